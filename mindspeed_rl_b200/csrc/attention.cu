@@ -594,10 +594,12 @@ MSRL_API int msrl_flash_attn_varlen_fwd(const void* q, const void* k, const void
                                         const long long* layouts12, void* o, long long o_stride_t,
                                         float* lse, const int* cu_q, const int* cu_k, int batch,
                                         int max_q, int nh, int nkv, long long Tq, int D,
-                                        int causal, cudaStream_t st) {
+                                        float scale, int causal, cudaStream_t st) {
   if (batch == 0 || Tq == 0) return 0;
   if (nh % nkv != 0) return (int)cudaErrorInvalidValue;
   AttnParams p = make_params(q, k, v, layouts12, o, o_stride_t, lse, cu_q, cu_k, nh, nkv, Tq, D, causal);
+  p.scale = scale;
+  p.scale_log2 = scale * kLog2e;
   if (D == 128) return launch_fwd<128>(p, batch, max_q, st);
   if (D == 64) return launch_fwd<64>(p, batch, max_q, st);
   return (int)cudaErrorInvalidValue;

@@ -872,7 +872,7 @@ MSRL_API int msrl_flash_attn_varlen_fwd_tcgen05(const void* q, const void* k, co
                                                 const long long* lay, void* o, long long o_stride_t,
                                                 float* lse, const int* cu_q, const int* cu_k, int batch,
                                                 int max_q, int nh, int nkv, long long Tq, long long Tk,
-                                                int D, int causal, int* error, cudaStream_t st) {
+                                                int D, float scale, int causal, int* error, cudaStream_t st) {
   if (batch == 0 || Tq == 0) return 0;
   if (D != fa5::D || nh % nkv != 0 || (o_stride_t % 8) != 0 || (reinterpret_cast<uintptr_t>(o) & 15) != 0)
     return (int)cudaErrorNotSupported;
@@ -899,7 +899,7 @@ MSRL_API int msrl_flash_attn_varlen_fwd_tcgen05(const void* q, const void* k, co
   p.nh = nh;
   p.nkv = nkv;
   p.Tq = Tq;
-  p.scale_log2 = 1.4426950408889634f / sqrtf((float)D);
+  p.scale_log2 = scale * 1.4426950408889634f;
   p.causal = causal;
   p.q_col0 = 0; p.q_group_stride = (int)lay[1]; p.q_hpg = (int)lay[2]; p.q_head_stride = (int)lay[3];
   p.k_col0 = 0; p.k_group_stride = (int)lay[5]; p.k_hpg = (int)lay[6]; p.k_head_stride = (int)lay[7];

@@ -29,6 +29,9 @@ NVCC_FLAGS = [
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
     "--expt-relaxed-constexpr", "-Xptxas", "-v",
 ]
+# kernels whose results are specified in 32-bit (an fp32 residual, recurrent state, fp32 attention): compiled
+# without the approximate divisions, square roots, exponentials and flush-to-zero of --use_fast_math
+PRECISE = {"residual_stream", "delta_rule", "latent_attention", "grouped_gemm_simt"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 
@@ -50,7 +53,8 @@ def _compile_one(src: Path, force: bool, log_dir: Path) -> Path:
     if not force and obj.exists() and obj.stat().st_mtime >= stamp:
         return obj
     if src.suffix == ".cu":
-        cmd = [_nvcc(), *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
+        flags = [f for f in NVCC_FLAGS if f != "--use_fast_math" or src.stem not in PRECISE]
+        cmd = [_nvcc(), *flags, "-I", str(CSRC), "-c", str(src), "-o", str(obj)]
     else:
         cmd = ["g++", *CXX_FLAGS, "-I", str(CSRC), "-I", "/usr/local/cuda/include", "-c", str(src),
                "-o", str(obj)]

@@ -1,0 +1,529 @@
+// Gated delta rule with a decay per key channel, for prompts (prefill portions) and single-token decode steps.
+//
+// Per value head h, with key head hk = h / (H / KVH), state S [dim, vdim] in fp32:
+//
+//   q, k, v = silu(causal conv over time of the projections)          (last tap = current token)
+//   q = q / |q| * dim^-1/2,  k = k / |k|                              (|x| = sqrt(sum x^2 + unit_eps))
+//   g = exp(-exp(A_log[h]) * softplus(a + dt_bias))   [dim],   beta = sigmoid(b)
+//   S <- g * S;  u = beta * (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   y = o / rms(o) * norm * sigmoid(gate)
+//
+// What a sequence carries from step to step lives in a state slot: S, and a ring of the last `taps` inputs of
+// the short convolutions (entry p % taps holds the projections of position p).  With `taps` entries, one more
+// than the next token needs, the entry a step writes is never one that the same step reads.  Positions
+// before the sequence's start count as zero, so a slot needs no clearing when it is used again.
+//
+//   prefill: `prep` (conv, silu, unit norms, decays, step sizes of every token), `scan` (the recurrence: one
+//            block per sequence, head and column group; S in registers, LPC lanes share a column) and
+//            `out` (norm and gate);
+//   decode:  one fused kernel per (sequence, head): all of the above with S read and written once, coalesced.
+//
+// Both sum (S^T k, S^T q) over the decayed state in one pass: o = (gS)^T q + (k.q) u.
+#include "dtype_utils.cuh"
+
+namespace msrl {
+
+template <typename T>
+struct DeltaIn {
+  const T* proj;             // [tokens, ld]: q | k | v | b ... sections at the given columns
+  long long ld;
+  int q_col, k_col, v_col, b_col;
+  const T* a;                // [tokens, H * dim] decay projection
+  long long a_ld;
+  const float* conv;         // [2 * KVH * dim + H * vdim, taps]
+  int taps;
+  const float* a_log;        // [H]
+  const float* dt_bias;      // [H * dim]
+  T* ring;                   // [slots, taps, channels]
+  float* state;              // [slots, H, dim, vdim]
+  int H, KVH, dim, vdim;
+  float unit_eps;
+};
+
+// silu of the short convolution for one channel: `col` is its column in proj, `ch` its ring / weight row,
+// `i` the token's index inside this portion (row t of proj), `pos` its position in the sequence
+template <typename T>
+__device__ __forceinline__ float conv_silu(const DeltaIn<T>& p, long long t, int i, int pos, long long slot, int col,
+                                           int ch) {
+  const int channels = 2 * p.KVH * p.dim + p.H * p.vdim;
+  float s = 0.f;
+  for (int j = 0; j < p.taps; ++j) {
+    const int back = p.taps - 1 - j;
+    if (pos - back < 0) continue;
+    const float x = i - back >= 0 ? ldf(p.proj + (t - back) * p.ld + col)
+                                  : ldf(p.ring + (slot * p.taps + (pos - back) % p.taps) * channels + ch);
+    s += x * p.conv[(long long)ch * p.taps + j];
+  }
+  return s * sigmoid_f(s);
+}
+
+constexpr int DELTA_MAX_DIM = 256;
+
+// ---- prefill: everything that does not depend on the state -------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_prep_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const int* start_pos, const long long* slots,
+                  float* qn, float* kn, float* kq, float* vv, float* g, float* beta) {
+  const long long t = blockIdx.x;
+  const int b = tok_seq[t];
+  const int i = (int)(t - cu[b]);
+  const int pos = start_pos[b] + i;
+  const long long slot = slots[b];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int kd = p.KVH * p.dim;
+  const float qscale = 1.f / sqrtf((float)p.dim);
+  for (int hk = warp; hk < p.KVH; hk += 8) {
+    float q[DELTA_MAX_DIM / 32], k[DELTA_MAX_DIM / 32];
+    float qq = 0.f, kk = 0.f, qk = 0.f;
+#pragma unroll
+    for (int n = 0; n < DELTA_MAX_DIM / 32; ++n) {
+      const int d = n * 32 + lane;
+      if (d < p.dim) {
+        const int ch = hk * p.dim + d;
+        q[n] = conv_silu(p, t, i, pos, slot, p.q_col + ch, ch);
+        k[n] = conv_silu(p, t, i, pos, slot, p.k_col + ch, kd + ch);
+        qq += q[n] * q[n];
+        kk += k[n] * k[n];
+        qk += q[n] * k[n];
+      }
+    }
+    const float qs = qscale / sqrtf(warp_sum(qq) + p.unit_eps), ks = 1.f / sqrtf(warp_sum(kk) + p.unit_eps);
+    qk = warp_sum(qk) * qs * ks;
+#pragma unroll
+    for (int n = 0; n < DELTA_MAX_DIM / 32; ++n) {
+      const int d = n * 32 + lane;
+      if (d < p.dim) {
+        qn[t * kd + hk * p.dim + d] = q[n] * qs;
+        kn[t * kd + hk * p.dim + d] = k[n] * ks;
+      }
+    }
+    if (lane == 0) kq[t * p.KVH + hk] = qk;
+  }
+  const int nv = p.H * p.vdim;
+  for (int c = threadIdx.x; c < nv; c += 256) vv[t * nv + c] = conv_silu(p, t, i, pos, slot, p.v_col + c, 2 * kd + c);
+  const int ng = p.H * p.dim;
+  for (int c = threadIdx.x; c < ng; c += 256)
+    g[t * ng + c] = expf(-expf(p.a_log[c / p.dim]) * softplus_f(ldf(p.a + t * p.a_ld + c) + p.dt_bias[c]));
+  for (int h = threadIdx.x; h < p.H; h += 256) beta[t * p.H + h] = sigmoid_f(ldf(p.proj + t * p.ld + p.b_col + h));
+}
+
+// ---- prefill: the recurrence --------------------------------------------------------------------------
+__device__ __forceinline__ void cp_async4(void* smem, const void* gmem) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(smem_u32(smem)), "l"(gmem));
+}
+__device__ __forceinline__ void cp_async16b(void* smem, const void* gmem) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_u32(smem)), "l"(gmem));
+}
+
+constexpr int SCAN_TB = 16;      // tokens staged at a time
+
+// LPC lanes share a column, each with DPL rows (row = 4 * (LPC * n + lane) + j); COLS columns per block
+template <int DPL, int LPC, int COLS, bool VEC>
+__global__ void __launch_bounds__(COLS * LPC)
+delta_scan_kernel(const float* qn, const float* kn, const float* kq, const float* vv, const float* g,
+                  const float* beta, float* state, const int* cu, const int* start_pos, const long long* slots, int H,
+                  int KVH, int dim, int vdim, float* o) {
+  constexpr int DP = DPL * LPC, THREADS = COLS * LPC;
+  extern __shared__ __align__(16) float sm[];
+  // two buffers of [q TB*DP | k TB*DP | g TB*DP | v TB*COLS | beta TB | kq TB]
+  constexpr int BUF = SCAN_TB * (3 * DP + COLS + 2);
+  const int h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * COLS;
+  const int hk = h / (H / KVH);
+  const long long t0 = cu[b];
+  const int len = cu[b + 1] - cu[b];
+  if (len <= 0) return;
+  const int col_l = threadIdx.x / LPC, lr = threadIdx.x % LPC;
+  const int col = c0 + col_l;
+  const bool on = col < vdim;
+  const long long slot = slots[b];
+  float* Sg = state + ((slot * H + h) * dim) * (long long)vdim + col;
+
+  for (int i = threadIdx.x; i < 2 * BUF; i += THREADS) sm[i] = 0.f;      // pad rows stay zero
+  float s[DPL];
+  const bool fresh = start_pos[b] == 0;
+#pragma unroll
+  for (int n = 0; n < DPL; ++n) {
+    const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
+    s[n] = (!fresh && on && r < dim) ? Sg[(long long)r * vdim] : 0.f;
+  }
+  __syncthreads();
+
+  auto stage = [&](int blk) {
+    float* buf = sm + (blk & 1) * BUF;
+    const int first = blk * SCAN_TB, n = min(SCAN_TB, len - first);
+    if constexpr (VEC) {
+      const int per = dim / 4;
+      for (int i = threadIdx.x; i < n * per; i += THREADS) {
+        const int tt = i / per, d = (i % per) * 4;
+        const long long t = t0 + first + tt;
+        cp_async16b(buf + tt * DP + d, qn + (t * KVH + hk) * dim + d);
+        cp_async16b(buf + SCAN_TB * DP + tt * DP + d, kn + (t * KVH + hk) * dim + d);
+        cp_async16b(buf + 2 * SCAN_TB * DP + tt * DP + d, g + (t * H + h) * dim + d);
+      }
+    } else {
+      for (int i = threadIdx.x; i < n * dim; i += THREADS) {
+        const int tt = i / dim, d = i % dim;
+        const long long t = t0 + first + tt;
+        cp_async4(buf + tt * DP + d, qn + (t * KVH + hk) * dim + d);
+        cp_async4(buf + SCAN_TB * DP + tt * DP + d, kn + (t * KVH + hk) * dim + d);
+        cp_async4(buf + 2 * SCAN_TB * DP + tt * DP + d, g + (t * H + h) * dim + d);
+      }
+    }
+    float* bv = buf + 3 * SCAN_TB * DP;
+    for (int i = threadIdx.x; i < n * COLS; i += THREADS) {
+      const int tt = i / COLS, c = i % COLS;
+      if (c0 + c < vdim) cp_async4(bv + i, vv + ((t0 + first + tt) * H + h) * vdim + c0 + c);
+    }
+    float* bb = bv + SCAN_TB * COLS;
+    for (int i = threadIdx.x; i < 2 * n; i += THREADS) {
+      const int tt = i % n;
+      if (i < n) cp_async4(bb + tt, beta + (t0 + first + tt) * H + h);
+      else cp_async4(bb + SCAN_TB + tt, kq + (t0 + first + tt) * KVH + hk);
+    }
+    asm volatile("cp.async.commit_group;\n" ::);
+  };
+
+  const int blocks = (len + SCAN_TB - 1) / SCAN_TB;
+  stage(0);
+  for (int blk = 0; blk < blocks; ++blk) {
+    if (blk + 1 < blocks) {
+      stage(blk + 1);
+      asm volatile("cp.async.wait_group 1;\n" ::);
+    } else {
+      asm volatile("cp.async.wait_group 0;\n" ::);
+    }
+    __syncthreads();
+    const float* buf = sm + (blk & 1) * BUF;
+    const int first = blk * SCAN_TB, n = min(SCAN_TB, len - first);
+    const float* bv = buf + 3 * SCAN_TB * DP;
+    const float* bb = bv + SCAN_TB * COLS;
+#pragma unroll 2
+    for (int tt = 0; tt < n; ++tt) {
+      const float4* q4 = reinterpret_cast<const float4*>(buf + tt * DP) + lr;
+      const float4* k4 = reinterpret_cast<const float4*>(buf + SCAN_TB * DP + tt * DP) + lr;
+      const float4* g4 = reinterpret_cast<const float4*>(buf + 2 * SCAN_TB * DP + tt * DP) + lr;
+      float pk[4] = {0.f, 0.f, 0.f, 0.f}, pq[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int m = 0; m < DPL / 4; ++m) {
+        const float4 gg = g4[m * LPC], kk = k4[m * LPC], qq = q4[m * LPC];
+        s[4 * m + 0] *= gg.x; s[4 * m + 1] *= gg.y; s[4 * m + 2] *= gg.z; s[4 * m + 3] *= gg.w;
+        pk[0] += s[4 * m + 0] * kk.x; pk[1] += s[4 * m + 1] * kk.y;
+        pk[2] += s[4 * m + 2] * kk.z; pk[3] += s[4 * m + 3] * kk.w;
+        pq[0] += s[4 * m + 0] * qq.x; pq[1] += s[4 * m + 1] * qq.y;
+        pq[2] += s[4 * m + 2] * qq.z; pq[3] += s[4 * m + 3] * qq.w;
+      }
+      float dk = (pk[0] + pk[1]) + (pk[2] + pk[3]), dq = (pq[0] + pq[1]) + (pq[2] + pq[3]);
+#pragma unroll
+      for (int x = LPC / 2; x > 0; x >>= 1) {
+        dk += __shfl_xor_sync(0xffffffffu, dk, x);
+        dq += __shfl_xor_sync(0xffffffffu, dq, x);
+      }
+      const float u = bb[tt] * (bv[tt * COLS + col_l] - dk);
+#pragma unroll
+      for (int m = 0; m < DPL / 4; ++m) {
+        const float4 kk = k4[m * LPC];
+        s[4 * m + 0] += kk.x * u; s[4 * m + 1] += kk.y * u;
+        s[4 * m + 2] += kk.z * u; s[4 * m + 3] += kk.w * u;
+      }
+      if (lr == 0 && on) o[((t0 + first + tt) * H + h) * vdim + col] = dq + bb[SCAN_TB + tt] * u;
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int n = 0; n < DPL; ++n) {
+    const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
+    if (on && r < dim) Sg[(long long)r * vdim] = s[n];
+  }
+}
+
+// ---- prefill: the last inputs of the convolutions ------------------------------------------------------
+template <typename T>
+__global__ void delta_ring_kernel(const DeltaIn<T> p, const int* cu, const int* start_pos, const long long* slots) {
+  const int b = blockIdx.y;
+  const int kd = p.KVH * p.dim, channels = 2 * kd + p.H * p.vdim;
+  const int len = cu[b + 1] - cu[b];
+  const int ch = blockIdx.x * blockDim.x + threadIdx.x;
+  if (ch >= channels) return;
+  const int col = ch < kd ? p.q_col + ch : ch < 2 * kd ? p.k_col + ch - kd : p.v_col + ch - 2 * kd;
+  for (int i = max(0, len - p.taps); i < len; ++i) {
+    const int pos = start_pos[b] + i;
+    p.ring[(slots[b] * p.taps + pos % p.taps) * channels + ch] = p.proj[(cu[b] + i) * p.ld + col];
+  }
+}
+
+// ---- prefill: norm and gate ------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_out_kernel(const float* o, const T* gate, long long gate_ld, const float* norm, float eps, T* y, long long rows,
+                 int H, int vdim) {
+  const long long r = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);     // (token, head)
+  const int lane = threadIdx.x & 31;
+  if (r >= rows) return;
+  const long long t = r / H;
+  const int h = (int)(r % H);
+  const float* x = o + r * vdim;
+  float ss = 0.f;
+  for (int c = lane; c < vdim; c += 32) ss += x[c] * x[c];
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)vdim + eps);
+  for (int c = lane; c < vdim; c += 32)
+    stf(y + r * vdim + c, x[c] * inv * norm[c] * sigmoid_f(ldf(gate + t * gate_ld + h * vdim + c)));
+}
+
+// ---- decode: one token per sequence, everything in one kernel -----------------------------------------------
+// block = (head, sequence).  Threads tile the state as [row groups RG][column groups of V]; a thread keeps its
+// NI row slices in registers between the decayed dot products and the rank-one update.
+template <typename T, int V, int NI, int THREADS>
+__global__ void __launch_bounds__(THREADS)
+delta_decode_kernel(const DeltaIn<T> p, const T* gate, long long gate_ld, const float* norm, float eps,
+                    const int* positions, const long long* slots, T* y) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float red[32];
+  __shared__ float scal[3];
+  const int h = blockIdx.x, b = blockIdx.y;
+  const long long slot = slots[b];
+  if (slot < 0) return;
+  const int dim = p.dim, vdim = p.vdim, kd = p.KVH * dim, channels = 2 * kd + p.H * vdim;
+  const int rep = p.H / p.KVH, hk = h / rep;
+  const int pos = positions[b];
+  const int CW = vdim / V, RG = THREADS / CW;
+  float* sq = sm;
+  float* sk = sq + dim;
+  float* sg = sk + dim;
+  float* sv = sg + dim;
+  float* su = sv + vdim;
+  float* so = su + vdim;
+  float* part = so + vdim;                       // [RG][2][vdim]
+  const int rg = threadIdx.x / CW, cg = threadIdx.x % CW;
+  const bool on = rg < RG;
+  float* S = p.state + ((slot * p.H + h) * dim) * (long long)vdim + cg * V;
+  float s[NI][4];
+#pragma unroll
+  for (int n = 0; n < NI; ++n) {
+    const int r = rg + n * RG;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) s[n][j] = 0.f;
+    if (on && r < dim && pos > 0) ldv<V>(S + (long long)r * vdim, s[n]);
+  }
+  const bool lead = h % rep == 0;                // writes the key head's ring entries
+  T* ring = p.ring + (slot * p.taps + pos % p.taps) * channels;
+  const T* row = p.proj + (long long)b * p.ld;
+  for (int d = threadIdx.x; d < dim; d += THREADS) {
+    const int ch = hk * dim + d;
+    sq[d] = conv_silu(p, b, 0, pos, slot, p.q_col + ch, ch);
+    sk[d] = conv_silu(p, b, 0, pos, slot, p.k_col + ch, kd + ch);
+    sg[d] = expf(-expf(p.a_log[h]) * softplus_f(ldf(p.a + b * p.a_ld + h * dim + d) + p.dt_bias[h * dim + d]));
+    if (lead) {
+      ring[ch] = row[p.q_col + ch];
+      ring[kd + ch] = row[p.k_col + ch];
+    }
+  }
+  for (int c = threadIdx.x; c < vdim; c += THREADS) {
+    const int ch = h * vdim + c;
+    sv[c] = conv_silu(p, b, 0, pos, slot, p.v_col + ch, 2 * kd + ch);
+    ring[2 * kd + ch] = row[p.v_col + ch];
+  }
+  __syncthreads();
+  {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (warp < 3) {
+      const float* x = warp == 1 ? sk : sq;
+      const float* z = warp == 0 ? sq : sk;
+      float a = 0.f;
+      for (int d = lane; d < dim; d += 32) a += x[d] * z[d];
+      a = warp_sum(a);
+      if (lane == 0) scal[warp] = a;
+    }
+  }
+  float pk[4] = {0.f, 0.f, 0.f, 0.f}, pq[4] = {0.f, 0.f, 0.f, 0.f};
+  if (on) {
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int r = rg + n * RG;
+      if (r < dim) {
+        const float gr = sg[r], kr = sk[r], qr = sq[r];
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          s[n][j] *= gr;
+          pk[j] += s[n][j] * kr;
+          pq[j] += s[n][j] * qr;
+        }
+      }
+    }
+    stv<V>(part + (rg * 2 + 0) * vdim + cg * V, pk);
+    stv<V>(part + (rg * 2 + 1) * vdim + cg * V, pq);
+  }
+  __syncthreads();
+  const float qs = 1.f / (sqrtf(scal[0] + p.unit_eps) * sqrtf((float)dim)), ks = 1.f / sqrtf(scal[1] + p.unit_eps);
+  const float kq = scal[2] * qs * ks;
+  const float beta = sigmoid_f(ldf(row + p.b_col + h));
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < vdim; c += THREADS) {
+    float dk = 0.f, dq = 0.f;
+    for (int r = 0; r < RG; ++r) {
+      dk += part[(r * 2 + 0) * vdim + c];
+      dq += part[(r * 2 + 1) * vdim + c];
+    }
+    const float u = beta * (sv[c] - dk * ks);
+    const float oc = dq * qs + kq * u;
+    su[c] = u * ks;
+    so[c] = oc;
+    ss += oc * oc;
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)vdim + eps);     // also orders su before the reads below
+  if (on) {
+    float u[4];
+    ldv<V>(su + cg * V, u);
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int r = rg + n * RG;
+      if (r < dim) {
+        const float kr = sk[r];
+#pragma unroll
+        for (int j = 0; j < V; ++j) s[n][j] += kr * u[j];
+        stv<V>(S + (long long)r * vdim, s[n]);
+      }
+    }
+  }
+  for (int c = threadIdx.x; c < vdim; c += THREADS)
+    stf(y + ((long long)b * p.H + h) * vdim + c,
+        so[c] * inv * norm[c] * sigmoid_f(ldf(gate + b * gate_ld + h * vdim + c)));
+}
+
+}  // namespace msrl
+
+using namespace msrl;
+
+// ints: taps, H, KVH, dim, vdim, q_col, k_col, v_col, b_col
+template <typename T>
+static DeltaIn<T> delta_in(const void* proj, long long ld, const void* a, long long a_ld, const float* conv,
+                           const float* a_log, const float* dt_bias, void* ring, float* state, const int* ints,
+                           float unit_eps) {
+  DeltaIn<T> p{};
+  p.proj = (const T*)proj;
+  p.ld = ld;
+  p.a = (const T*)a;
+  p.a_ld = a_ld;
+  p.conv = conv;
+  p.a_log = a_log;
+  p.dt_bias = dt_bias;
+  p.ring = (T*)ring;
+  p.state = state;
+  p.taps = ints[0];
+  p.H = ints[1];
+  p.KVH = ints[2];
+  p.dim = ints[3];
+  p.vdim = ints[4];
+  p.q_col = ints[5];
+  p.k_col = ints[6];
+  p.v_col = ints[7];
+  p.b_col = ints[8];
+  p.unit_eps = unit_eps;
+  return p;
+}
+
+template <typename F>
+static int allow_smem(F* kernel, size_t bytes) {
+  if (bytes <= 48 * 1024) return 0;
+  return (int)cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+}
+
+template <int DPL, int LPC, int COLS>
+static int launch_scan(const float* qn, const float* kn, const float* kq, const float* vv, const float* g,
+                       const float* beta, float* state, const int* cu, const int* start_pos, const long long* slots,
+                       int batch, int H, int KVH, int dim, int vdim, float* o, cudaStream_t st) {
+  const size_t smem = 2 * sizeof(float) * SCAN_TB * (3 * DPL * LPC + COLS + 2);
+  const dim3 grid((unsigned)((vdim + COLS - 1) / COLS), (unsigned)H, (unsigned)batch);
+  if (dim % 4 == 0) {
+    const int e = allow_smem(delta_scan_kernel<DPL, LPC, COLS, true>, smem);
+    if (e) return e;
+    delta_scan_kernel<DPL, LPC, COLS, true><<<grid, COLS * LPC, smem, st>>>(qn, kn, kq, vv, g, beta, state, cu,
+                                                                            start_pos, slots, H, KVH, dim, vdim, o);
+  } else {
+    const int e = allow_smem(delta_scan_kernel<DPL, LPC, COLS, false>, smem);
+    if (e) return e;
+    delta_scan_kernel<DPL, LPC, COLS, false><<<grid, COLS * LPC, smem, st>>>(qn, kn, kq, vv, g, beta, state, cu,
+                                                                             start_pos, slots, H, KVH, dim, vdim, o);
+  }
+  return (int)cudaGetLastError();
+}
+
+// scratch (fp32): qn, kn [tokens, KVH, dim], kq [tokens, KVH], vv, o [tokens, H, vdim], g [tokens, H, dim],
+// beta [tokens, H]
+MSRL_API int msrl_delta_prefill(const void* proj, long long ld, const void* a, long long a_ld, const float* conv,
+                                const float* a_log, const float* dt_bias, void* ring, float* state, const int* ints,
+                                float unit_eps, const void* gate, long long gate_ld, const float* norm, float eps,
+                                const int* tok_seq, const int* cu, const int* start_pos, const long long* slots,
+                                int tokens, int batch, float* qn, float* kn, float* kq, float* vv, float* g,
+                                float* beta, float* o, void* y, int is_f32, cudaStream_t st) {
+  if (tokens == 0 || batch == 0) return 0;
+  const int H = ints[1], KVH = ints[2], dim = ints[3], vdim = ints[4];
+  if (dim > DELTA_MAX_DIM || H % KVH != 0 || batch > 65535 || H > 65535) return (int)cudaErrorInvalidValue;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const DeltaIn<T> p = delta_in<T>(proj, ld, a, a_ld, conv, a_log, dt_bias, ring, state, ints, unit_eps);
+    delta_prep_kernel<T><<<tokens, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, qn, kn, kq, vv, g, beta);
+    int e;
+    if (dim <= 32) e = launch_scan<8, 4, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st);
+    else if (dim <= 64) e = launch_scan<16, 4, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st);
+    else if (dim <= 128) e = launch_scan<16, 8, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st);
+    else e = launch_scan<32, 8, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st);
+    if (e) return e;
+    const int channels = 2 * KVH * dim + H * vdim;
+    delta_ring_kernel<T><<<dim3((unsigned)((channels + 255) / 256), (unsigned)batch), 256, 0, st>>>(p, cu, start_pos, slots);
+    const long long rows = (long long)tokens * H;
+    delta_out_kernel<T><<<(unsigned)((rows + 7) / 8), 256, 0, st>>>(o, (const T*)gate, gate_ld, norm, eps, (T*)y, rows, H, vdim);
+    return (int)cudaGetLastError();
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+template <typename T, int V, int NI, int THREADS>
+static int launch_delta_decode(const DeltaIn<T>& p, const T* gate, long long gate_ld, const float* norm, float eps,
+                               const int* positions, const long long* slots, T* y, int batch, cudaStream_t st) {
+  const int rg = THREADS / (p.vdim / V);
+  const size_t smem = sizeof(float) * (3 * (size_t)p.dim + 3 * (size_t)p.vdim + 2 * (size_t)rg * p.vdim);
+  const int e = allow_smem(delta_decode_kernel<T, V, NI, THREADS>, smem);
+  if (e) return e;
+  delta_decode_kernel<T, V, NI, THREADS><<<dim3((unsigned)p.H, (unsigned)batch), THREADS, smem, st>>>(
+      p, gate, gate_ld, norm, eps, positions, slots, y);
+  return (int)cudaGetLastError();
+}
+
+template <typename T, int V>
+static int pick_delta_decode(const DeltaIn<T>& p, const T* gate, long long gate_ld, const float* norm, float eps,
+                             const int* positions, const long long* slots, T* y, int batch, cudaStream_t st) {
+  // rows per thread for a block size: the smallest block that keeps at most 16 row slices per thread
+  auto slices = [&](int threads) {
+    const int rg = threads / (p.vdim / V);
+    return rg == 0 ? 1 << 20 : (p.dim + rg - 1) / rg;
+  };
+#define MSRL_TRY(NI, THREADS) \
+  if (slices(THREADS) <= NI)  \
+    return launch_delta_decode<T, V, NI, THREADS>(p, gate, gate_ld, norm, eps, positions, slots, y, batch, st);
+  MSRL_TRY(4, 128)
+  MSRL_TRY(4, 256)
+  MSRL_TRY(16, 128)
+  MSRL_TRY(16, 256)
+  MSRL_TRY(16, 512)
+  MSRL_TRY(16, 1024)
+  MSRL_TRY(64, 512)
+#undef MSRL_TRY
+  return (int)cudaErrorInvalidValue;
+}
+
+MSRL_API int msrl_delta_decode(const void* proj, long long ld, const void* a, long long a_ld, const float* conv,
+                               const float* a_log, const float* dt_bias, void* ring, float* state, const int* ints,
+                               float unit_eps, const void* gate, long long gate_ld, const float* norm, float eps,
+                               const int* positions, const long long* slots, int batch, void* y, int is_f32,
+                               cudaStream_t st) {
+  if (batch == 0) return 0;
+  if (ints[3] > DELTA_MAX_DIM || ints[1] % ints[2] != 0 || batch > 65535) return (int)cudaErrorInvalidValue;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const DeltaIn<T> p = delta_in<T>(proj, ld, a, a_ld, conv, a_log, dt_bias, ring, state, ints, unit_eps);
+    return p.vdim % 4 == 0
+               ? pick_delta_decode<T, 4>(p, (const T*)gate, gate_ld, norm, eps, positions, slots, (T*)y, batch, st)
+               : pick_delta_decode<T, 1>(p, (const T*)gate, gate_ld, norm, eps, positions, slots, (T*)y, batch, st);
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}

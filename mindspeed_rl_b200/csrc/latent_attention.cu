@@ -1,0 +1,654 @@
+// Latent attention over a paged cache of one latent row per token.
+//
+// A cache row is [latent (RP, zero padded) | rotated key part (CP - RP, zero padded)]: all heads share it.
+// Scores are (q_unrotated . W_uk c + q_rotated . k_rotated) * scale and values W_uv c; the up-projections are
+// linear, so prompts expand them per head and decode steps fold them into the query (q W_uk) and the output
+// (W_uv sum p c) and attend to the rows themselves.
+//
+//   prep        RMS norm of the latent, interleaved rotation of the shared key part and of every head's query
+//               part (fp32), cache write; the row also goes to `lat` (prompts), the rotated query part to the
+//               decode query
+//   gather      cache rows of given (sequence, position) pairs, for prompt portions after the first
+//   spread      the rotated key part into every head's expanded key
+//   attn_simt   soft-max attention of packed sequences for any head sizes, fp32 arithmetic
+//   decode_simt one query per sequence over the paged rows, any sizes, fp32 arithmetic
+//   decode_mma  the same on the tensor cores for bf16: a block takes 16 / 32 / 64 heads of one sequence and a
+//               range of its keys, so that a row is read once for all of them; `combine` merges the ranges
+#include "dtype_utils.cuh"
+#include "mma_utils.cuh"
+
+namespace msrl {
+namespace mla {
+
+template <typename T>
+struct PrepArgs {
+  T* qkv;                      // [tokens, ld]
+  long long ld;
+  int H, q_stride, dn, dr;     // head h's query: columns h * q_stride + [0, dn) unrotated, then dr rotated
+  int dkv_col, rank;
+  const float* norm_w;
+  float eps;
+  const float* table;          // [positions, rot_dims]: cos | sin
+  int rot_dims, table_rows;
+  const int* positions;
+  const long long* slots;      // cache row per token, < 0: not cached
+  T* cache;
+  int RP, CP;
+  T* lat;                      // [tokens, CP] or null
+  T* qdec;                     // [tokens, H, CP] or null: receives the rotated query part at column RP
+};
+
+template <typename T>
+__device__ __forceinline__ float rotated(const T* x, int d, const float* cs, int rot_dims) {
+  if (d >= rot_dims) return ldf(x + d);
+  const int half = rot_dims / 2, i = d >> 1;
+  const float c = cs[i], s = cs[half + i];
+  const float u = ldf(x + (d & ~1)), v = ldf(x + (d | 1));
+  return (d & 1) ? v * c + u * s : u * c - v * s;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) prep_kernel(const PrepArgs<T> p) {
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  T* row = p.qkv + t * p.ld;
+  const T* lat_in = row + p.dkv_col;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < p.rank; c += 256) {
+    const float x = ldf(lat_in + c);
+    ss += x * x;
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)p.rank + p.eps);
+  const int pos = min(max(p.positions[t], 0), p.table_rows - 1);
+  const float* cs = p.table + (long long)pos * p.rot_dims;
+  const long long slot = p.slots[t];
+  T* crow = slot >= 0 ? p.cache + slot * p.CP : nullptr;
+  T* lrow = p.lat != nullptr ? p.lat + t * p.CP : nullptr;
+  for (int c = threadIdx.x; c < p.CP; c += 256) {
+    float v = 0.f;
+    if (c < p.rank) v = ldf(lat_in + c) * inv * p.norm_w[c];
+    else if (c >= p.RP && c < p.RP + p.dr) v = rotated(lat_in + p.rank, c - p.RP, cs, p.rot_dims);
+    if (crow != nullptr) stf(crow + c, v);
+    if (lrow != nullptr) stf(lrow + c, v);
+  }
+  if (p.qdec != nullptr) {
+    const int w = p.CP - p.RP;
+    for (int i = threadIdx.x; i < p.H * w; i += 256) {
+      const int h = i / w, d = i % w;
+      stf(p.qdec + (t * p.H + h) * p.CP + p.RP + d,
+          d < p.dr ? rotated(row + h * p.q_stride + p.dn, d, cs, p.rot_dims) : 0.f);
+    }
+  } else {
+    // in place: one thread owns both entries of a pair
+    const int half = p.rot_dims / 2;
+    for (int i = threadIdx.x; i < p.H * half; i += 256) {
+      const int h = i / half, d = 2 * (i % half);
+      T* x = row + h * p.q_stride + p.dn;
+      const float a = rotated(x, d, cs, p.rot_dims), b = rotated(x, d + 1, cs, p.rot_dims);
+      stf(x + d, a);
+      stf(x + d + 1, b);
+    }
+  }
+}
+
+// rows of 16-byte vectors
+__global__ void gather_kernel(const uint4* cache, const int* block_tables, int max_blocks, int block_size,
+                              const int* token_seq, const int* token_pos, uint4* out, long long rows, int vecs) {
+  const long long r = (long long)blockIdx.x * (blockDim.x / 32) + (threadIdx.x >> 5);
+  if (r >= rows) return;
+  const int pos = token_pos[r];
+  const long long slot = (long long)block_tables[(long long)token_seq[r] * max_blocks + pos / block_size] * block_size +
+                         pos % block_size;
+  for (int c = threadIdx.x & 31; c < vecs; c += 32) out[r * vecs + c] = cache[slot * vecs + c];
+}
+
+// kv[t, h * stride + dn + d] = lat[t, RP + d]
+template <typename T>
+__global__ void spread_kernel(const T* lat, int CP, int RP, T* kv, long long ld, int H, int stride, int dn, int dr,
+                              long long tokens) {
+  const long long t = blockIdx.x;
+  for (int i = threadIdx.x; i < H * dr; i += blockDim.x)
+    kv[t * ld + (i / dr) * stride + dn + i % dr] = lat[t * CP + RP + i % dr];
+}
+
+// ---- soft-max attention of packed sequences on the CUDA cores ------------------------------------------
+template <typename T>
+struct SimtArgs {
+  const T *q, *k, *v;
+  long long q_ld, k_ld, v_ld;
+  int q_stride, k_stride, v_stride;      // head strides
+  int dq, dv;
+  const int *cu_q, *cu_k;
+  float scale;
+  T* out;                                // [tokens, H * o_stride]
+  long long o_ld;
+  int o_stride;
+};
+
+constexpr int SB = 32;                   // query rows and keys per tile
+
+template <typename T, int ACC>
+__global__ void __launch_bounds__(256) attn_simt_kernel(const SimtArgs<T> p) {
+  extern __shared__ float smf[];
+  const int ldq = p.dq + 1;
+  float* sQ = smf;
+  float* sK = sQ + SB * ldq;
+  float* sV = sK + SB * ldq;
+  float* sP = sV + SB * p.dv;            // [SB][SB + 1]
+  const int h = blockIdx.y, b = blockIdx.z;
+  const int q0 = p.cu_q[b], qlen = p.cu_q[b + 1] - q0, k0 = p.cu_k[b], klen = p.cu_k[b + 1] - k0;
+  const int m0 = blockIdx.x * SB;
+  if (m0 >= qlen) return;
+  const int off = klen - qlen;           // bottom-right aligned causal mask
+  const int row = threadIdx.x >> 3, part = threadIdx.x & 7;
+  for (int i = threadIdx.x; i < SB * p.dq; i += 256) {
+    const int r = i / p.dq, d = i % p.dq;
+    sQ[r * ldq + d] = m0 + r < qlen ? ldf(p.q + (long long)(q0 + m0 + r) * p.q_ld + h * p.q_stride + d) : 0.f;
+  }
+  float acc[ACC];
+#pragma unroll
+  for (int i = 0; i < ACC; ++i) acc[i] = 0.f;
+  float m_run = -INFINITY, l_run = 0.f;
+  const int kmax = min(klen, m0 + SB + off);
+  for (int kb = 0; kb < kmax; kb += SB) {
+    __syncthreads();
+    for (int i = threadIdx.x; i < SB * p.dq; i += 256) {
+      const int r = i / p.dq, d = i % p.dq;
+      sK[r * ldq + d] = kb + r < klen ? ldf(p.k + (long long)(k0 + kb + r) * p.k_ld + h * p.k_stride + d) : 0.f;
+    }
+    for (int i = threadIdx.x; i < SB * p.dv; i += 256) {
+      const int r = i / p.dv, d = i % p.dv;
+      sV[r * p.dv + d] = kb + r < klen ? ldf(p.v + (long long)(k0 + kb + r) * p.v_ld + h * p.v_stride + d) : 0.f;
+    }
+    __syncthreads();
+    float s[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int d = 0; d < p.dq; ++d) {
+      const float x = sQ[row * ldq + d];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[j] += x * sK[(part + 8 * j) * ldq + d];
+    }
+    float mx = -INFINITY;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int key = kb + part + 8 * j;
+      s[j] = key < klen && key <= m0 + row + off ? s[j] * p.scale : -INFINITY;
+      mx = fmaxf(mx, s[j]);
+    }
+#pragma unroll
+    for (int x = 4; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+    const float m_new = fmaxf(m_run, mx);
+    const float m_use = m_new == -INFINITY ? 0.f : m_new;
+    const float corr = expf(m_run - m_use);
+    float sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      s[j] = expf(s[j] - m_use);
+      sum += s[j];
+      sP[row * (SB + 1) + part + 8 * j] = s[j];
+    }
+#pragma unroll
+    for (int x = 4; x > 0; x >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, x);
+    l_run = l_run * corr + sum;
+    m_run = m_new;
+    __syncwarp();                        // a row's eight threads share a warp
+#pragma unroll
+    for (int i = 0; i < ACC; ++i) {
+      const int c = part + 8 * i;
+      if (c < p.dv) {
+        float a = acc[i] * corr;
+        for (int j = 0; j < SB; ++j) a += sP[row * (SB + 1) + j] * sV[j * p.dv + c];
+        acc[i] = a;
+      }
+    }
+  }
+  if (m0 + row < qlen) {
+    const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+#pragma unroll
+    for (int i = 0; i < ACC; ++i) {
+      const int c = part + 8 * i;
+      if (c < p.dv) stf(p.out + (long long)(q0 + m0 + row) * p.o_ld + h * p.o_stride + c, acc[i] * inv);
+    }
+  }
+}
+
+// ---- decode on the CUDA cores -----------------------------------------------------------------------------
+constexpr int DS_ACC = 8;                // latent columns per thread: RP <= 2048
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+decode_simt_kernel(const T* q, const T* cache, const int* block_tables, int max_blocks, int block_size,
+                   const int* context_lens, float scale, int CP, int RP, T* out) {
+  extern __shared__ float smf[];
+  __shared__ float sS[32];
+  float* sQ = smf;
+  const int h = blockIdx.x, b = blockIdx.y, H = gridDim.x;
+  const int n = context_lens[b];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* qr = q + ((long long)b * H + h) * CP;
+  for (int c = threadIdx.x; c < CP; c += 256) sQ[c] = ldf(qr + c);
+  const int* bt = block_tables + (long long)b * max_blocks;
+  float acc[DS_ACC];
+#pragma unroll
+  for (int i = 0; i < DS_ACC; ++i) acc[i] = 0.f;
+  float m_run = -INFINITY, l_run = 0.f;
+  for (int kb = 0; kb < n; kb += 32) {
+    __syncthreads();
+    for (int j = warp; j < 32; j += 8) {
+      const int key = kb + j;
+      float s = -INFINITY;
+      if (key < n) {
+        const T* r = cache + ((long long)bt[key / block_size] * block_size + key % block_size) * CP;
+        s = 0.f;
+        for (int c = lane; c < CP; c += 32) s += sQ[c] * ldf(r + c);
+        s = warp_sum(s) * scale;
+      }
+      if (lane == 0) sS[j] = s;
+    }
+    __syncthreads();
+    float m_new = m_run;
+    for (int j = 0; j < 32; ++j) m_new = fmaxf(m_new, sS[j]);
+    const float corr = expf(m_run - m_new);
+    l_run *= corr;
+    m_run = m_new;
+#pragma unroll
+    for (int i = 0; i < DS_ACC; ++i) acc[i] *= corr;
+    const int keys = min(32, n - kb);
+    for (int j = 0; j < keys; ++j) {
+      const int key = kb + j;
+      const float pj = expf(sS[j] - m_new);
+      l_run += pj;
+      const T* r = cache + ((long long)bt[key / block_size] * block_size + key % block_size) * CP;
+#pragma unroll
+      for (int i = 0; i < DS_ACC; ++i) {
+        const int c = threadIdx.x + 256 * i;
+        if (c < RP) acc[i] += pj * ldf(r + c);
+      }
+    }
+  }
+  const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+#pragma unroll
+  for (int i = 0; i < DS_ACC; ++i) {
+    const int c = threadIdx.x + 256 * i;
+    if (c < RP) stf(out + ((long long)b * H + h) * RP + c, acc[i] * inv);
+  }
+}
+
+// ---- decode on the tensor cores (bf16) -------------------------------------------------------------------
+struct MmaArgs {
+  const __nv_bfloat16* q;      // [B, H, CP]
+  const __nv_bfloat16* cache;  // [rows, CP]
+  const int* block_tables;
+  int max_blocks, block_size;
+  const int* context_lens;
+  float scale_log2;
+  int H, CP, RP, nsplit;
+  float* part_o;               // [B, H, nsplit, RP]
+  float* part_ml;              // [B, H, nsplit, 2]
+  __nv_bfloat16* out;          // [B, H, RP], written directly when nsplit == 1
+};
+
+// MT 16-head tiles per block, NT 8-column output tiles per warp (RP <= 64 * NT), KT keys per tile
+template <int MT, int NT, int KT>
+__global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
+  constexpr int HM = 16 * MT, WK = 8 / MT, NK8 = KT / 8 / WK;      // warps: WK key groups x MT head tiles
+  constexpr int TPR = 256 / HM, KPT = KT / TPR;                    // soft-max: threads per head row, keys per thread
+  constexpr int LDS_S = KT + 4, LDS_P = KT + 8;
+  static_assert(NK8 >= 1 && KPT >= 1, "tile sizes");
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int ld = p.CP + 8;
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(raw);
+  __nv_bfloat16* sKV = sQ + HM * ld;                               // two buffers
+  float* sS = reinterpret_cast<float*>(sKV + 2 * KT * ld);
+  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(sS + HM * LDS_S);
+  float* sCorr = reinterpret_cast<float*>(sP + HM * LDS_P);        // [HM]
+  float* sL = sCorr + HM;                                          // [HM]
+  const int split = blockIdx.x, h0 = blockIdx.y * HM, b = blockIdx.z;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n = p.context_lens[b];
+  const int tiles = (n + KT - 1) / KT, per = (tiles + p.nsplit - 1) / p.nsplit;
+  const int first = split * per, last = min(tiles, first + per);
+  const int vecs = p.CP / 8;
+  const int* bt = p.block_tables + (long long)b * p.max_blocks;
+
+  auto load_tile = [&](int tile, int buf) {
+    __nv_bfloat16* dst = sKV + buf * KT * ld;
+    for (int r = warp; r < KT; r += 8) {
+      const int key = tile * KT + r;
+      const bool ok = key < n;
+      const long long slot = ok ? (long long)bt[key / p.block_size] * p.block_size + key % p.block_size : 0;
+      const __nv_bfloat16* src = p.cache + slot * p.CP;
+      for (int c = lane; c < vecs; c += 32) cp_async16(dst + r * ld + c * 8, src + c * 8, ok);
+    }
+    cp_async_commit();
+  };
+
+  float o[MT][NT][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) o[m][i][j] = 0.f;
+  const int srow = threadIdx.x / TPR, spart = threadIdx.x % TPR;
+  float m_run = -INFINITY, l_run = 0.f;
+  const int wm = warp / WK, wk = warp % WK;                        // scores: head tile and key group of this warp
+  const int col0 = warp * NT * 8;                                  // output columns of this warp
+
+  if (first < last) {
+    for (int r = warp; r < HM; r += 8) {
+      const bool ok = h0 + r < p.H;
+      const __nv_bfloat16* src = p.q + ((long long)b * p.H + (ok ? h0 + r : 0)) * p.CP;
+      for (int c = lane; c < vecs; c += 32) cp_async16(sQ + r * ld + c * 8, src + c * 8, ok);
+    }
+    load_tile(first, 0);
+  }
+  for (int tile = first; tile < last; ++tile) {
+    const int buf = (tile - first) & 1;
+    if (tile + 1 < last) {
+      load_tile(tile + 1, buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const __nv_bfloat16* kv = sKV + buf * KT * ld;
+    // scores of 16 heads x 8 * NK8 keys per warp
+    float s[NK8][4];
+#pragma unroll
+    for (int i = 0; i < NK8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+    const int key0 = wk * NK8 * 8;
+#pragma unroll 4
+    for (int kk = 0; kk < p.CP / 16; ++kk) {
+      uint32_t a[4];
+      ldmatrix_x4(a, smem_u32(sQ + (wm * 16 + (lane & 15)) * ld + kk * 16 + (lane >> 4) * 8));
+      if constexpr (NK8 == 2) {
+        uint32_t f[4];
+        ldmatrix_x4(f, smem_u32(kv + (key0 + (lane & 7) + (lane >> 4) * 8) * ld + kk * 16 + ((lane >> 3) & 1) * 8));
+        mma_16816(s[0], a, f[0], f[1]);
+        mma_16816(s[1], a, f[2], f[3]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < NK8; ++i) {
+          uint32_t f[2];
+          asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n"
+                       : "=r"(f[0]), "=r"(f[1])
+                       : "r"(smem_u32(kv + (key0 + i * 8 + (lane & 7)) * ld + kk * 16 + ((lane >> 3) & 1) * 8)));
+          mma_16816(s[i], a, f[0], f[1]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NK8; ++i) {
+      float* d = sS + (wm * 16 + (lane >> 2)) * LDS_S + key0 + i * 8 + (lane & 3) * 2;
+      d[0] = s[i][0];
+      d[1] = s[i][1];
+      d[8 * LDS_S] = s[i][2];
+      d[8 * LDS_S + 1] = s[i][3];
+    }
+    __syncthreads();
+    // soft-max of one head row by TPR neighbouring threads
+    {
+      float v[KPT], mx = -INFINITY;
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) {
+        const int k = spart + i * TPR;
+        v[i] = tile * KT + k < n ? sS[srow * LDS_S + k] * p.scale_log2 : -INFINITY;
+        mx = fmaxf(mx, v[i]);
+      }
+#pragma unroll
+      for (int x = TPR / 2; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+      const float m_new = fmaxf(m_run, mx);                        // finite: a tile holds at least one key
+      const float corr = exp2f(m_run - m_new);
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < KPT; ++i) {
+        const float e = exp2f(v[i] - m_new);
+        sum += e;
+        sP[srow * LDS_P + spart + i * TPR] = __float2bfloat16_rn(e);
+      }
+#pragma unroll
+      for (int x = TPR / 2; x > 0; x >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, x);
+      l_run = l_run * corr + sum;
+      m_run = m_new;
+      if (spart == 0) sCorr[srow] = corr;
+    }
+    __syncthreads();
+    // o = o * corr + P V, V = the latent columns of the same tile
+    if (col0 < p.RP) {
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        const float ca = sCorr[m * 16 + (lane >> 2)], cb = sCorr[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+          o[m][i][0] *= ca;
+          o[m][i][1] *= ca;
+          o[m][i][2] *= cb;
+          o[m][i][3] *= cb;
+        }
+      }
+#pragma unroll
+      for (int kc = 0; kc < KT / 16; ++kc) {
+        uint32_t a[MT][4];
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+          ldmatrix_x4(a[m], smem_u32(sP + (m * 16 + (lane & 15)) * LDS_P + kc * 16 + (lane >> 4) * 8));
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+          if (col0 + i * 8 < p.RP) {                               // uniform over the warp
+            uint32_t f[2];
+            asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n"
+                         : "=r"(f[0]), "=r"(f[1])
+                         : "r"(smem_u32(kv + (kc * 16 + (lane & 15)) * ld + col0 + i * 8)));
+#pragma unroll
+            for (int m = 0; m < MT; ++m) mma_16816(o[m][i], a[m], f[0], f[1]);
+          }
+        }
+      }
+    }
+    __syncthreads();
+  }
+  if (spart == 0) {
+    sL[srow] = l_run;
+    if (p.nsplit > 1 && h0 + srow < p.H) {
+      float* ml = p.part_ml + (((long long)b * p.H + h0 + srow) * p.nsplit + split) * 2;
+      ml[0] = m_run;
+      ml[1] = l_run;
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int m = 0; m < MT; ++m) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = m * 16 + (lane >> 2) + half * 8;
+      if (h0 + r >= p.H) continue;
+      const float l = sL[r], inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const int c = col0 + i * 8 + (lane & 3) * 2;
+        if (c >= p.RP) continue;
+        const float x = o[m][i][2 * half], y = o[m][i][2 * half + 1];
+        if (p.nsplit == 1) {
+          *reinterpret_cast<__nv_bfloat162*>(p.out + ((long long)b * p.H + h0 + r) * p.RP + c) =
+              __floats2bfloat162_rn(x * inv, y * inv);
+        } else {
+          *reinterpret_cast<float2*>(p.part_o + (((long long)b * p.H + h0 + r) * p.nsplit + split) * p.RP + c) =
+              make_float2(x, y);
+        }
+      }
+    }
+  }
+}
+
+__global__ void combine_kernel(const float* part_o, const float* part_ml, int nsplit, int RP, __nv_bfloat16* out) {
+  const long long r = blockIdx.x;
+  float m = -INFINITY;
+  for (int s = 0; s < nsplit; ++s) m = fmaxf(m, part_ml[(r * nsplit + s) * 2]);
+  float l = 0.f;
+  for (int s = 0; s < nsplit; ++s) {
+    const float ls = part_ml[(r * nsplit + s) * 2 + 1];
+    if (ls > 0.f) l += ls * exp2f(part_ml[(r * nsplit + s) * 2] - m);
+  }
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  for (int c = threadIdx.x; c < RP; c += blockDim.x) {
+    float a = 0.f;
+    for (int s = 0; s < nsplit; ++s)
+      if (part_ml[(r * nsplit + s) * 2 + 1] > 0.f)
+        a += part_o[(r * nsplit + s) * RP + c] * exp2f(part_ml[(r * nsplit + s) * 2] - m);
+    out[r * RP + c] = __float2bfloat16_rn(a * inv);
+  }
+}
+
+template <int MT, int NT, int KT>
+static int launch_mma(const MmaArgs& p, int batch, cudaStream_t st) {
+  constexpr int HM = 16 * MT;
+  const size_t smem = sizeof(__nv_bfloat16) * (size_t)(HM + 2 * KT) * (p.CP + 8) + sizeof(float) * HM * (KT + 4) +
+                      sizeof(__nv_bfloat16) * HM * (KT + 8) + sizeof(float) * 2 * HM;
+  if (smem > 227 * 1024) return (int)cudaErrorNotSupported;
+  cudaError_t e = cudaFuncSetAttribute(decode_mma_kernel<MT, NT, KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return (int)e;
+  const dim3 grid((unsigned)p.nsplit, (unsigned)((p.H + HM - 1) / HM), (unsigned)batch);
+  decode_mma_kernel<MT, NT, KT><<<grid, 256, smem, st>>>(p);
+  if (p.nsplit > 1)
+    combine_kernel<<<(unsigned)(batch * p.H), 128, 0, st>>>(p.part_o, p.part_ml, p.nsplit, p.RP, p.out);
+  return (int)cudaGetLastError();
+}
+
+template <int NT>
+static int pick_mma(const MmaArgs& p, int batch, cudaStream_t st) {
+  if (p.H <= 16) return launch_mma<1, NT, 64>(p, batch, st);
+  if (p.H <= 32) return launch_mma<2, NT, 64>(p, batch, st);
+  return launch_mma<4, NT, 32>(p, batch, st);
+}
+
+}  // namespace mla
+}  // namespace msrl
+
+using namespace msrl;
+
+// ints: H, q_stride, dn, dr, dkv_col, rank, rot_dims, table_rows, RP, CP
+MSRL_API int msrl_latent_prep(void* qkv, long long ld, const int* ints, const float* norm_w, float eps,
+                              const float* table, const int* positions, const long long* slots, void* cache, void* lat,
+                              void* qdec, int tokens, int is_f32, cudaStream_t st) {
+  if (tokens == 0) return 0;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    mla::PrepArgs<T> p{};
+    p.qkv = (T*)qkv;
+    p.ld = ld;
+    p.H = ints[0];
+    p.q_stride = ints[1];
+    p.dn = ints[2];
+    p.dr = ints[3];
+    p.dkv_col = ints[4];
+    p.rank = ints[5];
+    p.rot_dims = ints[6];
+    p.table_rows = ints[7];
+    p.RP = ints[8];
+    p.CP = ints[9];
+    p.norm_w = norm_w;
+    p.eps = eps;
+    p.table = table;
+    p.positions = positions;
+    p.slots = slots;
+    p.cache = (T*)cache;
+    p.lat = (T*)lat;
+    p.qdec = (T*)qdec;
+    mla::prep_kernel<T><<<tokens, 256, 0, st>>>(p);
+    return (int)cudaGetLastError();
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_latent_gather(const void* cache, const int* block_tables, int max_blocks, int block_size,
+                                const int* token_seq, const int* token_pos, void* out, long long rows, int row_bytes,
+                                cudaStream_t st) {
+  if (rows == 0) return 0;
+  if (row_bytes % 16 != 0) return (int)cudaErrorInvalidValue;
+  mla::gather_kernel<<<(unsigned)((rows + 7) / 8), 256, 0, st>>>((const uint4*)cache, block_tables, max_blocks,
+                                                                 block_size, token_seq, token_pos, (uint4*)out, rows,
+                                                                 row_bytes / 16);
+  return (int)cudaGetLastError();
+}
+
+MSRL_API int msrl_latent_spread(const void* lat, int CP, int RP, void* kv, long long ld, int H, int stride, int dn,
+                                int dr, int tokens, int is_f32, cudaStream_t st) {
+  if (tokens == 0 || dr == 0) return 0;
+  if (is_f32)
+    mla::spread_kernel<float><<<tokens, 256, 0, st>>>((const float*)lat, CP, RP, (float*)kv, ld, H, stride, dn, dr, tokens);
+  else
+    mla::spread_kernel<__nv_bfloat16><<<tokens, 256, 0, st>>>((const __nv_bfloat16*)lat, CP, RP, (__nv_bfloat16*)kv, ld, H,
+                                                              stride, dn, dr, tokens);
+  return (int)cudaGetLastError();
+}
+
+// lds: q, k, v, out row strides; ints: q, k, v, out head strides, dq, dv
+MSRL_API int msrl_attn_simt(const void* q, const void* k, const void* v, void* out, const long long* lds,
+                            const int* ints, const int* cu_q, const int* cu_k, int batch, int max_q, int H, float scale,
+                            int is_f32, cudaStream_t st) {
+  if (batch == 0 || max_q == 0) return 0;
+  const int dq = ints[4], dv = ints[5];
+  if (dv > 512 || batch > 65535 || H > 65535) return (int)cudaErrorNotSupported;
+  const size_t smem = sizeof(float) * (2 * (size_t)mla::SB * (dq + 1) + (size_t)mla::SB * dv + mla::SB * (mla::SB + 1));
+  if (smem > 227 * 1024) return (int)cudaErrorNotSupported;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    mla::SimtArgs<T> p{(const T*)q, (const T*)k, (const T*)v, lds[0], lds[1], lds[2], ints[0], ints[1], ints[2],
+                       dq, dv, cu_q, cu_k, scale, (T*)out, lds[3], ints[3]};
+    const dim3 grid((unsigned)((max_q + mla::SB - 1) / mla::SB), (unsigned)H, (unsigned)batch);
+    auto go = [&](auto kernel) {
+      cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return (int)e;
+      kernel<<<grid, 256, smem, st>>>(p);
+      return (int)cudaGetLastError();
+    };
+    if (dv <= 64) return go(mla::attn_simt_kernel<T, 8>);
+    if (dv <= 128) return go(mla::attn_simt_kernel<T, 16>);
+    if (dv <= 256) return go(mla::attn_simt_kernel<T, 32>);
+    return go(mla::attn_simt_kernel<T, 64>);
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_latent_decode_simt(const void* q, const void* cache, const int* block_tables, int max_blocks,
+                                     int block_size, const int* context_lens, float scale, int batch, int H, int CP,
+                                     int RP, void* out, int is_f32, cudaStream_t st) {
+  if (batch == 0) return 0;
+  if (RP > 256 * mla::DS_ACC || batch > 65535 || CP > 12000) return (int)cudaErrorNotSupported;
+  const dim3 grid((unsigned)H, (unsigned)batch);
+  if (is_f32)
+    mla::decode_simt_kernel<float><<<grid, 256, CP * sizeof(float), st>>>((const float*)q, (const float*)cache, block_tables,
+                                                                          max_blocks, block_size, context_lens, scale, CP, RP,
+                                                                          (float*)out);
+  else
+    mla::decode_simt_kernel<__nv_bfloat16><<<grid, 256, CP * sizeof(float), st>>>(
+        (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, block_tables, max_blocks, block_size, context_lens, scale, CP,
+        RP, (__nv_bfloat16*)out);
+  return (int)cudaGetLastError();
+}
+
+// key ranges per (sequence, head group) so that one wave of blocks covers the machine
+MSRL_API int msrl_latent_decode_nsplit(int batch, int H, int max_context) {
+  const int groups = H <= 32 ? 1 : (H + 63) / 64;
+  const int blocks = batch * groups;
+  int n = blocks > 0 ? sm_count() / blocks : 1;
+  const int most = (max_context + 127) / 128;
+  if (n > most) n = most;
+  if (n > 64) n = 64;
+  return n < 1 ? 1 : n;
+}
+
+// part_o [B, H, nsplit, RP] and part_ml [B, H, nsplit, 2] fp32 (unused when nsplit == 1)
+MSRL_API int msrl_latent_decode_mma(const void* q, const void* cache, const int* block_tables, int max_blocks,
+                                    int block_size, const int* context_lens, float scale, int batch, int H, int CP,
+                                    int RP, int nsplit, float* part_o, float* part_ml, void* out, cudaStream_t st) {
+  if (batch == 0) return 0;
+  if (CP % 16 != 0 || RP % 16 != 0 || RP > 512 || batch > 65535) return (int)cudaErrorNotSupported;
+  mla::MmaArgs p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, block_tables, max_blocks, block_size,
+                 context_lens, scale * 1.4426950408889634f, H, CP, RP, nsplit, part_o, part_ml, (__nv_bfloat16*)out};
+  if (RP <= 128) return mla::pick_mma<2>(p, batch, st);
+  if (RP <= 256) return mla::pick_mma<4>(p, batch, st);
+  return mla::pick_mma<8>(p, batch, st);
+}

@@ -1,0 +1,275 @@
+// Kernels around an fp32 residual stream (bf16 or fp32 activations, selected by `is_f32`).
+//
+//   embed_norm        resid[t] = scale * table[id[t]];                        y[t] = norm(resid[t])
+//   add_norm          resid[t] += delta[t];                                   y[t] = norm(resid[t])
+//   moe_combine_norm  resid[t] += w * sum_j e[pos(t, j)] + sig(h[t].sg) * sh[t];  y[t] = norm(resid[t])
+//
+// norm(x) = x * rsqrt(mean(x^2) + eps) * (offset + weight), all in fp32; y is stored in the activation
+// type.  One block per row; the row stays in registers between the sum and the norm (longer rows than the
+// register budget re-read the residual they just wrote).  A null `y` skips the norm.
+//
+//   glu               act(gate) * up of rows [gate | up]: silu, tanh-gelu, or the clamped swish with (up + 1)
+#include "dtype_utils.cuh"
+
+namespace msrl {
+
+constexpr int RS_THREADS = 256;
+
+enum { SRC_EMBED = 0, SRC_DELTA = 1, SRC_MOE = 2 };
+
+template <typename T>
+struct RowArgs {
+  float* resid;
+  const float* norm_w;
+  T* y;
+  int W;
+  float eps, offset;
+  // SRC_EMBED
+  const long long* ids;
+  const T* table;
+  float scale;
+  // SRC_DELTA
+  const T* delta;
+  // SRC_MOE
+  const T* e;
+  const int* pos;
+  int top;
+  float expert_w;
+  const T* h;
+  const T* sg;
+  const T* shared;
+};
+
+template <typename T, int V, int NPT, int SRC>
+__global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p) {
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  const int W = p.W;
+  float* res = p.resid + t * W;
+  const T* tab = nullptr;
+  if constexpr (SRC == SRC_EMBED) tab = p.table + p.ids[t] * W;
+  float sig = 0.f;
+  if constexpr (SRC == SRC_MOE) {
+    if (p.shared != nullptr) {
+      sig = 1.f;
+      if (p.sg != nullptr) {
+        float s = 0.f;
+        for (int c = threadIdx.x * V; c < W; c += RS_THREADS * V) {
+          float a[4], b[4];
+          ldv<V>(p.h + t * W + c, a);
+          ldv<V>(p.sg + c, b);
+#pragma unroll
+          for (int i = 0; i < V; ++i) s += a[i] * b[i];
+        }
+        sig = sigmoid_f(block_sum(s, red));
+      }
+    }
+  }
+  auto value = [&](int c, float (&f)[4]) {
+    if constexpr (SRC == SRC_EMBED) {
+      ldv<V>(tab + c, f);
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] *= p.scale;
+    } else if constexpr (SRC == SRC_DELTA) {
+      float d[4];
+      ldv<V>(res + c, f);
+      ldv<V>(p.delta + t * W + c, d);
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] += d[i];
+    } else {
+      float d[4], acc[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int j = 0; j < p.top; ++j) {
+        ldv<V>(p.e + (long long)p.pos[t * p.top + j] * W + c, d);
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] += d[i];
+      }
+      ldv<V>(res + c, f);
+#pragma unroll
+      for (int i = 0; i < V; ++i) acc[i] *= p.expert_w;
+      if (p.shared != nullptr) {
+        ldv<V>(p.shared + t * W + c, d);
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] += sig * d[i];
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] += acc[i];
+    }
+  };
+  float keep[NPT][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NPT; ++k) {
+    const int c = (k * RS_THREADS + threadIdx.x) * V;
+    if (c < W) {
+      value(c, keep[k]);
+      stv<V>(res + c, keep[k]);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss += keep[k][i] * keep[k][i];
+    }
+  }
+  for (int c = (NPT * RS_THREADS + threadIdx.x) * V; c < W; c += RS_THREADS * V) {
+    float f[4];
+    value(c, f);
+    stv<V>(res + c, f);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss += f[i] * f[i];
+  }
+  if (p.y == nullptr) return;
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + p.eps);
+  T* y = p.y + t * W;
+#pragma unroll
+  for (int k = 0; k < NPT; ++k) {
+    const int c = (k * RS_THREADS + threadIdx.x) * V;
+    if (c < W) {
+      float w[4];
+      ldv<V>(p.norm_w + c, w);
+#pragma unroll
+      for (int i = 0; i < V; ++i) w[i] = keep[k][i] * r * (p.offset + w[i]);
+      stv<V>(y + c, w);
+    }
+  }
+  for (int c = (NPT * RS_THREADS + threadIdx.x) * V; c < W; c += RS_THREADS * V) {
+    float f[4], w[4];
+    ldv<V>(res + c, f);
+    ldv<V>(p.norm_w + c, w);
+#pragma unroll
+    for (int i = 0; i < V; ++i) w[i] = f[i] * r * (p.offset + w[i]);
+    stv<V>(y + c, w);
+  }
+}
+
+template <typename T, int SRC>
+int launch_row_norm(const RowArgs<T>& p, long long rows, cudaStream_t st) {
+  if (rows == 0) return 0;
+  if (p.W % 4 == 0) {
+    const int units = (p.W / 4 + RS_THREADS - 1) / RS_THREADS;
+    if (units <= 1) row_norm_kernel<T, 4, 1, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+    else if (units <= 2) row_norm_kernel<T, 4, 2, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+    else if (units <= 4) row_norm_kernel<T, 4, 4, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+    else row_norm_kernel<T, 4, 8, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+  } else {
+    row_norm_kernel<T, 1, 4, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+  }
+  return (int)cudaGetLastError();
+}
+
+enum { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMPED_SWISH = 2 };
+
+template <int KIND>
+__device__ __forceinline__ float glu_one(float g, float u, float limit, float alpha) {
+  if constexpr (KIND == GLU_SILU) {
+    return g * sigmoid_f(g) * u;
+  } else if constexpr (KIND == GLU_GELU_TANH) {
+    const float k = 0.7978845608028654f;                 // sqrt(2 / pi)
+    return 0.5f * g * (1.f + tanhf(k * (g + 0.044715f * g * g * g))) * u;
+  } else {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoid_f(alpha * g) * (u + 1.f);
+  }
+}
+
+// x [rows, 2F] -> y [rows, F]; rows of a 128-row tile whose tile_expert is negative are skipped, and inside a
+// tile the pad rows past the expert's count
+template <typename T, int V, int KIND>
+__global__ void __launch_bounds__(256)
+glu_kernel(const T* x, T* y, int F, float limit, float alpha, const int* tile_expert, const int* counts,
+           const int* offsets) {
+  const long long r = blockIdx.x;
+  if (tile_expert != nullptr) {
+    const int e = tile_expert[r / 128];
+    if (e < 0 || r - offsets[e] >= counts[e]) return;
+  }
+  const int c = (blockIdx.y * 256 + threadIdx.x) * V;
+  if (c >= F) return;
+  float g[4], u[4];
+  ldv<V>(x + r * 2 * F + c, g);
+  ldv<V>(x + r * 2 * F + F + c, u);
+#pragma unroll
+  for (int i = 0; i < V; ++i) g[i] = glu_one<KIND>(g[i], u[i], limit, alpha);
+  stv<V>(y + r * F + c, g);
+}
+
+template <typename T, int V>
+int launch_glu(const T* x, T* y, long long rows, int F, int kind, float limit, float alpha, const int* tile_expert,
+               const int* counts, const int* offsets, cudaStream_t st) {
+  const dim3 grid((unsigned)rows, (unsigned)((F / V + 255) / 256));
+  if (kind == GLU_SILU)
+    glu_kernel<T, V, GLU_SILU><<<grid, 256, 0, st>>>(x, y, F, limit, alpha, tile_expert, counts, offsets);
+  else if (kind == GLU_GELU_TANH)
+    glu_kernel<T, V, GLU_GELU_TANH><<<grid, 256, 0, st>>>(x, y, F, limit, alpha, tile_expert, counts, offsets);
+  else
+    glu_kernel<T, V, GLU_CLAMPED_SWISH><<<grid, 256, 0, st>>>(x, y, F, limit, alpha, tile_expert, counts, offsets);
+  return (int)cudaGetLastError();
+}
+
+}  // namespace msrl
+
+using namespace msrl;
+
+template <typename T>
+static RowArgs<T> base_args(float* resid, const float* norm_w, void* y, int W, float eps, float offset) {
+  RowArgs<T> p{};
+  p.resid = resid;
+  p.norm_w = norm_w;
+  p.y = (T*)y;
+  p.W = W;
+  p.eps = eps;
+  p.offset = offset;
+  return p;
+}
+
+MSRL_API int msrl_embed_norm(const long long* ids, const void* table, float scale, float* resid, const float* norm_w,
+                             void* y, long long rows, int W, float eps, float offset, int is_f32, cudaStream_t st) {
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    RowArgs<T> p = base_args<T>(resid, norm_w, y, W, eps, offset);
+    p.ids = ids;
+    p.table = (const T*)table;
+    p.scale = scale;
+    return launch_row_norm<T, SRC_EMBED>(p, rows, st);
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_add_norm(const void* delta, float* resid, const float* norm_w, void* y, long long rows, int W,
+                           float eps, float offset, int is_f32, cudaStream_t st) {
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    RowArgs<T> p = base_args<T>(resid, norm_w, y, W, eps, offset);
+    p.delta = (const T*)delta;
+    return launch_row_norm<T, SRC_DELTA>(p, rows, st);
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_moe_combine_norm(const void* e, const int* pos, int top, float expert_w, const void* h,
+                                   const void* sg, const void* shared, float* resid, const float* norm_w, void* y,
+                                   long long rows, int W, float eps, float offset, int is_f32, cudaStream_t st) {
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    RowArgs<T> p = base_args<T>(resid, norm_w, y, W, eps, offset);
+    p.e = (const T*)e;
+    p.pos = pos;
+    p.top = top;
+    p.expert_w = expert_w;
+    p.h = (const T*)h;
+    p.sg = (const T*)sg;
+    p.shared = (const T*)shared;
+    return launch_row_norm<T, SRC_MOE>(p, rows, st);
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_glu_fwd(const void* x, void* y, long long rows, int F, int kind, float limit, float alpha,
+                          const int* tile_expert, const int* counts, const int* offsets, int is_f32,
+                          cudaStream_t st) {
+  if (rows == 0 || F == 0) return 0;
+  if (kind < 0 || kind > 2) return (int)cudaErrorInvalidValue;
+  const bool v4 = F % 4 == 0;
+  if (is_f32)
+    return v4 ? launch_glu<float, 4>((const float*)x, (float*)y, rows, F, kind, limit, alpha, tile_expert, counts, offsets, st)
+              : launch_glu<float, 1>((const float*)x, (float*)y, rows, F, kind, limit, alpha, tile_expert, counts, offsets, st);
+  return v4 ? launch_glu<__nv_bfloat16, 4>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, F, kind, limit, alpha, tile_expert, counts, offsets, st)
+            : launch_glu<__nv_bfloat16, 1>((const __nv_bfloat16*)x, (__nv_bfloat16*)y, rows, F, kind, limit, alpha, tile_expert, counts, offsets, st);
+}

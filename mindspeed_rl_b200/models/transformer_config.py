@@ -90,6 +90,9 @@ class TransformerConfig:
             self.num_query_groups = self.num_attention_heads
             self.kv_channels = self.qk_head_dim + self.qk_pos_emb_head_dim
 
+    is_hybrid = False        # one block repeated (``models.hybrid_config`` lists layers one by one)
+    is_recurrent = False     # nothing but the KV cache is carried from token to token
+
     @property
     def head_dim(self) -> int:
         return self.kv_channels

@@ -78,7 +78,10 @@ def moe_permute(x: torch.Tensor, plan: MoePlan, w: Optional[torch.Tensor] = None
     """``x [T, H]`` -> expert-grouped ``[max_rows, H]`` (row of slot (t, j) = ``w[t, j] * x[t]``);
     pad rows of used segments are zero, rows past the last segment are not touched."""
     t, h = x.shape
-    if _lib.use_kernels(x):
+    if x.dtype == torch.float32 and x.is_cuda and w is None and h % 4 == 0:
+        # rows are only moved: an fp32 row is a bf16 row of twice the length
+        return moe_permute(x.contiguous().view(torch.bfloat16), plan).view(torch.float32)
+    if x.dtype == torch.bfloat16 and h % 8 == 0 and _lib.use_kernels(x):
         x = x.contiguous()
         xp = guard.empty(plan.max_rows, h, dtype=x.dtype, device=x.device)
         wf = None if w is None else w.reshape(-1).float().contiguous()
@@ -86,7 +89,7 @@ def moe_permute(x: torch.Tensor, plan: MoePlan, w: Optional[torch.Tensor] = None
                                            c_int(plan.num_experts), ptr(plan.counts), ptr(plan.offsets), ptr(xp),
                                            c_ll(h), stream()), "moe_permute")
         return xp
-    xp = torch.zeros(plan.max_rows, h, dtype=x.dtype, device=x.device)
+    xp = torch.zeros(plan.max_rows, h, dtype=x.dtype, device=x.device)     # CPU, or rows the kernel cannot move
     rows = x.repeat_interleave(plan.k, dim=0)
     if w is not None:
         rows = (rows.float() * w.reshape(-1, 1).float()).to(x.dtype)
@@ -182,4 +185,21 @@ def grouped_gemm(a: torch.Tensor, plan: MoePlan, b2d: torch.Tensor, b_mn_major: 
         else:
             be = b2d[e * ey:e * ey + n, e * ex:e * ex + k]
             torch.matmul(a[r0:r0 + cnt], be.t(), out=c[r0:r0 + cnt])
+    return c
+
+
+def grouped_gemm_nt(a: torch.Tensor, plan: MoePlan, w: torch.Tensor) -> torch.Tensor:
+    """``c[r] = a[r] @ w[e].T`` for the rows of expert e, ``w [E, N, K]`` contiguous.  bf16 shapes that fit the
+    tcgen05 kernel run there; fp32 (true 32-bit products) and other bf16 shapes on the CUDA cores
+    (``csrc/grouped_gemm_simt.cu``).  Nothing is read back to the host."""
+    e, n, k = w.shape
+    if not _lib.use_kernels(a, w):
+        return grouped_gemm(a, plan, w.reshape(e * n, k), False, 0, n, n)
+    if a.dtype == torch.bfloat16 and k % 64 == 0 and n % 8 == 0 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
+        return grouped_gemm(a, plan, w.view(e * n, k), False, 0, n, n)
+    assert a.is_contiguous() and w.is_contiguous() and a.shape == (plan.max_rows, k) and a.dtype == w.dtype
+    c = guard.empty(plan.max_rows, n, dtype=a.dtype, device=a.device)
+    check(_lib.load().msrl_grouped_gemm_simt(ptr(a), ptr(w), ptr(c), c_int(plan.max_rows), c_int(n), c_int(k),
+                                             ptr(plan.tile_expert), ptr(plan.counts), ptr(plan.offsets),
+                                             c_int(1 if a.dtype == torch.float32 else 0), stream()), "grouped_gemm_simt")
     return c

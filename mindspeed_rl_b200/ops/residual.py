@@ -1,0 +1,106 @@
+"""Kernels around an fp32 residual stream: embedding, residual add and expert combine, each with the norm that
+follows fused in, and the gated activations.
+
+The residual ``[T, W]`` is fp32 and updated in place; norm weights are fp32, the activations bf16 or fp32.
+``norm(x) = x / sqrt(mean(x^2) + eps) * (offset + w)`` in fp32.  CUDA path: ``csrc/residual_stream.cu``; CPU
+tensors run the PyTorch formulation.
+"""
+from __future__ import annotations
+
+from typing import Optional, Tuple
+
+import torch
+import torch.nn.functional as F
+
+from . import guard
+
+from . import _lib
+from ._lib import c_float, c_int, c_ll, check, ptr, stream
+
+
+def _is_f32(t: torch.Tensor):
+    if t.dtype not in (torch.float32, torch.bfloat16):
+        raise TypeError(f"bf16 or fp32 activations expected, got {t.dtype}")
+    return c_int(1 if t.dtype == torch.float32 else 0)
+
+
+def _norm_ref(x: torch.Tensor, w: torch.Tensor, eps: float, offset: float, dtype) -> torch.Tensor:
+    return (x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (offset + w)).to(dtype)
+
+
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, w: torch.Tensor, eps: float,
+               offset: float = 0.0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``(residual fp32, norm(residual))`` of ``residual = table[ids] * scale``."""
+    t, h = ids.numel(), table.shape[1]
+    if _lib.use_kernels(ids, table, w):
+        resid = guard.empty(t, h, device=table.device, dtype=torch.float32)
+        y = guard.empty(t, h, device=table.device, dtype=table.dtype)
+        check(_lib.load().msrl_embed_norm(ptr(ids), ptr(table), c_float(scale), ptr(resid), ptr(w), ptr(y), c_ll(t),
+                                          c_int(h), c_float(eps), c_float(offset), _is_f32(table), stream()), "embed_norm")
+        return resid, y
+    resid = table[ids].float() * scale
+    return resid, _norm_ref(resid, w, eps, offset, table.dtype)
+
+
+def add_norm_(resid: torch.Tensor, delta: torch.Tensor, w: torch.Tensor, eps: float, offset: float = 0.0
+              ) -> torch.Tensor:
+    """``resid += delta`` in place; returns ``norm(resid)`` in ``delta``'s type."""
+    t, h = resid.shape
+    if _lib.use_kernels(resid, delta, w):
+        delta = delta.contiguous()
+        y = guard.empty(t, h, device=resid.device, dtype=delta.dtype)
+        check(_lib.load().msrl_add_norm(ptr(delta), ptr(resid), ptr(w), ptr(y), c_ll(t), c_int(h), c_float(eps),
+                                        c_float(offset), _is_f32(delta), stream()), "add_norm")
+        return y
+    resid.add_(delta.float())
+    return _norm_ref(resid, w, eps, offset, delta.dtype)
+
+
+def moe_combine_norm_(resid: torch.Tensor, expert_rows: torch.Tensor, pos: torch.Tensor, top: int, expert_w: float,
+                      h: torch.Tensor, shared: Optional[torch.Tensor], shared_gate: Optional[torch.Tensor],
+                      w: torch.Tensor, eps: float, offset: float = 0.0) -> torch.Tensor:
+    """``resid[t] += expert_w * sum_j expert_rows[pos[t, j]] + sigmoid(h[t] . shared_gate) * shared[t]`` in
+    place; returns ``norm(resid)``.  ``pos [T * top]`` are the rows of a dispatch plan (``ops.moe``); without
+    ``shared`` the second term is left out."""
+    t, width = resid.shape
+    if _lib.use_kernels(resid, expert_rows, pos, h):
+        y = guard.empty(t, width, device=resid.device, dtype=h.dtype)
+        check(_lib.load().msrl_moe_combine_norm(
+            ptr(expert_rows), ptr(pos), c_int(top), c_float(expert_w), ptr(h.contiguous()), ptr(shared_gate),
+            ptr(shared), ptr(resid), ptr(w), ptr(y), c_ll(t), c_int(width), c_float(eps), c_float(offset), _is_f32(h),
+            stream()), "moe_combine_norm")
+        return y
+    add = expert_rows[pos.long()].float().view(t, top, width).sum(1) * expert_w
+    if shared is not None:
+        sig = 1.0 if shared_gate is None else torch.sigmoid(h.float() @ shared_gate.float().reshape(-1, 1))
+        add = add + sig * shared.float()
+    resid.add_(add)
+    return _norm_ref(resid, w, eps, offset, h.dtype)
+
+
+GLU_KINDS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
+
+
+def glu_fwd(gate_up: torch.Tensor, act: str, limit: float = 0.0, alpha: float = 1.0, plan=None) -> torch.Tensor:
+    """Gated activation of ``[rows, gate | up]``: ``silu(g) * u``, ``gelu_tanh(g) * u`` or ``clamped_swish``:
+    ``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)``.  With a
+    dispatch ``plan`` the rows are expert-grouped and pad rows are left untouched."""
+    kind = GLU_KINDS[act]
+    rows, f = gate_up.shape[0], gate_up.shape[-1] // 2
+    if _lib.use_kernels(gate_up):
+        x = gate_up.contiguous()
+        y = guard.empty(rows, f, device=x.device, dtype=x.dtype)
+        check(_lib.load().msrl_glu_fwd(ptr(x), ptr(y), c_ll(rows), c_int(f), c_int(kind), c_float(limit), c_float(alpha),
+                                       ptr(plan.tile_expert if plan is not None else None),
+                                       ptr(plan.counts if plan is not None else None),
+                                       ptr(plan.offsets if plan is not None else None), _is_f32(x), stream()), "glu_fwd")
+        return y
+    g, u = gate_up.float().split(f, dim=-1)
+    if act == "silu":
+        y = F.silu(g) * u
+    elif act == "gelu_tanh":
+        y = F.gelu(g, approximate="tanh") * u
+    else:
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        y = g * torch.sigmoid(alpha * g) * (u + 1.0)
+    return y.to(gate_up.dtype)

@@ -30,7 +30,8 @@ from ..obs.io_counter import count_d2h, to_device, to_host
 from ..parallel.tp_comm import NO_TP, TPComm
 from .base_engine import BaseInferEngine
 from .block_manager import BlockManager
-from .model_runner import KVCache, ModelRunner, RolloutWeights
+from .layer_cache import HybridCache, StateSlots
+from .model_runner import ModelRunner, RolloutWeights
 from .scheduler import (PrefillItem, RequestGroup, SamplingParams, Scheduler, SchedulerOutput, SeqStatus,
                         Sequence)
 
@@ -87,32 +88,38 @@ class LLMEngine(BaseInferEngine):
         self.scheduler: Optional[Scheduler] = None
         self._step_counter = 0
         self.host_time = collections.defaultdict(float)   # wall-clock seconds per host-side section
-        nkv_local = max(cfg.num_query_groups // self.comm.world_size, 1)
-        nh_local = cfg.num_attention_heads // self.comm.world_size
-        # shared prompts are rounded down to the tensor-core prefix kernel's key tile (0: the mma.sync kernel takes any length)
-        self._prefix_tile = ops.decode_prefix_tile(nh_local, nkv_local, cfg.head_dim, block_size) \
-            if torch.device(device).type == "cuda" else 0
-        self.runner.prefix_tile = self._prefix_tile
-        self._group_max = ops.decode_group_max(nh_local, nkv_local, self._prefix_tile)
-        self.shared_prefix_decode = os.environ.get("MSRL_SHARED_PREFIX_DECODE", "1") == "1"
+        self._prefix_tile, self._group_max, self.shared_prefix_decode = 0, 1, False
+        if cfg.is_recurrent and enable_prefix_caching:
+            raise ValueError("prefix caching restores cached keys only, not the recurrent state behind them; "
+                             "turn enable_prefix_caching off for models with recurrent layers")
+        if not cfg.is_hybrid:
+            nkv_local = max(cfg.num_query_groups // self.comm.world_size, 1)
+            nh_local = cfg.num_attention_heads // self.comm.world_size
+            # shared prompts are rounded down to the tensor-core prefix kernel's key tile (0: the mma.sync kernel takes any length)
+            if torch.device(device).type == "cuda":
+                self._prefix_tile = ops.decode_prefix_tile(nh_local, nkv_local, cfg.head_dim, block_size)
+            self.runner.prefix_tile = self._prefix_tile
+            self._group_max = ops.decode_group_max(nh_local, nkv_local, self._prefix_tile)
+            self.shared_prefix_decode = os.environ.get("MSRL_SHARED_PREFIX_DECODE", "1") == "1"
+        self._replayed: Dict[str, Sequence] = {}        # sequences driven by ``replay``
         self.lookahead_decode = os.environ.get("MSRL_LOOKAHEAD_DECODE", "1") == "1" and lockstep_group is None
         self.stats = dict(prefill_tokens=0, decode_tokens=0, steps=0, preemptions=0, lookahead_steps=0)
 
     # ---- cache lifecycle -----------------------------------------------------------------------
     def kv_bytes_per_block(self) -> int:
-        c = self.cfg
-        nkv = c.num_query_groups // self.comm.world_size
-        return KVCache.bytes_per_block(c.num_layers, self.block_size, nkv, c.head_dim, c.params_dtype)
+        return self.runner.bytes_per_block(self.block_size)
+
+    def state_bytes(self) -> int:
+        """Memory of the recurrent-state slots (0 for models without recurrent layers)."""
+        return self.max_num_seqs * HybridCache.bytes_per_slot(self.cfg) if self.cfg.is_hybrid else 0
 
     def init_cache(self, num_blocks: int) -> None:
-        c = self.cfg
-        nkv = c.num_query_groups // self.comm.world_size
-        cache = KVCache(c.num_layers, num_blocks, self.block_size, nkv, c.head_dim, c.params_dtype,
-                        self.device)
-        self.runner.bind_cache(cache)
+        self.runner.bind_cache(self.runner.make_cache(num_blocks, self.block_size, self.max_num_seqs))
         self.bm = BlockManager(num_blocks, self.block_size, self.enable_prefix_caching)
+        self.state_slots = StateSlots(self.max_num_seqs) if self.cfg.is_recurrent else None
         self.scheduler = Scheduler(self.bm, self.max_num_seqs, self.max_num_batched_tokens,
-                                   self.max_model_len)
+                                   self.max_model_len, self.state_slots)
+        self._replayed.clear()
 
     def free_cache(self) -> None:
         if os.environ.get("MSRL_ENGINE_PROFILE", "0") == "1" and self.host_time:
@@ -152,6 +159,9 @@ class LLMEngine(BaseInferEngine):
         rid = request_id or f"req-{self._request_counter:010d}"
         if rid in self.scheduler.groups:
             raise ValueError(f"request id {rid} is already in flight")
+        if self.cfg.is_recurrent and params.n > self.max_num_seqs:
+            raise ValueError(f"{params.n} samples of one prompt need as many recurrent-state slots (max_num_seqs is "
+                             f"{self.max_num_seqs})")
         lead = Sequence(rid, list(int(t) for t in prompt_token_ids), params, sample_index=0)
         if mm is not None and mm.get("vit_embeds") is not None:
             if self.enable_prefix_caching:
@@ -274,9 +284,11 @@ class LLMEngine(BaseInferEngine):
         elif len(seq.output_ids) >= p.max_tokens or seq.total_len >= self.max_model_len:
             self.scheduler.finish(seq, SeqStatus.FINISHED_LENGTH)
 
-    def _run_prefill(self, items: List[PrefillItem]) -> None:
+    def _prefill_logits(self, items: List[PrefillItem], rows: List[List[int]]) -> torch.Tensor:
+        """Run prompt portions as one batch; ``rows[i]`` are the places inside portion i whose logits are
+        returned, in order."""
         dev = self.device
-        ids, pos, slots, cu, last_rows, finishing = [], [], [], [0], [], []
+        ids, pos, slots, cu, last_rows = [], [], [], [0], []
         need_prefix = any(it.start > 0 for it in items)
         tok_seq, tok_pos, cu_k = [], [], [0]
         for row, it in enumerate(items):
@@ -285,10 +297,8 @@ class LLMEngine(BaseInferEngine):
             ids.extend(all_ids[it.start:it.start + it.length])
             pos.extend(range(it.start, it.start + it.length))
             slots.append(self.bm.slots(s.seq_id, it.start, it.length))
+            last_rows.extend(cu[-1] + r for r in rows[row])
             cu.append(cu[-1] + it.length)
-            if it.completes_prompt:
-                last_rows.append(cu[-1] - 1)
-                finishing.append(s)
             if need_prefix:
                 end = it.start + it.length
                 tok_seq.extend([row] * end)
@@ -305,12 +315,22 @@ class LLMEngine(BaseInferEngine):
             pt, _ = self._ship([tok_seq, tok_pos])
             prefix = dict(block_tables=to_device(bt, torch.int32, dev), token_seq=pt[0].to(torch.int32),
                           token_pos=pt[1].to(torch.int32), cu_k=to_device(cu_k, torch.int32, dev))
+        state = None
+        if self.cfg.is_hybrid:
+            st, _ = self._ship([[it.start for it in items], [it.seq.state_slot for it in items]])
+            owner = np.repeat(np.arange(len(items)), [it.length for it in items])
+            state = dict(token_seq=to_device(owner, torch.int32, dev), start_pos=st[0].to(torch.int32), slots=st[1])
         logits = self.runner.prefill(t_ids, t_pos, t_slots, t_cu, max(it.length for it in items), t_last,
-                                     prefix, self._prefill_mm(items, ids, pos))
+                                     prefix, self._prefill_mm(items, ids, pos), state)
         self.stats["prefill_tokens"] += len(ids)
         for it in items:
             it.seq.num_computed = it.start + it.length
             self.bm.commit(it.seq.seq_id, it.seq.all_ids, it.seq.num_computed)
+        return logits
+
+    def _run_prefill(self, items: List[PrefillItem]) -> None:
+        finishing = [it.seq for it in items if it.completes_prompt]
+        logits = self._prefill_logits(items, [[it.length - 1] if it.completes_prompt else [] for it in items])
         if not finishing:
             return
         # fork n-sample groups, then sample one token per resulting sequence
@@ -323,6 +343,8 @@ class LLMEngine(BaseInferEngine):
                 for child, (src, dst) in self.scheduler.fork_group(lead):
                     if src >= 0:
                         self.runner.cache.copy_block(src, dst)
+                    if child.state_slot >= 0:
+                        self.runner.cache.copy_slot(lead.state_slot, child.state_slot)
                     rows.append(r)
                     seqs.append(child)
         keys, floats, need_filter, need_eos = self._sampling_rows(seqs)
@@ -390,6 +412,7 @@ class LLMEngine(BaseInferEngine):
                 multiple=max(1, self._prefix_tile))
             if grouped:
                 rows += [ks, gpre] + [list(col) for col in zip(*grows)]
+        rows.append([s.state_slot for s in seqs])
         t1 = time.perf_counter()
         it_, ft = self._ship(rows, floats)
         max_ctx = max(lens)
@@ -403,7 +426,8 @@ class LLMEngine(BaseInferEngine):
         if prev is not None:
             ids = prev["tokens"] if last == list(range(len(prev["seqs"]))) else prev["tokens"][it_[0]]
         t2 = time.perf_counter()
-        logits = self.runner.decode(ids, it_[1].to(torch.int32), it_[2], bt, it_[3].to(torch.int32), max_ctx, groups)
+        logits = self.runner.decode(ids, it_[1].to(torch.int32), it_[2], bt, it_[3].to(torch.int32), max_ctx, groups,
+                                    it_[-1] if self.cfg.is_recurrent else None)
         self.stats["decode_tokens"] += b
         tokens, logprobs = self._sample_device(logits, it_[4], ft, need_filter, need_eos)
         tokens = tokens.long()
@@ -476,6 +500,66 @@ class LLMEngine(BaseInferEngine):
             if any(s.finished for s in cont):
                 break                              # regroup without the finished sequences
         self._finish_decode(h)
+
+    # ---- given token ids instead of sampled ones ------------------------------------------------------
+    def replay(self, entries: Seq_[Tuple[str, Seq_[int], Seq_[int]]], end: Seq_[str] = ()) -> torch.Tensor:
+        """One teacher-forced step.  ``entries``: ``(request id, next tokens, wanted places among them)``; a new id
+        starts a sequence, a known one continues from the cache and state that earlier calls left.  Returns the
+        logits of the wanted places (``[n, V]``, entry by entry).  ``end``: requests that give back what they hold.
+
+        Sequences are admitted, batched and released by the scheduler and managers of generation: single tokens of
+        running sequences are a decode step, everything else prompt portions under the token budget."""
+        portions, single = [], []
+        for i, (rid, tokens, want) in enumerate(entries):
+            tokens = [int(t) for t in tokens]
+            seq = self._replayed.get(rid)
+            if seq is None:
+                seq = Sequence(rid, tokens, SamplingParams(max_tokens=self.max_model_len))
+                self.scheduler.admit(seq)
+                self._replayed[rid] = seq
+            else:
+                self.bm.append(seq.seq_id, len(tokens))
+                seq.output_ids.extend(tokens)
+                seq.prefill_target = seq.total_len
+            if seq.total_len > self.max_model_len:
+                raise ValueError(f"request {rid} exceeds max_model_len ({self.max_model_len})")
+            if len(tokens) == 1 and seq.num_computed > 0:
+                single.append((i, seq, want))
+            else:
+                portions.append((i, seq, seq.num_computed, len(tokens), want))
+        out: List[Optional[torch.Tensor]] = [None] * len(entries)
+        while portions:
+            budget, batch, rows, left = self.max_num_batched_tokens, [], [], []
+            for i, seq, start, n, want in portions:
+                take = min(n, budget)
+                if take > 0:
+                    batch.append((i, PrefillItem(seq, start, take)))
+                    rows.append([w for w in want if w < take])
+                    budget -= take
+                if take < n:
+                    left.append((i, seq, start + take, n - take, [w - take for w in want if w >= take]))
+            logits = self._prefill_logits([it for _, it in batch], rows)
+            for (i, _), part in zip(batch, logits.split([len(r) for r in rows])):
+                out[i] = part if out[i] is None else torch.cat([out[i], part])
+            portions = left
+        if single:
+            seqs = [s for _, s, _ in single]
+            lens = [s.total_len for s in seqs]
+            slots = [int(self.bm.slots(s.seq_id, n - 1, 1)[0]) for s, n in zip(seqs, lens)]
+            it_, _ = self._ship([[s.all_ids[-1] for s in seqs], [n - 1 for n in lens], slots, lens,
+                                 [s.state_slot for s in seqs]])
+            max_blocks = (max(lens) + self.block_size - 1) // self.block_size
+            bt = to_device(self.bm.block_tables([s.seq_id for s in seqs], max_blocks), torch.int32, self.device)
+            logits = self.runner.decode(it_[0], it_[1].to(torch.int32), it_[2], bt, it_[3].to(torch.int32), max(lens),
+                                        None, it_[4] if self.cfg.is_recurrent else None)
+            self.stats["decode_tokens"] += len(seqs)
+            for (i, s, want), n, row in zip(single, lens, logits.clone()):
+                s.num_computed = n
+                out[i] = row[None][[0] * len(want)]
+        for rid in end:
+            self.scheduler.finish(self._replayed.pop(rid), SeqStatus.FINISHED_STOPPED)
+        parts = [p for p in out if p is not None]
+        return torch.cat(parts) if parts else torch.empty(0, self.cfg.vocab_size, device=self.device)
 
     def _to_output(self, group: RequestGroup) -> RequestOutput:
         reasons = {SeqStatus.FINISHED_STOPPED: "stop", SeqStatus.FINISHED_LENGTH: "length",

@@ -1,0 +1,171 @@
+"""Token mixers of layer-by-layer decoders (``models.hybrid_config``) in the rollout engine.
+
+A mixer owns the fused weights of one layer and reads / writes the carried state of one layer run through the
+:class:`StepMeta` of the step.  ``prefill`` takes packed prompt portions, ``decode`` one token per sequence; both
+return the mixer's output before the residual add.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Dict, List, Optional
+
+import torch
+
+from .. import ops
+from ..ops.delta import DeltaLayout, DeltaWeights
+from ..ops.gemm import linear_fwd
+from ..ops.latent import LatentLayout
+
+
+@dataclass
+class StepMeta:
+    """Where the tokens of a step sit: shared by all layers of the step."""
+    ids: torch.Tensor                       # [T] int64
+    positions: torch.Tensor                 # [T] int32
+    slots: torch.Tensor                     # [T] int64 cache row of every token (-1: none)
+    state_slots: torch.Tensor               # [B] int64 recurrent-state slot of every sequence (-1: none)
+    max_model_len: int
+    # prompt portions
+    cu_q: Optional[torch.Tensor] = None     # [B + 1] int32
+    max_q: int = 0
+    tok_seq: Optional[torch.Tensor] = None  # [T] int32
+    start_pos: Optional[torch.Tensor] = None  # [B] int32 position of a portion's first token
+    prefix: Optional[dict] = None           # see ModelRunner.prefill
+    # decode steps
+    block_tables: Optional[torch.Tensor] = None
+    context_lens: Optional[torch.Tensor] = None
+    max_context: int = 0
+
+    @property
+    def is_decode(self) -> bool:
+        return self.block_tables is not None
+
+
+def _pad_rows(w: torch.Tensor, rows: int) -> torch.Tensor:
+    if w.shape[0] == rows:
+        return w
+    return torch.cat([w, w.new_zeros(rows - w.shape[0], *w.shape[1:])])
+
+
+def _pad_cols(w: torch.Tensor, cols: int) -> torch.Tensor:
+    if w.shape[-1] == cols:
+        return w
+    return torch.cat([w, w.new_zeros(*w.shape[:-1], cols - w.shape[-1])], dim=-1)
+
+
+def _pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+def stack_sections(parts: List[torch.Tensor]):
+    """Rows of several projections of one input as one weight; every section starts on a multiple of eight
+    columns of the product (zero rows in between).  Returns the weight and the section starts."""
+    cols, start, padded = [], 0, []
+    for p in parts:
+        cols.append(start)
+        padded.append(_pad_rows(p, _pad8(p.shape[0])))
+        start += padded[-1].shape[0]
+    return torch.cat(padded).contiguous(), cols
+
+
+class LatentAttention:
+    """Heads are padded to a size the tensor-core attention kernels serve (zero rows and columns in the weights,
+    so that the products are unchanged); other sizes and fp32 run unpadded on the CUDA cores."""
+
+    def __init__(self, spec, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.spec, self.eps = spec, eps
+        h, dn, dr, dv, r = spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank
+        qp, vp = dn + dr, dv
+        if dtype == torch.bfloat16 and max(qp, vp) <= 128:
+            qp = vp = 64 if max(qp, vp) <= 64 else 128
+        q = _pad_cols(w["q"].view(h, dn + dr, -1).transpose(1, 2), qp).transpose(1, 2).reshape(h * qp, -1)
+        fused, cols = stack_sections([q, w["dkv"]])
+        self.lay = lay = LatentLayout(h, dn, dr, dv, r, qp, vp, cols[1], spec.rot.dims)
+        uk = _pad_cols(w["uk"], lay.RP).view(h, dn, lay.RP)
+        uv = _pad_cols(w["uv"], lay.RP).view(h, dv, lay.RP)
+        k_rows = torch.cat([uk, uk.new_zeros(h, qp - dn, lay.RP)], dim=1)
+        v_rows = torch.cat([uv, uv.new_zeros(h, vp - dv, lay.RP)], dim=1)
+
+        def put(t):
+            return t.to(device=device, dtype=dtype).contiguous()
+
+        self.w_in = put(fused)
+        self.w_kv = put(torch.cat([k_rows.reshape(h * qp, lay.RP), v_rows.reshape(h * vp, lay.RP)]))
+        self.w_k = self.w_kv[:h * qp].view(h, qp, lay.RP)[:, :dn]       # [H, dn, RP]: folds W_uk into the query
+        self.w_v = self.w_kv[h * qp:].view(h, vp, lay.RP)               # [H, vp, RP]
+        self.w_o = put(_pad_cols(w["o"].view(-1, h, dv), vp).reshape(-1, h * vp))
+        self.norm = w["dkv.norm"].to(device=device, dtype=torch.float32).contiguous()
+
+    def _table(self, meta: StepMeta) -> torch.Tensor:
+        # whole powers of two, so that engines with different length limits share tables
+        rows = 1 << max(meta.max_model_len - 1, 1).bit_length()
+        return ops.rope_table(rows, self.spec.rot.dims, self.spec.rot.base, self.w_in.device)
+
+    def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        lay, pre = self.lay, meta.prefix
+        proj = linear_fwd(x, self.w_in)
+        rows = ops.latent_prep(proj, lay, self.norm, self.eps, self._table(meta), meta.positions, meta.slots,
+                               cache.latent[run], want_rows=pre is None)
+        cu_k = meta.cu_q
+        if pre is not None:
+            rows = ops.latent_gather(cache.latent[run], pre["block_tables"], pre["token_seq"], pre["token_pos"])
+            cu_k = pre["cu_k"]
+        kv = linear_fwd(rows[:, :lay.RP], self.w_kv)
+        ops.latent_spread_(kv, rows, lay)
+        attn = ops.latent_prefill_attention(proj, kv, lay, meta.cu_q, cu_k, meta.max_q, self.spec.scale)
+        return linear_fwd(attn, self.w_o)
+
+    def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        lay, b = self.lay, x.shape[0]
+        proj = linear_fwd(x, self.w_in)
+        q = torch.empty(b, lay.heads, lay.CP, dtype=x.dtype, device=x.device)
+        ops.latent_prep(proj, lay, self.norm, self.eps, self._table(meta), meta.positions, meta.slots,
+                        cache.latent[run], want_rows=False, decode_q=q)
+        heads = proj[:, :lay.heads * lay.qp].view(b, lay.heads, lay.qp)
+        torch.bmm(heads[..., :lay.dn].transpose(0, 1), self.w_k, out=q[..., :lay.RP].transpose(0, 1))
+        lat = ops.latent_decode_attention(q, cache.latent[run], lay, meta.block_tables, meta.context_lens,
+                                          meta.max_context, self.spec.scale)
+        attn = torch.empty(b, lay.heads, lay.vp, dtype=x.dtype, device=x.device)
+        torch.bmm(lat.transpose(0, 1), self.w_v.transpose(1, 2), out=attn.transpose(0, 1))
+        return linear_fwd(attn.view(b, lay.heads * lay.vp), self.w_o)
+
+
+class ChannelDelta:
+    def __init__(self, spec, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.spec, self.eps = spec, eps
+        fused, cols = stack_sections([w["q"], w["k"], w["v"], w["b"], w["a1"], w["g1"]])
+        self.lay = DeltaLayout(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.conv, *cols[:4],
+                               unit_eps=spec.unit_eps)
+        ra, rg = _pad8(w["a1"].shape[0]), _pad8(w["g1"].shape[0])
+        self.a_cols, self.g_cols = slice(cols[4], cols[4] + ra), slice(cols[5], cols[5] + rg)
+
+        def put(t, dt=dtype):
+            return t.to(device=device, dtype=dt).contiguous()
+
+        f32 = torch.float32
+        self.w_in = put(fused)
+        self.w_a2, self.w_g2 = put(_pad_cols(w["a2"], ra)), put(_pad_cols(w["g2"], rg))
+        self.w_o = put(w["o"])
+        self.state = DeltaWeights(conv=put(torch.cat([w["q.conv"], w["k.conv"], w["v.conv"]]), f32),
+                                  a_log=put(w["A_log"], f32), dt_bias=put(w["dt_bias"], f32), norm=put(w["norm"], f32))
+        if self.state.conv.shape != (self.lay.channels, spec.conv):
+            raise ValueError(f"convolution weights {tuple(self.state.conv.shape)} do not fit {spec}")
+
+    def _project(self, x: torch.Tensor):
+        proj = linear_fwd(x, self.w_in)
+        return proj, linear_fwd(proj[:, self.a_cols], self.w_a2), linear_fwd(proj[:, self.g_cols], self.w_g2)
+
+    def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        proj, a, gate = self._project(x)
+        y = ops.delta_prefill(proj, a, gate, self.lay, self.state, cache.ring[run], cache.state[run], meta.tok_seq,
+                              meta.cu_q, meta.start_pos, meta.state_slots, self.eps)
+        return linear_fwd(y, self.w_o)
+
+    def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        proj, a, gate = self._project(x)
+        y = ops.delta_decode(proj, a, gate, self.lay, self.state, cache.ring[run], cache.state[run], meta.positions,
+                             meta.state_slots, self.eps)
+        return linear_fwd(y, self.w_o)
+
+
+MIXERS = {"latent_attention": LatentAttention, "channel_delta": ChannelDelta}

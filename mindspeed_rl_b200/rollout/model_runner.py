@@ -8,6 +8,10 @@ rollout phase (reference contract: ``VLLMInferEngine.sync_model_weights``,
 Two entry points: ``prefill`` (packed prompt chunks, varlen attention, KV written to the cache)
 and ``decode`` (one token per sequence, paged attention).  Decode steps are replayed from CUDA
 graphs captured per batch-size bucket; all graph inputs live in static buffers.
+
+Decoders that are composed layer by layer (``models.hybrid_config``) bind ``HybridWeights`` and a
+``HybridCache`` instead; they run through the same two entry points, graphs and buffers, with an
+fp32 residual stream and the mixers and feed-forwards of ``rollout.mixers`` / ``rollout.feed_forward``.
 """
 from __future__ import annotations
 
@@ -21,6 +25,8 @@ from ..models.transformer_config import TransformerConfig
 from ..ops import QKVLayout
 from ..ops.gemm import linear_fwd
 from ..parallel.tp_comm import NO_TP, TPComm
+from .layer_cache import HybridCache
+from .mixers import StepMeta
 
 
 @dataclass
@@ -46,6 +52,11 @@ class RolloutWeights:
     lm_head: torch.Tensor
     qkv_layout: QKVLayout
     vocab_start: int = 0
+
+    def signature(self):
+        """Addresses of what captured graphs read."""
+        return (self.embed.data_ptr(), self.lm_head.data_ptr(),
+                tuple((l.qkv_w if l.qkv_w is not None else l.o_w).data_ptr() for l in self.layers))
 
 
 class KVCache:
@@ -84,6 +95,9 @@ class ModelRunner:
         self._rope = None
         self._graphs: Dict[tuple, dict] = {}
         self._static: Optional[dict] = None
+        if cfg.is_hybrid and self.comm.world_size > 1:
+            raise NotImplementedError(f"{cfg.architecture} is served on one GPU per replica (tensor parallel size 1)")
+        self.layer_probe = None   # callable(run, residual [T, W] fp32) after every layer run of a hybrid decoder (eager steps)
         self.prefix_tile = 0      # key tile of the tcgen05 shared-prefix kernel (set by the engine; 0 = mma.sync kernel)
 
     # ------------------------------------------------------------------------------------------
@@ -91,12 +105,24 @@ class ModelRunner:
         """(Re)bind parameters; graphs stay valid as long as the tensors keep their addresses."""
         old = self.weights
         self.weights = weights
-        if weights is None or old is None or self._signature(old) != self._signature(weights):
+        if weights is None or old is None or old.signature() != weights.signature():
             self._graphs.clear()
 
-    @staticmethod
-    def _signature(w: RolloutWeights):
-        return (w.embed.data_ptr(), w.lm_head.data_ptr(), tuple((l.qkv_w if l.qkv_w is not None else l.o_w).data_ptr() for l in w.layers))
+    def bytes_per_block(self, block_size: int) -> int:
+        c = self.cfg
+        if c.is_hybrid:
+            return HybridCache.bytes_per_block(c, block_size)
+        return KVCache.bytes_per_block(c.num_layers, block_size, c.num_query_groups // self.comm.world_size, c.head_dim,
+                                       c.params_dtype)
+
+    def make_cache(self, num_blocks: int, block_size: int, num_slots: int):
+        """The cache of this model: paged K / V, or what the layers of a hybrid decoder carry (``num_slots``
+        sequences at most keep recurrent state)."""
+        c = self.cfg
+        if c.is_hybrid:
+            return HybridCache(c, num_blocks, block_size, num_slots, self.device)
+        return KVCache(c.num_layers, num_blocks, block_size, c.num_query_groups // self.comm.world_size, c.head_dim,
+                       c.params_dtype, self.device)
 
     def bind_cache(self, cache: Optional[KVCache]) -> None:
         self.cache = cache
@@ -173,6 +199,27 @@ class ModelRunner:
                                   want_rstd=False)
         return x
 
+    def _forward_hybrid(self, meta: StepMeta) -> torch.Tensor:
+        """Final hidden states ``[T, H]`` of a layer-by-layer decoder: the fp32 residual is updated in place by
+        kernels that add and take the next norm in one pass."""
+        w, c, cache = self.weights, self.cfg, self.cache
+        eps, off = c.norm_epsilon, c.norm_offset
+        order = c.run_order
+        resid, x = ops.embed_norm(meta.ids, w.embed, c.embedding_scale, w.layers[order[0]].norm1, eps, off)
+        for run, li in enumerate(order):
+            lw = w.layers[li]
+            after = w.layers[order[run + 1]].norm1 if run + 1 < len(order) else w.final_norm
+            mix = lw.mixer.decode if meta.is_decode else lw.mixer.prefill
+            delta = mix(x, meta, cache, run)
+            if lw.ff is None:
+                x = ops.add_norm_(resid, delta, after, eps, off)
+            else:
+                x = ops.add_norm_(resid, delta, lw.norm2, eps, off)
+                x = lw.ff.forward_norm_(resid, x, meta.ids, after, eps, off)
+            if self.layer_probe is not None:
+                self.layer_probe(run, resid)
+        return x
+
     def _logits(self, x: torch.Tensor) -> torch.Tensor:
         return linear_fwd(x, self.weights.lm_head)
 
@@ -180,14 +227,22 @@ class ModelRunner:
     @torch.no_grad()
     def prefill(self, ids: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor,
                 cu_q: torch.Tensor, max_q: int, last_index: torch.Tensor,
-                prefix: Optional[dict] = None, mm: Optional[dict] = None) -> torch.Tensor:
+                prefix: Optional[dict] = None, mm: Optional[dict] = None,
+                state: Optional[dict] = None) -> torch.Tensor:
         """Run packed prompt chunks. ``last_index`` selects the rows whose logits are needed.
 
         ``prefix`` (for chunks that start inside a sequence) carries ``block_tables``,
         ``token_seq``, ``token_pos``, ``cu_k``: the K/V of ``[0, chunk_end)`` is gathered from the
         cache after this chunk's K/V has been written.
+
+        ``state`` (hybrid decoders): ``token_seq [T]`` and ``start_pos [B]`` (int32), ``slots [B]`` (int64, the
+        recurrent-state slot of every sequence).
         """
         cache = self.cache
+        if self.cfg.is_hybrid:
+            meta = StepMeta(ids, positions, slots, state["slots"], self.max_model_len, cu_q=cu_q, max_q=max_q,
+                            tok_seq=state["token_seq"], start_pos=state["start_pos"], prefix=prefix)
+            return self._logits(self._forward_hybrid(meta)[last_index])
 
         def attend(li, qkv, lay):
             ops.kv_cache_write(qkv, lay, slots, cache.k[li], cache.v[li])
@@ -204,8 +259,13 @@ class ModelRunner:
         return self._logits(x[last_index])
 
     # ------------------------------------------------------------------------------------------
-    def _decode_eager(self, ids, positions, slots, block_tables, context_lens, max_context, groups=None):
+    def _decode_eager(self, ids, positions, slots, block_tables, context_lens, max_context, groups=None,
+                      state_slots=None):
         cache = self.cache
+        if self.cfg.is_hybrid:
+            meta = StepMeta(ids, positions, slots, state_slots, self.max_model_len, block_tables=block_tables,
+                            context_lens=context_lens, max_context=max_context)
+            return self._logits(self._forward_hybrid(meta))
 
         def attend(li, qkv, lay):
             ops.kv_cache_write(qkv, lay, slots, cache.k[li], cache.v[li])
@@ -225,6 +285,7 @@ class ModelRunner:
                       slots=torch.full((cap,), -1, dtype=torch.int64, device=dev),
                       block_tables=torch.zeros(cap, max_blocks, dtype=torch.int32, device=dev),
                       context_lens=torch.zeros(cap, dtype=torch.int32, device=dev),
+                      state_slots=torch.full((cap,), -1, dtype=torch.int64, device=dev),
                       key_start=torch.zeros(cap, dtype=torch.int32, device=dev),
                       group_rows=torch.full((cap, 8), -1, dtype=torch.int32, device=dev),
                       group_prefix=torch.zeros(cap, dtype=torch.int32, device=dev))
@@ -235,11 +296,12 @@ class ModelRunner:
     @torch.no_grad()
     def decode(self, ids: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor,
                block_tables: torch.Tensor, context_lens: torch.Tensor, max_context: int,
-               groups=None) -> torch.Tensor:
+               groups=None, state_slots: Optional[torch.Tensor] = None) -> torch.Tensor:
         """One token per sequence -> logits ``[B, V_local]``.  ``groups`` (see
         ``ops.paged_decode_attention``; an optional fourth entry gives the number of groups that have
         members, which come first in the tables) turns on shared-prefix attention for n-sample groups.
-        Shared prefixes must be multiples of ``self.prefix_tile`` keys when that is non-zero."""
+        Shared prefixes must be multiples of ``self.prefix_tile`` keys when that is non-zero.  ``state_slots``
+        ``[B]``: the recurrent-state slot of every sequence (hybrid decoders)."""
         b = ids.shape[0]
         bucket = next((s for s in self.graph_batch_sizes if s >= b), None)
         n_groups = b
@@ -251,7 +313,8 @@ class ModelRunner:
         if self.enforce_eager or bucket is None:
             if groups is not None:
                 groups = (groups[0], groups[1][:n_groups], groups[2][:n_groups])
-            return self._decode_eager(ids, positions, slots, block_tables, context_lens, max_context, groups)
+            return self._decode_eager(ids, positions, slots, block_tables, context_lens, max_context, groups,
+                                      state_slots)
         max_blocks = (self.max_model_len + self.cache.block_size - 1) // self.cache.block_size
         st = self._ensure_static(max_blocks)
         st["ids"][:b].copy_(ids)
@@ -261,6 +324,9 @@ class ModelRunner:
         st["context_lens"][:b].copy_(context_lens)
         st["context_lens"][b:bucket].zero_()
         st["block_tables"][:b, :block_tables.shape[1]].copy_(block_tables)
+        if state_slots is not None:
+            st["state_slots"][:b].copy_(state_slots)
+            st["state_slots"][b:bucket].fill_(-1)
         grouped = groups is not None
         if grouped:
             st["key_start"][:b].copy_(groups[0])
@@ -278,12 +344,17 @@ class ModelRunner:
     def _capture(self, bucket: int, st: dict, grouped: bool = False, n_groups: int = 0) -> dict:
         groups = (st["key_start"][:bucket], st["group_rows"][:n_groups], st["group_prefix"][:n_groups]) if grouped else None
         args = (st["ids"][:bucket], st["positions"][:bucket], st["slots"][:bucket],
-                st["block_tables"][:bucket], st["context_lens"][:bucket], self.max_model_len, groups)
+                st["block_tables"][:bucket], st["context_lens"][:bucket], self.max_model_len, groups,
+                st["state_slots"][:bucket])
+        # the warm-up runs the step for real: a recurrent state must not advance twice, so it sees no state slots
+        live = st["state_slots"].clone()
+        st["state_slots"].fill_(-1)
         side = torch.cuda.Stream()
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):       # warm-up: sizes scratch buffers outside the capture
             self._decode_eager(*args)
         torch.cuda.current_stream().wait_stream(side)
+        st["state_slots"].copy_(live)
         graph = torch.cuda.CUDAGraph()
         with torch.cuda.graph(graph):
             logits = self._decode_eager(*args)

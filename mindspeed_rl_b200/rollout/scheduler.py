@@ -7,6 +7,9 @@ KV cache runs out of blocks during decode, the most recently admitted sequence i
 its blocks are released and it re-enters the waiting queue with ``prompt + generated so far``
 as its new prompt (recompute policy).  A request that asks for ``n`` samples prefills its
 prompt once; the ``n`` sequences are forked from it and share the prompt's KV blocks.
+
+Models with recurrent layers also keep a state slot per running sequence (``StateSlots``): it is taken
+together with the blocks when a sequence is admitted or forked and returned with them.
 """
 from __future__ import annotations
 
@@ -78,6 +81,7 @@ class Sequence:
     mm_embeds: Optional[object] = None
     mm_positions: Optional[object] = None
     pos_delta: int = 0
+    state_slot: int = -1           # recurrent-state slot while the sequence runs (-1: none)
 
     @property
     def all_ids(self) -> List[int]:
@@ -128,8 +132,9 @@ class SchedulerOutput:
 
 class Scheduler:
     def __init__(self, block_manager: BlockManager, max_num_seqs: int, max_num_batched_tokens: int,
-                 max_model_len: int):
+                 max_model_len: int, state_slots=None):
         self.bm = block_manager
+        self.state_slots = state_slots
         self.max_num_seqs = max_num_seqs
         self.max_num_batched_tokens = max_num_batched_tokens
         self.max_model_len = max_model_len
@@ -171,6 +176,9 @@ class Scheduler:
         if seq.seq_id in self._allocated:
             self.bm.free(seq.seq_id)
             self._allocated.discard(seq.seq_id)
+        if seq.state_slot >= 0:
+            self.state_slots.free(seq.state_slot)
+            seq.state_slot = -1
 
     def finish(self, seq: Sequence, status: SeqStatus) -> None:
         seq.status = status
@@ -190,6 +198,20 @@ class Scheduler:
         g = self.groups.get(seq.request_id)
         return g.params.n if (g is not None and not g.forked) else 1
 
+    def admit(self, seq: Sequence) -> None:
+        """Reserve blocks for all tokens the sequence has (and a state slot) and put it among the running
+        ones.  Raises :class:`OutOfBlocks` with nothing changed when it does not fit right now."""
+        if self.state_slots is not None and self.state_slots.num_free < self._reserve_children(seq):
+            raise OutOfBlocks()
+        cached = self.bm.allocate(seq.seq_id, seq.all_ids)
+        self._allocated.add(seq.seq_id)
+        if self.state_slots is not None:
+            seq.state_slot = self.state_slots.allocate()
+        seq.status = SeqStatus.RUNNING
+        seq.num_computed = cached
+        seq.prefill_target = seq.total_len
+        self.running.append(seq)
+
     def schedule(self) -> SchedulerOutput:
         """Pick the work of the next engine step.
 
@@ -205,7 +227,8 @@ class Scheduler:
                 n = min(budget, s.prefill_target - s.num_computed)
                 out.prefill.append(PrefillItem(s, s.num_computed, n))
                 budget -= n
-        slots_left = self.max_num_seqs - len(self.running)
+        # a prompt still in prefill will fork into its n samples: their places are taken already
+        slots_left = self.max_num_seqs - sum(self._reserve_children(s) for s in self.running)
         while self.waiting and budget > 0:
             s = self.waiting[0]
             need_seqs = self._reserve_children(s)
@@ -218,15 +241,10 @@ class Scheduler:
                     self.groups[s.request_id].forked = True
                 continue
             try:
-                cached = self.bm.allocate(s.seq_id, s.all_ids)
+                self.admit(s)
             except OutOfBlocks:
                 break
-            self._allocated.add(s.seq_id)
             self.waiting.popleft()
-            s.status = SeqStatus.RUNNING
-            s.num_computed = cached
-            s.prefill_target = s.total_len
-            self.running.append(s)
             slots_left -= need_seqs
             n = min(budget, s.prefill_target - s.num_computed)
             out.prefill.append(PrefillItem(s, s.num_computed, n))
@@ -272,6 +290,8 @@ class Scheduler:
             child.num_computed = lead.num_computed
             pair = self.bm.fork(lead.seq_id, child.seq_id)
             self._allocated.add(child.seq_id)
+            if self.state_slots is not None:
+                child.state_slot = self.state_slots.allocate()
             g.seqs.append(child)
             self.running.append(child)
             created.append((child, pair))
