@@ -35,6 +35,18 @@ PRECISE = {"residual_stream", "delta_rule", "latent_attention", "grouped_gemm_si
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 
+# kernels of one use (hybrid: the forward of layer-by-layer decoders, without the sampler), linked into a library of their own (``_C/libmsrl_<group>.so``): a process that serves one model
+# family from a fresh checkout compiles these and nothing else
+GROUPS = {
+    "hybrid": ("residual_stream", "delta_rule", "latent_attention", "grouped_gemm_simt", "moe", "moe_gemm_tcgen05",
+               "attention", "attention_tcgen05", "gemm2cta_tcgen05"),
+}
+
+
+def group_path(name: str) -> Path:
+    return OUT_DIR / f"libmsrl_{name}.so"
+
+
 def _nvcc() -> str:
     cand = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
     if not os.path.exists(cand):
@@ -69,35 +81,58 @@ def sources() -> List[Path]:
     return sorted(CSRC.glob("*.cu")) + sorted(CSRC.glob("*.cpp"))
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
+def _stale(lib: Path, deps: List[Path], force: bool = False) -> bool:
+    return force or not lib.exists() or any(o.stat().st_mtime > lib.stat().st_mtime for o in deps)
+
+
+def _link(lib: Path, objs: List[Path], cuda: bool) -> None:
+    # linked beside its place and moved there: a process that finds the library finds a whole one
+    tmp = lib.with_name(f"{lib.name}.{os.getpid()}")
+    if cuda:
+        cmd = [_nvcc(), "-shared", "-o", str(tmp), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a",
+               "-cudart", "static", "-Xcompiler", "-fPIC", "-Xlinker", "-z,noexecstack"]
+    else:
+        cmd = ["g++", "-shared", "-o", str(tmp), *map(str, objs), "-pthread"]
+    res = subprocess.run(cmd, capture_output=True, text=True)
+    if res.returncode != 0:
+        raise RuntimeError(f"link of {lib.name} failed:\n{res.stdout}\n{res.stderr}")
+    os.replace(tmp, lib)
+
+
+def _compile_all(srcs: List[Path], force: bool) -> List[Path]:
     OBJ_DIR.mkdir(parents=True, exist_ok=True)
     log_dir = OUT_DIR / "logs"
     log_dir.mkdir(exist_ok=True)
-    srcs = sources()
     with cf.ThreadPoolExecutor(max_workers=min(8, len(srcs) or 1)) as pool:
-        objs = list(pool.map(lambda s: _compile_one(s, force, log_dir), srcs))
+        return list(pool.map(lambda s: _compile_one(s, force, log_dir), srcs))
+
+
+def build_group(name: str) -> Path:
+    """Compile and link one group's kernels and the host-only library."""
+    cu = [CSRC / f"{stem}.cu" for stem in GROUPS[name]]
+    host = sorted(CSRC.glob("*.cpp"))
+    objs = _compile_all(cu + host, force=False)
+    lib = group_path(name)
+    if _stale(lib, objs[:len(cu)]):
+        _link(lib, objs[:len(cu)], cuda=True)
+    if host and _stale(HOST_LIB_PATH, objs[len(cu):]):
+        _link(HOST_LIB_PATH, objs[len(cu):], cuda=False)
+    return lib
+
+
+def build(force: bool = False, verbose: bool = False) -> Path:
+    srcs = sources()
+    objs = _compile_all(srcs, force)
     cu_objs = [o for s, o in zip(srcs, objs) if s.suffix == ".cu"]
     host_objs = [o for s, o in zip(srcs, objs) if s.suffix == ".cpp"]
-
-    def stale(lib, deps):
-        return force or not lib.exists() or any(o.stat().st_mtime > lib.stat().st_mtime for o in deps)
-
-    if cu_objs and stale(LIB_PATH, cu_objs):
-        cmd = [_nvcc(), "-shared", "-o", str(LIB_PATH), *map(str, cu_objs),
-               "-gencode", "arch=compute_100a,code=sm_100a", "-cudart", "static", "-Xcompiler", "-fPIC",
-               "-Xlinker", "-z,noexecstack"]
-        res = subprocess.run(cmd, capture_output=True, text=True)
-        if res.returncode != 0:
-            raise RuntimeError(f"link failed:\n{res.stdout}\n{res.stderr}")
-    if host_objs and stale(HOST_LIB_PATH, host_objs):
+    if cu_objs and _stale(LIB_PATH, cu_objs, force):
+        _link(LIB_PATH, cu_objs, cuda=True)
+    if host_objs and _stale(HOST_LIB_PATH, host_objs, force):
         # host-only runtime pieces (block manager, ...) load on machines without CUDA
-        cmd = ["g++", "-shared", "-o", str(HOST_LIB_PATH), *map(str, host_objs), "-pthread"]
-        res = subprocess.run(cmd, capture_output=True, text=True)
-        if res.returncode != 0:
-            raise RuntimeError(f"host link failed:\n{res.stdout}\n{res.stderr}")
+        _link(HOST_LIB_PATH, host_objs, cuda=False)
     if verbose:
         for s in srcs:
-            log = log_dir / (s.stem + ".log")
+            log = OUT_DIR / "logs" / (s.stem + ".log")
             if log.exists():
                 sys.stdout.write(f"== {s.name}\n{log.read_text()}\n")
     return LIB_PATH

@@ -43,6 +43,21 @@ def load() -> ctypes.CDLL:
     return _lib
 
 
+def use_group(name: str) -> None:
+    """Serve this process from the kernels of one group (``csrc.build.GROUPS``), compiling what is missing.  The
+    full library is preferred where it has been built from the present sources."""
+    global _LIB_PATH
+    from ..csrc import build as _build
+
+    newest = max(p.stat().st_mtime for p in _build.CSRC.iterdir() if p.suffix in (".cu", ".cuh", ".h"))
+    if _LIB_PATH.exists() and _LIB_PATH.stat().st_mtime >= newest and _build.HOST_LIB_PATH.exists():
+        return
+    path = _build.build_group(name)
+    if _lib is not None:
+        raise RuntimeError("the kernel library is loaded already")
+    _LIB_PATH = path
+
+
 def available() -> bool:
     return _LIB_PATH.exists()
 
