@@ -35,8 +35,9 @@ PRECISE = {"residual_stream", "delta_rule", "latent_attention", "grouped_gemm_si
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 
-# kernels of one use (hybrid: the forward of layer-by-layer decoders, without the sampler), linked into a library of their own (``_C/libmsrl_<group>.so``): a process that serves one model
-# family from a fresh checkout compiles these and nothing else
+# kernels of one use, linked into a library of their own (``_C/libmsrl_<group>.so``): a process that serves one
+# model family from a fresh checkout compiles these and nothing else.  hybrid: the forward of layer-by-layer decoders
+# (without the sampler)
 GROUPS = {
     "hybrid": ("residual_stream", "delta_rule", "latent_attention", "grouped_gemm_simt", "moe", "moe_gemm_tcgen05",
                "attention", "attention_tcgen05", "gemm2cta_tcgen05"),
