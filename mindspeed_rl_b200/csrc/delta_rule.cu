@@ -41,18 +41,36 @@ struct DeltaIn {
 };
 
 // silu of the short convolution for one channel: `col` is its column in proj, `ch` its ring / weight row,
-// `i` the token's index inside this portion (row t of proj), `pos` its position in the sequence
-template <typename T>
+// `i` the token's index inside this portion (row t of proj), `pos` its position in the sequence.  TAPS > 0 fixes
+// the number of taps so that all loads are in flight together.
+template <int TAPS, typename T>
 __device__ __forceinline__ float conv_silu(const DeltaIn<T>& p, long long t, int i, int pos, long long slot, int col,
                                            int ch) {
   const int channels = 2 * p.KVH * p.dim + p.H * p.vdim;
+  const int taps = TAPS > 0 ? TAPS : p.taps;
+  const T* ring = p.ring + slot * taps * channels + ch;
   float s = 0.f;
-  for (int j = 0; j < p.taps; ++j) {
-    const int back = p.taps - 1 - j;
-    if (pos - back < 0) continue;
-    const float x = i - back >= 0 ? ldf(p.proj + (t - back) * p.ld + col)
-                                  : ldf(p.ring + (slot * p.taps + (pos - back) % p.taps) * channels + ch);
-    s += x * p.conv[(long long)ch * p.taps + j];
+  if constexpr (TAPS > 0) {
+    float x[TAPS], w[TAPS];
+    const int at = pos % TAPS;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      const int back = TAPS - 1 - j;
+      const int entry = at - back < 0 ? at - back + TAPS : at - back;
+      x[j] = 0.f;
+      if (pos - back >= 0)
+        x[j] = ldf(i - back >= 0 ? p.proj + (t - back) * p.ld + col : ring + (long long)entry * channels);
+      w[j] = p.conv[(long long)ch * TAPS + j];
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) s += x[j] * w[j];
+  } else {
+    for (int j = 0; j < taps; ++j) {
+      const int back = taps - 1 - j;
+      if (pos - back < 0) continue;
+      s += ldf(i - back >= 0 ? p.proj + (t - back) * p.ld + col : ring + (long long)((pos - back) % taps) * channels) *
+           p.conv[(long long)ch * taps + j];
+    }
   }
   return s * sigmoid_f(s);
 }
@@ -80,8 +98,8 @@ delta_prep_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const i
       const int d = n * 32 + lane;
       if (d < p.dim) {
         const int ch = hk * p.dim + d;
-        q[n] = conv_silu(p, t, i, pos, slot, p.q_col + ch, ch);
-        k[n] = conv_silu(p, t, i, pos, slot, p.k_col + ch, kd + ch);
+        q[n] = conv_silu<0>(p, t, i, pos, slot, p.q_col + ch, ch);
+        k[n] = conv_silu<0>(p, t, i, pos, slot, p.k_col + ch, kd + ch);
         qq += q[n] * q[n];
         kk += k[n] * k[n];
         qk += q[n] * k[n];
@@ -100,11 +118,151 @@ delta_prep_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const i
     if (lane == 0) kq[t * p.KVH + hk] = qk;
   }
   const int nv = p.H * p.vdim;
-  for (int c = threadIdx.x; c < nv; c += 256) vv[t * nv + c] = conv_silu(p, t, i, pos, slot, p.v_col + c, 2 * kd + c);
+  for (int c = threadIdx.x; c < nv; c += 256) vv[t * nv + c] = conv_silu<0>(p, t, i, pos, slot, p.v_col + c, 2 * kd + c);
   const int ng = p.H * p.dim;
   for (int c = threadIdx.x; c < ng; c += 256)
     g[t * ng + c] = expf(-expf(p.a_log[c / p.dim]) * softplus_f(ldf(p.a + t * p.a_ld + c) + p.dt_bias[c]));
   for (int h = threadIdx.x; h < p.H; h += 256) beta[t * p.H + h] = sigmoid_f(ldf(p.proj + t * p.ld + p.b_col + h));
+}
+
+// The same for the usual shapes (dim a multiple of 4 up to 128, vdim a multiple of 4, up to 4 taps): a warp walks
+// PREP_TT consecutive tokens with the convolution window of its channels in registers, four channels per lane, so
+// that every projection is read once.  Warps: one per key head (q and k), then 128 v channels or 128 decay channels.
+constexpr int PREP_TT = 16;
+
+template <int TAPS, typename T>
+struct ConvWindow {
+  float w[TAPS][4], x[TAPS][4];
+  const T* src;
+  __device__ __forceinline__ void weights(const float* conv, int ch) {
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) w[j][c] = conv[(long long)(ch + c) * TAPS + j];
+  }
+  // window entries before token t (index i of its portion, position pos); x[TAPS - 1] is the token's own
+  __device__ __forceinline__ void fill(const DeltaIn<T>& p, long long t, int i, int pos, long long slot, int col, int ch) {
+    const int channels = 2 * p.KVH * p.dim + p.H * p.vdim;
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j) {
+      const int back = TAPS - 1 - j;            // shifted once more before use: entry j + 1 holds position pos - back
+#pragma unroll
+      for (int c = 0; c < 4; ++c) x[j + 1][c] = 0.f;
+      if (pos - back >= 0) {
+        if (i - back >= 0) ldf4(p.proj + (t - back) * p.ld + col, x[j + 1]);
+        else ldf4(p.ring + (slot * TAPS + (pos - back) % TAPS) * channels + ch, x[j + 1]);
+      }
+    }
+  }
+  __device__ __forceinline__ void step(const T* row, float (&y)[4]) {
+#pragma unroll
+    for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) x[j][c] = x[j + 1][c];
+    ldf4(row, x[TAPS - 1]);
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      float s = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) s += x[j][c] * w[j][c];
+      y[c] = s * sigmoid_f(s);
+    }
+  }
+};
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256)
+delta_prep_fast_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const int* start_pos,
+                       const long long* slots, int tokens, float* qn, float* kn, float* kq, float* vv, float* g,
+                       float* beta) {
+  const int lane = threadIdx.x & 31;
+  const int unit = blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int kd = p.KVH * p.dim, nv = p.H * p.vdim, ng = p.H * p.dim;
+  const int uv = (nv + 127) / 128, ug = (ng + 127) / 128;
+  const int t0 = blockIdx.y * PREP_TT, t1 = min(tokens, t0 + PREP_TT);
+  if (unit < p.KVH) {
+    const int d = lane * 4, ch = unit * p.dim + d;
+    const bool on = d < p.dim;
+    const float qscale = 1.f / sqrtf((float)p.dim);
+    ConvWindow<TAPS, T> cq, ck;
+    if (on) {
+      cq.weights(p.conv, ch);
+      ck.weights(p.conv, kd + ch);
+    }
+    int seq = -1;
+    for (int t = t0; t < t1; ++t) {
+      const int b = tok_seq[t];
+      if (b != seq) {
+        seq = b;
+        const int i = t - cu[b], pos = start_pos[b] + i;
+        if (on) {
+          cq.fill(p, t, i, pos, slots[b], p.q_col + ch, ch);
+          ck.fill(p, t, i, pos, slots[b], p.k_col + ch, kd + ch);
+        }
+      }
+      float q[4] = {0.f, 0.f, 0.f, 0.f}, k[4] = {0.f, 0.f, 0.f, 0.f};
+      if (on) {
+        cq.step(p.proj + t * p.ld + p.q_col + ch, q);
+        ck.step(p.proj + t * p.ld + p.k_col + ch, k);
+      }
+      float qq = 0.f, kk = 0.f, qk = 0.f;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        qq += q[c] * q[c];
+        kk += k[c] * k[c];
+        qk += q[c] * k[c];
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        qq += __shfl_xor_sync(0xffffffffu, qq, o);
+        kk += __shfl_xor_sync(0xffffffffu, kk, o);
+        qk += __shfl_xor_sync(0xffffffffu, qk, o);
+      }
+      const float qs = qscale / sqrtf(qq + p.unit_eps), ks = 1.f / sqrtf(kk + p.unit_eps);
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        q[c] *= qs;
+        k[c] *= ks;
+      }
+      if (on) {
+        stf4(qn + (long long)t * kd + ch, q);
+        stf4(kn + (long long)t * kd + ch, k);
+      }
+      if (lane == 0) kq[(long long)t * p.KVH + unit] = qk * qs * ks;
+    }
+  } else if (unit < p.KVH + uv) {
+    const int c = (unit - p.KVH) * 128 + lane * 4;
+    if (c >= nv) return;
+    ConvWindow<TAPS, T> cv;
+    cv.weights(p.conv, 2 * kd + c);
+    int seq = -1;
+    for (int t = t0; t < t1; ++t) {
+      const int b = tok_seq[t];
+      if (b != seq) {
+        seq = b;
+        const int i = t - cu[b];
+        cv.fill(p, t, i, start_pos[b] + i, slots[b], p.v_col + c, 2 * kd + c);
+      }
+      float y[4];
+      cv.step(p.proj + t * p.ld + p.v_col + c, y);
+      stf4(vv + (long long)t * nv + c, y);
+    }
+  } else if (unit < p.KVH + uv + ug) {
+    const int c = (unit - p.KVH - uv) * 128 + lane * 4;
+    if (c >= ng) return;
+    const float rate = -expf(p.a_log[c / p.dim]);            // dim is a multiple of 4: one head per lane
+    const float bias[4] = {p.dt_bias[c], p.dt_bias[c + 1], p.dt_bias[c + 2], p.dt_bias[c + 3]};
+    for (int t = t0; t < t1; ++t) {
+      float x[4];
+      ldf4(p.a + t * p.a_ld + c, x);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) x[j] = expf(rate * softplus_f(x[j] + bias[j]));
+      stf4(g + (long long)t * ng + c, x);
+    }
+  } else if (unit == p.KVH + uv + ug) {
+    for (int t = t0; t < t1; ++t)
+      for (int h = lane; h < p.H; h += 32) beta[(long long)t * p.H + h] = sigmoid_f(ldf(p.proj + t * p.ld + p.b_col + h));
+  }
 }
 
 // ---- prefill: the recurrence --------------------------------------------------------------------------
@@ -113,6 +271,29 @@ __device__ __forceinline__ void cp_async4(void* smem, const void* gmem) {
 }
 __device__ __forceinline__ void cp_async16b(void* smem, const void* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_u32(smem)), "l"(gmem));
+}
+
+// two fp32 lanes per instruction (each lane rounds like the scalar operation)
+using f2 = unsigned long long;
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
+  f2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
+  f2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ f2 pack2(float lo, float hi) {
+  f2 d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float2 unpack2(f2 a) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(a));
+  return r;
 }
 
 constexpr int SCAN_TB = 16;      // tokens staged at a time
@@ -139,12 +320,13 @@ delta_scan_kernel(const float* qn, const float* kn, const float* kq, const float
   float* Sg = state + ((slot * H + h) * dim) * (long long)vdim + col;
 
   for (int i = threadIdx.x; i < 2 * BUF; i += THREADS) sm[i] = 0.f;      // pad rows stay zero
-  float s[DPL];
+  f2 s[DPL / 2];
   const bool fresh = start_pos[b] == 0;
 #pragma unroll
-  for (int n = 0; n < DPL; ++n) {
+  for (int n = 0; n < DPL; n += 2) {
     const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
-    s[n] = (!fresh && on && r < dim) ? Sg[(long long)r * vdim] : 0.f;
+    const bool have = !fresh && on;
+    s[n / 2] = pack2(have && r < dim ? Sg[(long long)r * vdim] : 0.f, have && r + 1 < dim ? Sg[(long long)(r + 1) * vdim] : 0.f);
   }
   __syncthreads();
 
@@ -197,42 +379,48 @@ delta_scan_kernel(const float* qn, const float* kn, const float* kq, const float
     const int first = blk * SCAN_TB, n = min(SCAN_TB, len - first);
     const float* bv = buf + 3 * SCAN_TB * DP;
     const float* bb = bv + SCAN_TB * COLS;
+    auto rows = [&](int which, int tt) {
+      return reinterpret_cast<const ulonglong2*>(buf + (which * SCAN_TB + tt) * DP) + lr;
+    };
 #pragma unroll 2
     for (int tt = 0; tt < n; ++tt) {
-      const float4* q4 = reinterpret_cast<const float4*>(buf + tt * DP) + lr;
-      const float4* k4 = reinterpret_cast<const float4*>(buf + SCAN_TB * DP + tt * DP) + lr;
-      const float4* g4 = reinterpret_cast<const float4*>(buf + 2 * SCAN_TB * DP + tt * DP) + lr;
-      float pk[4] = {0.f, 0.f, 0.f, 0.f}, pq[4] = {0.f, 0.f, 0.f, 0.f};
+      const ulonglong2 *q4 = rows(0, tt), *k4 = rows(1, tt), *g4 = rows(2, tt);
+      const float bt = bb[tt], vt = bv[tt * COLS + col_l], kqt = bb[SCAN_TB + tt];
+      f2 kk[DPL / 2];
+      f2 pk[2] = {0ull, 0ull}, pq[2] = {0ull, 0ull};
 #pragma unroll
       for (int m = 0; m < DPL / 4; ++m) {
-        const float4 gg = g4[m * LPC], kk = k4[m * LPC], qq = q4[m * LPC];
-        s[4 * m + 0] *= gg.x; s[4 * m + 1] *= gg.y; s[4 * m + 2] *= gg.z; s[4 * m + 3] *= gg.w;
-        pk[0] += s[4 * m + 0] * kk.x; pk[1] += s[4 * m + 1] * kk.y;
-        pk[2] += s[4 * m + 2] * kk.z; pk[3] += s[4 * m + 3] * kk.w;
-        pq[0] += s[4 * m + 0] * qq.x; pq[1] += s[4 * m + 1] * qq.y;
-        pq[2] += s[4 * m + 2] * qq.z; pq[3] += s[4 * m + 3] * qq.w;
+        const ulonglong2 gg = g4[m * LPC], kv = k4[m * LPC], qq = q4[m * LPC];
+        kk[2 * m] = kv.x;
+        kk[2 * m + 1] = kv.y;
+        s[2 * m] = mul2(s[2 * m], gg.x);
+        s[2 * m + 1] = mul2(s[2 * m + 1], gg.y);
+        pk[0] = fma2(s[2 * m], kv.x, pk[0]);
+        pk[1] = fma2(s[2 * m + 1], kv.y, pk[1]);
+        pq[0] = fma2(s[2 * m], qq.x, pq[0]);
+        pq[1] = fma2(s[2 * m + 1], qq.y, pq[1]);
       }
-      float dk = (pk[0] + pk[1]) + (pk[2] + pk[3]), dq = (pq[0] + pq[1]) + (pq[2] + pq[3]);
+      const float2 k0 = unpack2(pk[0]), k1 = unpack2(pk[1]), q0 = unpack2(pq[0]), q1 = unpack2(pq[1]);
+      float dk = (k0.x + k0.y) + (k1.x + k1.y), dq = (q0.x + q0.y) + (q1.x + q1.y);
 #pragma unroll
       for (int x = LPC / 2; x > 0; x >>= 1) {
         dk += __shfl_xor_sync(0xffffffffu, dk, x);
         dq += __shfl_xor_sync(0xffffffffu, dq, x);
       }
-      const float u = bb[tt] * (bv[tt * COLS + col_l] - dk);
+      const float u = bt * (vt - dk);
+      const f2 uu = pack2(u, u);
 #pragma unroll
-      for (int m = 0; m < DPL / 4; ++m) {
-        const float4 kk = k4[m * LPC];
-        s[4 * m + 0] += kk.x * u; s[4 * m + 1] += kk.y * u;
-        s[4 * m + 2] += kk.z * u; s[4 * m + 3] += kk.w * u;
-      }
-      if (lr == 0 && on) o[((t0 + first + tt) * H + h) * vdim + col] = dq + bb[SCAN_TB + tt] * u;
+      for (int m = 0; m < DPL / 2; ++m) s[m] = fma2(kk[m], uu, s[m]);
+      if (lr == 0 && on) o[((t0 + first + tt) * H + h) * vdim + col] = dq + kqt * u;
     }
     __syncthreads();
   }
 #pragma unroll
-  for (int n = 0; n < DPL; ++n) {
+  for (int n = 0; n < DPL; n += 2) {
     const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
-    if (on && r < dim) Sg[(long long)r * vdim] = s[n];
+    const float2 v = unpack2(s[n / 2]);
+    if (on && r < dim) Sg[(long long)r * vdim] = v.x;
+    if (on && r + 1 < dim) Sg[(long long)(r + 1) * vdim] = v.y;
   }
 }
 
@@ -272,8 +460,8 @@ delta_out_kernel(const float* o, const T* gate, long long gate_ld, const float* 
 // ---- decode: one token per sequence, everything in one kernel -----------------------------------------------
 // block = (head, sequence).  Threads tile the state as [row groups RG][column groups of V]; a thread keeps its
 // NI row slices in registers between the decayed dot products and the rank-one update.
-template <typename T, int V, int NI, int THREADS>
-__global__ void __launch_bounds__(THREADS)
+template <typename T, int V, int NI, int THREADS, int TAPS>
+__global__ void __launch_bounds__(THREADS, NI * V <= 32 && THREADS == 512 ? 2 : 1)
 delta_decode_kernel(const DeltaIn<T> p, const T* gate, long long gate_ld, const float* norm, float eps,
                     const int* positions, const long long* slots, T* y) {
   extern __shared__ __align__(16) float sm[];
@@ -307,21 +495,17 @@ delta_decode_kernel(const DeltaIn<T> p, const T* gate, long long gate_ld, const 
   const bool lead = h % rep == 0;                // writes the key head's ring entries
   T* ring = p.ring + (slot * p.taps + pos % p.taps) * channels;
   const T* row = p.proj + (long long)b * p.ld;
-  for (int d = threadIdx.x; d < dim; d += THREADS) {
-    const int ch = hk * dim + d;
-    sq[d] = conv_silu(p, b, 0, pos, slot, p.q_col + ch, ch);
-    sk[d] = conv_silu(p, b, 0, pos, slot, p.k_col + ch, kd + ch);
+  // q | k | v channels of this head side by side, one per thread
+  for (int x = threadIdx.x; x < 2 * dim + vdim; x += THREADS) {
+    const int d = x < dim ? x : x < 2 * dim ? x - dim : x - 2 * dim;
+    const int ch = x < 2 * dim ? hk * dim + d : h * vdim + d;
+    const int base = x < dim ? 0 : x < 2 * dim ? kd : 2 * kd;
+    const int col = (x < dim ? p.q_col : x < 2 * dim ? p.k_col : p.v_col) + ch;
+    (x < dim ? sq : x < 2 * dim ? sk : sv)[d] = conv_silu<TAPS>(p, b, 0, pos, slot, col, base + ch);
+    if (lead || x >= 2 * dim) ring[base + ch] = row[col];
+  }
+  for (int d = threadIdx.x; d < dim; d += THREADS)
     sg[d] = expf(-expf(p.a_log[h]) * softplus_f(ldf(p.a + b * p.a_ld + h * dim + d) + p.dt_bias[h * dim + d]));
-    if (lead) {
-      ring[ch] = row[p.q_col + ch];
-      ring[kd + ch] = row[p.k_col + ch];
-    }
-  }
-  for (int c = threadIdx.x; c < vdim; c += THREADS) {
-    const int ch = h * vdim + c;
-    sv[c] = conv_silu(p, b, 0, pos, slot, p.v_col + ch, 2 * kd + ch);
-    ring[2 * kd + ch] = row[p.v_col + ch];
-  }
   __syncthreads();
   {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -461,12 +645,25 @@ MSRL_API int msrl_delta_prefill(const void* proj, long long ld, const void* a, l
   auto run = [&](auto tag) {
     using T = decltype(tag);
     const DeltaIn<T> p = delta_in<T>(proj, ld, a, a_ld, conv, a_log, dt_bias, ring, state, ints, unit_eps);
-    delta_prep_kernel<T><<<tokens, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, qn, kn, kq, vv, g, beta);
+    const bool usual = dim % 4 == 0 && dim <= 128 && vdim % 4 == 0 && p.q_col % 4 == 0 && p.k_col % 4 == 0 &&
+                       p.v_col % 4 == 0 && ld % 4 == 0 && a_ld % 4 == 0;
+    const int units = KVH + (H * vdim + 127) / 128 + (H * dim + 127) / 128 + 1;
+    const dim3 tiles((unsigned)((units + 7) / 8), (unsigned)((tokens + PREP_TT - 1) / PREP_TT));
+#define MSRL_PREP(N) delta_prep_fast_kernel<T, N><<<tiles, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, tokens, qn, kn, kq, vv, g, beta)
+    if (usual && p.taps == 4 && tiles.y <= 65535) MSRL_PREP(4);
+    else if (usual && p.taps == 3 && tiles.y <= 65535) MSRL_PREP(3);
+    else if (usual && p.taps == 2 && tiles.y <= 65535) MSRL_PREP(2);
+    else delta_prep_kernel<T><<<tokens, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, qn, kn, kq, vv, g, beta);
+#undef MSRL_PREP
+    // four lanes a column spend fewer instructions, eight hide a token's latency better when few blocks run
+    const bool many = (long long)batch * H * ((vdim + 31) / 32) >= 4LL * sm_count();
     int e;
-    if (dim <= 32) e = launch_scan<8, 4, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st);
-    else if (dim <= 64) e = launch_scan<16, 4, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st);
-    else if (dim <= 128) e = launch_scan<16, 8, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st);
-    else e = launch_scan<32, 8, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st);
+#define MSRL_SCAN(D, L) launch_scan<D, L, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st)
+    if (dim <= 32) e = MSRL_SCAN(8, 4);
+    else if (dim <= 64) e = many ? MSRL_SCAN(16, 4) : MSRL_SCAN(8, 8);
+    else if (dim <= 128) e = many ? MSRL_SCAN(32, 4) : MSRL_SCAN(16, 8);
+    else e = MSRL_SCAN(32, 8);
+#undef MSRL_SCAN
     if (e) return e;
     const int channels = 2 * KVH * dim + H * vdim;
     delta_ring_kernel<T><<<dim3((unsigned)((channels + 255) / 256), (unsigned)batch), 256, 0, st>>>(p, cu, start_pos, slots);
@@ -477,22 +674,36 @@ MSRL_API int msrl_delta_prefill(const void* proj, long long ld, const void* a, l
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
-template <typename T, int V, int NI, int THREADS>
-static int launch_delta_decode(const DeltaIn<T>& p, const T* gate, long long gate_ld, const float* norm, float eps,
+template <typename T, int V, int NI, int THREADS, int TAPS>
+static int launch_delta_decode_taps(const DeltaIn<T>& p, const T* gate, long long gate_ld, const float* norm, float eps,
                                const int* positions, const long long* slots, T* y, int batch, cudaStream_t st) {
   const int rg = THREADS / (p.vdim / V);
   const size_t smem = sizeof(float) * (3 * (size_t)p.dim + 3 * (size_t)p.vdim + 2 * (size_t)rg * p.vdim);
-  const int e = allow_smem(delta_decode_kernel<T, V, NI, THREADS>, smem);
+  const int e = allow_smem(delta_decode_kernel<T, V, NI, THREADS, TAPS>, smem);
   if (e) return e;
-  delta_decode_kernel<T, V, NI, THREADS><<<dim3((unsigned)p.H, (unsigned)batch), THREADS, smem, st>>>(
+  delta_decode_kernel<T, V, NI, THREADS, TAPS><<<dim3((unsigned)p.H, (unsigned)batch), THREADS, smem, st>>>(
       p, gate, gate_ld, norm, eps, positions, slots, y);
   return (int)cudaGetLastError();
+}
+
+template <typename T, int V, int NI, int THREADS>
+static int launch_delta_decode(const DeltaIn<T>& p, const T* gate, long long gate_ld, const float* norm, float eps,
+                               const int* positions, const long long* slots, T* y, int batch, cudaStream_t st) {
+  if constexpr (V == 4 && NI <= 8) {
+    if (p.taps == 4)
+      return launch_delta_decode_taps<T, V, NI, THREADS, 4>(p, gate, gate_ld, norm, eps, positions, slots, y, batch, st);
+    if (p.taps == 3)
+      return launch_delta_decode_taps<T, V, NI, THREADS, 3>(p, gate, gate_ld, norm, eps, positions, slots, y, batch, st);
+    if (p.taps == 2)
+      return launch_delta_decode_taps<T, V, NI, THREADS, 2>(p, gate, gate_ld, norm, eps, positions, slots, y, batch, st);
+  }
+  return launch_delta_decode_taps<T, V, NI, THREADS, 0>(p, gate, gate_ld, norm, eps, positions, slots, y, batch, st);
 }
 
 template <typename T, int V>
 static int pick_delta_decode(const DeltaIn<T>& p, const T* gate, long long gate_ld, const float* norm, float eps,
                              const int* positions, const long long* slots, T* y, int batch, cudaStream_t st) {
-  // rows per thread for a block size: the smallest block that keeps at most 16 row slices per thread
+  // the smallest block that keeps few row slices per thread: registers for two blocks of 512 threads on an SM
   auto slices = [&](int threads) {
     const int rg = threads / (p.vdim / V);
     return rg == 0 ? 1 << 20 : (p.dim + rg - 1) / rg;
@@ -502,8 +713,9 @@ static int pick_delta_decode(const DeltaIn<T>& p, const T* gate, long long gate_
     return launch_delta_decode<T, V, NI, THREADS>(p, gate, gate_ld, norm, eps, positions, slots, y, batch, st);
   MSRL_TRY(4, 128)
   MSRL_TRY(4, 256)
-  MSRL_TRY(16, 128)
-  MSRL_TRY(16, 256)
+  MSRL_TRY(8, 128)
+  MSRL_TRY(8, 256)
+  MSRL_TRY(8, 512)
   MSRL_TRY(16, 512)
   MSRL_TRY(16, 1024)
   MSRL_TRY(64, 512)

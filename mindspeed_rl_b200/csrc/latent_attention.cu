@@ -107,6 +107,16 @@ template <typename T>
 __global__ void spread_kernel(const T* lat, int CP, int RP, T* kv, long long ld, int H, int stride, int dn, int dr,
                               long long tokens) {
   const long long t = blockIdx.x;
+  if (dr % 4 == 0 && dn % 4 == 0 && stride % 4 == 0 && ld % 4 == 0) {
+    const int quads = dr / 4;
+    for (int i = threadIdx.x; i < H * quads; i += blockDim.x) {
+      const int h = i / quads, d = (i - h * quads) * 4;
+      float x[4];
+      ldf4(lat + t * CP + RP + d, x);
+      stf4(kv + t * ld + h * stride + dn + d, x);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < H * dr; i += blockDim.x)
     kv[t * ld + (i / dr) * stride + dn + i % dr] = lat[t * CP + RP + i % dr];
 }
@@ -310,14 +320,18 @@ __global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
   const int vecs = p.CP / 8;
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
 
-  auto load_tile = [&](int tile, int buf) {
+  // cache row of the key that lane l of a warp looks up for its warp's row l (rows warp, warp + 8, ...); -1: none
+  auto look_up = [&](int tile) -> int {
+    const int key = tile * KT + warp + 8 * lane;
+    return lane < KT / 8 && key < n ? bt[key / p.block_size] * p.block_size + key % p.block_size : -1;
+  };
+  auto load_tile = [&](int slots_of_lane, int buf) {
     __nv_bfloat16* dst = sKV + buf * KT * ld;
-    for (int r = warp; r < KT; r += 8) {
-      const int key = tile * KT + r;
-      const bool ok = key < n;
-      const long long slot = ok ? (long long)bt[key / p.block_size] * p.block_size + key % p.block_size : 0;
-      const __nv_bfloat16* src = p.cache + slot * p.CP;
-      for (int c = lane; c < vecs; c += 32) cp_async16(dst + r * ld + c * 8, src + c * 8, ok);
+#pragma unroll
+    for (int i = 0; i < KT / 8; ++i) {
+      const int slot = __shfl_sync(0xffffffffu, slots_of_lane, i);
+      const __nv_bfloat16* src = p.cache + (long long)max(slot, 0) * p.CP;
+      for (int c = lane; c < vecs; c += 32) cp_async16(dst + (warp + 8 * i) * ld + c * 8, src + c * 8, slot >= 0);
     }
     cp_async_commit();
   };
@@ -340,12 +354,14 @@ __global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
       const __nv_bfloat16* src = p.q + ((long long)b * p.H + (ok ? h0 + r : 0)) * p.CP;
       for (int c = lane; c < vecs; c += 32) cp_async16(sQ + r * ld + c * 8, src + c * 8, ok);
     }
-    load_tile(first, 0);
+    load_tile(look_up(first), 0);
   }
+  int ahead = first + 1 < last ? look_up(first + 1) : -1;          // rows of the tile that is loaded next
   for (int tile = first; tile < last; ++tile) {
     const int buf = (tile - first) & 1;
     if (tile + 1 < last) {
-      load_tile(tile + 1, buf ^ 1);
+      load_tile(ahead, buf ^ 1);
+      if (tile + 2 < last) ahead = look_up(tile + 2);
       cp_async_wait<1>();
     } else {
       cp_async_wait<0>();
@@ -353,21 +369,20 @@ __global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
     __syncthreads();
     const __nv_bfloat16* kv = sKV + buf * KT * ld;
     // scores of 16 heads x 8 * NK8 keys per warp
-    float s[NK8][4];
+    float s[NK8][4], s2[NK8][4];                                   // even and odd steps of the reduction
 #pragma unroll
     for (int i = 0; i < NK8; ++i)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+      for (int j = 0; j < 4; ++j) s[i][j] = s2[i][j] = 0.f;
     const int key0 = wk * NK8 * 8;
-#pragma unroll 4
-    for (int kk = 0; kk < p.CP / 16; ++kk) {
+    auto k_step = [&](int kk, float (&acc)[NK8][4]) {
       uint32_t a[4];
       ldmatrix_x4(a, smem_u32(sQ + (wm * 16 + (lane & 15)) * ld + kk * 16 + (lane >> 4) * 8));
       if constexpr (NK8 == 2) {
         uint32_t f[4];
         ldmatrix_x4(f, smem_u32(kv + (key0 + (lane & 7) + (lane >> 4) * 8) * ld + kk * 16 + ((lane >> 3) & 1) * 8));
-        mma_16816(s[0], a, f[0], f[1]);
-        mma_16816(s[1], a, f[2], f[3]);
+        mma_16816(acc[0], a, f[0], f[1]);
+        mma_16816(acc[1], a, f[2], f[3]);
       } else {
 #pragma unroll
         for (int i = 0; i < NK8; ++i) {
@@ -375,10 +390,22 @@ __global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
           asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n"
                        : "=r"(f[0]), "=r"(f[1])
                        : "r"(smem_u32(kv + (key0 + i * 8 + (lane & 7)) * ld + kk * 16 + ((lane >> 3) & 1) * 8)));
-          mma_16816(s[i], a, f[0], f[1]);
+          mma_16816(acc[i], a, f[0], f[1]);
         }
       }
+    };
+    const int steps = p.CP / 16;
+    int kk = 0;
+#pragma unroll 2
+    for (; kk + 1 < steps; kk += 2) {
+      k_step(kk, s);
+      k_step(kk + 1, s2);
     }
+    if (kk < steps) k_step(kk, s);
+#pragma unroll
+    for (int i = 0; i < NK8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) s[i][j] += s2[i][j];
 #pragma unroll
     for (int i = 0; i < NK8; ++i) {
       float* d = sS + (wm * 16 + (lane >> 2)) * LDS_S + key0 + i * 8 + (lane & 3) * 2;

@@ -385,6 +385,9 @@ def main():
     ap.add_argument("--small", action="store_true")
     ap.add_argument("--iters", type=int, default=10)
     args = ap.parse_args()
+    from .microbench_hybrid import CASES as hybrid
+
+    CASES.update(hybrid)
     names = [n for n in args.only.split(",") if n] or list(CASES)
     for n in names:
         CASES[n](args.small, args.iters)

@@ -1,0 +1,122 @@
+"""Micro-benchmark cases of the layer-by-layer decoders' kernels, at the layer sizes of a model of some ten billion
+parameters (32 heads of 128, latent rank 512, width 2304).  Run through ``ops.microbench --only hybrid_*``.
+
+Roofline of the recurrence: its state arithmetic is fp32 on the CUDA cores (4 multiply-adds per state entry and
+token), counted against 128 fp32 multiply-adds per SM and clock at the maximum clock.
+"""
+from __future__ import annotations
+
+import torch
+
+from . import (DeltaLayout, DeltaWeights, LatentLayout, add_norm_, delta_decode, delta_prefill, embed_norm, glu_fwd,
+               latent_decode_attention, latent_prefill_attention, latent_prep, latent_spread_, moe_combine_norm_, rope_table)
+from . import moe as K
+from .microbench import report, timeit
+
+
+def fp32_tflops() -> float:
+    p = torch.cuda.get_device_properties(0)
+    clock = getattr(p, "clock_rate", 1965000) * 1e3
+    return p.multi_processor_count * 128 * 2 * clock / 1e12
+
+
+def _delta(t, heads=32, dim=128, vdim=128, taps=4):
+    kd, hv = heads * dim, heads * vdim
+    lay = DeltaLayout(heads, heads, dim, vdim, taps, 0, kd, 2 * kd, 2 * kd + hv)
+    proj = torch.randn(t, 2 * kd + hv + heads + 256, device="cuda").bfloat16()
+    a, gate = torch.randn(t, kd, device="cuda").bfloat16(), torch.randn(t, hv, device="cuda").bfloat16()
+    w = DeltaWeights(torch.randn(lay.channels, taps, device="cuda"), torch.zeros(heads, device="cuda") - 2,
+                     torch.zeros(kd, device="cuda"), torch.ones(vdim, device="cuda"))
+    return lay, proj, a, gate, w
+
+
+def case_delta(small: bool, iters: int):
+    for b, n in ([(1, 2048)] if small else [(1, 8192), (8, 1024), (32, 256)]):
+        t = b * n
+        lay, proj, a, gate, w = _delta(t)
+        ring = torch.zeros(b, lay.taps, lay.channels, device="cuda").bfloat16()
+        state = torch.zeros(b, lay.heads, lay.dim, lay.vdim, device="cuda")
+        cu = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda")
+        seq = torch.arange(b, dtype=torch.int32, device="cuda").repeat_interleave(n)
+        start, slots = torch.zeros(b, dtype=torch.int32, device="cuda"), torch.arange(b, device="cuda")
+        ms = timeit(lambda: delta_prefill(proj, a, gate, lay, w, ring, state, seq, cu, start, slots, 1e-5), iters)
+        fma = 4.0 * t * lay.heads * lay.dim * lay.vdim
+        report(f"delta_prefill {b}x{n} heads=32 dim=128", ms, bytes_=2.0 * t * (lay.channels + 3 * lay.heads * lay.vdim),
+               note=f"{2 * fma / ms / 1e9:.1f} TFLOP/s fp32 = {2 * fma / ms / 1e9 / fp32_tflops():.3f} of nominal fp32")
+    for b in ([32] if small else [1, 32, 256]):
+        lay, proj, a, gate, w = _delta(b)
+        ring = torch.zeros(b, lay.taps, lay.channels, device="cuda").bfloat16()
+        state = torch.zeros(b, lay.heads, lay.dim, lay.vdim, device="cuda")
+        pos = torch.full((b,), 100, dtype=torch.int32, device="cuda")
+        slots = torch.randperm(b, device="cuda")
+        ms = timeit(lambda: delta_decode(proj, a, gate, lay, w, ring, state, pos, slots, 1e-5), iters)
+        report(f"delta_decode B={b} heads=32 dim=128", ms, bytes_=2.0 * state.numel() * 4 + b * lay.channels * 2 * 8)
+
+
+def case_latent(small: bool, iters: int):
+    for heads in (16, 32, 64, 128):
+        lay = LatentLayout(heads, 64, 64, 128, 512, 128, 128, heads * 128, 64)
+        for b, ctx in ([(16, 1024)] if small else [(256, 2048), (32, 2048), (1, 8192)]):
+            nb = b * ctx // 16
+            cache = torch.randn(nb, 16, lay.CP, device="cuda").bfloat16()
+            bt = torch.randperm(nb, device="cuda").to(torch.int32).view(b, -1)
+            cl = torch.full((b,), ctx, dtype=torch.int32, device="cuda")
+            q = torch.randn(b, heads, lay.CP, device="cuda").bfloat16()
+            ms = timeit(lambda: latent_decode_attention(q, cache, lay, bt, cl, ctx, 0.05), iters)
+            report(f"latent_decode H={heads} B={b} ctx={ctx}", ms, bytes_=2.0 * b * ctx * lay.CP,
+                   flops=2.0 * b * ctx * heads * (lay.CP + lay.RP))
+    heads, t, n = 32, (2048 if small else 16384), 2048
+    for dn, dr, dv, p in ((64, 64, 128, 128), (128, 64, 128, 192)):
+        lay = LatentLayout(heads, dn, dr, dv, 512, p, 128, heads * p, dr)
+        proj = torch.randn(t, heads * p + 576, device="cuda").bfloat16()
+        kv = torch.randn(t, heads * (p + 128), device="cuda").bfloat16()
+        cu = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda")
+        ms = timeit(lambda: latent_prefill_attention(proj, kv, lay, cu, cu, n, 0.08), iters)
+        report(f"latent_prefill_attention {t // n}x{n} H=32 qk={dn + dr} v={dv}", ms,
+               flops=2.0 * t * (n / 2) * heads * (dn + dr + dv))
+        pos = torch.arange(t, dtype=torch.int32, device="cuda") % n
+        slots = torch.arange(t, device="cuda")
+        cache = torch.empty(t // 16, 16, lay.CP, device="cuda").bfloat16()
+        tab = rope_table(4096, dr, 1e4, proj.device)
+        nw = torch.ones(512, device="cuda")
+        ms = timeit(lambda: latent_prep(proj, lay, nw, 1e-5, tab, pos, slots, cache, True), iters)
+        report(f"latent_prep T={t} H=32 rot={dr}", ms, bytes_=2.0 * t * (2 * heads * dr + 3 * lay.CP))
+        rows = torch.randn(t, lay.CP, device="cuda").bfloat16()
+        ms = timeit(lambda: latent_spread_(kv, rows, lay), iters)
+        report(f"latent_spread T={t} H=32 rot={dr}", ms, bytes_=2.0 * t * (heads * dr + dr))
+
+
+def case_stream(small: bool, iters: int):
+    t, h, f = (4096, 2304, 4096) if small else (16384, 3584, 18944)
+    resid, w = torch.zeros(t, h, device="cuda"), torch.zeros(h, device="cuda")
+    x = torch.randn(t, h, device="cuda").bfloat16()
+    ms = timeit(lambda: add_norm_(resid, x, w, 1e-5, 1.0), iters)
+    report(f"add_norm {t}x{h} (fp32 residual)", ms, bytes_=t * h * 12.0)
+    table, ids = torch.randn(32768, h, device="cuda").bfloat16(), torch.randint(0, 32768, (t,), device="cuda")
+    ms = timeit(lambda: embed_norm(ids, table, 1.0, w, 1e-5, 1.0), iters)
+    report(f"embed_norm {t}x{h}", ms, bytes_=t * h * 8.0)
+    for act in ("gelu_tanh", "clamped_swish"):
+        gu = torch.randn(t, 2 * f, device="cuda").bfloat16()
+        ms = timeit(lambda: glu_fwd(gu, act, 7.0, 1.702), iters)
+        report(f"glu {act} {t}x{f}", ms, bytes_=6.0 * t * f)
+        del gu
+    e, k, h, f = 64, 8, 2304, 1024
+    for t in ([2048] if small else [16384, 256]):
+        x = torch.randn(t, h, device="cuda").bfloat16()
+        idx = torch.stack([torch.randperm(e, device="cuda")[:k] for _ in range(256)]).repeat((t + 255) // 256, 1)[:t]
+        plan = K.moe_plan(idx, e)
+        w1, w2 = (torch.randn(e, n, c, device="cuda").bfloat16() for n, c in ((2 * f, h), (h, f)))
+        xp = K.moe_permute(x, plan)
+        ms = timeit(lambda: K.grouped_gemm_nt(xp, plan, w1), iters)
+        report(f"grouped_gemm_nt w1 rows={t * k} E={e}", ms, bytes_=2.0 * w1.numel() + 2.0 * t * k * (h + 2 * f), flops=2.0 * t * k * h * 2 * f)
+        gu = K.grouped_gemm_nt(xp, plan, w1)
+        ms = timeit(lambda: glu_fwd(gu, "clamped_swish", 7.0, 1.702, plan=plan), iters)
+        report(f"glu clamped_swish by expert rows={t * k} F={f}", ms, bytes_=6.0 * t * k * f)
+        y = K.grouped_gemm_nt(glu_fwd(gu, "clamped_swish", 7.0, 1.702, plan=plan), plan, w2)
+        resid, sh, sg = torch.zeros(t, h, device="cuda"), torch.randn(t, h, device="cuda").bfloat16(), torch.randn(h, device="cuda").bfloat16()
+        w = torch.zeros(h, device="cuda")
+        ms = timeit(lambda: moe_combine_norm_(resid, y, plan.pos, k, 1.0 / k, x, sh, sg, w, 1e-5, 1.0), iters)
+        report(f"moe_combine_norm T={t} k={k} H={h}", ms, bytes_=t * h * (2.0 * k + 4 + 8 + 2))
+
+
+CASES = {"hybrid_delta": case_delta, "hybrid_latent": case_latent, "hybrid_stream": case_stream}

@@ -24,7 +24,8 @@ from mindspeed_rl_b200.rollout.scheduler import SamplingParams
 
 CUDA = pytest.param("cuda", marks=pytest.mark.gpu)
 DEVICES = ["cpu", CUDA]
-TOL = {torch.float32: 3e-5, torch.bfloat16: 4e-2}
+# bf16: the positions of the worst rounding (nearly tied scores, small norms) reach several times the mean
+TOL = {torch.float32: 3e-5, torch.bfloat16: 9e-2}
 
 
 @functools.lru_cache(maxsize=None)
@@ -53,6 +54,8 @@ def close(got, want, dtype=torch.float32, tol=None):
     assert got.shape == want.shape
     err = (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean().sqrt()
     assert float(err.max()) < (tol or TOL[dtype]), (float(err.max()), int(err.argmax()))
+    if tol is None and dtype == torch.bfloat16:
+        assert float(err.mean()) < 1.5e-2, float(err.mean())
 
 
 def run_schedule(eng, seq, cuts, rid="r", end=True):
