@@ -33,7 +33,10 @@ constexpr uint32_t TILE_HALF = 128 * 64 * 2;          // one [128 rows x 64 cols
 constexpr uint32_t TILE_BYTES = 2 * TILE_HALF;         // 32 KiB
 constexpr uint32_t SMEM_Q = 0;
 constexpr uint32_t TMEM_COLS = 512;                    // backward kernels
-constexpr uint32_t fwd_smem_bytes(int bn) { return TILE_BYTES + 4u * (2u * bn * 64 * 2) + 128u * bn * 2; }
+// nqk: 64-column halves of a query / key head (values have two)
+constexpr uint32_t fwd_smem_bytes(int bn, int nqk) {
+  return nqk * TILE_HALF + 2u * (nqk + 2u) * (bn * 64 * 2) + 128u * bn * 2;
+}
 constexpr int OUT_PITCH = 144;
 constexpr int SOFTMAX_WARPS = 8, TMA_WARP = 8, MMA_WARP = 9, THREADS = 320;
 
@@ -61,9 +64,10 @@ __device__ __forceinline__ int head_col(int col0, int gs, int hpg, int hs, int h
 
 // BN = keys per tile.  128: one CTA per SM (192 KiB of shared memory, 512 TMEM columns).  64: two
 // CTAs per SM (112 KiB, 256 columns each), so that one CTA's soft-max, prologue and epilogue overlap
-// the other's tensor work.
-template <int BN>
-__global__ void __launch_bounds__(THREADS, BN == 128 ? 1 : 2)
+// the other's tensor work.  NQK = 64-column halves of a query / key head: 2, or 3 for the 192-wide heads of latent
+// attention (128 unrotated + 64 rotated entries, values 128), then one CTA per SM.
+template <int BN, int NQK>
+__global__ void __launch_bounds__(THREADS, BN == 128 || NQK == 3 ? 1 : 2)
 fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                       const __grid_constant__ CUtensorMap map_v, const __grid_constant__ Params p) {
   extern __shared__ unsigned char smem_raw[];
@@ -71,8 +75,8 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       (reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   __shared__ uint64_t q_full, k_full[2], v_full[2], k_empty[2], v_empty[2], s_full[2], s_free[2], p_ready, pv_done;
   __shared__ uint32_t tmem_slot;
-  constexpr uint32_t KV_HALF = BN * 64 * 2, KV_BYTES = 2 * KV_HALF;
-  constexpr uint32_t SMEM_K = TILE_BYTES, SMEM_V = SMEM_K + 2 * KV_BYTES, SMEM_P = SMEM_V + 2 * KV_BYTES;
+  constexpr uint32_t KV_HALF = BN * 64 * 2, KV_BYTES = 2 * KV_HALF, K_BYTES = NQK * KV_HALF;
+  constexpr uint32_t SMEM_K = NQK * TILE_HALF, SMEM_V = SMEM_K + 2 * K_BYTES, SMEM_P = SMEM_V + 2 * KV_BYTES;
   constexpr uint32_t TMEM_COLS = BN == 128 ? 512 : 256;      // S0 [0,BN) S1 [BN,2BN) O [2BN, 2BN+128)
   constexpr int HALF = BN / 2, NCH = HALF / 32;              // key columns per soft-max thread
 
@@ -92,7 +96,7 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     // less than a full KiB of slack when two CTAs share an SM)
     uint32_t dyn;
     asm volatile("mov.u32 %0, %%dynamic_smem_size;\n" : "=r"(dyn));
-    if ((uint32_t)(smem - smem_raw) + fwd_smem_bytes(BN) > dyn) {
+    if ((uint32_t)(smem - smem_raw) + fwd_smem_bytes(BN, NQK) > dyn) {
       if (threadIdx.x == 0) atomicCAS(p.error, 0, ERR_SMEM);
       return;
     }
@@ -130,19 +134,19 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       const int qc = head_col(p.q_col0, p.q_group_stride, p.q_hpg, p.q_head_stride, h);
       const int kc = head_col(p.k_col0, p.k_group_stride, p.k_hpg, p.k_head_stride, hk);
       const int vc = head_col(p.v_col0, p.v_group_stride, p.v_hpg, p.v_head_stride, hk);
-      mbar_expect_tx(&q_full, TILE_BYTES);
-      tma_load_2d(smem + SMEM_Q, &map_q, &q_full, qc, q0 + m0);
-      tma_load_2d(smem + SMEM_Q + TILE_HALF, &map_q, &q_full, qc + 64, q0 + m0);
+      mbar_expect_tx(&q_full, NQK * TILE_HALF);
+#pragma unroll
+      for (int i = 0; i < NQK; ++i) tma_load_2d(smem + SMEM_Q + i * TILE_HALF, &map_q, &q_full, qc + i * 64, q0 + m0);
       bool ok = true;
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int st = j & 1;
         const uint32_t use = j >> 1;
         if (use > 0) ok = mbar_wait(&k_empty[st], (use - 1) & 1, p.error, ERR_EMPTY);
         if (!ok) break;
-        mbar_expect_tx(&k_full[st], KV_BYTES);
-        unsigned char* sk = smem + SMEM_K + st * KV_BYTES;
-        tma_load_2d(sk, &map_k, &k_full[st], kc, k0 + j * BN);
-        tma_load_2d(sk + KV_HALF, &map_k, &k_full[st], kc + 64, k0 + j * BN);
+        mbar_expect_tx(&k_full[st], K_BYTES);
+        unsigned char* sk = smem + SMEM_K + st * K_BYTES;
+#pragma unroll
+        for (int i = 0; i < NQK; ++i) tma_load_2d(sk + i * KV_HALF, &map_k, &k_full[st], kc + i * 64, k0 + j * BN);
         if (use > 0) ok = mbar_wait(&v_empty[st], (use - 1) & 1, p.error, ERR_EMPTY);
         if (!ok) break;
         mbar_expect_tx(&v_full[st], KV_BYTES);
@@ -162,9 +166,9 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         if (!mbar_wait(&k_full[st], (j >> 1) & 1, p.error, ERR_K)) return false;
         if (j >= 2 && !mbar_wait(&s_free[st], ((j >> 1) - 1) & 1, p.error, ERR_S)) return false;
         fence_after();
-        const uint32_t k_addr = smem_u32(smem + SMEM_K + st * KV_BYTES);
+        const uint32_t k_addr = smem_u32(smem + SMEM_K + st * K_BYTES);
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {
+        for (int kk = 0; kk < NQK * 4; ++kk) {
           umma(tmem + st * BN, desc_sw128(q_addr + (kk >> 2) * TILE_HALF + (kk & 3) * 32, 16, 1024),
                desc_sw128(k_addr + (kk >> 2) * KV_HALF + (kk & 3) * 32, 16, 1024), id_s,
                kk > 0 ? 1u : 0u);
@@ -855,16 +859,17 @@ static bool fa5_make_map(CUtensorMap* map, const void* base, long long rows, lon
             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-static long long fa5_width(int heads, long long gs, long long hpg, long long hs) {
+static long long fa5_width(int heads, long long gs, long long hpg, long long hs, int head_dim = fa5::D) {
   long long w = 0;
   for (int h = 0; h < heads; ++h) {
-    const long long c = (h / hpg) * gs + (h % hpg) * hs + fa5::D;
+    const long long c = (h / hpg) * gs + (h % hpg) * hs + head_dim;
     w = c > w ? c : w;
   }
   return w;
 }
 
-// Same contract as msrl_flash_attn_varlen_fwd (attention.cu) for head dim 128, plus the number of
+// Same contract as msrl_flash_attn_varlen_fwd (attention.cu) for head dim 128, or query / key heads of 192 (`D`)
+// with values of 128, plus the number of
 // key rows `Tk` and a device status word (0 = ok; 11..17 = a bounded wait ran out).  Layout
 // arrays: {stride_t, group_stride, heads_per_group, head_stride} for q, k, v (12 values).
 // Returns cudaErrorNotSupported for shapes this kernel does not cover: the caller falls back.
@@ -874,7 +879,7 @@ MSRL_API int msrl_flash_attn_varlen_fwd_tcgen05(const void* q, const void* k, co
                                                 int max_q, int nh, int nkv, long long Tq, long long Tk,
                                                 int D, float scale, int causal, int* error, cudaStream_t st) {
   if (batch == 0 || Tq == 0) return 0;
-  if (D != fa5::D || nh % nkv != 0 || (o_stride_t % 8) != 0 || (reinterpret_cast<uintptr_t>(o) & 15) != 0)
+  if ((D != fa5::D && D != 192) || nh % nkv != 0 || (o_stride_t % 8) != 0 || (reinterpret_cast<uintptr_t>(o) & 15) != 0)
     return (int)cudaErrorNotSupported;
   for (int i = 0; i < 3; ++i) {
     const long long* l = lay + 4 * i;
@@ -885,10 +890,11 @@ MSRL_API int msrl_flash_attn_varlen_fwd_tcgen05(const void* q, const void* k, co
     const char* e = getenv("MSRL_ATTN_KEY_TILE");
     bn = (e != nullptr && atoi(e) == 128) ? 128 : 64;
   }
+  const int nqk = D / 64, kt = nqk == 3 ? 64 : bn;       // 192: only 64-key tiles fit
   CUtensorMap mq, mk, mv;
-  if (!fa5_make_map(&mq, q, Tq, fa5_width(nh, lay[1], lay[2], lay[3]), lay[0]) ||
-      !fa5_make_map(&mk, k, Tk, fa5_width(nkv, lay[5], lay[6], lay[7]), lay[4], bn) ||
-      !fa5_make_map(&mv, v, Tk, fa5_width(nkv, lay[9], lay[10], lay[11]), lay[8], bn))
+  if (!fa5_make_map(&mq, q, Tq, fa5_width(nh, lay[1], lay[2], lay[3], D), lay[0]) ||
+      !fa5_make_map(&mk, k, Tk, fa5_width(nkv, lay[5], lay[6], lay[7], D), lay[4], kt) ||
+      !fa5_make_map(&mv, v, Tk, fa5_width(nkv, lay[9], lay[10], lay[11]), lay[8], kt))
     return (int)cudaErrorNotSupported;
   fa5::Params p{};
   p.o = (__nv_bfloat16*)o;
@@ -905,20 +911,17 @@ MSRL_API int msrl_flash_attn_varlen_fwd_tcgen05(const void* q, const void* k, co
   p.k_col0 = 0; p.k_group_stride = (int)lay[5]; p.k_hpg = (int)lay[6]; p.k_head_stride = (int)lay[7];
   p.v_col0 = 0; p.v_group_stride = (int)lay[9]; p.v_hpg = (int)lay[10]; p.v_head_stride = (int)lay[11];
   p.error = error;
-  static bool attr_set = false;
-  const int smem = (int)fa5::fwd_smem_bytes(bn) + (bn == 128 ? 1024 : 896);   // 64: two CTAs in 228 KiB
-  if (!attr_set) {
-    cudaError_t e = bn == 128
-        ? cudaFuncSetAttribute(fa5::fa_fwd_tcgen05_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem)
-        : cudaFuncSetAttribute(fa5::fa_fwd_tcgen05_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  static bool attr_set[2] = {false, false};
+  const int smem = (int)fa5::fwd_smem_bytes(kt, nqk) + (kt == 64 && nqk == 2 ? 896 : 1024);   // 64, 2: two CTAs in 228 KiB
+  auto* kernel = nqk == 3 ? fa5::fa_fwd_tcgen05_kernel<64, 3>
+                          : bn == 128 ? fa5::fa_fwd_tcgen05_kernel<128, 2> : fa5::fa_fwd_tcgen05_kernel<64, 2>;
+  if (!attr_set[nqk - 2]) {
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
-    attr_set = true;
+    attr_set[nqk - 2] = true;
   }
   dim3 grid((max_q + fa5::BM - 1) / fa5::BM, nh, batch);
-  if (bn == 128)
-    fa5::fa_fwd_tcgen05_kernel<128><<<grid, fa5::THREADS, smem, st>>>(mq, mk, mv, p);
-  else
-    fa5::fa_fwd_tcgen05_kernel<64><<<grid, fa5::THREADS, smem, st>>>(mq, mk, mv, p);
+  kernel<<<grid, fa5::THREADS, smem, st>>>(mq, mk, mv, p);
   return (int)cudaGetLastError();
 }
 

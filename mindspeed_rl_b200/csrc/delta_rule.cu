@@ -154,14 +154,12 @@ struct ConvWindow {
       }
     }
   }
-  __device__ __forceinline__ void step(const T* row, float (&y)[4]) {
-#pragma unroll
-    for (int j = 0; j + 1 < TAPS; ++j)
-#pragma unroll
-      for (int c = 0; c < 4; ++c) x[j][c] = x[j + 1][c];
-    ldf4(row, x[TAPS - 1]);
+  __device__ __forceinline__ void step(const float (&in)[4], float (&y)[4]) {
 #pragma unroll
     for (int c = 0; c < 4; ++c) {
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j) x[j][c] = x[j + 1][c];
+      x[TAPS - 1][c] = in[c];
       float s = 0.f;
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) s += x[j][c] * w[j][c];
@@ -169,6 +167,8 @@ struct ConvWindow {
     }
   }
 };
+
+constexpr int PREP_U = 4;       // tokens whose projections are loaded together
 
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256)
@@ -190,45 +190,61 @@ delta_prep_fast_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, co
       ck.weights(p.conv, kd + ch);
     }
     int seq = -1;
-    for (int t = t0; t < t1; ++t) {
-      const int b = tok_seq[t];
-      if (b != seq) {
-        seq = b;
-        const int i = t - cu[b], pos = start_pos[b] + i;
+    float rq[PREP_U][4], rk[PREP_U][4];
+    int sq[PREP_U];
+    for (int tb = t0; tb < t1; tb += PREP_U) {
+#pragma unroll
+      for (int x = 0; x < PREP_U; ++x) {
+        const int t = min(tb + x, t1 - 1);
+        sq[x] = tok_seq[t];
         if (on) {
-          cq.fill(p, t, i, pos, slots[b], p.q_col + ch, ch);
-          ck.fill(p, t, i, pos, slots[b], p.k_col + ch, kd + ch);
+          ldf4(p.proj + t * p.ld + p.q_col + ch, rq[x]);
+          ldf4(p.proj + t * p.ld + p.k_col + ch, rk[x]);
         }
       }
-      float q[4] = {0.f, 0.f, 0.f, 0.f}, k[4] = {0.f, 0.f, 0.f, 0.f};
-      if (on) {
-        cq.step(p.proj + t * p.ld + p.q_col + ch, q);
-        ck.step(p.proj + t * p.ld + p.k_col + ch, k);
-      }
-      float qq = 0.f, kk = 0.f, qk = 0.f;
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        qq += q[c] * q[c];
-        kk += k[c] * k[c];
-        qk += q[c] * k[c];
-      }
+      for (int x = 0; x < PREP_U; ++x) {
+        const int t = tb + x;
+        if (t >= t1) break;
+        const int b = sq[x];
+        if (b != seq) {
+          seq = b;
+          const int i = t - cu[b], pos = start_pos[b] + i;
+          if (on) {
+            cq.fill(p, t, i, pos, slots[b], p.q_col + ch, ch);
+            ck.fill(p, t, i, pos, slots[b], p.k_col + ch, kd + ch);
+          }
+        }
+        float q[4] = {0.f, 0.f, 0.f, 0.f}, k[4] = {0.f, 0.f, 0.f, 0.f};
+        if (on) {
+          cq.step(rq[x], q);
+          ck.step(rk[x], k);
+        }
+        float qq = 0.f, kk = 0.f, qk = 0.f;
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        qq += __shfl_xor_sync(0xffffffffu, qq, o);
-        kk += __shfl_xor_sync(0xffffffffu, kk, o);
-        qk += __shfl_xor_sync(0xffffffffu, qk, o);
-      }
-      const float qs = qscale / sqrtf(qq + p.unit_eps), ks = 1.f / sqrtf(kk + p.unit_eps);
+        for (int c = 0; c < 4; ++c) {
+          qq += q[c] * q[c];
+          kk += k[c] * k[c];
+          qk += q[c] * k[c];
+        }
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        q[c] *= qs;
-        k[c] *= ks;
+        for (int o = 16; o > 0; o >>= 1) {
+          qq += __shfl_xor_sync(0xffffffffu, qq, o);
+          kk += __shfl_xor_sync(0xffffffffu, kk, o);
+          qk += __shfl_xor_sync(0xffffffffu, qk, o);
+        }
+        const float qs = qscale / sqrtf(qq + p.unit_eps), ks = 1.f / sqrtf(kk + p.unit_eps);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          q[c] *= qs;
+          k[c] *= ks;
+        }
+        if (on) {
+          stf4(qn + (long long)t * kd + ch, q);
+          stf4(kn + (long long)t * kd + ch, k);
+        }
+        if (lane == 0) kq[(long long)t * p.KVH + unit] = qk * qs * ks;
       }
-      if (on) {
-        stf4(qn + (long long)t * kd + ch, q);
-        stf4(kn + (long long)t * kd + ch, k);
-      }
-      if (lane == 0) kq[(long long)t * p.KVH + unit] = qk * qs * ks;
     }
   } else if (unit < p.KVH + uv) {
     const int c = (unit - p.KVH) * 128 + lane * 4;
@@ -236,22 +252,35 @@ delta_prep_fast_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, co
     ConvWindow<TAPS, T> cv;
     cv.weights(p.conv, 2 * kd + c);
     int seq = -1;
-    for (int t = t0; t < t1; ++t) {
-      const int b = tok_seq[t];
-      if (b != seq) {
-        seq = b;
-        const int i = t - cu[b];
-        cv.fill(p, t, i, start_pos[b] + i, slots[b], p.v_col + c, 2 * kd + c);
+    float rv[PREP_U][4];
+    int sq[PREP_U];
+    for (int tb = t0; tb < t1; tb += PREP_U) {
+#pragma unroll
+      for (int x = 0; x < PREP_U; ++x) {
+        const int t = min(tb + x, t1 - 1);
+        sq[x] = tok_seq[t];
+        ldf4(p.proj + t * p.ld + p.v_col + c, rv[x]);
       }
-      float y[4];
-      cv.step(p.proj + t * p.ld + p.v_col + c, y);
-      stf4(vv + (long long)t * nv + c, y);
+#pragma unroll
+      for (int x = 0; x < PREP_U; ++x) {
+        const int t = tb + x;
+        if (t >= t1) break;
+        if (sq[x] != seq) {
+          seq = sq[x];
+          const int i = t - cu[seq];
+          cv.fill(p, t, i, start_pos[seq] + i, slots[seq], p.v_col + c, 2 * kd + c);
+        }
+        float y[4];
+        cv.step(rv[x], y);
+        stf4(vv + (long long)t * nv + c, y);
+      }
     }
   } else if (unit < p.KVH + uv + ug) {
     const int c = (unit - p.KVH - uv) * 128 + lane * 4;
     if (c >= ng) return;
     const float rate = -expf(p.a_log[c / p.dim]);            // dim is a multiple of 4: one head per lane
     const float bias[4] = {p.dt_bias[c], p.dt_bias[c + 1], p.dt_bias[c + 2], p.dt_bias[c + 3]};
+#pragma unroll 4
     for (int t = t0; t < t1; ++t) {
       float x[4];
       ldf4(p.a + t * p.a_ld + c, x);
@@ -298,13 +327,14 @@ __device__ __forceinline__ float2 unpack2(f2 a) {
 
 constexpr int SCAN_TB = 16;      // tokens staged at a time
 
-// LPC lanes share a column, each with DPL rows (row = 4 * (LPC * n + lane) + j); COLS columns per block
-template <int DPL, int LPC, int COLS, bool VEC>
-__global__ void __launch_bounds__(COLS * LPC)
+// LPC lanes share CPT neighbouring columns, each lane with DPL rows of them (row = 4 * (LPC * n + lane) + j);
+// COLS columns per block.  Every value of q, k and g that a thread loads serves its CPT columns.
+template <int DPL, int LPC, int CPT, int COLS, bool VEC>
+__global__ void __launch_bounds__(COLS / CPT * LPC)
 delta_scan_kernel(const float* qn, const float* kn, const float* kq, const float* vv, const float* g,
                   const float* beta, float* state, const int* cu, const int* start_pos, const long long* slots, int H,
                   int KVH, int dim, int vdim, float* o) {
-  constexpr int DP = DPL * LPC, THREADS = COLS * LPC;
+  constexpr int DP = DPL * LPC, THREADS = COLS / CPT * LPC;
   extern __shared__ __align__(16) float sm[];
   // two buffers of [q TB*DP | k TB*DP | g TB*DP | v TB*COLS | beta TB | kq TB]
   constexpr int BUF = SCAN_TB * (3 * DP + COLS + 2);
@@ -313,21 +343,23 @@ delta_scan_kernel(const float* qn, const float* kn, const float* kq, const float
   const long long t0 = cu[b];
   const int len = cu[b + 1] - cu[b];
   if (len <= 0) return;
-  const int col_l = threadIdx.x / LPC, lr = threadIdx.x % LPC;
+  const int col_l = threadIdx.x / LPC * CPT, lr = threadIdx.x % LPC;
   const int col = c0 + col_l;
-  const bool on = col < vdim;
   const long long slot = slots[b];
   float* Sg = state + ((slot * H + h) * dim) * (long long)vdim + col;
 
   for (int i = threadIdx.x; i < 2 * BUF; i += THREADS) sm[i] = 0.f;      // pad rows stay zero
-  f2 s[DPL / 2];
+  f2 s[CPT][DPL / 2];
   const bool fresh = start_pos[b] == 0;
 #pragma unroll
-  for (int n = 0; n < DPL; n += 2) {
-    const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
-    const bool have = !fresh && on;
-    s[n / 2] = pack2(have && r < dim ? Sg[(long long)r * vdim] : 0.f, have && r + 1 < dim ? Sg[(long long)(r + 1) * vdim] : 0.f);
-  }
+  for (int c = 0; c < CPT; ++c)
+#pragma unroll
+    for (int n = 0; n < DPL; n += 2) {
+      const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
+      const bool have = !fresh && col + c < vdim;
+      s[c][n / 2] = pack2(have && r < dim ? Sg[(long long)r * vdim + c] : 0.f,
+                          have && r + 1 < dim ? Sg[(long long)(r + 1) * vdim + c] : 0.f);
+    }
   __syncthreads();
 
   auto stage = [&](int blk) {
@@ -385,43 +417,67 @@ delta_scan_kernel(const float* qn, const float* kn, const float* kq, const float
 #pragma unroll 2
     for (int tt = 0; tt < n; ++tt) {
       const ulonglong2 *q4 = rows(0, tt), *k4 = rows(1, tt), *g4 = rows(2, tt);
-      const float bt = bb[tt], vt = bv[tt * COLS + col_l], kqt = bb[SCAN_TB + tt];
+      const float bt = bb[tt], kqt = bb[SCAN_TB + tt];
       f2 kk[DPL / 2];
-      f2 pk[2] = {0ull, 0ull}, pq[2] = {0ull, 0ull};
+      f2 pk[CPT][2], pq[CPT][2];
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) pk[c][0] = pk[c][1] = pq[c][0] = pq[c][1] = 0ull;
 #pragma unroll
       for (int m = 0; m < DPL / 4; ++m) {
         const ulonglong2 gg = g4[m * LPC], kv = k4[m * LPC], qq = q4[m * LPC];
         kk[2 * m] = kv.x;
         kk[2 * m + 1] = kv.y;
-        s[2 * m] = mul2(s[2 * m], gg.x);
-        s[2 * m + 1] = mul2(s[2 * m + 1], gg.y);
-        pk[0] = fma2(s[2 * m], kv.x, pk[0]);
-        pk[1] = fma2(s[2 * m + 1], kv.y, pk[1]);
-        pq[0] = fma2(s[2 * m], qq.x, pq[0]);
-        pq[1] = fma2(s[2 * m + 1], qq.y, pq[1]);
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+          s[c][2 * m] = mul2(s[c][2 * m], gg.x);
+          s[c][2 * m + 1] = mul2(s[c][2 * m + 1], gg.y);
+          pk[c][0] = fma2(s[c][2 * m], kv.x, pk[c][0]);
+          pk[c][1] = fma2(s[c][2 * m + 1], kv.y, pk[c][1]);
+          pq[c][0] = fma2(s[c][2 * m], qq.x, pq[c][0]);
+          pq[c][1] = fma2(s[c][2 * m + 1], qq.y, pq[c][1]);
+        }
       }
-      const float2 k0 = unpack2(pk[0]), k1 = unpack2(pk[1]), q0 = unpack2(pq[0]), q1 = unpack2(pq[1]);
-      float dk = (k0.x + k0.y) + (k1.x + k1.y), dq = (q0.x + q0.y) + (q1.x + q1.y);
+      float dk[CPT], dq[CPT];
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) {
+        const float2 k0 = unpack2(pk[c][0]), k1 = unpack2(pk[c][1]), q0 = unpack2(pq[c][0]), q1 = unpack2(pq[c][1]);
+        dk[c] = (k0.x + k0.y) + (k1.x + k1.y);
+        dq[c] = (q0.x + q0.y) + (q1.x + q1.y);
+      }
 #pragma unroll
       for (int x = LPC / 2; x > 0; x >>= 1) {
-        dk += __shfl_xor_sync(0xffffffffu, dk, x);
-        dq += __shfl_xor_sync(0xffffffffu, dq, x);
-      }
-      const float u = bt * (vt - dk);
-      const f2 uu = pack2(u, u);
 #pragma unroll
-      for (int m = 0; m < DPL / 2; ++m) s[m] = fma2(kk[m], uu, s[m]);
-      if (lr == 0 && on) o[((t0 + first + tt) * H + h) * vdim + col] = dq + kqt * u;
+        for (int c = 0; c < CPT; ++c) dk[c] += __shfl_xor_sync(0xffffffffu, dk[c], x);
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) dq[c] += __shfl_xor_sync(0xffffffffu, dq[c], x);
+      }
+#pragma unroll
+      for (int c = 0; c < CPT; ++c) {
+        const float u = bt * (bv[tt * COLS + col_l + c] - dk[c]);
+        const f2 uu = pack2(u, u);
+#pragma unroll
+        for (int m = 0; m < DPL / 2; ++m) s[c][m] = fma2(kk[m], uu, s[c][m]);
+        dq[c] += kqt * u;
+      }
+      // one lane per column writes it
+      if (lr < CPT) {
+        float mine = dq[0];
+#pragma unroll
+        for (int c = 1; c < CPT; ++c) mine = lr == c ? dq[c] : mine;
+        if (col + lr < vdim) o[((t0 + first + tt) * H + h) * vdim + col + lr] = mine;
+      }
     }
     __syncthreads();
   }
 #pragma unroll
-  for (int n = 0; n < DPL; n += 2) {
-    const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
-    const float2 v = unpack2(s[n / 2]);
-    if (on && r < dim) Sg[(long long)r * vdim] = v.x;
-    if (on && r + 1 < dim) Sg[(long long)(r + 1) * vdim] = v.y;
-  }
+  for (int c = 0; c < CPT; ++c)
+#pragma unroll
+    for (int n = 0; n < DPL; n += 2) {
+      const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
+      const float2 v = unpack2(s[c][n / 2]);
+      if (col + c < vdim && r < dim) Sg[(long long)r * vdim + c] = v.x;
+      if (col + c < vdim && r + 1 < dim) Sg[(long long)(r + 1) * vdim + c] = v.y;
+    }
 }
 
 // ---- prefill: the last inputs of the convolutions ------------------------------------------------------
@@ -611,21 +667,21 @@ static int allow_smem(F* kernel, size_t bytes) {
   return (int)cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
 }
 
-template <int DPL, int LPC, int COLS>
+template <int DPL, int LPC, int CPT, int COLS>
 static int launch_scan(const float* qn, const float* kn, const float* kq, const float* vv, const float* g,
                        const float* beta, float* state, const int* cu, const int* start_pos, const long long* slots,
                        int batch, int H, int KVH, int dim, int vdim, float* o, cudaStream_t st) {
   const size_t smem = 2 * sizeof(float) * SCAN_TB * (3 * DPL * LPC + COLS + 2);
   const dim3 grid((unsigned)((vdim + COLS - 1) / COLS), (unsigned)H, (unsigned)batch);
   if (dim % 4 == 0) {
-    const int e = allow_smem(delta_scan_kernel<DPL, LPC, COLS, true>, smem);
+    const int e = allow_smem(delta_scan_kernel<DPL, LPC, CPT, COLS, true>, smem);
     if (e) return e;
-    delta_scan_kernel<DPL, LPC, COLS, true><<<grid, COLS * LPC, smem, st>>>(qn, kn, kq, vv, g, beta, state, cu,
+    delta_scan_kernel<DPL, LPC, CPT, COLS, true><<<grid, COLS / CPT * LPC, smem, st>>>(qn, kn, kq, vv, g, beta, state, cu,
                                                                             start_pos, slots, H, KVH, dim, vdim, o);
   } else {
-    const int e = allow_smem(delta_scan_kernel<DPL, LPC, COLS, false>, smem);
+    const int e = allow_smem(delta_scan_kernel<DPL, LPC, CPT, COLS, false>, smem);
     if (e) return e;
-    delta_scan_kernel<DPL, LPC, COLS, false><<<grid, COLS * LPC, smem, st>>>(qn, kn, kq, vv, g, beta, state, cu,
+    delta_scan_kernel<DPL, LPC, CPT, COLS, false><<<grid, COLS / CPT * LPC, smem, st>>>(qn, kn, kq, vv, g, beta, state, cu,
                                                                              start_pos, slots, H, KVH, dim, vdim, o);
   }
   return (int)cudaGetLastError();
@@ -655,14 +711,12 @@ MSRL_API int msrl_delta_prefill(const void* proj, long long ld, const void* a, l
     else if (usual && p.taps == 2 && tiles.y <= 65535) MSRL_PREP(2);
     else delta_prep_kernel<T><<<tokens, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, qn, kn, kq, vv, g, beta);
 #undef MSRL_PREP
-    // four lanes a column spend fewer instructions, eight hide a token's latency better when few blocks run
-    const bool many = (long long)batch * H * ((vdim + 31) / 32) >= 4LL * sm_count();
     int e;
-#define MSRL_SCAN(D, L) launch_scan<D, L, 32>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st)
-    if (dim <= 32) e = MSRL_SCAN(8, 4);
-    else if (dim <= 64) e = many ? MSRL_SCAN(16, 4) : MSRL_SCAN(8, 8);
-    else if (dim <= 128) e = many ? MSRL_SCAN(32, 4) : MSRL_SCAN(16, 8);
-    else e = MSRL_SCAN(32, 8);
+#define MSRL_SCAN(D, L, C, N) launch_scan<D, L, C, N>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st)
+    if (dim <= 32) e = MSRL_SCAN(8, 4, 1, 32);
+    else if (dim <= 64) e = MSRL_SCAN(8, 8, 2, 32);
+    else if (dim <= 128) e = MSRL_SCAN(16, 8, 2, 32);
+    else e = MSRL_SCAN(32, 8, 1, 32);
 #undef MSRL_SCAN
     if (e) return e;
     const int channels = 2 * KVH * dim + H * vdim;

@@ -129,12 +129,12 @@ def latent_prefill_attention(proj: torch.Tensor, kv: torch.Tensor, lay: LatentLa
     if _lib.use_kernels(proj, kv, cu_q, cu_k):
         v = kv.view(-1)[h * lay.qp:]
         out = guard.empty(t, h * lay.vp, device=proj.device, dtype=proj.dtype)
-        if proj.dtype == torch.bfloat16 and lay.qp == lay.vp and lay.qp in (64, 128):
+        if proj.dtype == torch.bfloat16 and (lay.qp, lay.vp) in ((64, 64), (128, 128), (192, 128)):
             from .gemm import _status_word
             st = (proj.stride(0), kv.stride(0))
             spec = (ctypes.c_longlong * 12)(st[0], 0, h, lay.qp, st[1], 0, h, lay.qp, st[1], 0, h, lay.vp)
             lse = guard.empty(h, t, device=proj.device, dtype=torch.float32)
-            if lay.qp == 128 and use_tcgen05_attention():
+            if lay.qp >= 128 and use_tcgen05_attention():
                 rc = _lib.load().msrl_flash_attn_varlen_fwd_tcgen05(
                     ptr(proj), ptr(kv), ptr(v), spec, ptr(out), c_ll(h * lay.vp), ptr(lse), ptr(cu_q), ptr(cu_k),
                     c_int(batch), c_int(max_q), c_int(h), c_int(h), c_ll(t), c_ll(kv.shape[0]), c_int(lay.qp),
@@ -142,11 +142,12 @@ def latent_prefill_attention(proj: torch.Tensor, kv: torch.Tensor, lay: LatentLa
                 if rc != _NOT_SUPPORTED:
                     check(rc, "flash_attn_varlen_fwd_tcgen05")
                     return out
-            check(_lib.load().msrl_flash_attn_varlen_fwd(
-                ptr(proj), ptr(kv), ptr(v), spec, ptr(out), c_ll(h * lay.vp), ptr(lse), ptr(cu_q), ptr(cu_k),
-                c_int(batch), c_int(max_q), c_int(h), c_int(h), c_ll(t), c_int(lay.qp), c_float(scale), c_int(1),
-                stream()), "flash_attn_varlen_fwd")
-            return out
+            if lay.qp <= 128:
+                check(_lib.load().msrl_flash_attn_varlen_fwd(
+                    ptr(proj), ptr(kv), ptr(v), spec, ptr(out), c_ll(h * lay.vp), ptr(lse), ptr(cu_q), ptr(cu_k),
+                    c_int(batch), c_int(max_q), c_int(h), c_int(h), c_ll(t), c_int(lay.qp), c_float(scale), c_int(1),
+                    stream()), "flash_attn_varlen_fwd")
+                return out
         lds = (ctypes.c_longlong * 4)(proj.stride(0), kv.stride(0), kv.stride(0), h * lay.vp)
         ints = (ctypes.c_int * 6)(lay.qp, lay.qp, lay.vp, lay.vp, lay.dn + lay.dr, lay.vp)
         check(_lib.load().msrl_attn_simt(ptr(proj), ptr(kv), ptr(v), ptr(out), lds, ints, ptr(cu_q), ptr(cu_k),

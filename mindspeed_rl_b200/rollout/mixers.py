@@ -76,8 +76,9 @@ class LatentAttention:
         self.spec, self.eps = spec, eps
         h, dn, dr, dv, r = spec.heads, spec.dim, spec.rot_dim, spec.vdim, spec.kv_rank
         qp, vp = dn + dr, dv
-        if dtype == torch.bfloat16 and max(qp, vp) <= 128:
-            qp = vp = 64 if max(qp, vp) <= 64 else 128
+        if dtype == torch.bfloat16 and vp <= 128 and qp <= 192:
+            vp = 64 if max(qp, vp) <= 64 else 128
+            qp = 192 if qp > 128 else vp
         q = _pad_cols(w["q"].view(h, dn + dr, -1).transpose(1, 2), qp).transpose(1, 2).reshape(h * qp, -1)
         fused, cols = stack_sections([q, w["dkv"]])
         self.lay = lay = LatentLayout(h, dn, dr, dv, r, qp, vp, cols[1], spec.rot.dims)
