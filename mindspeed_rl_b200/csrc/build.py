@@ -31,7 +31,8 @@ NVCC_FLAGS = [
 ]
 # kernels whose results are specified in 32-bit (an fp32 residual, recurrent state, fp32 attention): compiled
 # without the approximate divisions, square roots, exponentials and flush-to-zero of --use_fast_math
-PRECISE = {"residual_stream", "delta_rule", "latent_attention", "grouped_gemm_simt"}
+PRECISE = {"residual_stream", "delta_rule", "latent_attention", "latent_decode_tcgen05",
+           "grouped_gemm_simt"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 
@@ -39,7 +40,7 @@ CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 # model family from a fresh checkout compiles these and nothing else.  hybrid: the forward of layer-by-layer decoders
 # (without the sampler)
 GROUPS = {
-    "hybrid": ("residual_stream", "delta_rule", "latent_attention", "grouped_gemm_simt", "moe", "moe_gemm_tcgen05",
+    "hybrid": ("residual_stream", "delta_rule", "latent_attention", "latent_decode_tcgen05", "grouped_gemm_simt", "moe", "moe_gemm_tcgen05",
                "attention", "attention_tcgen05", "gemm2cta_tcgen05"),
 }
 

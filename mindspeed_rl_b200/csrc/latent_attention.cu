@@ -12,8 +12,9 @@
 //   spread      the rotated key part into every head's expanded key
 //   attn_simt   soft-max attention of packed sequences for any head sizes, fp32 arithmetic
 //   decode_simt one query per sequence over the paged rows, any sizes, fp32 arithmetic
-//   decode_mma  the same on the tensor cores for bf16: a block takes 16 / 32 / 64 heads of one sequence and a
-//               range of its keys, so that a row is read once for all of them; `combine` merges the ranges
+//   decode_mma  the same on the legacy tensor path for bf16 (block sizes that latent_decode_tcgen05.cu does not
+//               take): a block takes 16 / 32 / 64 heads of one sequence and a range of its keys, so that a row is
+//               read once for all of them; `combine` merges the ranges
 #include "dtype_utils.cuh"
 #include "mma_utils.cuh"
 
@@ -656,15 +657,30 @@ MSRL_API int msrl_latent_decode_simt(const void* q, const void* cache, const int
   return (int)cudaGetLastError();
 }
 
-// key ranges per (sequence, head group) so that one wave of blocks covers the machine
+// Key ranges per (sequence, head group): the count that finishes first when whole waves of one block per SM walk
+// their tiles of 64 keys and every block pays for its start, its end and the merge.
 MSRL_API int msrl_latent_decode_nsplit(int batch, int H, int max_context) {
-  const int groups = H <= 32 ? 1 : (H + 63) / 64;
-  const int blocks = batch * groups;
-  int n = blocks > 0 ? sm_count() / blocks : 1;
-  const int most = (max_context + 127) / 128;
-  if (n > most) n = most;
-  if (n > 64) n = 64;
-  return n < 1 ? 1 : n;
+  const long long blocks = (long long)batch * (H <= 32 ? 1 : (H + 63) / 64);
+  const int tiles = (max_context + 63) / 64, sms = sm_count();
+  int best = 1;
+  double least = 1e30;
+  for (int n = 1; n <= 64 && n <= (tiles + 1) / 2 + 1; ++n) {
+    const double waves = (double)((blocks * n + sms - 1) / sms);
+    const double cost = waves * ((tiles + n - 1) / n + 2.5) + (n > 1 ? 1.0 : 0.0);
+    if (cost < least) {
+      least = cost;
+      best = n;
+    }
+  }
+  return best;
+}
+
+// merge of the key ranges that msrl_latent_decode_tcgen05 leaves in part_o / part_ml
+MSRL_API int msrl_latent_decode_combine(const float* part_o, const float* part_ml, int batch, int H, int RP, int nsplit,
+                                        void* out, cudaStream_t st) {
+  if (batch == 0) return 0;
+  mla::combine_kernel<<<(unsigned)(batch * H), 128, 0, st>>>(part_o, part_ml, nsplit, RP, (__nv_bfloat16*)out);
+  return (int)cudaGetLastError();
 }
 
 // part_o [B, H, nsplit, RP] and part_ml [B, H, nsplit, 2] fp32 (unused when nsplit == 1)

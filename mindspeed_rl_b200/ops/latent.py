@@ -171,9 +171,10 @@ def latent_prefill_attention(proj: torch.Tensor, kv: torch.Tensor, lay: LatentLa
 
 def latent_decode_attention(q: torch.Tensor, cache: torch.Tensor, lay: LatentLayout, block_tables: torch.Tensor,
                             context_lens: torch.Tensor, max_context: int, scale: float,
-                            nsplit: Optional[int] = None) -> torch.Tensor:
+                            nsplit: Optional[int] = None, use_tcgen05: bool = True) -> torch.Tensor:
     """One query per sequence, ``q [B, heads, CP]`` in cache-row space, over the sequence's cached rows ->
-    weighted latents ``[B, heads, RP]``."""
+    weighted latents ``[B, heads, RP]``.  ``nsplit``: key ranges per sequence (default: what fills the machine);
+    ``use_tcgen05=False`` keeps to the ``mma.sync`` kernel (comparison runs)."""
     b, h, cp = q.shape
     bs = cache.shape[1]
     if _lib.use_kernels(q, cache, block_tables, context_lens):
@@ -185,6 +186,18 @@ def latent_decode_attention(q: torch.Tensor, cache: torch.Tensor, lay: LatentLay
             if n > 1:
                 part_o = _workspace("latent_part_o", b * h * n * lay.RP, q.device)
                 part_ml = _workspace("latent_part_ml", b * h * n * 2, q.device)
+            if use_tcgen05:
+                from .gemm import _status_word
+                rc = L.msrl_latent_decode_tcgen05(
+                    ptr(q), ptr(cache), c_ll(cache.shape[0]), ptr(block_tables), c_int(block_tables.shape[1]), c_int(bs),
+                    ptr(context_lens), c_float(scale), c_int(b), c_int(h), c_int(cp), c_int(lay.RP), c_int(n), ptr(part_o),
+                    ptr(part_ml), ptr(out), ptr(_status_word(q.device)), stream())
+                if rc != _NOT_SUPPORTED:
+                    check(rc, "latent_decode_tcgen05")
+                    if n > 1:
+                        check(L.msrl_latent_decode_combine(ptr(part_o), ptr(part_ml), c_int(b), c_int(h), c_int(lay.RP),
+                                                           c_int(n), ptr(out), stream()), "latent_decode_combine")
+                    return out
             rc = L.msrl_latent_decode_mma(ptr(q), ptr(cache), ptr(block_tables), c_int(block_tables.shape[1]), c_int(bs),
                                           ptr(context_lens), c_float(scale), c_int(b), c_int(h), c_int(cp),
                                           c_int(lay.RP), c_int(n), ptr(part_o), ptr(part_ml), ptr(out), stream())

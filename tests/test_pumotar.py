@@ -309,7 +309,7 @@ def test_decode_attention_keys_at_borders(device, heads, rank, dr):
         targets += [0, 1, 15, 16, 63, 64]
         b = len(lens)
         perm = torch.randperm(b * blocks, generator=torch.Generator().manual_seed(1)).view(b, blocks)
-        cache = torch.full((b * blocks, bs, lay.CP), 7.0)            # what freed pages hold must not matter
+        cache = torch.full((b * blocks, bs, lay.CP), float("nan") if device == "cuda" else 7.0)   # what freed pages hold must not matter
         q = torch.empty(b, heads, lay.CP)
         want = torch.empty(b, heads, lay.RP, dtype=torch.float64)
         for i, (m, target) in enumerate(zip(lens, targets)):
@@ -321,10 +321,10 @@ def test_decode_attention_keys_at_borders(device, heads, rank, dr):
             want[i] = s @ rows[:, :lay.RP].double()
             if m > 1:
                 assert float(s[0, target]) > 0.9                     # the key does stand out
-        for nsplit in (None, 1, 3, 5):
+        for nsplit, t5 in ((None, True), (1, True), (3, True), (5, False), (1, False)):
             got = ops.latent_decode_attention(q.to(device, dtype), cache.to(device, dtype), lay,
                                               perm.to(device, torch.int32), torch.tensor(lens, dtype=torch.int32, device=device),
-                                              n, 0.5, nsplit=nsplit)
+                                              n, 0.5, nsplit=nsplit, use_tcgen05=t5)
             close(got.reshape(b * heads, -1), want.reshape(b * heads, -1), dtype, tol=1e-5 if dtype == torch.float32 else 1.5e-2)
 
 
