@@ -36,7 +36,6 @@ constexpr int SM_WARPS = 8, TMA_WARP = 8, MMA_WARP = 9, THREADS = 320;
 enum { ERR_SMEM = 60, ERR_Q = 61, ERR_K = 62, ERR_S = 63, ERR_P = 64, ERR_PV = 65, ERR_EMPTY = 66, ERR_FREE = 67 };
 
 struct Params {
-  const __nv_bfloat16* q;      // [B, H, CP]
   const int* block_tables;
   int max_blocks, block_size;
   const int* context_lens;
@@ -49,6 +48,13 @@ struct Params {
   int* error;
 };
 
+__device__ __forceinline__ bool mbar_test(uint64_t* bar, uint32_t parity) {       // one look, no suspension
+  uint32_t ok;
+  asm volatile("{\n\t.reg .pred p;\n\tmbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}\n"
+               : "=r"(ok) : "r"(smem_u32(bar)), "r"(parity) : "memory");
+  return ok != 0;
+}
+
 __host__ __device__ inline uint32_t smem_bytes(int hb, int chunks) {
   return (uint32_t)chunks * hb * 128u + 2u * chunks * CHUNK + hb * 128u;
 }
@@ -57,7 +63,8 @@ constexpr uint32_t idesc_a_mn(int m, int n) { return idesc_bf16(m, n, false) | (
 
 template <int HB>
 __global__ void __launch_bounds__(THREADS, 1)
-latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_constant__ Params p) {
+latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_constant__ CUtensorMap map_q,
+                     const __grid_constant__ Params p) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>(
       (reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
@@ -99,7 +106,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_const
   unsigned char* sP = sK + 2 * stage_bytes;
 
   if (threadIdx.x == 0) {
-    mbar_init(&q_full, SM_WARPS);
+    mbar_init(&q_full, 1);
     for (int i = 0; i < 2; ++i) {
       mbar_init(&k_full[i], 1);
       mbar_init(&k_empty[i], 1);
@@ -128,6 +135,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_const
       const int bs = p.block_size, per_tile = KT / bs, last_block = (n + bs - 1) / bs;
       const int boxes = (p.CP + 63) / 64;
       const uint32_t box_bytes = (uint32_t)bs * 128u;
+      // HB rows from the first head on; rows past this sequence's heads belong to the next one or are zero, and
+      // their scores are never used
+      mbar_expect_tx(&q_full, (uint32_t)boxes * q_chunk);
+      for (int c = 0; c < boxes; ++c) tma_load_2d(sQ + c * q_chunk, &map_q, &q_full, c * 64, (int)row0);
       bool ok = true;
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int st = j & 1;
@@ -171,7 +182,20 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_const
       if (ok) ok = issue_s(0);
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int st = j & 1;
-        if (j + 1 < n_tiles) ok = issue_s(j + 1);       // the next tile's scores run during this soft-max
+        // The next tile's scores run during this soft-max, unless its rows are still on their way when P is ready:
+        // the product comes first then, because it frees the stage that the tile after waits for.
+        bool next = j + 1 < n_tiles, ahead = false;
+        for (int poll = 0; next && poll < 4096; ++poll) {
+          if (mbar_test(&k_full[st ^ 1], ((j + 1) >> 1) & 1)) {
+            ahead = true;
+            break;
+          }
+          if (mbar_test(&p_ready, j & 1)) break;
+        }
+        if (ahead) {
+          ok = issue_s(j + 1);
+          next = false;
+        }
         if (!ok) break;
         ok = mbar_wait(&p_ready, j & 1, p.error, ERR_P);
         if (!ok) break;
@@ -185,25 +209,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_const
         }
         commit(&pv_done);
         commit(&k_empty[st]);
+        if (next) ok = issue_s(j + 1);
       }
     }
   } else {
-    // ---------------- query, soft-max, output ----------------
-    // query rows: K-major, 128-byte swizzle (16-byte chunk index XOR row % 8); missing heads are zero
-    {
-      const int vecs = p.CP / 8;
-      for (int r = warp; r < HB; r += SM_WARPS) {
-        const __nv_bfloat16* src = p.q + (row0 + (r < heads ? r : 0)) * p.CP;
-        for (int c = lane; c < vecs; c += 32) {
-          uint4 v = make_uint4(0u, 0u, 0u, 0u);
-          if (r < heads) v = *reinterpret_cast<const uint4*>(src + c * 8);
-          *reinterpret_cast<uint4*>(sQ + (c >> 3) * q_chunk + (r >> 3) * 1024 + (r & 7) * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
-        }
-      }
-      asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&q_full);
-    }
+    // ---------------- soft-max, output ----------------
     const int wg = warp >> 2, quarter = warp & 3;
     const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
     const bool scores = quarter < NQ;                   // this warp's lanes hold heads
@@ -344,13 +354,13 @@ static PFN_cuTensorMapEncodeTiled_v12000 encode_fn() {
   return fn;
 }
 
-// the paged cache as [num_blocks * block_size rows, CP columns]; box = one block of rows x 64 columns
-static bool make_map(CUtensorMap* map, const void* base, long long rows, int CP, int block_size) {
+// a [rows, CP] bf16 matrix (the paged cache, all query heads); box = `box_rows` rows x 64 columns
+static bool make_map(CUtensorMap* map, const void* base, long long rows, int CP, int box_rows) {
   auto fn = encode_fn();
   if (fn == nullptr || (reinterpret_cast<uintptr_t>(base) & 15) != 0 || CP % 8 != 0) return false;
   cuuint64_t dims[2] = {(cuuint64_t)CP, (cuuint64_t)rows};
   cuuint64_t strides[1] = {(cuuint64_t)CP * 2};
-  cuuint32_t box[2] = {64u, (cuuint32_t)block_size};
+  cuuint32_t box[2] = {64u, (cuuint32_t)box_rows};
   cuuint32_t estr[2] = {1, 1};
   return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
@@ -358,7 +368,9 @@ static bool make_map(CUtensorMap* map, const void* base, long long rows, int CP,
 }
 
 template <int HB>
-static int launch(const CUtensorMap& map, const Params& p, int batch, cudaStream_t st) {
+static int launch(const CUtensorMap& map, const void* q, const Params& p, int batch, cudaStream_t st) {
+  CUtensorMap map_q;
+  if (!make_map(&map_q, q, (long long)batch * p.H, p.CP, HB)) return (int)cudaErrorNotSupported;
   const int smem = (int)smem_bytes(HB, p.chunks) + 1024;
   if (smem > 231 * 1000) return (int)cudaErrorNotSupported;      // static shared memory shares the 227 KiB
   static int allowed = 0;
@@ -368,7 +380,7 @@ static int launch(const CUtensorMap& map, const Params& p, int batch, cudaStream
     allowed = smem;
   }
   const dim3 grid((unsigned)p.nsplit, (unsigned)((p.H + HB - 1) / HB), (unsigned)batch);
-  latent_decode_kernel<HB><<<grid, THREADS, smem, st>>>(map, p);
+  latent_decode_kernel<HB><<<grid, THREADS, smem, st>>>(map, map_q, p);
   return (int)cudaGetLastError();
 }
 
@@ -390,8 +402,8 @@ MSRL_API int msrl_latent_decode_tcgen05(const void* q, const void* cache, long l
   CUtensorMap map;
   if (!ld5::make_map(&map, cache, num_blocks * block_size, CP, block_size)) return (int)cudaErrorNotSupported;
   const int boxes = (CP + 63) / 64, blocks = 2 * ((RP + 127) / 128);
-  ld5::Params p{(const __nv_bfloat16*)q, block_tables, max_blocks, block_size, context_lens,
+  ld5::Params p{block_tables, max_blocks, block_size, context_lens,
                 scale * 1.4426950408889634f, H, CP, RP, nsplit, boxes > blocks ? boxes : blocks, part_o, part_ml,
                 (__nv_bfloat16*)out, error};
-  return H <= 32 ? ld5::launch<32>(map, p, batch, st) : ld5::launch<64>(map, p, batch, st);
+  return H <= 32 ? ld5::launch<32>(map, q, p, batch, st) : ld5::launch<64>(map, q, p, batch, st);
 }
