@@ -52,6 +52,10 @@ def parse_args():
     ap.add_argument("--steps", type=int, default=1)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
+    ap.add_argument("--workload", default="grpo", choices=["grpo", "serve"],
+                    help="grpo: the headline benchmark; serve: prefill and decode throughput of the layer-by-layer "
+                         "decoder (Pumotar) beside the latent-attention decoder of equal size, one JSON line per case")
+    ap.add_argument("--serve-sizes", default="", help="comma-separated subset of the serve workload's sizes")
     ap.add_argument("--model", default="qwen25_7b")
     ap.add_argument("--prompts-per-gpu", type=int, default=32)
     ap.add_argument("--samples", type=int, default=8)
@@ -146,6 +150,12 @@ def main():
     args = parse_args()
     if args.impl == "reference":
         reference_arm(args)
+        return
+    if args.workload == "serve":
+        from mindspeed_rl_b200.rollout import serve_bench
+
+        serve_bench.run(args.steps, args.warmup, [x for x in args.serve_sizes.split(",") if x],
+                        emit=lambda line: print(line, flush=True))
         return
     import torch
     import torch.distributed as dist

@@ -72,7 +72,7 @@ __device__ __forceinline__ float conv_silu(const DeltaIn<T>& p, long long t, int
            p.conv[(long long)ch * taps + j];
     }
   }
-  return s * sigmoid_f(s);
+  return s * sigmoid_t<T>(s);
 }
 
 constexpr int DELTA_MAX_DIM = 256;
@@ -163,7 +163,7 @@ struct ConvWindow {
       float s = 0.f;
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) s += x[j][c] * w[j][c];
-      y[c] = s * sigmoid_f(s);
+      y[c] = s * sigmoid_t<T>(s);
     }
   }
 };

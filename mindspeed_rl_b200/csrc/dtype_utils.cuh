@@ -44,6 +44,12 @@ __device__ __forceinline__ void stv(T* p, const float (&f)[4]) {
 }
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+// for activations that are stored in T: bf16 results do not need the last bits of the exponential and the division
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float x) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-x));
+  else return sigmoid_f(x);
+}
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 }  // namespace msrl

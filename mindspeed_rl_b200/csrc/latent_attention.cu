@@ -48,6 +48,76 @@ __device__ __forceinline__ float rotated(const T* x, int d, const float* cs, int
   return (d & 1) ? v * c + u * s : u * c - v * s;
 }
 
+// entries d .. d + 3 (d a multiple of 4) of a rotated part whose rot_dims is a multiple of 4
+template <typename T>
+__device__ __forceinline__ void rotated4(const T* x, int d, const float* cs, int rot_dims, float (&y)[4]) {
+  ldf4(x + d, y);
+  if (d < rot_dims) {
+    const int half = rot_dims / 2, i = d >> 1;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const float c = cs[i + k], s = cs[half + i + k], u = y[2 * k], v = y[2 * k + 1];
+      y[2 * k] = u * c - v * s;
+      y[2 * k + 1] = v * c + u * s;
+    }
+  }
+}
+
+// prep for sizes and columns that are multiples of 4: four entries per load and store
+template <typename T>
+__global__ void __launch_bounds__(256) prep4_kernel(const PrepArgs<T> p) {
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  T* row = p.qkv + t * p.ld;
+  const T* lat_in = row + p.dkv_col;
+  float ss = 0.f;
+  for (int c = threadIdx.x * 4; c < p.rank; c += 1024) {
+    float x[4];
+    ldf4(lat_in + c, x);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) ss += x[j] * x[j];
+  }
+  const int pos = min(max(p.positions[t], 0), p.table_rows - 1);
+  const float* cs = p.table + (long long)pos * p.rot_dims;
+  const long long slot = p.slots[t];
+  // queries first: they do not wait for the norm
+  if (p.qdec != nullptr) {
+    const int w = (p.CP - p.RP) / 4;
+    for (int i = threadIdx.x; i < p.H * w; i += 256) {
+      const int h = i / w, d = (i - h * w) * 4;
+      float y[4] = {0.f, 0.f, 0.f, 0.f};
+      if (d < p.dr) rotated4(row + h * p.q_stride + p.dn, d, cs, p.rot_dims, y);
+      stf4(p.qdec + (t * p.H + h) * p.CP + p.RP + d, y);
+    }
+  } else {
+    const int quads = p.rot_dims / 4;
+    for (int i = threadIdx.x; i < p.H * quads; i += 256) {
+      const int h = i / quads, d = (i - h * quads) * 4;
+      T* x = row + h * p.q_stride + p.dn;
+      float y[4];
+      rotated4(x, d, cs, p.rot_dims, y);
+      stf4(x + d, y);
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)p.rank + p.eps);
+  T* crow = slot >= 0 ? p.cache + slot * p.CP : nullptr;
+  T* lrow = p.lat != nullptr ? p.lat + t * p.CP : nullptr;
+  for (int c = threadIdx.x * 4; c < p.CP; c += 1024) {
+    float y[4] = {0.f, 0.f, 0.f, 0.f};
+    if (c < p.rank) {
+      float w[4];
+      ldf4(lat_in + c, y);
+      ldf4(p.norm_w + c, w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) y[j] *= inv * w[j];
+    } else if (c >= p.RP && c < p.RP + p.dr) {
+      rotated4(lat_in + p.rank, c - p.RP, cs, p.rot_dims, y);
+    }
+    if (crow != nullptr) stf4(crow + c, y);
+    if (lrow != nullptr) stf4(lrow + c, y);
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) prep_kernel(const PrepArgs<T> p) {
   __shared__ float red[32];
@@ -584,7 +654,9 @@ MSRL_API int msrl_latent_prep(void* qkv, long long ld, const int* ints, const fl
     p.cache = (T*)cache;
     p.lat = (T*)lat;
     p.qdec = (T*)qdec;
-    mla::prep_kernel<T><<<tokens, 256, 0, st>>>(p);
+    const bool by4 = ((p.rank | p.dr | p.dn | p.rot_dims | p.q_stride | p.dkv_col | (int)(ld & 3)) & 3) == 0;
+    if (by4) mla::prep4_kernel<T><<<tokens, 256, 0, st>>>(p);
+    else mla::prep_kernel<T><<<tokens, 256, 0, st>>>(p);
     return (int)cudaGetLastError();
   };
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});

@@ -155,17 +155,18 @@ int launch_row_norm(const RowArgs<T>& p, long long rows, cudaStream_t st) {
 
 enum { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMPED_SWISH = 2 };
 
-template <int KIND>
+// 0.5 (1 + tanh(z)) = sigmoid(2 z) carries the tanh form of gelu on the sigmoid of the storage type
+template <int KIND, typename T>
 __device__ __forceinline__ float glu_one(float g, float u, float limit, float alpha) {
   if constexpr (KIND == GLU_SILU) {
-    return g * sigmoid_f(g) * u;
+    return g * sigmoid_t<T>(g) * u;
   } else if constexpr (KIND == GLU_GELU_TANH) {
-    const float k = 0.7978845608028654f;                 // sqrt(2 / pi)
-    return 0.5f * g * (1.f + tanhf(k * (g + 0.044715f * g * g * g))) * u;
+    const float k = 2.f * 0.7978845608028654f;           // 2 sqrt(2 / pi)
+    return g * sigmoid_t<T>(k * (g + 0.044715f * g * g * g)) * u;
   } else {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
-    return g * sigmoid_f(alpha * g) * (u + 1.f);
+    return g * sigmoid_t<T>(alpha * g) * (u + 1.f);
   }
 }
 
@@ -180,20 +181,32 @@ glu_kernel(const T* x, T* y, int F, float limit, float alpha, const int* tile_ex
     const int e = tile_expert[r / 128];
     if (e < 0 || r - offsets[e] >= counts[e]) return;
   }
-  const int c = (blockIdx.y * 256 + threadIdx.x) * V;
-  if (c >= F) return;
-  float g[4], u[4];
-  ldv<V>(x + r * 2 * F + c, g);
-  ldv<V>(x + r * 2 * F + F + c, u);
+  // two vectors a thread, both loads in flight
+  float g[2][4], u[2][4];
+  const int c0 = (blockIdx.y * 512 + threadIdx.x) * V;
 #pragma unroll
-  for (int i = 0; i < V; ++i) g[i] = glu_one<KIND>(g[i], u[i], limit, alpha);
-  stv<V>(y + r * F + c, g);
+  for (int k = 0; k < 2; ++k) {
+    const int c = c0 + k * 256 * V;
+    if (c < F) {
+      ldv<V>(x + r * 2 * F + c, g[k]);
+      ldv<V>(x + r * 2 * F + F + c, u[k]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const int c = c0 + k * 256 * V;
+    if (c < F) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) g[k][i] = glu_one<KIND, T>(g[k][i], u[k][i], limit, alpha);
+      stv<V>(y + r * F + c, g[k]);
+    }
+  }
 }
 
 template <typename T, int V>
 int launch_glu(const T* x, T* y, long long rows, int F, int kind, float limit, float alpha, const int* tile_expert,
                const int* counts, const int* offsets, cudaStream_t st) {
-  const dim3 grid((unsigned)rows, (unsigned)((F / V + 255) / 256));
+  const dim3 grid((unsigned)rows, (unsigned)((F / V + 511) / 512));
   if (kind == GLU_SILU)
     glu_kernel<T, V, GLU_SILU><<<grid, 256, 0, st>>>(x, y, F, limit, alpha, tile_expert, counts, offsets);
   else if (kind == GLU_GELU_TANH)

@@ -1,0 +1,200 @@
+"""Serving throughput of a layer-by-layer decoder beside the closest repeated-block decoder of equal size.
+
+``bench.py --workload serve`` runs it: random weights, prompts and decode batches through ``LLMEngine`` (the
+scheduler, cache, graphs and sampler of generation).  The closest existing model is the latent-attention (MLA)
+decoder with routed experts: same width, heads, head sizes, latent rank, feed-forward sizes, experts and layer
+count.  It caches full per-head keys and values; the layer-by-layer decoder caches latent rows and recurrent
+state.  ``mixed`` puts one latent-attention layer after three recurrent ones, ``latent`` uses latent attention
+everywhere.  One JSON line per measurement: tokens/s from CUDA events around the engine calls.
+"""
+from __future__ import annotations
+
+import json
+from dataclasses import dataclass
+from typing import List
+
+import torch
+
+from ..models.hybrid_config import ChannelDeltaSpec, GluSpec, HybridConfig, LatentAttentionSpec, LayerSpec, Rotary, TableMoESpec
+from ..models.transformer_config import TransformerConfig
+from .engine import LLMEngine
+from .scheduler import SamplingParams
+
+
+@dataclass(frozen=True)
+class Size:
+    name: str
+    width: int
+    heads: int
+    rank: int
+    ff: int
+    experts: int
+    top: int
+    expert_ff: int
+    layers: int = 4
+    vocab: int = 32768
+    dn: int = 64
+    dr: int = 64
+    dv: int = 128
+
+
+SIZES = (Size("1k", 1024, 8, 256, 4096, 32, 4, 512), Size("2k", 2304, 32, 512, 9216, 64, 8, 1024),
+         Size("4k", 4096, 32, 512, 12288, 64, 4, 2048))
+PREFILL = ((1, 8192), (8, 2048))
+DECODE = ((1, 2048), (32, 2048), (256, 2048))
+NEW_TOKENS = 64
+
+
+def hybrid_config(s: Size, pattern: str) -> HybridConfig:
+    latent = LayerSpec("latent_attention", LatentAttentionSpec(s.heads, s.dn, s.dr, s.dv, s.rank, (s.dn + s.dr) ** -0.5,
+                                                               Rotary(s.dr, 10000.0)))
+    delta = LayerSpec("channel_delta", ChannelDeltaSpec(s.heads, s.heads, 128, 128, 4))
+    dense = GluSpec(s.ff, "gelu_tanh")
+    act = dict(act="clamped_swish", limit=7.0, alpha=1.702)
+    moe = TableMoESpec(s.experts, s.top, GluSpec(s.expert_ff, **act), GluSpec(s.expert_ff, **act))
+    layers = []
+    for i in range(s.layers):
+        m = latent if pattern == "latent" or i % 4 == 3 else delta
+        layers.append(LayerSpec(m.type, m.mixer, dense if i == 0 else moe))
+    return HybridConfig("Pumotar", s.vocab, s.width, layers, 1e-5)
+
+
+def random_state(cfg: HybridConfig, device) -> dict:
+    """Random checkpoint tensors of a configuration (drawn on the device)."""
+    g = torch.Generator(device=device).manual_seed(0)
+    w, out = cfg.hidden_size, {}
+
+    def lin(name, rows, cols):
+        out[name] = (torch.randn(rows, cols, generator=g, device=device) * cols ** -0.5).to(cfg.params_dtype)
+
+    def vec(name, n, mean=0.0):
+        out[name] = torch.full((n,), mean, device=device)
+
+    def glu(p, ff):
+        lin(p + "gate", ff, w)
+        lin(p + "up", ff, w)
+        lin(p + "down", w, ff)
+
+    lin("embed", cfg.vocab_size, w)
+    vec("final.norm", w)
+    for i, l in enumerate(cfg.layers):
+        p, m = f"l{i}.mix.", l.mixer
+        vec(f"l{i}.norm1", w)
+        vec(f"l{i}.norm2", w)
+        if l.type == "latent_attention":
+            lin(p + "q", m.heads * (m.dim + m.rot_dim), w)
+            lin(p + "dkv", m.kv_rank + m.rot_dim, w)
+            vec(p + "dkv.norm", m.kv_rank, 1.0)
+            lin(p + "uk", m.heads * m.dim, m.kv_rank)
+            lin(p + "uv", m.heads * m.vdim, m.kv_rank)
+            lin(p + "o", w, m.heads * m.vdim)
+        else:
+            kd, hv = m.kv_heads * m.dim, m.heads * m.vdim
+            for n, rows in (("q", kd), ("k", kd), ("v", hv)):
+                lin(p + n, rows, w)
+                out[p + n + ".conv"] = torch.randn(rows, m.conv, generator=g, device=device) * 0.5
+            lin(p + "b", m.heads, w)
+            vec(p + "A_log", m.heads, -2.0)
+            vec(p + "norm", m.vdim, 1.0)
+            vec(p + "dt_bias", m.heads * m.dim)
+            for a, n in (("a", m.heads * m.dim), ("g", hv)):
+                lin(p + a + "1", 128, w)
+                lin(p + a + "2", n, 128)
+            lin(p + "o", w, hv)
+        p = f"l{i}.mlp."
+        if isinstance(l.mlp, TableMoESpec):
+            for e in range(l.mlp.experts):
+                glu(f"{p}e{e}.", l.mlp.expert.ff)
+            out[p + "table"] = torch.rand(cfg.vocab_size, l.mlp.experts, generator=g, device=device).topk(l.mlp.top, -1).indices
+            glu(p + "shared.", l.mlp.shared.ff)
+            lin(p + "shared.sg", 1, w)
+        else:
+            glu(p, l.mlp.ff)
+    return out
+
+
+def mla_config(s: Size) -> TransformerConfig:
+    return TransformerConfig(num_layers=s.layers, hidden_size=s.width, ffn_hidden_size=s.ff, num_attention_heads=s.heads,
+                             num_query_groups=s.heads, vocab_size=s.vocab, norm_epsilon=1e-5, max_position_embeddings=16384,
+                             untie_embeddings_and_output_weights=False, num_experts=s.experts, moe_router_topk=s.top,
+                             moe_ffn_hidden_size=s.expert_ff, n_shared_experts=1, first_k_dense_replace=1,
+                             multi_latent_attention=True, kv_lora_rank=s.rank, qk_head_dim=s.dn, qk_pos_emb_head_dim=s.dr,
+                             v_head_dim=s.dv)
+
+
+def build(s: Size, model: str, device):
+    if model == "mla":
+        from ..models.gpt import GPTModel
+        from ..reshard.alias import alias_rollout_weights
+
+        cfg = mla_config(s)
+        return cfg, alias_rollout_weights(GPTModel(cfg, device=device))
+    from .hybrid_weights import build_hybrid_weights
+
+    cfg = hybrid_config(s, model)
+    return cfg, build_hybrid_weights(cfg, random_state(cfg, device), device)
+
+
+def _timed(fn) -> float:
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    e0.record()
+    fn()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1)
+
+
+def run(steps: int, warmup: int, sizes=None, models=("mla", "latent", "mixed"), emit=print) -> List[dict]:
+    dev = torch.device("cuda")
+    rows = []
+    for s in SIZES:
+        if sizes and s.name not in sizes:
+            continue
+        gen = torch.Generator().manual_seed(1)
+        for model in models:
+            cfg, weights = build(s, model, dev)
+            bs = max(b for b, _ in DECODE)
+            ctx = max(n for _, n in DECODE) + NEW_TOKENS
+            eng = LLMEngine(cfg, dev, max_num_seqs=bs, max_num_batched_tokens=16384, max_model_len=8192 + 16, block_size=16,
+                            enforce_eager=False, graph_batch_sizes=tuple(b for b, _ in DECODE))
+            eng.runner.bind_weights(weights)
+            eng.init_cache(bs * ((ctx + 15) // 16 + 1))
+            base = dict(workload="serve", model=model, size=s.name, width=s.width, heads=s.heads, layers=s.layers,
+                        kv_bytes_per_token=eng.kv_bytes_per_block() // 16, state_bytes_per_seq=eng.state_bytes() // bs,
+                        dtype="bf16", data="synthetic: uniform random ids, random weights")
+            for b, n in PREFILL:
+                prompts = torch.randint(0, s.vocab, (b, n), generator=gen).tolist()
+
+                def prefill():
+                    eng.replay([(str(i), p, [n - 1]) for i, p in enumerate(prompts)], [str(i) for i in range(b)])
+
+                for _ in range(max(warmup, 3)):
+                    prefill()
+                ms = sorted(_timed(prefill) for _ in range(max(steps, 3)))[max(steps, 3) // 2]
+                rows.append(dict(base, case=f"prefill {b}x{n}", ms=round(ms, 3), tokens_per_s=round(b * n / ms * 1e3)))
+                emit(json.dumps(rows[-1]))
+            for b, n in DECODE:
+                prompts = torch.randint(0, s.vocab, (b, n), generator=gen).tolist()
+                params = SamplingParams(temperature=1.0, max_tokens=NEW_TOKENS + 1, ignore_eos=True, seed=1)
+
+                def decode():
+                    for p in prompts:
+                        eng.add_request(None, p, params)
+                    while any(q.num_computed < len(q.prompt_ids) for q in eng.scheduler.running) or eng.scheduler.waiting:
+                        eng.step()
+
+                    def rest():
+                        while eng.has_unfinished_requests():
+                            eng.step()
+                    return _timed(rest)
+
+                for _ in range(1):
+                    decode()
+                ms = sorted(decode() for _ in range(max(steps, 3)))[max(steps, 3) // 2]
+                rows.append(dict(base, case=f"decode B={b} ctx={n}", ms_per_step=round(ms / NEW_TOKENS, 4),
+                                 tokens_per_s=round(b * NEW_TOKENS / ms * 1e3)))
+                emit(json.dumps(rows[-1]))
+            del eng, weights
+            torch.cuda.empty_cache()
+    return rows
