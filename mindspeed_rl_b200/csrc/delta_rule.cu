@@ -15,7 +15,8 @@
 //
 //   prefill: `prep` (conv, silu, unit norms, decays, step sizes of every token), `scan` (the recurrence: one
 //            block per sequence, head and column group; S in registers, LPC lanes share a column) and
-//            `out` (norm and gate);
+//            `out` (norm and gate).  The usual shapes run the recurrence four tokens at a time
+//            (`delta_group_kernel`, `delta_group_scan_kernel`), the others token by token;
 //   decode:  one fused kernel per (sequence, head): all of the above with S read and written once, coalesced.
 //
 // Both sum (S^T k, S^T q) over the decayed state in one pass: o = (gS)^T q + (k.q) u.
@@ -125,9 +126,8 @@ delta_prep_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const i
   for (int h = threadIdx.x; h < p.H; h += 256) beta[t * p.H + h] = sigmoid_f(ldf(p.proj + t * p.ld + p.b_col + h));
 }
 
-// The same for the usual shapes (dim a multiple of 4 up to 128, vdim a multiple of 4, up to 4 taps): a warp walks
-// PREP_TT consecutive tokens with the convolution window of its channels in registers, four channels per lane, so
-// that every projection is read once.  Warps: one per key head (q and k), then 128 v channels or 128 decay channels.
+// ---- prefill, usual shapes (dim a multiple of 4 up to 128, vdim a multiple of 4, 2 to 4 taps): a warp walks
+// consecutive tokens with the convolution window of its channels in registers, four channels per lane.
 constexpr int PREP_TT = 16;
 
 template <int TAPS, typename T>
@@ -170,127 +170,203 @@ struct ConvWindow {
 
 constexpr int PREP_U = 4;       // tokens whose projections are loaded together
 
+// v of every token: warps of 128 channels, PREP_TT tokens each
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256)
-delta_prep_fast_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const int* start_pos,
-                       const long long* slots, int tokens, float* qn, float* kn, float* kq, float* vv, float* g,
-                       float* beta) {
-  const int lane = threadIdx.x & 31;
-  const int unit = blockIdx.x * 8 + (threadIdx.x >> 5);
-  const int kd = p.KVH * p.dim, nv = p.H * p.vdim, ng = p.H * p.dim;
-  const int uv = (nv + 127) / 128, ug = (ng + 127) / 128;
+delta_value_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const int* start_pos, const long long* slots,
+                   int tokens, float* vv) {
+  const int kd = p.KVH * p.dim, nv = p.H * p.vdim;
+  const int c = (blockIdx.x * 8 + (threadIdx.x >> 5)) * 128 + (threadIdx.x & 31) * 4;
   const int t0 = blockIdx.y * PREP_TT, t1 = min(tokens, t0 + PREP_TT);
-  if (unit < p.KVH) {
-    const int d = lane * 4, ch = unit * p.dim + d;
-    const bool on = d < p.dim;
-    const float qscale = 1.f / sqrtf((float)p.dim);
-    ConvWindow<TAPS, T> cq, ck;
-    if (on) {
-      cq.weights(p.conv, ch);
-      ck.weights(p.conv, kd + ch);
-    }
-    int seq = -1;
-    float rq[PREP_U][4], rk[PREP_U][4];
-    int sq[PREP_U];
-    for (int tb = t0; tb < t1; tb += PREP_U) {
+  if (c >= nv) return;
+  ConvWindow<TAPS, T> cv;
+  cv.weights(p.conv, 2 * kd + c);
+  int seq = -1;
+  float rv[PREP_U][4];
+  int sq[PREP_U];
+  for (int tb = t0; tb < t1; tb += PREP_U) {
 #pragma unroll
-      for (int x = 0; x < PREP_U; ++x) {
-        const int t = min(tb + x, t1 - 1);
-        sq[x] = tok_seq[t];
-        if (on) {
-          ldf4(p.proj + t * p.ld + p.q_col + ch, rq[x]);
-          ldf4(p.proj + t * p.ld + p.k_col + ch, rk[x]);
+    for (int x = 0; x < PREP_U; ++x) {
+      const int t = min(tb + x, t1 - 1);
+      sq[x] = tok_seq[t];
+      ldf4(p.proj + t * p.ld + p.v_col + c, rv[x]);
+    }
+#pragma unroll
+    for (int x = 0; x < PREP_U; ++x) {
+      const int t = tb + x;
+      if (t >= t1) break;
+      if (sq[x] != seq) {
+        seq = sq[x];
+        const int i = t - cu[seq];
+        cv.fill(p, t, i, start_pos[seq] + i, slots[seq], p.v_col + c, 2 * kd + c);
+      }
+      float y[4];
+      cv.step(rv[x], y);
+      stf4(vv + (long long)t * nv + c, y);
+    }
+  }
+}
+
+// Groups of four tokens.  With G_j = g_0 ... g_j inside a group and S the state before it,
+//
+//   r_j = S^T (G_j k_j)                    u_j = beta_j (v_j - r_j - sum_{i<j} a_ji u_i)
+//   p_j = S^T (G_j q_j)                    o_j = p_j + sum_{i<=j} b_ji u_i
+//   S  <- G_3 S + sum_j (k_j g_{j+1} ... g_3) u_j^T
+//   a_ji = k_j . (g_{i+1} ... g_j k_i)     b_ji = q_j . (g_{i+1} ... g_j k_i)
+//
+// which is the recurrence with the tokens' mutual terms taken out of the state: only products of decays (never a
+// quotient) appear.  A group and head is one record: G k (4 x DP), G q (4 x DP), the write vectors (4 x DP), G_3 (DP),
+// a (6), b (10), beta (4), padding (4).  A sequence's groups start at its first token; record slot of its group n:
+// cu[b] / 4 + b + n.  Missing tokens of a last group have k = q = 0, g = 1, beta = 0.
+constexpr int GRP = 4, COEF = 24;
+
+__host__ __device__ constexpr int group_floats(int dp) { return 13 * dp + COEF; }
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256)
+delta_group_kernel(const DeltaIn<T> p, const int* cu, const int* start_pos, const long long* slots, int batch,
+                   int total_slots, int DP, float* rec) {
+  const int lane = threadIdx.x & 31, h = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (h >= p.H) return;
+  const int hk = h / (p.H / p.KVH), kd = p.KVH * p.dim;
+  const int d = lane * 4, ch = hk * p.dim + d;
+  const bool on = d < p.dim, pad = !on && d < DP;
+  const int CH = group_floats(DP);
+  const float rate = -expf(p.a_log[h]);
+  const float qscale = 1.f / sqrtf((float)p.dim);
+  ConvWindow<TAPS, T> cq, ck;
+  float bias[4] = {0.f, 0.f, 0.f, 0.f};
+  if (on) {
+    cq.weights(p.conv, ch);
+    ck.weights(p.conv, kd + ch);
+#pragma unroll
+    for (int c = 0; c < 4; ++c) bias[c] = p.dt_bias[h * p.dim + d + c];
+  }
+  const int s0 = blockIdx.y * 4, s1 = min(total_slots, s0 + 4);
+  int last_b = -1;
+  for (int s = s0; s < s1; ++s) {
+    int lo = 0, hi = batch - 1;                          // the last sequence whose first slot is at most s
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (cu[mid] / GRP + mid <= s) lo = mid;
+      else hi = mid - 1;
+    }
+    const int b = lo, len = cu[b + 1] - cu[b], i0 = (s - (cu[b] / GRP + b)) * GRP;
+    if (i0 >= len) {                                     // a slot between two sequences
+      last_b = -1;
+      continue;
+    }
+    const int t0 = cu[b] + i0, cnt = min(GRP, len - i0);
+    float q[GRP][4], k[GRP][4], g[GRP][4];
+#pragma unroll
+    for (int j = 0; j < GRP; ++j) {
+      const long long t = t0 + min(j, cnt - 1);
+#pragma unroll
+      for (int c = 0; c < 4; ++c) q[j][c] = k[j][c] = g[j][c] = 0.f;
+      if (on) {
+        ldf4(p.proj + t * p.ld + p.q_col + ch, q[j]);
+        ldf4(p.proj + t * p.ld + p.k_col + ch, k[j]);
+        ldf4(p.a + t * p.a_ld + h * p.dim + d, g[j]);
+      }
+    }
+    if (on && b != last_b) {
+      const int pos = start_pos[b] + i0;
+      cq.fill(p, t0, i0, pos, slots[b], p.q_col + ch, ch);
+      ck.fill(p, t0, i0, pos, slots[b], p.k_col + ch, kd + ch);
+    }
+    last_b = b;
+    float beta = 0.f;
+    if (lane < cnt) beta = sigmoid_f(ldf(p.proj + (long long)(t0 + lane) * p.ld + p.b_col + h));
+    float v[8];
+#pragma unroll
+    for (int j = 0; j < GRP; ++j) {
+      v[2 * j] = v[2 * j + 1] = 0.f;
+      if (on && j < cnt) {
+        cq.step(q[j], q[j]);
+        ck.step(k[j], k[j]);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          g[j][c] = expf(rate * softplus_f(g[j][c] + bias[c]));
+          v[2 * j] += q[j][c] * q[j][c];
+          v[2 * j + 1] += k[j][c] * k[j][c];
+        }
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          q[j][c] = k[j][c] = 0.f;
+          g[j][c] = 1.f;
         }
       }
+    }
 #pragma unroll
-      for (int x = 0; x < PREP_U; ++x) {
-        const int t = tb + x;
-        if (t >= t1) break;
-        const int b = sq[x];
-        if (b != seq) {
-          seq = b;
-          const int i = t - cu[b], pos = start_pos[b] + i;
-          if (on) {
-            cq.fill(p, t, i, pos, slots[b], p.q_col + ch, ch);
-            ck.fill(p, t, i, pos, slots[b], p.k_col + ch, kd + ch);
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int x = 0; x < 8; ++x) v[x] += __shfl_xor_sync(0xffffffffu, v[x], o);
+#pragma unroll
+    for (int j = 0; j < GRP; ++j) {
+      const float qs = qscale / sqrtf(v[2 * j] + p.unit_eps), ks = 1.f / sqrtf(v[2 * j + 1] + p.unit_eps);
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        q[j][c] *= qs;
+        k[j][c] *= ks;
+      }
+    }
+    // mutual terms: w = g_{i+1} ... g_j k_i, extended token by token
+    float co[16];
+#pragma unroll
+    for (int x = 0; x < 16; ++x) co[x] = 0.f;
+#pragma unroll
+    for (int i = 0; i < GRP; ++i) {
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        float w = k[i][c];
+#pragma unroll
+        for (int j = i; j < GRP; ++j) {
+          if (j > i) {
+            w *= g[j][c];
+            co[j * (j - 1) / 2 + i] += k[j][c] * w;
           }
+          co[6 + j * (j + 1) / 2 + i] += q[j][c] * w;
         }
-        float q[4] = {0.f, 0.f, 0.f, 0.f}, k[4] = {0.f, 0.f, 0.f, 0.f};
-        if (on) {
-          cq.step(rq[x], q);
-          ck.step(rk[x], k);
-        }
-        float qq = 0.f, kk = 0.f, qk = 0.f;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int x = 0; x < 16; ++x) co[x] += __shfl_xor_sync(0xffffffffu, co[x], o);
+    float* r = rec + ((long long)s * p.H + h) * CH;
+    if (on || pad) {
+      float cum[4] = {1.f, 1.f, 1.f, 1.f}, tail[4] = {1.f, 1.f, 1.f, 1.f}, y[4];
+#pragma unroll
+      for (int j = 0; j < GRP; ++j) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          qq += q[c] * q[c];
-          kk += k[c] * k[c];
-          qk += q[c] * k[c];
+          cum[c] *= g[j][c];
+          y[c] = k[j][c] * cum[c];
         }
+        stf4(r + j * DP + d, y);
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          qq += __shfl_xor_sync(0xffffffffu, qq, o);
-          kk += __shfl_xor_sync(0xffffffffu, kk, o);
-          qk += __shfl_xor_sync(0xffffffffu, qk, o);
-        }
-        const float qs = qscale / sqrtf(qq + p.unit_eps), ks = 1.f / sqrtf(kk + p.unit_eps);
+        for (int c = 0; c < 4; ++c) y[c] = q[j][c] * cum[c];
+        stf4(r + (GRP + j) * DP + d, y);
+      }
+      stf4(r + 12 * DP + d, cum);
+#pragma unroll
+      for (int j = GRP - 1; j >= 0; --j) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          q[c] *= qs;
-          k[c] *= ks;
+          y[c] = k[j][c] * tail[c];
+          tail[c] *= g[j][c];
         }
-        if (on) {
-          stf4(qn + (long long)t * kd + ch, q);
-          stf4(kn + (long long)t * kd + ch, k);
-        }
-        if (lane == 0) kq[(long long)t * p.KVH + unit] = qk * qs * ks;
+        stf4(r + (8 + j) * DP + d, y);
       }
     }
-  } else if (unit < p.KVH + uv) {
-    const int c = (unit - p.KVH) * 128 + lane * 4;
-    if (c >= nv) return;
-    ConvWindow<TAPS, T> cv;
-    cv.weights(p.conv, 2 * kd + c);
-    int seq = -1;
-    float rv[PREP_U][4];
-    int sq[PREP_U];
-    for (int tb = t0; tb < t1; tb += PREP_U) {
+    if (lane < COEF) {
+      float mine = 0.f;
 #pragma unroll
-      for (int x = 0; x < PREP_U; ++x) {
-        const int t = min(tb + x, t1 - 1);
-        sq[x] = tok_seq[t];
-        ldf4(p.proj + t * p.ld + p.v_col + c, rv[x]);
-      }
-#pragma unroll
-      for (int x = 0; x < PREP_U; ++x) {
-        const int t = tb + x;
-        if (t >= t1) break;
-        if (sq[x] != seq) {
-          seq = sq[x];
-          const int i = t - cu[seq];
-          cv.fill(p, t, i, start_pos[seq] + i, slots[seq], p.v_col + c, 2 * kd + c);
-        }
-        float y[4];
-        cv.step(rv[x], y);
-        stf4(vv + (long long)t * nv + c, y);
-      }
+      for (int x = 0; x < 16; ++x) mine = lane == x ? co[x] : mine;
+      const float bt = __shfl_sync(0x00ffffffu, beta, lane >= 16 && lane < 20 ? lane - 16 : 0);
+      r[13 * DP + lane] = lane < 16 ? mine : lane < 20 ? bt : 0.f;
     }
-  } else if (unit < p.KVH + uv + ug) {
-    const int c = (unit - p.KVH - uv) * 128 + lane * 4;
-    if (c >= ng) return;
-    const float rate = -expf(p.a_log[c / p.dim]);            // dim is a multiple of 4: one head per lane
-    const float bias[4] = {p.dt_bias[c], p.dt_bias[c + 1], p.dt_bias[c + 2], p.dt_bias[c + 3]};
-#pragma unroll 4
-    for (int t = t0; t < t1; ++t) {
-      float x[4];
-      ldf4(p.a + t * p.a_ld + c, x);
-#pragma unroll
-      for (int j = 0; j < 4; ++j) x[j] = expf(rate * softplus_f(x[j] + bias[j]));
-      stf4(g + (long long)t * ng + c, x);
-    }
-  } else if (unit == p.KVH + uv + ug) {
-    for (int t = t0; t < t1; ++t)
-      for (int h = lane; h < p.H; h += 32) beta[(long long)t * p.H + h] = sigmoid_f(ldf(p.proj + t * p.ld + p.b_col + h));
   }
 }
 
@@ -465,6 +541,172 @@ delta_scan_kernel(const float* qn, const float* kn, const float* kq, const float
 #pragma unroll
         for (int c = 1; c < CPT; ++c) mine = lr == c ? dq[c] : mine;
         if (col + lr < vdim) o[((t0 + first + tt) * H + h) * vdim + col + lr] = mine;
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int c = 0; c < CPT; ++c)
+#pragma unroll
+    for (int n = 0; n < DPL; n += 2) {
+      const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
+      const float2 v = unpack2(s[c][n / 2]);
+      if (col + c < vdim && r < dim) Sg[(long long)r * vdim + c] = v.x;
+      if (col + c < vdim && r + 1 < dim) Sg[(long long)(r + 1) * vdim + c] = v.y;
+    }
+}
+
+// ---- prefill: the recurrence over groups of four tokens ------------------------------------------------
+// Same lane layout as delta_scan_kernel with LPC = 8 and two columns per thread.  A group costs one pass over the
+// state for its eight dot products and one for its four writes, and one exchange between lanes.
+constexpr int SG = 2;            // groups staged at a time
+
+template <int DPL, int COLS>
+__global__ void __launch_bounds__(COLS * 4)
+delta_group_scan_kernel(const float* rec, const float* vv, float* state, const int* cu, const int* start_pos,
+                        const long long* slots, int H, int dim, int vdim, float* o) {
+  constexpr int LPC = 8, CPT = 2, DP = DPL * LPC, THREADS = COLS / CPT * LPC, CH = group_floats(DP);
+  constexpr int BUF = SG * (CH + GRP * COLS);
+  extern __shared__ __align__(16) float sm[];            // two buffers of SG x [record | v of four tokens]
+  const int h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * COLS;
+  const long long t0 = cu[b];
+  const int len = cu[b + 1] - cu[b];
+  if (len <= 0) return;
+  const int col_l = threadIdx.x / LPC * CPT, lr = threadIdx.x % LPC, col = c0 + col_l;
+  const float* rb = rec + ((long long)(cu[b] / GRP + b) * H + h) * CH;
+  float* Sg = state + ((slots[b] * H + h) * dim) * (long long)vdim + col;
+  const bool fresh = start_pos[b] == 0;
+  f2 s[CPT][DPL / 2];
+#pragma unroll
+  for (int c = 0; c < CPT; ++c)
+#pragma unroll
+    for (int n = 0; n < DPL; n += 2) {
+      const int r = 4 * (LPC * (n / 4) + lr) + (n & 3);
+      const bool have = !fresh && col + c < vdim;
+      s[c][n / 2] = pack2(have && r < dim ? Sg[(long long)r * vdim + c] : 0.f,
+                          have && r + 1 < dim ? Sg[(long long)(r + 1) * vdim + c] : 0.f);
+    }
+  for (int i = threadIdx.x; i < 2 * BUF; i += THREADS) sm[i] = 0.f;      // columns past vdim, missing tokens: finite
+  __syncthreads();
+
+  const int groups = (len + GRP - 1) / GRP, rounds = (groups + SG - 1) / SG;
+  auto stage = [&](int rd) {
+    float* buf = sm + (rd & 1) * BUF;
+#pragma unroll
+    for (int x = 0; x < SG; ++x) {
+      const int gi = rd * SG + x;
+      if (gi < groups) {
+        const float* src = rb + (long long)gi * H * CH;
+        float* dst = buf + x * (CH + GRP * COLS);
+        for (int i = threadIdx.x; i < CH / 4; i += THREADS) cp_async16b(dst + i * 4, src + i * 4);
+        for (int i = threadIdx.x; i < GRP * COLS / 4; i += THREADS) {
+          const int tt = i / (COLS / 4), c = (i % (COLS / 4)) * 4;
+          if (gi * GRP + tt < len && c0 + c < vdim)
+            cp_async16b(dst + CH + tt * COLS + c, vv + ((t0 + gi * GRP + tt) * H + h) * vdim + c0 + c);
+        }
+      }
+    }
+    asm volatile("cp.async.commit_group;\n" ::);
+  };
+
+  stage(0);
+  for (int rd = 0; rd < rounds; ++rd) {
+    if (rd + 1 < rounds) {
+      stage(rd + 1);
+      asm volatile("cp.async.wait_group 1;\n" ::);
+    } else {
+      asm volatile("cp.async.wait_group 0;\n" ::);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int x = 0; x < SG; ++x) {
+      const int gi = rd * SG + x;
+      if (gi >= groups) break;
+      const float* r = sm + (rd & 1) * BUF + x * (CH + GRP * COLS);
+      const float* co = r + 13 * DP;
+      auto rows = [&](int which) { return reinterpret_cast<const ulonglong2*>(r + which * DP) + lr; };
+      f2 acc[2 * GRP][CPT];                              // r_0 .. r_3, p_0 .. p_3
+#pragma unroll
+      for (int v = 0; v < 2 * GRP; ++v)
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) acc[v][c] = 0ull;
+#pragma unroll
+      for (int m = 0; m < DPL / 4; ++m)
+#pragma unroll
+        for (int v = 0; v < 2 * GRP; ++v) {
+          const ulonglong2 w = rows(v)[m * LPC];
+#pragma unroll
+          for (int c = 0; c < CPT; ++c) {
+            acc[v][c] = fma2(s[c][2 * m], w.x, acc[v][c]);
+            acc[v][c] = fma2(s[c][2 * m + 1], w.y, acc[v][c]);
+          }
+        }
+      // sums over the eight lanes: lane l ends with value l of both columns
+      float val[2 * GRP][CPT];
+#pragma unroll
+      for (int v = 0; v < 2 * GRP; ++v)
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+          const float2 t = unpack2(acc[v][c]);
+          val[v][c] = t.x + t.y;
+        }
+#pragma unroll
+      for (int half = 4; half > 0; half >>= 1) {
+        const bool up = lr & half;
+#pragma unroll
+        for (int v = 0; v < half; ++v)
+#pragma unroll
+          for (int c = 0; c < CPT; ++c) {
+            const float mine = up ? val[v + half][c] : val[v][c], theirs = up ? val[v][c] : val[v + half][c];
+            val[v][c] = mine + __shfl_xor_sync(0xffffffffu, theirs, half);
+          }
+      }
+      // every lane solves for the four writes
+      float u[GRP][CPT];
+#pragma unroll
+      for (int j = 0; j < GRP; ++j) {
+        const float bt = co[16 + j];
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+          float t = r[CH + j * COLS + col_l + c] - __shfl_sync(0xffffffffu, val[0][c], j, 8);
+#pragma unroll
+          for (int i = 0; i < j; ++i) t -= co[j * (j - 1) / 2 + i] * u[i][c];
+          u[j][c] = bt * t;
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < DPL / 4; ++m) {
+        const ulonglong2 ga = rows(12)[m * LPC];
+#pragma unroll
+        for (int c = 0; c < CPT; ++c) {
+          s[c][2 * m] = mul2(s[c][2 * m], ga.x);
+          s[c][2 * m + 1] = mul2(s[c][2 * m + 1], ga.y);
+        }
+#pragma unroll
+        for (int j = 0; j < GRP; ++j) {
+          const ulonglong2 w = rows(8 + j)[m * LPC];
+#pragma unroll
+          for (int c = 0; c < CPT; ++c) {
+            const f2 uu = pack2(u[j][c], u[j][c]);
+            s[c][2 * m] = fma2(w.x, uu, s[c][2 * m]);
+            s[c][2 * m + 1] = fma2(w.y, uu, s[c][2 * m + 1]);
+          }
+        }
+      }
+      // lane 4 + j holds p_j and writes token j
+      const int j = lr - GRP;
+      if (j >= 0 && gi * GRP + j < len) {
+        const float* bj = co + 6 + j * (j + 1) / 2;
+        float y[CPT] = {val[0][0], val[0][1]};
+#pragma unroll
+        for (int i = 0; i < GRP; ++i)
+          if (i <= j) {
+            const float w = bj[i];
+            y[0] += w * u[i][0];
+            y[1] += w * u[i][1];
+          }
+        float* dst = o + ((t0 + gi * GRP + j) * H + h) * vdim + col;
+        if (col + 1 < vdim) *reinterpret_cast<float2*>(dst) = make_float2(y[0], y[1]);   // vdim is a multiple of 4
       }
     }
     __syncthreads();
@@ -687,37 +929,78 @@ static int launch_scan(const float* qn, const float* kn, const float* kq, const 
   return (int)cudaGetLastError();
 }
 
-// scratch (fp32): qn, kn [tokens, KVH, dim], kq [tokens, KVH], vv, o [tokens, H, vdim], g [tokens, H, dim],
-// beta [tokens, H]
+template <int DPL>
+static int launch_group_scan(const float* rec, const float* vv, float* state, const int* cu, const int* start_pos,
+                             const long long* slots, int batch, int H, int dim, int vdim, float* o, cudaStream_t st) {
+  constexpr int COLS = 32;
+  const size_t smem = 2 * sizeof(float) * SG * (group_floats(DPL * 8) + GRP * COLS);
+  const int e = allow_smem(delta_group_scan_kernel<DPL, COLS>, smem);
+  if (e) return e;
+  const dim3 grid((unsigned)((vdim + COLS - 1) / COLS), (unsigned)H, (unsigned)batch);
+  delta_group_scan_kernel<DPL, COLS><<<grid, COLS * 4, smem, st>>>(rec, vv, state, cu, start_pos, slots, H, dim, vdim, o);
+  return (int)cudaGetLastError();
+}
+
+// the shapes of the grouped path (four channels per lane, at most four taps)
+static bool grouped_shape(const int* ints, long long ld, long long a_ld) {
+  const int taps = ints[0], dim = ints[3], vdim = ints[4];
+  return dim % 4 == 0 && dim <= 128 && vdim % 4 == 0 && taps >= 2 && taps <= 4 && ints[5] % 4 == 0 && ints[6] % 4 == 0 &&
+         ints[7] % 4 == 0 && ld % 4 == 0 && a_ld % 4 == 0;
+}
+static int padded_dim(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : 128; }
+
+// fp32 scratch of msrl_delta_prefill
+MSRL_API long long msrl_delta_prefill_scratch(const int* ints, long long ld, long long a_ld, int tokens, int batch) {
+  const long long H = ints[1], KVH = ints[2], dim = ints[3], vdim = ints[4], t = tokens;
+  if (grouped_shape(ints, ld, a_ld))
+    return 8 + 2 * t * H * vdim + (t / GRP + batch) * H * group_floats(padded_dim((int)dim));
+  return 2 * t * H * vdim + 2 * t * KVH * dim + t * H * dim + t * (KVH + H) + 64;
+}
+
 MSRL_API int msrl_delta_prefill(const void* proj, long long ld, const void* a, long long a_ld, const float* conv,
                                 const float* a_log, const float* dt_bias, void* ring, float* state, const int* ints,
                                 float unit_eps, const void* gate, long long gate_ld, const float* norm, float eps,
                                 const int* tok_seq, const int* cu, const int* start_pos, const long long* slots,
-                                int tokens, int batch, float* qn, float* kn, float* kq, float* vv, float* g,
-                                float* beta, float* o, void* y, int is_f32, cudaStream_t st) {
+                                int tokens, int batch, float* scratch, void* y, int is_f32, cudaStream_t st) {
   if (tokens == 0 || batch == 0) return 0;
   const int H = ints[1], KVH = ints[2], dim = ints[3], vdim = ints[4];
   if (dim > DELTA_MAX_DIM || H % KVH != 0 || batch > 65535 || H > 65535) return (int)cudaErrorInvalidValue;
   auto run = [&](auto tag) {
     using T = decltype(tag);
     const DeltaIn<T> p = delta_in<T>(proj, ld, a, a_ld, conv, a_log, dt_bias, ring, state, ints, unit_eps);
-    const bool usual = dim % 4 == 0 && dim <= 128 && vdim % 4 == 0 && p.q_col % 4 == 0 && p.k_col % 4 == 0 &&
-                       p.v_col % 4 == 0 && ld % 4 == 0 && a_ld % 4 == 0;
-    const int units = KVH + (H * vdim + 127) / 128 + (H * dim + 127) / 128 + 1;
-    const dim3 tiles((unsigned)((units + 7) / 8), (unsigned)((tokens + PREP_TT - 1) / PREP_TT));
-#define MSRL_PREP(N) delta_prep_fast_kernel<T, N><<<tiles, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, tokens, qn, kn, kq, vv, g, beta)
-    if (usual && p.taps == 4 && tiles.y <= 65535) MSRL_PREP(4);
-    else if (usual && p.taps == 3 && tiles.y <= 65535) MSRL_PREP(3);
-    else if (usual && p.taps == 2 && tiles.y <= 65535) MSRL_PREP(2);
-    else delta_prep_kernel<T><<<tokens, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, qn, kn, kq, vv, g, beta);
-#undef MSRL_PREP
+    auto up4 = [](long long n) { return (n + 3) / 4 * 4; };       // every array starts on 16 bytes
+    const long long nv = up4((long long)tokens * H * vdim);
+    float *vv = scratch, *o = vv + nv;
     int e;
+    const int gslots = tokens / GRP + batch;
+    const dim3 vgrid((unsigned)((H * vdim + 1023) / 1024), (unsigned)((tokens + PREP_TT - 1) / PREP_TT));
+    const dim3 ggrid((unsigned)((H + 7) / 8), (unsigned)((gslots + 3) / 4));
+    if (grouped_shape(ints, ld, a_ld) && vgrid.y <= 65535 && ggrid.y <= 65535) {
+      float* rec = o + nv;
+      const int DP = padded_dim(dim);
+#define MSRL_PREP(N)                                                                                       \
+  do {                                                                                                     \
+    delta_value_kernel<T, N><<<vgrid, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, tokens, vv);           \
+    delta_group_kernel<T, N><<<ggrid, 256, 0, st>>>(p, cu, start_pos, slots, batch, gslots, DP, rec);        \
+  } while (0)
+      if (p.taps == 4) MSRL_PREP(4);
+      else if (p.taps == 3) MSRL_PREP(3);
+      else MSRL_PREP(2);
+#undef MSRL_PREP
+      if (DP == 32) e = launch_group_scan<4>(rec, vv, state, cu, start_pos, slots, batch, H, dim, vdim, o, st);
+      else if (DP == 64) e = launch_group_scan<8>(rec, vv, state, cu, start_pos, slots, batch, H, dim, vdim, o, st);
+      else e = launch_group_scan<16>(rec, vv, state, cu, start_pos, slots, batch, H, dim, vdim, o, st);
+    } else {
+      const long long nk = up4((long long)tokens * KVH * dim);
+      float *qn = o + nv, *kn = qn + nk, *g = kn + nk, *beta = g + up4((long long)tokens * H * dim), *kq = beta + up4((long long)tokens * H);
+      delta_prep_kernel<T><<<tokens, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, qn, kn, kq, vv, g, beta);
 #define MSRL_SCAN(D, L, C, N) launch_scan<D, L, C, N>(qn, kn, kq, vv, g, beta, state, cu, start_pos, slots, batch, H, KVH, dim, vdim, o, st)
-    if (dim <= 32) e = MSRL_SCAN(8, 4, 1, 32);
-    else if (dim <= 64) e = MSRL_SCAN(8, 8, 2, 32);
-    else if (dim <= 128) e = MSRL_SCAN(16, 8, 2, 32);
-    else e = MSRL_SCAN(32, 8, 1, 32);
+      if (dim <= 32) e = MSRL_SCAN(8, 4, 1, 32);
+      else if (dim <= 64) e = MSRL_SCAN(8, 8, 2, 32);
+      else if (dim <= 128) e = MSRL_SCAN(16, 8, 2, 32);
+      else e = MSRL_SCAN(32, 8, 1, 32);
 #undef MSRL_SCAN
+    }
     if (e) return e;
     const int channels = 2 * KVH * dim + H * vdim;
     delta_ring_kernel<T><<<dim3((unsigned)((channels + 255) / 256), (unsigned)batch), 256, 0, st>>>(p, cu, start_pos, slots);

@@ -103,21 +103,16 @@ def delta_prefill(proj: torch.Tensor, a: torch.Tensor, gate: torch.Tensor, lay: 
     in slot ``slots[b]``) -> gated, normed outputs ``[T, heads * vdim]``; ring and state are updated."""
     t, batch = proj.shape[0], cu.numel() - 1
     if _lib.use_kernels(proj, a, gate, ring, state, cu):
-        dev = proj.device
-
-        def scratch(*shape):
-            return guard.empty(*shape, device=dev, dtype=torch.float32)
-
-        qn, kn = scratch(t, lay.kv_heads, lay.dim), scratch(t, lay.kv_heads, lay.dim)
-        kq, beta = scratch(t, lay.kv_heads), scratch(t, lay.heads)
-        vv, o = scratch(t, lay.heads, lay.vdim), scratch(t, lay.heads, lay.vdim)
-        g = scratch(t, lay.heads, lay.dim)
-        y = guard.empty(t, lay.heads * lay.vdim, device=dev, dtype=proj.dtype)
-        check(_lib.load().msrl_delta_prefill(
+        L, ints = _lib.load(), lay.ints()
+        L.msrl_delta_prefill_scratch.restype = c_ll
+        n = L.msrl_delta_prefill_scratch(ints, c_ll(proj.stride(0)), c_ll(a.stride(0)), c_int(t), c_int(batch))
+        scratch = guard.empty(int(n), device=proj.device, dtype=torch.float32)
+        y = guard.empty(t, lay.heads * lay.vdim, device=proj.device, dtype=proj.dtype)
+        check(L.msrl_delta_prefill(
             ptr(proj), c_ll(proj.stride(0)), ptr(a), c_ll(a.stride(0)), ptr(w.conv), ptr(w.a_log), ptr(w.dt_bias),
-            ptr(ring), ptr(state), lay.ints(), c_float(lay.unit_eps), ptr(gate), c_ll(gate.stride(0)), ptr(w.norm),
-            c_float(eps), ptr(tok_seq), ptr(cu), ptr(start_pos), ptr(slots), c_int(t), c_int(batch), ptr(qn), ptr(kn),
-            ptr(kq), ptr(vv), ptr(g), ptr(beta), ptr(o), ptr(y), _is_f32(proj), stream()), "delta_prefill")
+            ptr(ring), ptr(state), ints, c_float(lay.unit_eps), ptr(gate), c_ll(gate.stride(0)), ptr(w.norm),
+            c_float(eps), ptr(tok_seq), ptr(cu), ptr(start_pos), ptr(slots), c_int(t), c_int(batch), ptr(scratch), ptr(y),
+            _is_f32(proj), stream()), "delta_prefill")
         return y
     return _reference(proj, a, gate, lay, w, ring, state, cu.tolist(), start_pos, slots, eps)
 
