@@ -223,7 +223,7 @@ constexpr int GRP = 4, COEF = 24;
 __host__ __device__ constexpr int group_floats(int dp) { return 13 * dp + COEF; }
 
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 delta_group_kernel(const DeltaIn<T> p, const int* cu, const int* start_pos, const long long* slots, int batch,
                    int total_slots, int DP, float* rec) {
   const int lane = threadIdx.x & 31, h = blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -557,15 +557,16 @@ delta_scan_kernel(const float* qn, const float* kn, const float* kq, const float
 }
 
 // ---- prefill: the recurrence over groups of four tokens ------------------------------------------------
-// Same lane layout as delta_scan_kernel with LPC = 8 and two columns per thread.  A group costs one pass over the
-// state for its eight dot products and one for its four writes, and one exchange between lanes.
+// Lane layout of delta_scan_kernel with sixteen lanes on four neighbouring columns: what a thread reads of a record
+// serves four columns.  A group costs one pass over the state for its eight dot products and one for its four
+// writes, and one exchange between lanes.
 constexpr int SG = 2;            // groups staged at a time
 
 template <int DPL, int COLS>
 __global__ void __launch_bounds__(COLS * 4)
 delta_group_scan_kernel(const float* rec, const float* vv, float* state, const int* cu, const int* start_pos,
                         const long long* slots, int H, int dim, int vdim, float* o) {
-  constexpr int LPC = 8, CPT = 2, DP = DPL * LPC, THREADS = COLS / CPT * LPC, CH = group_floats(DP);
+  constexpr int LPC = 16, CPT = 4, DP = DPL * LPC, THREADS = COLS / CPT * LPC, CH = group_floats(DP);
   constexpr int BUF = SG * (CH + GRP * COLS);
   extern __shared__ __align__(16) float sm[];            // two buffers of SG x [record | v of four tokens]
   const int h = blockIdx.y, b = blockIdx.z, c0 = blockIdx.x * COLS;
@@ -641,7 +642,7 @@ delta_group_scan_kernel(const float* rec, const float* vv, float* state, const i
             acc[v][c] = fma2(s[c][2 * m + 1], w.y, acc[v][c]);
           }
         }
-      // sums over the eight lanes: lane l ends with value l of both columns
+      // sums over the sixteen lanes: lane l ends with value l / 2 of columns 2 (l % 2) and 2 (l % 2) + 1
       float val[2 * GRP][CPT];
 #pragma unroll
       for (int v = 0; v < 2 * GRP; ++v)
@@ -652,14 +653,20 @@ delta_group_scan_kernel(const float* rec, const float* vv, float* state, const i
         }
 #pragma unroll
       for (int half = 4; half > 0; half >>= 1) {
-        const bool up = lr & half;
+        const bool up = lr & (2 * half);
 #pragma unroll
         for (int v = 0; v < half; ++v)
 #pragma unroll
           for (int c = 0; c < CPT; ++c) {
             const float mine = up ? val[v + half][c] : val[v][c], theirs = up ? val[v][c] : val[v + half][c];
-            val[v][c] = mine + __shfl_xor_sync(0xffffffffu, theirs, half);
+            val[v][c] = mine + __shfl_xor_sync(0xffffffffu, theirs, 2 * half);
           }
+      }
+      float two[2];
+#pragma unroll
+      for (int c = 0; c < 2; ++c) {
+        const float mine = lr & 1 ? val[0][c + 2] : val[0][c], theirs = lr & 1 ? val[0][c] : val[0][c + 2];
+        two[c] = mine + __shfl_xor_sync(0xffffffffu, theirs, 1);
       }
       // every lane solves for the four writes
       float u[GRP][CPT];
@@ -668,7 +675,7 @@ delta_group_scan_kernel(const float* rec, const float* vv, float* state, const i
         const float bt = co[16 + j];
 #pragma unroll
         for (int c = 0; c < CPT; ++c) {
-          float t = r[CH + j * COLS + col_l + c] - __shfl_sync(0xffffffffu, val[0][c], j, 8);
+          float t = r[CH + j * COLS + col_l + c] - __shfl_sync(0xffffffffu, two[c & 1], 2 * j + (c >> 1), LPC);
 #pragma unroll
           for (int i = 0; i < j; ++i) t -= co[j * (j - 1) / 2 + i] * u[i][c];
           u[j][c] = bt * t;
@@ -693,20 +700,19 @@ delta_group_scan_kernel(const float* rec, const float* vv, float* state, const i
           }
         }
       }
-      // lane 4 + j holds p_j and writes token j
-      const int j = lr - GRP;
+      // lanes 8 + 2 j and 9 + 2 j hold p_j and write token j
+      const int j = lr / 2 - GRP, cp = 2 * (lr & 1);
       if (j >= 0 && gi * GRP + j < len) {
         const float* bj = co + 6 + j * (j + 1) / 2;
-        float y[CPT] = {val[0][0], val[0][1]};
 #pragma unroll
         for (int i = 0; i < GRP; ++i)
           if (i <= j) {
             const float w = bj[i];
-            y[0] += w * u[i][0];
-            y[1] += w * u[i][1];
+            two[0] += w * (cp ? u[i][2] : u[i][0]);
+            two[1] += w * (cp ? u[i][3] : u[i][1]);
           }
-        float* dst = o + ((t0 + gi * GRP + j) * H + h) * vdim + col;
-        if (col + 1 < vdim) *reinterpret_cast<float2*>(dst) = make_float2(y[0], y[1]);   // vdim is a multiple of 4
+        float* dst = o + ((t0 + gi * GRP + j) * H + h) * vdim + col + cp;
+        if (col + cp + 1 < vdim) *reinterpret_cast<float2*>(dst) = make_float2(two[0], two[1]);   // vdim % 4 == 0
       }
     }
     __syncthreads();
@@ -933,7 +939,7 @@ template <int DPL>
 static int launch_group_scan(const float* rec, const float* vv, float* state, const int* cu, const int* start_pos,
                              const long long* slots, int batch, int H, int dim, int vdim, float* o, cudaStream_t st) {
   constexpr int COLS = 32;
-  const size_t smem = 2 * sizeof(float) * SG * (group_floats(DPL * 8) + GRP * COLS);
+  const size_t smem = 2 * sizeof(float) * SG * (group_floats(DPL * 16) + GRP * COLS);
   const int e = allow_smem(delta_group_scan_kernel<DPL, COLS>, smem);
   if (e) return e;
   const dim3 grid((unsigned)((vdim + COLS - 1) / COLS), (unsigned)H, (unsigned)batch);
@@ -947,7 +953,7 @@ static bool grouped_shape(const int* ints, long long ld, long long a_ld) {
   return dim % 4 == 0 && dim <= 128 && vdim % 4 == 0 && taps >= 2 && taps <= 4 && ints[5] % 4 == 0 && ints[6] % 4 == 0 &&
          ints[7] % 4 == 0 && ld % 4 == 0 && a_ld % 4 == 0;
 }
-static int padded_dim(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : 128; }
+static int padded_dim(int dim) { return dim <= 64 ? 64 : 128; }
 
 // fp32 scratch of msrl_delta_prefill
 MSRL_API long long msrl_delta_prefill_scratch(const int* ints, long long ld, long long a_ld, int tokens, int batch) {
@@ -987,9 +993,8 @@ MSRL_API int msrl_delta_prefill(const void* proj, long long ld, const void* a, l
       else if (p.taps == 3) MSRL_PREP(3);
       else MSRL_PREP(2);
 #undef MSRL_PREP
-      if (DP == 32) e = launch_group_scan<4>(rec, vv, state, cu, start_pos, slots, batch, H, dim, vdim, o, st);
-      else if (DP == 64) e = launch_group_scan<8>(rec, vv, state, cu, start_pos, slots, batch, H, dim, vdim, o, st);
-      else e = launch_group_scan<16>(rec, vv, state, cu, start_pos, slots, batch, H, dim, vdim, o, st);
+      if (DP == 64) e = launch_group_scan<4>(rec, vv, state, cu, start_pos, slots, batch, H, dim, vdim, o, st);
+      else e = launch_group_scan<8>(rec, vv, state, cu, start_pos, slots, batch, H, dim, vdim, o, st);
     } else {
       const long long nk = up4((long long)tokens * KVH * dim);
       float *qn = o + nv, *kn = qn + nk, *g = kn + nk, *beta = g + up4((long long)tokens * H * dim), *kq = beta + up4((long long)tokens * H);
