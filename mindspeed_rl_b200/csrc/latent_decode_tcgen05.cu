@@ -389,8 +389,8 @@ static int launch(const CUtensorMap& map, const void* q, const Params& p, int ba
 
 using namespace msrl;
 
-// Contract of msrl_latent_decode_mma (latent_attention.cu) without the merge of key ranges, plus the number of cache
-// blocks and a status word.  Returns cudaErrorNotSupported for shapes it does not cover.
+// The arguments of msrl_latent_decode_mma (latent_attention.cu) plus the number of cache blocks and a status word; key
+// ranges are left in part_o / part_ml for msrl_latent_decode_combine.  Returns cudaErrorNotSupported for shapes it does not cover.
 MSRL_API int msrl_latent_decode_tcgen05(const void* q, const void* cache, long long num_blocks, const int* block_tables,
                                         int max_blocks, int block_size, const int* context_lens, float scale, int batch,
                                         int H, int CP, int RP, int nsplit, float* part_o, float* part_ml, void* out,

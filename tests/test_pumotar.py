@@ -166,30 +166,32 @@ def test_looped_layers_run_in_order_with_a_cache_each():
 
 
 @pytest.mark.parametrize("device", DEVICES)
-def test_delta_recurrence_far_write(device):
+@pytest.mark.parametrize("taps", [1, 3])
+def test_delta_recurrence_far_write(device, taps):
     """A value written under a key of its own is read back unchanged many tokens later when the decay is one, and is
     lost when the key's channels decay."""
-    lay = ops.DeltaLayout(1, 1, 8, 6, 1, 0, 8, 16, 24)
-    n, far = 200, 3
+    lay = ops.DeltaLayout(1, 1, 8, 8, taps, 0, 8, 16, 24)
+    n, far = 203, 6
     proj = torch.zeros(n, 32)
     proj[:, 8 + 1] = 5.0                                   # all other tokens write under channel 1
     proj[far, 8:16] = torch.eye(8)[4] * 5.0
-    proj[far, 16:22] = torch.arange(1.0, 7.0)
+    proj[far, 16:24] = torch.arange(1.0, 9.0)
     proj[-1, 0:8] = torch.eye(8)[4] * 5.0                  # the last token asks for channel 4
     proj[:, 24] = 20.0                                     # write strength one
-    conv = torch.ones(lay.channels, 1)
-    gate = torch.full((n, 6), 30.0)
+    conv = torch.zeros(lay.channels, taps)
+    conv[:, -1] = 1.0                                      # the current token only
+    gate = torch.full((n, 8), 30.0)
     for decay, keeps in ((-40.0, True), (3.0, False)):
-        w = ops.DeltaWeights(conv, torch.zeros(1), torch.full((8,), decay), torch.ones(6))
-        ring, state = torch.zeros(2, 1, lay.channels), torch.zeros(2, 1, 8, 6)
+        w = ops.DeltaWeights(conv, torch.zeros(1), torch.full((8,), decay), torch.ones(8))
+        ring, state = torch.zeros(2, taps, lay.channels), torch.zeros(2, 1, 8, 8)
         t = dict(device=device)
         cu = torch.tensor([0, n], dtype=torch.int32)
         out = ops.delta_prefill(proj.to(**t), torch.zeros(n, 8, **t), gate.to(**t), lay,
                                 ops.DeltaWeights(*(x.to(**t) for x in (w.conv, w.a_log, w.dt_bias, w.norm))), ring.to(**t),
                                 state.to(**t), torch.zeros(n, dtype=torch.int32, **t), cu.to(**t),
                                 torch.zeros(1, dtype=torch.int32, **t), torch.tensor([1], **t), 1e-6)
-        v = O.silu(torch.arange(1.0, 7.0).double())
-        want = v / v.pow(2).mean().sqrt() if keeps else torch.zeros(6).double()
+        v = O.silu(torch.arange(1.0, 9.0).double())
+        want = v / v.pow(2).mean().sqrt() if keeps else torch.zeros(8).double()
         assert torch.allclose(out[-1].double().cpu(), want, atol=2e-4), (decay, out[-1])
 
 
@@ -274,6 +276,21 @@ def test_single_tokens_from_the_start(device):
 
 
 @pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("case", ["latent", "delta_grouped"])
+def test_one_kind_of_layer_only(device, case):
+    """A model without recurrent layers takes no state slots, one without attention no cache memory."""
+    cfg = M.config([(MIXER_CASES[case], M.moe()), (MIXER_CASES[case], None)], loop=(1, 2, 2))
+    w = M.weights(cfg, 8)
+    seq = M.tokens(40, cfg["vocab"])
+    want = O.forward(cfg, w, seq)
+    eng = make_engine(None, device, cfg=cfg, w=w, graphs=(1,) if device == "cuda" else ())
+    assert (eng.state_slots is None) == (case == "latent") and (eng.kv_bytes_per_block() == 0) == (case != "latent")
+    close(run_schedule(eng, seq, [11, 6, 1]), want)
+    out = eng.generate([seq[:9]], SamplingParams(n=2, temperature=0.0, max_tokens=5))[0].outputs
+    assert out[0].token_ids == out[1].token_ids and out[0].token_ids[0] == int(want[8].argmax())
+
+
+@pytest.mark.parametrize("device", DEVICES)
 def test_long_decoding(device):
     n = 220
     eng = make_engine("mixed", device, graphs=(1, 2) if device == "cuda" else ())
@@ -298,10 +315,10 @@ def _peaked(n, lay, target, seed=0):
 
 
 @pytest.mark.parametrize("device", DEVICES)
-@pytest.mark.parametrize("heads,rank,dr", [(3, 24, 8), (20, 72, 16), (40, 130, 24), (70, 40, 16), (4, 300, 32)])
-def test_decode_attention_keys_at_borders(device, heads, rank, dr):
+@pytest.mark.parametrize("heads,rank,dr,bs", [(3, 24, 8, 16), (20, 72, 16, 8), (40, 130, 24, 32), (70, 40, 16, 64), (4, 300, 32, 4)])
+def test_decode_attention_keys_at_borders(device, heads, rank, dr, bs):
     lay = ops.LatentLayout(heads, 8, dr, 8, rank, 8 + dr, 8, 0, dr)
-    bs, n = 16, 333
+    n = 333
     blocks = (n + bs - 1) // bs
     for dtype in (torch.float32,) if device == "cpu" else (torch.float32, torch.bfloat16):
         targets = [0, 15, 16, 31, 63, 64, 127, 128, 200, n - 2, n - 1]
