@@ -33,6 +33,7 @@ struct AttnParams {
   float scale;             // 1/sqrt(D)
   float scale_log2;        // scale * log2(e)
   int causal;
+  int window;                 // forward: keys a query sees, itself included (0: all)
   // backward only
   const __nv_bfloat16* dout;  // same layout as o
   float* delta;               // [nh, Tq] rowsum(dO * O)
@@ -65,14 +66,15 @@ __global__ void __launch_bounds__(128) fa_fwd_kernel(const AttnParams p) {
   int kmax = klen;
   if (p.causal) kmax = min(klen, m0 + BM + off);
   const int n_tiles = (kmax + BN - 1) / BN;
+  const int t0 = p.window > 0 ? max(m0 + off - p.window + 1, 0) / BN : 0;    // first tile inside any row's window
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int qrow = lane >> 2, qcol = (lane & 3) * 2;
 
   load_tile_async<BM, D, LD, THREADS>(sQ, p.q, p.Lq, h, q0, m0, qlen);
-  if (n_tiles > 0) {
-    load_tile_async<BN, D, LD, THREADS>(sK, p.k, p.Lk, hk, k0, 0, klen);
-    load_tile_async<BN, D, LD, THREADS>(sV, p.v, p.Lv, hk, k0, 0, klen);
+  if (n_tiles > t0) {
+    load_tile_async<BN, D, LD, THREADS>(sK, p.k, p.Lk, hk, k0, t0 * BN, klen);
+    load_tile_async<BN, D, LD, THREADS>(sV, p.v, p.Lv, hk, k0, t0 * BN, klen);
   }
   cp_async_commit();
 
@@ -84,8 +86,8 @@ __global__ void __launch_bounds__(128) fa_fwd_kernel(const AttnParams p) {
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.f, 0.f};
 
-  for (int it = 0; it < n_tiles; ++it) {
-    const int st = it & 1;
+  for (int it = t0; it < n_tiles; ++it) {
+    const int st = (it - t0) & 1;
     if (it + 1 < n_tiles) {
       load_tile_async<BN, D, LD, THREADS>(sK + (st ^ 1) * BN * LD, p.k, p.Lk, hk, k0, (it + 1) * BN, klen);
       load_tile_async<BN, D, LD, THREADS>(sV + (st ^ 1) * BN * LD, p.v, p.Lv, hk, k0, (it + 1) * BN, klen);
@@ -121,7 +123,8 @@ __global__ void __launch_bounds__(128) fa_fwd_kernel(const AttnParams p) {
 
     // mask + online softmax (exp2 domain)
     const int kbase = it * BN;
-    const bool need_mask = (kbase + BN > klen) || (p.causal && (kbase + BN - 1 > m0 + off));
+    const bool need_mask = (kbase + BN > klen) || (p.causal && (kbase + BN - 1 > m0 + off)) ||
+                           (p.window > 0 && kbase <= m0 + BM - 1 + off - p.window);
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int nt = 0; nt < BN / 8; ++nt) {
@@ -131,7 +134,8 @@ __global__ void __launch_bounds__(128) fa_fwd_kernel(const AttnParams p) {
         if (need_mask) {
           const int key = kbase + nt * 8 + qcol + (j & 1);
           const int row = m0 + warp * 16 + qrow + ((j >> 1) << 3);
-          const bool ok = (key < klen) && (!p.causal || key <= row + off);
+          const bool ok = (key < klen) && (!p.causal || key <= row + off) &&
+                          (p.window <= 0 || key > row + off - p.window);
           v = ok ? v : -INFINITY;
         }
         s[nt][j] = v;
@@ -594,12 +598,13 @@ MSRL_API int msrl_flash_attn_varlen_fwd(const void* q, const void* k, const void
                                         const long long* layouts12, void* o, long long o_stride_t,
                                         float* lse, const int* cu_q, const int* cu_k, int batch,
                                         int max_q, int nh, int nkv, long long Tq, int D,
-                                        float scale, int causal, cudaStream_t st) {
+                                        float scale, int causal, int window, cudaStream_t st) {
   if (batch == 0 || Tq == 0) return 0;
-  if (nh % nkv != 0) return (int)cudaErrorInvalidValue;
+  if (nh % nkv != 0 || (window > 0 && !causal)) return (int)cudaErrorInvalidValue;
   AttnParams p = make_params(q, k, v, layouts12, o, o_stride_t, lse, cu_q, cu_k, nh, nkv, Tq, D, causal);
   p.scale = scale;
   p.scale_log2 = scale * kLog2e;
+  p.window = window;
   if (D == 128) return launch_fwd<128>(p, batch, max_q, st);
   if (D == 64) return launch_fwd<64>(p, batch, max_q, st);
   return (int)cudaErrorInvalidValue;

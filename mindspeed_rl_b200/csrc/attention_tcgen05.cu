@@ -52,6 +52,7 @@ struct Params {
   long long Tq;
   float scale_log2;
   int causal;
+  int window;                                          // keys a query sees, itself included (0: all)
   int q_col0, q_group_stride, q_hpg, q_head_stride;    // column of head h inside a row of the Q tensor map
   int k_col0, k_group_stride, k_hpg, k_head_stride;
   int v_col0, v_group_stride, v_hpg, v_head_stride;
@@ -89,7 +90,9 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const int off = klen - qlen;
   int kmax = klen;
   if (p.causal) kmax = min(klen, m0 + BM + off);
-  const int n_tiles = kmax > 0 ? (kmax + BN - 1) / BN : 0;
+  // tiles [t0, t0 + n_tiles): those inside some row's window
+  const int t0 = p.window > 0 ? max(m0 + off - p.window + 1, 0) / BN : 0;
+  const int n_tiles = max((max(kmax, 0) + BN - 1) / BN - t0, 0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   {
     // the tiles must fit behind the 1024-byte alignment of the dynamic segment (the launch leaves
@@ -146,13 +149,13 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         mbar_expect_tx(&k_full[st], K_BYTES);
         unsigned char* sk = smem + SMEM_K + st * K_BYTES;
 #pragma unroll
-        for (int i = 0; i < NQK; ++i) tma_load_2d(sk + i * KV_HALF, &map_k, &k_full[st], kc + i * 64, k0 + j * BN);
+        for (int i = 0; i < NQK; ++i) tma_load_2d(sk + i * KV_HALF, &map_k, &k_full[st], kc + i * 64, k0 + (t0 + j) * BN);
         if (use > 0) ok = mbar_wait(&v_empty[st], (use - 1) & 1, p.error, ERR_EMPTY);
         if (!ok) break;
         mbar_expect_tx(&v_full[st], KV_BYTES);
         unsigned char* sv = smem + SMEM_V + st * KV_BYTES;
-        tma_load_2d(sv, &map_v, &v_full[st], vc, k0 + j * BN);
-        tma_load_2d(sv + KV_HALF, &map_v, &v_full[st], vc + 64, k0 + j * BN);
+        tma_load_2d(sv, &map_v, &v_full[st], vc, k0 + (t0 + j) * BN);
+        tma_load_2d(sv + KV_HALF, &map_v, &v_full[st], vc + 64, k0 + (t0 + j) * BN);
       }
     }
   } else if (warp == MMA_WARP) {
@@ -218,9 +221,11 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       ok = mbar_wait_warp(&s_full[sb], (j >> 1) & 1, p.error, ERR_S);
       if (!ok) break;
       fence_after();
-      const int kbase = j * BN;
-      const bool need_mask = (kbase + BN > klen) || (p.causal && (kbase + BN - 1 > m0 + off));
-      const int limit = min(klen, p.causal ? grow + off + 1 : klen) - kbase;   // valid columns of this row
+      const int kbase = (t0 + j) * BN;
+      const bool need_mask = (kbase + BN > klen) || (p.causal && (kbase + BN - 1 > m0 + off)) ||
+                             (p.window > 0 && kbase <= m0 + BM - 1 + off - p.window);
+      const int limit = min(klen, p.causal ? grow + off + 1 : klen) - kbase;   // valid columns of this row: [from, limit)
+      const int from = p.window > 0 ? grow + off + 1 - p.window - kbase : 0;
       float s[HALF], t[32];
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
       // the other half: maximum only
@@ -230,7 +235,7 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         tmem_ld32(tmem + lane_base + sb * BN + col0, t);
         if (need_mask) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i) t[i] = (col0 + i < limit) ? t[i] : -INFINITY;
+          for (int i = 0; i < 32; ++i) t[i] = (col0 + i < limit && col0 + i >= from) ? t[i] : -INFINITY;
         }
 #pragma unroll
         for (int i = 0; i < 32; i += 4) {
@@ -248,7 +253,7 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           float v = t[i];
-          if (need_mask) v = (col0 + i < limit) ? v : -INFINITY;
+          if (need_mask) v = (col0 + i < limit && col0 + i >= from) ? v : -INFINITY;
           s[c * 32 + i] = v;
         }
 #pragma unroll
@@ -877,8 +882,10 @@ MSRL_API int msrl_flash_attn_varlen_fwd_tcgen05(const void* q, const void* k, co
                                                 const long long* lay, void* o, long long o_stride_t,
                                                 float* lse, const int* cu_q, const int* cu_k, int batch,
                                                 int max_q, int nh, int nkv, long long Tq, long long Tk,
-                                                int D, float scale, int causal, int* error, cudaStream_t st) {
+                                                int D, float scale, int causal, int window, int* error,
+                                                cudaStream_t st) {
   if (batch == 0 || Tq == 0) return 0;
+  if (window > 0 && !causal) return (int)cudaErrorInvalidValue;
   if ((D != fa5::D && D != 192) || nh % nkv != 0 || (o_stride_t % 8) != 0 || (reinterpret_cast<uintptr_t>(o) & 15) != 0)
     return (int)cudaErrorNotSupported;
   for (int i = 0; i < 3; ++i) {
@@ -907,6 +914,7 @@ MSRL_API int msrl_flash_attn_varlen_fwd_tcgen05(const void* q, const void* k, co
   p.Tq = Tq;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.causal = causal;
+  p.window = window;
   p.q_col0 = 0; p.q_group_stride = (int)lay[1]; p.q_hpg = (int)lay[2]; p.q_head_stride = (int)lay[3];
   p.k_col0 = 0; p.k_group_stride = (int)lay[5]; p.k_hpg = (int)lay[6]; p.k_head_stride = (int)lay[7];
   p.v_col0 = 0; p.v_group_stride = (int)lay[9]; p.v_hpg = (int)lay[10]; p.v_head_stride = (int)lay[11];

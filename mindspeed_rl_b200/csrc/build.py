@@ -31,17 +31,18 @@ NVCC_FLAGS = [
 ]
 # kernels whose results are specified in 32-bit (an fp32 residual, recurrent state, fp32 attention): compiled
 # without the approximate divisions, square roots, exponentials and flush-to-zero of --use_fast_math
-PRECISE = {"residual_stream", "delta_rule", "latent_attention", "latent_decode_tcgen05",
-           "grouped_gemm_simt"}
+PRECISE = {"residual_stream", "delta_rule", "latent_attention", "latent_decode_tcgen05", "grouped_gemm_simt",
+           "matrix_memory", "qkv_prep", "attention_simt", "moe"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 
-# kernels of one use, linked into a library of their own (``_C/libmsrl_<group>.so``): a process that serves one
-# model family from a fresh checkout compiles these and nothing else.  hybrid: the forward of layer-by-layer decoders
-# (without the sampler)
+# kernels of one model family, linked into a library of their own (``_C/libmsrl_<group>.so``): a process that serves the
+# family from a fresh checkout compiles these and nothing else (the forward of the family, without the sampler)
+_STREAM = ("residual_stream", "grouped_gemm_simt", "moe", "moe_gemm_tcgen05", "attention", "attention_tcgen05", "attention_simt",
+           "paged_rows", "gemm2cta_tcgen05")
 GROUPS = {
-    "hybrid": ("residual_stream", "delta_rule", "latent_attention", "latent_decode_tcgen05", "grouped_gemm_simt", "moe", "moe_gemm_tcgen05",
-               "attention", "attention_tcgen05", "gemm2cta_tcgen05"),
+    "pumotar": (*_STREAM, "delta_rule", "latent_attention", "latent_decode_tcgen05"),
+    "sunatar": (*_STREAM, "matrix_memory", "qkv_prep", "decode", "decode_prefix_tcgen05"),
 }
 
 

@@ -90,43 +90,49 @@ struct DecodeParams {
   const int* group_prefix;  // [n_groups] shared keys of the group
   int npre;                 // prefix splits (slots 0 .. npre-1)
   int block_shift;          // log2(block_size), or -1 when it is not a power of two
+  int window;               // keys a query sees, itself included (0: all)
 };
 
 constexpr int kGroupMax = 8;
 
-template <int D>
+// Query / key heads of DK and value heads of DV entries.  A CTA serves 16 query heads of a KV group; larger groups take
+// several (blockIdx.y = KV head x head tile).
+template <int DK, int DV>
 __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p) {
-  constexpr int CH = 64, LD = D + 8, THREADS = 128;
+  constexpr int CH = 64, LD = DK + 8, LDV = DV + 8, THREADS = 128;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem_raw);  // 16 x LD
   __nv_bfloat16* sK = sQ + 16 * LD;                                 // 2 x CH x LD
-  __nv_bfloat16* sV = sK + 2 * CH * LD;                             // 2 x CH x LD
+  __nv_bfloat16* sV = sK + 2 * CH * LD;                             // 2 x CH x LDV
 
-  const int b = blockIdx.x, hk = blockIdx.y, sp = blockIdx.z;
-  const int rep = p.nh / p.nkv;
+  const int group = p.nh / p.nkv, tiles = (group + 15) / 16;
+  const int b = blockIdx.x, hk = blockIdx.y / tiles, sp = blockIdx.z;
+  const int h0 = hk * group + blockIdx.y % tiles * 16, rep = min(group - blockIdx.y % tiles * 16, 16);
   const int ctx = p.context_lens[b];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int frow = lane >> 2, fcol = (lane & 3) * 2;
 
-  const int k0 = (p.key_start != nullptr) ? min(p.key_start[b], ctx) : 0;
+  const int k0 = (p.key_start != nullptr) ? min(p.key_start[b], ctx)
+                                               : (p.window > 0 ? max(ctx - p.window, 0) : 0);
   int per_split = (ctx - k0 + p.nsplit - 1) / p.nsplit;
   per_split = ((per_split + CH - 1) / CH) * CH;
   const int kbeg = k0 + sp * per_split;
   const int kend = min(ctx, kbeg + per_split);
   const int n_chunks = (kend > kbeg) ? (kend - kbeg + CH - 1) / CH : 0;
 
-  // Q rows: the `rep` heads of this KV group; rows >= rep are zero
-  for (int i = threadIdx.x; i < 16 * (D / 8); i += THREADS) {
-    const int r = i / (D / 8), c = i % (D / 8);
+  // Q rows: `rep` heads of this KV group; rows >= rep are zero
+  for (int i = threadIdx.x; i < 16 * (DK / 8); i += THREADS) {
+    const int r = i / (DK / 8), c = i % (DK / 8);
     const bool ok = r < rep;
-    const __nv_bfloat16* src = p.q + head_offset(p.Lq, b, hk * rep + (ok ? r : 0)) + c * 8;
+    const __nv_bfloat16* src = p.q + head_offset(p.Lq, b, h0 + (ok ? r : 0)) + c * 8;
     cp_async16(sQ + r * LD + c * 8, src, ok);
   }
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
   auto issue = [&](int chunk, int stage) {
     const int base = kbeg + chunk * CH;
-    for (int i = threadIdx.x; i < CH * (D / 8); i += THREADS) {
-      const int r = i / (D / 8), c = i % (D / 8);
+    constexpr int VEC = (DK > DV ? DK : DV) / 8;
+    for (int i = threadIdx.x; i < CH * VEC; i += THREADS) {
+      const int r = i / VEC, c = i % VEC;
       const int key = base + r;
       const bool ok = key < kend;
       const int kk = ok ? key : kbeg;
@@ -138,17 +144,17 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p)
         blk = __ldg(bt + kk / p.block_size);
         off = kk % p.block_size;
       }
-      const long long src = (((long long)blk * p.block_size + off) * p.nkv + hk) * D + c * 8;
-      cp_async16(sK + (stage * CH + r) * LD + c * 8, p.k_cache + src, ok);
-      cp_async16(sV + (stage * CH + r) * LD + c * 8, p.v_cache + src, ok);
+      const long long row = ((long long)blk * p.block_size + off) * p.nkv + hk;
+      if (DK >= DV || c < DK / 8) cp_async16(sK + (stage * CH + r) * LD + c * 8, p.k_cache + row * DK + c * 8, ok);
+      if (DV >= DK || c < DV / 8) cp_async16(sV + (stage * CH + r) * LDV + c * 8, p.v_cache + row * DV + c * 8, ok);
     }
   };
   if (n_chunks > 0) issue(0, 0);
   cp_async_commit();
 
-  float o_acc[D / 8][4];
+  float o_acc[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i)
+  for (int i = 0; i < DV / 8; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) o_acc[i][j] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
@@ -164,10 +170,10 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p)
     }
     __syncthreads();
     const __nv_bfloat16* tK = sK + (st * CH + warp * 16) * LD;  // this warp's 16 keys
-    const __nv_bfloat16* tV = sV + (st * CH + warp * 16) * LD;
+    const __nv_bfloat16* tV = sV + (st * CH + warp * 16) * LDV;
     float s[2][4] = {{0, 0, 0, 0}, {0, 0, 0, 0}};
 #pragma unroll
-    for (int kk = 0; kk < D / 16; ++kk) {
+    for (int kk = 0; kk < DK / 16; ++kk) {
       uint32_t a[4], bfr[4];
       ldmatrix_x4(a, smem_u32(sQ + (lane & 15) * LD + kk * 16 + (lane >> 4) * 8));
       ldmatrix_x4(bfr, smem_u32(tK + ((lane & 7) + (lane >> 4) * 8) * LD + kk * 16 + ((lane >> 3) & 1) * 8));
@@ -212,9 +218,9 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p)
     a[2] = pack_bf16(s[1][0], s[1][1]);
     a[3] = pack_bf16(s[1][2], s[1][3]);
 #pragma unroll
-    for (int dp = 0; dp < D / 16; ++dp) {
+    for (int dp = 0; dp < DV / 16; ++dp) {
       uint32_t bfr[4];
-      ldmatrix_x4_trans(bfr, smem_u32(tV + (lane & 15) * LD + dp * 16 + (lane >> 4) * 8));
+      ldmatrix_x4_trans(bfr, smem_u32(tV + (lane & 15) * LDV + dp * 16 + (lane >> 4) * 8));
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         o_acc[2 * dp][j] *= corr[0];
@@ -236,8 +242,8 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p)
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
   }
-  float* sO = reinterpret_cast<float*>(sK);        // [4][16][D]
-  float* sM = sO + 4 * 16 * D;                     // [4][16]
+  float* sO = reinterpret_cast<float*>(sK);        // [4][16][DV]
+  float* sM = sO + 4 * 16 * DV;                     // [4][16]
   float* sL = sM + 4 * 16;                         // [4][16]
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
@@ -247,14 +253,14 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p)
       sL[warp * 16 + row] = l_run[r];
     }
 #pragma unroll
-    for (int dt = 0; dt < D / 8; ++dt) {
-      sO[(warp * 16 + row) * D + dt * 8 + fcol] = o_acc[dt][2 * r];
-      sO[(warp * 16 + row) * D + dt * 8 + fcol + 1] = o_acc[dt][2 * r + 1];
+    for (int dt = 0; dt < DV / 8; ++dt) {
+      sO[(warp * 16 + row) * DV + dt * 8 + fcol] = o_acc[dt][2 * r];
+      sO[(warp * 16 + row) * DV + dt * 8 + fcol + 1] = o_acc[dt][2 * r + 1];
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < rep * D; i += THREADS) {
-    const int r = i / D, d = i % D;
+  for (int i = threadIdx.x; i < rep * DV; i += THREADS) {
+    const int r = i / DV, d = i % DV;
     float m = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) m = fmaxf(m, sM[w * 16 + r]);
@@ -264,15 +270,15 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p)
     for (int w = 0; w < 4; ++w) {
       const float c = exp2f(sM[w * 16 + r] - mu);
       l += sL[w * 16 + r] * c;
-      o += sO[(w * 16 + r) * D + d] * c;
+      o += sO[(w * 16 + r) * DV + d] * c;
     }
-    const int h = hk * rep + r;
+    const int h = h0 + r;
     if (p.slot_total == 1) {
-      p.out[(long long)b * p.out_stride + (long long)h * D + d] =
+      p.out[(long long)b * p.out_stride + (long long)h * DV + d] =
           __float2bfloat16(l > 0.f ? o / l : 0.f);
     } else {
       const long long pi = ((long long)b * p.nh + h) * p.slot_total + p.slot_base + sp;
-      p.part_o[pi * D + d] = o;
+      p.part_o[pi * DV + d] = o;
       if (d == 0) {
         p.part_ml[pi * 2] = m;
         p.part_ml[pi * 2 + 1] = l;
@@ -933,13 +939,13 @@ static int launch_paged_decode(const void* q, const long long* q_layout4, const 
     if (e != cudaSuccess) return (int)e;
   }
   if (D == 128) {
-    e = cudaFuncSetAttribute(paged_decode_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    e = cudaFuncSetAttribute(paged_decode_kernel<128, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    paged_decode_kernel<128><<<grid, 128, smem, st>>>(p);
+    paged_decode_kernel<128, 128><<<grid, 128, smem, st>>>(p);
   } else {
-    e = cudaFuncSetAttribute(paged_decode_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    e = cudaFuncSetAttribute(paged_decode_kernel<64, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    paged_decode_kernel<64><<<grid, 128, smem, st>>>(p);
+    paged_decode_kernel<64, 64><<<grid, 128, smem, st>>>(p);
   }
   e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
@@ -960,6 +966,52 @@ MSRL_API int msrl_paged_decode(const void* q, const long long* q_layout4, const 
   return launch_paged_decode(q, q_layout4, k_cache, v_cache, block_tables, max_blocks, context_lens, out,
                              out_stride, part_o, part_ml, B, nh, nkv, D, block_size, nsplit, nullptr, nullptr,
                              nullptr, 0, 0, st);
+}
+
+template <int DK, int DV>
+static int launch_window_decode(const DecodeParams& p, int B, cudaStream_t st) {
+  constexpr size_t smem = (size_t)(16 * (DK + 8) + 128 * (DK + 8) + 128 * (DV + 8)) * sizeof(__nv_bfloat16);
+  const cudaError_t e = cudaFuncSetAttribute(paged_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e != cudaSuccess) return (int)e;
+  const int tiles = (p.nh / p.nkv + 15) / 16;
+  paged_decode_kernel<DK, DV><<<dim3((unsigned)B, (unsigned)(p.nkv * tiles), (unsigned)p.nsplit), 128, smem, st>>>(p);
+  if (p.nsplit > 1)
+    paged_decode_merge_kernel<DV><<<(unsigned)(((long long)B * p.nh + 3) / 4), 128, 0, st>>>(p, B);
+  return (int)cudaGetLastError();
+}
+
+// One query per sequence over the last `window` (0: all) cached keys: k_cache [blocks, block_size, nkv, dk], v_cache
+// [.., dv], any group size, explicit scale.  part_o [B, nh, nsplit, dv] and part_ml [B, nh, nsplit, 2]: scratch.
+MSRL_API int msrl_paged_decode_window(const void* q, const long long* q_layout4, const void* k_cache, const void* v_cache,
+                                      const int* block_tables, int max_blocks, const int* context_lens, void* out,
+                                      long long out_stride, float* part_o, float* part_ml, int B, int nh, int nkv, int dk,
+                                      int dv, int block_size, float scale, int window, int nsplit, cudaStream_t st) {
+  if (B == 0) return 0;
+  if (nh % nkv != 0 || nsplit < 1 || nsplit > 65535) return (int)cudaErrorInvalidValue;
+  DecodeParams p{};
+  p.slot_total = nsplit;
+  p.q = (const __nv_bfloat16*)q;
+  p.Lq = HeadLayout{q_layout4[0], (int)q_layout4[1], (int)q_layout4[2], (int)q_layout4[3]};
+  p.k_cache = (const __nv_bfloat16*)k_cache;
+  p.v_cache = (const __nv_bfloat16*)v_cache;
+  p.block_tables = block_tables;
+  p.context_lens = context_lens;
+  p.out = (__nv_bfloat16*)out;
+  p.out_stride = out_stride;
+  p.part_o = part_o;
+  p.part_ml = part_ml;
+  p.max_blocks = max_blocks;
+  p.block_size = block_size;
+  p.block_shift = (block_size & (block_size - 1)) == 0 ? __builtin_ctz(block_size) : -1;
+  p.nh = nh;
+  p.nkv = nkv;
+  p.nsplit = nsplit;
+  p.scale_log2 = scale * kLog2eD;
+  p.window = window;
+  if (dk == 128 && dv == 128) return launch_window_decode<128, 128>(p, B, st);
+  if (dk == 64 && dv == 64) return launch_window_decode<64, 64>(p, B, st);
+  if (dk == 192 && dv == 128) return launch_window_decode<192, 128>(p, B, st);
+  return (int)cudaErrorNotSupported;
 }
 
 MSRL_API int msrl_paged_decode_group_max(int nh, int nkv) {

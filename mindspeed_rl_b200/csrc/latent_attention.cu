@@ -8,9 +8,7 @@
 //   prep        RMS norm of the latent, interleaved rotation of the shared key part and of every head's query
 //               part (fp32), cache write; the row also goes to `lat` (prompts), the rotated query part to the
 //               decode query
-//   gather      cache rows of given (sequence, position) pairs, for prompt portions after the first
 //   spread      the rotated key part into every head's expanded key
-//   attn_simt   soft-max attention of packed sequences for any head sizes, fp32 arithmetic
 //   decode_simt one query per sequence over the paged rows, any sizes, fp32 arithmetic
 //   decode_mma  the same on the legacy tensor path for bf16 (block sizes that latent_decode_tcgen05.cu does not
 //               take): a block takes 16 / 32 / 64 heads of one sequence and a range of its keys, so that a row is
@@ -162,17 +160,6 @@ __global__ void __launch_bounds__(256) prep_kernel(const PrepArgs<T> p) {
   }
 }
 
-// rows of 16-byte vectors
-__global__ void gather_kernel(const uint4* cache, const int* block_tables, int max_blocks, int block_size,
-                              const int* token_seq, const int* token_pos, uint4* out, long long rows, int vecs) {
-  const long long r = (long long)blockIdx.x * (blockDim.x / 32) + (threadIdx.x >> 5);
-  if (r >= rows) return;
-  const int pos = token_pos[r];
-  const long long slot = (long long)block_tables[(long long)token_seq[r] * max_blocks + pos / block_size] * block_size +
-                         pos % block_size;
-  for (int c = threadIdx.x & 31; c < vecs; c += 32) out[r * vecs + c] = cache[slot * vecs + c];
-}
-
 // kv[t, h * stride + dn + d] = lat[t, RP + d]
 template <typename T>
 __global__ void spread_kernel(const T* lat, int CP, int RP, T* kv, long long ld, int H, int stride, int dn, int dr,
@@ -190,106 +177,6 @@ __global__ void spread_kernel(const T* lat, int CP, int RP, T* kv, long long ld,
   }
   for (int i = threadIdx.x; i < H * dr; i += blockDim.x)
     kv[t * ld + (i / dr) * stride + dn + i % dr] = lat[t * CP + RP + i % dr];
-}
-
-// ---- soft-max attention of packed sequences on the CUDA cores ------------------------------------------
-template <typename T>
-struct SimtArgs {
-  const T *q, *k, *v;
-  long long q_ld, k_ld, v_ld;
-  int q_stride, k_stride, v_stride;      // head strides
-  int dq, dv;
-  const int *cu_q, *cu_k;
-  float scale;
-  T* out;                                // [tokens, H * o_stride]
-  long long o_ld;
-  int o_stride;
-};
-
-constexpr int SB = 32;                   // query rows and keys per tile
-
-template <typename T, int ACC>
-__global__ void __launch_bounds__(256) attn_simt_kernel(const SimtArgs<T> p) {
-  extern __shared__ float smf[];
-  const int ldq = p.dq + 1;
-  float* sQ = smf;
-  float* sK = sQ + SB * ldq;
-  float* sV = sK + SB * ldq;
-  float* sP = sV + SB * p.dv;            // [SB][SB + 1]
-  const int h = blockIdx.y, b = blockIdx.z;
-  const int q0 = p.cu_q[b], qlen = p.cu_q[b + 1] - q0, k0 = p.cu_k[b], klen = p.cu_k[b + 1] - k0;
-  const int m0 = blockIdx.x * SB;
-  if (m0 >= qlen) return;
-  const int off = klen - qlen;           // bottom-right aligned causal mask
-  const int row = threadIdx.x >> 3, part = threadIdx.x & 7;
-  for (int i = threadIdx.x; i < SB * p.dq; i += 256) {
-    const int r = i / p.dq, d = i % p.dq;
-    sQ[r * ldq + d] = m0 + r < qlen ? ldf(p.q + (long long)(q0 + m0 + r) * p.q_ld + h * p.q_stride + d) : 0.f;
-  }
-  float acc[ACC];
-#pragma unroll
-  for (int i = 0; i < ACC; ++i) acc[i] = 0.f;
-  float m_run = -INFINITY, l_run = 0.f;
-  const int kmax = min(klen, m0 + SB + off);
-  for (int kb = 0; kb < kmax; kb += SB) {
-    __syncthreads();
-    for (int i = threadIdx.x; i < SB * p.dq; i += 256) {
-      const int r = i / p.dq, d = i % p.dq;
-      sK[r * ldq + d] = kb + r < klen ? ldf(p.k + (long long)(k0 + kb + r) * p.k_ld + h * p.k_stride + d) : 0.f;
-    }
-    for (int i = threadIdx.x; i < SB * p.dv; i += 256) {
-      const int r = i / p.dv, d = i % p.dv;
-      sV[r * p.dv + d] = kb + r < klen ? ldf(p.v + (long long)(k0 + kb + r) * p.v_ld + h * p.v_stride + d) : 0.f;
-    }
-    __syncthreads();
-    float s[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int d = 0; d < p.dq; ++d) {
-      const float x = sQ[row * ldq + d];
-#pragma unroll
-      for (int j = 0; j < 4; ++j) s[j] += x * sK[(part + 8 * j) * ldq + d];
-    }
-    float mx = -INFINITY;
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int key = kb + part + 8 * j;
-      s[j] = key < klen && key <= m0 + row + off ? s[j] * p.scale : -INFINITY;
-      mx = fmaxf(mx, s[j]);
-    }
-#pragma unroll
-    for (int x = 4; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
-    const float m_new = fmaxf(m_run, mx);
-    const float m_use = m_new == -INFINITY ? 0.f : m_new;
-    const float corr = expf(m_run - m_use);
-    float sum = 0.f;
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      s[j] = expf(s[j] - m_use);
-      sum += s[j];
-      sP[row * (SB + 1) + part + 8 * j] = s[j];
-    }
-#pragma unroll
-    for (int x = 4; x > 0; x >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, x);
-    l_run = l_run * corr + sum;
-    m_run = m_new;
-    __syncwarp();                        // a row's eight threads share a warp
-#pragma unroll
-    for (int i = 0; i < ACC; ++i) {
-      const int c = part + 8 * i;
-      if (c < p.dv) {
-        float a = acc[i] * corr;
-        for (int j = 0; j < SB; ++j) a += sP[row * (SB + 1) + j] * sV[j * p.dv + c];
-        acc[i] = a;
-      }
-    }
-  }
-  if (m0 + row < qlen) {
-    const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-#pragma unroll
-    for (int i = 0; i < ACC; ++i) {
-      const int c = part + 8 * i;
-      if (c < p.dv) stf(p.out + (long long)(q0 + m0 + row) * p.o_ld + h * p.o_stride + c, acc[i] * inv);
-    }
-  }
 }
 
 // ---- decode on the CUDA cores -----------------------------------------------------------------------------
@@ -662,17 +549,6 @@ MSRL_API int msrl_latent_prep(void* qkv, long long ld, const int* ints, const fl
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
-MSRL_API int msrl_latent_gather(const void* cache, const int* block_tables, int max_blocks, int block_size,
-                                const int* token_seq, const int* token_pos, void* out, long long rows, int row_bytes,
-                                cudaStream_t st) {
-  if (rows == 0) return 0;
-  if (row_bytes % 16 != 0) return (int)cudaErrorInvalidValue;
-  mla::gather_kernel<<<(unsigned)((rows + 7) / 8), 256, 0, st>>>((const uint4*)cache, block_tables, max_blocks,
-                                                                 block_size, token_seq, token_pos, (uint4*)out, rows,
-                                                                 row_bytes / 16);
-  return (int)cudaGetLastError();
-}
-
 MSRL_API int msrl_latent_spread(const void* lat, int CP, int RP, void* kv, long long ld, int H, int stride, int dn,
                                 int dr, int tokens, int is_f32, cudaStream_t st) {
   if (tokens == 0 || dr == 0) return 0;
@@ -682,34 +558,6 @@ MSRL_API int msrl_latent_spread(const void* lat, int CP, int RP, void* kv, long 
     mla::spread_kernel<__nv_bfloat16><<<tokens, 256, 0, st>>>((const __nv_bfloat16*)lat, CP, RP, (__nv_bfloat16*)kv, ld, H,
                                                               stride, dn, dr, tokens);
   return (int)cudaGetLastError();
-}
-
-// lds: q, k, v, out row strides; ints: q, k, v, out head strides, dq, dv
-MSRL_API int msrl_attn_simt(const void* q, const void* k, const void* v, void* out, const long long* lds,
-                            const int* ints, const int* cu_q, const int* cu_k, int batch, int max_q, int H, float scale,
-                            int is_f32, cudaStream_t st) {
-  if (batch == 0 || max_q == 0) return 0;
-  const int dq = ints[4], dv = ints[5];
-  if (dv > 512 || batch > 65535 || H > 65535) return (int)cudaErrorNotSupported;
-  const size_t smem = sizeof(float) * (2 * (size_t)mla::SB * (dq + 1) + (size_t)mla::SB * dv + mla::SB * (mla::SB + 1));
-  if (smem > 227 * 1024) return (int)cudaErrorNotSupported;
-  auto run = [&](auto tag) {
-    using T = decltype(tag);
-    mla::SimtArgs<T> p{(const T*)q, (const T*)k, (const T*)v, lds[0], lds[1], lds[2], ints[0], ints[1], ints[2],
-                       dq, dv, cu_q, cu_k, scale, (T*)out, lds[3], ints[3]};
-    const dim3 grid((unsigned)((max_q + mla::SB - 1) / mla::SB), (unsigned)H, (unsigned)batch);
-    auto go = [&](auto kernel) {
-      cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-      if (e != cudaSuccess) return (int)e;
-      kernel<<<grid, 256, smem, st>>>(p);
-      return (int)cudaGetLastError();
-    };
-    if (dv <= 64) return go(mla::attn_simt_kernel<T, 8>);
-    if (dv <= 128) return go(mla::attn_simt_kernel<T, 16>);
-    if (dv <= 256) return go(mla::attn_simt_kernel<T, 32>);
-    return go(mla::attn_simt_kernel<T, 64>);
-  };
-  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
 MSRL_API int msrl_latent_decode_simt(const void* q, const void* cache, const int* block_tables, int max_blocks,

@@ -6,6 +6,7 @@
 //             the grouped GEMM's row count is bounded by slots + 128 * experts on the host side.
 //   permute   x[token] (optionally scaled by the slot's weight) -> rows of the expert-grouped
 //             buffer; pad rows of every segment are zeroed.
+//   route_top the experts of the largest sigmoid scores of every token, with their scores
 //   combine   out[token] = sum_k w[token, k] * y[row(token, k)]   (fp32 accumulation; w optional)
 //   slot_dot  dw[token, k] = <dout[token], y[row(token, k)]>      (gradient of the combine weights)
 //
@@ -123,6 +124,64 @@ moe_permute_kernel(const __nv_bfloat16* x, long long ldx, const int* pos, const 
   }
 }
 
+// fp32 rows of any length
+__global__ void __launch_bounds__(128)
+moe_permute_f32_kernel(const float* x, const int* pos, const float* w, int T, int k, int H, const int* counts,
+                       const int* offsets, float* xp) {
+  const int b = blockIdx.x;
+  if (b < T) {
+    for (int j = 0; j < k; ++j) {
+      const long long r = pos[b * k + j];
+      const float s = w != nullptr ? w[b * k + j] : 1.f;
+      for (int c = threadIdx.x; c < H; c += 128) xp[r * H + c] = s * x[(long long)b * H + c];
+    }
+  } else {
+    const int e = b - T;
+    for (long long i = (long long)(offsets[e] + counts[e]) * H + threadIdx.x; i < (long long)offsets[e + 1] * H; i += 128)
+      xp[i] = 0.f;
+  }
+}
+
+// One warp per token.  Logits stay in registers (NPL per lane); the largest is taken out `top` times.  They are
+// ordered by logit: the sigmoid is monotone but saturates.
+template <int NPL>
+__global__ void __launch_bounds__(256)
+route_top_kernel(const float* logits, int T, int E, int top, long long* idx, float* score) {
+  const long long t = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (t >= T) return;
+  float z[NPL];
+#pragma unroll
+  for (int n = 0; n < NPL; ++n) z[n] = n * 32 + lane < E ? logits[t * E + n * 32 + lane] : -INFINITY;
+  unsigned taken = 0;                                  // bit n: this lane's entry n is out
+  for (int j = 0; j < top; ++j) {
+    float best = -INFINITY;
+    int at = 0x7fffffff;
+#pragma unroll
+    for (int n = 0; n < NPL; ++n) {
+      if (n * 32 + lane < E && !(taken >> n & 1) && (at == 0x7fffffff || z[n] > best)) {
+        best = z[n];
+        at = n * 32 + lane;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float b2 = __shfl_xor_sync(0xffffffffu, best, o);
+      const int a2 = __shfl_xor_sync(0xffffffffu, at, o);
+      const bool valid = a2 != 0x7fffffff;
+      if (valid && (at == 0x7fffffff || b2 > best || (b2 == best && a2 < at))) {
+        best = b2;
+        at = a2;
+      }
+    }
+    if ((at & 31) == lane) taken |= 1u << (at >> 5);
+    if (lane == 0) {
+      idx[t * top + j] = at;
+      score[t * top + j] = 1.f / (1.f + expf(-best));
+    }
+  }
+}
+
 __global__ void __launch_bounds__(128)
 moe_combine_kernel(const __nv_bfloat16* y, long long ldy, const int* pos, const float* w, int k, int H,
                    __nv_bfloat16* out, long long ldo, int accumulate) {
@@ -198,6 +257,24 @@ MSRL_API int msrl_moe_permute(const void* x, long long ldx, const int* pos, cons
   if (T + n_experts == 0) return 0;
   moe_permute_kernel<<<T + n_experts, 128, 0, st>>>((const __nv_bfloat16*)x, ldx, pos, w, T, k, H, counts, offsets,
                                                     (__nv_bfloat16*)xp, ldp);
+  return (int)cudaGetLastError();
+}
+
+MSRL_API int msrl_moe_permute_f32(const float* x, const int* pos, const float* w, int T, int k, int H, int n_experts,
+                                  const int* counts, const int* offsets, float* xp, cudaStream_t st) {
+  if (T + n_experts == 0) return 0;
+  moe_permute_f32_kernel<<<T + n_experts, 128, 0, st>>>(x, pos, w, T, k, H, counts, offsets, xp);
+  return (int)cudaGetLastError();
+}
+
+// logits [T, E] -> idx, score [T, top]; at most 1024 experts
+MSRL_API int msrl_route_top(const float* logits, int T, int E, int top, long long* idx, float* score, cudaStream_t st) {
+  if (T == 0) return 0;
+  if (E < 1 || E > 1024 || top < 1 || top > E) return (int)cudaErrorInvalidValue;
+  const unsigned grid = (unsigned)((T + 7) / 8);
+  if (E <= 64) route_top_kernel<2><<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
+  else if (E <= 256) route_top_kernel<8><<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
+  else route_top_kernel<32><<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
   return (int)cudaGetLastError();
 }
 

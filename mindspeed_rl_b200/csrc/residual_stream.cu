@@ -1,11 +1,11 @@
 // Kernels around an fp32 residual stream (bf16 or fp32 activations, selected by `is_f32`).
 //
 //   embed_norm        resid[t] = scale * table[id[t]];                        y[t] = norm(resid[t])
-//   add_norm          resid[t] += delta[t];                                   y[t] = norm(resid[t])
-//   moe_combine_norm  resid[t] += w * sum_j e[pos(t, j)] + sig(h[t].sg) * sh[t];  y[t] = norm(resid[t])
+//   add_norm          resid[t] += delta[t] + delta2[t];                       y[t] = norm(resid[t])
+//   moe_combine_norm  resid[t] += w * sum_j e[pos(t, j)] + sig(h[t].sg) * sh[t] + delta2[t];  y[t] = norm(resid[t])
 //
-// norm(x) = x * rsqrt(mean(x^2) + eps) * (offset + weight), all in fp32; y is stored in the activation
-// type.  One block per row; the row stays in registers between the sum and the norm (longer rows than the
+// norm(x) = x / sqrt(mean(x^2) + eps) * (offset + weight), all in fp32, with x less its mean when `centered` (the
+// squares are then summed in a pass of their own over the kept row); y is stored in the activation type.  One block per row; the row stays in registers between the sum and the norm (longer rows than the
 // register budget re-read the residual they just wrote).  A null `y` skips the norm.
 //
 //   glu               act(gate) * up of rows [gate | up]: silu, tanh-gelu, or the clamped swish with (up + 1)
@@ -24,6 +24,8 @@ struct RowArgs {
   T* y;
   int W;
   float eps, offset;
+  int centered;
+  const T* delta2;                        // SRC_DELTA, SRC_MOE: one more term, or null
   // SRC_EMBED
   const long long* ids;
   const T* table;
@@ -76,6 +78,11 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
       ldv<V>(p.delta + t * W + c, d);
 #pragma unroll
       for (int i = 0; i < V; ++i) f[i] += d[i];
+      if (p.delta2 != nullptr) {
+        ldv<V>(p.delta2 + t * W + c, d);
+#pragma unroll
+        for (int i = 0; i < V; ++i) f[i] += d[i];
+      }
     } else {
       float d[4], acc[4] = {0.f, 0.f, 0.f, 0.f};
       for (int j = 0; j < p.top; ++j) {
@@ -91,12 +98,17 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
 #pragma unroll
         for (int i = 0; i < V; ++i) acc[i] += sig * d[i];
       }
+      if (p.delta2 != nullptr) {
+        ldv<V>(p.delta2 + t * W + c, d);
+#pragma unroll
+        for (int i = 0; i < V; ++i) acc[i] += d[i];
+      }
 #pragma unroll
       for (int i = 0; i < V; ++i) f[i] += acc[i];
     }
   };
   float keep[NPT][4];
-  float ss = 0.f;
+  float ss = 0.f, sum = 0.f;
 #pragma unroll
   for (int k = 0; k < NPT; ++k) {
     const int c = (k * RS_THREADS + threadIdx.x) * V;
@@ -104,7 +116,10 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
       value(c, keep[k]);
       stv<V>(res + c, keep[k]);
 #pragma unroll
-      for (int i = 0; i < V; ++i) ss += keep[k][i] * keep[k][i];
+      for (int i = 0; i < V; ++i) {
+        ss += keep[k][i] * keep[k][i];
+        sum += keep[k][i];
+      }
     }
   }
   for (int c = (NPT * RS_THREADS + threadIdx.x) * V; c < W; c += RS_THREADS * V) {
@@ -112,9 +127,33 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
     value(c, f);
     stv<V>(res + c, f);
 #pragma unroll
-    for (int i = 0; i < V; ++i) ss += f[i] * f[i];
+    for (int i = 0; i < V; ++i) {
+      ss += f[i] * f[i];
+      sum += f[i];
+    }
   }
   if (p.y == nullptr) return;
+  float mean = 0.f;
+  if (p.centered) {
+    mean = block_sum(sum, red) / (float)W;
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NPT; ++k) {
+      if ((k * RS_THREADS + threadIdx.x) * V < W) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+          keep[k][i] -= mean;
+          ss += keep[k][i] * keep[k][i];
+        }
+      }
+    }
+    for (int c = (NPT * RS_THREADS + threadIdx.x) * V; c < W; c += RS_THREADS * V) {
+      float f[4];
+      ldv<V>(res + c, f);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss += (f[i] - mean) * (f[i] - mean);
+    }
+  }
   const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + p.eps);
   T* y = p.y + t * W;
 #pragma unroll
@@ -133,7 +172,7 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
     ldv<V>(res + c, f);
     ldv<V>(p.norm_w + c, w);
 #pragma unroll
-    for (int i = 0; i < V; ++i) w[i] = f[i] * r * (p.offset + w[i]);
+    for (int i = 0; i < V; ++i) w[i] = (f[i] - mean) * r * (p.offset + w[i]);
     stv<V>(y + c, w);
   }
 }
@@ -221,7 +260,8 @@ int launch_glu(const T* x, T* y, long long rows, int F, int kind, float limit, f
 using namespace msrl;
 
 template <typename T>
-static RowArgs<T> base_args(float* resid, const float* norm_w, void* y, int W, float eps, float offset) {
+static RowArgs<T> base_args(float* resid, const float* norm_w, void* y, int W, float eps, float offset,
+                            int centered) {
   RowArgs<T> p{};
   p.resid = resid;
   p.norm_w = norm_w;
@@ -229,14 +269,16 @@ static RowArgs<T> base_args(float* resid, const float* norm_w, void* y, int W, f
   p.W = W;
   p.eps = eps;
   p.offset = offset;
+  p.centered = centered;
   return p;
 }
 
 MSRL_API int msrl_embed_norm(const long long* ids, const void* table, float scale, float* resid, const float* norm_w,
-                             void* y, long long rows, int W, float eps, float offset, int is_f32, cudaStream_t st) {
+                             void* y, long long rows, int W, float eps, float offset, int centered, int is_f32,
+                             cudaStream_t st) {
   auto run = [&](auto tag) {
     using T = decltype(tag);
-    RowArgs<T> p = base_args<T>(resid, norm_w, y, W, eps, offset);
+    RowArgs<T> p = base_args<T>(resid, norm_w, y, W, eps, offset, centered);
     p.ids = ids;
     p.table = (const T*)table;
     p.scale = scale;
@@ -245,23 +287,25 @@ MSRL_API int msrl_embed_norm(const long long* ids, const void* table, float scal
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
-MSRL_API int msrl_add_norm(const void* delta, float* resid, const float* norm_w, void* y, long long rows, int W,
-                           float eps, float offset, int is_f32, cudaStream_t st) {
+MSRL_API int msrl_add_norm(const void* delta, const void* delta2, float* resid, const float* norm_w, void* y,
+                           long long rows, int W, float eps, float offset, int centered, int is_f32, cudaStream_t st) {
   auto run = [&](auto tag) {
     using T = decltype(tag);
-    RowArgs<T> p = base_args<T>(resid, norm_w, y, W, eps, offset);
+    RowArgs<T> p = base_args<T>(resid, norm_w, y, W, eps, offset, centered);
     p.delta = (const T*)delta;
+    p.delta2 = (const T*)delta2;
     return launch_row_norm<T, SRC_DELTA>(p, rows, st);
   };
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
 MSRL_API int msrl_moe_combine_norm(const void* e, const int* pos, int top, float expert_w, const void* h,
-                                   const void* sg, const void* shared, float* resid, const float* norm_w, void* y,
-                                   long long rows, int W, float eps, float offset, int is_f32, cudaStream_t st) {
+                                   const void* sg, const void* shared, const void* delta, float* resid,
+                                   const float* norm_w, void* y, long long rows, int W, float eps, float offset,
+                                   int centered, int is_f32, cudaStream_t st) {
   auto run = [&](auto tag) {
     using T = decltype(tag);
-    RowArgs<T> p = base_args<T>(resid, norm_w, y, W, eps, offset);
+    RowArgs<T> p = base_args<T>(resid, norm_w, y, W, eps, offset, centered);
     p.e = (const T*)e;
     p.pos = pos;
     p.top = top;
@@ -269,6 +313,7 @@ MSRL_API int msrl_moe_combine_norm(const void* e, const int* pos, int top, float
     p.h = (const T*)h;
     p.sg = (const T*)sg;
     p.shared = (const T*)shared;
+    p.delta2 = (const T*)delta;
     return launch_row_norm<T, SRC_MOE>(p, rows, st);
   };
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});

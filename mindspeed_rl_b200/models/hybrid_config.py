@@ -2,23 +2,66 @@
 
 A :class:`HybridConfig` lists its layers one by one: each has a token mixer of some type with its own sizes
 and a feed-forward of some kind (or none), and a range of layers may be run several times in a row with the
-same weights.  The layer types are small dataclasses in two tables (``MIXERS``, ``FEED_FORWARDS``), so that
+same weights.  The layer types are small dataclasses; a :class:`Design` says which of them an architecture has
+under which names, its norm, how a layer adds its two sublayers and where its LM head is (``DESIGNS``), so that
 another design adds a type without touching the readers of the others.  :meth:`HybridConfig.from_json` reads
 the ``config.json`` of a model folder.
+
+A mixer spec tells the cache what a sequence carries for it: ``paged_rows(dtype)``, shapes of one token's rows in
+paged memory by name, and ``slot_state(dtype)``, shapes and types of the state of one sequence by name.
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional, Tuple
 
 import torch
 
+from ..ops.latent import pad16
+
+
+def padded_heads(dq: int, dv: int, dtype: torch.dtype) -> Tuple[int, int]:
+    """Query / key and value head sizes as they are stored: bf16 heads are padded to a pair that the tensor-core
+    attention kernels serve; other sizes and fp32 (CUDA cores) to whole 16-byte vectors."""
+    if dtype != torch.bfloat16 or dv > 128 or dq > 192:
+        unit = 16 // dtype.itemsize
+        return -(-dq // unit) * unit, -(-dv // unit) * unit
+    vp = 64 if max(dq, dv) <= 64 else 128
+    return (192 if dq > 128 else vp), vp
+
+
+@dataclass(frozen=True)
+class WavelengthScaling:
+    """Frequencies of wavelengths above ``original / low`` are divided by ``factor``, those below
+    ``original / high`` kept, and the ones between are blended linearly in ``original / wavelength``."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+    def scaled(self, f: float) -> float:
+        turns = self.original * f / (2.0 * math.pi)          # whole turns over the original length
+        if turns > self.high:
+            return f
+        if turns < self.low:
+            return f / self.factor
+        s = (turns - self.low) / (self.high - self.low)
+        return (1.0 - s) * f / self.factor + s * f
+
 
 @dataclass(frozen=True)
 class Rotary:
-    """Rotary positions on the first ``dims`` entries of a vector, neighbours paired (2i with 2i + 1)."""
+    """Rotary positions on the first ``dims`` entries of a vector: neighbours paired (2i with 2i + 1), or
+    with ``halves`` entry i with entry i + dims / 2."""
     dims: int
     base: float
+    halves: bool = False
+    scaling: Optional[WavelengthScaling] = None
+
+    def frequencies(self) -> Tuple[float, ...]:
+        fs = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        return tuple(self.scaling.scaled(f) if self.scaling is not None else f for f in fs)
 
 
 @dataclass(frozen=True)
@@ -33,6 +76,13 @@ class LatentAttentionSpec:
     scale: float
     rot: Rotary
     recurrent = False
+    window = None
+
+    def paged_rows(self, dtype) -> Dict[str, Tuple[int, ...]]:
+        return {"latent": (pad16(self.kv_rank) + pad16(self.rot_dim),)}
+
+    def slot_state(self, dtype) -> dict:
+        return {}
 
     @classmethod
     def from_json(cls, m: dict) -> "LatentAttentionSpec":
@@ -55,12 +105,87 @@ class ChannelDeltaSpec:
     unit_eps: float = 1e-6
     recurrent = True
 
+    @property
+    def channels(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    def paged_rows(self, dtype) -> dict:
+        return {}
+
+    def slot_state(self, dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
+        return {"ring": ((self.conv, self.channels), dtype), "state": ((self.heads, self.dim, self.vdim), torch.float32)}
+
     @classmethod
     def from_json(cls, m: dict) -> "ChannelDeltaSpec":
         out = cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]))
         if out.heads % out.kv_heads:
             raise ValueError(f"{out.heads} heads do not divide into {out.kv_heads} key heads")
         return out
+
+
+@dataclass(frozen=True)
+class WindowAttentionSpec:
+    """Soft-max attention of grouped heads over the last ``window`` tokens (None: all), with biased projections, an
+    RMS norm over the whole query and the whole key projection, partial rotation, and values mixed with those of
+    the first layer that has ``value_mix``."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: Rotary
+    window: Optional[int] = None
+    value_mix: bool = False
+    recurrent = False
+
+    def padded(self, dtype) -> Tuple[int, int]:
+        return padded_heads(self.dim, self.vdim, dtype)
+
+    def paged_rows(self, dtype) -> Dict[str, Tuple[int, ...]]:
+        qp, vp = self.padded(dtype)
+        return {"k": (self.kv_heads, qp), "v": (self.kv_heads, vp)}
+
+    def slot_state(self, dtype) -> dict:
+        return {}
+
+    @classmethod
+    def from_json(cls, m: dict) -> "WindowAttentionSpec":
+        r, sc, mask = m["rot"], m["rot"].get("scaling"), m.get("mask")
+        rot = Rotary(int(r["dims"]), float(r["base"]), halves=True,
+                     scaling=None if not sc else WavelengthScaling(float(sc["factor"]), float(sc["low"]), float(sc["high"]),
+                                                                   float(sc["original"])))
+        out = cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), rot,
+                  None if not mask else int(mask["size"]), bool(m.get("v_mix", False)))
+        if out.heads % out.kv_heads:
+            raise ValueError(f"{out.heads} heads do not divide into {out.kv_heads} key heads")
+        if rot.dims % 2 or rot.dims > out.dim:
+            raise ValueError(f"rotary dims {rot.dims} must be even and at most dim ({out.dim})")
+        if out.window is not None and out.window < 1:
+            raise ValueError(f"a window of {out.window} tokens sees nothing")
+        return out
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    """Matrix memory with exponential gates, stabilised by a running maximum that starts at zero; gate logits are
+    soft-capped at ``gate_cap``.  Heads are stored in multiples of 16."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+    floor: float = 1e-6                  # added to the normaliser
+    recurrent = True
+
+    def slot_state(self, dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
+        f32, dp, vp = torch.float32, pad16(self.dim), pad16(self.vdim)
+        return {"memory": ((self.heads, dp, vp), f32), "norm": ((self.heads, dp), f32), "peak": ((self.heads,), f32)}
+
+    def paged_rows(self, dtype) -> dict:
+        return {}
+
+    @classmethod
+    def from_json(cls, m: dict) -> "MatrixMemorySpec":
+        return cls(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
 
 
 @dataclass(frozen=True)
@@ -94,8 +219,44 @@ class TableMoESpec:
                    clamped(m["shared"]) if m.get("shared") else None)
 
 
-MIXERS = {"latent_attention": LatentAttentionSpec, "channel_delta": ChannelDeltaSpec}
-FEED_FORWARDS = {"dense": GluSpec, "moe": TableMoESpec}
+@dataclass(frozen=True)
+class ScoredMoESpec:
+    """Experts of the largest router scores (sigmoid of 32-bit logits), each run on its input times its score, plus
+    an optional shared expert."""
+    experts: int
+    top: int
+    expert: GluSpec
+    shared: Optional[GluSpec] = None
+
+    @classmethod
+    def from_json(cls, m: dict) -> "ScoredMoESpec":
+        r, sh = m["router"], m.get("shared")
+        out = cls(int(r["experts"]), int(r["top"]), GluSpec(int(m["expert"]["ff"]), "silu"),
+                  GluSpec(int(sh["ff"]), "silu") if sh else None)
+        if not 0 < out.top <= out.experts:
+            raise ValueError(f"top {out.top} of {out.experts} experts")
+        return out
+
+
+@dataclass(frozen=True)
+class Design:
+    """What the layers of one architecture have in common.  ``parallel``: both sublayers read one norm and are added
+    together; otherwise the feed-forward reads a second norm of the sum.  ``centered``: norms subtract the mean.
+    ``norm_offset``: the stored weight of a norm is an offset from this value."""
+    mixers: Dict[str, Any]
+    feed_forwards: Dict[str, Any]
+    parallel: bool = False
+    centered: bool = False
+    norm_offset: float = 0.0
+    tied_head: bool = True
+
+
+DESIGNS = {
+    "Pumotar": Design({"latent_attention": LatentAttentionSpec, "channel_delta": ChannelDeltaSpec},
+                      {"dense": GluSpec, "moe": TableMoESpec}, norm_offset=1.0),
+    "Sunatar": Design({"attention": WindowAttentionSpec, "mlstm": MatrixMemorySpec}, {"moe": ScoredMoESpec},
+                      parallel=True, centered=True, tied_head=False),
+}
 
 
 @dataclass(frozen=True)
@@ -112,7 +273,6 @@ class HybridConfig:
     hidden_size: int
     layers: List[LayerSpec]
     norm_epsilon: float
-    norm_offset: float = 1.0             # the stored weight of a pre-norm is an offset from this value
     embedding_scale: float = 1.0
     loop: Optional[Tuple[int, int, int]] = None      # (start, stop, times)
     params_dtype: torch.dtype = torch.bfloat16
@@ -124,6 +284,13 @@ class HybridConfig:
             a, b, n = self.loop
             if not (0 <= a <= b <= len(self.layers)) or n < 1:
                 raise ValueError(f"loop {self.loop} does not fit {len(self.layers)} layers")
+        mixed = {l.mixer.kv_heads * l.mixer.vdim for l in self.layers if getattr(l.mixer, "value_mix", False)}
+        if len(mixed) > 1:
+            raise ValueError(f"layers that mix values with the first one's have different value sizes: {sorted(mixed)}")
+
+    @property
+    def design(self) -> Design:
+        return DESIGNS[self.architecture]
 
     # ---- what a sequence runs through ----------------------------------------------------------
     @property
@@ -145,19 +312,24 @@ class HybridConfig:
 
     @property
     def is_moe(self) -> bool:
-        return any(isinstance(l.mlp, TableMoESpec) for l in self.layers)
+        return any(isinstance(l.mlp, (TableMoESpec, ScoredMoESpec)) for l in self.layers)
+
+    @property
+    def windows(self) -> Tuple[Optional[int], ...]:
+        """Distinct key ranges of the attention layers (None: all earlier tokens)."""
+        return tuple({l.mixer.window: None for l in self.layers if not l.mixer.recurrent})
 
     @classmethod
     def from_json(cls, cfg: dict, dtype: torch.dtype = torch.bfloat16) -> "HybridConfig":
-        layers = []
+        layers, design = [], DESIGNS[cfg["architecture"]]
         for i, l in enumerate(cfg["layers"]):
-            if l["type"] not in MIXERS:
+            if l["type"] not in design.mixers:
                 raise ValueError(f"layer {i}: unknown mixer type {l['type']!r}")
             mlp = l.get("mlp")
-            if mlp is not None and mlp["kind"] not in FEED_FORWARDS:
+            if mlp is not None and mlp["kind"] not in design.feed_forwards:
                 raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
-            layers.append(LayerSpec(l["type"], MIXERS[l["type"]].from_json(l["mixer"]),
-                                    None if mlp is None else FEED_FORWARDS[mlp["kind"]].from_json(mlp)))
+            layers.append(LayerSpec(l["type"], design.mixers[l["type"]].from_json(l["mixer"]),
+                                    None if mlp is None else design.feed_forwards[mlp["kind"]].from_json(mlp)))
         lp = cfg.get("loop")
         return cls(architecture=cfg["architecture"], vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
                    layers=layers, norm_epsilon=float(cfg["norm"]["eps"]),

@@ -9,7 +9,7 @@ from __future__ import annotations
 import json
 import os
 from dataclasses import dataclass
-from typing import Any, Callable, Dict, Tuple
+from typing import Any, Callable, Dict, Optional, Tuple
 
 import torch
 
@@ -21,6 +21,7 @@ from .transformer_config import TransformerConfig
 class ModelFamily:
     config: Callable[[dict, torch.dtype], Any]                                  # (config.json, dtype) -> config
     weights: Callable[[Any, Dict[str, torch.Tensor], Any], Any]                 # (config, tensors, device) -> weights
+    kernels: Optional[str] = None        # group of kernels that serves the family (``csrc.build.GROUPS``; None: all)
 
 
 _FAMILIES: Dict[str, ModelFamily] = {}
@@ -45,6 +46,16 @@ def read_config(path: str, dtype: torch.dtype = torch.bfloat16):
     with open(os.path.join(path, "config.json")) as fh:
         raw = json.load(fh)
     return _FAMILIES[architecture_of(raw)].config(raw, dtype), raw
+
+
+def use_kernels_of(path: str) -> None:
+    """Serve this process from the kernels that the model of a folder needs, compiling them if they are not there."""
+    from ..ops import _lib
+
+    with open(os.path.join(path, "config.json")) as fh:
+        group = _FAMILIES[architecture_of(json.load(fh))].kernels
+    if group is not None:
+        _lib.use_group(group)
 
 
 def load_model(path: str, dtype: torch.dtype = torch.bfloat16, device="cuda"):
@@ -98,6 +109,7 @@ def _decoder_weights(cfg, state, device):
     return alias_rollout_weights(model)
 
 
-register("Pumotar", ModelFamily(HybridConfig.from_json, _hybrid_weights))
+register("Pumotar", ModelFamily(HybridConfig.from_json, _hybrid_weights, "pumotar"))
+register("Sunatar", ModelFamily(HybridConfig.from_json, _hybrid_weights, "sunatar"))
 for _name in ("Qwen2ForCausalLM", "Qwen3ForCausalLM", "Qwen3MoeForCausalLM"):
     register(_name, ModelFamily(_decoder_config, _decoder_weights))

@@ -100,7 +100,7 @@ def attn_varlen_fwd(qkv: torch.Tensor, layout: QKVLayout, cu_seqlens: torch.Tens
             rc = _lib.load().msrl_flash_attn_varlen_fwd_tcgen05(
                 ptr(flat[qs[0]:]), ptr(kb), ptr(vb), lay, ptr(out), c_ll(nh * hd), ptr(lse),
                 ptr(cu_seqlens), ptr(cu_k), c_int(batch), c_int(int(max_seqlen)), c_int(nh), c_int(nkv),
-                c_ll(t), c_ll(tk), c_int(hd), c_float(1.0 / math.sqrt(hd)), c_int(1 if causal else 0),
+                c_ll(t), c_ll(tk), c_int(hd), c_float(1.0 / math.sqrt(hd)), c_int(1 if causal else 0), c_int(0),
                 ptr(_status_word(qkv.device)), stream())
             if rc != _NOT_SUPPORTED:
                 check(rc, "flash_attn_varlen_fwd_tcgen05")
@@ -108,7 +108,7 @@ def attn_varlen_fwd(qkv: torch.Tensor, layout: QKVLayout, cu_seqlens: torch.Tens
         check(_lib.load().msrl_flash_attn_varlen_fwd(
             ptr(flat[qs[0]:]), ptr(kb), ptr(vb), lay, ptr(out), c_ll(nh * hd), ptr(lse),
             ptr(cu_seqlens), ptr(cu_k), c_int(batch), c_int(int(max_seqlen)), c_int(nh), c_int(nkv),
-            c_ll(t), c_int(hd), c_float(1.0 / math.sqrt(hd)), c_int(1 if causal else 0), stream()),
+            c_ll(t), c_int(hd), c_float(1.0 / math.sqrt(hd)), c_int(1 if causal else 0), c_int(0), stream()),
             "flash_attn_varlen_fwd")
         return out, lse
     q, k, v = layout.split(qkv)
@@ -178,14 +178,14 @@ def attn_kv_fwd(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_q: torch.T
             rc = _lib.load().msrl_flash_attn_varlen_fwd_tcgen05(
                 ptr(q), ptr(k), ptr(v), lay, ptr(out), c_ll(nh * hd), ptr(lse), ptr(cu_q), ptr(cu_k), c_int(batch),
                 c_int(int(max_q)), c_int(nh), c_int(nkv), c_ll(tq), c_ll(tk), c_int(hd), c_float(1.0 / math.sqrt(hd)),
-                c_int(1 if causal else 0), ptr(_status_word(q.device)), stream())
+                c_int(1 if causal else 0), c_int(0), ptr(_status_word(q.device)), stream())
             if rc != _NOT_SUPPORTED:
                 check(rc, "flash_attn_varlen_fwd_tcgen05")
                 return out, lse
         check(_lib.load().msrl_flash_attn_varlen_fwd(
             ptr(q), ptr(k), ptr(v), lay, ptr(out), c_ll(nh * hd), ptr(lse), ptr(cu_q), ptr(cu_k), c_int(batch),
             c_int(int(max_q)), c_int(nh), c_int(nkv), c_ll(tq), c_int(hd), c_float(1.0 / math.sqrt(hd)),
-            c_int(1 if causal else 0), stream()), "flash_attn_varlen_fwd")
+            c_int(1 if causal else 0), c_int(0), stream()), "flash_attn_varlen_fwd")
         return out, lse
     o, lse = _ref_attention(q, k, v, cu_q, cu_k, causal)
     return o.reshape(tq, nh * hd).to(q.dtype), lse

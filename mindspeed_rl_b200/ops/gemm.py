@@ -154,6 +154,14 @@ def linear_fwd(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = 
     return torch.matmul(x, w.t())
 
 
+def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``x [T, K] @ w [N, K].T`` with a 32-bit result: few output columns (router and gate logits), whatever the
+    operands' type."""
+    if x.is_cuda and x.dtype != torch.float32:
+        return torch.mm(x, w.t(), out_dtype=torch.float32)
+    return torch.matmul(x.float(), w.float().t())
+
+
 def linear_dgrad(dy: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     """``dy [T, N] @ w [N, K]``: input gradient of a linear, reading ``w`` where it is."""
     if dy.is_cuda and _pair_pays(dy.shape[0], w.shape[1]) and pair_usable(dy, w) and _lib.use_kernels(dy, w):

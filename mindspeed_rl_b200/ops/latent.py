@@ -100,7 +100,7 @@ def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, token_seq: to
     t = token_seq.numel()
     if _lib.use_kernels(cache, block_tables, token_seq, token_pos):
         out = guard.empty(t, cp, device=cache.device, dtype=cache.dtype)
-        check(_lib.load().msrl_latent_gather(ptr(cache), ptr(block_tables), c_int(block_tables.shape[1]), c_int(bs),
+        check(_lib.load().msrl_rows_gather(ptr(cache), ptr(block_tables), c_int(block_tables.shape[1]), c_int(bs),
                                              ptr(token_seq), ptr(token_pos), ptr(out), c_ll(t),
                                              c_int(cp * cache.element_size()), stream()), "latent_gather")
         return out
@@ -138,7 +138,7 @@ def latent_prefill_attention(proj: torch.Tensor, kv: torch.Tensor, lay: LatentLa
                 rc = _lib.load().msrl_flash_attn_varlen_fwd_tcgen05(
                     ptr(proj), ptr(kv), ptr(v), spec, ptr(out), c_ll(h * lay.vp), ptr(lse), ptr(cu_q), ptr(cu_k),
                     c_int(batch), c_int(max_q), c_int(h), c_int(h), c_ll(t), c_ll(kv.shape[0]), c_int(lay.qp),
-                    c_float(scale), c_int(1), ptr(_status_word(proj.device)), stream())
+                    c_float(scale), c_int(1), c_int(0), ptr(_status_word(proj.device)), stream())
                 if rc != _NOT_SUPPORTED:
                     check(rc, "flash_attn_varlen_fwd_tcgen05")
                     return out
@@ -146,10 +146,10 @@ def latent_prefill_attention(proj: torch.Tensor, kv: torch.Tensor, lay: LatentLa
                 check(_lib.load().msrl_flash_attn_varlen_fwd(
                     ptr(proj), ptr(kv), ptr(v), spec, ptr(out), c_ll(h * lay.vp), ptr(lse), ptr(cu_q), ptr(cu_k),
                     c_int(batch), c_int(max_q), c_int(h), c_int(h), c_ll(t), c_int(lay.qp), c_float(scale), c_int(1),
-                    stream()), "flash_attn_varlen_fwd")
+                    c_int(0), stream()), "flash_attn_varlen_fwd")
                 return out
         lds = (ctypes.c_longlong * 4)(proj.stride(0), kv.stride(0), kv.stride(0), h * lay.vp)
-        ints = (ctypes.c_int * 6)(lay.qp, lay.qp, lay.vp, lay.vp, lay.dn + lay.dr, lay.vp)
+        ints = (ctypes.c_int * 8)(lay.qp, lay.qp, lay.vp, lay.vp, lay.dn + lay.dr, lay.vp, 1, 0)
         check(_lib.load().msrl_attn_simt(ptr(proj), ptr(kv), ptr(v), ptr(out), lds, ints, ptr(cu_q), ptr(cu_k),
                                          c_int(batch), c_int(max_q), c_int(h), c_float(scale), _is_f32(proj), stream()),
               "attn_simt")

@@ -12,7 +12,7 @@ formulation that is also the test oracle.  Reference behaviour:
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -74,6 +74,21 @@ def moe_plan(expert_of: torch.Tensor, num_experts: int) -> MoePlan:
     return MoePlan(counts.int(), offsets.int(), pos.int(), tiles, rows, t, k, num_experts)
 
 
+def route_top(logits: torch.Tensor, top: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Router logits ``[T, E]`` fp32 -> ``(expert ids [T, top] int64, their scores [T, top] fp32)``: the ``top`` largest
+    ``sigmoid(logit)`` in descending order (equal logits: the lower expert first), scores not renormalised."""
+    t, e = logits.shape
+    if _lib.use_kernels(logits):
+        logits = logits.contiguous()
+        idx = guard.empty(t, top, dtype=torch.int64, device=logits.device)
+        score = guard.empty(t, top, dtype=torch.float32, device=logits.device)
+        check(_lib.load().msrl_route_top(ptr(logits), c_int(t), c_int(e), c_int(top), ptr(idx), ptr(score), stream()),
+              "route_top")
+        return idx, score
+    z, idx = torch.sort(logits, dim=-1, descending=True, stable=True)
+    return idx[:, :top].contiguous(), torch.sigmoid(z[:, :top])
+
+
 def moe_permute(x: torch.Tensor, plan: MoePlan, w: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``x [T, H]`` -> expert-grouped ``[max_rows, H]`` (row of slot (t, j) = ``w[t, j] * x[t]``);
     pad rows of used segments are zero, rows past the last segment are not touched."""
@@ -81,6 +96,14 @@ def moe_permute(x: torch.Tensor, plan: MoePlan, w: Optional[torch.Tensor] = None
     if x.dtype == torch.float32 and x.is_cuda and w is None and h % 4 == 0:
         # rows are only moved: an fp32 row is a bf16 row of twice the length
         return moe_permute(x.contiguous().view(torch.bfloat16), plan).view(torch.float32)
+    if x.dtype == torch.float32 and _lib.use_kernels(x):
+        x = x.contiguous()
+        xp = guard.empty(plan.max_rows, h, dtype=x.dtype, device=x.device)
+        wf = None if w is None else w.reshape(-1).float().contiguous()
+        check(_lib.load().msrl_moe_permute_f32(ptr(x), ptr(plan.pos), ptr(wf), c_int(t), c_int(plan.k), c_int(h),
+                                               c_int(plan.num_experts), ptr(plan.counts), ptr(plan.offsets), ptr(xp),
+                                               stream()), "moe_permute_f32")
+        return xp
     if x.dtype == torch.bfloat16 and h % 8 == 0 and _lib.use_kernels(x):
         x = x.contiguous()
         xp = guard.empty(plan.max_rows, h, dtype=x.dtype, device=x.device)

@@ -2,12 +2,13 @@
 follows fused in, and the gated activations.
 
 The residual ``[T, W]`` is fp32 and updated in place; norm weights are fp32, the activations bf16 or fp32.
-``norm(x) = x / sqrt(mean(x^2) + eps) * (offset + w)`` in fp32.  CUDA path: ``csrc/residual_stream.cu``; CPU
+``norm(x) = x / sqrt(mean(x^2) + eps) * (offset + w)`` in fp32; ``centered`` norms subtract the row's mean from x
+first (a layer norm without bias).  CUDA path: ``csrc/residual_stream.cu``; CPU
 tensors run the PyTorch formulation.
 """
 from __future__ import annotations
 
-from typing import Optional, Tuple
+from typing import NamedTuple, Optional, Tuple
 
 import torch
 import torch.nn.functional as F
@@ -24,58 +25,74 @@ def _is_f32(t: torch.Tensor):
     return c_int(1 if t.dtype == torch.float32 else 0)
 
 
-def _norm_ref(x: torch.Tensor, w: torch.Tensor, eps: float, offset: float, dtype) -> torch.Tensor:
+class Norm(NamedTuple):
+    """Arguments of a norm in the order of the functions below."""
+    weight: torch.Tensor
+    eps: float
+    offset: float = 0.0
+    centered: bool = False
+
+
+def _norm_ref(x: torch.Tensor, w: torch.Tensor, eps: float, offset: float, centered: bool, dtype) -> torch.Tensor:
+    if centered:
+        x = x - x.mean(-1, keepdim=True)
     return (x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (offset + w)).to(dtype)
 
 
 def embed_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, w: torch.Tensor, eps: float,
-               offset: float = 0.0) -> Tuple[torch.Tensor, torch.Tensor]:
+               offset: float = 0.0, centered: bool = False) -> Tuple[torch.Tensor, torch.Tensor]:
     """``(residual fp32, norm(residual))`` of ``residual = table[ids] * scale``."""
     t, h = ids.numel(), table.shape[1]
     if _lib.use_kernels(ids, table, w):
         resid = guard.empty(t, h, device=table.device, dtype=torch.float32)
         y = guard.empty(t, h, device=table.device, dtype=table.dtype)
         check(_lib.load().msrl_embed_norm(ptr(ids), ptr(table), c_float(scale), ptr(resid), ptr(w), ptr(y), c_ll(t),
-                                          c_int(h), c_float(eps), c_float(offset), _is_f32(table), stream()), "embed_norm")
+                                          c_int(h), c_float(eps), c_float(offset), c_int(centered), _is_f32(table), stream()),
+              "embed_norm")
         return resid, y
     resid = table[ids].float() * scale
-    return resid, _norm_ref(resid, w, eps, offset, table.dtype)
+    return resid, _norm_ref(resid, w, eps, offset, centered, table.dtype)
 
 
-def add_norm_(resid: torch.Tensor, delta: torch.Tensor, w: torch.Tensor, eps: float, offset: float = 0.0
-              ) -> torch.Tensor:
-    """``resid += delta`` in place; returns ``norm(resid)`` in ``delta``'s type."""
+def add_norm_(resid: torch.Tensor, delta: torch.Tensor, w: torch.Tensor, eps: float, offset: float = 0.0,
+              centered: bool = False, delta2: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``resid += delta (+ delta2)`` in place; returns ``norm(resid)`` in ``delta``'s type."""
     t, h = resid.shape
     if _lib.use_kernels(resid, delta, w):
         delta = delta.contiguous()
+        delta2 = None if delta2 is None else delta2.contiguous()
         y = guard.empty(t, h, device=resid.device, dtype=delta.dtype)
-        check(_lib.load().msrl_add_norm(ptr(delta), ptr(resid), ptr(w), ptr(y), c_ll(t), c_int(h), c_float(eps),
-                                        c_float(offset), _is_f32(delta), stream()), "add_norm")
+        check(_lib.load().msrl_add_norm(ptr(delta), ptr(delta2), ptr(resid), ptr(w), ptr(y), c_ll(t), c_int(h), c_float(eps),
+                                        c_float(offset), c_int(centered), _is_f32(delta), stream()), "add_norm")
         return y
-    resid.add_(delta.float())
-    return _norm_ref(resid, w, eps, offset, delta.dtype)
+    resid.add_(delta.float() if delta2 is None else delta.float() + delta2.float())
+    return _norm_ref(resid, w, eps, offset, centered, delta.dtype)
 
 
 def moe_combine_norm_(resid: torch.Tensor, expert_rows: torch.Tensor, pos: torch.Tensor, top: int, expert_w: float,
                       h: torch.Tensor, shared: Optional[torch.Tensor], shared_gate: Optional[torch.Tensor],
-                      w: torch.Tensor, eps: float, offset: float = 0.0) -> torch.Tensor:
-    """``resid[t] += expert_w * sum_j expert_rows[pos[t, j]] + sigmoid(h[t] . shared_gate) * shared[t]`` in
+                      w: torch.Tensor, eps: float, offset: float = 0.0, centered: bool = False,
+                      delta: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``resid[t] += expert_w * sum_j expert_rows[pos[t, j]] + sigmoid(h[t] . shared_gate) * shared[t] + delta[t]`` in
     place; returns ``norm(resid)``.  ``pos [T * top]`` are the rows of a dispatch plan (``ops.moe``); without
-    ``shared`` the second term is left out."""
+    ``shared`` or ``delta`` their term is left out, without ``shared_gate`` the shared term counts in full."""
     t, width = resid.shape
     if _lib.use_kernels(resid, expert_rows, pos, h):
         y = guard.empty(t, width, device=resid.device, dtype=h.dtype)
+        delta = None if delta is None else delta.contiguous()
         check(_lib.load().msrl_moe_combine_norm(
             ptr(expert_rows), ptr(pos), c_int(top), c_float(expert_w), ptr(h.contiguous()), ptr(shared_gate),
-            ptr(shared), ptr(resid), ptr(w), ptr(y), c_ll(t), c_int(width), c_float(eps), c_float(offset), _is_f32(h),
-            stream()), "moe_combine_norm")
+            ptr(shared), ptr(delta), ptr(resid), ptr(w), ptr(y), c_ll(t), c_int(width), c_float(eps), c_float(offset),
+            c_int(centered), _is_f32(h), stream()), "moe_combine_norm")
         return y
     add = expert_rows[pos.long()].float().view(t, top, width).sum(1) * expert_w
     if shared is not None:
         sig = 1.0 if shared_gate is None else torch.sigmoid(h.float() @ shared_gate.float().reshape(-1, 1))
         add = add + sig * shared.float()
+    if delta is not None:
+        add = add + delta.float()
     resid.add_(add)
-    return _norm_ref(resid, w, eps, offset, h.dtype)
+    return _norm_ref(resid, w, eps, offset, centered, h.dtype)
 
 
 GLU_KINDS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}

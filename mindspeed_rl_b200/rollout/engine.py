@@ -290,7 +290,6 @@ class LLMEngine(BaseInferEngine):
         dev = self.device
         ids, pos, slots, cu, last_rows = [], [], [], [0], []
         need_prefix = any(it.start > 0 for it in items)
-        tok_seq, tok_pos, cu_k = [], [], [0]
         for row, it in enumerate(items):
             s = it.seq
             all_ids = s.all_ids
@@ -299,11 +298,6 @@ class LLMEngine(BaseInferEngine):
             slots.append(self.bm.slots(s.seq_id, it.start, it.length))
             last_rows.extend(cu[-1] + r for r in rows[row])
             cu.append(cu[-1] + it.length)
-            if need_prefix:
-                end = it.start + it.length
-                tok_seq.extend([row] * end)
-                tok_pos.extend(range(end))
-                cu_k.append(cu_k[-1] + end)
         tok, _ = self._ship([ids, pos, np.concatenate(slots).tolist()])
         t_ids, t_pos, t_slots = tok[0], tok[1].to(torch.int32), tok[2]
         t_cu = to_device(cu, torch.int32, dev)
@@ -312,9 +306,10 @@ class LLMEngine(BaseInferEngine):
         if need_prefix:
             max_blocks = max(len(self.bm.block_table(it.seq.seq_id)) for it in items)
             bt = self.bm.block_tables([it.seq.seq_id for it in items], max_blocks)
-            pt, _ = self._ship([tok_seq, tok_pos])
-            prefix = dict(block_tables=to_device(bt, torch.int32, dev), token_seq=pt[0].to(torch.int32),
-                          token_pos=pt[1].to(torch.int32), cu_k=to_device(cu_k, torch.int32, dev))
+            bt = to_device(bt, torch.int32, dev)
+            prefix = {w: self._prefix_keys(items, bt, w) for w in (self.cfg.windows if self.cfg.is_hybrid else (None,))}
+            if not self.cfg.is_hybrid:
+                prefix = prefix[None]
         state = None
         if self.cfg.is_hybrid:
             st, _ = self._ship([[it.start for it in items], [it.seq.state_slot for it in items]])
@@ -327,6 +322,19 @@ class LLMEngine(BaseInferEngine):
             it.seq.num_computed = it.start + it.length
             self.bm.commit(it.seq.seq_id, it.seq.all_ids, it.seq.num_computed)
         return logits
+
+    def _prefix_keys(self, items: List[PrefillItem], block_tables: torch.Tensor, window: Optional[int]) -> dict:
+        """Cache positions that the tokens of prompt portions look at: everything up to a portion's end, or from the
+        first key inside the portion's first window."""
+        ends = np.array([it.start + it.length for it in items])
+        first = np.zeros_like(ends) if window is None else np.maximum([it.start - window + 1 for it in items], 0)
+        n = ends - first
+        cu = np.concatenate([[0], np.cumsum(n)])
+        owner = np.repeat(np.arange(len(items)), n)
+        pos = np.arange(cu[-1]) - cu[owner] + first[owner]
+        pt, _ = self._ship([owner, pos])
+        return dict(block_tables=block_tables, token_seq=pt[0].to(torch.int32), token_pos=pt[1].to(torch.int32),
+                    cu_k=to_device(cu.tolist(), torch.int32, self.device))
 
     def _run_prefill(self, items: List[PrefillItem]) -> None:
         finishing = [it.seq for it in items if it.completes_prompt]

@@ -1,18 +1,19 @@
 """Feed-forwards of layer-by-layer decoders in the rollout engine.
 
-``forward_norm_`` adds the feed-forward of ``h`` to the fp32 residual and returns the next norm of the sum, so
-that the add (and for expert layers the combine) and the norm are one kernel.
+``forward`` does the feed-forward's work on ``h`` up to what is left to add; ``finish_`` adds it (and, in layers whose
+sublayers run in parallel, the mixer's output ``delta``) to the fp32 residual and returns the next norm of the sum, so
+that the add (and for expert layers the combine) and the norm are one kernel.  ``norm``: an ``ops.Norm``.
 """
 from __future__ import annotations
 
-from typing import Dict
+from typing import Dict, Optional, Tuple
 
 import torch
 
 from .. import ops
-from ..models.hybrid_config import GluSpec, TableMoESpec
+from ..models.hybrid_config import GluSpec, ScoredMoESpec, TableMoESpec
 from ..ops import moe as K
-from ..ops.gemm import linear_fwd
+from ..ops.gemm import linear_f32, linear_fwd
 from .mixers import _pad_cols, _pad_rows
 
 
@@ -22,19 +23,22 @@ class Glu:
         self.gate_up = torch.cat([w["gate"], w["up"]]).to(device=device, dtype=dtype).contiguous()
         self.down = w["down"].to(device=device, dtype=dtype).contiguous()
 
-    def forward(self, h: torch.Tensor) -> torch.Tensor:
+    def __call__(self, h: torch.Tensor) -> torch.Tensor:
         s = self.spec
         return linear_fwd(ops.glu_fwd(linear_fwd(h, self.gate_up), s.act, s.limit, s.alpha), self.down)
 
-    def forward_norm_(self, resid, h, ids, norm_w, eps, offset) -> torch.Tensor:
-        return ops.add_norm_(resid, self.forward(h), norm_w, eps, offset)
+    def forward(self, h: torch.Tensor, ids: torch.Tensor) -> torch.Tensor:
+        return self(h)
+
+    def finish_(self, resid, h, done, norm, delta: Optional[torch.Tensor] = None) -> torch.Tensor:
+        return ops.add_norm_(resid, done, *norm, delta2=delta)
 
 
-class TableMoE:
-    """The router is a table from token id to expert ids: the dispatch plan of a step depends on its ids only.
-    Expert widths are padded to the grouped GEMM's reduction tile (zero rows: both activations vanish there)."""
+class GroupedExperts:
+    """Stacked expert weights and what every expert layer does once it knows its dispatch plan.  Expert widths are
+    padded to the grouped GEMM's reduction tile (zero rows: the activations vanish there)."""
 
-    def __init__(self, spec: TableMoESpec, w: Dict[str, torch.Tensor], dtype, device):
+    def __init__(self, spec, w: Dict[str, torch.Tensor], dtype, device):
         self.spec = spec
         f = spec.expert.ff
         fp = (f + 63) // 64 * 64 if dtype == torch.bfloat16 else f
@@ -44,27 +48,56 @@ class TableMoE:
             down.append(_pad_cols(w[f"e{e}.down"], fp))
         self.w1 = torch.stack(up).to(device=device, dtype=dtype).contiguous()        # [E, 2F, W]
         self.w2 = torch.stack(down).to(device=device, dtype=dtype).contiguous()      # [E, W, F]
+        self.shared = self.shared_gate = None
+        if spec.shared is not None:
+            self.shared = Glu(spec.shared, {k: w["shared." + k] for k in ("gate", "up", "down")}, dtype, device)
+
+    def run(self, h: torch.Tensor, plan: K.MoePlan, input_w: Optional[torch.Tensor] = None
+            ) -> Tuple[torch.Tensor, K.MoePlan, Optional[torch.Tensor]]:
+        s = self.spec
+        gu = K.grouped_gemm_nt(K.moe_permute(h, plan, input_w), plan, self.w1)
+        act = ops.glu_fwd(gu, s.expert.act, s.expert.limit, s.expert.alpha, plan=plan)
+        y = K.grouped_gemm_nt(act, plan, self.w2)
+        return y, plan, self.shared(h) if self.shared is not None else None
+
+    def finish_(self, resid, h, done, norm, delta: Optional[torch.Tensor] = None) -> torch.Tensor:
+        y, plan, shared = done
+        return ops.moe_combine_norm_(resid, y, plan.pos, self.spec.top, self.output_w, h, shared, self.shared_gate, *norm,
+                                     delta=delta)
+
+
+class TableMoE(GroupedExperts):
+    """The router is a table from token id to expert ids: the dispatch plan of a step depends on its ids only."""
+
+    def __init__(self, spec: TableMoESpec, w: Dict[str, torch.Tensor], dtype, device):
+        super().__init__(spec, w, dtype, device)
         table = w["table"].to(torch.int64)
         if table.shape[1] != spec.top or int(table.min()) < 0 or int(table.max()) >= spec.experts:
             raise ValueError(f"expert table {tuple(table.shape)} does not fit {spec.experts} experts, top {spec.top}")
         self.table = table.to(device)
-        self.shared = self.shared_gate = None
+        self.output_w = 1.0 / spec.top
         if spec.shared is not None:
-            self.shared = Glu(spec.shared, {k: w["shared." + k] for k in ("gate", "up", "down")}, dtype, device)
             self.shared_gate = w["shared.sg"].reshape(-1).to(device=device, dtype=dtype).contiguous()
 
-    def forward_norm_(self, resid, h, ids, norm_w, eps, offset) -> torch.Tensor:
-        s = self.spec
-        plan = K.moe_plan(self.table[ids], s.experts)
-        gu = K.grouped_gemm_nt(K.moe_permute(h, plan), plan, self.w1)
-        act = ops.glu_fwd(gu, s.expert.act, s.expert.limit, s.expert.alpha, plan=plan)
-        y = K.grouped_gemm_nt(act, plan, self.w2)
-        shared = self.shared.forward(h) if self.shared is not None else None
-        return ops.moe_combine_norm_(resid, y, plan.pos, s.top, 1.0 / s.top, h, shared, self.shared_gate, norm_w, eps,
-                                     offset)
+    def forward(self, h: torch.Tensor, ids: torch.Tensor):
+        return self.run(h, K.moe_plan(self.table[ids], self.spec.experts))
+
+
+class ScoredMoE(GroupedExperts):
+    """Router logits are 32-bit; a chosen expert's score scales the rows that go into it."""
+    output_w = 1.0
+
+    def __init__(self, spec: ScoredMoESpec, w: Dict[str, torch.Tensor], dtype, device):
+        super().__init__(spec, w, dtype, device)
+        self.router = w["router"].to(device=device, dtype=dtype).contiguous()
+
+    def forward(self, h: torch.Tensor, ids: torch.Tensor):
+        idx, score = K.route_top(linear_f32(h, self.router), self.spec.top)
+        return self.run(h, K.moe_plan(idx, self.spec.experts), score)
+
+
+FEED_FORWARDS = {GluSpec: Glu, TableMoESpec: TableMoE, ScoredMoESpec: ScoredMoE}
 
 
 def build_feed_forward(spec, w: Dict[str, torch.Tensor], dtype, device):
-    if spec is None:
-        return None
-    return (TableMoE if isinstance(spec, TableMoESpec) else Glu)(spec, w, dtype, device)
+    return None if spec is None else FEED_FORWARDS[type(spec)](spec, w, dtype, device)

@@ -44,8 +44,9 @@ class _Taken(dict):
 
 
 def build_hybrid_weights(cfg: HybridConfig, state: Dict[str, torch.Tensor], device) -> HybridWeights:
-    """``state``: checkpoint tensors (``embed``, ``final.norm``, ``l<i>.norm1``, ``l<i>.mix.*``, ``l<i>.mlp.*``).
-    The LM head is the embedding table.  A name that no layer asks for is an error."""
+    """``state``: checkpoint tensors (``embed``, ``final.norm``, ``l<i>.norm1``, ``l<i>.mix.*``, ``l<i>.mlp.*``, and
+    ``l<i>.norm2`` and ``head`` where the design has them; else the LM head is the embedding table).  A name that no
+    layer asks for is an error."""
     dt = cfg.params_dtype
     used = {"embed", "final.norm"}
 
@@ -57,17 +58,24 @@ def build_hybrid_weights(cfg: HybridConfig, state: Dict[str, torch.Tensor], devi
     for i, spec in enumerate(cfg.layers):
         p = f"l{i}."
         layer = HybridLayer(f32(p + "norm1"),
-                            MIXERS[spec.type](spec.mixer, _Taken(state, p + "mix.", used), cfg.norm_epsilon, dt, device))
+                            MIXERS[type(spec.mixer)](spec.mixer, _Taken(state, p + "mix.", used), cfg.norm_epsilon, dt, device))
         if spec.mlp is not None:
-            layer.norm2 = f32(p + "norm2")
+            if not cfg.design.parallel:
+                layer.norm2 = f32(p + "norm2")
             layer.ff = build_feed_forward(spec.mlp, _Taken(state, p + "mlp.", used), dt, device)
         layers.append(layer)
+    def table(name):
+        used.add(name)
+        t = state[name].to(device=device, dtype=dt).contiguous()
+        if tuple(t.shape) != (cfg.vocab_size, cfg.hidden_size):
+            raise ValueError(f"{name} {tuple(t.shape)} does not fit {cfg.vocab_size} x {cfg.hidden_size}")
+        return t
+
+    embed = table("embed")
+    head = embed if cfg.design.tied_head else table("head")
     extra = sorted(set(state) - used)
     # a layer without a feed-forward may still carry an unused second norm
     extra = [n for n in extra if not n.endswith(".norm2")]
     if extra:
         raise ValueError(f"tensors without a place in the model: {extra[:8]}")
-    embed = state["embed"].to(device=device, dtype=dt).contiguous()
-    if tuple(embed.shape) != (cfg.vocab_size, cfg.hidden_size):
-        raise ValueError(f"embedding {tuple(embed.shape)} does not fit {cfg.vocab_size} x {cfg.hidden_size}")
-    return HybridWeights(embed, layers, f32("final.norm"), embed)
+    return HybridWeights(embed, layers, f32("final.norm"), head)

@@ -1,19 +1,18 @@
-"""Carried state of decoders whose layers differ: paged latent rows and recurrent state slots.
+"""Carried state of decoders whose layers differ: paged rows (latents, keys and values) and recurrent state slots.
 
 ``HybridCache`` holds one entry per layer *run* (a layer that is run several times in a row has an entry per
-pass): latent-attention runs own paged rows ``[num_blocks, block_size, CP]`` addressed through the block manager's
-tables, recurrent runs own ``ring [slots, taps, channels]`` and ``state [slots, heads, dim, vdim]`` (fp32)
-addressed by a state slot per sequence.  ``StateSlots`` hands the slots out; the scheduler takes one when it
+pass): attention runs own paged rows ``[num_blocks, block_size, ...]`` addressed through the block manager's
+tables, recurrent runs own state tensors ``[slots, ...]`` addressed by a state slot per sequence.  ``StateSlots`` hands the slots out; the scheduler takes one when it
 admits or forks a sequence and returns it when the sequence ends or is preempted.
 """
 from __future__ import annotations
 
-from typing import List, Optional
+import math
+from typing import Dict, List
 
 import torch
 
 from ..models.hybrid_config import HybridConfig
-from ..ops.latent import pad16
 
 
 class OutOfSlots(RuntimeError):
@@ -46,58 +45,42 @@ class StateSlots:
         self._free.append(slot)
 
 
-def latent_row_width(spec) -> int:
-    return pad16(spec.kv_rank) + pad16(spec.rot_dim)
-
-
-def delta_channels(spec) -> int:
-    return 2 * spec.kv_heads * spec.dim + spec.heads * spec.vdim
-
-
 class HybridCache:
+    """``rows[run]``: paged memory by name, ``[num_blocks, block_size, *row]``; ``slots[run]``: state by name,
+    ``[num_slots, *shape]``.  What a layer has is what its mixer spec asks for."""
+
     def __init__(self, cfg: HybridConfig, num_blocks: int, block_size: int, num_slots: int, device):
         self.num_blocks, self.block_size, self.num_slots = num_blocks, block_size, num_slots
         dev = torch.device(device)
         # every row and slot is written before it is read (a sequence's first token ignores what its slot holds),
         # so nothing is cleared on the GPU; the CPU path multiplies by masks and wants finite values
         alloc = torch.empty if dev.type == "cuda" else torch.zeros
-        self.latent: List[Optional[torch.Tensor]] = []
-        self.ring: List[Optional[torch.Tensor]] = []
-        self.state: List[Optional[torch.Tensor]] = []
+        self.rows: List[Dict[str, torch.Tensor]] = []
+        self.slots: List[Dict[str, torch.Tensor]] = []
+        dt = cfg.params_dtype
         for li in cfg.run_order:
             m = cfg.layers[li].mixer
-            if m.recurrent:
-                self.latent.append(None)
-                self.ring.append(alloc(num_slots, m.conv, delta_channels(m), dtype=cfg.params_dtype, device=dev))
-                self.state.append(alloc(num_slots, m.heads, m.dim, m.vdim, dtype=torch.float32, device=dev))
-            else:
-                self.latent.append(alloc(num_blocks, block_size, latent_row_width(m), dtype=cfg.params_dtype, device=dev))
-                self.ring.append(None)
-                self.state.append(None)
+            self.rows.append({n: alloc(num_blocks, block_size, *shape, dtype=dt, device=dev)
+                              for n, shape in m.paged_rows(dt).items()})
+            self.slots.append({n: alloc(num_slots, *shape, dtype=t, device=dev) for n, (shape, t) in m.slot_state(dt).items()})
 
     @staticmethod
     def bytes_per_block(cfg: HybridConfig, block_size: int) -> int:
-        size = torch.empty(0, dtype=cfg.params_dtype).element_size()
-        return sum(block_size * latent_row_width(cfg.layers[li].mixer) * size for li in cfg.run_order
-                   if not cfg.layers[li].mixer.recurrent)
+        dt = cfg.params_dtype
+        return sum(block_size * math.prod(shape) * dt.itemsize for li in cfg.run_order
+                   for shape in cfg.layers[li].mixer.paged_rows(dt).values())
 
     @staticmethod
     def bytes_per_slot(cfg: HybridConfig) -> int:
-        size = torch.empty(0, dtype=cfg.params_dtype).element_size()
-        total = 0
-        for li in cfg.run_order:
-            m = cfg.layers[li].mixer
-            if m.recurrent:
-                total += m.conv * delta_channels(m) * size + m.heads * m.dim * m.vdim * 4
-        return total
+        return sum(math.prod(shape) * t.itemsize for li in cfg.run_order
+                   for shape, t in cfg.layers[li].mixer.slot_state(cfg.params_dtype).values())
 
     def copy_block(self, src: int, dst: int) -> None:
-        for c in self.latent:
-            if c is not None:
+        for rows in self.rows:
+            for c in rows.values():
                 c[dst].copy_(c[src])
 
     def copy_slot(self, src: int, dst: int) -> None:
-        for pair in (self.ring, self.state):
-            for c in pair:
-                if c is not None:
-                    c[dst].copy_(c[src])
+        for slots in self.slots:
+            for c in slots.values():
+                c[dst].copy_(c[src])

@@ -12,9 +12,12 @@ from typing import Dict, List, Optional
 import torch
 
 from .. import ops
+from ..models.hybrid_config import ChannelDeltaSpec, LatentAttentionSpec, MatrixMemorySpec, WindowAttentionSpec
 from ..ops.delta import DeltaLayout, DeltaWeights
-from ..ops.gemm import linear_fwd
-from ..ops.latent import LatentLayout
+from ..ops.gemm import linear_f32, linear_fwd
+from ..ops.latent import LatentLayout, pad16
+from ..ops.matrix_memory import MemoryLayout, MemoryWeights
+from ..ops.window import GroupedHeads, ValueSource
 
 
 @dataclass
@@ -30,11 +33,16 @@ class StepMeta:
     max_q: int = 0
     tok_seq: Optional[torch.Tensor] = None  # [T] int32
     start_pos: Optional[torch.Tensor] = None  # [B] int32 position of a portion's first token
-    prefix: Optional[dict] = None           # see ModelRunner.prefill
+    prefix: Optional[dict] = None           # by key range (``HybridConfig.windows``); see ModelRunner.prefill
     # decode steps
     block_tables: Optional[torch.Tensor] = None
     context_lens: Optional[torch.Tensor] = None
     max_context: int = 0
+    # values of the first layer that mixes values, kept for the later ones of the step
+    first_values: Optional[ValueSource] = None
+
+    def prefix_of(self, window: Optional[int]) -> Optional[dict]:
+        return None if self.prefix is None else self.prefix[window]
 
     @property
     def is_decode(self) -> bool:
@@ -55,6 +63,14 @@ def _pad_cols(w: torch.Tensor, cols: int) -> torch.Tensor:
 
 def _pad8(n: int) -> int:
     return (n + 7) // 8 * 8
+
+
+def _pad_heads(w: torch.Tensor, heads: int, dim: int, to: int) -> torch.Tensor:
+    """Rows (or entries) of ``heads`` heads of ``dim``, each head zero padded to ``to``."""
+    if dim == to:
+        return w
+    x = w.reshape(heads, dim, *w.shape[1:])
+    return torch.cat([x, x.new_zeros(heads, to - dim, *w.shape[1:])], dim=1).reshape(heads * to, *w.shape[1:])
 
 
 def stack_sections(parts: List[torch.Tensor]):
@@ -103,13 +119,13 @@ class LatentAttention:
         return ops.rope_table(rows, self.spec.rot.dims, self.spec.rot.base, self.w_in.device)
 
     def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
-        lay, pre = self.lay, meta.prefix
+        lay, pre = self.lay, meta.prefix_of(None)
         proj = linear_fwd(x, self.w_in)
         rows = ops.latent_prep(proj, lay, self.norm, self.eps, self._table(meta), meta.positions, meta.slots,
-                               cache.latent[run], want_rows=pre is None)
+                               cache.rows[run]["latent"], want_rows=pre is None)
         cu_k = meta.cu_q
         if pre is not None:
-            rows = ops.latent_gather(cache.latent[run], pre["block_tables"], pre["token_seq"], pre["token_pos"])
+            rows = ops.latent_gather(cache.rows[run]["latent"], pre["block_tables"], pre["token_seq"], pre["token_pos"])
             cu_k = pre["cu_k"]
         kv = linear_fwd(rows[:, :lay.RP], self.w_kv)
         ops.latent_spread_(kv, rows, lay)
@@ -121,10 +137,10 @@ class LatentAttention:
         proj = linear_fwd(x, self.w_in)
         q = torch.empty(b, lay.heads, lay.CP, dtype=x.dtype, device=x.device)
         ops.latent_prep(proj, lay, self.norm, self.eps, self._table(meta), meta.positions, meta.slots,
-                        cache.latent[run], want_rows=False, decode_q=q)
+                        cache.rows[run]["latent"], want_rows=False, decode_q=q)
         heads = proj[:, :lay.heads * lay.qp].view(b, lay.heads, lay.qp)
         torch.bmm(heads[..., :lay.dn].transpose(0, 1), self.w_k, out=q[..., :lay.RP].transpose(0, 1))
-        lat = ops.latent_decode_attention(q, cache.latent[run], lay, meta.block_tables, meta.context_lens,
+        lat = ops.latent_decode_attention(q, cache.rows[run]["latent"], lay, meta.block_tables, meta.context_lens,
                                           meta.max_context, self.spec.scale)
         attn = torch.empty(b, lay.heads, lay.vp, dtype=x.dtype, device=x.device)
         torch.bmm(lat.transpose(0, 1), self.w_v.transpose(1, 2), out=attn.transpose(0, 1))
@@ -158,15 +174,108 @@ class ChannelDelta:
 
     def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
         proj, a, gate = self._project(x)
-        y = ops.delta_prefill(proj, a, gate, self.lay, self.state, cache.ring[run], cache.state[run], meta.tok_seq,
+        y = ops.delta_prefill(proj, a, gate, self.lay, self.state, cache.slots[run]["ring"], cache.slots[run]["state"], meta.tok_seq,
                               meta.cu_q, meta.start_pos, meta.state_slots, self.eps)
         return linear_fwd(y, self.w_o)
 
     def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
         proj, a, gate = self._project(x)
-        y = ops.delta_decode(proj, a, gate, self.lay, self.state, cache.ring[run], cache.state[run], meta.positions,
+        y = ops.delta_decode(proj, a, gate, self.lay, self.state, cache.slots[run]["ring"], cache.slots[run]["state"], meta.positions,
                              meta.state_slots, self.eps)
         return linear_fwd(y, self.w_o)
 
 
-MIXERS = {"latent_attention": LatentAttention, "channel_delta": ChannelDelta}
+class WindowAttention:
+    """Grouped-head attention over a window of paged keys and values.  Heads are stored padded (``padded_heads``):
+    zero rows and columns in the weights, so that sums of squares and products are unchanged."""
+
+    def __init__(self, spec, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.spec, self.eps = spec, eps
+        h, g = spec.heads, spec.kv_heads
+        qp, vp = spec.padded(dtype)
+        f32 = torch.float32
+
+        def put(t, dt=dtype):
+            return t.to(device=device, dtype=dt).contiguous()
+
+        def pad(t, heads, dim, to):
+            return _pad_heads(t, heads, dim, to)
+
+        parts = [(w["q"], w["q.b"], h, spec.dim, qp), (w["k"], w["k.b"], g, spec.dim, qp), (w["v"], w["v.b"], g, spec.vdim, vp)]
+        fused, cols = stack_sections([pad(t, n, d, p) for t, _, n, d, p in parts])
+        bias = torch.zeros(fused.shape[0], dtype=w["q.b"].dtype)
+        for c, (_, b, n, d, p) in zip(cols, parts):
+            bias[c:c + n * p] = pad(b, n, d, p)
+        self.lay = GroupedHeads(h, g, spec.dim, spec.vdim, qp, vp, *cols)
+        self.w_in, self.b_in = put(fused), put(bias)
+        self.q_norm = put(pad(w["q.norm"], h, spec.dim, qp), f32)
+        self.k_norm = put(pad(w["k.norm"], g, spec.dim, qp), f32)
+        self.mix = put(w["vmix"].reshape(1), f32) if spec.value_mix else None
+        if not spec.value_mix and "vmix" in w:
+            w["vmix"]                                                   # stored but without a use
+        self.w_o = put(_pad_cols(w["o"].reshape(-1, h, spec.vdim), vp).reshape(-1, h * vp))
+
+    def _project(self, x: torch.Tensor, meta: StepMeta, rows: Dict[str, torch.Tensor]) -> torch.Tensor:
+        """Normed, rotated and mixed q | k | v rows, written to the cache."""
+        lay, spec = self.lay, self.spec
+        proj = linear_fwd(x, self.w_in, self.b_in)
+        length = 1 << max(meta.max_model_len - 1, 1).bit_length()       # see LatentAttention._table
+        table = ops.angle_table(length, spec.rot.frequencies(), x.device)
+        first = meta.first_values if spec.value_mix else None
+        ops.qkv_prep_(proj, lay, self.q_norm, self.k_norm, self.eps, table, meta.positions, meta.slots, rows["k"], rows["v"],
+                      first, self.mix)
+        if spec.value_mix and first is None:
+            meta.first_values = lay.values(proj)
+        return proj
+
+    def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        rows, pre, spec = cache.rows[run], meta.prefix_of(self.spec.window), self.spec
+        proj = self._project(x, meta, rows)
+        kv, cu_k = None, meta.cu_q
+        if pre is not None:
+            kv = tuple(ops.rows_gather(rows[n], pre["block_tables"], pre["token_seq"], pre["token_pos"]) for n in ("k", "v"))
+            cu_k = pre["cu_k"]
+        attn = ops.window_prefill_attention(proj, self.lay, meta.cu_q, cu_k, meta.max_q, spec.scale, spec.window, kv)
+        return linear_fwd(attn, self.w_o)
+
+    def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        rows, spec = cache.rows[run], self.spec
+        proj = self._project(x, meta, rows)
+        attn = ops.window_decode_attention(proj, self.lay, rows["k"], rows["v"], meta.block_tables, meta.context_lens,
+                                           meta.max_context, spec.scale, spec.window)
+        return linear_fwd(attn, self.w_o)
+
+
+class MatrixMemory:
+    """Head rows are padded to multiples of 16 (zero rows: padded keys and values leave the memory's padding zero);
+    gate logits are a product of their own with a 32-bit result."""
+
+    def __init__(self, spec, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.spec, self.eps = spec, eps
+        h, d, dv = spec.heads, spec.dim, spec.vdim
+        dp, vp = pad16(d), pad16(dv)
+
+        def put(t, dt=dtype):
+            return t.to(device=device, dtype=dt).contiguous()
+
+        fused, cols = stack_sections([_pad_heads(w["q"], h, d, dp), _pad_heads(w["k"], h, d, dp),
+                                      _pad_heads(w["v"], h, dv, vp), _pad_heads(w["g"], h, dv, vp)])
+        self.lay = MemoryLayout(h, dp, vp, dv, *cols, scale=d ** -0.5, cap=spec.gate_cap, floor=spec.floor)
+        self.w_in, self.w_gates = put(fused), put(torch.cat([w["i"], w["f"]]))
+        self.memory = MemoryWeights(bias=put(torch.cat([w["i.b"], w["f.b"]]), torch.float32),
+                                    norm=put(_pad_heads(w["norm"], h, dv, vp), torch.float32))
+        self.w_o = put(_pad_cols(w["o"].reshape(-1, h, dv), vp).reshape(-1, h * vp))
+
+    def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        y = ops.memory_prefill(linear_fwd(x, self.w_in), linear_f32(x, self.w_gates), self.lay, self.memory, cache.slots[run],
+                               meta.cu_q, meta.max_q, meta.start_pos, meta.state_slots, self.eps)
+        return linear_fwd(y, self.w_o)
+
+    def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        y = ops.memory_decode(linear_fwd(x, self.w_in), linear_f32(x, self.w_gates), self.lay, self.memory, cache.slots[run],
+                              meta.positions, meta.state_slots, self.eps)
+        return linear_fwd(y, self.w_o)
+
+
+MIXERS = {LatentAttentionSpec: LatentAttention, ChannelDeltaSpec: ChannelDelta, WindowAttentionSpec: WindowAttention,
+          MatrixMemorySpec: MatrixMemory}

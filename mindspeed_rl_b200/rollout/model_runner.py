@@ -97,6 +97,7 @@ class ModelRunner:
         self._static: Optional[dict] = None
         if cfg.is_hybrid and self.comm.world_size > 1:
             raise NotImplementedError(f"{cfg.architecture} is served on one GPU per replica (tensor parallel size 1)")
+        self._side = None         # second stream of captured decode steps
         self.layer_probe = None   # callable(run, residual [T, W] fp32) after every layer run of a hybrid decoder (eager steps)
         self.prefix_tile = 0      # key tile of the tcgen05 shared-prefix kernel (set by the engine; 0 = mma.sync kernel)
 
@@ -203,22 +204,47 @@ class ModelRunner:
         """Final hidden states ``[T, H]`` of a layer-by-layer decoder: the fp32 residual is updated in place by
         kernels that add and take the next norm in one pass."""
         w, c, cache = self.weights, self.cfg, self.cache
-        eps, off = c.norm_epsilon, c.norm_offset
-        order = c.run_order
-        resid, x = ops.embed_norm(meta.ids, w.embed, c.embedding_scale, w.layers[order[0]].norm1, eps, off)
+        order, parallel = c.run_order, c.design.parallel
+
+        def norm(weight):
+            return ops.Norm(weight, c.norm_epsilon, c.design.norm_offset, c.design.centered)
+
+        resid, x = ops.embed_norm(meta.ids, w.embed, c.embedding_scale, *norm(w.layers[order[0]].norm1))
         for run, li in enumerate(order):
             lw = w.layers[li]
-            after = w.layers[order[run + 1]].norm1 if run + 1 < len(order) else w.final_norm
+            after = norm(w.layers[order[run + 1]].norm1 if run + 1 < len(order) else w.final_norm)
             mix = lw.mixer.decode if meta.is_decode else lw.mixer.prefill
-            delta = mix(x, meta, cache, run)
-            if lw.ff is None:
-                x = ops.add_norm_(resid, delta, after, eps, off)
+            if parallel and lw.ff is not None:
+                join = self._beside(meta, lambda: lw.ff.forward(x, meta.ids))
+                delta = mix(x, meta, cache, run)
+                x = lw.ff.finish_(resid, x, join(), after, delta)
+            elif lw.ff is not None:
+                x = ops.add_norm_(resid, mix(x, meta, cache, run), *norm(lw.norm2))
+                x = lw.ff.finish_(resid, x, lw.ff.forward(x, meta.ids), after)
             else:
-                x = ops.add_norm_(resid, delta, lw.norm2, eps, off)
-                x = lw.ff.forward_norm_(resid, x, meta.ids, after, eps, off)
+                x = ops.add_norm_(resid, mix(x, meta, cache, run), *after)
             if self.layer_probe is not None:
                 self.layer_probe(run, resid)
         return x
+
+    def _beside(self, meta: StepMeta, work):
+        """Start ``work`` beside what the caller launches next; the returned function waits for it and gives its
+        result.  Small decode steps leave most of the machine idle, so there the two run on two streams (inside
+        a capture the fork and the join become edges of the graph); elsewhere one after the other."""
+        if not (meta.is_decode and meta.ids.is_cuda and torch.cuda.is_current_stream_capturing()):
+            return work
+        main = torch.cuda.current_stream()
+        if self._side is None:
+            self._side = torch.cuda.Stream(self.device)
+        side = self._side
+        side.wait_stream(main)
+        with torch.cuda.stream(side):
+            out = work()
+
+        def join():
+            main.wait_stream(side)
+            return out
+        return join
 
     def _logits(self, x: torch.Tensor) -> torch.Tensor:
         return linear_fwd(x, self.weights.lm_head)
@@ -233,7 +259,8 @@ class ModelRunner:
 
         ``prefix`` (for chunks that start inside a sequence) carries ``block_tables``,
         ``token_seq``, ``token_pos``, ``cu_k``: the K/V of ``[0, chunk_end)`` is gathered from the
-        cache after this chunk's K/V has been written.
+        cache after this chunk's K/V has been written.  Hybrid decoders get one such dictionary per key range
+        of their attention layers (``HybridConfig.windows``), which lists only the keys inside the range.
 
         ``state`` (hybrid decoders): ``token_seq [T]`` and ``start_pos [B]`` (int32), ``slots [B]`` (int64, the
         recurrent-state slot of every sequence).

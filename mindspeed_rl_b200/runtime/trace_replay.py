@@ -38,14 +38,13 @@ def parse(argv=None):
 def build_engine(args):
     import torch
 
-    from ..models.registry import load_model
-    from ..ops import _lib
+    from ..models.registry import load_model, use_kernels_of
     from ..rollout.engine import LLMEngine
 
     if args.device == "cuda":
         if not torch.cuda.is_available():
             raise RuntimeError("no CUDA device (use --device cpu for the PyTorch formulation)")
-        _lib.use_group("hybrid")
+        use_kernels_of(args.model)
     torch.backends.cuda.matmul.allow_tf32 = False
     torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
     cfg, weights = load_model(args.model, getattr(torch, args.dtype), args.device)

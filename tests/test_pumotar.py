@@ -159,8 +159,8 @@ def test_looped_layers_run_in_order_with_a_cache_each():
     assert HybridConfig.from_json(M.ZOO["grouped_heads"]).run_order == [0, 1]
     eng = make_engine("mixed", "cpu")
     cache = eng.runner.cache
-    assert [c is not None for c in cache.latent] == [False, True, False, True, False]
-    ptrs = [c.data_ptr() for c in cache.latent if c is not None] + [c.data_ptr() for c in cache.state if c is not None]
+    assert ["latent" in c for c in cache.rows] == [False, True, False, True, False]
+    ptrs = [c["latent"].data_ptr() for c in cache.rows if c] + [c["state"].data_ptr() for c in cache.slots if c]
     assert len(set(ptrs)) == 5
     assert eng.kv_bytes_per_block() == 2 * 16 * (32 + 16) * 4 and eng.state_bytes() > 0
 
