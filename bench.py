@@ -54,8 +54,9 @@ def parse_args():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="grpo", choices=["grpo", "serve"],
                     help="grpo: the headline benchmark; serve: prefill and decode throughput of the layer-by-layer "
-                         "decoder (Pumotar) beside the latent-attention decoder of equal size, one JSON line per case")
+                         "decoders (Pumotar, Sunatar) beside the closest decoders of equal size, one JSON line per case")
     ap.add_argument("--serve-sizes", default="", help="comma-separated subset of the serve workload's sizes")
+    ap.add_argument("--serve-models", default="", help="comma-separated subset of the serve workload's models")
     ap.add_argument("--model", default="qwen25_7b")
     ap.add_argument("--prompts-per-gpu", type=int, default=32)
     ap.add_argument("--samples", type=int, default=8)
@@ -155,6 +156,7 @@ def main():
         from mindspeed_rl_b200.rollout import serve_bench
 
         serve_bench.run(args.steps, args.warmup, [x for x in args.serve_sizes.split(",") if x],
+                        [x for x in args.serve_models.split(",") if x],
                         emit=lambda line: print(line, flush=True))
         return
     import torch

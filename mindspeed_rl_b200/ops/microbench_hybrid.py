@@ -8,8 +8,10 @@ from __future__ import annotations
 
 import torch
 
-from . import (DeltaLayout, DeltaWeights, LatentLayout, add_norm_, delta_decode, delta_prefill, embed_norm, glu_fwd,
-               latent_decode_attention, latent_prefill_attention, latent_prep, latent_spread_, moe_combine_norm_, rope_table)
+from . import (DeltaLayout, DeltaWeights, GroupedHeads, LatentLayout, MemoryLayout, MemoryWeights, add_norm_, angle_table,
+               delta_decode, delta_prefill, embed_norm, glu_fwd, latent_decode_attention, latent_prefill_attention, latent_prep,
+               latent_spread_, memory_decode, memory_prefill, moe_combine_norm_, qkv_prep_, rope_table, rows_gather,
+               window_decode_attention, window_prefill_attention)
 from . import moe as K
 from .microbench import report, timeit
 
@@ -119,4 +121,82 @@ def case_stream(small: bool, iters: int):
         report(f"moe_combine_norm T={t} k={k} H={h}", ms, bytes_=t * h * (2.0 * k + 4 + 8 + 2))
 
 
-CASES = {"hybrid_delta": case_delta, "hybrid_latent": case_latent, "hybrid_stream": case_stream}
+def _memory(t, slots, heads, dim, vdim):
+    n = heads * (2 * dim + 2 * vdim)
+    lay = MemoryLayout(heads, dim, vdim, vdim, 0, heads * dim, 2 * heads * dim, heads * (2 * dim + vdim), dim ** -0.5, 15.0)
+    w = MemoryWeights(torch.zeros(2 * heads, device="cuda"), torch.ones(heads * vdim, device="cuda"))
+    state = {"memory": torch.zeros(slots, heads, dim, vdim, device="cuda"), "norm": torch.zeros(slots, heads, dim, device="cuda"),
+             "peak": torch.zeros(slots, heads, device="cuda")}
+    return lay, torch.randn(t, n, device="cuda").bfloat16(), torch.randn(t, 2 * heads, device="cuda"), w, state
+
+
+def case_memory(small: bool, iters: int):
+    """Roofline of prompts: the rows read and written once (the recurrence's products are far below the tensor peak)."""
+    for heads, dim, vdim in ((32, 128, 128), (8, 256, 512)):
+        for b, n in ([(1, 2048)] if small else [(1, 8192), (8, 1024), (32, 256)]):
+            t = b * n
+            lay, proj, z, w, state = _memory(t, b, heads, dim, vdim)
+            cu = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda")
+            start, slots = torch.zeros(b, dtype=torch.int32, device="cuda"), torch.arange(b, device="cuda")
+            ms = timeit(lambda: memory_prefill(proj, z, lay, w, state, cu, n, start, slots, 1e-5), iters)
+            report(f"memory_prefill {b}x{n} heads={heads} {dim}x{vdim}", ms, bytes_=2.0 * t * heads * (2 * dim + 3 * vdim),
+                   flops=4.0 * t * heads * dim * vdim)
+        for b in ([32] if small else [1, 32, 256]):
+            lay, proj, z, w, state = _memory(b, b, heads, dim, vdim)
+            pos, slots = torch.full((b,), 100, dtype=torch.int32, device="cuda"), torch.randperm(b, device="cuda")
+            ms = timeit(lambda: memory_decode(proj, z, lay, w, state, pos, slots, 1e-5), iters)
+            report(f"memory_decode B={b} heads={heads} {dim}x{vdim}", ms, bytes_=8.0 * state["memory"].numel())
+
+
+def case_window(small: bool, iters: int):
+    h, g, d = 32, 8, 128
+    lay = GroupedHeads(h, g, d, d, d, d, 0, h * d, (h + g) * d)
+    t, n = (2048, 2048) if small else (16384, 8192)
+    for window in (None, 4096, 1024):
+        proj = torch.randn(t, (h + 2 * g) * d, device="cuda").bfloat16()
+        cu = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda")
+        w = min(window or n, n)
+        pairs = t // n * (w * (w + 1) / 2 + (n - w) * w)
+        ms = timeit(lambda: window_prefill_attention(proj, lay, cu, cu, n, d ** -0.5, window), iters)
+        report(f"window_prefill_attention {t // n}x{n} H={h}/{g} window={window}", ms, flops=4.0 * pairs * h * d)
+    pos, slots = torch.arange(t, dtype=torch.int32, device="cuda") % n, torch.arange(t, device="cuda")
+    kc, vc = (torch.empty(t // 16, 16, g, d, device="cuda").bfloat16() for _ in range(2))
+    tab = angle_table(8192, tuple(1e4 ** (-i / 64) for i in range(64)), proj.device)
+    qn, kn, mix = torch.ones(h * d, device="cuda"), torch.ones(g * d, device="cuda"), torch.full((1,), 0.3, device="cuda")
+    other = lay.values(torch.randn_like(proj))
+    ms = timeit(lambda: qkv_prep_(proj, lay, qn, kn, 1e-5, tab, pos, slots, kc, vc, other, mix), iters)
+    report(f"qkv_prep T={t} H={h}/{g} d={d}", ms, bytes_=2.0 * t * d * (2 * h + 4 * g + 3 * g))
+    bt = torch.randperm(t // 16, device="cuda").to(torch.int32).view(1, -1)
+    seq, at = torch.zeros(t, dtype=torch.int32, device="cuda"), torch.arange(t, dtype=torch.int32, device="cuda")
+    ms = timeit(lambda: rows_gather(kc, bt, seq, at), iters)
+    report(f"rows_gather T={t} row={g * d}", ms, bytes_=4.0 * t * g * d)
+    for b, ctx, window in ([(16, 1024, None)] if small else [(256, 2048, None), (256, 8192, 1024), (32, 8192, 4096), (1, 8192, 4096)]):
+        nb = b * ctx // 16
+        kc, vc = (torch.randn(nb, 16, g, d, device="cuda").bfloat16() for _ in range(2))
+        bt = torch.randperm(nb, device="cuda").to(torch.int32).view(b, -1)
+        cl = torch.full((b,), ctx, dtype=torch.int32, device="cuda")
+        q = torch.randn(b, (h + 2 * g) * d, device="cuda").bfloat16()
+        ms = timeit(lambda: window_decode_attention(q, lay, kc, vc, bt, cl, ctx, d ** -0.5, window), iters)
+        report(f"window_decode H={h}/{g} B={b} ctx={ctx} window={window}", ms, bytes_=4.0 * b * min(ctx, window or ctx) * g * d)
+
+
+def case_routed(small: bool, iters: int):
+    """What scored experts in parallel layers add: router, weighted permutation, centred norm with the mixer's output."""
+    e, k, h = 64, 8, 2304
+    for t in ([2048] if small else [16384, 256]):
+        x, z = torch.randn(t, h, device="cuda").bfloat16(), torch.randn(t, e, device="cuda")
+        ms = timeit(lambda: K.route_top(z, k), iters)
+        report(f"route_top T={t} E={e} k={k}", ms, bytes_=t * (4.0 * e + 12 * k))
+        idx, score = K.route_top(z, k)
+        plan = K.moe_plan(idx, e)
+        ms = timeit(lambda: K.moe_permute(x, plan, score), iters)
+        report(f"moe_permute weighted T={t} k={k} H={h}", ms, bytes_=2.0 * t * h * (k + 1))
+        y, sh, mixer = torch.randn(plan.max_rows, h, device="cuda").bfloat16(), torch.randn_like(x), torch.randn_like(x)
+        resid, w = torch.zeros(t, h, device="cuda"), torch.ones(h, device="cuda")
+        ms = timeit(lambda: moe_combine_norm_(resid, y, plan.pos, k, 1.0, x, sh, None, w, 1e-5, 0.0, True, delta=mixer), iters)
+        report(f"moe_combine_norm centred + mixer T={t} k={k} H={h}", ms, bytes_=t * h * (2.0 * k + 4 + 8 + 2))
+        ms = timeit(lambda: add_norm_(resid, mixer, w, 1e-5, 0.0, True), iters)
+        report(f"add_norm centred {t}x{h}", ms, bytes_=t * h * 12.0)
+
+
+CASES = {"hybrid_memory": case_memory, "hybrid_window": case_window, "hybrid_routed": case_routed, "hybrid_delta": case_delta, "hybrid_latent": case_latent, "hybrid_stream": case_stream}

@@ -1,11 +1,17 @@
-"""Serving throughput of a layer-by-layer decoder beside the closest repeated-block decoder of equal size.
+"""Serving throughput of layer-by-layer decoders beside the closest repeated-block decoders of equal size.
 
 ``bench.py --workload serve`` runs it: random weights, prompts and decode batches through ``LLMEngine`` (the
-scheduler, cache, graphs and sampler of generation).  The closest existing model is the latent-attention (MLA)
-decoder with routed experts: same width, heads, head sizes, latent rank, feed-forward sizes, experts and layer
-count.  It caches full per-head keys and values; the layer-by-layer decoder caches latent rows and recurrent
-state.  ``mixed`` puts one latent-attention layer after three recurrent ones, ``latent`` uses latent attention
-everywhere.  One JSON line per measurement: tokens/s from CUDA events around the engine calls.
+scheduler, cache, graphs and sampler of generation).
+
+Pumotar: ``latent`` has latent attention everywhere, ``mixed`` one such layer after three recurrent ones.  Closest
+existing model: ``mla``, the latent-attention decoder with routed experts of the same width, heads, head sizes, latent
+rank, feed-forward sizes, experts and layer count; it caches full per-head keys and values.
+
+Sunatar: ``window`` has window attention everywhere, ``memory`` the matrix memory everywhere, ``sunatar`` one
+matrix-memory layer in four.  Closest existing models: ``gqa``, the grouped-head decoder with routed and shared experts
+of the same width, heads, experts and layer count (full attention), and for the recurrent layers ``mixed``.
+
+One JSON line per measurement: tokens/s from CUDA events around the engine calls.
 """
 from __future__ import annotations
 
@@ -15,7 +21,8 @@ from typing import List
 
 import torch
 
-from ..models.hybrid_config import ChannelDeltaSpec, GluSpec, HybridConfig, LatentAttentionSpec, LayerSpec, Rotary, TableMoESpec
+from ..models.hybrid_config import (ChannelDeltaSpec, GluSpec, HybridConfig, LatentAttentionSpec, LayerSpec, MatrixMemorySpec,
+                                    Rotary, ScoredMoESpec, TableMoESpec, WavelengthScaling, WindowAttentionSpec)
 from ..models.transformer_config import TransformerConfig
 from .engine import LLMEngine
 from .scheduler import SamplingParams
@@ -43,9 +50,26 @@ SIZES = (Size("1k", 1024, 8, 256, 4096, 32, 4, 512), Size("2k", 2304, 32, 512, 9
 PREFILL = ((1, 8192), (8, 2048))
 DECODE = ((1, 2048), (32, 2048), (256, 2048))
 NEW_TOKENS = 64
+WINDOW = 1024
+MODELS = ("mla", "latent", "mixed", "gqa", "window", "memory", "sunatar")
+
+
+def sunatar_config(s: Size, pattern: str) -> HybridConfig:
+    rot = Rotary(64, 500000.0, halves=True, scaling=WavelengthScaling(8.0, 1.0, 4.0, 8192))
+    window = LayerSpec("attention", WindowAttentionSpec(s.heads, s.heads // 4, 128, 128, 128 ** -0.5, rot, WINDOW, True))
+    memory = LayerSpec("mlstm", MatrixMemorySpec(s.heads, 128, 128, 15.0))
+    glu = GluSpec(s.expert_ff, "silu")
+    moe = ScoredMoESpec(s.experts, s.top, glu, glu)
+    layers = []
+    for i in range(s.layers):
+        m = memory if pattern == "memory" or (pattern == "sunatar" and i % 4 == 2) else window
+        layers.append(LayerSpec(m.type, m.mixer, moe))
+    return HybridConfig("Sunatar", s.vocab, s.width, layers, 1e-5)
 
 
 def hybrid_config(s: Size, pattern: str) -> HybridConfig:
+    if pattern in ("window", "memory", "sunatar"):
+        return sunatar_config(s, pattern)
     latent = LayerSpec("latent_attention", LatentAttentionSpec(s.heads, s.dn, s.dr, s.dv, s.rank, (s.dn + s.dr) ** -0.5,
                                                                Rotary(s.dr, 10000.0)))
     delta = LayerSpec("channel_delta", ChannelDeltaSpec(s.heads, s.heads, 128, 128, 4))
@@ -76,17 +100,37 @@ def random_state(cfg: HybridConfig, device) -> dict:
         lin(p + "down", w, ff)
 
     lin("embed", cfg.vocab_size, w)
-    vec("final.norm", w)
+    ones = 1.0 - cfg.design.norm_offset
+    vec("final.norm", w, ones)
+    if not cfg.design.tied_head:
+        lin("head", cfg.vocab_size, w)
     for i, l in enumerate(cfg.layers):
         p, m = f"l{i}.mix.", l.mixer
-        vec(f"l{i}.norm1", w)
-        vec(f"l{i}.norm2", w)
+        vec(f"l{i}.norm1", w, ones)
+        if not cfg.design.parallel:
+            vec(f"l{i}.norm2", w)
         if l.type == "latent_attention":
             lin(p + "q", m.heads * (m.dim + m.rot_dim), w)
             lin(p + "dkv", m.kv_rank + m.rot_dim, w)
             vec(p + "dkv.norm", m.kv_rank, 1.0)
             lin(p + "uk", m.heads * m.dim, m.kv_rank)
             lin(p + "uv", m.heads * m.vdim, m.kv_rank)
+            lin(p + "o", w, m.heads * m.vdim)
+        elif l.type == "attention":
+            for n, rows in (("q", m.heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
+                lin(p + n, rows, w)
+                vec(p + n + ".b", rows)
+            vec(p + "q.norm", m.heads * m.dim, 1.0)
+            vec(p + "k.norm", m.kv_heads * m.dim, 1.0)
+            out[p + "vmix"] = torch.tensor(0.3, device=device)
+            lin(p + "o", w, m.heads * m.vdim)
+        elif l.type == "mlstm":
+            for n, rows in (("q", m.heads * m.dim), ("k", m.heads * m.dim), ("v", m.heads * m.vdim), ("g", m.heads * m.vdim),
+                            ("i", m.heads), ("f", m.heads)):
+                lin(p + n, rows, w)
+            vec(p + "i.b", m.heads)
+            vec(p + "f.b", m.heads, 3.0)
+            vec(p + "norm", m.heads * m.vdim, 1.0)
             lin(p + "o", w, m.heads * m.vdim)
         else:
             kd, hv = m.kv_heads * m.dim, m.heads * m.vdim
@@ -102,7 +146,12 @@ def random_state(cfg: HybridConfig, device) -> dict:
                 lin(p + a + "2", n, 128)
             lin(p + "o", w, hv)
         p = f"l{i}.mlp."
-        if isinstance(l.mlp, TableMoESpec):
+        if isinstance(l.mlp, ScoredMoESpec):
+            for e in range(l.mlp.experts):
+                glu(f"{p}e{e}.", l.mlp.expert.ff)
+            lin(p + "router", l.mlp.experts, w)
+            glu(p + "shared.", l.mlp.shared.ff)
+        elif isinstance(l.mlp, TableMoESpec):
             for e in range(l.mlp.experts):
                 glu(f"{p}e{e}.", l.mlp.expert.ff)
             out[p + "table"] = torch.rand(cfg.vocab_size, l.mlp.experts, generator=g, device=device).topk(l.mlp.top, -1).indices
@@ -122,12 +171,19 @@ def mla_config(s: Size) -> TransformerConfig:
                              v_head_dim=s.dv)
 
 
+def gqa_config(s: Size) -> TransformerConfig:
+    return TransformerConfig(num_layers=s.layers, hidden_size=s.width, ffn_hidden_size=s.ff, num_attention_heads=s.heads,
+                             num_query_groups=s.heads // 4, kv_channels=128, vocab_size=s.vocab, norm_epsilon=1e-5,
+                             max_position_embeddings=16384, qk_layernorm=True, untie_embeddings_and_output_weights=True,
+                             num_experts=s.experts, moe_router_topk=s.top, moe_ffn_hidden_size=s.expert_ff, n_shared_experts=1)
+
+
 def build(s: Size, model: str, device):
-    if model == "mla":
+    if model in ("mla", "gqa"):
         from ..models.gpt import GPTModel
         from ..reshard.alias import alias_rollout_weights
 
-        cfg = mla_config(s)
+        cfg = mla_config(s) if model == "mla" else gqa_config(s)
         return cfg, alias_rollout_weights(GPTModel(cfg, device=device))
     from .hybrid_weights import build_hybrid_weights
 
@@ -145,14 +201,14 @@ def _timed(fn) -> float:
     return e0.elapsed_time(e1)
 
 
-def run(steps: int, warmup: int, sizes=None, models=("mla", "latent", "mixed"), emit=print) -> List[dict]:
+def run(steps: int, warmup: int, sizes=None, models=None, emit=print) -> List[dict]:
     dev = torch.device("cuda")
     rows = []
     for s in SIZES:
         if sizes and s.name not in sizes:
             continue
         gen = torch.Generator().manual_seed(1)
-        for model in models:
+        for model in models or MODELS:
             cfg, weights = build(s, model, dev)
             bs = max(b for b, _ in DECODE)
             ctx = max(n for _, n in DECODE) + NEW_TOKENS
