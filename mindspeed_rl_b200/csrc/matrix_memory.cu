@@ -19,42 +19,15 @@
 //               chunk_state   U = sum_s e^(a_s - max a) k_s v_s^T of every chunk
 //               carry         running state over the chunks, element by element; leaves the state before every chunk
 //               chunk_out     (Q K^T with the weights) V + (Q S) with the weights, denominators, norm and gate
-//             Products run on the tensor cores with 32-bit operands (weights times keys, weighted scores, the state)
-//             taken apart into three bf16 terms of 24 bits together; the other operand is exact, sums are fp32.
+//             chunk_state and chunk_out are in matrix_memory_tcgen05.cu.
 #include <cooperative_groups.h>
 
-#include "dtype_utils.cuh"
-#include "mma_utils.cuh"
+#include "matrix_memory.cuh"
 
 namespace msrl {
 namespace mem {
 
 namespace cg = cooperative_groups;
-
-template <typename T>
-struct Args {
-  const T* proj;                         // [tokens, ld]: q | k | v | gate sections at the given columns
-  long long ld;
-  const float* z;                        // [tokens, z_ld]: input gate logits [H] | forget gate logits [H]
-  long long z_ld;
-  int H, dim, vdim, rms_dim, q_col, k_col, v_col, g_col;
-  float scale, cap, floor, eps;
-  const float* bias;                     // [2 H]
-  const float* norm;                     // [H * vdim]
-  float *memory, *nrm, *peak;
-  const int* cu;
-  const int* start;                      // position of a portion's first token
-  const long long* slots;
-  T* y;                                  // [tokens, H * vdim]
-};
-
-template <typename T>
-__device__ __forceinline__ void log_gates(const Args<T>& p, long long t, int h, float& i, float& f) {
-  const float* z = p.z + t * p.z_ld + h;
-  i = p.cap * tanhf((z[0] + p.bias[h]) / p.cap);
-  const float x = p.cap * tanhf((z[p.H] + p.bias[p.H + h]) / p.cap);
-  f = fminf(x, 0.f) - log1pf(expf(-fabsf(x)));
-}
 
 // ---- decode -----------------------------------------------------------------------------------------------
 constexpr int DB = 8, DC = 4;            // state rows of a thread in flight, output columns of a thread (of 256 DC)
@@ -304,170 +277,8 @@ __global__ void __launch_bounds__(256) finish_kernel(const Args<T> p, const floa
   }
 }
 
-// ---- prompts in chunks (bf16) -------------------------------------------------------------------------------
+// ---- prompts in chunks (bf16): the pass over the chunks ------------------------------------------------------------
 using bf16 = __nv_bfloat16;
-constexpr int C = 128, VW = 128, LDV = VW + 8, SB = 64, DBLK = 32;
-constexpr int TERMS = 3;
-
-struct Chunks {
-  float* state;                          // [chunks, H, dim * vdim + dim]: U and its n part, then the state before the chunk
-  float *top, *sum, *before;             // [chunks, H]: max a, sum of f, m before the chunk
-  float *a, *run, *b;                    // [H, tokens]: a, running max of a, sum of f inside the chunk
-  float* o;                              // [tokens, H * vdim] when a head does not fit one block's columns
-  int tokens;
-};
-
-__device__ __forceinline__ long long chunk_id(int t0, int b, int j) { return t0 / C + b + j; }
-
-// x (two values of a fragment register) as TERMS bf16 registers whose sum is x to 24 bits
-__device__ __forceinline__ void split(float x0, float x1, uint32_t (&r)[TERMS]) {
-#pragma unroll
-  for (int i = 0; i < TERMS; ++i) {
-    const __nv_bfloat162 v = __floats2bfloat162_rn(x0, x1);
-    r[i] = *reinterpret_cast<const uint32_t*>(&v);
-    const float2 f = __bfloat1622float2(v);
-    x0 -= f.x;
-    x1 -= f.y;
-  }
-}
-
-// rows [row0, row0 + ROWS) of a section (`cols` wide, a multiple of 8) into shared memory; rows past `len` and columns
-// [cols, fill) are zero
-__device__ __forceinline__ void load_rows(bf16* dst, int ld, const bf16* src, long long src_ld, int rows, int row0, int len,
-                                          int cols, int fill) {
-  const int vecs = fill / 8;
-  for (int i = threadIdx.x; i < rows * vecs; i += 256) {
-    const int r = i / vecs, c = (i - r * vecs) * 8;
-    const bool ok = row0 + r < len && c < cols;
-    cp_async16(dst + r * ld + c, src + (long long)(ok ? row0 + r : 0) * src_ld + (ok ? c : 0), ok);
-  }
-}
-
-// grid (chunks x column blocks, H, B)
-__global__ void __launch_bounds__(256, 2) chunk_state_kernel(const Args<bf16> p, const Chunks ch) {
-  extern __shared__ __align__(16) unsigned char raw[];
-  __shared__ float w[C];
-  const int ldk = p.dim + 8, vblocks = (p.vdim + VW - 1) / VW;
-  bf16* sK = reinterpret_cast<bf16*>(raw);
-  bf16* sV = sK + C * ldk;
-  const int j = blockIdx.x / vblocks, vb = blockIdx.x % vblocks, h = blockIdx.y, b = blockIdx.z;
-  const int t0 = p.cu[b], len = min(p.cu[b + 1] - t0 - j * C, C);
-  if (len <= 0) return;
-  const long long first = t0 + j * C, id = chunk_id(t0, b, j) * p.H + h;
-  const int width = min(VW, p.vdim - vb * VW);
-  const bf16* rows = p.proj + first * p.ld;
-  load_rows(sK, ldk, rows + p.k_col + h * p.dim, p.ld, C, 0, len, p.dim, p.dim);
-  load_rows(sV, LDV, rows + p.v_col + h * p.vdim + vb * VW, p.ld, C, 0, len, width, width);
-  cp_async_commit();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (warp == 0) {                       // gates of the chunk, four tokens per lane
-    float a[4], run[4], bs[4], sum = 0.f;
-#pragma unroll
-    for (int x = 0; x < 4; ++x) {
-      const int s = lane * 4 + x;
-      float gi = -INFINITY, gf = 0.f;
-      if (s < len) log_gates(p, first + s, h, gi, gf);
-      a[x] = gi;
-      sum += gf;
-      bs[x] = sum;
-    }
-    float before = sum;
-#pragma unroll
-    for (int d = 1; d < 32; d <<= 1) {
-      const float o = __shfl_up_sync(0xffffffffu, before, d);
-      if (lane >= d) before += o;
-    }
-    const float total = __shfl_sync(0xffffffffu, before, 31);
-    before -= sum;
-    float top = -INFINITY;
-#pragma unroll
-    for (int x = 0; x < 4; ++x) {
-      bs[x] += before;
-      a[x] -= bs[x];
-      top = fmaxf(top, a[x]);
-      run[x] = top;
-    }
-    float peak = top;
-#pragma unroll
-    for (int d = 1; d < 32; d <<= 1) {
-      const float o = __shfl_up_sync(0xffffffffu, peak, d);
-      if (lane >= d) peak = fmaxf(peak, o);
-    }
-    const float all = __shfl_sync(0xffffffffu, peak, 31);
-    float left = __shfl_up_sync(0xffffffffu, peak, 1);
-    if (lane == 0) left = -INFINITY;
-#pragma unroll
-    for (int x = 0; x < 4; ++x) {
-      const int s = lane * 4 + x;
-      w[s] = expf(a[x] - all);
-      if (vb == 0 && s < len) {
-        const long long at = (long long)h * ch.tokens + first + s;
-        ch.a[at] = a[x];
-        ch.run[at] = fmaxf(run[x], left);
-        ch.b[at] = bs[x];
-      }
-    }
-    if (vb == 0 && lane == 0) {
-      ch.top[id] = all;
-      ch.sum[id] = total;
-    }
-  }
-  cp_async_wait<0>();
-  __syncthreads();
-  float* U = ch.state + id * ((long long)p.dim * p.vdim + p.dim);
-  if (vb == 0) {
-    for (int d = threadIdx.x; d < p.dim; d += 256) {
-      float s = 0.f;
-      for (int x = 0; x < len; ++x) s += w[x] * __bfloat162float(sK[x * ldk + d]);
-      U[(long long)p.dim * p.vdim + d] = s;
-    }
-  }
-  const int steps = (len + 15) / 16, ntile = width / 8;
-  for (int mt = warp; mt < p.dim / 16; mt += 8) {
-    float acc[VW / 8][4];
-#pragma unroll
-    for (int n = 0; n < VW / 8; ++n)
-#pragma unroll
-      for (int x = 0; x < 4; ++x) acc[n][x] = 0.f;
-    for (int ks = 0; ks < steps; ++ks) {
-      // K^T fragment: rows = key entries, columns = tokens
-      uint32_t kf[4], at[TERMS][4];
-      ldmatrix_x4_trans(kf, smem_u32(sK + (ks * 16 + (lane >> 4) * 8 + (lane & 7)) * ldk + mt * 16 + ((lane >> 3) & 1) * 8));
-      const float2 wl = *reinterpret_cast<const float2*>(w + ks * 16 + (lane & 3) * 2);
-      const float2 wh = *reinterpret_cast<const float2*>(w + ks * 16 + 8 + (lane & 3) * 2);
-#pragma unroll
-      for (int r = 0; r < 4; ++r) {
-        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&kf[r]));
-        const float2 ww = r < 2 ? wl : wh;
-        uint32_t t3[TERMS];
-        split(f.x * ww.x, f.y * ww.y, t3);
-#pragma unroll
-        for (int i = 0; i < TERMS; ++i) at[i][r] = t3[i];
-      }
-#pragma unroll
-      for (int n = 0; n < VW / 16; ++n) {
-        if (n * 2 < ntile) {
-          uint32_t vf[4];
-          ldmatrix_x4_trans(vf, smem_u32(sV + (ks * 16 + (lane & 15)) * LDV + n * 16 + (lane >> 4) * 8));
-#pragma unroll
-          for (int i = 0; i < TERMS; ++i) {
-            mma_16816(acc[2 * n], at[i], vf[0], vf[1]);
-            mma_16816(acc[2 * n + 1], at[i], vf[2], vf[3]);
-          }
-        }
-      }
-    }
-    const int d = mt * 16 + (lane >> 2);
-#pragma unroll
-    for (int n = 0; n < VW / 8; ++n) {
-      if (n < ntile) {
-        float* dst = U + (long long)d * p.vdim + vb * VW + n * 8 + (lane & 3) * 2;
-        *reinterpret_cast<float2*>(dst) = make_float2(acc[n][0], acc[n][1]);
-        *reinterpret_cast<float2*>(dst + 8ll * p.vdim) = make_float2(acc[n][2], acc[n][3]);
-      }
-    }
-  }
-}
 
 __device__ __forceinline__ float4 blend(float x, const float4& a, float y, const float4& b) {
   return make_float4(x * a.x + y * b.x, x * a.y + y * b.y, x * a.z + y * b.z, x * a.w + y * b.w);
@@ -527,224 +338,6 @@ __global__ void carry_peak_kernel(const Args<bf16> p, const Chunks ch, int batch
   if (len <= 0 || slot < 0) return;
   const long long id = chunk_id(t0, b, (len - 1) / C) * p.H + h;
   p.peak[slot * p.H + h] = ch.sum[id] + fmaxf(ch.before[id], ch.top[id]);
-}
-
-// grid (chunks x column blocks, H, B); NT column tiles of 8 per block
-template <int NT>
-__global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, const Chunks ch) {
-  extern __shared__ __align__(16) unsigned char raw[];
-  __shared__ float sa[C], sM[C], sInter[C], sExp[C], sDen[C];
-  const int ld = p.dim + 8, vblocks = (p.vdim + VW - 1) / VW;
-  bf16* sQ = reinterpret_cast<bf16*>(raw);
-  float* sN = reinterpret_cast<float*>(sQ + C * ld);
-  bf16* sK = reinterpret_cast<bf16*>(sN + p.dim);
-  bf16* sV = sK + SB * ld;
-  bf16* sS = sK;                         // terms of a state block: [TERMS][DBLK][LDV], before the keys and values
-  const int j = blockIdx.x / vblocks, vb = blockIdx.x % vblocks, h = blockIdx.y, b = blockIdx.z;
-  const int t0 = p.cu[b], len = min(p.cu[b + 1] - t0 - j * C, C);
-  if (len <= 0) return;
-  const long long first = t0 + j * C, id = chunk_id(t0, b, j) * p.H + h, size = (long long)p.dim * p.vdim;
-  const bool inter = j > 0 || p.start[b] > 0;                     // a state before the chunk
-  const int width = min(VW, p.vdim - vb * VW), ntile = width / 8;
-  const bf16* rows = p.proj + first * p.ld;
-  load_rows(sQ, ld, rows + p.q_col + h * p.dim, p.ld, C, 0, len, p.dim, p.dim);
-  cp_async_commit();
-  const float* S = ch.state + id * (size + p.dim);
-  if (threadIdx.x < C) {
-    const int s = threadIdx.x;
-    const long long at = (long long)h * ch.tokens + first + s;
-    const float m = ch.before[id], M = s < len ? fmaxf(m, ch.run[at]) : 0.f;
-    sa[s] = s < len ? ch.a[at] : -INFINITY;
-    sM[s] = M;
-    sInter[s] = s < len ? expf(m - M) * p.scale : 0.f;
-    sExp[s] = s < len ? expf(-(ch.b[at] + M)) : 0.f;
-  }
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r0 = warp * 16;
-  float acc[NT][4];
-#pragma unroll
-  for (int n = 0; n < NT; ++n)
-#pragma unroll
-    for (int x = 0; x < 4; ++x) acc[n][x] = 0.f;
-  if (inter) {
-    for (int d = threadIdx.x; d < p.dim; d += 256) sN[d] = S[size + d];
-    float4 x[DBLK * VW / 4 / 256];
-    auto fetch = [&](int d0) {
-#pragma unroll
-      for (int i = 0; i < DBLK * VW / 4 / 256; ++i) {
-        const int idx = i * 256 + threadIdx.x, r = idx / (VW / 4), c = idx % (VW / 4) * 4;
-        x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (d0 + r < p.dim && c < width) x[i] = *reinterpret_cast<const float4*>(S + (long long)(d0 + r) * p.vdim + vb * VW + c);
-      }
-    };
-    fetch(0);
-    for (int d0 = 0; d0 < p.dim; d0 += DBLK) {
-      __syncthreads();
-#pragma unroll
-      for (int i = 0; i < DBLK * VW / 4 / 256; ++i) {
-        const int idx = i * 256 + threadIdx.x, r = idx / (VW / 4), c = idx % (VW / 4) * 4;
-        uint32_t lo[TERMS], hi[TERMS];
-        split(x[i].x, x[i].y, lo);
-        split(x[i].z, x[i].w, hi);
-#pragma unroll
-        for (int k = 0; k < TERMS; ++k)
-          *reinterpret_cast<uint2*>(sS + (k * DBLK + r) * LDV + c) = make_uint2(lo[k], hi[k]);
-      }
-      if (d0 + DBLK < p.dim) fetch(d0 + DBLK);
-      if (d0 == 0) cp_async_wait<0>();
-      __syncthreads();
-#pragma unroll
-      for (int kk = 0; kk < DBLK / 16; ++kk) {
-        if (d0 + kk * 16 < p.dim && r0 < len) {
-          uint32_t q[4];
-          ldmatrix_x4(q, smem_u32(sQ + (r0 + (lane & 15)) * ld + d0 + kk * 16 + (lane >> 4) * 8));
-#pragma unroll
-          for (int n = 0; n < NT / 2; ++n) {
-            if (n * 2 < ntile) {
-#pragma unroll
-              for (int k = 0; k < TERMS; ++k) {
-                uint32_t f[4];
-                ldmatrix_x4_trans(f, smem_u32(sS + (k * DBLK + kk * 16 + (lane & 15)) * LDV + n * 16 + (lane >> 4) * 8));
-                mma_16816(acc[2 * n], q, f[0], f[1]);
-                mma_16816(acc[2 * n + 1], q, f[2], f[3]);
-              }
-            }
-          }
-        }
-      }
-    }
-    {
-      // q . n of every row, two threads a row
-      const int r = threadIdx.x >> 1;
-      float s = 0.f;
-      for (int d = (threadIdx.x & 1) * 2; d < p.dim; d += 4) {
-        const float2 q = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sQ + r * ld + d));
-        s += q.x * sN[d] + q.y * sN[d + 1];
-      }
-      s += __shfl_xor_sync(0xffffffffu, s, 1);
-      if ((threadIdx.x & 1) == 0) sDen[r] = s;
-    }
-    const float i0 = sInter[r0 + (lane >> 2)], i1 = sInter[r0 + (lane >> 2) + 8];
-#pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      acc[n][0] *= i0;
-      acc[n][1] *= i0;
-      acc[n][2] *= i1;
-      acc[n][3] *= i1;
-    }
-  }
-  const int tr = r0 + (lane >> 2);       // this thread's rows: tr, tr + 8
-  float rs[2] = {0.f, 0.f};
-  for (int s0 = 0; s0 < len; s0 += SB) {
-    __syncthreads();
-    load_rows(sK, ld, rows + p.k_col + h * p.dim, p.ld, SB, s0, len, p.dim, p.dim);
-    load_rows(sV, LDV, rows + p.v_col + h * p.vdim + vb * VW, p.ld, SB, s0, len, width, width);
-    cp_async_commit();
-    cp_async_wait<0>();
-    __syncthreads();
-    if (s0 > r0 + 15 || r0 >= len) continue;
-    const int tiles = min((r0 + 15 - s0) / 16 + 1, SB / 16);      // 16-token tiles that some row of the warp sees
-    float sc[SB / 8][4];
-#pragma unroll
-    for (int n = 0; n < SB / 8; ++n)
-#pragma unroll
-      for (int x = 0; x < 4; ++x) sc[n][x] = 0.f;
-    for (int kk = 0; kk < p.dim / 16; ++kk) {
-      uint32_t q[4];
-      ldmatrix_x4(q, smem_u32(sQ + (r0 + (lane & 15)) * ld + kk * 16 + (lane >> 4) * 8));
-#pragma unroll
-      for (int n = 0; n < SB / 16; ++n) {
-        if (n < tiles) {
-          uint32_t f[4];
-          ldmatrix_x4(f, smem_u32(sK + (n * 16 + (lane & 7) + (lane >> 4) * 8) * ld + kk * 16 + ((lane >> 3) & 1) * 8));
-          mma_16816(sc[2 * n], q, f[0], f[1]);
-          mma_16816(sc[2 * n + 1], q, f[2], f[3]);
-        }
-      }
-    }
-#pragma unroll
-    for (int n = 0; n < SB / 16; ++n) {
-      if (n < tiles) {
-        uint32_t at[TERMS][4];
-#pragma unroll
-        for (int u = 0; u < 2; ++u) {
-#pragma unroll
-          for (int x = 0; x < 4; ++x) {
-            const int s = s0 + (2 * n + u) * 8 + (lane & 3) * 2 + (x & 1), t = tr + (x >> 1) * 8;
-            const float v = s <= t ? sc[2 * n + u][x] * p.scale * expf(sa[s] - sM[t]) : 0.f;
-            sc[2 * n + u][x] = v;
-            rs[x >> 1] += v;
-          }
-        }
-        // accumulator pairs -> A fragment registers (rows lane / 4 and + 8, columns 2 (lane % 4) and + 8)
-#pragma unroll
-        for (int r = 0; r < 4; ++r) {
-          uint32_t t3[TERMS];
-          split(sc[2 * n + (r >> 1)][(r & 1) * 2], sc[2 * n + (r >> 1)][(r & 1) * 2 + 1], t3);
-#pragma unroll
-          for (int k = 0; k < TERMS; ++k) at[k][r] = t3[k];
-        }
-#pragma unroll
-        for (int c = 0; c < NT / 2; ++c) {
-          if (c * 2 < ntile) {
-            uint32_t f[4];
-            ldmatrix_x4_trans(f, smem_u32(sV + (n * 16 + (lane & 15)) * LDV + c * 16 + (lane >> 4) * 8));
-#pragma unroll
-            for (int k = 0; k < TERMS; ++k) {
-              mma_16816(acc[2 * c], at[k], f[0], f[1]);
-              mma_16816(acc[2 * c + 1], at[k], f[2], f[3]);
-            }
-          }
-        }
-      }
-    }
-  }
-  if (r0 >= len) return;                 // no barrier follows
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    const int t = tr + r * 8;
-    float den = rs[r] + __shfl_xor_sync(0xffffffffu, rs[r], 1);
-    den += __shfl_xor_sync(0xffffffffu, den, 2);
-    if (inter) den += sInter[t] * sDen[t];
-    const float inv = 1.f / (fmaxf(fabsf(den), sExp[t]) + p.floor);
-    float ss = 0.f;
-#pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      acc[n][2 * r] *= inv;
-      acc[n][2 * r + 1] *= inv;
-      ss += acc[n][2 * r] * acc[n][2 * r] + acc[n][2 * r + 1] * acc[n][2 * r + 1];
-    }
-    ss += __shfl_xor_sync(0xffffffffu, ss, 1);
-    ss += __shfl_xor_sync(0xffffffffu, ss, 2);
-    if (t >= len) continue;
-    const int c0 = h * p.vdim + vb * VW + (lane & 3) * 2;
-    if (vblocks > 1) {
-      float* o = ch.o + (first + t) * p.H * p.vdim + c0;
-#pragma unroll
-      for (int n = 0; n < NT; ++n)
-        if (n < ntile) *reinterpret_cast<float2*>(o + n * 8) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
-      continue;
-    }
-    const float nr = 1.f / sqrtf(ss / (float)p.rms_dim + p.eps);
-    const bf16* g = p.proj + (first + t) * p.ld + p.g_col + c0;
-    bf16* y = p.y + (first + t) * p.H * p.vdim + c0;
-#pragma unroll
-    for (int n = 0; n < NT; ++n) {
-      if (n < ntile) {
-        const float2 gg = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(g + n * 8));
-        const float2 w = *reinterpret_cast<const float2*>(p.norm + c0 + n * 8);
-        *reinterpret_cast<__nv_bfloat162*>(y + n * 8) =
-            __floats2bfloat162_rn(acc[n][2 * r] * nr * w.x * sigmoid_f(gg.x), acc[n][2 * r + 1] * nr * w.y * sigmoid_f(gg.y));
-      }
-    }
-  }
-}
-
-template <typename T>
-Args<T> make_args(const void* proj, long long ld, const float* z, long long z_ld, const int* ints, const float* floats,
-                  const float* bias, const float* norm, float* memory, float* nrm, float* peak, const int* cu,
-                  const int* start, const long long* slots, void* y) {
-  return Args<T>{(const T*)proj, ld, z, z_ld, ints[0], ints[1], ints[2], ints[3], ints[4], ints[5], ints[6], ints[7],
-                 floats[0], floats[1], floats[2], floats[3], bias, norm, memory, nrm, peak, cu, start, slots, (T*)y};
 }
 
 }  // namespace mem
@@ -817,24 +410,28 @@ MSRL_API int msrl_memory_prefill(const void* proj, long long ld, const float* z,
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
-static size_t memory_out_smem(int dim) {
-  const size_t kv = (size_t)mem::SB * (dim + 8) + (size_t)mem::SB * mem::LDV, s = (size_t)mem::TERMS * mem::DBLK * mem::LDV;
-  return ((size_t)mem::C * (dim + 8) + (kv > s ? kv : s)) * 2 + dim * 4;
-}
-
 MSRL_API int msrl_memory_chunked_serves(const int* ints) { return ints[1] <= 256 && ints[1] % 16 == 0 && ints[2] % 16 == 0; }
 
 // floats
 MSRL_API long long msrl_memory_chunk_scratch(const int* ints, int tokens, int batch) {
   const long long H = ints[0], dim = ints[1], vdim = ints[2], chunks = tokens / mem::C + batch;
-  return chunks * H * (dim * vdim + dim + 4) + 3 * H * tokens + 16 + (vdim > mem::VW ? (long long)tokens * H * vdim : 0);
+  return chunks * H * (dim * vdim + dim + 4) + 3 * H * tokens + 16 + (vdim > 128 ? (long long)tokens * H * vdim : 0);
 }
 
-// The same for bf16 rows, in chunks; column starts and ld are multiples of 8
+// matrix_memory_tcgen05.cu
+namespace msrl {
+namespace mem {
+int launch_chunk_state(const Args<__nv_bfloat16>& p, const Chunks& ch, int most, int batch, int* error, cudaStream_t st);
+int launch_chunk_out(const Args<__nv_bfloat16>& p, const Chunks& ch, int most, int batch, int* error, cudaStream_t st);
+}  // namespace mem
+}  // namespace msrl
+
+// The same for bf16 rows, in chunks; column starts and ld are multiples of 8.  error: device status word (0 = ok)
 MSRL_API int msrl_memory_prefill_chunked(const void* proj, long long ld, const float* z, long long z_ld, const int* ints,
                                          const float* floats, const float* bias, const float* norm, float* memory,
                                          float* nrm, float* peak, const int* cu, const int* start, const long long* slots,
-                                         float* scratch, void* y, int tokens, int batch, int max_q, cudaStream_t st) {
+                                         float* scratch, void* y, int tokens, int batch, int max_q, int* error,
+                                         cudaStream_t st) {
   if (batch == 0 || tokens == 0) return 0;
   const int H = ints[0], dim = ints[1], vdim = ints[2];
   if (!msrl_memory_chunked_serves(ints) || ld % 8 != 0 || batch > 65535 || H > 65535) return (int)cudaErrorNotSupported;
@@ -854,22 +451,13 @@ MSRL_API int msrl_memory_prefill_chunked(const void* proj, long long ld, const f
   ch.o = ch.b + (long long)H * tokens;
   ch.o += (16 - (reinterpret_cast<uintptr_t>(ch.o) & 15)) / 4 % 4;
   ch.tokens = tokens;
-  const int vblocks = (vdim + mem::VW - 1) / mem::VW, most = (max_q + mem::C - 1) / mem::C;
-  const dim3 grid((unsigned)(most * vblocks), (unsigned)H, (unsigned)batch);
-  const int smem_state = (mem::C * (dim + 8) + mem::C * mem::LDV) * 2, smem_out = (int)memory_out_smem(dim);
-  cudaError_t e = cudaFuncSetAttribute(mem::chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_state);
-  if (e != cudaSuccess) return (int)e;
-  mem::chunk_state_kernel<<<grid, 256, smem_state, st>>>(p, ch);
+  const int most = (max_q + mem::C - 1) / mem::C;
+  int rc = mem::launch_chunk_state(p, ch, most, batch, error, st);
+  if (rc != 0) return rc;
   mem::carry_kernel<<<dim3((unsigned)((size + 1023) / 1024), (unsigned)H, (unsigned)batch), 256, 0, st>>>(p, ch);
   mem::carry_peak_kernel<<<(unsigned)(((long long)batch * H + 127) / 128), 128, 0, st>>>(p, ch, batch);
-  auto go = [&](auto kernel) {
-    e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_out);
-    if (e != cudaSuccess) return (int)e;
-    kernel<<<grid, 256, smem_out, st>>>(p, ch);
-    return (int)cudaGetLastError();
-  };
-  const int rc = vdim <= 64 ? go(mem::chunk_out_kernel<8>) : go(mem::chunk_out_kernel<16>);
-  if (rc != 0 || vblocks == 1) return rc;
+  rc = mem::launch_chunk_out(p, ch, most, batch, error, st);
+  if (rc != 0 || vdim <= 128) return rc;
   const long long rows = (long long)tokens * H;
   mem::finish_kernel<__nv_bfloat16><<<(unsigned)((rows + 7) / 8), 256, 0, st>>>(p, ch.o, rows);
   return (int)cudaGetLastError();

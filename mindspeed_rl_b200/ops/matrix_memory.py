@@ -8,7 +8,7 @@ Per head, with log gates ``i = cap tanh(z_i / cap)`` and ``f = log sigmoid(cap t
 
 A sequence starts with S, n and m zero.  ``slots`` holds the state of all sequences: ``memory [slots, H, dim, vdim]``,
 ``norm [slots, H, dim]`` and ``peak [slots, H]``, all fp32; a sequence's first token ignores what its slot holds.  CUDA
-path: ``csrc/matrix_memory.cu``; CPU tensors run the PyTorch formulation.
+path: ``csrc/matrix_memory.cu``, ``csrc/matrix_memory_tcgen05.cu``; CPU tensors run the PyTorch formulation.
 """
 from __future__ import annotations
 
@@ -24,6 +24,7 @@ from . import guard
 from . import _lib
 from ._lib import c_float, c_int, c_ll, check, ptr, stream
 from .elementwise import _workspace
+from .gemm import _status_word
 from .residual import _is_f32
 
 CHUNK = 128            # tokens that the chunked prompt kernels take at a time
@@ -106,8 +107,8 @@ def memory_prefill(proj: torch.Tensor, z: torch.Tensor, lay: MemoryLayout, w: Me
             size = L.msrl_memory_chunk_scratch
             size.restype = ctypes.c_longlong
             scratch = _workspace("memory_chunks", int(size(lay.ints(), c_int(t), c_int(batch))), proj.device)
-            check(L.msrl_memory_prefill_chunked(*args, ptr(scratch), ptr(y), c_int(t), c_int(batch), c_int(max_q), stream()),
-                  "memory_prefill_chunked")
+            check(L.msrl_memory_prefill_chunked(*args, ptr(scratch), ptr(y), c_int(t), c_int(batch), c_int(max_q),
+                                                ptr(_status_word(proj.device)), stream()), "memory_prefill_chunked")
             return y
         o = _workspace("memory_out", t * lay.heads * lay.vdim, proj.device)
         check(L.msrl_memory_prefill(*args, ptr(o), ptr(y), c_int(t), c_int(batch), _is_f32(proj), stream()), "memory_prefill")
