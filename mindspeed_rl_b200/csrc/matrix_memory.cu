@@ -272,7 +272,7 @@ __global__ void __launch_bounds__(256) finish_kernel(const Args<T> p, const floa
     ldf4(p.proj + t * p.ld + p.g_col + h * p.vdim + c, g);
     ldf4(p.norm + h * p.vdim + c, w);
 #pragma unroll
-    for (int i = 0; i < 4; ++i) f[i] *= inv * w[i] * sigmoid_f(g[i]);
+    for (int i = 0; i < 4; ++i) f[i] *= inv * w[i] * sigmoid_t<T>(g[i]);
     stf4(p.y + r * p.vdim + c, f);
   }
 }

@@ -3,15 +3,15 @@
 // One CTA takes one chunk of 128 tokens, one head and up to 128 value columns:
 //
 //   chunk_state   U [dim, columns] = (w K)^T V: the gates of the chunk are summed and maximised by one warp, the keys times
-//                 their weights go to shared memory as MN-major A operand, 32 tokens at a time (two buffers), V is the
-//                 MN-major B operand
+//                 their weights go to shared memory as MN-major A operand, 32 tokens at a time, V is the MN-major B
+//                 operand
 //   chunk_out     S = Q K^T;  O1 = Q S0, the state before the chunk going through shared memory 32 rows at a time;
 //                 P = S with the weights, as K-major A operand over the dead Q and K;  O2 = P V into the columns of S;
 //                 y = (weight O1 + O2) / denominator, normed and gated
 //
 // 32-bit operands (weighted keys, P, the state) are taken apart into three bf16 terms of 24 bits together, one product
-// each; the other operand is exact and sums are fp32.  Two CTAs share an SM (dim <= 128), so that the copies and
-// conversions of one run beside the products of the other.  All tiles are 128-byte-swizzled.
+// each; the other operand is exact and sums are fp32.  Two or three CTAs share an SM (dim <= 128), so that the copies and
+// conversions of one run beside the products of the other  All tiles are 128-byte-swizzled.
 //
 // Every mbarrier wait is bounded; on expiry the kernel records a code in the status word, skips the rest, frees
 // TMEM and returns.
@@ -31,7 +31,7 @@ constexpr int VW = 128;                  // value columns of a CTA
 constexpr int TERMS = 3, TB = 32;        // bf16 terms of a 32-bit operand; tokens or state rows per converted block
 constexpr uint32_t HALF = C * 128;       // [128 rows x 64 columns] bf16
 constexpr uint32_t BLK = TB * 128;       // [32 rows x 64 columns]
-constexpr uint32_t TMEM_COLS = 256;
+constexpr float LOG2E = 1.4426950408889634f;
 constexpr int PITCH = 36;                // floats per row of a warp's [32 x 32] staging patch
 
 enum { ERR_A = 80, ERR_DONE = 81, ERR_S = 82, ERR_Q = 83, ERR_PV = 84 };
@@ -49,6 +49,17 @@ __device__ __forceinline__ uint32_t piece(int r, int c) { return (r >> 3) * 1024
 // 128 rows of a section (`cols` wide) into swizzled halves; rows past `len` are zero
 __device__ __forceinline__ void load_tile(unsigned char* dst, const bf16* src, long long ld, int len, int cols) {
   const int vecs = cols / 8;
+  if (vecs == 16) {                      // 128 columns: a thread keeps its column piece
+    const int c = threadIdx.x & 15, r0 = threadIdx.x >> 4;
+    unsigned char* to = dst + (c >> 3) * HALF + piece(r0, c & 7);  // 16 rows on: the same place two row groups later
+    const bf16* from = src + (long long)r0 * ld + c * 8;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const bool ok = r0 + i * 16 < len;
+      cp_async16(to + i * 2048, ok ? from + (long long)(i * 16) * ld : src, ok);
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < C * vecs; i += 256) {
     const int r = i / vecs, c = i - r * vecs;
     const bool ok = r < len;
@@ -69,60 +80,77 @@ __device__ __forceinline__ bf16x8 take_term(float* v) {
   return out;
 }
 
-__device__ __forceinline__ void alloc_tmem(uint32_t* slot) {
-  asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(smem_u32(slot)), "r"(TMEM_COLS));
+__device__ __forceinline__ void alloc_tmem(uint32_t* slot, uint32_t columns) {
+  asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(smem_u32(slot)), "r"(columns));
   asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::);
 }
-__device__ __forceinline__ void free_tmem(uint32_t tmem) {
-  asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;\n" ::"r"(tmem), "r"(TMEM_COLS));
+__device__ __forceinline__ void free_tmem(uint32_t tmem, uint32_t columns) {
+  asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;\n" ::"r"(tmem), "r"(columns));
 }
 
 __host__ __device__ inline int key_halves(int dim) { return (dim + 63) / 64; }
 __host__ __device__ inline uint32_t state_smem(int dim) {
-  return 2u * HALF + 2u * TERMS * (dim > 128 ? 4u : 2u) * BLK;
+  const uint32_t terms = TERMS * (dim > 128 ? 4u : 2u) * BLK, patches = 8u * 32 * PITCH * 4;
+  return 2u * HALF + (terms > patches ? terms : patches);
 }
 __host__ __device__ inline uint32_t out_keys_bytes(int dim) {      // Q and K, later P
   const uint32_t b = 2u * key_halves(dim) * HALF;
   return b > 4u * HALF ? b : 4u * HALF;
 }
 
-// grid (chunks x column blocks, H, B)
-__global__ void __launch_bounds__(256, 2) chunk_state_kernel(const Args<bf16> p, const Chunks ch, int* error) {
+// MB 128-row blocks of keys (dim <= 128 MB).  grid (chunks x column blocks, H, B)
+template <int MB>
+__global__ void __launch_bounds__(256, MB == 1 ? 3 : 2) chunk_state_kernel(const Args<bf16> p, const Chunks ch, int* error) {
   extern __shared__ unsigned char raw[];
-  __shared__ float w[C];
-  __shared__ uint64_t used[2], done;
+  __shared__ float w[C], gate_f[C];
+  __shared__ uint64_t used, done;
   __shared__ uint32_t tmem_slot;
+  constexpr uint32_t TMEM = 128 * MB, term_bytes = MB * 2 * BLK;
   const int vblocks = (p.vdim + VW - 1) / VW;
   const int j = blockIdx.x / vblocks, vb = blockIdx.x % vblocks, h = blockIdx.y, b = blockIdx.z;
   const int t0 = p.cu[b], len = min(p.cu[b + 1] - t0 - j * C, C);
   if (len <= 0) return;                  // uniform for the CTA, before any allocation
   unsigned char* sV = align1k(raw);
   unsigned char* sA = sV + 2 * HALF;
-  const int mblocks = p.dim > 128 ? 2 : 1;
-  const uint32_t term_bytes = mblocks * 2 * BLK, buf_bytes = TERMS * term_bytes;
   const long long first = t0 + j * C, id = chunk_id(t0, b, j) * p.H + h;
   const int width = min(VW, p.vdim - vb * VW);
   const bf16* rows = p.proj + first * p.ld;
   load_tile(sV, rows + p.v_col + h * p.vdim + vb * VW, p.ld, len, width);
   cp_async_commit();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  // keys: a thread keeps its eight entries and takes rows `kr`, `kr` + lanes, ... of a block
+  const int vecs = p.dim / 8, lanes = 256 / vecs, kc = threadIdx.x % vecs, kr = threadIdx.x / vecs;
+  const bf16* keys = rows + p.k_col + h * p.dim + kc * 8;
+  constexpr int ROWS = 2 * MB;           // rows of a thread in a block: 32 / lanes, at most 2 MB
+  bf16x8 next[ROWS];
+  auto fetch = [&](int blk) {
+#pragma unroll
+    for (int i = 0; i < ROWS; ++i) {
+      const int r = kr + i * lanes;
+      if (kr < lanes && r < TB && blk * TB + r < len) next[i] = ld8(keys + (long long)(blk * TB + r) * p.ld);
+    }
+  };
+  fetch(0);
   if (threadIdx.x == 32) {
-    mbar_init(&used[0], 1);
-    mbar_init(&used[1], 1);
+    mbar_init(&used, 1);
     mbar_init(&done, 1);
     asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
   }
   __syncwarp();
-  if (warp == 1) alloc_tmem(&tmem_slot);
-  if (warp == 0) {                       // gates of the chunk, four tokens per lane
+  if (warp == 1) alloc_tmem(&tmem_slot, TMEM);
+  if (threadIdx.x < C) {                 // log gates, one token per thread
+    float gi = -INFINITY, gf = 0.f;
+    if (threadIdx.x < len) log_gates(p, first + threadIdx.x, h, gi, gf);
+    w[threadIdx.x] = gi;
+    gate_f[threadIdx.x] = gf;
+    asm volatile("bar.sync 1, 128;\n" ::: "memory");
+  }
+  if (warp == 0) {                       // sums and maxima over the chunk, four tokens per lane
     float a[4], run[4], bs[4], sum = 0.f;
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
-      const int s = lane * 4 + x;
-      float gi = -INFINITY, gf = 0.f;
-      if (s < len) log_gates(p, first + s, h, gi, gf);
-      a[x] = gi;
-      sum += gf;
+      a[x] = w[lane * 4 + x];
+      sum += gate_f[lane * 4 + x];
       bs[x] = sum;
     }
     float before = sum;
@@ -166,19 +194,6 @@ __global__ void __launch_bounds__(256, 2) chunk_state_kernel(const Args<bf16> p,
       ch.sum[id] = total;
     }
   }
-  // keys: a thread keeps its eight entries and takes rows `kr`, `kr` + lanes, ... of a block
-  const int vecs = p.dim / 8, lanes = 256 / vecs, kc = threadIdx.x % vecs, kr = threadIdx.x / vecs;
-  const bf16* keys = rows + p.k_col + h * p.dim + kc * 8;
-  constexpr int AHEAD = 4;               // rows of a thread in a block: 32 / lanes, at most 4 (dim <= 256)
-  bf16x8 next[AHEAD];
-  auto fetch = [&](int blk) {
-#pragma unroll
-    for (int i = 0; i < AHEAD; ++i) {
-      const int r = kr + i * lanes;
-      if (kr < lanes && r < TB && blk * TB + r < len) next[i] = ld8(keys + (long long)(blk * TB + r) * p.ld);
-    }
-  };
-  fetch(0);
   float nsum[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
   cp_async_wait<0>();
   fence_before();
@@ -188,10 +203,9 @@ __global__ void __launch_bounds__(256, 2) chunk_state_kernel(const Args<bf16> p,
   const int blocks = (len + TB - 1) / TB;
   bool ok = true;
   for (int blk = 0; blk < blocks; ++blk) {
-    unsigned char* buf = sA + (blk & 1) * buf_bytes;
-    if (blk >= 2) ok = mbar_wait_warp(&used[blk & 1], ((blk >> 1) - 1) & 1, error, ERR_A);
+    if (blk > 0) ok = mbar_wait_warp(&used, (blk - 1) & 1, error, ERR_A);
 #pragma unroll
-    for (int i = 0; i < AHEAD; ++i) {
+    for (int i = 0; i < ROWS; ++i) {
       const int r = kr + i * lanes, s = blk * TB + r;
       if (ok && kr < lanes && r < TB) {
         float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
@@ -203,9 +217,9 @@ __global__ void __launch_bounds__(256, 2) chunk_state_kernel(const Args<bf16> p,
             nsum[x] += f[x];
           }
         }
+        unsigned char* to = sA + (kc >> 3) * BLK + piece(r, kc & 7);
 #pragma unroll
-        for (int k = 0; k < TERMS; ++k)
-          *reinterpret_cast<bf16x8*>(buf + k * term_bytes + (kc >> 3) * BLK + piece(r, kc & 7)) = take_term(f);
+        for (int k = 0; k < TERMS; ++k) *reinterpret_cast<bf16x8*>(to + k * term_bytes) = take_term(f);
       }
     }
     if (blk + 1 < blocks) fetch(blk + 1);
@@ -215,14 +229,16 @@ __global__ void __launch_bounds__(256, 2) chunk_state_kernel(const Args<bf16> p,
     if (warp == 0 && elect_one()) {
       fence_after();
       const uint32_t id_u = with_n(idesc_both_mn(128), width);
-      const uint32_t a0 = smem_u32(buf), v0 = smem_u32(sV) + blk * BLK;
-      for (int mb = 0; mb < mblocks; ++mb)
+      const uint32_t a0 = smem_u32(sA), v0 = smem_u32(sV) + blk * BLK;
+#pragma unroll
+      for (int mb = 0; mb < MB; ++mb)
+#pragma unroll
         for (int k = 0; k < TERMS; ++k)
 #pragma unroll
           for (int kk = 0; kk < TB / 16; ++kk)
             umma(tmem + mb * 128, desc_sw128(a0 + k * term_bytes + mb * 2 * BLK + kk * 2048, BLK, 1024),
                  desc_sw128(v0 + kk * 2048, HALF, 1024), id_u, (blk > 0 || k > 0 || kk > 0) ? 1u : 0u);
-      commit(&used[blk & 1]);
+      commit(&used);
       if (blk + 1 == blocks) commit(&done);
     }
     __syncwarp();
@@ -235,7 +251,7 @@ __global__ void __launch_bounds__(256, 2) chunk_state_kernel(const Args<bf16> p,
     float* U = ch.state + id * (size + p.dim);
     const int quarter = warp & 3, wg = warp >> 2;
     float* patch = reinterpret_cast<float*>(sA) + warp * 32 * PITCH;
-    for (int mb = 0; mb < mblocks; ++mb) {
+    for (int mb = 0; mb < MB; ++mb) {
       const int d0 = mb * 128 + quarter * 32;
       for (int c0 = wg * 64; c0 < min(wg * 64 + 64, width); c0 += 32) {
         float v[32];
@@ -269,7 +285,7 @@ __global__ void __launch_bounds__(256, 2) chunk_state_kernel(const Args<bf16> p,
   }
   fence_before();
   __syncthreads();
-  if (warp == 1) free_tmem(tmem);
+  if (warp == 1) free_tmem(tmem, TMEM);
 }
 
 // grid (chunks x column blocks, H, B)
@@ -278,6 +294,7 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
   __shared__ float sa[C], sM[C], sInter[C], sExp[C], sDen[C], part[2][C];
   __shared__ uint64_t s_full, q_done, pv_done;
   __shared__ uint32_t tmem_slot;
+  constexpr uint32_t TMEM = 256;
   const int vblocks = (p.vdim + VW - 1) / VW;
   const int j = blockIdx.x / vblocks, vb = blockIdx.x % vblocks, h = blockIdx.y, b = blockIdx.z;
   const int t0 = p.cu[b], len = min(p.cu[b + 1] - t0 - j * C, C);
@@ -302,7 +319,7 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
     mbar_init(&pv_done, 1);
     asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
   }
-  if (warp == 1) alloc_tmem(&tmem_slot);
+  if (warp == 1) alloc_tmem(&tmem_slot, TMEM);
   const float* S = ch.state + id * (size + p.dim);
   float4 x[TB * VW / 4 / 256];
   auto fetch = [&](int d0) {
@@ -321,8 +338,8 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
     const int s = threadIdx.x;
     const long long at = (long long)h * ch.tokens + first + s;
     const float m = ch.before[id], M = s < len ? fmaxf(m, ch.run[at]) : 0.f;
-    sa[s] = s < len ? ch.a[at] : -INFINITY;
-    sM[s] = M;
+    sa[s] = s < len ? ch.a[at] * LOG2E : -INFINITY;
+    sM[s] = M * LOG2E;
     sInter[s] = s < len ? expf(m - M) * p.scale : 0.f;
     sExp[s] = s < len ? expf(-(ch.b[at] + M)) : 0.f;
   }
@@ -413,11 +430,17 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
         float t[32];
-        tmem_ld32(tmem + lane_base + wg * 64 + c * 32, t);
+        const int s0 = wg * 64 + c * 32;
+        if (s0 > quarter * 32 + 31) {    // past the diagonal for all rows of the warp
+#pragma unroll
+          for (int i = 0; i < 32; ++i) v[c * 32 + i] = 0.f;
+          continue;
+        }
+        tmem_ld32(tmem + lane_base + s0, t);
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          const int s = wg * 64 + c * 32 + i;
-          const float e = s <= row ? t[i] * p.scale * expf(sa[s] - M) : 0.f;
+          float e = t[i] * p.scale * exp2f(fminf(sa[s0 + i] - M, 0.f));       // at most 0 up to the diagonal
+          e = s0 + i <= row ? e : 0.f;
           v[c * 32 + i] = e;
           sum += e;
         }
@@ -481,55 +504,66 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
     const float weight = sInter[row];
     if (inter) den += weight * sDen[row];
     const float inv = 1.f / (fmaxf(fabsf(den), sExp[row]) + p.floor);
-    auto columns = [&](int c0, float (&v)[32]) {                  // o of 32 columns of the thread's row
-      tmem_ld32(tmem + lane_base + c0, v);
-      if (inter) {
-        float u[32];
-        tmem_ld32(tmem_o1 + lane_base + c0, u);
+    float o[2][32], ss = 0.f;            // the thread's row, its half of the columns
 #pragma unroll
-        for (int i = 0; i < 32; ++i) v[i] += weight * u[i];
+    for (int c = 0; c < 2; ++c) {
+      const int c0 = wg * 64 + c * 32;
+      if (c0 < width) {
+        tmem_ld32(tmem + lane_base + c0, o[c]);
+        if (inter) {
+          float u[32];
+          tmem_ld32(tmem_o1 + lane_base + c0, u);
+#pragma unroll
+          for (int i = 0; i < 32; ++i) o[c][i] += weight * u[i];
+        }
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          o[c][i] *= inv;
+          ss += c0 + i < width ? o[c][i] * o[c][i] : 0.f;
+        }
       }
-#pragma unroll
-      for (int i = 0; i < 32; ++i) v[i] *= inv;
-    };
+    }
     float scale = 1.f;
     if (vblocks == 1) {
-      float ss = 0.f;
-      for (int c0 = wg * 64; c0 < min(wg * 64 + 64, width); c0 += 32) {
-        float v[32];
-        columns(c0, v);
-#pragma unroll
-        for (int i = 0; i < 32; ++i) ss += c0 + i < width ? v[i] * v[i] : 0.f;
-      }
       __syncthreads();                   // every thread has read its denominators
       part[wg][row] = ss;
       __syncthreads();
       scale = 1.f / sqrtf((part[0][row] + part[1][row]) / (float)p.rms_dim + p.eps);
     }
     float* patch = reinterpret_cast<float*>(sQ) + warp * 32 * PITCH;
-    for (int c0 = wg * 64; c0 < min(wg * 64 + 64, width); c0 += 32) {
-      float v[32];
-      columns(c0, v);
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int c0 = wg * 64 + x * 32;
+      if (c0 >= width) break;
 #pragma unroll
       for (int i = 0; i < 8; ++i)
         *reinterpret_cast<float4*>(patch + lane * PITCH + i * 4) =
-            make_float4(v[i * 4] * scale, v[i * 4 + 1] * scale, v[i * 4 + 2] * scale, v[i * 4 + 3] * scale);
+            make_float4(o[x][i * 4] * scale, o[x][i * 4 + 1] * scale, o[x][i * 4 + 2] * scale, o[x][i * 4 + 3] * scale);
       __syncwarp();
+      const int c = c0 + (lane & 7) * 4, col = h * p.vdim + vb * VW + c;
+      float wn[4] = {0.f, 0.f, 0.f, 0.f};
+      uint2 gate[8];                     // all loads before the first store
+      if (vblocks == 1 && c < width) {
+        ldf4(p.norm + col, wn);
+#pragma unroll
+        for (int it = 0; it < 8; ++it) {
+          const int t = min(quarter * 32 + it * 4 + (lane >> 3), len - 1);
+          gate[it] = *reinterpret_cast<const uint2*>(p.proj + (first + t) * p.ld + p.g_col + col);
+        }
+      }
 #pragma unroll
       for (int it = 0; it < 8; ++it) {
-        const int r = it * 4 + (lane >> 3), t = quarter * 32 + r, c = c0 + (lane & 7) * 4;
+        const int r = it * 4 + (lane >> 3), t = quarter * 32 + r;
         if (t < len && c < width) {
           const float4 f = *reinterpret_cast<const float4*>(patch + r * PITCH + (lane & 7) * 4);
-          const int col = h * p.vdim + vb * VW + c;
           const long long at = (first + t) * p.H * p.vdim + col;
           if (vblocks > 1) {
             *reinterpret_cast<float4*>(ch.o + at) = f;
           } else {
-            float g[4], wn[4];
-            ldf4(p.proj + (first + t) * p.ld + p.g_col + col, g);
-            ldf4(p.norm + col, wn);
-            const float y[4] = {f.x * wn[0] * sigmoid_f(g[0]), f.y * wn[1] * sigmoid_f(g[1]), f.z * wn[2] * sigmoid_f(g[2]),
-                                f.w * wn[3] * sigmoid_f(g[3])};
+            const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[it].x));
+            const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[it].y));
+            const float y[4] = {f.x * wn[0] * sigmoid_t<bf16>(g0.x), f.y * wn[1] * sigmoid_t<bf16>(g0.y),
+                                f.z * wn[2] * sigmoid_t<bf16>(g1.x), f.w * wn[3] * sigmoid_t<bf16>(g1.y)};
             stf4(p.y + at, y);
           }
         }
@@ -539,7 +573,7 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
   }
   fence_before();
   __syncthreads();
-  if (warp == 1) free_tmem(tmem);
+  if (warp == 1) free_tmem(tmem, TMEM);
 }
 
 static int set_smem(const void* kernel, int bytes) {
@@ -547,10 +581,11 @@ static int set_smem(const void* kernel, int bytes) {
 }
 
 int launch_chunk_state(const Args<bf16>& p, const Chunks& ch, int most, int batch, int* error, cudaStream_t st) {
-  const int smem = (int)state_smem(p.dim) + 1024, rc = set_smem((const void*)chunk_state_kernel, smem);
+  auto* kernel = p.dim > 128 ? chunk_state_kernel<2> : chunk_state_kernel<1>;
+  const int smem = (int)state_smem(p.dim) + 1024, rc = set_smem((const void*)kernel, smem);
   if (rc != 0) return rc;
   const dim3 grid((unsigned)(most * ((p.vdim + VW - 1) / VW)), (unsigned)p.H, (unsigned)batch);
-  chunk_state_kernel<<<grid, 256, smem, st>>>(p, ch, error);
+  kernel<<<grid, 256, smem, st>>>(p, ch, error);
   return (int)cudaGetLastError();
 }
 
