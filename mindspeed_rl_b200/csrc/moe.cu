@@ -142,42 +142,40 @@ moe_permute_f32_kernel(const float* x, const int* pos, const float* w, int T, in
   }
 }
 
-// One warp per token.  Logits stay in registers (NPL per lane); the largest is taken out `top` times.  They are
-// ordered by logit: the sigmoid is monotone but saturates.
+// One warp per token.  Logits stay in registers (NPL per lane) as integers of the same order; the largest is taken out
+// `top` times.  They are ordered by logit: the sigmoid is monotone but saturates.
 template <int NPL>
 __global__ void __launch_bounds__(256)
 route_top_kernel(const float* logits, int T, int E, int top, long long* idx, float* score) {
   const long long t = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (t >= T) return;
-  float z[NPL];
+  unsigned key[NPL];                                   // 0: out of range or taken
 #pragma unroll
-  for (int n = 0; n < NPL; ++n) z[n] = n * 32 + lane < E ? logits[t * E + n * 32 + lane] : -INFINITY;
-  unsigned taken = 0;                                  // bit n: this lane's entry n is out
+  for (int n = 0; n < NPL; ++n) {
+    key[n] = 0;
+    if (n * 32 + lane < E) {
+      const unsigned b = __float_as_uint(logits[t * E + n * 32 + lane]);
+      key[n] = max(b & 0x80000000u ? ~b : b | 0x80000000u, 1u);
+    }
+  }
   for (int j = 0; j < top; ++j) {
-    float best = -INFINITY;
-    int at = 0x7fffffff;
+    unsigned mine = 0;
 #pragma unroll
-    for (int n = 0; n < NPL; ++n) {
-      if (n * 32 + lane < E && !(taken >> n & 1) && (at == 0x7fffffff || z[n] > best)) {
-        best = z[n];
-        at = n * 32 + lane;
-      }
-    }
+    for (int n = 0; n < NPL; ++n) mine = max(mine, key[n]);
+    const unsigned best = __reduce_max_sync(0xffffffffu, mine);
+    unsigned at = 0xffffffffu;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float b2 = __shfl_xor_sync(0xffffffffu, best, o);
-      const int a2 = __shfl_xor_sync(0xffffffffu, at, o);
-      const bool valid = a2 != 0x7fffffff;
-      if (valid && (at == 0x7fffffff || b2 > best || (b2 == best && a2 < at))) {
-        best = b2;
-        at = a2;
-      }
-    }
-    if ((at & 31) == lane) taken |= 1u << (at >> 5);
+    for (int n = NPL - 1; n >= 0; --n)
+      if (key[n] == best) at = n * 32 + lane;          // this lane's lowest expert with that logit
+    const unsigned first = __reduce_min_sync(0xffffffffu, at);
+#pragma unroll
+    for (int n = 0; n < NPL; ++n)
+      if (n * 32 + lane == first) key[n] = 0;
     if (lane == 0) {
-      idx[t * top + j] = at;
-      score[t * top + j] = 1.f / (1.f + expf(-best));
+      const float z = __uint_as_float(best & 0x80000000u ? best & 0x7fffffffu : ~best);
+      idx[t * top + j] = first;
+      score[t * top + j] = 1.f / (1.f + expf(-z));
     }
   }
 }

@@ -5,8 +5,9 @@
 //   moe_combine_norm  resid[t] += w * sum_j e[pos(t, j)] + sig(h[t].sg) * sh[t] + delta2[t];  y[t] = norm(resid[t])
 //
 // norm(x) = x / sqrt(mean(x^2) + eps) * (offset + weight), all in fp32, with x less its mean when `centered` (the
-// squares are then summed in a pass of their own over the kept row); y is stored in the activation type.  One block per row; the row stays in registers between the sum and the norm (longer rows than the
-// register budget re-read the residual they just wrote).  A null `y` skips the norm.
+// squares are then summed in a pass of their own over the kept row); y is stored in the activation type.  One block
+// per row; the row stays in registers between the sum and the norm (longer rows than the register budget re-read the
+// residual they just wrote).  A null `y` skips the norm.
 //
 //   glu               act(gate) * up of rows [gate | up]: silu, tanh-gelu, or the clamped swish with (up + 1)
 #include "dtype_utils.cuh"
@@ -42,7 +43,8 @@ struct RowArgs {
   const T* shared;
 };
 
-template <typename T, int V, int NPT, int SRC>
+// FULL: with the options `centered` and `delta2`
+template <typename T, int V, int NPT, int SRC, bool FULL>
 __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
@@ -78,7 +80,7 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
       ldv<V>(p.delta + t * W + c, d);
 #pragma unroll
       for (int i = 0; i < V; ++i) f[i] += d[i];
-      if (p.delta2 != nullptr) {
+      if (FULL && p.delta2 != nullptr) {
         ldv<V>(p.delta2 + t * W + c, d);
 #pragma unroll
         for (int i = 0; i < V; ++i) f[i] += d[i];
@@ -98,7 +100,7 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
 #pragma unroll
         for (int i = 0; i < V; ++i) acc[i] += sig * d[i];
       }
-      if (p.delta2 != nullptr) {
+      if (FULL && p.delta2 != nullptr) {
         ldv<V>(p.delta2 + t * W + c, d);
 #pragma unroll
         for (int i = 0; i < V; ++i) acc[i] += d[i];
@@ -118,7 +120,7 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
 #pragma unroll
       for (int i = 0; i < V; ++i) {
         ss += keep[k][i] * keep[k][i];
-        sum += keep[k][i];
+        if (FULL) sum += keep[k][i];
       }
     }
   }
@@ -129,12 +131,12 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
 #pragma unroll
     for (int i = 0; i < V; ++i) {
       ss += f[i] * f[i];
-      sum += f[i];
+      if (FULL) sum += f[i];
     }
   }
   if (p.y == nullptr) return;
   float mean = 0.f;
-  if (p.centered) {
+  if (FULL && p.centered) {
     mean = block_sum(sum, red) / (float)W;
     ss = 0.f;
 #pragma unroll
@@ -177,19 +179,24 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
   }
 }
 
+template <typename T, int SRC, bool FULL>
+int launch_rows(const RowArgs<T>& p, long long rows, cudaStream_t st) {
+  if (p.W % 4 == 0) {
+    const int units = (p.W / 4 + RS_THREADS - 1) / RS_THREADS;
+    if (units <= 1) row_norm_kernel<T, 4, 1, SRC, FULL><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+    else if (units <= 2) row_norm_kernel<T, 4, 2, SRC, FULL><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+    else if (units <= 4) row_norm_kernel<T, 4, 4, SRC, FULL><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+    else row_norm_kernel<T, 4, 8, SRC, FULL><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+  } else {
+    row_norm_kernel<T, 1, 4, SRC, FULL><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
+  }
+  return (int)cudaGetLastError();
+}
+
 template <typename T, int SRC>
 int launch_row_norm(const RowArgs<T>& p, long long rows, cudaStream_t st) {
   if (rows == 0) return 0;
-  if (p.W % 4 == 0) {
-    const int units = (p.W / 4 + RS_THREADS - 1) / RS_THREADS;
-    if (units <= 1) row_norm_kernel<T, 4, 1, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
-    else if (units <= 2) row_norm_kernel<T, 4, 2, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
-    else if (units <= 4) row_norm_kernel<T, 4, 4, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
-    else row_norm_kernel<T, 4, 8, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
-  } else {
-    row_norm_kernel<T, 1, 4, SRC><<<(unsigned)rows, RS_THREADS, 0, st>>>(p);
-  }
-  return (int)cudaGetLastError();
+  return p.centered || p.delta2 != nullptr ? launch_rows<T, SRC, true>(p, rows, st) : launch_rows<T, SRC, false>(p, rows, st);
 }
 
 enum { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMPED_SWISH = 2 };

@@ -576,14 +576,15 @@ def test_samples_of_a_prompt_fork_state_and_pages(device):
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("name", ["many_heads", "values_regrouped", "memory_first"])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-def test_graph_decode_is_the_eager_decode(dtype):
+def test_graph_decode_is_the_eager_decode(dtype, name):
     """A captured step (its sublayers on two streams) advances every state exactly once, also the step whose capture it
     is."""
-    seqs = [M.tokens(40, M.ZOO["many_heads"]["vocab"], s) for s in range(3)]
+    seqs = [M.tokens(40, M.ZOO[name]["vocab"], s) for s in range(3)]
     got = []
     for graphs in ((), (4,)):
-        eng = engine("many_heads", "cuda", dtype, graphs=graphs)
+        eng = engine(name, "cuda", dtype, graphs=graphs)
         eng.replay([(str(i), s[:20 + i], []) for i, s in enumerate(seqs)])
         steps = [eng.replay([(str(i), [s[20 + i + k]], [0]) for i, s in enumerate(seqs)]).float().cpu() for k in range(10)]
         got.append(torch.stack(steps))
