@@ -8,13 +8,14 @@ another design adds a type without touching the readers of the others.  :meth:`H
 the ``config.json`` of a model folder.
 
 A mixer spec tells the cache what a sequence carries for it: ``paged_rows(dtype)``, shapes of one token's rows in
-paged memory by name, and ``slot_state(dtype)``, shapes and types of the state of one sequence by name.
+paged memory by name, and ``slot_state(dtype)``, shapes and types of the state of one sequence by name.  Specs with
+paged rows have ``keys``, the range of earlier tokens that a token sees (:data:`KeyRange`).
 """
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional, Tuple
+from typing import Any, Callable, Dict, List, NamedTuple, Optional, Tuple, Union
 
 import torch
 
@@ -29,6 +30,48 @@ def padded_heads(dq: int, dv: int, dtype: torch.dtype) -> Tuple[int, int]:
         return -(-dq // unit) * unit, -(-dv // unit) * unit
     vp = 64 if max(dq, dv) <= 64 else 128
     return (192 if dq > 128 else vp), vp
+
+
+class Chunk(NamedTuple):
+    """A token sees the earlier tokens of its own chunk; chunks of ``size`` tokens count from the sequence's start."""
+    size: int
+
+    @classmethod
+    def of(cls, mask: Optional[dict]) -> Optional["Chunk"]:
+        return None if not mask else cls(_positive(mask["size"], "chunk"))
+
+
+KeyRange = Union[None, int, Chunk]       # all earlier tokens, the last n up to the token itself, or its chunk
+
+
+def first_key(keys: KeyRange, pos):
+    """First position that the token at ``pos`` (an integer or an array of them) sees."""
+    if keys is None:
+        return pos * 0
+    if isinstance(keys, Chunk):
+        return pos // keys.size * keys.size
+    return (pos - keys + 1) * (pos >= keys)
+
+
+def _positive(n, what: str) -> int:
+    if int(n) < 1:
+        raise ValueError(f"a {what} of {n} tokens sees nothing")
+    return int(n)
+
+
+def _window_of(mask: Optional[dict]) -> Optional[int]:
+    return None if not mask else _positive(mask["size"], "window")
+
+
+def _check_heads(spec):
+    if spec.heads % spec.kv_heads:
+        raise ValueError(f"{spec.heads} heads do not divide into {spec.kv_heads} key heads")
+    return spec
+
+
+def _check_rotary(rot: "Rotary", limit: int, name: str) -> None:
+    if rot.dims % 2 or rot.dims > limit:
+        raise ValueError(f"rotary dims {rot.dims} must be even and at most {name} ({limit})")
 
 
 @dataclass(frozen=True)
@@ -67,7 +110,9 @@ class Rotary:
 @dataclass(frozen=True)
 class LatentAttentionSpec:
     """Causal soft-max attention whose keys and values are up-projections of one cached latent per token.
-    ``dim`` unrotated and ``rot_dim`` rotated query / key entries per head; the rotated key part is shared."""
+    ``dim`` unrotated and ``rot_dim`` rotated query / key entries per head; the rotated key part is shared.
+    ``q_rank``: queries go through a normed latent of their own; ``sink``: a learned number per head joins the soft-max
+    sum; ``head_gate``: a sigmoid per head scales the head's output."""
     heads: int
     dim: int
     rot_dim: int
@@ -75,8 +120,14 @@ class LatentAttentionSpec:
     kv_rank: int
     scale: float
     rot: Rotary
-    recurrent = False
-    window = None
+    q_rank: Optional[int] = None
+    window: Optional[int] = None
+    sink: bool = False
+    head_gate: bool = False
+
+    @property
+    def keys(self) -> KeyRange:
+        return self.window
 
     def paged_rows(self, dtype) -> Dict[str, Tuple[int, ...]]:
         return {"latent": (pad16(self.kv_rank) + pad16(self.rot_dim),)}
@@ -85,13 +136,17 @@ class LatentAttentionSpec:
         return {}
 
     @classmethod
-    def from_json(cls, m: dict) -> "LatentAttentionSpec":
-        rot = Rotary(int(m["rot"]["dims"]), float(m["rot"]["base"]))
+    def from_json(cls, m: dict, halves: bool = False, **options) -> "LatentAttentionSpec":
+        rot = Rotary(int(m["rot"]["dims"]), float(m["rot"]["base"]), halves)
         out = cls(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]),
-                  float(m["scale"]), rot)
-        if rot.dims % 2 or rot.dims > out.rot_dim:
-            raise ValueError(f"rotary dims {rot.dims} must be even and at most rot_dim ({out.rot_dim})")
+                  float(m["scale"]), rot, **options)
+        _check_rotary(rot, out.rot_dim, "rot_dim")
         return out
+
+    @classmethod
+    def gated_from_json(cls, m: dict) -> "LatentAttentionSpec":
+        """With a query latent, half-split rotation, a window, a sink and a gate per head."""
+        return cls.from_json(m, halves=True, q_rank=int(m["q_rank"]), window=_window_of(m.get("mask")), sink=True, head_gate=True)
 
 
 @dataclass(frozen=True)
@@ -103,7 +158,6 @@ class ChannelDeltaSpec:
     vdim: int
     conv: int
     unit_eps: float = 1e-6
-    recurrent = True
 
     @property
     def channels(self) -> int:
@@ -117,10 +171,12 @@ class ChannelDeltaSpec:
 
     @classmethod
     def from_json(cls, m: dict) -> "ChannelDeltaSpec":
-        out = cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]))
-        if out.heads % out.kv_heads:
-            raise ValueError(f"{out.heads} heads do not divide into {out.kv_heads} key heads")
-        return out
+        return _check_heads(cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"])))
+
+
+@dataclass(frozen=True)
+class HeadDeltaSpec(ChannelDeltaSpec):
+    """The delta rule with one decay per head, projected without a bottleneck, and a silu output gate."""
 
 
 @dataclass(frozen=True)
@@ -136,7 +192,10 @@ class WindowAttentionSpec:
     rot: Rotary
     window: Optional[int] = None
     value_mix: bool = False
-    recurrent = False
+
+    @property
+    def keys(self) -> KeyRange:
+        return self.window
 
     def padded(self, dtype) -> Tuple[int, int]:
         return padded_heads(self.dim, self.vdim, dtype)
@@ -154,14 +213,49 @@ class WindowAttentionSpec:
         rot = Rotary(int(r["dims"]), float(r["base"]), halves=True,
                      scaling=None if not sc else WavelengthScaling(float(sc["factor"]), float(sc["low"]), float(sc["high"]),
                                                                    float(sc["original"])))
-        out = cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), rot,
-                  None if not mask else int(mask["size"]), bool(m.get("v_mix", False)))
-        if out.heads % out.kv_heads:
-            raise ValueError(f"{out.heads} heads do not divide into {out.kv_heads} key heads")
-        if rot.dims % 2 or rot.dims > out.dim:
-            raise ValueError(f"rotary dims {rot.dims} must be even and at most dim ({out.dim})")
-        if out.window is not None and out.window < 1:
-            raise ValueError(f"a window of {out.window} tokens sees nothing")
+        out = _check_heads(cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), rot,
+                               _window_of(mask), bool(m.get("v_mix", False))))
+        _check_rotary(rot, out.dim, "dim")
+        return out
+
+
+@dataclass(frozen=True)
+class ConvAttentionSpec:
+    """Soft-max attention of grouped heads with short convolutions on q, k and v (carried like a recurrent state), an RMS
+    norm per query and key head, partial interleaved rotation, soft-capped scores (0: not capped), a key range, and a
+    sigmoid gate per head."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+    scale: float
+    rot: Rotary
+    softcap: float = 0.0
+    keys: KeyRange = None
+
+    @property
+    def channels(self) -> int:
+        return (self.heads + self.kv_heads) * self.dim + self.kv_heads * self.vdim
+
+    def padded(self, dtype) -> Tuple[int, int]:
+        return padded_heads(self.dim, self.vdim, dtype)
+
+    def paged_rows(self, dtype) -> Dict[str, Tuple[int, ...]]:
+        qp, vp = self.padded(dtype)
+        return {"k": (self.kv_heads, qp), "v": (self.kv_heads, vp)}
+
+    def slot_state(self, dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
+        return {"ring": ((self.conv, self.channels), dtype)}
+
+    @classmethod
+    def from_json(cls, m: dict) -> "ConvAttentionSpec":
+        rot = Rotary(int(m["rot"]["dims"]), float(m["rot"]["base"]))
+        out = _check_heads(cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]),
+                               float(m["scale"]), rot, float(m.get("softcap") or 0.0), Chunk.of(m.get("mask"))))
+        _check_rotary(rot, out.dim, "dim")
+        if out.softcap < 0.0:
+            raise ValueError(f"scores cannot be capped at {out.softcap}")
         return out
 
 
@@ -174,7 +268,6 @@ class MatrixMemorySpec:
     vdim: int
     gate_cap: float
     floor: float = 1e-6                  # added to the normaliser
-    recurrent = True
 
     def slot_state(self, dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
         f32, dp, vp = torch.float32, pad16(self.dim), pad16(self.vdim)
@@ -239,23 +332,52 @@ class ScoredMoESpec:
 
 
 @dataclass(frozen=True)
+class SoftmaxMoESpec:
+    """Experts of the largest corrected scores: the score is a soft-max (32-bit) over all router outputs, the correction a
+    stored number per output that counts for the choice only.  Outputs past ``experts`` are ``identity`` experts, which
+    give back their input.  A chosen expert's output is weighted by its score."""
+    experts: int
+    top: int
+    expert: GluSpec
+    identity: int = 0
+    shared: Optional[GluSpec] = None
+
+    @property
+    def outputs(self) -> int:
+        return self.experts + self.identity
+
+    @classmethod
+    def from_json(cls, m: dict) -> "SoftmaxMoESpec":
+        r = m["router"]
+        out = cls(int(r["experts"]), int(r["top"]), GluSpec(int(m["expert"]["ff"]), "silu"), int(r.get("identity") or 0))
+        if not 0 < out.top <= out.outputs:
+            raise ValueError(f"top {out.top} of {out.outputs} experts")
+        return out
+
+
+@dataclass(frozen=True)
 class Design:
-    """What the layers of one architecture have in common.  ``parallel``: both sublayers read one norm and are added
-    together; otherwise the feed-forward reads a second norm of the sum.  ``centered``: norms subtract the mean.
-    ``norm_offset``: the stored weight of a norm is an offset from this value."""
-    mixers: Dict[str, Any]
-    feed_forwards: Dict[str, Any]
+    """What the layers of one architecture have in common.  ``mixers`` and ``feed_forwards``: readers of a layer's entry
+    by its type.  ``parallel``: both sublayers read one norm and are added together; ``post_norm``: the sublayers read the
+    residual itself and their outputs are normed before they are added; otherwise the feed-forward reads a second norm of
+    the sum.  ``centered``: norms subtract the mean.  ``norm_offset``: the stored weight of a norm is an offset from this
+    value."""
+    mixers: Dict[str, Callable[[dict], Any]]
+    feed_forwards: Dict[str, Callable[[dict], Any]]
     parallel: bool = False
+    post_norm: bool = False
     centered: bool = False
     norm_offset: float = 0.0
     tied_head: bool = True
 
 
 DESIGNS = {
-    "Pumotar": Design({"latent_attention": LatentAttentionSpec, "channel_delta": ChannelDeltaSpec},
-                      {"dense": GluSpec, "moe": TableMoESpec}, norm_offset=1.0),
-    "Sunatar": Design({"attention": WindowAttentionSpec, "mlstm": MatrixMemorySpec}, {"moe": ScoredMoESpec},
-                      parallel=True, centered=True, tied_head=False),
+    "Pumotar": Design({"latent_attention": LatentAttentionSpec.from_json, "channel_delta": ChannelDeltaSpec.from_json},
+                      {"dense": GluSpec.from_json, "moe": TableMoESpec.from_json}, norm_offset=1.0),
+    "Sunatar": Design({"attention": WindowAttentionSpec.from_json, "mlstm": MatrixMemorySpec.from_json},
+                      {"moe": ScoredMoESpec.from_json}, parallel=True, centered=True, tied_head=False),
+    "Gapevik": Design({"attention": ConvAttentionSpec.from_json, "latent_attention": LatentAttentionSpec.gated_from_json,
+                       "delta": HeadDeltaSpec.from_json}, {"moe": SoftmaxMoESpec.from_json}, post_norm=True),
 }
 
 
@@ -264,6 +386,7 @@ class LayerSpec:
     type: str
     mixer: Any
     mlp: Any = None
+    weights_of: Optional[int] = None     # the layer whose tensors this one uses (None: its own)
 
 
 @dataclass
@@ -274,6 +397,7 @@ class HybridConfig:
     layers: List[LayerSpec]
     norm_epsilon: float
     embedding_scale: float = 1.0
+    residual_mult: float = 1.0                       # factor on what a sublayer adds (post-norm designs)
     loop: Optional[Tuple[int, int, int]] = None      # (start, stop, times)
     params_dtype: torch.dtype = torch.bfloat16
     extra: Dict[str, Any] = field(default_factory=dict)
@@ -284,6 +408,8 @@ class HybridConfig:
             a, b, n = self.loop
             if not (0 <= a <= b <= len(self.layers)) or n < 1:
                 raise ValueError(f"loop {self.loop} does not fit {len(self.layers)} layers")
+        for i in range(len(self.layers)):
+            self.owner(i)
         mixed = {l.mixer.kv_heads * l.mixer.vdim for l in self.layers if getattr(l.mixer, "value_mix", False)}
         if len(mixed) > 1:
             raise ValueError(f"layers that mix values with the first one's have different value sizes: {sorted(mixed)}")
@@ -291,6 +417,19 @@ class HybridConfig:
     @property
     def design(self) -> Design:
         return DESIGNS[self.architecture]
+
+    def owner(self, i: int) -> int:
+        """The layer whose tensors layer ``i`` uses."""
+        j, seen = i, set()
+        while self.layers[j].weights_of is not None:
+            seen.add(j)
+            j = self.layers[j].weights_of
+            if not 0 <= j < len(self.layers) or j in seen:
+                raise ValueError(f"layer {i} uses the tensors of layer {j}, which has none")
+        mine, other = self.layers[i], self.layers[j]
+        if (mine.type, mine.mixer, mine.mlp) != (other.type, other.mixer, other.mlp):
+            raise ValueError(f"layer {i} uses the tensors of layer {j} but differs from it")
+        return j
 
     # ---- what a sequence runs through ----------------------------------------------------------
     @property
@@ -308,16 +447,17 @@ class HybridConfig:
 
     @property
     def is_recurrent(self) -> bool:
-        return any(l.mixer.recurrent for l in self.layers)
+        """Sequences carry state besides paged rows."""
+        return any(l.mixer.slot_state(self.params_dtype) for l in self.layers)
 
     @property
     def is_moe(self) -> bool:
-        return any(isinstance(l.mlp, (TableMoESpec, ScoredMoESpec)) for l in self.layers)
+        return any(isinstance(l.mlp, (TableMoESpec, ScoredMoESpec, SoftmaxMoESpec)) for l in self.layers)
 
     @property
-    def windows(self) -> Tuple[Optional[int], ...]:
-        """Distinct key ranges of the attention layers (None: all earlier tokens)."""
-        return tuple({l.mixer.window: None for l in self.layers if not l.mixer.recurrent})
+    def windows(self) -> Tuple[KeyRange, ...]:
+        """Distinct key ranges of the attention layers."""
+        return tuple({l.mixer.keys: None for l in self.layers if l.mixer.paged_rows(self.params_dtype)})
 
     @classmethod
     def from_json(cls, cfg: dict, dtype: torch.dtype = torch.bfloat16) -> "HybridConfig":
@@ -328,11 +468,14 @@ class HybridConfig:
             mlp = l.get("mlp")
             if mlp is not None and mlp["kind"] not in design.feed_forwards:
                 raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
-            layers.append(LayerSpec(l["type"], design.mixers[l["type"]].from_json(l["mixer"]),
-                                    None if mlp is None else design.feed_forwards[mlp["kind"]].from_json(mlp)))
+            of = l.get("weights_of")
+            layers.append(LayerSpec(l["type"], design.mixers[l["type"]](l["mixer"]),
+                                    None if mlp is None else design.feed_forwards[mlp["kind"]](mlp),
+                                    None if of is None else int(of)))
         lp = cfg.get("loop")
         return cls(architecture=cfg["architecture"], vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
                    layers=layers, norm_epsilon=float(cfg["norm"]["eps"]),
                    embedding_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
+                   residual_mult=float(cfg.get("residual_mult", 1.0)),
                    loop=None if not lp else (int(lp["start"]), int(lp["stop"]), int(lp["times"])),
                    params_dtype=dtype)

@@ -111,5 +111,6 @@ def _decoder_weights(cfg, state, device):
 
 register("Pumotar", ModelFamily(HybridConfig.from_json, _hybrid_weights, "pumotar"))
 register("Sunatar", ModelFamily(HybridConfig.from_json, _hybrid_weights, "sunatar"))
+register("Gapevik", ModelFamily(HybridConfig.from_json, _hybrid_weights, "gapevik"))
 for _name in ("Qwen2ForCausalLM", "Qwen3ForCausalLM", "Qwen3MoeForCausalLM"):
     register(_name, ModelFamily(_decoder_config, _decoder_weights))

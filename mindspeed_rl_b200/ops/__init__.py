@@ -14,13 +14,15 @@ from .decode import (build_decode_groups, decode_group_max, decode_prefix_tile, 
 from .rl import (gae, group_norm_advantage, loss_weights, policy_loss_fwd_bwd,
                  policy_loss_reference, value_loss_fwd_bwd, value_loss_reference)
 from .optim import adamw_step, cast_f32_to_bf16, clip_coefficient, sumsq_accumulate
-from .residual import Norm, add_norm_, embed_norm, glu_fwd, moe_combine_norm_
+from .score_form import PLAIN, ScoreForm
+from .residual import Norm, PostNorm, add_norm_, embed, embed_norm, glu_fwd, moe_combine_norm_, moe_post_add_, post_add_
 from .latent import (LatentLayout, latent_decode_attention, latent_gather, latent_prefill_attention, latent_prep,
-                     latent_spread_)
+                     latent_rotate_queries, latent_spread_)
 from .delta import DeltaLayout, DeltaWeights, delta_decode, delta_prefill
 from .matrix_memory import MemoryLayout, MemoryWeights, memory_decode, memory_prefill
 from .window import (GroupedHeads, ValueSource, angle_table, qkv_prep_, rows_gather, window_decode_attention,
                      window_prefill_attention)
+from .conv_qkv import ConvHeads, ConvNormWeights, conv_qkv_decode, conv_qkv_prefill
 from .lmhead import lmhead_logprob_bwd, lmhead_logprob_fwd
 
 __all__ = [n for n in dir() if not n.startswith("_")]

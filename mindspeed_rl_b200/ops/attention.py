@@ -19,6 +19,7 @@ from . import guard
 
 from . import _lib
 from ._lib import c_float, c_int, c_ll, check, ptr, stream
+from .score_form import PLAIN
 from .elementwise import _workspace
 from .layouts import QKVLayout
 
@@ -101,15 +102,15 @@ def attn_varlen_fwd(qkv: torch.Tensor, layout: QKVLayout, cu_seqlens: torch.Tens
                 ptr(flat[qs[0]:]), ptr(kb), ptr(vb), lay, ptr(out), c_ll(nh * hd), ptr(lse),
                 ptr(cu_seqlens), ptr(cu_k), c_int(batch), c_int(int(max_seqlen)), c_int(nh), c_int(nkv),
                 c_ll(t), c_ll(tk), c_int(hd), c_float(1.0 / math.sqrt(hd)), c_int(1 if causal else 0), c_int(0),
-                ptr(_status_word(qkv.device)), stream())
+                *PLAIN.args(), ptr(_status_word(qkv.device)), stream())
             if rc != _NOT_SUPPORTED:
                 check(rc, "flash_attn_varlen_fwd_tcgen05")
                 return out, lse
         check(_lib.load().msrl_flash_attn_varlen_fwd(
             ptr(flat[qs[0]:]), ptr(kb), ptr(vb), lay, ptr(out), c_ll(nh * hd), ptr(lse),
             ptr(cu_seqlens), ptr(cu_k), c_int(batch), c_int(int(max_seqlen)), c_int(nh), c_int(nkv),
-            c_ll(t), c_int(hd), c_float(1.0 / math.sqrt(hd)), c_int(1 if causal else 0), c_int(0), stream()),
-            "flash_attn_varlen_fwd")
+            c_ll(t), c_int(hd), c_float(1.0 / math.sqrt(hd)), c_int(1 if causal else 0), c_int(0), *PLAIN.args(),
+            stream()), "flash_attn_varlen_fwd")
         return out, lse
     q, k, v = layout.split(qkv)
     if kv is not None:
@@ -178,14 +179,14 @@ def attn_kv_fwd(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_q: torch.T
             rc = _lib.load().msrl_flash_attn_varlen_fwd_tcgen05(
                 ptr(q), ptr(k), ptr(v), lay, ptr(out), c_ll(nh * hd), ptr(lse), ptr(cu_q), ptr(cu_k), c_int(batch),
                 c_int(int(max_q)), c_int(nh), c_int(nkv), c_ll(tq), c_ll(tk), c_int(hd), c_float(1.0 / math.sqrt(hd)),
-                c_int(1 if causal else 0), c_int(0), ptr(_status_word(q.device)), stream())
+                c_int(1 if causal else 0), c_int(0), *PLAIN.args(), ptr(_status_word(q.device)), stream())
             if rc != _NOT_SUPPORTED:
                 check(rc, "flash_attn_varlen_fwd_tcgen05")
                 return out, lse
         check(_lib.load().msrl_flash_attn_varlen_fwd(
             ptr(q), ptr(k), ptr(v), lay, ptr(out), c_ll(nh * hd), ptr(lse), ptr(cu_q), ptr(cu_k), c_int(batch),
             c_int(int(max_q)), c_int(nh), c_int(nkv), c_ll(tq), c_int(hd), c_float(1.0 / math.sqrt(hd)),
-            c_int(1 if causal else 0), c_int(0), stream()), "flash_attn_varlen_fwd")
+            c_int(1 if causal else 0), c_int(0), *PLAIN.args(), stream()), "flash_attn_varlen_fwd")
         return out, lse
     o, lse = _ref_attention(q, k, v, cu_q, cu_k, causal)
     return o.reshape(tq, nh * hd).to(q.dtype), lse

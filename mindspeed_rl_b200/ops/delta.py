@@ -1,4 +1,4 @@
-"""Gated delta rule with per-channel decay over state slots: prompt portions and decode steps.
+"""Gated delta rule with a decay per key channel or per head over state slots: prompt portions and decode steps.
 
 The weights of a layer (:class:`DeltaWeights`) and the carried state of all sequences (``ring``, ``state``) are
 described in ``csrc/delta_rule.cu``, the CUDA path; CPU tensors run the PyTorch formulation.
@@ -32,21 +32,23 @@ class DeltaLayout:
     v_col: int
     b_col: int
     unit_eps: float = 1e-6
+    head_decay: bool = False      # one decay per head instead of one per key channel
+    silu_gate: bool = False       # the output gate is silu instead of sigmoid
 
     @property
     def channels(self) -> int:
         return 2 * self.kv_heads * self.dim + self.heads * self.vdim
 
     def ints(self):
-        return (ctypes.c_int * 9)(self.taps, self.heads, self.kv_heads, self.dim, self.vdim, self.q_col, self.k_col,
-                                  self.v_col, self.b_col)
+        return (ctypes.c_int * 11)(self.taps, self.heads, self.kv_heads, self.dim, self.vdim, self.q_col, self.k_col,
+                                   self.v_col, self.b_col, int(self.head_decay), int(self.silu_gate))
 
 
 @dataclass
 class DeltaWeights:
     conv: torch.Tensor        # [channels, taps] fp32 (q, k, v channels in order)
     a_log: torch.Tensor       # [heads] fp32
-    dt_bias: torch.Tensor     # [heads * dim] fp32
+    dt_bias: torch.Tensor     # [heads * dim] fp32, or [heads] with one decay per head
     norm: torch.Tensor        # [vdim] fp32
 
 
@@ -66,14 +68,14 @@ def _recur(proj, a, gate, lay: DeltaLayout, w: DeltaWeights, hist, s, eps):
     q, k, v = unit(y[:, :kd]) / math.sqrt(lay.dim), unit(y[:, kd:2 * kd]), y[:, 2 * kd:].view(t, lay.heads, lay.vdim)
     beta = torch.sigmoid(proj[:, lay.b_col:lay.b_col + lay.heads].float())
     g = torch.exp(-torch.exp(w.a_log).view(1, -1, 1)
-                  * F.softplus(a.float() + w.dt_bias, threshold=60.0).view(t, lay.heads, lay.dim))
+                  * F.softplus(a.float() + w.dt_bias, threshold=60.0).view(t, lay.heads, -1))
     o = torch.empty(t, lay.heads, lay.vdim)
     for i in range(t):
         s.mul_(g[i].unsqueeze(-1))
         u = beta[i].unsqueeze(-1) * (v[i] - torch.einsum("hdv,hd->hv", s, k[i]))
         s.add_(k[i].unsqueeze(-1) * u.unsqueeze(1))
         o[i] = torch.einsum("hdv,hd->hv", s, q[i])
-    o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w.norm * torch.sigmoid(gate.float()).view_as(o)
+    o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w.norm * (F.silu if lay.silu_gate else torch.sigmoid)(gate.float()).view_as(o)
     return o.view(t, -1).to(proj.dtype), ext
 
 
@@ -100,7 +102,7 @@ def delta_prefill(proj: torch.Tensor, a: torch.Tensor, gate: torch.Tensor, lay: 
                   ring: torch.Tensor, state: torch.Tensor, tok_seq: torch.Tensor, cu: torch.Tensor,
                   start_pos: torch.Tensor, slots: torch.Tensor, eps: float) -> torch.Tensor:
     """Packed prompt portions (``cu [B + 1]``; sequence b starts at position ``start_pos[b]`` and carries its state
-    in slot ``slots[b]``) -> gated, normed outputs ``[T, heads * vdim]``; ring and state are updated."""
+    in slot ``slots[b]``; ``a [T, heads * dim or heads]``: decay projection) -> gated, normed outputs ``[T, heads * vdim]``; ring and state are updated."""
     t, batch = proj.shape[0], cu.numel() - 1
     if _lib.use_kernels(proj, a, gate, ring, state, cu):
         L, ints = _lib.load(), lay.ints()

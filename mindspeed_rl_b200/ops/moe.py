@@ -43,7 +43,8 @@ def max_rows(n_slots: int, num_experts: int) -> int:
 
 
 def moe_plan(expert_of: torch.Tensor, num_experts: int) -> MoePlan:
-    """``expert_of [T, k]`` (int64) -> :class:`MoePlan`; slots of an expert keep their order."""
+    """``expert_of [T, k]`` (int64) -> :class:`MoePlan`; slots of an expert keep their order.  Slots with an id outside
+    ``[0, num_experts)`` have no row (``pos`` -1)."""
     t, k = expert_of.shape
     n = t * k
     rows = max_rows(n, num_experts)
@@ -59,15 +60,15 @@ def moe_plan(expert_of: torch.Tensor, num_experts: int) -> MoePlan:
         check(_lib.load().msrl_moe_plan(ptr(flat), c_int(n), c_int(num_experts), ptr(scratch), ptr(counts),
                                         ptr(offsets), ptr(pos), ptr(tiles), c_int(rows // PAD), stream()), "moe_plan")
         return MoePlan(counts, offsets, pos, tiles, rows, t, k, num_experts)
-    counts = torch.bincount(flat, minlength=num_experts)
+    counts = torch.bincount(flat[(flat >= 0) & (flat < num_experts)], minlength=num_experts)
     padded = (counts + PAD - 1) // PAD * PAD
     offsets = torch.zeros(num_experts + 1, dtype=torch.int64, device=dev)
     offsets[1:] = padded.cumsum(0)
+    pos = torch.full((n,), -1, dtype=torch.int64, device=dev)
     order = torch.argsort(flat, stable=True)
-    rank = guard.empty(n, dtype=torch.int64, device=dev)
+    order = order[(flat[order] >= 0) & (flat[order] < num_experts)]
     start = counts.cumsum(0) - counts
-    rank[order] = torch.arange(n, device=dev) - start[flat[order]]
-    pos = offsets[flat] + rank
+    pos[order] = offsets[flat[order]] + torch.arange(order.numel(), device=dev) - start[flat[order]]
     tiles = torch.full((rows // PAD,), -1, dtype=torch.int32, device=dev)
     for e in range(num_experts):
         tiles[int(offsets[e]) // PAD:int(offsets[e + 1]) // PAD] = e
@@ -87,6 +88,23 @@ def route_top(logits: torch.Tensor, top: int) -> Tuple[torch.Tensor, torch.Tenso
         return idx, score
     z, idx = torch.sort(logits, dim=-1, descending=True, stable=True)
     return idx[:, :top].contiguous(), torch.sigmoid(z[:, :top])
+
+
+def route_softmax_top(logits: torch.Tensor, correction: torch.Tensor, top: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Router logits ``[T, E]`` fp32 -> ``(ids [T, top] int64, scores [T, top] fp32)``: the ``top`` largest of
+    ``softmax(logits) + correction`` in descending order (equal ones: the lower id first) with their soft-max scores,
+    which the correction does not enter and which are not renormalised."""
+    t, e = logits.shape
+    if _lib.use_kernels(logits, correction):
+        logits = logits.contiguous()
+        idx = guard.empty(t, top, dtype=torch.int64, device=logits.device)
+        score = guard.empty(t, top, dtype=torch.float32, device=logits.device)
+        check(_lib.load().msrl_route_softmax_top(ptr(logits), ptr(correction), c_int(t), c_int(e), c_int(top), ptr(idx),
+                                                 ptr(score), stream()), "route_softmax_top")
+        return idx, score
+    s = torch.softmax(logits, dim=-1)
+    idx = torch.sort(s + correction, dim=-1, descending=True, stable=True).indices[:, :top].contiguous()
+    return idx, s.gather(1, idx)
 
 
 def moe_permute(x: torch.Tensor, plan: MoePlan, w: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -116,7 +134,8 @@ def moe_permute(x: torch.Tensor, plan: MoePlan, w: Optional[torch.Tensor] = None
     rows = x.repeat_interleave(plan.k, dim=0)
     if w is not None:
         rows = (rows.float() * w.reshape(-1, 1).float()).to(x.dtype)
-    xp[plan.pos.long()] = rows
+    used = plan.pos >= 0
+    xp[plan.pos[used].long()] = rows[used]
     return xp
 
 

@@ -3,7 +3,8 @@ follows fused in, and the gated activations.
 
 The residual ``[T, W]`` is fp32 and updated in place; norm weights are fp32, the activations bf16 or fp32.
 ``norm(x) = x / sqrt(mean(x^2) + eps) * (offset + w)`` in fp32; ``centered`` norms subtract the row's mean from x
-first (a layer norm without bias).  CUDA path: ``csrc/residual_stream.cu``; CPU
+first (a layer norm without bias).  ``post_*`` functions norm what a sublayer gives before it is added and hand on the
+residual itself, rounded to the activation type.  CUDA path: ``csrc/residual_stream.cu``; CPU
 tensors run the PyTorch formulation.
 """
 from __future__ import annotations
@@ -33,6 +34,13 @@ class Norm(NamedTuple):
     centered: bool = False
 
 
+class PostNorm(NamedTuple):
+    """Norm of a sublayer's output ``d`` and its factor: ``resid += mult * d / sqrt(mean(d^2) + eps) * weight``."""
+    weight: torch.Tensor
+    eps: float
+    mult: float = 1.0
+
+
 def _norm_ref(x: torch.Tensor, w: torch.Tensor, eps: float, offset: float, centered: bool, dtype) -> torch.Tensor:
     if centered:
         x = x - x.mean(-1, keepdim=True)
@@ -52,6 +60,55 @@ def embed_norm(ids: torch.Tensor, table: torch.Tensor, scale: float, w: torch.Te
         return resid, y
     resid = table[ids].float() * scale
     return resid, _norm_ref(resid, w, eps, offset, centered, table.dtype)
+
+
+def embed(ids: torch.Tensor, table: torch.Tensor, scale: float) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``(residual fp32, residual in the table's type)`` of ``residual = table[ids] * scale``."""
+    t, h = ids.numel(), table.shape[1]
+    if _lib.use_kernels(ids, table):
+        resid = guard.empty(t, h, device=table.device, dtype=torch.float32)
+        y = guard.empty(t, h, device=table.device, dtype=table.dtype)
+        check(_lib.load().msrl_embed_norm(ptr(ids), ptr(table), c_float(scale), ptr(resid), None, ptr(y), c_ll(t),
+                                          c_int(h), c_float(0.0), c_float(0.0), c_int(0), _is_f32(table), stream()), "embed")
+        return resid, y
+    resid = table[ids].float() * scale
+    return resid, resid.to(table.dtype, copy=True)
+
+
+def _post_ref(resid, d, post: PostNorm, after: Optional[Norm], dtype):
+    resid.add_(post.mult * (d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + post.eps) * post.weight))
+    return resid.to(dtype, copy=True) if after is None else _norm_ref(resid, *after, dtype)
+
+
+def post_add_(resid: torch.Tensor, delta: torch.Tensor, post: PostNorm, after: Optional[Norm] = None) -> torch.Tensor:
+    """Add the normed ``delta`` in place; returns the sum (or, with ``after``, that norm of it) in ``delta``'s type."""
+    if _lib.use_kernels(resid, delta, post.weight):
+        return _post(resid, post, after, delta.dtype, delta=delta.contiguous())
+    return _post_ref(resid, delta.float(), post, after, delta.dtype)
+
+
+def moe_post_add_(resid: torch.Tensor, expert_rows: torch.Tensor, pos: torch.Tensor, weights: torch.Tensor, post: PostNorm,
+                  after: Optional[Norm] = None, shared: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The same for ``d[t] = sum_j weights[t, j] * expert_rows[pos[t, j]] (+ shared[t])``; a negative ``pos`` is an expert
+    that gives back its input, the residual's row.  ``weights [T, top]`` fp32."""
+    if _lib.use_kernels(resid, expert_rows, pos, weights):
+        return _post(resid, post, after, expert_rows.dtype, rows=expert_rows, pos=pos, weights=weights.contiguous(), shared=shared)
+    pos = pos.long().view(resid.shape[0], -1)
+    rows = torch.where((pos < 0)[..., None], resid[:, None, :], expert_rows[pos.clamp(min=0)].float())
+    d = (rows * weights[..., None]).sum(1)
+    return _post_ref(resid, d if shared is None else d + shared.float(), post, after, expert_rows.dtype)
+
+
+def _post(resid, post, after, dtype, delta=None, rows=None, pos=None, weights=None, shared=None):
+    t, width = resid.shape
+    if after is not None and (after.centered or after.offset):
+        raise ValueError("the norm behind a post-normed layer is a plain RMS norm")
+    y = guard.empty(t, width, device=resid.device, dtype=dtype)
+    check(_lib.load().msrl_post_add(
+        ptr(delta), ptr(rows), ptr(pos), ptr(weights), c_int(0 if weights is None else weights.shape[1]), ptr(shared), ptr(resid),
+        ptr(post.weight), c_float(post.eps), c_float(post.mult), ptr(after.weight if after else None),
+        c_float(after.eps if after else 0.0), ptr(y), c_ll(t), c_int(width), _is_f32(y), stream()), "post_add")
+    return y
 
 
 def add_norm_(resid: torch.Tensor, delta: torch.Tensor, w: torch.Tensor, eps: float, offset: float = 0.0,

@@ -4,7 +4,8 @@ Query / key heads of ``dim`` and value heads of ``vdim`` entries are stored padd
 (:class:`GroupedHeads`); the pad entries are zero.  ``qkv_prep_`` turns fused projection rows into what attention and
 the cache take: RMS norm over the whole query and the whole key projection, partial rotation (entry i with entry
 i + dims / 2), and values mixed with those of another layer, in one kernel (``csrc/qkv_prep.cu``).  Token i sees the
-``window`` tokens up to and including itself (None: all).  Prompt attention: ``csrc/attention_tcgen05.cu``,
+``window`` tokens up to and including itself (None: all); decode steps may see their ``chunk`` of tokens instead (prompts in
+chunks are packed as one sequence per chunk).  ``ops.ScoreForm``: soft cap, sink and gates.  Prompt attention: ``csrc/attention_tcgen05.cu``,
 ``csrc/attention.cu``; decode: ``csrc/decode.cu``; fp32 and head sizes outside those: ``csrc/attention_simt.cu``.  CPU
 tensors run the PyTorch formulation.
 """
@@ -24,6 +25,7 @@ from .attention import _NOT_SUPPORTED, use_tcgen05_attention
 from .elementwise import _workspace
 from .latent import latent_gather
 from .residual import _is_f32
+from .score_form import PLAIN, ScoreForm
 
 TENSOR_CORE_HEADS = ((64, 64), (128, 128), (192, 128))
 
@@ -110,7 +112,7 @@ def rows_gather(cache: torch.Tensor, block_tables: torch.Tensor, token_seq: torc
 
 def window_prefill_attention(proj: torch.Tensor, lay: GroupedHeads, cu_q: torch.Tensor, cu_k: torch.Tensor, max_q: int,
                              scale: float, window: Optional[int], kv: Optional[Tuple[torch.Tensor, torch.Tensor]] = None,
-                             use_tcgen05: bool = True) -> torch.Tensor:
+                             use_tcgen05: bool = True, form: ScoreForm = PLAIN) -> torch.Tensor:
     """Causal window attention of the query heads of prepared rows -> ``[T, heads * vp]``.  Keys and values are those of
     the same rows, or ``kv = (k [Tk, kv_heads, qp], v [Tk, kv_heads, vp])`` delimited by ``cu_k`` (bottom-right aligned
     when a sequence has more keys than queries)."""
@@ -133,20 +135,20 @@ def window_prefill_attention(proj: torch.Tensor, lay: GroupedHeads, cu_q: torch.
                 rc = L.msrl_flash_attn_varlen_fwd_tcgen05(
                     ptr(q), ptr(k), ptr(v), spec, ptr(out), c_ll(h * lay.vp), ptr(lse), ptr(cu_q), ptr(cu_k), c_int(batch),
                     c_int(max_q), c_int(h), c_int(g), c_ll(t), c_ll(tk), c_int(lay.qp), c_float(scale), c_int(1), win,
-                    ptr(_status_word(proj.device)), stream())
+                    *form.args(), ptr(_status_word(proj.device)), stream())
                 if rc != _NOT_SUPPORTED:
                     check(rc, "flash_attn_varlen_fwd_tcgen05")
                     return out
             if lay.qp <= 128:
                 check(L.msrl_flash_attn_varlen_fwd(
                     ptr(q), ptr(k), ptr(v), spec, ptr(out), c_ll(h * lay.vp), ptr(lse), ptr(cu_q), ptr(cu_k), c_int(batch),
-                    c_int(max_q), c_int(h), c_int(g), c_ll(t), c_int(lay.qp), c_float(scale), c_int(1), win, stream()),
-                    "flash_attn_varlen_fwd")
+                    c_int(max_q), c_int(h), c_int(g), c_ll(t), c_int(lay.qp), c_float(scale), c_int(1), win, *form.args(),
+                    stream()), "flash_attn_varlen_fwd")
                 return out
         lds = (ctypes.c_longlong * 4)(ld, kld, vld, h * lay.vp)
         ints = (ctypes.c_int * 8)(lay.qp, lay.qp, lay.vp, lay.vp, lay.qp, lay.vp, h // g, window or 0)
         check(L.msrl_attn_simt(ptr(q), ptr(k), ptr(v), ptr(out), lds, ints, ptr(cu_q), ptr(cu_k), c_int(batch), c_int(max_q),
-                               c_int(h), c_float(scale), _is_f32(proj), stream()), "attn_simt")
+                               c_int(h), c_float(scale), *form.args(), _is_f32(proj), stream()), "attn_simt")
         return out
     q, k, v = lay.split(proj)
     if kv is not None:
@@ -159,16 +161,17 @@ def window_prefill_attention(proj: torch.Tensor, lay: GroupedHeads, cu_q: torch.
         qi, ki, vi = q[cq[b]:cq[b + 1]], k[ck[b]:ck[b + 1]], v[ck[b]:ck[b + 1]]
         back = torch.arange(qi.shape[0])[:, None] + (ki.shape[0] - qi.shape[0]) - torch.arange(ki.shape[0])
         hide = (back < 0) | (back >= (window or back.shape[1] + 1))
-        s = (torch.einsum("qhd,khd->hqk", qi, ki) * scale).masked_fill(hide, float("-inf"))
-        out[cq[b]:cq[b + 1]] = torch.einsum("hqk,khd->qhd", torch.softmax(s, dim=-1), vi)
-    return out.view(t, h * lay.vp).to(proj.dtype)
+        p = form.weights(torch.einsum("qhd,khd->hqk", qi, ki) * scale, hide)
+        out[cq[b]:cq[b + 1]] = torch.einsum("hqk,khd->qhd", p, vi)
+    return form.gated(out).view(t, h * lay.vp).to(proj.dtype)
 
 
 def window_decode_attention(proj: torch.Tensor, lay: GroupedHeads, k_cache: torch.Tensor, v_cache: torch.Tensor,
                             block_tables: torch.Tensor, context_lens: torch.Tensor, max_context: int, scale: float,
-                            window: Optional[int], nsplit: Optional[int] = None) -> torch.Tensor:
-    """One query per sequence (prepared rows; the cache holds their own keys too) over the last ``window`` cached tokens
-    -> ``[B, heads * vp]``.  ``nsplit``: key ranges per sequence (default: what fills the machine)."""
+                            window: Optional[int], nsplit: Optional[int] = None, chunk: Optional[int] = None,
+                            form: ScoreForm = PLAIN) -> torch.Tensor:
+    """One query per sequence (prepared rows; the cache holds their own keys too) over the last ``window`` cached tokens,
+    or those of its ``chunk`` -> ``[B, heads * vp]``.  ``nsplit``: key ranges per sequence (default: what fills the machine)."""
     b, h, g = proj.shape[0], lay.heads, lay.kv_heads
     bs = k_cache.shape[1]
     if _lib.use_kernels(proj, k_cache, v_cache, block_tables, context_lens):
@@ -176,7 +179,7 @@ def window_decode_attention(proj: torch.Tensor, lay: GroupedHeads, k_cache: torc
         out = guard.empty(b, h * lay.vp, device=proj.device, dtype=proj.dtype)
         q = proj.view(-1)[lay.q_col:]
         if proj.dtype == torch.bfloat16 and (lay.qp, lay.vp) in TENSOR_CORE_HEADS:
-            longest = min(int(max_context), window or int(max_context))
+            longest = min(int(max_context), window or chunk or int(max_context))
             n = nsplit or int(L.msrl_paged_decode_nsplit(c_int(b), c_int(g * ((h // g + 15) // 16)), c_int(longest)))
             part_o = _workspace("decode_part_o", b * h * n * lay.vp, proj.device)
             part_ml = _workspace("decode_part_ml", b * h * n * 2, proj.device)
@@ -184,20 +187,21 @@ def window_decode_attention(proj: torch.Tensor, lay: GroupedHeads, k_cache: torc
             check(L.msrl_paged_decode_window(
                 ptr(q), spec, ptr(k_cache), ptr(v_cache), ptr(block_tables), c_int(block_tables.shape[1]), ptr(context_lens),
                 ptr(out), c_ll(h * lay.vp), ptr(part_o), ptr(part_ml), c_int(b), c_int(h), c_int(g), c_int(lay.qp), c_int(lay.vp),
-                c_int(bs), c_float(scale), c_int(window or 0), c_int(n), stream()), "paged_decode_window")
+                c_int(bs), c_float(scale), c_int(window or 0), c_int(chunk or 0), *form.args(), c_int(n), stream()),
+                "paged_decode_window")
             return out
-        ints = (ctypes.c_int * 8)(h, g, lay.qp, lay.vp, bs, block_tables.shape[1], window or 0, lay.qp)
+        ints = (ctypes.c_int * 9)(h, g, lay.qp, lay.vp, bs, block_tables.shape[1], window or 0, lay.qp, chunk or 0)
         check(L.msrl_paged_decode_simt(ptr(q), c_ll(proj.stride(0)), ptr(k_cache), ptr(v_cache), ptr(block_tables),
-                                       ptr(context_lens), ptr(out), ints, c_int(b), c_float(scale), _is_f32(proj), stream()),
-              "paged_decode_simt")
+                                       ptr(context_lens), ptr(out), ints, c_int(b), c_float(scale), *form.args(), _is_f32(proj),
+                                       stream()), "paged_decode_simt")
         return out
     q = lay.split(proj)[0].float()
     out = torch.zeros(b, h, lay.vp)
     for i in range(b):
         n = int(context_lens[i])
-        pos = torch.arange(max(0, n - (window or n)), n)
+        pos = torch.arange(max(n - 1, 0) // chunk * chunk if chunk else max(0, n - (window or n)), n)
         at = block_tables[i, (pos // bs).long()].long() * bs + pos % bs
         k, v = (c.view(-1, *c.shape[2:])[at].float().repeat_interleave(h // g, dim=1) for c in (k_cache, v_cache))
-        p = torch.softmax(torch.einsum("hd,jhd->hj", q[i], k) * scale, dim=-1)
+        p = form.weights(torch.einsum("hd,jhd->hj", q[i], k) * scale)
         out[i] = torch.einsum("hj,jhd->hd", p, v)
-    return out.view(b, h * lay.vp).to(proj.dtype)
+    return form.gated(out).view(b, h * lay.vp).to(proj.dtype)

@@ -25,12 +25,14 @@ import numpy as np
 import torch
 
 from .. import ops
+from ..models.hybrid_config import Chunk, KeyRange, first_key
 from ..models.transformer_config import TransformerConfig
 from ..obs.io_counter import count_d2h, to_device, to_host
 from ..parallel.tp_comm import NO_TP, TPComm
 from .base_engine import BaseInferEngine
 from .block_manager import BlockManager
 from .layer_cache import HybridCache, StateSlots
+from .mixers import KeySpan
 from .model_runner import ModelRunner, RolloutWeights
 from .scheduler import (PrefillItem, RequestGroup, SamplingParams, Scheduler, SchedulerOutput, SeqStatus,
                         Sequence)
@@ -302,14 +304,16 @@ class LLMEngine(BaseInferEngine):
         t_ids, t_pos, t_slots = tok[0], tok[1].to(torch.int32), tok[2]
         t_cu = to_device(cu, torch.int32, dev)
         t_last = to_device(last_rows, torch.int64, dev)
-        prefix = None
+        prefix = bt = None
         if need_prefix:
             max_blocks = max(len(self.bm.block_table(it.seq.seq_id)) for it in items)
             bt = self.bm.block_tables([it.seq.seq_id for it in items], max_blocks)
             bt = to_device(bt, torch.int32, dev)
-            prefix = {w: self._prefix_keys(items, bt, w) for w in (self.cfg.windows if self.cfg.is_hybrid else (None,))}
-            if not self.cfg.is_hybrid:
-                prefix = prefix[None]
+        if self.cfg.is_hybrid:
+            prefix = {keys: self._key_span(items, bt, keys) for keys in self.cfg.windows if need_prefix or isinstance(keys, Chunk)}
+        elif need_prefix:
+            span = self._key_span(items, bt, None)
+            prefix = dict(span.cached, cu_k=span.cu_k)
         state = None
         if self.cfg.is_hybrid:
             st, _ = self._ship([[it.start for it in items], [it.seq.state_slot for it in items]])
@@ -323,18 +327,29 @@ class LLMEngine(BaseInferEngine):
             self.bm.commit(it.seq.seq_id, it.seq.all_ids, it.seq.num_computed)
         return logits
 
-    def _prefix_keys(self, items: List[PrefillItem], block_tables: torch.Tensor, window: Optional[int]) -> dict:
-        """Cache positions that the tokens of prompt portions look at: everything up to a portion's end, or from the
-        first key inside the portion's first window."""
-        ends = np.array([it.start + it.length for it in items])
-        first = np.zeros_like(ends) if window is None else np.maximum([it.start - window + 1 for it in items], 0)
-        n = ends - first
-        cu = np.concatenate([[0], np.cumsum(n)])
-        owner = np.repeat(np.arange(len(items)), n)
-        pos = np.arange(cu[-1]) - cu[owner] + first[owner]
-        pt, _ = self._ship([owner, pos])
-        return dict(block_tables=block_tables, token_seq=pt[0].to(torch.int32), token_pos=pt[1].to(torch.int32),
-                    cu_k=to_device(cu.tolist(), torch.int32, self.device))
+    def _key_span(self, items: List[PrefillItem], block_tables: Optional[torch.Tensor], keys: KeyRange) -> KeySpan:
+        """What the tokens of prompt portions look at: the cached keys (``block_tables``; None: fresh prompts, whose keys are
+        their own rows) from the first one that a portion's first token sees to the portion's end.  Layers that see chunks
+        get a packed sequence per chunk."""
+        starts = np.array([it.start for it in items])
+        ends = starts + np.array([it.length for it in items])
+        first = first_key(keys, starts)
+        len_q, len_k = ends - starts, ends - first
+        if isinstance(keys, Chunk):
+            len_q, len_k = [], []
+            for lo, at, end in zip(first, starts, ends):
+                edges = np.append(np.arange(lo, end, keys.size), end)      # chunk borders; the first may lie before the portion
+                len_k.extend(np.diff(edges))
+                len_q.extend(np.diff(np.maximum(edges, at)))
+        cu_q, cu_k = (to_device(np.concatenate([[0], np.cumsum(n)]).tolist(), torch.int32, self.device) for n in (len_q, len_k))
+        cached = None
+        if block_tables is not None:
+            n = ends - first
+            owner = np.repeat(np.arange(len(items)), n)
+            pos = np.arange(n.sum()) - (np.cumsum(n) - n)[owner] + first[owner]
+            pt, _ = self._ship([owner, pos])
+            cached = dict(block_tables=block_tables, token_seq=pt[0].to(torch.int32), token_pos=pt[1].to(torch.int32))
+        return KeySpan(cu_q, cu_k, int(max(len_q)), cached)
 
     def _run_prefill(self, items: List[PrefillItem]) -> None:
         finishing = [it.seq for it in items if it.completes_prompt]

@@ -2,7 +2,8 @@
 
 ``forward`` does the feed-forward's work on ``h`` up to what is left to add; ``finish_`` adds it (and, in layers whose
 sublayers run in parallel, the mixer's output ``delta``) to the fp32 residual and returns the next norm of the sum, so
-that the add (and for expert layers the combine) and the norm are one kernel.  ``norm``: an ``ops.Norm``.
+that the add (and for expert layers the combine) and the norm are one kernel.  ``norm``: an ``ops.Norm``.  In designs
+that norm a sublayer's output, ``finish_post_`` takes the place of ``finish_``; ``post``: an ``ops.PostNorm``.
 """
 from __future__ import annotations
 
@@ -11,7 +12,7 @@ from typing import Dict, Optional, Tuple
 import torch
 
 from .. import ops
-from ..models.hybrid_config import GluSpec, ScoredMoESpec, TableMoESpec
+from ..models.hybrid_config import GluSpec, ScoredMoESpec, SoftmaxMoESpec, TableMoESpec
 from ..ops import moe as K
 from ..ops.gemm import linear_f32, linear_fwd
 from .mixers import _pad_cols, _pad_rows
@@ -32,6 +33,9 @@ class Glu:
 
     def finish_(self, resid, h, done, norm, delta: Optional[torch.Tensor] = None) -> torch.Tensor:
         return ops.add_norm_(resid, done, *norm, delta2=delta)
+
+    def finish_post_(self, resid, done, post, after) -> torch.Tensor:
+        return ops.post_add_(resid, done, post, after)
 
 
 class GroupedExperts:
@@ -96,7 +100,28 @@ class ScoredMoE(GroupedExperts):
         return self.run(h, K.moe_plan(idx, self.spec.experts), score)
 
 
-FEED_FORWARDS = {GluSpec: Glu, TableMoESpec: TableMoE, ScoredMoESpec: ScoredMoE}
+class SoftmaxMoE(GroupedExperts):
+    """Router scores are a 32-bit soft-max; what is chosen also depends on a correction per output.  Identity experts have
+    no rows in the dispatch plan: the combine takes their input, the residual, where it adds the others."""
+
+    def __init__(self, spec: SoftmaxMoESpec, w: Dict[str, torch.Tensor], dtype, device):
+        super().__init__(spec, w, dtype, device)
+        self.router = w["router"].to(device=device, dtype=dtype).contiguous()
+        self.correction = w["correction"].reshape(-1).to(device=device, dtype=torch.float32).contiguous()
+        if self.router.shape[0] != spec.outputs or self.correction.numel() != spec.outputs:
+            raise ValueError(f"router {tuple(self.router.shape)} and correction {self.correction.numel()} do not fit {spec.outputs} "
+                             "outputs")
+
+    def forward(self, h: torch.Tensor, ids: torch.Tensor):
+        idx, score = K.route_softmax_top(linear_f32(h, self.router), self.correction, self.spec.top)
+        return *self.run(h, K.moe_plan(idx, self.spec.experts)), score
+
+    def finish_post_(self, resid, done, post, after) -> torch.Tensor:
+        y, plan, shared, score = done
+        return ops.moe_post_add_(resid, y, plan.pos, score, post, after, shared)
+
+
+FEED_FORWARDS = {GluSpec: Glu, TableMoESpec: TableMoE, ScoredMoESpec: ScoredMoE, SoftmaxMoESpec: SoftmaxMoE}
 
 
 def build_feed_forward(spec, w: Dict[str, torch.Tensor], dtype, device):

@@ -45,8 +45,8 @@ class _Taken(dict):
 
 def build_hybrid_weights(cfg: HybridConfig, state: Dict[str, torch.Tensor], device) -> HybridWeights:
     """``state``: checkpoint tensors (``embed``, ``final.norm``, ``l<i>.norm1``, ``l<i>.mix.*``, ``l<i>.mlp.*``, and
-    ``l<i>.norm2`` and ``head`` where the design has them; else the LM head is the embedding table).  A name that no
-    layer asks for is an error."""
+    ``l<i>.norm2`` and ``head`` where the design has them; else the LM head is the embedding table).  A layer that uses
+    another one's tensors has none, and shares its objects.  A name that no layer asks for is an error."""
     dt = cfg.params_dtype
     used = {"embed", "final.norm"}
 
@@ -54,8 +54,10 @@ def build_hybrid_weights(cfg: HybridConfig, state: Dict[str, torch.Tensor], devi
         used.add(name)
         return state[name].to(device=device, dtype=torch.float32).contiguous()
 
-    layers = []
+    layers: List[Optional[HybridLayer]] = [None] * len(cfg.layers)
     for i, spec in enumerate(cfg.layers):
+        if cfg.owner(i) != i:
+            continue
         p = f"l{i}."
         layer = HybridLayer(f32(p + "norm1"),
                             MIXERS[type(spec.mixer)](spec.mixer, _Taken(state, p + "mix.", used), cfg.norm_epsilon, dt, device))
@@ -63,7 +65,9 @@ def build_hybrid_weights(cfg: HybridConfig, state: Dict[str, torch.Tensor], devi
             if not cfg.design.parallel:
                 layer.norm2 = f32(p + "norm2")
             layer.ff = build_feed_forward(spec.mlp, _Taken(state, p + "mlp.", used), dt, device)
-        layers.append(layer)
+        layers[i] = layer
+    layers = [layers[cfg.owner(i)] for i in range(len(layers))]
+
     def table(name):
         used.add(name)
         t = state[name].to(device=device, dtype=dt).contiguous()

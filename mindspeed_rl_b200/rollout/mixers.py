@@ -7,17 +7,28 @@ return the mixer's output before the residual add.
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Dict, List, Optional
+from typing import Dict, List, NamedTuple, Optional
 
 import torch
 
 from .. import ops
-from ..models.hybrid_config import ChannelDeltaSpec, LatentAttentionSpec, MatrixMemorySpec, WindowAttentionSpec
+from ..models.hybrid_config import (ChannelDeltaSpec, Chunk, ConvAttentionSpec, HeadDeltaSpec, KeyRange, LatentAttentionSpec,
+                                    MatrixMemorySpec, WindowAttentionSpec)
+from ..ops.conv_qkv import ConvHeads, ConvNormWeights
 from ..ops.delta import DeltaLayout, DeltaWeights
 from ..ops.gemm import linear_f32, linear_fwd
 from ..ops.latent import LatentLayout, pad16
 from ..ops.matrix_memory import MemoryLayout, MemoryWeights
 from ..ops.window import GroupedHeads, ValueSource
+
+
+class KeySpan(NamedTuple):
+    """Queries and keys of a prompt step as packed sequences of one attention call (a layer that sees chunks has a
+    sequence per chunk)."""
+    cu_q: torch.Tensor
+    cu_k: torch.Tensor
+    max_q: int
+    cached: Optional[dict] = None           # block_tables, token_seq, token_pos of the keys; None: the step's own rows
 
 
 @dataclass
@@ -33,7 +44,7 @@ class StepMeta:
     max_q: int = 0
     tok_seq: Optional[torch.Tensor] = None  # [T] int32
     start_pos: Optional[torch.Tensor] = None  # [B] int32 position of a portion's first token
-    prefix: Optional[dict] = None           # by key range (``HybridConfig.windows``); see ModelRunner.prefill
+    spans: Optional[Dict[KeyRange, KeySpan]] = None     # where a key range needs more than the packed portions
     # decode steps
     block_tables: Optional[torch.Tensor] = None
     context_lens: Optional[torch.Tensor] = None
@@ -41,8 +52,9 @@ class StepMeta:
     # values of the first layer that mixes values, kept for the later ones of the step
     first_values: Optional[ValueSource] = None
 
-    def prefix_of(self, window: Optional[int]) -> Optional[dict]:
-        return None if self.prefix is None else self.prefix[window]
+    def span_of(self, keys: KeyRange) -> KeySpan:
+        span = None if self.spans is None else self.spans.get(keys)
+        return span or KeySpan(self.cu_q, self.cu_q, self.max_q)
 
     @property
     def is_decode(self) -> bool:
@@ -73,6 +85,11 @@ def _pad_heads(w: torch.Tensor, heads: int, dim: int, to: int) -> torch.Tensor:
     return torch.cat([x, x.new_zeros(heads, to - dim, *w.shape[1:])], dim=1).reshape(heads * to, *w.shape[1:])
 
 
+def _table_rows(meta: StepMeta) -> int:
+    """Length of rotation tables: whole powers of two, so that engines with different length limits share them."""
+    return 1 << max(meta.max_model_len - 1, 1).bit_length()
+
+
 def stack_sections(parts: List[torch.Tensor]):
     """Rows of several projections of one input as one weight; every section starts on a multiple of eight
     columns of the product (zero rows in between).  Returns the weight and the section starts."""
@@ -95,78 +112,100 @@ class LatentAttention:
         if dtype == torch.bfloat16 and vp <= 128 and qp <= 192:
             vp = 64 if max(qp, vp) <= 64 else 128
             qp = 192 if qp > 128 else vp
-        q = _pad_cols(w["q"].view(h, dn + dr, -1).transpose(1, 2), qp).transpose(1, 2).reshape(h * qp, -1)
-        fused, cols = stack_sections([q, w["dkv"]])
-        self.lay = lay = LatentLayout(h, dn, dr, dv, r, qp, vp, cols[1], spec.rot.dims)
+
+        def put(t, dt=dtype):
+            return t.to(device=device, dtype=dt).contiguous()
+
+        q = w["uq" if spec.q_rank else "q"]
+        q = _pad_cols(q.view(h, dn + dr, -1).transpose(1, 2), qp).transpose(1, 2).reshape(h * qp, -1)
+        fused, cols = stack_sections([w["dq"] if spec.q_rank else q, w["dkv"]] + ([w["g"]] if spec.head_gate else []))
+        self.lay = lay = LatentLayout(h, dn, dr, dv, r, qp, vp, cols[1], spec.rot.dims, spec.rot.halves, spec.q_rank or 0, cols[0])
+        if spec.q_rank:
+            self.w_uq = put(_pad_cols(q, lay.QP))
+            self.q_norm = put(w["dq.norm"], torch.float32)
+        self.g_cols = slice(cols[2], cols[2] + h) if spec.head_gate else None
+        self.sink = put(w["sink"].reshape(-1), torch.float32) if spec.sink else None
         uk = _pad_cols(w["uk"], lay.RP).view(h, dn, lay.RP)
         uv = _pad_cols(w["uv"], lay.RP).view(h, dv, lay.RP)
         k_rows = torch.cat([uk, uk.new_zeros(h, qp - dn, lay.RP)], dim=1)
         v_rows = torch.cat([uv, uv.new_zeros(h, vp - dv, lay.RP)], dim=1)
-
-        def put(t):
-            return t.to(device=device, dtype=dtype).contiguous()
-
         self.w_in = put(fused)
         self.w_kv = put(torch.cat([k_rows.reshape(h * qp, lay.RP), v_rows.reshape(h * vp, lay.RP)]))
         self.w_k = self.w_kv[:h * qp].view(h, qp, lay.RP)[:, :dn]       # [H, dn, RP]: folds W_uk into the query
         self.w_v = self.w_kv[h * qp:].view(h, vp, lay.RP)               # [H, vp, RP]
         self.w_o = put(_pad_cols(w["o"].view(-1, h, dv), vp).reshape(-1, h * vp))
-        self.norm = w["dkv.norm"].to(device=device, dtype=torch.float32).contiguous()
+        self.norm = put(w["dkv.norm"], torch.float32)
 
-    def _table(self, meta: StepMeta) -> torch.Tensor:
-        # whole powers of two, so that engines with different length limits share tables
-        rows = 1 << max(meta.max_model_len - 1, 1).bit_length()
-        return ops.rope_table(rows, self.spec.rot.dims, self.spec.rot.base, self.w_in.device)
+    def _form(self, proj: torch.Tensor) -> ops.ScoreForm:
+        return ops.ScoreForm(0.0, None if self.g_cols is None else proj[:, self.g_cols], self.sink)
+
+    def _queries(self, proj: torch.Tensor, meta: StepMeta, stored: torch.Tensor, want_rows: bool, decode_q=None):
+        """Rows that begin with the prepared query heads, and the step's cache rows."""
+        lay, rot = self.lay, self.spec.rot
+        table = ops.rope_table(_table_rows(meta), rot.dims, rot.base, self.w_in.device)
+        args = (proj, lay, self.norm, self.eps, table, meta.positions, meta.slots, stored, want_rows)
+        if not lay.q_rank:
+            return proj, ops.latent_prep(*args, decode_q=decode_q)
+        rows, cq = ops.latent_prep(*args, q_norm=self.q_norm)
+        q = linear_fwd(cq, self.w_uq)
+        ops.latent_rotate_queries(q, lay, table, meta.positions, decode_q)
+        return q, rows
 
     def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
-        lay, pre = self.lay, meta.prefix_of(None)
+        lay, spec, span, stored = self.lay, self.spec, meta.span_of(self.spec.keys), cache.rows[run]["latent"]
         proj = linear_fwd(x, self.w_in)
-        rows = ops.latent_prep(proj, lay, self.norm, self.eps, self._table(meta), meta.positions, meta.slots,
-                               cache.rows[run]["latent"], want_rows=pre is None)
-        cu_k = meta.cu_q
-        if pre is not None:
-            rows = ops.latent_gather(cache.rows[run]["latent"], pre["block_tables"], pre["token_seq"], pre["token_pos"])
-            cu_k = pre["cu_k"]
+        q, rows = self._queries(proj, meta, stored, want_rows=span.cached is None)
+        if span.cached is not None:
+            rows = ops.latent_gather(stored, **span.cached)
         kv = linear_fwd(rows[:, :lay.RP], self.w_kv)
         ops.latent_spread_(kv, rows, lay)
-        attn = ops.latent_prefill_attention(proj, kv, lay, meta.cu_q, cu_k, meta.max_q, self.spec.scale)
+        attn = ops.latent_prefill_attention(q, kv, lay, span.cu_q, span.cu_k, span.max_q, spec.scale, spec.window, self._form(proj))
         return linear_fwd(attn, self.w_o)
 
     def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
-        lay, b = self.lay, x.shape[0]
+        lay, b, stored = self.lay, x.shape[0], cache.rows[run]["latent"]
         proj = linear_fwd(x, self.w_in)
         q = torch.empty(b, lay.heads, lay.CP, dtype=x.dtype, device=x.device)
-        ops.latent_prep(proj, lay, self.norm, self.eps, self._table(meta), meta.positions, meta.slots,
-                        cache.rows[run]["latent"], want_rows=False, decode_q=q)
-        heads = proj[:, :lay.heads * lay.qp].view(b, lay.heads, lay.qp)
+        heads, _ = self._queries(proj, meta, stored, want_rows=False, decode_q=q)
+        heads = heads[:, :lay.heads * lay.qp].view(b, lay.heads, lay.qp)
         torch.bmm(heads[..., :lay.dn].transpose(0, 1), self.w_k, out=q[..., :lay.RP].transpose(0, 1))
-        lat = ops.latent_decode_attention(q, cache.rows[run]["latent"], lay, meta.block_tables, meta.context_lens,
-                                          meta.max_context, self.spec.scale)
+        lat = ops.latent_decode_attention(q, stored, lay, meta.block_tables, meta.context_lens, meta.max_context, self.spec.scale,
+                                          window=self.spec.window, form=self._form(proj))
         attn = torch.empty(b, lay.heads, lay.vp, dtype=x.dtype, device=x.device)
         torch.bmm(lat.transpose(0, 1), self.w_v.transpose(1, 2), out=attn.transpose(0, 1))
         return linear_fwd(attn.view(b, lay.heads * lay.vp), self.w_o)
 
 
 class ChannelDelta:
+    """Decays and the output gate come through bottlenecks of two products."""
+    head_decay = silu_gate = False
+
     def __init__(self, spec, w: Dict[str, torch.Tensor], eps: float, dtype, device):
         self.spec, self.eps = spec, eps
-        fused, cols = stack_sections([w["q"], w["k"], w["v"], w["b"], w["a1"], w["g1"]])
-        self.lay = DeltaLayout(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.conv, *cols[:4],
-                               unit_eps=spec.unit_eps)
-        ra, rg = _pad8(w["a1"].shape[0]), _pad8(w["g1"].shape[0])
-        self.a_cols, self.g_cols = slice(cols[4], cols[4] + ra), slice(cols[5], cols[5] + rg)
+        decay, gate = self._inputs(w)
+        fused, cols = stack_sections([w["q"], w["k"], w["v"], w["b"], decay, gate])
+        self.lay = DeltaLayout(spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.conv, *cols[:4], unit_eps=spec.unit_eps,
+                               head_decay=self.head_decay, silu_gate=self.silu_gate)
+        self.a_cols, self.g_cols = (slice(c, c + _pad8(p.shape[0])) for c, p in ((cols[4], decay), (cols[5], gate)))
 
         def put(t, dt=dtype):
             return t.to(device=device, dtype=dt).contiguous()
 
         f32 = torch.float32
         self.w_in = put(fused)
-        self.w_a2, self.w_g2 = put(_pad_cols(w["a2"], ra)), put(_pad_cols(w["g2"], rg))
+        self._outputs(w, put)
         self.w_o = put(w["o"])
         self.state = DeltaWeights(conv=put(torch.cat([w["q.conv"], w["k.conv"], w["v.conv"]]), f32),
                                   a_log=put(w["A_log"], f32), dt_bias=put(w["dt_bias"], f32), norm=put(w["norm"], f32))
         if self.state.conv.shape != (self.lay.channels, spec.conv):
             raise ValueError(f"convolution weights {tuple(self.state.conv.shape)} do not fit {spec}")
+
+    def _inputs(self, w):
+        return w["a1"], w["g1"]
+
+    def _outputs(self, w, put):
+        self.w_a2 = put(_pad_cols(w["a2"], _pad8(w["a1"].shape[0])))
+        self.w_g2 = put(_pad_cols(w["g2"], _pad8(w["g1"].shape[0])))
 
     def _project(self, x: torch.Tensor):
         proj = linear_fwd(x, self.w_in)
@@ -183,6 +222,26 @@ class ChannelDelta:
         y = ops.delta_decode(proj, a, gate, self.lay, self.state, cache.slots[run]["ring"], cache.slots[run]["state"], meta.positions,
                              meta.state_slots, self.eps)
         return linear_fwd(y, self.w_o)
+
+
+class HeadDelta(ChannelDelta):
+    """One decay per head; decays and the output gate are sections of the fused projection."""
+    head_decay = silu_gate = True
+
+    def _inputs(self, w):
+        return w["a"], w["g"]
+
+    def _outputs(self, w, put):
+        pass
+
+    def _project(self, x: torch.Tensor):
+        proj, s = linear_fwd(x, self.w_in), self.spec
+        return proj, proj[:, self.a_cols][:, :s.heads], proj[:, self.g_cols][:, :s.heads * s.vdim]
+
+
+def _cached_kv(rows: Dict[str, torch.Tensor], span: KeySpan):
+    """Keys and values that a prompt step looks at, or None where they are its own rows."""
+    return None if span.cached is None else tuple(ops.rows_gather(rows[n], **span.cached) for n in ("k", "v"))
 
 
 class WindowAttention:
@@ -219,8 +278,7 @@ class WindowAttention:
         """Normed, rotated and mixed q | k | v rows, written to the cache."""
         lay, spec = self.lay, self.spec
         proj = linear_fwd(x, self.w_in, self.b_in)
-        length = 1 << max(meta.max_model_len - 1, 1).bit_length()       # see LatentAttention._table
-        table = ops.angle_table(length, spec.rot.frequencies(), x.device)
+        table = ops.angle_table(_table_rows(meta), spec.rot.frequencies(), x.device)
         first = meta.first_values if spec.value_mix else None
         ops.qkv_prep_(proj, lay, self.q_norm, self.k_norm, self.eps, table, meta.positions, meta.slots, rows["k"], rows["v"],
                       first, self.mix)
@@ -229,13 +287,10 @@ class WindowAttention:
         return proj
 
     def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
-        rows, pre, spec = cache.rows[run], meta.prefix_of(self.spec.window), self.spec
+        rows, span, spec = cache.rows[run], meta.span_of(self.spec.keys), self.spec
         proj = self._project(x, meta, rows)
-        kv, cu_k = None, meta.cu_q
-        if pre is not None:
-            kv = tuple(ops.rows_gather(rows[n], pre["block_tables"], pre["token_seq"], pre["token_pos"]) for n in ("k", "v"))
-            cu_k = pre["cu_k"]
-        attn = ops.window_prefill_attention(proj, self.lay, meta.cu_q, cu_k, meta.max_q, spec.scale, spec.window, kv)
+        attn = ops.window_prefill_attention(proj, self.lay, span.cu_q, span.cu_k, span.max_q, spec.scale, spec.window,
+                                            _cached_kv(rows, span))
         return linear_fwd(attn, self.w_o)
 
     def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
@@ -243,6 +298,53 @@ class WindowAttention:
         proj = self._project(x, meta, rows)
         attn = ops.window_decode_attention(proj, self.lay, rows["k"], rows["v"], meta.block_tables, meta.context_lens,
                                            meta.max_context, spec.scale, spec.window)
+        return linear_fwd(attn, self.w_o)
+
+
+class ConvAttention:
+    """Short convolutions, per-head norms and rotation between the projection and grouped-head attention.  The projection's
+    heads are stored as they are; prepared rows and the cache hold them padded (``padded_heads``)."""
+
+    def __init__(self, spec, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.spec, self.eps = spec, eps
+        h, g = spec.heads, spec.kv_heads
+        qp, vp = spec.padded(dtype)
+
+        def put(t, dt=dtype):
+            return t.to(device=device, dtype=dt).contiguous()
+
+        fused, cols = stack_sections([w["q"], w["k"], w["v"], w["g"]])
+        self.heads = GroupedHeads(h, g, spec.dim, spec.vdim, qp, vp, 0, h * qp, (h + g) * qp)
+        self.lay = ConvHeads(self.heads, spec.conv, *cols[:3])
+        self.g_cols = slice(cols[3], cols[3] + h)
+        self.w_in = put(fused)
+        f32 = torch.float32
+        self.prep = ConvNormWeights(put(torch.cat([w["q.conv"], w["k.conv"], w["v.conv"]]), f32), put(w["q.norm"], f32),
+                                    put(w["k.norm"], f32))
+        if self.prep.conv.shape != (spec.channels, spec.conv):
+            raise ValueError(f"convolution weights {tuple(self.prep.conv.shape)} do not fit {spec}")
+        self.w_o = put(_pad_cols(w["o"].reshape(-1, h, spec.vdim), vp).reshape(-1, h * vp))
+
+    def _prepare(self, prep, x, meta: StepMeta, cache, run: int, *where):
+        proj, rows = linear_fwd(x, self.w_in), cache.rows[run]
+        table = ops.angle_table(_table_rows(meta), self.spec.rot.frequencies(), x.device)
+        out = prep(proj, self.lay, self.prep, self.eps, table, meta.positions, meta.slots, rows["k"], rows["v"],
+                   cache.slots[run]["ring"], meta.state_slots, *where)
+        return out, rows, ops.ScoreForm(self.spec.softcap, proj[:, self.g_cols])
+
+    def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        spec, span = self.spec, meta.span_of(self.spec.keys)
+        qkv, rows, form = self._prepare(ops.conv_qkv_prefill, x, meta, cache, run, meta.tok_seq, meta.cu_q, meta.start_pos)
+        attn = ops.window_prefill_attention(qkv, self.heads, span.cu_q, span.cu_k, span.max_q, spec.scale,
+                                            None if isinstance(spec.keys, Chunk) else spec.keys, _cached_kv(rows, span), form=form)
+        return linear_fwd(attn, self.w_o)
+
+    def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        keys = self.spec.keys
+        q, rows, form = self._prepare(ops.conv_qkv_decode, x, meta, cache, run)
+        attn = ops.window_decode_attention(q, self.heads, rows["k"], rows["v"], meta.block_tables, meta.context_lens,
+                                           meta.max_context, self.spec.scale, None if isinstance(keys, Chunk) else keys,
+                                           chunk=keys.size if isinstance(keys, Chunk) else None, form=form)
         return linear_fwd(attn, self.w_o)
 
 
@@ -277,5 +379,5 @@ class MatrixMemory:
         return linear_fwd(y, self.w_o)
 
 
-MIXERS = {LatentAttentionSpec: LatentAttention, ChannelDeltaSpec: ChannelDelta, WindowAttentionSpec: WindowAttention,
-          MatrixMemorySpec: MatrixMemory}
+MIXERS = {LatentAttentionSpec: LatentAttention, ChannelDeltaSpec: ChannelDelta, HeadDeltaSpec: HeadDelta,
+          WindowAttentionSpec: WindowAttention, ConvAttentionSpec: ConvAttention, MatrixMemorySpec: MatrixMemory}

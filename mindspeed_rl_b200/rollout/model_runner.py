@@ -205,6 +205,8 @@ class ModelRunner:
         kernels that add and take the next norm in one pass."""
         w, c, cache = self.weights, self.cfg, self.cache
         order, parallel = c.run_order, c.design.parallel
+        if c.design.post_norm:
+            return self._forward_post_norm(meta)
 
         def norm(weight):
             return ops.Norm(weight, c.norm_epsilon, c.design.norm_offset, c.design.centered)
@@ -223,6 +225,24 @@ class ModelRunner:
                 x = lw.ff.finish_(resid, x, lw.ff.forward(x, meta.ids), after)
             else:
                 x = ops.add_norm_(resid, mix(x, meta, cache, run), *after)
+            if self.layer_probe is not None:
+                self.layer_probe(run, resid)
+        return x
+
+    def _forward_post_norm(self, meta: StepMeta) -> torch.Tensor:
+        """The same for designs that norm what a sublayer gives: sublayers read the residual itself (in the activation
+        type), and one kernel norms, scales and adds their output."""
+        w, c, cache = self.weights, self.cfg, self.cache
+        order = c.run_order
+        resid, x = ops.embed(meta.ids, w.embed, c.embedding_scale)
+        for run, li in enumerate(order):
+            lw = w.layers[li]
+            post1, post2 = (None if n is None else ops.PostNorm(n, c.norm_epsilon, c.residual_mult) for n in (lw.norm1, lw.norm2))
+            after = ops.Norm(w.final_norm, c.norm_epsilon) if run + 1 == len(order) else None
+            mix = lw.mixer.decode if meta.is_decode else lw.mixer.prefill
+            x = ops.post_add_(resid, mix(x, meta, cache, run), post1, after if lw.ff is None else None)
+            if lw.ff is not None:
+                x = lw.ff.finish_post_(resid, lw.ff.forward(x, meta.ids), post2, after)
             if self.layer_probe is not None:
                 self.layer_probe(run, resid)
         return x
@@ -259,8 +279,8 @@ class ModelRunner:
 
         ``prefix`` (for chunks that start inside a sequence) carries ``block_tables``,
         ``token_seq``, ``token_pos``, ``cu_k``: the K/V of ``[0, chunk_end)`` is gathered from the
-        cache after this chunk's K/V has been written.  Hybrid decoders get one such dictionary per key range
-        of their attention layers (``HybridConfig.windows``), which lists only the keys inside the range.
+        cache after this chunk's K/V has been written.  Hybrid decoders get a ``KeySpan`` per key range of their
+        attention layers (``HybridConfig.windows``) that lists only the keys inside the range.
 
         ``state`` (hybrid decoders): ``token_seq [T]`` and ``start_pos [B]`` (int32), ``slots [B]`` (int64, the
         recurrent-state slot of every sequence).
@@ -268,7 +288,7 @@ class ModelRunner:
         cache = self.cache
         if self.cfg.is_hybrid:
             meta = StepMeta(ids, positions, slots, state["slots"], self.max_model_len, cu_q=cu_q, max_q=max_q,
-                            tok_seq=state["token_seq"], start_pos=state["start_pos"], prefix=prefix)
+                            tok_seq=state["token_seq"], start_pos=state["start_pos"], spans=prefix)
             return self._logits(self._forward_hybrid(meta)[last_index])
 
         def attend(li, qkv, lay):
