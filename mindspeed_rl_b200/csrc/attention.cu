@@ -14,6 +14,7 @@
 //
 // Replaces the reference's dependency on an external fused attention with
 // `set_actual_seq_len` (mindspeed_rl/models/base/base_training_engine.py:384-391).
+#include "head_tail.cuh"
 #include "mma_utils.cuh"
 
 namespace msrl {
@@ -34,6 +35,8 @@ struct AttnParams {
   float scale_log2;        // scale * log2(e)
   int causal;
   int window;                 // forward: keys a query sees, itself included (0: all)
+  float softcap;              // forward: cap of the scaled scores (0: none)
+  HeadTail<__nv_bfloat16> tail;
   // backward only
   const __nv_bfloat16* dout;  // same layout as o
   float* delta;               // [nh, Tq] rowsum(dO * O)
@@ -48,7 +51,7 @@ constexpr float kLn2 = 0.6931471805599453f;
 // ---------------------------------------------------------------------------------------------
 // Forward
 // ---------------------------------------------------------------------------------------------
-template <int D>
+template <int D, bool CAP>
 __global__ void __launch_bounds__(128) fa_fwd_kernel(const AttnParams p) {
   constexpr int BM = 64, BN = 64, LD = D + 8, THREADS = 128;
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -70,6 +73,7 @@ __global__ void __launch_bounds__(128) fa_fwd_kernel(const AttnParams p) {
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int qrow = lane >> 2, qcol = (lane & 3) * 2;
+  const SoftCap2 cap(CAP ? p.softcap : 1.f);
 
   load_tile_async<BM, D, LD, THREADS>(sQ, p.q, p.Lq, h, q0, m0, qlen);
   if (n_tiles > t0) {
@@ -131,6 +135,7 @@ __global__ void __launch_bounds__(128) fa_fwd_kernel(const AttnParams p) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         float v = s[nt][j] * p.scale_log2;
+        if constexpr (CAP) v = cap(v);
         if (need_mask) {
           const int key = kbase + nt * 8 + qcol + (j & 1);
           const int row = m0 + warp * 16 + qrow + ((j >> 1) << 3);
@@ -201,7 +206,7 @@ __global__ void __launch_bounds__(128) fa_fwd_kernel(const AttnParams p) {
   for (int r = 0; r < 2; ++r) {
     const int row = m0 + warp * 16 + qrow + r * 8;
     if (row >= qlen) continue;
-    const float inv = (l_run[r] > 0.f) ? 1.f / l_run[r] : 0.f;
+    const float inv = p.tail.scale2(q0 + row, h, m_run[r], l_run[r]);
     __nv_bfloat16* orow = p.o + (long long)(q0 + row) * p.o_stride_t + (long long)h * D;
 #pragma unroll
     for (int dt = 0; dt < D / 8; ++dt) {
@@ -529,10 +534,11 @@ template <int D>
 static int launch_fwd(const AttnParams& p, int batch, int max_q, cudaStream_t st) {
   constexpr int LD = D + 8;
   const size_t smem = (size_t)(64 + 4 * 64) * LD * sizeof(__nv_bfloat16);
-  cudaError_t e = cudaFuncSetAttribute(fa_fwd_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  auto* kernel = p.softcap > 0.f ? fa_fwd_kernel<D, true> : fa_fwd_kernel<D, false>;
+  cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   dim3 grid((max_q + 63) / 64, p.nh, batch);
-  fa_fwd_kernel<D><<<grid, 128, smem, st>>>(p);
+  kernel<<<grid, 128, smem, st>>>(p);
   return (int)cudaGetLastError();
 }
 
@@ -598,13 +604,16 @@ MSRL_API int msrl_flash_attn_varlen_fwd(const void* q, const void* k, const void
                                         const long long* layouts12, void* o, long long o_stride_t,
                                         float* lse, const int* cu_q, const int* cu_k, int batch,
                                         int max_q, int nh, int nkv, long long Tq, int D,
-                                        float scale, int causal, int window, cudaStream_t st) {
+                                        float scale, int causal, int window, float softcap, const void* gate,
+                                        long long gate_ld, const float* sink, cudaStream_t st) {
   if (batch == 0 || Tq == 0) return 0;
   if (nh % nkv != 0 || (window > 0 && !causal)) return (int)cudaErrorInvalidValue;
   AttnParams p = make_params(q, k, v, layouts12, o, o_stride_t, lse, cu_q, cu_k, nh, nkv, Tq, D, causal);
   p.scale = scale;
   p.scale_log2 = scale * kLog2e;
   p.window = window;
+  p.softcap = softcap;
+  p.tail = {(const __nv_bfloat16*)gate, gate_ld, sink};
   if (D == 128) return launch_fwd<128>(p, batch, max_q, st);
   if (D == 64) return launch_fwd<64>(p, batch, max_q, st);
   return (int)cudaErrorInvalidValue;

@@ -2,8 +2,10 @@
 // tensor-core kernels do not: true 32-bit products and unusual head sizes.
 //
 //   attn_simt     packed sequences, causal (bottom-right aligned), grouped heads, optional window
-//   decode_simt   one query per sequence over paged keys and values
-#include "dtype_utils.cuh"
+//   decode_simt   one query per sequence over paged keys and values, optional window or chunk
+//
+// Both take a soft cap on the scores, a sink and a gate per head (head_tail.cuh).
+#include "head_tail.cuh"
 
 namespace msrl {
 
@@ -16,7 +18,8 @@ struct SimtArgs {
   int dq, dv;
   int rep, window;                       // query heads per key head; keys a query sees (0: all)
   const int *cu_q, *cu_k;
-  float scale;
+  float scale, softcap;                  // softcap 0: not capped
+  HeadTail<T> tail;
   T* out;                                // [tokens, H * o_stride]
   long long o_ld;
   int o_stride;
@@ -70,7 +73,9 @@ __global__ void __launch_bounds__(256) attn_simt_kernel(const SimtArgs<T> p) {
     for (int j = 0; j < 4; ++j) {
       const int key = kb + part + 8 * j;
       const int back = m0 + row + off - key;
-      s[j] = key < klen && back >= 0 && back < window ? s[j] * p.scale : -INFINITY;
+      s[j] *= p.scale;
+      if (p.softcap > 0.f) s[j] = softcapped(s[j], p.softcap);
+      s[j] = key < klen && back >= 0 && back < window ? s[j] : -INFINITY;
       mx = fmaxf(mx, s[j]);
     }
 #pragma unroll
@@ -101,7 +106,7 @@ __global__ void __launch_bounds__(256) attn_simt_kernel(const SimtArgs<T> p) {
     }
   }
   if (m0 + row < qlen) {
-    const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+    const float inv = p.tail.scale(q0 + m0 + row, h, m_run, l_run);
 #pragma unroll
     for (int i = 0; i < ACC; ++i) {
       const int c = part + 8 * i;
@@ -118,8 +123,9 @@ struct PagedSimtArgs {
   const T *k, *v;                        // [blocks, block_size, G, qp] and [.., vp]
   const int *block_tables, *context_lens;
   T* out;                                // [B, H * vp]
-  int H, G, qp, vp, block_size, max_blocks, window, q_stride;
-  float scale;
+  int H, G, qp, vp, block_size, max_blocks, window, q_stride, chunk;      // chunk > 0: keys of the query's chunk
+  float scale, softcap;
+  HeadTail<T> tail;
 };
 
 constexpr int PS_ACC = 4;                // value columns per thread: vp <= 512
@@ -131,7 +137,7 @@ __global__ void __launch_bounds__(128) paged_decode_simt_kernel(const PagedSimtA
   __shared__ long long sRow[32];
   const int h = blockIdx.x, b = blockIdx.y, hk = h / (p.H / p.G);
   const int n = p.context_lens[b];
-  const int first = p.window > 0 ? max(n - p.window, 0) : 0;
+  const int first = p.chunk > 0 ? max(n - 1, 0) / p.chunk * p.chunk : p.window > 0 ? max(n - p.window, 0) : 0;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int c = threadIdx.x; c < p.qp; c += 128) sQ[c] = ldf(p.q + (long long)b * p.q_ld + h * p.q_stride + c);
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
@@ -148,6 +154,7 @@ __global__ void __launch_bounds__(128) paged_decode_simt_kernel(const PagedSimtA
         s = 0.f;
         for (int c = lane; c < p.qp; c += 32) s += sQ[c] * ldf(p.k + row * p.qp + c);
         s = warp_sum(s) * p.scale;
+        if (p.softcap > 0.f) s = softcapped(s, p.softcap);
       }
       if (lane == 0) {
         sS[j] = s;
@@ -173,7 +180,7 @@ __global__ void __launch_bounds__(128) paged_decode_simt_kernel(const PagedSimtA
       }
     }
   }
-  const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+  const float inv = p.tail.scale(b, h, m_run, l_run);
 #pragma unroll
   for (int i = 0; i < PS_ACC; ++i) {
     const int c = threadIdx.x + 128 * i;
@@ -188,7 +195,8 @@ using namespace msrl;
 // lds: q, k, v, out row strides; ints: q, k, v, out head strides, dq, dv, query heads per key head, window (0: all)
 MSRL_API int msrl_attn_simt(const void* q, const void* k, const void* v, void* out, const long long* lds,
                             const int* ints, const int* cu_q, const int* cu_k, int batch, int max_q, int H, float scale,
-                            int is_f32, cudaStream_t st) {
+                            float softcap, const void* gate, long long gate_ld, const float* sink, int is_f32,
+                            cudaStream_t st) {
   if (batch == 0 || max_q == 0) return 0;
   const int dq = ints[4], dv = ints[5];
   if (dv > 512 || batch > 65535 || H > 65535) return (int)cudaErrorNotSupported;
@@ -197,7 +205,7 @@ MSRL_API int msrl_attn_simt(const void* q, const void* k, const void* v, void* o
   auto run = [&](auto tag) {
     using T = decltype(tag);
     SimtArgs<T> p{(const T*)q, (const T*)k, (const T*)v, lds[0], lds[1], lds[2], ints[0], ints[1], ints[2],
-                  dq, dv, ints[6], ints[7], cu_q, cu_k, scale, (T*)out, lds[3], ints[3]};
+                  dq, dv, ints[6], ints[7], cu_q, cu_k, scale, softcap, {(const T*)gate, gate_ld, sink}, (T*)out, lds[3], ints[3]};
     const dim3 grid((unsigned)((max_q + SB - 1) / SB), (unsigned)H, (unsigned)batch);
     auto go = [&](auto kernel) {
       cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -213,16 +221,16 @@ MSRL_API int msrl_attn_simt(const void* q, const void* k, const void* v, void* o
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
-// ints: H, G, qp, vp, block size, block-table width, window (0: all), query head stride
+// ints: H, G, qp, vp, block size, block-table width, window (0: all), query head stride, chunk (0: none)
 MSRL_API int msrl_paged_decode_simt(const void* q, long long q_ld, const void* k, const void* v, const int* block_tables,
-                                    const int* context_lens, void* out, const int* ints, int batch, float scale, int is_f32,
-                                    cudaStream_t st) {
+                                    const int* context_lens, void* out, const int* ints, int batch, float scale, float softcap,
+                                    const void* gate, long long gate_ld, const float* sink, int is_f32, cudaStream_t st) {
   if (batch == 0) return 0;
   if (ints[3] > 128 * PS_ACC || ints[2] > 8192 || batch > 65535) return (int)cudaErrorNotSupported;
   auto run = [&](auto tag) {
     using T = decltype(tag);
     PagedSimtArgs<T> p{(const T*)q, q_ld, (const T*)k, (const T*)v, block_tables, context_lens, (T*)out, ints[0], ints[1],
-                       ints[2], ints[3], ints[4], ints[5], ints[6], ints[7], scale};
+                       ints[2], ints[3], ints[4], ints[5], ints[6], ints[7], ints[8], scale, softcap, {(const T*)gate, gate_ld, sink}};
     paged_decode_simt_kernel<T><<<dim3((unsigned)p.H, (unsigned)batch), 128, p.qp * sizeof(float), st>>>(p);
     return (int)cudaGetLastError();
   };

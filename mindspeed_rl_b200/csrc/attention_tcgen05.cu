@@ -21,6 +21,7 @@
 
 #include <cstdlib>
 
+#include "head_tail.cuh"
 #include "tcgen05_utils.cuh"
 
 namespace msrl {
@@ -53,6 +54,8 @@ struct Params {
   float scale_log2;
   int causal;
   int window;                                          // keys a query sees, itself included (0: all)
+  float softcap;                                       // cap of the scaled scores (forward with CAP)
+  HeadTail<__nv_bfloat16> tail;
   int q_col0, q_group_stride, q_hpg, q_head_stride;    // column of head h inside a row of the Q tensor map
   int k_col0, k_group_stride, k_hpg, k_head_stride;
   int v_col0, v_group_stride, v_hpg, v_head_stride;
@@ -66,8 +69,9 @@ __device__ __forceinline__ int head_col(int col0, int gs, int hpg, int hs, int h
 // BN = keys per tile.  128: one CTA per SM (192 KiB of shared memory, 512 TMEM columns).  64: two
 // CTAs per SM (112 KiB, 256 columns each), so that one CTA's soft-max, prologue and epilogue overlap
 // the other's tensor work.  NQK = 64-column halves of a query / key head: 2, or 3 for the 192-wide heads of latent
-// attention (128 unrotated + 64 rotated entries, values 128), then one CTA per SM.
-template <int BN, int NQK>
+// attention (128 unrotated + 64 rotated entries, values 128), then one CTA per SM.  CAP: soft-capped scores; the cap is
+// monotone, so running maxima are those of the raw scores.
+template <int BN, int NQK, bool CAP>
 __global__ void __launch_bounds__(THREADS, BN == 128 || NQK == 3 ? 1 : 2)
 fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                       const __grid_constant__ CUtensorMap map_v, const __grid_constant__ Params p) {
@@ -215,6 +219,7 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     unsigned char* sp = smem + SMEM_P + ((wg * HALF) >> 6) * TILE_HALF;   // the 64-column half tile of P
     constexpr int NCHUNK = HALF / 8;
     const int chunk0 = ((wg * HALF) & 63) >> 3;
+    const SoftCap2 cap(CAP ? p.softcap : 1.f);
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       const int sb = j & 1;
@@ -267,7 +272,8 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_free[sb]);              // the score buffer may be overwritten
-      const float mx = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * p.scale_log2;   // scale > 0
+      float mx = fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3)) * p.scale_log2;   // scale > 0
+      if (CAP && mx != -INFINITY) mx = cap(mx);
       // The running maximum follows the row maximum lazily: it moves only when the row maximum
       // passed it by more than 8 (a factor 256, harmless in fp32 sums and bf16 P), so that O is
       // rescaled in TMEM on few tiles only.
@@ -276,8 +282,26 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       const float m_use = (m_new == -INFINITY) ? 0.f : m_new;
       const float corr = exp2f(m_run - m_use);
       float sum0 = 0.f, sum1 = 0.f, sum2 = 0.f, sum3 = 0.f;
+      if constexpr (CAP) {
+#pragma unroll
+        for (int i = 0; i < HALF; ++i) {
+          const float v = cap(s[i] * p.scale_log2);
+          s[i] = need_mask && s[i] == -INFINITY ? -INFINITY : v;
+        }
+      }
 #pragma unroll
       for (int i = 0; i < HALF; i += 4) {
+        if constexpr (CAP) {
+          s[i] = exp2f(s[i] - m_use);
+          s[i + 1] = exp2f(s[i + 1] - m_use);
+          s[i + 2] = exp2f(s[i + 2] - m_use);
+          s[i + 3] = exp2f(s[i + 3] - m_use);
+          sum0 += s[i];
+          sum1 += s[i + 1];
+          sum2 += s[i + 2];
+          sum3 += s[i + 3];
+          continue;
+        }
         s[i] = exp2f(fmaf(s[i], p.scale_log2, -m_use));
         s[i + 1] = exp2f(fmaf(s[i + 1], p.scale_log2, -m_use));
         s[i + 2] = exp2f(fmaf(s[i + 2], p.scale_log2, -m_use));
@@ -322,7 +346,7 @@ fa_fwd_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     if (ok) {
       fence_after();
       const float l_row = l_part[0][row] + l_part[1][row];
-      const float inv_l = l_row > 0.f ? 1.f / l_row : 0.f;
+      const float inv_l = grow < qlen ? p.tail.scale2(q0 + grow, h, m_run, l_row) : 0.f;
       // O: 32 rows x 64 columns through this warp's patch (all tiles are consumed: any stage is free)
       unsigned char* patch = smem + warp * (32 * OUT_PITCH);
 #pragma unroll
@@ -882,7 +906,8 @@ MSRL_API int msrl_flash_attn_varlen_fwd_tcgen05(const void* q, const void* k, co
                                                 const long long* lay, void* o, long long o_stride_t,
                                                 float* lse, const int* cu_q, const int* cu_k, int batch,
                                                 int max_q, int nh, int nkv, long long Tq, long long Tk,
-                                                int D, float scale, int causal, int window, int* error,
+                                                int D, float scale, int causal, int window, float softcap,
+                                                const void* gate, long long gate_ld, const float* sink, int* error,
                                                 cudaStream_t st) {
   if (batch == 0 || Tq == 0) return 0;
   if (window > 0 && !causal) return (int)cudaErrorInvalidValue;
@@ -915,18 +940,22 @@ MSRL_API int msrl_flash_attn_varlen_fwd_tcgen05(const void* q, const void* k, co
   p.scale_log2 = scale * 1.4426950408889634f;
   p.causal = causal;
   p.window = window;
+  p.softcap = softcap;
+  p.tail = {(const __nv_bfloat16*)gate, gate_ld, sink};
   p.q_col0 = 0; p.q_group_stride = (int)lay[1]; p.q_hpg = (int)lay[2]; p.q_head_stride = (int)lay[3];
   p.k_col0 = 0; p.k_group_stride = (int)lay[5]; p.k_hpg = (int)lay[6]; p.k_head_stride = (int)lay[7];
   p.v_col0 = 0; p.v_group_stride = (int)lay[9]; p.v_hpg = (int)lay[10]; p.v_head_stride = (int)lay[11];
   p.error = error;
-  static bool attr_set[2] = {false, false};
+  static bool attr_set[2][2] = {{false, false}, {false, false}};
+  const bool capped = softcap > 0.f;
   const int smem = (int)fa5::fwd_smem_bytes(kt, nqk) + (kt == 64 && nqk == 2 ? 896 : 1024);   // 64, 2: two CTAs in 228 KiB
-  auto* kernel = nqk == 3 ? fa5::fa_fwd_tcgen05_kernel<64, 3>
-                          : bn == 128 ? fa5::fa_fwd_tcgen05_kernel<128, 2> : fa5::fa_fwd_tcgen05_kernel<64, 2>;
-  if (!attr_set[nqk - 2]) {
+  auto* kernel = nqk == 3 ? (capped ? fa5::fa_fwd_tcgen05_kernel<64, 3, true> : fa5::fa_fwd_tcgen05_kernel<64, 3, false>)
+                 : bn == 128 ? (capped ? fa5::fa_fwd_tcgen05_kernel<128, 2, true> : fa5::fa_fwd_tcgen05_kernel<128, 2, false>)
+                             : (capped ? fa5::fa_fwd_tcgen05_kernel<64, 2, true> : fa5::fa_fwd_tcgen05_kernel<64, 2, false>);
+  if (!attr_set[nqk - 2][capped]) {
     const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
-    attr_set[nqk - 2] = true;
+    attr_set[nqk - 2][capped] = true;
   }
   dim3 grid((max_q + fa5::BM - 1) / fa5::BM, nh, batch);
   kernel<<<grid, fa5::THREADS, smem, st>>>(mq, mk, mv, p);

@@ -32,7 +32,7 @@ NVCC_FLAGS = [
 # kernels whose results are specified in 32-bit (an fp32 residual, recurrent state, fp32 attention): compiled
 # without the approximate divisions, square roots, exponentials and flush-to-zero of --use_fast_math
 PRECISE = {"residual_stream", "delta_rule", "latent_attention", "latent_decode_tcgen05", "grouped_gemm_simt",
-           "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "attention_simt",
+           "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "conv_qkv", "attention_simt",
            "moe"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
@@ -43,6 +43,7 @@ _STREAM = ("residual_stream", "grouped_gemm_simt", "moe", "moe_gemm_tcgen05", "a
            "paged_rows", "gemm2cta_tcgen05")
 GROUPS = {
     "pumotar": (*_STREAM, "delta_rule", "latent_attention", "latent_decode_tcgen05"),
+    "gapevik": (*_STREAM, "delta_rule", "latent_attention", "latent_decode_tcgen05", "conv_qkv", "decode", "decode_prefix_tcgen05"),
     "sunatar": (*_STREAM, "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "decode", "decode_prefix_tcgen05"),
 }
 

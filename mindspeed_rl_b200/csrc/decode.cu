@@ -8,6 +8,7 @@
 //
 // These replace the rollout engine the reference imports (vLLM paged attention + sampler;
 // mindspeed_rl/models/rollout/vllm_engine.py:222-250,423-504).
+#include "head_tail.cuh"
 #include "mma_utils.cuh"
 
 namespace msrl {
@@ -91,6 +92,9 @@ struct DecodeParams {
   int npre;                 // prefix splits (slots 0 .. npre-1)
   int block_shift;          // log2(block_size), or -1 when it is not a power of two
   int window;               // keys a query sees, itself included (0: all)
+  int chunk;                // > 0: the keys of the query's chunk
+  float softcap;            // cap of the scaled scores (0: none)
+  HeadTail<__nv_bfloat16> tail;
 };
 
 constexpr int kGroupMax = 8;
@@ -113,7 +117,8 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p)
   const int frow = lane >> 2, fcol = (lane & 3) * 2;
 
   const int k0 = (p.key_start != nullptr) ? min(p.key_start[b], ctx)
-                                               : (p.window > 0 ? max(ctx - p.window, 0) : 0);
+                     : p.chunk > 0 ? max(ctx - 1, 0) / p.chunk * p.chunk
+                                   : (p.window > 0 ? max(ctx - p.window, 0) : 0);
   int per_split = (ctx - k0 + p.nsplit - 1) / p.nsplit;
   per_split = ((per_split + CH - 1) / CH) * CH;
   const int kbeg = k0 + sp * per_split;
@@ -185,9 +190,20 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p)
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
+      for (int j = 0; j < 4; ++j) s[nt][j] *= p.scale_log2;
+    if (p.softcap > 0.f) {
+      const SoftCap2 cap(p.softcap);
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) s[nt][j] = cap(s[nt][j]);
+    }
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int key = key0 + nt * 8 + fcol + (j & 1);
-        const float v = (key < kend) ? s[nt][j] * p.scale_log2 : -INFINITY;
+        const float v = (key < kend) ? s[nt][j] : -INFINITY;
         s[nt][j] = v;
         mx[j >> 1] = fmaxf(mx[j >> 1], v);
       }
@@ -275,7 +291,7 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const DecodeParams p)
     const int h = h0 + r;
     if (p.slot_total == 1) {
       p.out[(long long)b * p.out_stride + (long long)h * DV + d] =
-          __float2bfloat16(l > 0.f ? o / l : 0.f);
+          __float2bfloat16(o * p.tail.scale2(b, h, m, l));
     } else {
       const long long pi = ((long long)b * p.nh + h) * p.slot_total + p.slot_base + sp;
       p.part_o[pi * DV + d] = o;
@@ -509,11 +525,12 @@ __global__ void paged_decode_merge_kernel(const DecodeParams p, int B) {
   for (int s = 0; s < ns; ++s) l += ml[2 * s + 1] * exp2f(ml[2 * s] - mu);
   const long long b = gw / p.nh;
   const int h = (int)(gw % p.nh);
+  const float inv = p.tail.scale2(b, h, m, l);
   for (int d = lane; d < D; d += 32) {
     float o = 0.f;
     for (int s = 0; s < ns; ++s)
       o += p.part_o[(gw * ns + s) * D + d] * exp2f(ml[2 * s] - mu);
-    p.out[b * p.out_stride + (long long)h * D + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
+    p.out[b * p.out_stride + (long long)h * D + d] = __float2bfloat16(o * inv);
   }
 }
 
@@ -980,12 +997,13 @@ static int launch_window_decode(const DecodeParams& p, int B, cudaStream_t st) {
   return (int)cudaGetLastError();
 }
 
-// One query per sequence over the last `window` (0: all) cached keys: k_cache [blocks, block_size, nkv, dk], v_cache
+// One query per sequence over the last `window` (0: all) cached keys, or those of its `chunk`: k_cache [blocks, block_size, nkv, dk], v_cache
 // [.., dv], any group size, explicit scale.  part_o [B, nh, nsplit, dv] and part_ml [B, nh, nsplit, 2]: scratch.
 MSRL_API int msrl_paged_decode_window(const void* q, const long long* q_layout4, const void* k_cache, const void* v_cache,
                                       const int* block_tables, int max_blocks, const int* context_lens, void* out,
                                       long long out_stride, float* part_o, float* part_ml, int B, int nh, int nkv, int dk,
-                                      int dv, int block_size, float scale, int window, int nsplit, cudaStream_t st) {
+                                      int dv, int block_size, float scale, int window, int chunk, float softcap, const void* gate,
+                                      long long gate_ld, const float* sink, int nsplit, cudaStream_t st) {
   if (B == 0) return 0;
   if (nh % nkv != 0 || nsplit < 1 || nsplit > 65535) return (int)cudaErrorInvalidValue;
   DecodeParams p{};
@@ -1008,6 +1026,9 @@ MSRL_API int msrl_paged_decode_window(const void* q, const long long* q_layout4,
   p.nsplit = nsplit;
   p.scale_log2 = scale * kLog2eD;
   p.window = window;
+  p.chunk = chunk;
+  p.softcap = softcap;
+  p.tail = {(const __nv_bfloat16*)gate, gate_ld, sink};
   if (dk == 128 && dv == 128) return launch_window_decode<128, 128>(p, B, st);
   if (dk == 64 && dv == 64) return launch_window_decode<64, 64>(p, B, st);
   if (dk == 192 && dv == 128) return launch_window_decode<192, 128>(p, B, st);

@@ -1,17 +1,15 @@
-// Gated delta rule with a decay per key channel, for prompts (prefill portions) and single-token decode steps.
+// Gated delta rule with a decay per key channel or per head, for prompts (prefill portions) and single-token decode steps.
 //
 // Per value head h, with key head hk = h / (H / KVH), state S [dim, vdim] in fp32:
 //
 //   q, k, v = silu(causal conv over time of the projections)          (last tap = current token)
 //   q = q / |q| * dim^-1/2,  k = k / |k|                              (|x| = sqrt(sum x^2 + unit_eps))
-//   g = exp(-exp(A_log[h]) * softplus(a + dt_bias))   [dim],   beta = sigmoid(b)
+//   g = exp(-exp(A_log[h]) * softplus(a + dt_bias))   [dim] or one per head,   beta = sigmoid(b)
 //   S <- g * S;  u = beta * (v - S^T k);  S <- S + k u^T;  o = S^T q
-//   y = o / rms(o) * norm * sigmoid(gate)
+//   y = o / rms(o) * norm * (sigmoid or silu)(gate)
 //
-// What a sequence carries from step to step lives in a state slot: S, and a ring of the last `taps` inputs of
-// the short convolutions (entry p % taps holds the projections of position p).  With `taps` entries, one more
-// than the next token needs, the entry a step writes is never one that the same step reads.  Positions
-// before the sequence's start count as zero, so a slot needs no clearing when it is used again.
+// What a sequence carries from step to step lives in a state slot: S, and the ring of the short convolutions
+// (short_conv.cuh).
 //
 //   prefill: `prep` (conv, silu, unit norms, decays, step sizes of every token), `scan` (the recurrence: one
 //            block per sequence, head and column group; S in registers, LPC lanes share a column) and
@@ -20,59 +18,32 @@
 //   decode:  one fused kernel per (sequence, head): all of the above with S read and written once, coalesced.
 //
 // Both sum (S^T k, S^T q) over the decayed state in one pass: o = (gS)^T q + (k.q) u.
-#include "dtype_utils.cuh"
+#include "short_conv.cuh"
 
 namespace msrl {
 
 template <typename T>
-struct DeltaIn {
-  const T* proj;             // [tokens, ld]: q | k | v | b ... sections at the given columns
-  long long ld;
+struct DeltaIn : ConvIn<T> { // proj: q | k | v | b ... sections at the given columns
   int q_col, k_col, v_col, b_col;
-  const T* a;                // [tokens, H * dim] decay projection
+  const T* a;                // decay projection, [tokens, H * dim] (a_h = dim, a_d = 1) or [tokens, H] (a_h = 1, a_d = 0)
   long long a_ld;
-  const float* conv;         // [2 * KVH * dim + H * vdim, taps]
-  int taps;
+  int a_h, a_d;
+  int silu_gate;
   const float* a_log;        // [H]
-  const float* dt_bias;      // [H * dim]
-  T* ring;                   // [slots, taps, channels]
+  const float* dt_bias;      // like a row of a
   float* state;              // [slots, H, dim, vdim]
   int H, KVH, dim, vdim;
   float unit_eps;
+  __device__ __forceinline__ float decay(long long t, int h, int d) const {
+    const int c = h * a_h + d * a_d;
+    return expf(-expf(a_log[h]) * softplus_f(ldf(a + t * a_ld + c) + dt_bias[c]));
+  }
+  __device__ __forceinline__ float gate_of(float z) const { return silu_gate ? z * sigmoid_f(z) : sigmoid_f(z); }
 };
 
-// silu of the short convolution for one channel: `col` is its column in proj, `ch` its ring / weight row,
-// `i` the token's index inside this portion (row t of proj), `pos` its position in the sequence.  TAPS > 0 fixes
-// the number of taps so that all loads are in flight together.
 template <int TAPS, typename T>
-__device__ __forceinline__ float conv_silu(const DeltaIn<T>& p, long long t, int i, int pos, long long slot, int col,
-                                           int ch) {
-  const int channels = 2 * p.KVH * p.dim + p.H * p.vdim;
-  const int taps = TAPS > 0 ? TAPS : p.taps;
-  const T* ring = p.ring + slot * taps * channels + ch;
-  float s = 0.f;
-  if constexpr (TAPS > 0) {
-    float x[TAPS], w[TAPS];
-    const int at = pos % TAPS;
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) {
-      const int back = TAPS - 1 - j;
-      const int entry = at - back < 0 ? at - back + TAPS : at - back;
-      x[j] = 0.f;
-      if (pos - back >= 0)
-        x[j] = ldf(i - back >= 0 ? p.proj + (t - back) * p.ld + col : ring + (long long)entry * channels);
-      w[j] = p.conv[(long long)ch * TAPS + j];
-    }
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) s += x[j] * w[j];
-  } else {
-    for (int j = 0; j < taps; ++j) {
-      const int back = taps - 1 - j;
-      if (pos - back < 0) continue;
-      s += ldf(i - back >= 0 ? p.proj + (t - back) * p.ld + col : ring + (long long)((pos - back) % taps) * channels) *
-           p.conv[(long long)ch * taps + j];
-    }
-  }
+__device__ __forceinline__ float conv_silu(const DeltaIn<T>& p, long long t, int i, int pos, long long slot, int col, int ch) {
+  const float s = conv_one<TAPS>(static_cast<const ConvIn<T>&>(p), t, i, pos, slot, col, ch);
   return s * sigmoid_t<T>(s);
 }
 
@@ -122,7 +93,7 @@ delta_prep_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const i
   for (int c = threadIdx.x; c < nv; c += 256) vv[t * nv + c] = conv_silu<0>(p, t, i, pos, slot, p.v_col + c, 2 * kd + c);
   const int ng = p.H * p.dim;
   for (int c = threadIdx.x; c < ng; c += 256)
-    g[t * ng + c] = expf(-expf(p.a_log[c / p.dim]) * softplus_f(ldf(p.a + t * p.a_ld + c) + p.dt_bias[c]));
+    g[t * ng + c] = p.decay(t, c / p.dim, c % p.dim);
   for (int h = threadIdx.x; h < p.H; h += 256) beta[t * p.H + h] = sigmoid_f(ldf(p.proj + t * p.ld + p.b_col + h));
 }
 
@@ -130,43 +101,11 @@ delta_prep_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const i
 // consecutive tokens with the convolution window of its channels in registers, four channels per lane.
 constexpr int PREP_TT = 16;
 
-template <int TAPS, typename T>
-struct ConvWindow {
-  float w[TAPS][4], x[TAPS][4];
-  const T* src;
-  __device__ __forceinline__ void weights(const float* conv, int ch) {
+template <typename T>
+__device__ __forceinline__ void silu4(float (&y)[4]) {
 #pragma unroll
-    for (int c = 0; c < 4; ++c)
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j) w[j][c] = conv[(long long)(ch + c) * TAPS + j];
-  }
-  // window entries before token t (index i of its portion, position pos); x[TAPS - 1] is the token's own
-  __device__ __forceinline__ void fill(const DeltaIn<T>& p, long long t, int i, int pos, long long slot, int col, int ch) {
-    const int channels = 2 * p.KVH * p.dim + p.H * p.vdim;
-#pragma unroll
-    for (int j = 0; j + 1 < TAPS; ++j) {
-      const int back = TAPS - 1 - j;            // shifted once more before use: entry j + 1 holds position pos - back
-#pragma unroll
-      for (int c = 0; c < 4; ++c) x[j + 1][c] = 0.f;
-      if (pos - back >= 0) {
-        if (i - back >= 0) ldf4(p.proj + (t - back) * p.ld + col, x[j + 1]);
-        else ldf4(p.ring + (slot * TAPS + (pos - back) % TAPS) * channels + ch, x[j + 1]);
-      }
-    }
-  }
-  __device__ __forceinline__ void step(const float (&in)[4], float (&y)[4]) {
-#pragma unroll
-    for (int c = 0; c < 4; ++c) {
-#pragma unroll
-      for (int j = 0; j + 1 < TAPS; ++j) x[j][c] = x[j + 1][c];
-      x[TAPS - 1][c] = in[c];
-      float s = 0.f;
-#pragma unroll
-      for (int j = 0; j < TAPS; ++j) s += x[j][c] * w[j][c];
-      y[c] = s * sigmoid_t<T>(s);
-    }
-  }
-};
+  for (int c = 0; c < 4; ++c) y[c] *= sigmoid_t<T>(y[c]);
+}
 
 constexpr int PREP_U = 4;       // tokens whose projections are loaded together
 
@@ -202,6 +141,7 @@ delta_value_kernel(const DeltaIn<T> p, const int* tok_seq, const int* cu, const 
       }
       float y[4];
       cv.step(rv[x], y);
+      silu4<T>(y);
       stf4(vv + (long long)t * nv + c, y);
     }
   }
@@ -222,7 +162,7 @@ constexpr int GRP = 4, COEF = 24;
 
 __host__ __device__ constexpr int group_floats(int dp) { return 13 * dp + COEF; }
 
-template <typename T, int TAPS>
+template <typename T, int TAPS, bool HEAD>        // HEAD: one decay per head
 __global__ void __launch_bounds__(256, 2)
 delta_group_kernel(const DeltaIn<T> p, const int* cu, const int* start_pos, const long long* slots, int batch,
                    int total_slots, int DP, float* rec) {
@@ -240,7 +180,7 @@ delta_group_kernel(const DeltaIn<T> p, const int* cu, const int* start_pos, cons
     cq.weights(p.conv, ch);
     ck.weights(p.conv, kd + ch);
 #pragma unroll
-    for (int c = 0; c < 4; ++c) bias[c] = p.dt_bias[h * p.dim + d + c];
+    for (int c = 0; c < 4; ++c) bias[c] = p.dt_bias[HEAD ? h : h * p.dim + d + c];
   }
   const int s0 = blockIdx.y * 4, s1 = min(total_slots, s0 + 4);
   int last_b = -1;
@@ -266,7 +206,8 @@ delta_group_kernel(const DeltaIn<T> p, const int* cu, const int* start_pos, cons
       if (on) {
         ldf4(p.proj + t * p.ld + p.q_col + ch, q[j]);
         ldf4(p.proj + t * p.ld + p.k_col + ch, k[j]);
-        ldf4(p.a + t * p.a_ld + h * p.dim + d, g[j]);
+        if constexpr (HEAD) g[j][0] = ldf(p.a + t * p.a_ld + h);
+        else ldf4(p.a + t * p.a_ld + h * p.dim + d, g[j]);
       }
     }
     if (on && b != last_b) {
@@ -284,9 +225,11 @@ delta_group_kernel(const DeltaIn<T> p, const int* cu, const int* start_pos, cons
       if (on && j < cnt) {
         cq.step(q[j], q[j]);
         ck.step(k[j], k[j]);
+        silu4<T>(q[j]);
+        silu4<T>(k[j]);
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          g[j][c] = expf(rate * softplus_f(g[j][c] + bias[c]));
+          g[j][c] = HEAD && c > 0 ? g[j][0] : expf(rate * softplus_f(g[j][c] + bias[c]));
           v[2 * j] += q[j][c] * q[j][c];
           v[2 * j + 1] += k[j][c] * k[j][c];
         }
@@ -728,25 +671,10 @@ delta_group_scan_kernel(const float* rec, const float* vv, float* state, const i
     }
 }
 
-// ---- prefill: the last inputs of the convolutions ------------------------------------------------------
-template <typename T>
-__global__ void delta_ring_kernel(const DeltaIn<T> p, const int* cu, const int* start_pos, const long long* slots) {
-  const int b = blockIdx.y;
-  const int kd = p.KVH * p.dim, channels = 2 * kd + p.H * p.vdim;
-  const int len = cu[b + 1] - cu[b];
-  const int ch = blockIdx.x * blockDim.x + threadIdx.x;
-  if (ch >= channels) return;
-  const int col = ch < kd ? p.q_col + ch : ch < 2 * kd ? p.k_col + ch - kd : p.v_col + ch - 2 * kd;
-  for (int i = max(0, len - p.taps); i < len; ++i) {
-    const int pos = start_pos[b] + i;
-    p.ring[(slots[b] * p.taps + pos % p.taps) * channels + ch] = p.proj[(cu[b] + i) * p.ld + col];
-  }
-}
-
 // ---- prefill: norm and gate ------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256)
-delta_out_kernel(const float* o, const T* gate, long long gate_ld, const float* norm, float eps, T* y, long long rows,
+delta_out_kernel(const DeltaIn<T> p, const float* o, const T* gate, long long gate_ld, const float* norm, float eps, T* y, long long rows,
                  int H, int vdim) {
   const long long r = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);     // (token, head)
   const int lane = threadIdx.x & 31;
@@ -758,7 +686,7 @@ delta_out_kernel(const float* o, const T* gate, long long gate_ld, const float* 
   for (int c = lane; c < vdim; c += 32) ss += x[c] * x[c];
   const float inv = 1.f / sqrtf(warp_sum(ss) / (float)vdim + eps);
   for (int c = lane; c < vdim; c += 32)
-    stf(y + r * vdim + c, x[c] * inv * norm[c] * sigmoid_f(ldf(gate + t * gate_ld + h * vdim + c)));
+    stf(y + r * vdim + c, x[c] * inv * norm[c] * p.gate_of(ldf(gate + t * gate_ld + h * vdim + c)));
 }
 
 // ---- decode: one token per sequence, everything in one kernel -----------------------------------------------
@@ -809,7 +737,7 @@ delta_decode_kernel(const DeltaIn<T> p, const T* gate, long long gate_ld, const 
     if (lead || x >= 2 * dim) ring[base + ch] = row[col];
   }
   for (int d = threadIdx.x; d < dim; d += THREADS)
-    sg[d] = expf(-expf(p.a_log[h]) * softplus_f(ldf(p.a + b * p.a_ld + h * dim + d) + p.dt_bias[h * dim + d]));
+    sg[d] = p.decay(b, h, d);
   __syncthreads();
   {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -874,14 +802,14 @@ delta_decode_kernel(const DeltaIn<T> p, const T* gate, long long gate_ld, const 
   }
   for (int c = threadIdx.x; c < vdim; c += THREADS)
     stf(y + ((long long)b * p.H + h) * vdim + c,
-        so[c] * inv * norm[c] * sigmoid_f(ldf(gate + b * gate_ld + h * vdim + c)));
+        so[c] * inv * norm[c] * p.gate_of(ldf(gate + b * gate_ld + h * vdim + c)));
 }
 
 }  // namespace msrl
 
 using namespace msrl;
 
-// ints: taps, H, KVH, dim, vdim, q_col, k_col, v_col, b_col
+// ints: taps, H, KVH, dim, vdim, q_col, k_col, v_col, b_col, one decay per head, silu gate
 template <typename T>
 static DeltaIn<T> delta_in(const void* proj, long long ld, const void* a, long long a_ld, const float* conv,
                            const float* a_log, const float* dt_bias, void* ring, float* state, const int* ints,
@@ -905,6 +833,10 @@ static DeltaIn<T> delta_in(const void* proj, long long ld, const void* a, long l
   p.k_col = ints[6];
   p.v_col = ints[7];
   p.b_col = ints[8];
+  p.a_h = ints[9] ? 1 : p.dim;
+  p.a_d = ints[9] ? 0 : 1;
+  p.silu_gate = ints[10];
+  p.channels = 2 * p.KVH * p.dim + p.H * p.vdim;
   p.unit_eps = unit_eps;
   return p;
 }
@@ -951,7 +883,7 @@ static int launch_group_scan(const float* rec, const float* vv, float* state, co
 static bool grouped_shape(const int* ints, long long ld, long long a_ld) {
   const int taps = ints[0], dim = ints[3], vdim = ints[4];
   return dim % 4 == 0 && dim <= 128 && vdim % 4 == 0 && taps >= 2 && taps <= 4 && ints[5] % 4 == 0 && ints[6] % 4 == 0 &&
-         ints[7] % 4 == 0 && ld % 4 == 0 && a_ld % 4 == 0;
+         ints[7] % 4 == 0 && ld % 4 == 0 && (ints[9] || a_ld % 4 == 0);
 }
 static int padded_dim(int dim) { return dim <= 64 ? 64 : 128; }
 
@@ -987,7 +919,8 @@ MSRL_API int msrl_delta_prefill(const void* proj, long long ld, const void* a, l
 #define MSRL_PREP(N)                                                                                       \
   do {                                                                                                     \
     delta_value_kernel<T, N><<<vgrid, 256, 0, st>>>(p, tok_seq, cu, start_pos, slots, tokens, vv);           \
-    delta_group_kernel<T, N><<<ggrid, 256, 0, st>>>(p, cu, start_pos, slots, batch, gslots, DP, rec);        \
+    if (ints[9]) delta_group_kernel<T, N, true><<<ggrid, 256, 0, st>>>(p, cu, start_pos, slots, batch, gslots, DP, rec); \
+    else delta_group_kernel<T, N, false><<<ggrid, 256, 0, st>>>(p, cu, start_pos, slots, batch, gslots, DP, rec);        \
   } while (0)
       if (p.taps == 4) MSRL_PREP(4);
       else if (p.taps == 3) MSRL_PREP(3);
@@ -1007,10 +940,10 @@ MSRL_API int msrl_delta_prefill(const void* proj, long long ld, const void* a, l
 #undef MSRL_SCAN
     }
     if (e) return e;
-    const int channels = 2 * KVH * dim + H * vdim;
-    delta_ring_kernel<T><<<dim3((unsigned)((channels + 255) / 256), (unsigned)batch), 256, 0, st>>>(p, cu, start_pos, slots);
+    conv_ring_kernel<T><<<dim3((unsigned)((p.channels + 255) / 256), (unsigned)batch), 256, 0, st>>>(
+        p, KVH * dim, KVH * dim, p.q_col, p.k_col, p.v_col, cu, start_pos, slots);
     const long long rows = (long long)tokens * H;
-    delta_out_kernel<T><<<(unsigned)((rows + 7) / 8), 256, 0, st>>>(o, (const T*)gate, gate_ld, norm, eps, (T*)y, rows, H, vdim);
+    delta_out_kernel<T><<<(unsigned)((rows + 7) / 8), 256, 0, st>>>(p, o, (const T*)gate, gate_ld, norm, eps, (T*)y, rows, H, vdim);
     return (int)cudaGetLastError();
   };
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});

@@ -5,15 +5,19 @@
 // linear, so prompts expand them per head and decode steps fold them into the query (q W_uk) and the output
 // (W_uv sum p c) and attend to the rows themselves.
 //
-//   prep        RMS norm of the latent, interleaved rotation of the shared key part and of every head's query
-//               part (fp32), cache write; the row also goes to `lat` (prompts), the rotated query part to the
-//               decode query
+//   prep        RMS norm of the latent (and of the queries' own latent, where there is one), rotation of the shared
+//               key part and of every head's query part (fp32; neighbours, or entries half a part away), cache write;
+//               the row also goes to `lat` (prompts), the rotated query part to the decode query
 //   spread      the rotated key part into every head's expanded key
 //   decode_simt one query per sequence over the paged rows, any sizes, fp32 arithmetic
 //   decode_mma  the same on the legacy tensor path for bf16 (block sizes that latent_decode_tcgen05.cu does not
 //               take): a block takes 16 / 32 / 64 heads of one sequence and a range of its keys, so that a row is
 //               read once for all of them; `combine` merges the ranges
+//
+// Decode kernels see the last `window` rows (0: all), may add exp(sink[h]) to a head's soft-max sum and may scale a head
+// by sigmoid(gate).
 #include "dtype_utils.cuh"
+#include "head_tail.cuh"
 #include "mma_utils.cuh"
 
 namespace msrl {
@@ -21,43 +25,60 @@ namespace mla {
 
 template <typename T>
 struct PrepArgs {
-  T* qkv;                      // [tokens, ld]
+  T* qkv;                      // [tokens, ld] rows with the query heads (H of them; 0: they are not there)
   long long ld;
   int H, q_stride, dn, dr;     // head h's query: columns h * q_stride + [0, dn) unrotated, then dr rotated
-  int dkv_col, rank;
+  const T* latent;             // [tokens, ld] latent and shared key part, or null: queries only
+  int rank;
   const float* norm_w;
   float eps;
   const float* table;          // [positions, rot_dims]: cos | sin
-  int rot_dims, table_rows;
+  int rot_dims, table_rows, halves;
   const int* positions;
   const long long* slots;      // cache row per token, < 0: not cached
   T* cache;
   int RP, CP;
   T* lat;                      // [tokens, CP] or null
   T* qdec;                     // [tokens, H, CP] or null: receives the rotated query part at column RP
+  int q_rank, QP, dq;          // the queries' latent lies dq columns behind `latent`
+  const float* q_norm;
+  T* cq;                       // [tokens, QP] or null: it normed, zero padded
 };
 
+// entry d of a rotated part
 template <typename T>
-__device__ __forceinline__ float rotated(const T* x, int d, const float* cs, int rot_dims) {
+__device__ __forceinline__ float rotated(const T* x, int d, const float* cs, int rot_dims, int halves) {
   if (d >= rot_dims) return ldf(x + d);
-  const int half = rot_dims / 2, i = d >> 1;
+  const int half = rot_dims / 2, i = halves ? d % half : d >> 1;
+  const bool second = halves ? d >= half : d & 1;
   const float c = cs[i], s = cs[half + i];
-  const float u = ldf(x + (d & ~1)), v = ldf(x + (d | 1));
-  return (d & 1) ? v * c + u * s : u * c - v * s;
+  const float u = ldf(x + (halves ? i : d & ~1)), v = ldf(x + (halves ? i + half : d | 1));
+  return second ? v * c + u * s : u * c - v * s;
 }
 
-// entries d .. d + 3 (d a multiple of 4) of a rotated part whose rot_dims is a multiple of 4
+// entries d .. d + 3 (d a multiple of 4) of a rotated part whose rot_dims is a multiple of 4 (of 8 with halves)
 template <typename T>
-__device__ __forceinline__ void rotated4(const T* x, int d, const float* cs, int rot_dims, float (&y)[4]) {
+__device__ __forceinline__ void rotated4(const T* x, int d, const float* cs, int rot_dims, int halves, float (&y)[4]) {
   ldf4(x + d, y);
-  if (d < rot_dims) {
-    const int half = rot_dims / 2, i = d >> 1;
+  if (d >= rot_dims) return;
+  const int half = rot_dims / 2;
+  if (halves) {
+    const bool second = d >= half;
+    const int i = second ? d - half : d;
+    float o[4], c[4], s[4];
+    ldf4(x + (second ? i : d + half), o);
+    ldf4(cs + i, c);
+    ldf4(cs + half + i, s);
 #pragma unroll
-    for (int k = 0; k < 2; ++k) {
-      const float c = cs[i + k], s = cs[half + i + k], u = y[2 * k], v = y[2 * k + 1];
-      y[2 * k] = u * c - v * s;
-      y[2 * k + 1] = v * c + u * s;
-    }
+    for (int k = 0; k < 4; ++k) y[k] = second ? y[k] * c[k] + o[k] * s[k] : y[k] * c[k] - o[k] * s[k];
+    return;
+  }
+  const int i = d >> 1;
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const float c = cs[i + k], s = cs[half + i + k], u = y[2 * k], v = y[2 * k + 1];
+    y[2 * k] = u * c - v * s;
+    y[2 * k + 1] = v * c + u * s;
   }
 }
 
@@ -67,36 +88,72 @@ __global__ void __launch_bounds__(256) prep4_kernel(const PrepArgs<T> p) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   T* row = p.qkv + t * p.ld;
-  const T* lat_in = row + p.dkv_col;
-  float ss = 0.f;
-  for (int c = threadIdx.x * 4; c < p.rank; c += 1024) {
-    float x[4];
-    ldf4(lat_in + c, x);
+  const T* lat_in = p.latent + t * p.ld;
+  float ss = 0.f, sq = 0.f;
+  if (p.latent != nullptr) {
+    for (int c = threadIdx.x * 4; c < p.rank; c += 1024) {
+      float x[4];
+      ldf4(lat_in + c, x);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) ss += x[j] * x[j];
+      for (int j = 0; j < 4; ++j) ss += x[j] * x[j];
+    }
+    if (p.cq != nullptr)
+      for (int c = threadIdx.x * 4; c < p.q_rank; c += 1024) {
+        float x[4];
+        ldf4(lat_in + p.dq + c, x);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) sq += x[j] * x[j];
+      }
   }
   const int pos = min(max(p.positions[t], 0), p.table_rows - 1);
   const float* cs = p.table + (long long)pos * p.rot_dims;
-  const long long slot = p.slots[t];
   // queries first: they do not wait for the norm
-  if (p.qdec != nullptr) {
+  if (p.H > 0 && p.qdec != nullptr) {
     const int w = (p.CP - p.RP) / 4;
     for (int i = threadIdx.x; i < p.H * w; i += 256) {
       const int h = i / w, d = (i - h * w) * 4;
       float y[4] = {0.f, 0.f, 0.f, 0.f};
-      if (d < p.dr) rotated4(row + h * p.q_stride + p.dn, d, cs, p.rot_dims, y);
+      if (d < p.dr) rotated4(row + h * p.q_stride + p.dn, d, cs, p.rot_dims, p.halves, y);
       stf4(p.qdec + (t * p.H + h) * p.CP + p.RP + d, y);
     }
-  } else {
+  } else if (p.H > 0 && p.halves) {
+    // in place: one thread owns both entries of a pair
+    const int half = p.rot_dims / 2, quads = half / 4;
+    for (int i = threadIdx.x; i < p.H * quads; i += 256) {
+      const int h = i / quads, d = (i - h * quads) * 4;
+      T* x = row + h * p.q_stride + p.dn;
+      float a[4], b[4];
+      rotated4(x, d, cs, p.rot_dims, 1, a);
+      rotated4(x, d + half, cs, p.rot_dims, 1, b);
+      stf4(x + d, a);
+      stf4(x + d + half, b);
+    }
+  } else if (p.H > 0) {
     const int quads = p.rot_dims / 4;
     for (int i = threadIdx.x; i < p.H * quads; i += 256) {
       const int h = i / quads, d = (i - h * quads) * 4;
       T* x = row + h * p.q_stride + p.dn;
       float y[4];
-      rotated4(x, d, cs, p.rot_dims, y);
+      rotated4(x, d, cs, p.rot_dims, 0, y);
       stf4(x + d, y);
     }
   }
+  if (p.latent == nullptr) return;
+  if (p.cq != nullptr) {
+    const float inv = 1.f / sqrtf(block_sum(sq, red) / (float)p.q_rank + p.eps);
+    for (int c = threadIdx.x * 4; c < p.QP; c += 1024) {
+      float y[4] = {0.f, 0.f, 0.f, 0.f};
+      if (c < p.q_rank) {
+        float w[4];
+        ldf4(lat_in + p.dq + c, y);
+        ldf4(p.q_norm + c, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] *= inv * w[j];
+      }
+      stf4(p.cq + t * p.QP + c, y);
+    }
+  }
+  const long long slot = p.slots[t];
   const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)p.rank + p.eps);
   T* crow = slot >= 0 ? p.cache + slot * p.CP : nullptr;
   T* lrow = p.lat != nullptr ? p.lat + t * p.CP : nullptr;
@@ -109,7 +166,7 @@ __global__ void __launch_bounds__(256) prep4_kernel(const PrepArgs<T> p) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) y[j] *= inv * w[j];
     } else if (c >= p.RP && c < p.RP + p.dr) {
-      rotated4(lat_in + p.rank, c - p.RP, cs, p.rot_dims, y);
+      rotated4(lat_in + p.rank, c - p.RP, cs, p.rot_dims, p.halves, y);
     }
     if (crow != nullptr) stf4(crow + c, y);
     if (lrow != nullptr) stf4(lrow + c, y);
@@ -121,41 +178,53 @@ __global__ void __launch_bounds__(256) prep_kernel(const PrepArgs<T> p) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   T* row = p.qkv + t * p.ld;
-  const T* lat_in = row + p.dkv_col;
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < p.rank; c += 256) {
-    const float x = ldf(lat_in + c);
-    ss += x * x;
-  }
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)p.rank + p.eps);
   const int pos = min(max(p.positions[t], 0), p.table_rows - 1);
   const float* cs = p.table + (long long)pos * p.rot_dims;
-  const long long slot = p.slots[t];
-  T* crow = slot >= 0 ? p.cache + slot * p.CP : nullptr;
-  T* lrow = p.lat != nullptr ? p.lat + t * p.CP : nullptr;
-  for (int c = threadIdx.x; c < p.CP; c += 256) {
-    float v = 0.f;
-    if (c < p.rank) v = ldf(lat_in + c) * inv * p.norm_w[c];
-    else if (c >= p.RP && c < p.RP + p.dr) v = rotated(lat_in + p.rank, c - p.RP, cs, p.rot_dims);
-    if (crow != nullptr) stf(crow + c, v);
-    if (lrow != nullptr) stf(lrow + c, v);
+  if (p.latent != nullptr) {
+    const T* lat_in = p.latent + t * p.ld;
+    float ss = 0.f, sq = 0.f;
+    for (int c = threadIdx.x; c < p.rank; c += 256) {
+      const float x = ldf(lat_in + c);
+      ss += x * x;
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)p.rank + p.eps);
+    const long long slot = p.slots[t];
+    T* crow = slot >= 0 ? p.cache + slot * p.CP : nullptr;
+    T* lrow = p.lat != nullptr ? p.lat + t * p.CP : nullptr;
+    for (int c = threadIdx.x; c < p.CP; c += 256) {
+      float v = 0.f;
+      if (c < p.rank) v = ldf(lat_in + c) * inv * p.norm_w[c];
+      else if (c >= p.RP && c < p.RP + p.dr) v = rotated(lat_in + p.rank, c - p.RP, cs, p.rot_dims, p.halves);
+      if (crow != nullptr) stf(crow + c, v);
+      if (lrow != nullptr) stf(lrow + c, v);
+    }
+    if (p.cq != nullptr) {
+      for (int c = threadIdx.x; c < p.q_rank; c += 256) {
+        const float x = ldf(lat_in + p.dq + c);
+        sq += x * x;
+      }
+      const float iq = 1.f / sqrtf(block_sum(sq, red) / (float)p.q_rank + p.eps);
+      for (int c = threadIdx.x; c < p.QP; c += 256)
+        stf(p.cq + t * p.QP + c, c < p.q_rank ? ldf(lat_in + p.dq + c) * iq * p.q_norm[c] : 0.f);
+    }
   }
+  if (p.H == 0) return;
   if (p.qdec != nullptr) {
     const int w = p.CP - p.RP;
     for (int i = threadIdx.x; i < p.H * w; i += 256) {
       const int h = i / w, d = i % w;
       stf(p.qdec + (t * p.H + h) * p.CP + p.RP + d,
-          d < p.dr ? rotated(row + h * p.q_stride + p.dn, d, cs, p.rot_dims) : 0.f);
+          d < p.dr ? rotated(row + h * p.q_stride + p.dn, d, cs, p.rot_dims, p.halves) : 0.f);
     }
   } else {
     // in place: one thread owns both entries of a pair
     const int half = p.rot_dims / 2;
     for (int i = threadIdx.x; i < p.H * half; i += 256) {
-      const int h = i / half, d = 2 * (i % half);
+      const int h = i / half, j = i % half, d0 = p.halves ? j : 2 * j, d1 = p.halves ? j + half : 2 * j + 1;
       T* x = row + h * p.q_stride + p.dn;
-      const float a = rotated(x, d, cs, p.rot_dims), b = rotated(x, d + 1, cs, p.rot_dims);
-      stf(x + d, a);
-      stf(x + d + 1, b);
+      const float a = rotated(x, d0, cs, p.rot_dims, p.halves), b = rotated(x, d1, cs, p.rot_dims, p.halves);
+      stf(x + d0, a);
+      stf(x + d1, b);
     }
   }
 }
@@ -185,7 +254,7 @@ constexpr int DS_ACC = 8;                // latent columns per thread: RP <= 204
 template <typename T>
 __global__ void __launch_bounds__(256)
 decode_simt_kernel(const T* q, const T* cache, const int* block_tables, int max_blocks, int block_size,
-                   const int* context_lens, float scale, int CP, int RP, T* out) {
+                   const int* context_lens, float scale, int CP, int RP, int window, const HeadTail<T> tail, T* out) {
   extern __shared__ float smf[];
   __shared__ float sS[32];
   float* sQ = smf;
@@ -199,7 +268,7 @@ decode_simt_kernel(const T* q, const T* cache, const int* block_tables, int max_
 #pragma unroll
   for (int i = 0; i < DS_ACC; ++i) acc[i] = 0.f;
   float m_run = -INFINITY, l_run = 0.f;
-  for (int kb = 0; kb < n; kb += 32) {
+  for (int kb = window > 0 ? max(n - window, 0) : 0; kb < n; kb += 32) {
     __syncthreads();
     for (int j = warp; j < 32; j += 8) {
       const int key = kb + j;
@@ -233,7 +302,7 @@ decode_simt_kernel(const T* q, const T* cache, const int* block_tables, int max_
       }
     }
   }
-  const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+  const float inv = tail.scale(b, h, m_run, l_run);
 #pragma unroll
   for (int i = 0; i < DS_ACC; ++i) {
     const int c = threadIdx.x + 256 * i;
@@ -250,6 +319,8 @@ struct MmaArgs {
   const int* context_lens;
   float scale_log2;
   int H, CP, RP, nsplit;
+  int window;                  // keys a query sees, itself included (0: all)
+  HeadTail<__nv_bfloat16> tail;
   float* part_o;               // [B, H, nsplit, RP]
   float* part_ml;              // [B, H, nsplit, 2]
   __nv_bfloat16* out;          // [B, H, RP], written directly when nsplit == 1
@@ -273,8 +344,9 @@ __global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
   const int split = blockIdx.x, h0 = blockIdx.y * HM, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = p.context_lens[b];
-  const int tiles = (n + KT - 1) / KT, per = (tiles + p.nsplit - 1) / p.nsplit;
-  const int first = split * per, last = min(tiles, first + per);
+  const int lo = p.window > 0 ? max(n - p.window, 0) : 0, tile0 = lo / KT;      // first key, its tile
+  const int tiles = (n + KT - 1) / KT, per = (tiles - tile0 + p.nsplit - 1) / p.nsplit;
+  const int first = tile0 + split * per, last = min(tiles, first + per);
   const int vecs = p.CP / 8;
   const int* bt = p.block_tables + (long long)b * p.max_blocks;
 
@@ -379,7 +451,7 @@ __global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
 #pragma unroll
       for (int i = 0; i < KPT; ++i) {
         const int k = spart + i * TPR;
-        v[i] = tile * KT + k < n ? sS[srow * LDS_S + k] * p.scale_log2 : -INFINITY;
+        v[i] = tile * KT + k < n && tile * KT + k >= lo ? sS[srow * LDS_S + k] * p.scale_log2 : -INFINITY;
         mx = fmaxf(mx, v[i]);
       }
 #pragma unroll
@@ -435,7 +507,7 @@ __global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
     __syncthreads();
   }
   if (spart == 0) {
-    sL[srow] = l_run;
+    sL[srow] = p.nsplit == 1 && h0 + srow < p.H ? p.tail.scale2(b, h0 + srow, m_run, l_run) : 0.f;
     if (p.nsplit > 1 && h0 + srow < p.H) {
       float* ml = p.part_ml + (((long long)b * p.H + h0 + srow) * p.nsplit + split) * 2;
       ml[0] = m_run;
@@ -449,7 +521,7 @@ __global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
     for (int half = 0; half < 2; ++half) {
       const int r = m * 16 + (lane >> 2) + half * 8;
       if (h0 + r >= p.H) continue;
-      const float l = sL[r], inv = l > 0.f ? 1.f / l : 0.f;
+      const float inv = sL[r];
 #pragma unroll
       for (int i = 0; i < NT; ++i) {
         const int c = col0 + i * 8 + (lane & 3) * 2;
@@ -467,7 +539,8 @@ __global__ void __launch_bounds__(256, 1) decode_mma_kernel(const MmaArgs p) {
   }
 }
 
-__global__ void combine_kernel(const float* part_o, const float* part_ml, int nsplit, int RP, __nv_bfloat16* out) {
+__global__ void combine_kernel(const float* part_o, const float* part_ml, int H, int nsplit, int RP,
+                               const HeadTail<__nv_bfloat16> tail, __nv_bfloat16* out) {
   const long long r = blockIdx.x;
   float m = -INFINITY;
   for (int s = 0; s < nsplit; ++s) m = fmaxf(m, part_ml[(r * nsplit + s) * 2]);
@@ -476,7 +549,7 @@ __global__ void combine_kernel(const float* part_o, const float* part_ml, int ns
     const float ls = part_ml[(r * nsplit + s) * 2 + 1];
     if (ls > 0.f) l += ls * exp2f(part_ml[(r * nsplit + s) * 2] - m);
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = tail.scale2(r / H, (int)(r % H), m, l);
   for (int c = threadIdx.x; c < RP; c += blockDim.x) {
     float a = 0.f;
     for (int s = 0; s < nsplit; ++s)
@@ -497,7 +570,7 @@ static int launch_mma(const MmaArgs& p, int batch, cudaStream_t st) {
   const dim3 grid((unsigned)p.nsplit, (unsigned)((p.H + HM - 1) / HM), (unsigned)batch);
   decode_mma_kernel<MT, NT, KT><<<grid, 256, smem, st>>>(p);
   if (p.nsplit > 1)
-    combine_kernel<<<(unsigned)(batch * p.H), 128, 0, st>>>(p.part_o, p.part_ml, p.nsplit, p.RP, p.out);
+    combine_kernel<<<(unsigned)(batch * p.H), 128, 0, st>>>(p.part_o, p.part_ml, p.H, p.nsplit, p.RP, p.tail, p.out);
   return (int)cudaGetLastError();
 }
 
@@ -513,35 +586,45 @@ static int pick_mma(const MmaArgs& p, int batch, cudaStream_t st) {
 
 using namespace msrl;
 
-// ints: H, q_stride, dn, dr, dkv_col, rank, rot_dims, table_rows, RP, CP
-MSRL_API int msrl_latent_prep(void* qkv, long long ld, const int* ints, const float* norm_w, float eps,
-                              const float* table, const int* positions, const long long* slots, void* cache, void* lat,
-                              void* qdec, int tokens, int is_f32, cudaStream_t st) {
+// ints: H, q_stride, dn, dr, rank, rot_dims, table_rows, RP, CP, halves, q_rank, QP, column of the queries' latent less that
+// of the latent.  Without `latent` (same row stride as qkv) only queries are rotated, with H = 0 none.
+MSRL_API int msrl_latent_prep(void* qkv, long long ld, const void* latent, const int* ints, const float* norm_w, float eps,
+                              const float* q_norm, const float* table, const int* positions, const long long* slots,
+                              void* cache, void* lat, void* cq, void* qdec, int tokens, int is_f32, cudaStream_t st) {
   if (tokens == 0) return 0;
   auto run = [&](auto tag) {
     using T = decltype(tag);
     mla::PrepArgs<T> p{};
     p.qkv = (T*)qkv;
     p.ld = ld;
+    p.latent = (const T*)latent;
     p.H = ints[0];
     p.q_stride = ints[1];
     p.dn = ints[2];
     p.dr = ints[3];
-    p.dkv_col = ints[4];
-    p.rank = ints[5];
-    p.rot_dims = ints[6];
-    p.table_rows = ints[7];
-    p.RP = ints[8];
-    p.CP = ints[9];
+    p.rank = ints[4];
+    p.rot_dims = ints[5];
+    p.table_rows = ints[6];
+    p.RP = ints[7];
+    p.CP = ints[8];
+    p.halves = ints[9];
+    p.q_rank = ints[10];
+    p.QP = ints[11];
+    p.dq = ints[12];
     p.norm_w = norm_w;
     p.eps = eps;
+    p.q_norm = q_norm;
     p.table = table;
     p.positions = positions;
     p.slots = slots;
     p.cache = (T*)cache;
     p.lat = (T*)lat;
+    p.cq = (T*)cq;
     p.qdec = (T*)qdec;
-    const bool by4 = ((p.rank | p.dr | p.dn | p.rot_dims | p.q_stride | p.dkv_col | (int)(ld & 3)) & 3) == 0;
+    bool by4 = ((p.rank | p.dr | p.dn | p.rot_dims | p.q_stride | (int)(ld & 3)) & 3) == 0 &&
+               reinterpret_cast<uintptr_t>(latent) % (4 * sizeof(T)) == 0;
+    if (p.cq != nullptr) by4 = by4 && ((p.q_rank | p.dq) & 3) == 0;
+    if (p.halves) by4 = by4 && p.rot_dims % 8 == 0;
     if (by4) mla::prep4_kernel<T><<<tokens, 256, 0, st>>>(p);
     else mla::prep_kernel<T><<<tokens, 256, 0, st>>>(p);
     return (int)cudaGetLastError();
@@ -562,18 +645,19 @@ MSRL_API int msrl_latent_spread(const void* lat, int CP, int RP, void* kv, long 
 
 MSRL_API int msrl_latent_decode_simt(const void* q, const void* cache, const int* block_tables, int max_blocks,
                                      int block_size, const int* context_lens, float scale, int batch, int H, int CP,
-                                     int RP, void* out, int is_f32, cudaStream_t st) {
+                                     int RP, int window, const void* gate, long long gate_ld, const float* sink, void* out,
+                                     int is_f32, cudaStream_t st) {
   if (batch == 0) return 0;
   if (RP > 256 * mla::DS_ACC || batch > 65535 || CP > 12000) return (int)cudaErrorNotSupported;
   const dim3 grid((unsigned)H, (unsigned)batch);
   if (is_f32)
     mla::decode_simt_kernel<float><<<grid, 256, CP * sizeof(float), st>>>((const float*)q, (const float*)cache, block_tables,
-                                                                          max_blocks, block_size, context_lens, scale, CP, RP,
-                                                                          (float*)out);
+                                                                          max_blocks, block_size, context_lens, scale, CP, RP, window,
+                                                                          HeadTail<float>{(const float*)gate, gate_ld, sink}, (float*)out);
   else
     mla::decode_simt_kernel<__nv_bfloat16><<<grid, 256, CP * sizeof(float), st>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, block_tables, max_blocks, block_size, context_lens, scale, CP,
-        RP, (__nv_bfloat16*)out);
+        RP, window, HeadTail<__nv_bfloat16>{(const __nv_bfloat16*)gate, gate_ld, sink}, (__nv_bfloat16*)out);
   return (int)cudaGetLastError();
 }
 
@@ -597,20 +681,23 @@ MSRL_API int msrl_latent_decode_nsplit(int batch, int H, int max_context) {
 
 // merge of the key ranges that msrl_latent_decode_tcgen05 leaves in part_o / part_ml
 MSRL_API int msrl_latent_decode_combine(const float* part_o, const float* part_ml, int batch, int H, int RP, int nsplit,
-                                        void* out, cudaStream_t st) {
+                                        const void* gate, long long gate_ld, const float* sink, void* out, cudaStream_t st) {
   if (batch == 0) return 0;
-  mla::combine_kernel<<<(unsigned)(batch * H), 128, 0, st>>>(part_o, part_ml, nsplit, RP, (__nv_bfloat16*)out);
+  mla::combine_kernel<<<(unsigned)(batch * H), 128, 0, st>>>(
+      part_o, part_ml, H, nsplit, RP, HeadTail<__nv_bfloat16>{(const __nv_bfloat16*)gate, gate_ld, sink}, (__nv_bfloat16*)out);
   return (int)cudaGetLastError();
 }
 
 // part_o [B, H, nsplit, RP] and part_ml [B, H, nsplit, 2] fp32 (unused when nsplit == 1)
 MSRL_API int msrl_latent_decode_mma(const void* q, const void* cache, const int* block_tables, int max_blocks,
                                     int block_size, const int* context_lens, float scale, int batch, int H, int CP,
-                                    int RP, int nsplit, float* part_o, float* part_ml, void* out, cudaStream_t st) {
+                                    int RP, int nsplit, int window, const void* gate, long long gate_ld, const float* sink,
+                                    float* part_o, float* part_ml, void* out, cudaStream_t st) {
   if (batch == 0) return 0;
   if (CP % 16 != 0 || RP % 16 != 0 || RP > 512 || batch > 65535) return (int)cudaErrorNotSupported;
   mla::MmaArgs p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, block_tables, max_blocks, block_size,
-                 context_lens, scale * 1.4426950408889634f, H, CP, RP, nsplit, part_o, part_ml, (__nv_bfloat16*)out};
+                 context_lens, scale * 1.4426950408889634f, H, CP, RP, nsplit, window,
+                 {(const __nv_bfloat16*)gate, gate_ld, sink}, part_o, part_ml, (__nv_bfloat16*)out};
   if (RP <= 128) return mla::pick_mma<2>(p, batch, st);
   if (RP <= 256) return mla::pick_mma<4>(p, batch, st);
   return mla::pick_mma<8>(p, batch, st);

@@ -22,6 +22,7 @@
 #include <cuda.h>
 #include <cudaTypedefs.h>
 
+#include "head_tail.cuh"
 #include "tcgen05_utils.cuh"
 
 namespace msrl {
@@ -41,6 +42,8 @@ struct Params {
   const int* context_lens;
   float scale_log2;
   int H, CP, RP, nsplit;
+  int window;                  // keys a query sees, itself included (0: all)
+  HeadTail<__nv_bfloat16> tail;
   int chunks;                  // chunks of a ring stage: enough for CP columns and for whole 128-latent blocks
   float* part_o;               // [B, H, nsplit, RP]
   float* part_ml;              // [B, H, nsplit, 2]
@@ -79,8 +82,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_const
   const int split = blockIdx.x, h0 = blockIdx.y * HB, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = p.context_lens[b];
-  const int all_tiles = (n + KT - 1) / KT, per = (all_tiles + p.nsplit - 1) / p.nsplit;
-  const int first = split * per, n_tiles = min(all_tiles, first + per) - first;
+  const int lo = p.window > 0 ? max(n - p.window, 0) : 0, tile0 = lo / KT;      // first key, its tile
+  const int all_tiles = (n + KT - 1) / KT, per = (all_tiles - tile0 + p.nsplit - 1) / p.nsplit;
+  const int first = tile0 + split * per, n_tiles = min(all_tiles, first + per) - first;
   const int heads = min(HB, p.H - h0);
   const long long row0 = (long long)b * p.H + h0;       // first (sequence, head) of this CTA
   bool fits;
@@ -222,7 +226,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_const
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       const int sb = j & 1;
-      const int valid = min(KT, n - (first + j) * KT);
+      const int valid = min(KT, n - (first + j) * KT), from = lo - (first + j) * KT;      // keys [from, valid) of the tile
       float s[32];
       float corr = 1.f;
       ok = ok && mbar_wait_warp(&s_full[sb], (j >> 1) & 1, p.error, ERR_S);
@@ -232,11 +236,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_const
         float mx = -INFINITY;
         tmem_ld32(tmem + lane_base + sb * KT + (wg ^ 1) * 32, t);
 #pragma unroll
-        for (int i = 0; i < 32; ++i) mx = fmaxf(mx, (wg ^ 1) * 32 + i < valid ? t[i] : -INFINITY);
+        for (int i = 0; i < 32; ++i) mx = fmaxf(mx, (wg ^ 1) * 32 + i < valid && (wg ^ 1) * 32 + i >= from ? t[i] : -INFINITY);
         tmem_ld32(tmem + lane_base + sb * KT + wg * 32, s);
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          s[i] = wg * 32 + i < valid ? s[i] : -INFINITY;
+          s[i] = wg * 32 + i < valid && wg * 32 + i >= from ? s[i] : -INFINITY;
           mx = fmaxf(mx, s[i]);
         }
         fence_before();
@@ -304,6 +308,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_const
     if (ok) ok = mbar_wait_warp(&pv_done, (n_tiles - 1) & 1, p.error, ERR_PV);
     if (scores) l_part[wg][row] = l_run;
     asm volatile("bar.sync 1, 256;\n" ::: "memory");
+    if (scores && wg == 0 && row < heads && p.nsplit == 1)
+      corr_s[row] = p.tail.scale2(b, h0 + row, m_run, l_part[0][row] + l_part[1][row]);      // its last use was before the barrier
+    asm volatile("bar.sync 1, 256;\n" ::: "memory");
     if (scores && wg == 0 && row < heads && p.nsplit > 1) {
       float* ml = p.part_ml + ((row0 + row) * p.nsplit + split) * 2;
       ml[0] = ok ? m_run : -INFINITY;
@@ -324,8 +331,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map, const __grid_const
               const int h = x * 32 + i;
               if (h < heads) {
                 if (p.nsplit == 1) {
-                  const float l = l_part[0][h] + l_part[1][h];
-                  p.out[(row0 + h) * p.RP + c] = __float2bfloat16_rn(v[i] / l);
+                  p.out[(row0 + h) * p.RP + c] = __float2bfloat16_rn(v[i] * corr_s[h]);
                 } else {
                   p.part_o[((row0 + h) * p.nsplit + split) * p.RP + c] = v[i];
                 }
@@ -393,8 +399,9 @@ using namespace msrl;
 // ranges are left in part_o / part_ml for msrl_latent_decode_combine.  Returns cudaErrorNotSupported for shapes it does not cover.
 MSRL_API int msrl_latent_decode_tcgen05(const void* q, const void* cache, long long num_blocks, const int* block_tables,
                                         int max_blocks, int block_size, const int* context_lens, float scale, int batch,
-                                        int H, int CP, int RP, int nsplit, float* part_o, float* part_ml, void* out,
-                                        int* error, cudaStream_t st) {
+                                        int H, int CP, int RP, int nsplit, int window, const void* gate, long long gate_ld,
+                                        const float* sink, float* part_o, float* part_ml, void* out, int* error,
+                                        cudaStream_t st) {
   if (batch == 0) return 0;
   if (CP % 16 != 0 || RP % 16 != 0 || RP > 512 || batch > 65535 || !(scale > 0.f) || block_size < 8 ||
       ld5::KT % block_size != 0 || (reinterpret_cast<uintptr_t>(q) & 15) != 0)
@@ -403,7 +410,7 @@ MSRL_API int msrl_latent_decode_tcgen05(const void* q, const void* cache, long l
   if (!ld5::make_map(&map, cache, num_blocks * block_size, CP, block_size)) return (int)cudaErrorNotSupported;
   const int boxes = (CP + 63) / 64, blocks = 2 * ((RP + 127) / 128);
   ld5::Params p{block_tables, max_blocks, block_size, context_lens,
-                scale * 1.4426950408889634f, H, CP, RP, nsplit, boxes > blocks ? boxes : blocks, part_o, part_ml,
+                scale * 1.4426950408889634f, H, CP, RP, nsplit, window, {(const __nv_bfloat16*)gate, gate_ld, sink}, boxes > blocks ? boxes : blocks, part_o, part_ml,
                 (__nv_bfloat16*)out, error};
   return H <= 32 ? ld5::launch<32>(map, q, p, batch, st) : ld5::launch<64>(map, q, p, batch, st);
 }

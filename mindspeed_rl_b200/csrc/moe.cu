@@ -4,9 +4,11 @@
 //             offsets, the destination row of every slot (stable: slots of an expert keep their
 //             order), the expert of every 128-row tile.  Three small kernels, no host round trip:
 //             the grouped GEMM's row count is bounded by slots + 128 * experts on the host side.
+//             Slots with an id outside the experts have no row (destination -1).
 //   permute   x[token] (optionally scaled by the slot's weight) -> rows of the expert-grouped
 //             buffer; pad rows of every segment are zeroed.
 //   route_top the experts of the largest sigmoid scores of every token, with their scores
+//   route_softmax_top  those of the largest soft-max score plus correction, with their scores
 //   combine   out[token] = sum_k w[token, k] * y[row(token, k)]   (fp32 accumulation; w optional)
 //   slot_dot  dw[token, k] = <dout[token], y[row(token, k)]>      (gradient of the combine weights)
 //
@@ -28,7 +30,8 @@ moe_plan_local_kernel(const long long* expert_of, int n_slots, int n_experts, in
   for (int i = threadIdx.x; i < warps * n_experts; i += PLAN_THREADS) sh[i] = 0;
   __syncthreads();
   const int slot = blockIdx.x * PLAN_THREADS + threadIdx.x;
-  const int e = slot < n_slots ? (int)expert_of[slot] : -1;
+  int e = slot < n_slots ? (int)expert_of[slot] : -1;
+  if (e >= n_experts) e = -1;
   const unsigned peers = __match_any_sync(0xffffffffu, e);
   const int rank_in_warp = __popc(peers & ((1u << lane) - 1u));
   if (e >= 0 && rank_in_warp == 0) sh[warp * n_experts + e] = __popc(peers);
@@ -88,6 +91,10 @@ __global__ void moe_plan_pos_kernel(const long long* expert_of, int n_slots, int
   const int slot = blockIdx.x * PLAN_THREADS + threadIdx.x;
   if (slot >= n_slots) return;
   const int e = (int)expert_of[slot];
+  if (e < 0 || e >= n_experts) {
+    pos[slot] = -1;
+    return;
+  }
   pos[slot] = offsets[e] + block_hist[(long long)blockIdx.x * n_experts + e] + local_rank[slot];
 }
 
@@ -101,6 +108,7 @@ moe_permute_kernel(const __nv_bfloat16* x, long long ldx, const int* pos, const 
       const bf16x8 v = ld8(x + (long long)b * ldx + c);
       for (int j = 0; j < k; ++j) {
         const int r = pos[b * k + j];
+        if (r < 0) continue;
         if (w == nullptr) {
           st8(xp + (long long)r * ldp + c, v);
         } else {
@@ -132,6 +140,7 @@ moe_permute_f32_kernel(const float* x, const int* pos, const float* w, int T, in
   if (b < T) {
     for (int j = 0; j < k; ++j) {
       const long long r = pos[b * k + j];
+      if (r < 0) continue;
       const float s = w != nullptr ? w[b * k + j] : 1.f;
       for (int c = threadIdx.x; c < H; c += 128) xp[r * H + c] = s * x[(long long)b * H + c];
     }
@@ -177,6 +186,59 @@ route_top_kernel(const float* logits, int T, int E, int top, long long* idx, flo
       idx[t * top + j] = first;
       score[t * top + j] = 1.f / (1.f + expf(-z));
     }
+  }
+}
+
+__device__ __forceinline__ unsigned ordered_key(float x) {      // same order as the numbers, never 0
+  const unsigned b = __float_as_uint(x);
+  return max(b & 0x80000000u ? ~b : b | 0x80000000u, 1u);
+}
+
+// One warp per token.  Scores stay in registers, what decides (score + correction) beside them as integers.
+template <int NPL>
+__global__ void __launch_bounds__(256)
+route_softmax_top_kernel(const float* logits, const float* correction, int T, int E, int top, long long* idx, float* score) {
+  const long long t = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (t >= T) return;
+  float s[NPL], mx = -INFINITY, sum = 0.f;
+#pragma unroll
+  for (int n = 0; n < NPL; ++n) {
+    s[n] = n * 32 + lane < E ? logits[t * E + n * 32 + lane] : -INFINITY;
+    mx = fmaxf(mx, s[n]);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+#pragma unroll
+  for (int n = 0; n < NPL; ++n) {
+    s[n] = expf(s[n] - mx);
+    sum += s[n];
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+  unsigned key[NPL];                                   // 0: out of range or taken
+#pragma unroll
+  for (int n = 0; n < NPL; ++n) {
+    s[n] /= sum;
+    key[n] = n * 32 + lane < E ? ordered_key(s[n] + correction[n * 32 + lane]) : 0u;
+  }
+  for (int j = 0; j < top; ++j) {
+    unsigned mine = 0;
+#pragma unroll
+    for (int n = 0; n < NPL; ++n) mine = max(mine, key[n]);
+    const unsigned best = __reduce_max_sync(0xffffffffu, mine);
+    unsigned at = 0xffffffffu;
+#pragma unroll
+    for (int n = NPL - 1; n >= 0; --n)
+      if (key[n] == best) at = n * 32 + lane;          // this lane's lowest expert with that value
+    const unsigned first = __reduce_min_sync(0xffffffffu, at);
+#pragma unroll
+    for (int n = 0; n < NPL; ++n)
+      if (n * 32 + lane == first) {
+        key[n] = 0;
+        idx[t * top + j] = first;
+        score[t * top + j] = s[n];
+      }
   }
 }
 
@@ -273,6 +335,18 @@ MSRL_API int msrl_route_top(const float* logits, int T, int E, int top, long lon
   if (E <= 64) route_top_kernel<2><<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
   else if (E <= 256) route_top_kernel<8><<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
   else route_top_kernel<32><<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
+  return (int)cudaGetLastError();
+}
+
+// logits [T, E], correction [E] -> idx, score [T, top]; at most 1024 router outputs
+MSRL_API int msrl_route_softmax_top(const float* logits, const float* correction, int T, int E, int top, long long* idx,
+                                    float* score, cudaStream_t st) {
+  if (T == 0) return 0;
+  if (E < 1 || E > 1024 || top < 1 || top > E) return (int)cudaErrorInvalidValue;
+  const unsigned grid = (unsigned)((T + 7) / 8);
+  if (E <= 64) route_softmax_top_kernel<2><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
+  else if (E <= 256) route_softmax_top_kernel<8><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
+  else route_softmax_top_kernel<32><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
   return (int)cudaGetLastError();
 }
 

@@ -7,7 +7,10 @@
 // norm(x) = x / sqrt(mean(x^2) + eps) * (offset + weight), all in fp32, with x less its mean when `centered` (the
 // squares are then summed in a pass of their own over the kept row); y is stored in the activation type.  One block
 // per row; the row stays in registers between the sum and the norm (longer rows than the register budget re-read the
-// residual they just wrote).  A null `y` skips the norm.
+// residual they just wrote).  A null `y` skips the norm; without a norm weight y is the residual itself.
+//
+//   post_add          d = delta[t], or sum_j w[t, j] * e[pos(t, j)] + sh[t] where a negative pos stands for the residual's
+//                     row; resid[t] += mult * d / sqrt(mean(d^2) + eps) * weight;  y[t] = resid[t] or a norm of it
 //
 //   glu               act(gate) * up of rows [gate | up]: silu, tanh-gelu, or the clamped swish with (up + 1)
 #include "dtype_utils.cuh"
@@ -135,6 +138,20 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
     }
   }
   if (p.y == nullptr) return;
+  T* y = p.y + t * W;
+  if (SRC == SRC_EMBED && p.norm_w == nullptr) {
+#pragma unroll
+    for (int k = 0; k < NPT; ++k) {
+      const int c = (k * RS_THREADS + threadIdx.x) * V;
+      if (c < W) stv<V>(y + c, keep[k]);
+    }
+    for (int c = (NPT * RS_THREADS + threadIdx.x) * V; c < W; c += RS_THREADS * V) {
+      float f[4];
+      ldv<V>(res + c, f);
+      stv<V>(y + c, f);
+    }
+    return;
+  }
   float mean = 0.f;
   if (FULL && p.centered) {
     mean = block_sum(sum, red) / (float)W;
@@ -157,7 +174,6 @@ __global__ void __launch_bounds__(RS_THREADS) row_norm_kernel(const RowArgs<T> p
     }
   }
   const float r = 1.f / sqrtf(block_sum(ss, red) / (float)W + p.eps);
-  T* y = p.y + t * W;
 #pragma unroll
   for (int k = 0; k < NPT; ++k) {
     const int c = (k * RS_THREADS + threadIdx.x) * V;
@@ -197,6 +213,130 @@ template <typename T, int SRC>
 int launch_row_norm(const RowArgs<T>& p, long long rows, cudaStream_t st) {
   if (rows == 0) return 0;
   return p.centered || p.delta2 != nullptr ? launch_rows<T, SRC, true>(p, rows, st) : launch_rows<T, SRC, false>(p, rows, st);
+}
+
+template <typename T>
+struct PostArgs {
+  const T* delta;                         // the sublayer's rows, or null:
+  const T* e;                             // expert rows,
+  const int* pos;                         // [rows, top]
+  const float* weights;                   // [rows, top]
+  int top;
+  const T* shared;                        // one more term, or null
+  float* resid;
+  const float* norm_w;
+  float eps, mult;
+  const float* after_w;                   // norm of the sum, or null
+  float after_eps;
+  T* y;
+  int W;
+};
+
+// One block per row.  Rows up to NPT * 256 * V entries stay in registers; what is longer is computed again.
+template <typename T, int V, int NPT, bool MOE>
+__global__ void __launch_bounds__(RS_THREADS) post_add_kernel(const PostArgs<T> p) {
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  const int W = p.W;
+  float* res = p.resid + t * W;
+  T* y = p.y + t * W;
+  auto value = [&](int c, float (&r)[4], float (&d)[4]) {     // the residual's entries and the sublayer's
+    ldv<V>(res + c, r);
+    if constexpr (!MOE) {
+      ldv<V>(p.delta + t * W + c, d);
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) d[i] = 0.f;
+      for (int j = 0; j < p.top; ++j) {
+        const int at = p.pos[t * p.top + j];
+        const float w = p.weights[t * p.top + j];
+        float f[4];
+        if (at >= 0) ldv<V>(p.e + (long long)at * W + c, f);
+#pragma unroll
+        for (int i = 0; i < V; ++i) d[i] += w * (at >= 0 ? f[i] : r[i]);
+      }
+      if (p.shared != nullptr) {
+        float f[4];
+        ldv<V>(p.shared + t * W + c, f);
+#pragma unroll
+        for (int i = 0; i < V; ++i) d[i] += f[i];
+      }
+    }
+  };
+  float r[NPT][4], d[NPT][4], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NPT; ++k) {
+    const int c = (k * RS_THREADS + threadIdx.x) * V;
+    if (c < W) {
+      value(c, r[k], d[k]);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss += d[k][i] * d[k][i];
+    }
+  }
+  const int rest = (NPT * RS_THREADS + threadIdx.x) * V;
+  for (int c = rest; c < W; c += RS_THREADS * V) {
+    float a[4], b[4];
+    value(c, a, b);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss += b[i] * b[i];
+  }
+  const float inv = p.mult / sqrtf(block_sum(ss, red) / (float)W + p.eps);
+  float sum = 0.f;
+  auto add = [&](int c, float (&a)[4], const float (&b)[4]) {
+    float w[4];
+    ldv<V>(p.norm_w + c, w);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      a[i] += b[i] * inv * w[i];
+      sum += a[i] * a[i];
+    }
+    stv<V>(res + c, a);
+    if (p.after_w == nullptr) stv<V>(y + c, a);
+  };
+#pragma unroll
+  for (int k = 0; k < NPT; ++k) {
+    const int c = (k * RS_THREADS + threadIdx.x) * V;
+    if (c < W) add(c, r[k], d[k]);
+  }
+  for (int c = rest; c < W; c += RS_THREADS * V) {
+    float a[4], b[4];
+    value(c, a, b);
+    add(c, a, b);
+  }
+  if (p.after_w == nullptr) return;
+  const float q = 1.f / sqrtf(block_sum(sum, red) / (float)W + p.after_eps);
+  auto norm = [&](int c, const float (&a)[4]) {
+    float w[4];
+    ldv<V>(p.after_w + c, w);
+#pragma unroll
+    for (int i = 0; i < V; ++i) w[i] *= a[i] * q;
+    stv<V>(y + c, w);
+  };
+#pragma unroll
+  for (int k = 0; k < NPT; ++k) {
+    const int c = (k * RS_THREADS + threadIdx.x) * V;
+    if (c < W) norm(c, r[k]);
+  }
+  for (int c = rest; c < W; c += RS_THREADS * V) {
+    float a[4];
+    ldv<V>(res + c, a);
+    norm(c, a);
+  }
+}
+
+template <typename T, bool MOE>
+int launch_post(const PostArgs<T>& p, long long rows, cudaStream_t st) {
+  const unsigned g = (unsigned)rows;
+  if (p.W % 4 != 0) {
+    post_add_kernel<T, 1, 4, MOE><<<g, RS_THREADS, 0, st>>>(p);
+  } else {
+    const int units = (p.W / 4 + RS_THREADS - 1) / RS_THREADS;
+    if (units <= 1) post_add_kernel<T, 4, 1, MOE><<<g, RS_THREADS, 0, st>>>(p);
+    else if (units <= 2) post_add_kernel<T, 4, 2, MOE><<<g, RS_THREADS, 0, st>>>(p);
+    else if (units <= 4) post_add_kernel<T, 4, 4, MOE><<<g, RS_THREADS, 0, st>>>(p);
+    else post_add_kernel<T, 4, 8, MOE><<<g, RS_THREADS, 0, st>>>(p);
+  }
+  return (int)cudaGetLastError();
 }
 
 enum { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMPED_SWISH = 2 };
@@ -322,6 +462,20 @@ MSRL_API int msrl_moe_combine_norm(const void* e, const int* pos, int top, float
     p.shared = (const T*)shared;
     p.delta2 = (const T*)delta;
     return launch_row_norm<T, SRC_MOE>(p, rows, st);
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_post_add(const void* delta, const void* e, const int* pos, const float* weights, int top, const void* shared,
+                           float* resid, const float* norm_w, float eps, float mult, const float* after_w, float after_eps,
+                           void* y, long long rows, int W, int is_f32, cudaStream_t st) {
+  if (rows == 0) return 0;
+  if (delta == nullptr && (e == nullptr || pos == nullptr || weights == nullptr)) return (int)cudaErrorInvalidValue;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const PostArgs<T> p{(const T*)delta, (const T*)e, pos, weights, top, (const T*)shared, resid, norm_w, eps, mult, after_w,
+                        after_eps, (T*)y, W};
+    return delta == nullptr ? launch_post<T, true>(p, rows, st) : launch_post<T, false>(p, rows, st);
   };
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
