@@ -54,7 +54,7 @@ def parse_args():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="grpo", choices=["grpo", "serve"],
                     help="grpo: the headline benchmark; serve: prefill and decode throughput of the layer-by-layer "
-                         "decoders (Pumotar, Sunatar) beside the closest decoders of equal size, one JSON line per case")
+                         "decoders (Pumotar, Sunatar, Gapevik) beside the closest decoders of equal size, one JSON line per case")
     ap.add_argument("--serve-sizes", default="", help="comma-separated subset of the serve workload's sizes")
     ap.add_argument("--serve-models", default="", help="comma-separated subset of the serve workload's models")
     ap.add_argument("--model", default="qwen25_7b")

@@ -8,9 +8,10 @@ from __future__ import annotations
 
 import torch
 
-from . import (DeltaLayout, DeltaWeights, GroupedHeads, LatentLayout, MemoryLayout, MemoryWeights, add_norm_, angle_table,
-               delta_decode, delta_prefill, embed_norm, glu_fwd, latent_decode_attention, latent_prefill_attention, latent_prep,
-               latent_spread_, memory_decode, memory_prefill, moe_combine_norm_, qkv_prep_, rope_table, rows_gather,
+from . import (ConvHeads, ConvNormWeights, DeltaLayout, DeltaWeights, GroupedHeads, LatentLayout, MemoryLayout, MemoryWeights,
+               PostNorm, ScoreForm, add_norm_, angle_table, conv_qkv_decode, conv_qkv_prefill, delta_decode, delta_prefill, embed_norm,
+               glu_fwd, latent_decode_attention, latent_prefill_attention, latent_prep, latent_rotate_queries, latent_spread_,
+               memory_decode, memory_prefill, moe_combine_norm_, moe_post_add_, post_add_, qkv_prep_, rope_table, rows_gather,
                window_decode_attention, window_prefill_attention)
 from . import moe as K
 from .microbench import report, timeit
@@ -22,20 +23,26 @@ def fp32_tflops() -> float:
     return p.multi_processor_count * 128 * 2 * clock / 1e12
 
 
-def _delta(t, heads=32, dim=128, vdim=128, taps=4):
+def _delta(t, heads=32, dim=128, vdim=128, taps=4, head_decay=False):
     kd, hv = heads * dim, heads * vdim
-    lay = DeltaLayout(heads, heads, dim, vdim, taps, 0, kd, 2 * kd, 2 * kd + hv)
+    na = heads if head_decay else kd
+    lay = DeltaLayout(heads, heads, dim, vdim, taps, 0, kd, 2 * kd, 2 * kd + hv, head_decay=head_decay, silu_gate=head_decay)
     proj = torch.randn(t, 2 * kd + hv + heads + 256, device="cuda").bfloat16()
-    a, gate = torch.randn(t, kd, device="cuda").bfloat16(), torch.randn(t, hv, device="cuda").bfloat16()
+    a, gate = torch.randn(t, na, device="cuda").bfloat16(), torch.randn(t, hv, device="cuda").bfloat16()
     w = DeltaWeights(torch.randn(lay.channels, taps, device="cuda"), torch.zeros(heads, device="cuda") - 2,
-                     torch.zeros(kd, device="cuda"), torch.ones(vdim, device="cuda"))
+                     torch.zeros(na, device="cuda"), torch.ones(vdim, device="cuda"))
     return lay, proj, a, gate, w
 
 
-def case_delta(small: bool, iters: int):
+def case_head_delta(small: bool, iters: int):
+    case_delta(small, iters, True)
+
+
+def case_delta(small: bool, iters: int, head_decay: bool = False):
+    kind = " decay per head" if head_decay else ""
     for b, n in ([(1, 2048)] if small else [(1, 8192), (8, 1024), (32, 256)]):
         t = b * n
-        lay, proj, a, gate, w = _delta(t)
+        lay, proj, a, gate, w = _delta(t, head_decay=head_decay)
         ring = torch.zeros(b, lay.taps, lay.channels, device="cuda").bfloat16()
         state = torch.zeros(b, lay.heads, lay.dim, lay.vdim, device="cuda")
         cu = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda")
@@ -43,16 +50,16 @@ def case_delta(small: bool, iters: int):
         start, slots = torch.zeros(b, dtype=torch.int32, device="cuda"), torch.arange(b, device="cuda")
         ms = timeit(lambda: delta_prefill(proj, a, gate, lay, w, ring, state, seq, cu, start, slots, 1e-5), iters)
         fma = 4.0 * t * lay.heads * lay.dim * lay.vdim
-        report(f"delta_prefill {b}x{n} heads=32 dim=128", ms, bytes_=2.0 * t * (lay.channels + 3 * lay.heads * lay.vdim),
+        report(f"delta_prefill {b}x{n} heads=32 dim=128{kind}", ms, bytes_=2.0 * t * (lay.channels + 3 * lay.heads * lay.vdim),
                note=f"{2 * fma / ms / 1e9:.1f} TFLOP/s fp32 = {2 * fma / ms / 1e9 / fp32_tflops():.3f} of nominal fp32")
     for b in ([32] if small else [1, 32, 256]):
-        lay, proj, a, gate, w = _delta(b)
+        lay, proj, a, gate, w = _delta(b, head_decay=head_decay)
         ring = torch.zeros(b, lay.taps, lay.channels, device="cuda").bfloat16()
         state = torch.zeros(b, lay.heads, lay.dim, lay.vdim, device="cuda")
         pos = torch.full((b,), 100, dtype=torch.int32, device="cuda")
         slots = torch.randperm(b, device="cuda")
         ms = timeit(lambda: delta_decode(proj, a, gate, lay, w, ring, state, pos, slots, 1e-5), iters)
-        report(f"delta_decode B={b} heads=32 dim=128", ms, bytes_=2.0 * state.numel() * 4 + b * lay.channels * 2 * 8)
+        report(f"delta_decode B={b} heads=32 dim=128{kind}", ms, bytes_=2.0 * state.numel() * 4 + b * lay.channels * 2 * 8)
 
 
 def case_latent(small: bool, iters: int):
@@ -199,4 +206,102 @@ def case_routed(small: bool, iters: int):
         report(f"add_norm centred {t}x{h}", ms, bytes_=t * h * 12.0)
 
 
-CASES = {"hybrid_memory": case_memory, "hybrid_window": case_window, "hybrid_routed": case_routed, "hybrid_delta": case_delta, "hybrid_latent": case_latent, "hybrid_stream": case_stream}
+def case_conv(small: bool, iters: int):
+    """Convolved attention in chunks: preparation, soft-capped and gated prompt attention, decode over a chunk."""
+    h, g, d, size = 32, 8, 128, 1024
+    heads = GroupedHeads(h, g, d, d, d, d, 0, h * d, (h + g) * d)
+    lay = ConvHeads(heads, 4, 0, h * d, (h + g) * d)
+    w = ConvNormWeights(torch.randn(lay.channels, 4, device="cuda"), torch.ones(d, device="cuda"), torch.ones(d, device="cuda"))
+    tab = angle_table(8192, tuple(1e4 ** (-i / 32) for i in range(32)), "cuda")
+    t, n = (2048, 2048) if small else (16384, 8192)
+    b = t // n
+    proj = torch.randn(t, lay.row + 32, device="cuda").bfloat16()
+    gate = proj[:, lay.row:]
+    pos, slots = torch.arange(t, dtype=torch.int32, device="cuda") % n, torch.arange(t, device="cuda")
+    kc, vc = (torch.empty(t // 16, 16, g, d, device="cuda").bfloat16() for _ in range(2))
+    ring = torch.zeros(256, 4, lay.channels, device="cuda").bfloat16()
+    cu, seq = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda"), torch.arange(t, dtype=torch.int32, device="cuda") // n
+    start, state = torch.zeros(b, dtype=torch.int32, device="cuda"), torch.arange(b, device="cuda")
+    ms = timeit(lambda: conv_qkv_prefill(proj, lay, w, 1e-5, tab, pos, slots, kc, vc, ring, state, seq, cu, start), iters)
+    report(f"conv_qkv_prefill T={t} H={h}/{g} d={d}", ms, bytes_=2.0 * t * d * (2 * h + 6 * g))
+    for name, form, keys in (("plain", ScoreForm(), None), ("gated", ScoreForm(0.0, gate), None), ("capped and gated", ScoreForm(30.0, gate), None),
+                             ("capped and gated", ScoreForm(30.0, gate), size)):
+        cq = torch.arange(0, t + 1, keys or n, dtype=torch.int32, device="cuda")
+        ms = timeit(lambda: window_prefill_attention(proj, heads, cq, cq, keys or n, d ** -0.5, None, form=form), iters)
+        pairs = t * ((keys or n) + 1) / 2
+        report(f"prompt attention {name} {b}x{n} H={h}/{g} chunk={keys}", ms, flops=4.0 * pairs * h * d,
+               note=f"{ms * 1e6 / (pairs * h) * 1e3 * torch.cuda.get_device_properties(0).multi_processor_count:.1f} SM-ps per score")
+    for b, ctx in ([(16, 1024)] if small else [(256, 2048), (32, 8192), (1, 8192)]):
+        nb = b * ctx // 16
+        kc, vc = (torch.randn(nb, 16, g, d, device="cuda").bfloat16() for _ in range(2))
+        bt = torch.randperm(nb, device="cuda").to(torch.int32).view(b, -1)
+        cl = torch.full((b,), ctx, dtype=torch.int32, device="cuda")
+        pos, slots, state = cl - 1, bt[:, -1].long() * 16 + 15, torch.arange(b, device="cuda")
+        x = proj[:b]
+        ms = timeit(lambda: conv_qkv_decode(x, lay, w, 1e-5, tab, pos, slots, kc, vc, ring, state), iters)
+        report(f"conv_qkv_decode B={b} H={h}/{g}", ms, bytes_=2.0 * b * (lay.channels * 6 + lay.row) + 16.0 * lay.channels)
+        q = torch.randn(b, h * d, device="cuda").bfloat16()
+        for chunk in (None, size):
+            ms = timeit(lambda: window_decode_attention(q, heads, kc, vc, bt, cl, ctx, d ** -0.5, None, chunk=chunk,
+                                                        form=ScoreForm(30.0, gate[:b])), iters)
+            report(f"decode capped and gated H={h}/{g} B={b} ctx={ctx} chunk={chunk}", ms,
+                   bytes_=4.0 * b * ((ctx - 1) % chunk + 1 if chunk else ctx) * g * d)
+
+
+def case_gated_latent(small: bool, iters: int):
+    """Latent attention with a query latent, half-split rotation, window, sink and gates."""
+    for heads in (16, 32, 64):
+        lay = LatentLayout(heads, 64, 64, 128, 512, 128, 128, 768, 64, True, 768, 0)
+        for b, ctx, window in ([(16, 1024, None)] if small else [(256, 2048, None), (256, 2048, 1024), (32, 8192, 1024), (1, 8192, 1024)]):
+            nb = b * ctx // 16
+            cache = torch.randn(nb, 16, lay.CP, device="cuda").bfloat16()
+            bt = torch.randperm(nb, device="cuda").to(torch.int32).view(b, -1)
+            cl = torch.full((b,), ctx, dtype=torch.int32, device="cuda")
+            q, gate = torch.randn(b, heads, lay.CP, device="cuda").bfloat16(), torch.randn(b, heads, device="cuda").bfloat16()
+            form = ScoreForm(0.0, gate, torch.zeros(heads, device="cuda"))
+            ms = timeit(lambda: latent_decode_attention(q, cache, lay, bt, cl, ctx, 0.05, window=window, form=form), iters)
+            report(f"latent_decode gated, sink H={heads} B={b} ctx={ctx} window={window}", ms, bytes_=2.0 * b * min(ctx, window or ctx) * lay.CP)
+    heads, t, n = 32, (2048 if small else 16384), 2048
+    lay = LatentLayout(heads, 64, 64, 128, 512, 128, 128, 768, 64, True, 768, 0)
+    proj = torch.randn(t, 768 + 576 + 32, device="cuda").bfloat16()
+    q = torch.randn(t, heads * 128, device="cuda").bfloat16()
+    pos, slots = torch.arange(t, dtype=torch.int32, device="cuda") % n, torch.arange(t, device="cuda")
+    cache = torch.empty(t // 16, 16, lay.CP, device="cuda").bfloat16()
+    tab, nw, qw = rope_table(4096, 64, 1e4, proj.device), torch.ones(512, device="cuda"), torch.ones(768, device="cuda")
+    ms = timeit(lambda: latent_prep(proj, lay, nw, 1e-5, tab, pos, slots, cache, True, q_norm=qw), iters)
+    report(f"latent_prep with query latent T={t}", ms, bytes_=2.0 * t * (2 * 768 + 3 * lay.CP))
+    ms = timeit(lambda: latent_rotate_queries(q, lay, tab, pos), iters)
+    report(f"latent_rotate_queries T={t} H={heads} rot=64", ms, bytes_=4.0 * t * heads * 64)
+    kv = torch.randn(t, heads * 256, device="cuda").bfloat16()
+    cu = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda")
+    form = ScoreForm(0.0, proj[:, -32:], torch.zeros(heads, device="cuda"))
+    for window in (None, 1024):
+        ms = timeit(lambda: latent_prefill_attention(q, kv, lay, cu, cu, n, 0.08, window, form), iters)
+        w = window or n
+        report(f"latent_prefill_attention gated, sink {t // n}x{n} H=32 window={window}", ms,
+               flops=4.0 * (t // n) * (w * (w + 1) / 2 + (n - w) * w) * heads * 128)
+
+
+def case_post_norm(small: bool, iters: int):
+    """Post-norm adds and the soft-max router."""
+    e, k, h = 64, 8, 2304
+    for t in ([2048] if small else [16384, 256]):
+        z, corr = torch.randn(t, e + 8, device="cuda"), torch.zeros(e + 8, device="cuda")
+        ms = timeit(lambda: K.route_softmax_top(z, corr, k), iters)
+        report(f"route_softmax_top T={t} E={e + 8} k={k}", ms, bytes_=t * (4.0 * (e + 8) + 12 * k))
+        idx, score = K.route_softmax_top(z, corr, k)
+        plan = K.moe_plan(idx, e)
+        x, y = torch.randn(t, h, device="cuda").bfloat16(), torch.randn(plan.max_rows, h, device="cuda").bfloat16()
+        resid, w = torch.zeros(t, h, device="cuda"), torch.ones(h, device="cuda")
+        post = PostNorm(w, 1e-5, 0.5)
+        ms = timeit(lambda: K.moe_permute(x, plan), iters)
+        report(f"moe_permute T={t} k={k} of {e} + 8 H={h}", ms, bytes_=2.0 * t * h * (k * e / (e + 8) + 1))
+        ms = timeit(lambda: moe_post_add_(resid, y, plan.pos, score, post), iters)
+        report(f"moe_post_add T={t} k={k} H={h}", ms, bytes_=t * h * (2.0 * k * e / (e + 8) + 8 + 2))
+        ms = timeit(lambda: post_add_(resid, x, post), iters)
+        report(f"post_add {t}x{h}", ms, bytes_=t * h * 12.0)
+
+
+CASES = {"hybrid_conv": case_conv, "hybrid_gated_latent": case_gated_latent, "hybrid_head_delta": case_head_delta,
+         "hybrid_post_norm": case_post_norm, "hybrid_memory": case_memory, "hybrid_window": case_window, "hybrid_routed": case_routed,
+         "hybrid_delta": case_delta, "hybrid_latent": case_latent, "hybrid_stream": case_stream}

@@ -11,6 +11,10 @@ Sunatar: ``window`` has window attention everywhere, ``memory`` the matrix memor
 matrix-memory layer in four.  Closest existing models: ``gqa``, the grouped-head decoder with routed and shared experts
 of the same width, heads, experts and layer count (full attention), and for the recurrent layers ``mixed``.
 
+Gapevik: ``conv`` has convolved attention in chunks everywhere, ``gated`` latent attention with a query latent, window, sink
+and gates, ``delta`` the delta rule with a decay per head, ``gapevik`` the three in turn.  Closest existing models of the same
+width, heads, experts and layer count: ``window``, ``latent`` and ``mixed``.
+
 One JSON line per measurement: tokens/s from CUDA events around the engine calls.
 """
 from __future__ import annotations
@@ -21,8 +25,9 @@ from typing import List
 
 import torch
 
-from ..models.hybrid_config import (ChannelDeltaSpec, GluSpec, HybridConfig, LatentAttentionSpec, LayerSpec, MatrixMemorySpec,
-                                    Rotary, ScoredMoESpec, TableMoESpec, WavelengthScaling, WindowAttentionSpec)
+from ..models.hybrid_config import (ChannelDeltaSpec, Chunk, ConvAttentionSpec, GluSpec, HeadDeltaSpec, HybridConfig,
+                                    LatentAttentionSpec, LayerSpec, MatrixMemorySpec, Rotary, ScoredMoESpec, SoftmaxMoESpec,
+                                    TableMoESpec, WavelengthScaling, WindowAttentionSpec)
 from ..models.transformer_config import TransformerConfig
 from .engine import LLMEngine
 from .scheduler import SamplingParams
@@ -51,7 +56,7 @@ PREFILL = ((1, 8192), (8, 2048))
 DECODE = ((1, 2048), (32, 2048), (256, 2048))
 NEW_TOKENS = 64
 WINDOW = 1024
-MODELS = ("mla", "latent", "mixed", "gqa", "window", "memory", "sunatar")
+MODELS = ("mla", "latent", "mixed", "gqa", "window", "memory", "sunatar", "conv", "gated", "delta", "gapevik")
 
 
 def sunatar_config(s: Size, pattern: str) -> HybridConfig:
@@ -67,7 +72,20 @@ def sunatar_config(s: Size, pattern: str) -> HybridConfig:
     return HybridConfig("Sunatar", s.vocab, s.width, layers, 1e-5)
 
 
+def gapevik_config(s: Size, pattern: str) -> HybridConfig:
+    kinds = {"conv": ("attention", ConvAttentionSpec(s.heads, s.heads // 4, 128, 128, 4, 128 ** -0.5, Rotary(64, 500000.0), 30.0,
+                                                     Chunk(WINDOW))),
+             "gated": ("latent_attention", LatentAttentionSpec(s.heads, s.dn, s.dr, s.dv, s.rank, (s.dn + s.dr) ** -0.5,
+                                                               Rotary(s.dr, 10000.0, halves=True), 3 * s.rank // 2, WINDOW, True, True)),
+             "delta": ("delta", HeadDeltaSpec(s.heads, s.heads // 2, 128, 128, 4))}
+    moe = SoftmaxMoESpec(s.experts, s.top, GluSpec(s.expert_ff, "silu"), s.experts // 8)
+    layers = [LayerSpec(*kinds[pattern if pattern in kinds else tuple(kinds)[i % 3]], moe) for i in range(s.layers)]
+    return HybridConfig("Gapevik", s.vocab, s.width, layers, 1e-5, residual_mult=0.5)
+
+
 def hybrid_config(s: Size, pattern: str) -> HybridConfig:
+    if pattern in ("conv", "gated", "delta", "gapevik"):
+        return gapevik_config(s, pattern)
     if pattern in ("window", "memory", "sunatar"):
         return sunatar_config(s, pattern)
     latent = LayerSpec("latent_attention", LatentAttentionSpec(s.heads, s.dn, s.dr, s.dv, s.rank, (s.dn + s.dr) ** -0.5,
@@ -108,15 +126,30 @@ def random_state(cfg: HybridConfig, device) -> dict:
         p, m = f"l{i}.mix.", l.mixer
         vec(f"l{i}.norm1", w, ones)
         if not cfg.design.parallel:
-            vec(f"l{i}.norm2", w)
-        if l.type == "latent_attention":
-            lin(p + "q", m.heads * (m.dim + m.rot_dim), w)
+            vec(f"l{i}.norm2", w, ones)
+        if isinstance(m, LatentAttentionSpec):
+            if m.q_rank:
+                lin(p + "dq", m.q_rank, w)
+                vec(p + "dq.norm", m.q_rank, 1.0)
+            lin(p + ("uq" if m.q_rank else "q"), m.heads * (m.dim + m.rot_dim), m.q_rank or w)
+            if m.sink:
+                vec(p + "sink", m.heads)
+            if m.head_gate:
+                lin(p + "g", m.heads, w)
             lin(p + "dkv", m.kv_rank + m.rot_dim, w)
             vec(p + "dkv.norm", m.kv_rank, 1.0)
             lin(p + "uk", m.heads * m.dim, m.kv_rank)
             lin(p + "uv", m.heads * m.vdim, m.kv_rank)
             lin(p + "o", w, m.heads * m.vdim)
-        elif l.type == "attention":
+        elif isinstance(m, ConvAttentionSpec):
+            for n, rows in (("q", m.heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
+                lin(p + n, rows, w)
+                out[p + n + ".conv"] = torch.randn(rows, m.conv, generator=g, device=device) * 0.5
+            vec(p + "q.norm", m.dim, 1.0)
+            vec(p + "k.norm", m.dim, 1.0)
+            lin(p + "g", m.heads, w)
+            lin(p + "o", w, m.heads * m.vdim)
+        elif isinstance(m, WindowAttentionSpec):
             for n, rows in (("q", m.heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
                 lin(p + n, rows, w)
                 vec(p + n + ".b", rows)
@@ -124,7 +157,7 @@ def random_state(cfg: HybridConfig, device) -> dict:
             vec(p + "k.norm", m.kv_heads * m.dim, 1.0)
             out[p + "vmix"] = torch.tensor(0.3, device=device)
             lin(p + "o", w, m.heads * m.vdim)
-        elif l.type == "mlstm":
+        elif isinstance(m, MatrixMemorySpec):
             for n, rows in (("q", m.heads * m.dim), ("k", m.heads * m.dim), ("v", m.heads * m.vdim), ("g", m.heads * m.vdim),
                             ("i", m.heads), ("f", m.heads)):
                 lin(p + n, rows, w)
@@ -140,10 +173,15 @@ def random_state(cfg: HybridConfig, device) -> dict:
             lin(p + "b", m.heads, w)
             vec(p + "A_log", m.heads, -2.0)
             vec(p + "norm", m.vdim, 1.0)
-            vec(p + "dt_bias", m.heads * m.dim)
-            for a, n in (("a", m.heads * m.dim), ("g", hv)):
-                lin(p + a + "1", 128, w)
-                lin(p + a + "2", n, 128)
+            if isinstance(m, HeadDeltaSpec):
+                vec(p + "dt_bias", m.heads)
+                lin(p + "a", m.heads, w)
+                lin(p + "g", hv, w)
+            else:
+                vec(p + "dt_bias", m.heads * m.dim)
+                for a, n in (("a", m.heads * m.dim), ("g", hv)):
+                    lin(p + a + "1", 128, w)
+                    lin(p + a + "2", n, 128)
             lin(p + "o", w, hv)
         p = f"l{i}.mlp."
         if isinstance(l.mlp, ScoredMoESpec):
@@ -151,6 +189,11 @@ def random_state(cfg: HybridConfig, device) -> dict:
                 glu(f"{p}e{e}.", l.mlp.expert.ff)
             lin(p + "router", l.mlp.experts, w)
             glu(p + "shared.", l.mlp.shared.ff)
+        elif isinstance(l.mlp, SoftmaxMoESpec):
+            for e in range(l.mlp.experts):
+                glu(f"{p}e{e}.", l.mlp.expert.ff)
+            lin(p + "router", l.mlp.outputs, w)
+            vec(p + "correction", l.mlp.outputs)
         elif isinstance(l.mlp, TableMoESpec):
             for e in range(l.mlp.experts):
                 glu(f"{p}e{e}.", l.mlp.expert.ff)
