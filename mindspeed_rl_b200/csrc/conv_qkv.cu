@@ -51,21 +51,21 @@ struct HeadOf {
     if (p.cu == nullptr && !is_q) return nullptr;
     return p.out + t * p.out_ld + (is_q ? p.oq : is_v ? p.ov : p.ok) + h * pad;
   }
-  __device__ __forceinline__ T* cached(const ConvQkvArgs<T>& p, long long t) const {
-    const long long slot = p.slots[t];
+  __device__ __forceinline__ T* cached(const ConvQkvArgs<T>& p, long long slot) const {
     return is_q || slot < 0 ? nullptr : (is_v ? p.v_cache : p.k_cache) + (slot * p.G + h) * pad;
   }
 };
 
-constexpr int CQ_TT = 16, CQ_U = 4;      // tokens per warp, tokens loaded together
+constexpr int CQ_TT = 32, CQ_U = 4;      // tokens per warp, tokens in flight together
 
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256) conv_qkv4_kernel(const ConvQkvArgs<T> p, int per_warp) {
+__global__ void __launch_bounds__(256, 2) conv_qkv4_kernel(const ConvQkvArgs<T> p, int per_warp) {
   const int u = blockIdx.x * 8 + (threadIdx.x >> 5), d = (threadIdx.x & 31) * 4;
   if (u >= p.H + 2 * p.G) return;
   const HeadOf<T> hd(p, u);
   const int t0 = blockIdx.y * per_warp, t1 = min(p.tokens, t0 + per_warp);
   const bool on = d < hd.size, wr = d < hd.pad, decode = p.cu == nullptr;
+  const bool turned = on && !hd.is_v && d < p.rot, whole = p.rot % 4 == 0;
   ConvWindow<TAPS, T> cv;
   float w[4] = {0.f, 0.f, 0.f, 0.f};
   if (on) {
@@ -74,50 +74,78 @@ __global__ void __launch_bounds__(256) conv_qkv4_kernel(const ConvQkvArgs<T> p, 
   }
   int seq = -1;
   for (int tb = t0; tb < t1; tb += CQ_U) {
-    float x[CQ_U][4];
+    float y[CQ_U][4], cs[CQ_U][4];                       // cs: two cosines, two sines
     int sq[CQ_U], pos[CQ_U];
+    long long slot[CQ_U];
 #pragma unroll
     for (int n = 0; n < CQ_U; ++n) {
       const int t = min(tb + n, t1 - 1);
       sq[n] = decode ? t : p.tok_seq[t];
       pos[n] = p.positions[t];
+      slot[n] = hd.is_q ? -1 : p.slots[t];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) x[n][c] = 0.f;
-      if (on) ldf4(p.proj + t * p.ld + hd.col + d, x[n]);
+      for (int c = 0; c < 4; ++c) y[n][c] = 0.f;
+      if (on) ldf4(p.proj + t * p.ld + hd.col + d, y[n]);
+    }
+    if (turned) {
+#pragma unroll
+      for (int n = 0; n < CQ_U; ++n) {
+        const float* tab = p.table + (long long)min(max(pos[n], 0), p.table_rows - 1) * p.rot + (d >> 1);
+        if (whole) {
+          const float2 a = *reinterpret_cast<const float2*>(tab), b = *reinterpret_cast<const float2*>(tab + (p.rot >> 1));
+          cs[n][0] = a.x; cs[n][1] = a.y; cs[n][2] = b.x; cs[n][3] = b.y;
+        } else {
+          const bool two = d + 2 < p.rot;
+          cs[n][0] = tab[0];
+          cs[n][1] = two ? tab[1] : 1.f;
+          cs[n][2] = tab[p.rot >> 1];
+          cs[n][3] = two ? tab[(p.rot >> 1) + 1] : 0.f;
+        }
+      }
     }
 #pragma unroll
     for (int n = 0; n < CQ_U; ++n) {
       const int t = tb + n;
-      if (t >= t1) break;                                // uniform over the warp
+      if (t >= t1 || !on) continue;                      // what is past the end is not written
       if (sq[n] != seq) {
         seq = sq[n];
-        const long long slot = p.state_slots[seq];
-        if (on) {
-          if (slot < 0) cv.fill(p, t, 0, 0, 0, hd.col + d, hd.ch + d);      // a row that is not in use
-          else cv.fill(p, t, decode ? 0 : t - p.cu[seq], pos[n], slot, hd.col + d, hd.ch + d);
-          if (decode && slot >= 0) stf4(p.ring + (slot * TAPS + pos[n] % TAPS) * p.channels + hd.ch + d, x[n]);
-        }
+        const long long state = p.state_slots[seq];
+        if (state < 0) cv.fill(p, t, 0, 0, 0, hd.col + d, hd.ch + d);         // a row that is not in use
+        else cv.fill(p, t, decode ? 0 : t - p.cu[seq], pos[n], state, hd.col + d, hd.ch + d);
+        if (decode && state >= 0) stf4(p.ring + (state * TAPS + pos[n] % TAPS) * p.channels + hd.ch + d, y[n]);
       }
-      float y[4] = {0.f, 0.f, 0.f, 0.f};
-      if (on) cv.step(x[n], y);
-      if (!hd.is_v) {
-        const float inv = 1.f / sqrtf(warp_sum(y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3]) / (float)p.dim + p.eps);
+      cv.step(y[n], y[n]);
+    }
+    if (!hd.is_v) {
+      float ss[CQ_U];
 #pragma unroll
-        for (int c = 0; c < 4; ++c) y[c] *= inv * w[c];
-        const float* cs = p.table + (long long)min(max(pos[n], 0), p.table_rows - 1) * p.rot;
+      for (int n = 0; n < CQ_U; ++n) ss[n] = y[n][0] * y[n][0] + y[n][1] * y[n][1] + y[n][2] * y[n][2] + y[n][3] * y[n][3];
 #pragma unroll
-        for (int c = 0; c < 4; c += 2) {
-          if (d + c < p.rot) {
-            const float co = cs[(d + c) >> 1], si = cs[(p.rot + d + c) >> 1], a = y[c], b = y[c + 1];
-            y[c] = a * co - b * si;
-            y[c + 1] = b * co + a * si;
+      for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int n = 0; n < CQ_U; ++n) ss[n] += __shfl_xor_sync(0xffffffffu, ss[n], o);
+#pragma unroll
+      for (int n = 0; n < CQ_U; ++n) {
+        const float inv = 1.f / sqrtf(ss[n] / (float)p.dim + p.eps);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) y[n][c] *= inv * w[c];
+        if (turned) {
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            const float a = y[n][2 * c], b = y[n][2 * c + 1];
+            y[n][2 * c] = a * cs[n][c] - b * cs[n][2 + c];
+            y[n][2 * c + 1] = b * cs[n][c] + a * cs[n][2 + c];
           }
         }
       }
-      if (wr) {
-        T *o = hd.row(p, t), *k = hd.cached(p, t);
-        if (o != nullptr) stf4(o + d, y);
-        if (k != nullptr) stf4(k + d, y);
+    }
+#pragma unroll
+    for (int n = 0; n < CQ_U; ++n) {
+      const int t = tb + n;
+      if (t < t1 && wr) {
+        T *o = hd.row(p, t), *k = hd.cached(p, slot[n]);
+        if (o != nullptr) stf4(o + d, y[n]);
+        if (k != nullptr) stf4(k + d, y[n]);
       }
     }
   }
@@ -148,7 +176,7 @@ __global__ void __launch_bounds__(256) conv_qkv_kernel(const ConvQkvArgs<T> p) {
       inv = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
     }
     const float* w = hd.is_q ? p.q_norm : p.k_norm;
-    T *o = hd.row(p, t), *k = hd.cached(p, t);
+    T *o = hd.row(p, t), *k = hd.cached(p, p.slots[t]);
     for (int d = 2 * lane; d < hd.pad; d += 64) {
       float y[2] = {conv(d), conv(d + 1)};
       if (!hd.is_v) {

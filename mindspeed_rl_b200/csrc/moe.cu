@@ -344,8 +344,11 @@ MSRL_API int msrl_route_softmax_top(const float* logits, const float* correction
   if (T == 0) return 0;
   if (E < 1 || E > 1024 || top < 1 || top > E) return (int)cudaErrorInvalidValue;
   const unsigned grid = (unsigned)((T + 7) / 8);
-  if (E <= 64) route_softmax_top_kernel<2><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
-  else if (E <= 256) route_softmax_top_kernel<8><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
+  if (E <= 32) route_softmax_top_kernel<1><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
+  else if (E <= 64) route_softmax_top_kernel<2><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
+  else if (E <= 96) route_softmax_top_kernel<3><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
+  else if (E <= 160) route_softmax_top_kernel<5><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
+  else if (E <= 288) route_softmax_top_kernel<9><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
   else route_softmax_top_kernel<32><<<grid, 256, 0, st>>>(logits, correction, T, E, top, idx, score);
   return (int)cudaGetLastError();
 }

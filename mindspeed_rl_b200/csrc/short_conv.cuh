@@ -35,8 +35,9 @@ __device__ __forceinline__ float conv_one(const ConvIn<T>& p, long long t, int i
       x[j] = 0.f;
       if (pos - back >= 0)
         x[j] = ldf(i - back >= 0 ? p.proj + (t - back) * p.ld + col : ring + (long long)entry * p.channels);
-      w[j] = p.conv[(long long)ch * TAPS + j];
+      if (TAPS != 4) w[j] = p.conv[(long long)ch * TAPS + j];
     }
+    if constexpr (TAPS == 4) ldf4(p.conv + (long long)ch * TAPS, w);
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) s += x[j] * w[j];
   } else {
@@ -55,10 +56,14 @@ template <int TAPS, typename T>
 struct ConvWindow {
   float w[TAPS][4], x[TAPS][4];
   __device__ __forceinline__ void weights(const float* conv, int ch) {
+    // the 4 x TAPS weights lie side by side: ch is a multiple of 4
+    float f[TAPS][4];
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) ldf4(conv + (long long)ch * TAPS + i * 4, f[i]);
 #pragma unroll
     for (int c = 0; c < 4; ++c)
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) w[j][c] = conv[(long long)(ch + c) * TAPS + j];
+      for (int j = 0; j < TAPS; ++j) w[j][c] = f[(c * TAPS + j) / 4][(c * TAPS + j) % 4];
   }
   // window entries before token t (index i of its portion, position pos); x[TAPS - 1] is the token's own
   __device__ __forceinline__ void fill(const ConvIn<T>& p, long long t, int i, int pos, long long slot, int col, int ch) {

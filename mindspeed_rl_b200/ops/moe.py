@@ -130,13 +130,14 @@ def moe_permute(x: torch.Tensor, plan: MoePlan, w: Optional[torch.Tensor] = None
                                            c_int(plan.num_experts), ptr(plan.counts), ptr(plan.offsets), ptr(xp),
                                            c_ll(h), stream()), "moe_permute")
         return xp
-    xp = torch.zeros(plan.max_rows, h, dtype=x.dtype, device=x.device)     # CPU, or rows the kernel cannot move
+    # CPU, or rows the kernel cannot move; slots without a row meet in one behind the last
+    xp = torch.zeros(plan.max_rows + 1, h, dtype=x.dtype, device=x.device)
     rows = x.repeat_interleave(plan.k, dim=0)
     if w is not None:
         rows = (rows.float() * w.reshape(-1, 1).float()).to(x.dtype)
-    used = plan.pos >= 0
-    xp[plan.pos[used].long()] = rows[used]
-    return xp
+    pos = plan.pos.long()
+    xp[torch.where(pos < 0, plan.max_rows, pos)] = rows
+    return xp[:plan.max_rows]
 
 
 def moe_combine(y: torch.Tensor, plan: MoePlan, w: Optional[torch.Tensor] = None) -> torch.Tensor:
