@@ -7,8 +7,9 @@
 // Prepared rows hold the heads padded (qp, vp; pad entries are written as zeros), and so do the cache rows of k and v.
 // Prompt portions are followed by conv_ring_kernel; a decode step (one token per sequence) writes its ring entry itself.
 //
-//   conv_qkv4_kernel   heads of up to 128 entries, sizes and columns multiples of 4, 2 to 4 taps: a warp walks consecutive
-//                      tokens of one head with the convolution windows in registers, four channels per lane
+//   conv_qkv4_kernel, conv_qkv4_step_kernel   heads of up to 128 entries, sizes and columns multiples of 4, 2 to 4 taps: a
+//                      warp walks consecutive tokens of one head with the convolution windows in registers, four
+//                      channels per lane; in decode steps it takes one token
 //   conv_qkv_kernel    any sizes: a warp per token and head, every entry convolved where it is needed
 #include "short_conv.cuh"
 
@@ -56,98 +57,142 @@ struct HeadOf {
   }
 };
 
-constexpr int CQ_TT = 32, CQ_U = 4;      // tokens per warp, tokens in flight together
+constexpr int CQ_TT = 32, CQ_U = 4;      // tokens per warp (one a lane looks up), tokens in flight together
 
+template <typename T>
+__device__ __forceinline__ float inv_rms(float ss, float inv_n, float eps) {
+  if constexpr (sizeof(T) == 2) return rsqrtf(fmaf(ss, inv_n, eps));     // within 2^-22, far below the rounding of the result
+  else return 1.f / sqrtf(ss * inv_n + eps);
+}
+
+// cosines and sines of the two pairs from entry d on (a multiple of 4, below rot)
+__device__ __forceinline__ void pair_angles(const float* row, int d, int rot, float (&cs)[4]) {
+  const float* tab = row + (d >> 1);
+  if (rot % 4 == 0) {
+    const float2 a = *reinterpret_cast<const float2*>(tab), b = *reinterpret_cast<const float2*>(tab + (rot >> 1));
+    cs[0] = a.x; cs[1] = a.y; cs[2] = b.x; cs[3] = b.y;
+  } else {
+    const bool two = d + 2 < rot;
+    cs[0] = tab[0];
+    cs[1] = two ? tab[1] : 1.f;
+    cs[2] = tab[rot >> 1];
+    cs[3] = two ? tab[(rot >> 1) + 1] : 0.f;
+  }
+}
+__device__ __forceinline__ void turn_pairs(float (&y)[4], const float (&cs)[4]) {
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {
+    const float a = y[2 * c], b = y[2 * c + 1];
+    y[2 * c] = a * cs[c] - b * cs[2 + c];
+    y[2 * c + 1] = b * cs[c] + a * cs[2 + c];
+  }
+}
+
+// prompt portions
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256, 2) conv_qkv4_kernel(const ConvQkvArgs<T> p, int per_warp) {
-  const int u = blockIdx.x * 8 + (threadIdx.x >> 5), d = (threadIdx.x & 31) * 4;
+__global__ void __launch_bounds__(256, 2) conv_qkv4_kernel(const ConvQkvArgs<T> p) {
+  const int u = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, d = lane * 4;
   if (u >= p.H + 2 * p.G) return;
   const HeadOf<T> hd(p, u);
-  const int t0 = blockIdx.y * per_warp, t1 = min(p.tokens, t0 + per_warp);
-  const bool on = d < hd.size, wr = d < hd.pad, decode = p.cu == nullptr;
-  const bool turned = on && !hd.is_v && d < p.rot, whole = p.rot % 4 == 0;
+  const int t0 = blockIdx.y * CQ_TT, t1 = min(p.tokens, t0 + CQ_TT);
+  const bool on = d < hd.size, wr = d < hd.pad, turned = on && !hd.is_v && d < p.rot;
   ConvWindow<TAPS, T> cv;
   float w[4] = {0.f, 0.f, 0.f, 0.f};
   if (on) {
     cv.weights(p.conv, hd.ch + d);
     if (!hd.is_v) ldf4((hd.is_q ? p.q_norm : p.k_norm) + d, w);
   }
-  int seq = -1;
-  for (int tb = t0; tb < t1; tb += CQ_U) {
-    float y[CQ_U][4], cs[CQ_U][4];                       // cs: two cosines, two sines
-    int sq[CQ_U], pos[CQ_U];
-    long long slot[CQ_U];
-#pragma unroll
-    for (int n = 0; n < CQ_U; ++n) {
-      const int t = min(tb + n, t1 - 1);
-      sq[n] = decode ? t : p.tok_seq[t];
-      pos[n] = p.positions[t];
-      slot[n] = hd.is_q ? -1 : p.slots[t];
-#pragma unroll
-      for (int c = 0; c < 4; ++c) y[n][c] = 0.f;
-      if (on) ldf4(p.proj + t * p.ld + hd.col + d, y[n]);
-    }
-    if (turned) {
+  const float inv_n = 1.f / (float)p.dim;
+  T* cache = hd.is_q ? nullptr : (hd.is_v ? p.v_cache : p.k_cache) + hd.h * hd.pad + d;
+  const int cache_row = p.G * hd.pad;
+  const int mine = min(t0 + lane, t1 - 1), my_pos = p.positions[mine], my_slot = hd.is_q ? -1 : (int)p.slots[mine];
+  for (int ts = t0; ts < t1;) {                          // the sequences of this run, one after the other
+    const int b = p.tok_seq[ts], first = p.cu[b], te = min(t1, p.cu[b + 1]);
+    if (on) cv.fill(p, ts, ts - first, p.start_pos[b] + ts - first, p.state_slots[b], hd.col + d, hd.ch + d);
+    const T* src = p.proj + ts * p.ld + hd.col + d;
+    T* out = hd.row(p, ts) + d;
+    for (int tb = ts; tb < te; tb += CQ_U) {
+      const int last = te - 1 - tb;                      // what is computed past it is not written
+      float y[CQ_U][4];
 #pragma unroll
       for (int n = 0; n < CQ_U; ++n) {
-        const float* tab = p.table + (long long)min(max(pos[n], 0), p.table_rows - 1) * p.rot + (d >> 1);
-        if (whole) {
-          const float2 a = *reinterpret_cast<const float2*>(tab), b = *reinterpret_cast<const float2*>(tab + (p.rot >> 1));
-          cs[n][0] = a.x; cs[n][1] = a.y; cs[n][2] = b.x; cs[n][3] = b.y;
-        } else {
-          const bool two = d + 2 < p.rot;
-          cs[n][0] = tab[0];
-          cs[n][1] = two ? tab[1] : 1.f;
-          cs[n][2] = tab[p.rot >> 1];
-          cs[n][3] = two ? tab[(p.rot >> 1) + 1] : 0.f;
+#pragma unroll
+        for (int c = 0; c < 4; ++c) y[n][c] = 0.f;
+        if (on && n <= last) ldf4(src + n * p.ld, y[n]);
+      }
+      float cs[CQ_U][4];
+      if (!hd.is_v) {
+#pragma unroll
+        for (int n = 0; n < CQ_U; ++n) {
+          const int pos = __shfl_sync(0xffffffffu, my_pos, tb - t0 + min(n, last));
+          if (turned) pair_angles(p.table + min(max(pos, 0), p.table_rows - 1) * p.rot, d, p.rot, cs[n]);
         }
       }
-    }
+      if (on) cv.template steps<CQ_U>(y);
+      if (!hd.is_v) {
+        float ss[CQ_U];
 #pragma unroll
-    for (int n = 0; n < CQ_U; ++n) {
-      const int t = tb + n;
-      if (t >= t1 || !on) continue;                      // what is past the end is not written
-      if (sq[n] != seq) {
-        seq = sq[n];
-        const long long state = p.state_slots[seq];
-        if (state < 0) cv.fill(p, t, 0, 0, 0, hd.col + d, hd.ch + d);         // a row that is not in use
-        else cv.fill(p, t, decode ? 0 : t - p.cu[seq], pos[n], state, hd.col + d, hd.ch + d);
-        if (decode && state >= 0) stf4(p.ring + (state * TAPS + pos[n] % TAPS) * p.channels + hd.ch + d, y[n]);
+        for (int n = 0; n < CQ_U; ++n) ss[n] = y[n][0] * y[n][0] + y[n][1] * y[n][1] + y[n][2] * y[n][2] + y[n][3] * y[n][3];
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+          for (int n = 0; n < CQ_U; ++n) ss[n] += __shfl_xor_sync(0xffffffffu, ss[n], o);
+#pragma unroll
+        for (int n = 0; n < CQ_U; ++n) {
+          const float inv = inv_rms<T>(ss[n], inv_n, p.eps);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) y[n][c] *= inv * w[c];
+          if (turned) turn_pairs(y[n], cs[n]);
+        }
       }
-      cv.step(y[n], y[n]);
-    }
-    if (!hd.is_v) {
-      float ss[CQ_U];
-#pragma unroll
-      for (int n = 0; n < CQ_U; ++n) ss[n] = y[n][0] * y[n][0] + y[n][1] * y[n][1] + y[n][2] * y[n][2] + y[n][3] * y[n][3];
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1)
-#pragma unroll
-        for (int n = 0; n < CQ_U; ++n) ss[n] += __shfl_xor_sync(0xffffffffu, ss[n], o);
 #pragma unroll
       for (int n = 0; n < CQ_U; ++n) {
-        const float inv = 1.f / sqrtf(ss[n] / (float)p.dim + p.eps);
-#pragma unroll
-        for (int c = 0; c < 4; ++c) y[n][c] *= inv * w[c];
-        if (turned) {
-#pragma unroll
-          for (int c = 0; c < 2; ++c) {
-            const float a = y[n][2 * c], b = y[n][2 * c + 1];
-            y[n][2 * c] = a * cs[n][c] - b * cs[n][2 + c];
-            y[n][2 * c + 1] = b * cs[n][c] + a * cs[n][2 + c];
-          }
+        const int slot = hd.is_q ? -1 : __shfl_sync(0xffffffffu, my_slot, tb - t0 + min(n, last));
+        if (n <= last && wr) {
+          stf4(out + n * p.out_ld, y[n]);
+          if (slot >= 0) stf4(cache + (long long)slot * cache_row, y[n]);
         }
       }
+      src += CQ_U * p.ld;
+      out += CQ_U * p.out_ld;
     }
+    ts = te;
+  }
+}
+
+// decode: one token per sequence, a warp per head
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256) conv_qkv4_step_kernel(const ConvQkvArgs<T> p) {
+  const int u = blockIdx.x * 8 + (threadIdx.x >> 5), d = (threadIdx.x & 31) * 4;
+  if (u >= p.H + 2 * p.G) return;
+  const HeadOf<T> hd(p, u);
+  const long long t = blockIdx.y, state = p.state_slots[t], slot = p.slots[t];
+  const int pos = p.positions[t];
+  const bool on = d < hd.size;
+  float y[4] = {0.f, 0.f, 0.f, 0.f}, x[4], cs[4];
+  if (on) {
+    ConvWindow<TAPS, T> cv;
+    ldf4(p.proj + t * p.ld + hd.col + d, x);
+    cv.weights(p.conv, hd.ch + d);
+    cv.fill(p, t, 0, state < 0 ? 0 : pos, state, hd.col + d, hd.ch + d);      // without a state: no history
+    if (state >= 0) stf4(p.ring + (state * TAPS + pos % TAPS) * p.channels + hd.ch + d, x);
+    cv.step(x, y);
+  }
+  if (!hd.is_v) {
+    if (on && d < p.rot) pair_angles(p.table + min(max(pos, 0), p.table_rows - 1) * p.rot, d, p.rot, cs);
+    const float ss = warp_sum(y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3]);
+    if (on) {
+      float w[4];
+      ldf4((hd.is_q ? p.q_norm : p.k_norm) + d, w);
+      const float inv = inv_rms<T>(ss, 1.f / (float)p.dim, p.eps);
 #pragma unroll
-    for (int n = 0; n < CQ_U; ++n) {
-      const int t = tb + n;
-      if (t < t1 && wr) {
-        T *o = hd.row(p, t), *k = hd.cached(p, slot[n]);
-        if (o != nullptr) stf4(o + d, y[n]);
-        if (k != nullptr) stf4(k + d, y[n]);
-      }
+      for (int c = 0; c < 4; ++c) y[c] *= inv * w[c];
+      if (d < p.rot) turn_pairs(y, cs);
     }
+  }
+  if (d < hd.pad) {
+    T* o = hd.is_q ? hd.row(p, t) : hd.cached(p, slot);
+    if (o != nullptr) stf4(o + d, y);
   }
 }
 
@@ -254,13 +299,18 @@ MSRL_API int msrl_conv_qkv(const void* proj, long long ld, const int* ints, cons
     p.cu = cu;
     p.start_pos = start_pos;
     p.tokens = tokens;
-    const int units = p.H + 2 * p.G, per_warp = cu == nullptr ? 1 : CQ_TT;
-    const dim3 grid((unsigned)((units + 7) / 8), (unsigned)((tokens + per_warp - 1) / per_warp));
+    const bool decode = cu == nullptr;
+    const dim3 grid((unsigned)((p.H + 2 * p.G + 7) / 8), (unsigned)(decode ? tokens : (tokens + CQ_TT - 1) / CQ_TT));
     const int odd = p.dim | p.vdim | p.qp | p.vp | p.q_col | p.k_col | p.v_col | p.oq | p.ok | p.ov | (int)(ld & 3) | (int)(out_ld & 3);
-    if ((odd & 3) == 0 && p.qp <= 128 && p.vp <= 128 && p.taps >= 2 && p.taps <= 4 && grid.y <= 65535) {
-      if (p.taps == 4) conv_qkv4_kernel<T, 4><<<grid, 256, 0, st>>>(p, per_warp);
-      else if (p.taps == 3) conv_qkv4_kernel<T, 3><<<grid, 256, 0, st>>>(p, per_warp);
-      else conv_qkv4_kernel<T, 2><<<grid, 256, 0, st>>>(p, per_warp);
+    if ((odd & 3) == 0 && (long long)p.table_rows * p.rot < (1ll << 31) && p.qp <= 128 && p.vp <= 128 && p.taps >= 2 && p.taps <= 4 &&
+        grid.y <= 65535) {
+      auto go = [&](auto prompt, auto step) {
+        if (decode) step<<<grid, 256, 0, st>>>(p);
+        else prompt<<<grid, 256, 0, st>>>(p);
+      };
+      if (p.taps == 4) go(conv_qkv4_kernel<T, 4>, conv_qkv4_step_kernel<T, 4>);
+      else if (p.taps == 3) go(conv_qkv4_kernel<T, 3>, conv_qkv4_step_kernel<T, 3>);
+      else go(conv_qkv4_kernel<T, 2>, conv_qkv4_step_kernel<T, 2>);
     } else {
       conv_qkv_kernel<T><<<(unsigned)tokens, 256, 0, st>>>(p);
     }

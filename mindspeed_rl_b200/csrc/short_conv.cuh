@@ -35,9 +35,8 @@ __device__ __forceinline__ float conv_one(const ConvIn<T>& p, long long t, int i
       x[j] = 0.f;
       if (pos - back >= 0)
         x[j] = ldf(i - back >= 0 ? p.proj + (t - back) * p.ld + col : ring + (long long)entry * p.channels);
-      if (TAPS != 4) w[j] = p.conv[(long long)ch * TAPS + j];
+      w[j] = p.conv[(long long)ch * TAPS + j];
     }
-    if constexpr (TAPS == 4) ldf4(p.conv + (long long)ch * TAPS, w);
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) s += x[j] * w[j];
   } else {
@@ -76,6 +75,26 @@ struct ConvWindow {
         if (i - back >= 0) ldf4(p.proj + (t - back) * p.ld + col, x[j + 1]);
         else ldf4(p.ring + (slot * TAPS + (pos - back) % TAPS) * p.channels + ch, x[j + 1]);
       }
+    }
+  }
+  // U >= TAPS - 1 tokens at once: nothing is shifted in between
+  template <int U>
+  __device__ __forceinline__ void steps(float (&in)[U][4]) {
+    static_assert(U >= TAPS - 1, "the window must lie inside the tokens");
+    float last[TAPS > 1 ? TAPS - 1 : 1][4];
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j) last[j][c] = in[U - (TAPS - 1) + j][c];
+#pragma unroll
+      for (int n = U - 1; n >= 0; --n) {                 // from the last on: a token's input is still there for later ones
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) s += w[j][c] * (n + j < TAPS - 1 ? x[n + j + 1][c] : in[n + j < TAPS - 1 ? 0 : n + j - (TAPS - 1)][c]);
+        in[n][c] = s;
+      }
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j) x[j + 1][c] = last[j][c];
     }
   }
   __device__ __forceinline__ void step(const float (&in)[4], float (&y)[4]) {
