@@ -88,9 +88,24 @@ __device__ __forceinline__ void turn_pairs(float (&y)[4], const float (&cs)[4]) 
   }
 }
 
-// prompt portions
+// Sums over the warp of four values per lane: lanes 8 n to 8 n + 7 end with the sum of value n.
+__device__ __forceinline__ float sum_of_four(const float (&v)[4], int lane) {
+  float two[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const float keep = lane & 16 ? v[2 + i] : v[i], give = lane & 16 ? v[i] : v[2 + i];
+    two[i] = keep + __shfl_xor_sync(0xffffffffu, give, 16);
+  }
+  const float keep = lane & 8 ? two[1] : two[0], give = lane & 8 ? two[0] : two[1];
+  float s = keep + __shfl_xor_sync(0xffffffffu, give, 8);
+#pragma unroll
+  for (int o = 4; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+  return s;
+}
+
+// prompt portions: the tokens of a sequence follow one another from start_pos on
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256, 2) conv_qkv4_kernel(const ConvQkvArgs<T> p) {
+__global__ void __launch_bounds__(256, 3) conv_qkv4_kernel(const ConvQkvArgs<T> p) {
   const int u = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, d = lane * 4;
   if (u >= p.H + 2 * p.G) return;
   const HeadOf<T> hd(p, u);
@@ -105,10 +120,11 @@ __global__ void __launch_bounds__(256, 2) conv_qkv4_kernel(const ConvQkvArgs<T> 
   const float inv_n = 1.f / (float)p.dim;
   T* cache = hd.is_q ? nullptr : (hd.is_v ? p.v_cache : p.k_cache) + hd.h * hd.pad + d;
   const int cache_row = p.G * hd.pad;
-  const int mine = min(t0 + lane, t1 - 1), my_pos = p.positions[mine], my_slot = hd.is_q ? -1 : (int)p.slots[mine];
+  const int mine = min(t0 + lane, t1 - 1), my_slot = hd.is_q ? -1 : (int)p.slots[mine];
   for (int ts = t0; ts < t1;) {                          // the sequences of this run, one after the other
     const int b = p.tok_seq[ts], first = p.cu[b], te = min(t1, p.cu[b + 1]);
-    if (on) cv.fill(p, ts, ts - first, p.start_pos[b] + ts - first, p.state_slots[b], hd.col + d, hd.ch + d);
+    int pos = p.start_pos[b] + ts - first;
+    if (on) cv.fill(p, ts, ts - first, pos, p.state_slots[b], hd.col + d, hd.ch + d);
     const T* src = p.proj + ts * p.ld + hd.col + d;
     T* out = hd.row(p, ts) + d;
     for (int tb = ts; tb < te; tb += CQ_U) {
@@ -120,30 +136,24 @@ __global__ void __launch_bounds__(256, 2) conv_qkv4_kernel(const ConvQkvArgs<T> 
         for (int c = 0; c < 4; ++c) y[n][c] = 0.f;
         if (on && n <= last) ldf4(src + n * p.ld, y[n]);
       }
-      float cs[CQ_U][4];
-      if (!hd.is_v) {
-#pragma unroll
-        for (int n = 0; n < CQ_U; ++n) {
-          const int pos = __shfl_sync(0xffffffffu, my_pos, tb - t0 + min(n, last));
-          if (turned) pair_angles(p.table + min(max(pos, 0), p.table_rows - 1) * p.rot, d, p.rot, cs[n]);
-        }
-      }
       if (on) cv.template steps<CQ_U>(y);
       if (!hd.is_v) {
         float ss[CQ_U];
 #pragma unroll
         for (int n = 0; n < CQ_U; ++n) ss[n] = y[n][0] * y[n][0] + y[n][1] * y[n][1] + y[n][2] * y[n][2] + y[n][3] * y[n][3];
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1)
-#pragma unroll
-          for (int n = 0; n < CQ_U; ++n) ss[n] += __shfl_xor_sync(0xffffffffu, ss[n], o);
+        const float inv = inv_rms<T>(sum_of_four(ss, lane), inv_n, p.eps);      // of token lane / 8
 #pragma unroll
         for (int n = 0; n < CQ_U; ++n) {
-          const float inv = inv_rms<T>(ss[n], inv_n, p.eps);
+          const float r = __shfl_sync(0xffffffffu, inv, n * 8);
 #pragma unroll
-          for (int c = 0; c < 4; ++c) y[n][c] *= inv * w[c];
-          if (turned) turn_pairs(y[n], cs[n]);
+          for (int c = 0; c < 4; ++c) y[n][c] *= r * w[c];
+          if (turned) {
+            float cs[4];
+            pair_angles(p.table + min(pos + n, p.table_rows - 1) * p.rot, d, p.rot, cs);
+            turn_pairs(y[n], cs);
+          }
         }
+        pos += CQ_U;
       }
 #pragma unroll
       for (int n = 0; n < CQ_U; ++n) {
