@@ -88,7 +88,8 @@ def test_grpo_lora_cpu():
     from mindspeed_rl_b200.trainer.grpo_trainer import RayGRPOTrainer
 
     torch.manual_seed(0)
-    actor, rl, gen = build(n_prompts=4, n_samples=4, max_tokens=16, iters=2)
+    # enough tokens that some response earns the reward (one token in a thousand does), whatever the CPU's rounding draws
+    actor, rl, gen = build(n_prompts=8, n_samples=8, max_tokens=64, iters=2)
     actor.lora_r, actor.lora_alpha = 4, 8
     actor.lora_target_modules = ["linear_qkv", "linear_proj", "linear_fc1", "linear_fc2"]
     actor.lr = 1e-2
@@ -99,8 +100,8 @@ def test_grpo_lora_cpu():
     before = {k: v.clone() for k, v in core.state_dict().items()}
     trainer = RayGRPOTrainer(group, reward_list=[RuleReward(rl, None, actor)], train_iters=2, save_interval=0,
                              adv_estimator="group_norm", kl_penalty="low_var_kl", init_kl_coef=0.001,
-                             global_batch_size=4, n_samples_per_prompt=4, pad_token_id=0)
-    hist = trainer.fit(iter(SyntheticPromptLoader(4, 32, 1024, seed=0)))
+                             global_batch_size=8, n_samples_per_prompt=8, pad_token_id=0)
+    hist = trainer.fit(iter(SyntheticPromptLoader(8, 32, 1024, seed=0)))
     assert len(hist) == 2 and "actor/kl_loss" in hist[0]
     after = core.state_dict()
     moved = [k for k in before if not torch.equal(before[k], after[k])]
