@@ -18,6 +18,7 @@
 //   decode:  one fused kernel per (sequence, head): all of the above with S read and written once, coalesced.
 //
 // Both sum (S^T k, S^T q) over the decayed state in one pass: o = (gS)^T q + (k.q) u.
+#include "packed_f32.cuh"
 #include "short_conv.cuh"
 
 namespace msrl {
@@ -319,29 +320,6 @@ __device__ __forceinline__ void cp_async4(void* smem, const void* gmem) {
 }
 __device__ __forceinline__ void cp_async16b(void* smem, const void* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_u32(smem)), "l"(gmem));
-}
-
-// two fp32 lanes per instruction (each lane rounds like the scalar operation)
-using f2 = unsigned long long;
-__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
-  f2 d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
-  f2 d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ f2 pack2(float lo, float hi) {
-  f2 d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ float2 unpack2(f2 a) {
-  float2 r;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(a));
-  return r;
 }
 
 constexpr int SCAN_TB = 16;      // tokens staged at a time

@@ -7,6 +7,9 @@
 //   o = S'^T q / (max(|n' . q|, e^-m') + floor)            (q carries `scale`)
 //   y = o / rms(o) * norm * sigmoid(gate)
 //
+// or, with a constant decay per head in place of the gates (linear attention),  S' = decay S + k v^T,  o = S'^T q.  The output
+// gate is a sigmoid or a silu.
+//
 // What a sequence carries lives in a state slot (memory [slots, H, dim, vdim], norm [slots, H, dim], peak [slots, H]); the
 // first token of a sequence ignores what the slot holds.
 //
@@ -52,20 +55,29 @@ __global__ void __launch_bounds__(256) decode_kernel(const Args<T> p) {
   float* sq = sm;
   float* sk = sm + p.dim;
   const T* row = p.proj + b * p.ld;
+  const bool plain = p.decay != nullptr;
   float* nr = p.nrm + (slot * p.H + h) * p.dim;
-  float gi, gf;
-  log_gates(p, b, h, gi, gf);
-  const float m0 = fresh ? 0.f : p.peak[slot * p.H + h];
-  const float m = fmaxf(gf + m0, gi);
-  const float keep = fresh ? 0.f : expf(gf + m0 - m), take = expf(gi - m);
+  float m = 0.f, keep = 0.f, take = 1.f;
+  if (plain) {
+    if (!fresh) keep = p.decay[h];
+  } else {
+    float gi, gf;
+    log_gates(p, b, h, gi, gf);
+    const float m0 = fresh ? 0.f : p.peak[slot * p.H + h];
+    m = fmaxf(gf + m0, gi);
+    if (!fresh) keep = expf(gf + m0 - m);
+    take = expf(gi - m);
+  }
   float nq = 0.f;
   for (int d = threadIdx.x; d < p.dim; d += 256) {
     const float q = ldf(row + p.q_col + h * p.dim + d) * p.scale, k = take * ldf(row + p.k_col + h * p.dim + d);
     sq[d] = q;
     sk[d] = k;
-    nq += q * (fresh ? k : keep * nr[d] + k);
+    if (!plain) nq += q * (fresh ? k : keep * nr[d] + k);
   }
-  const float den = fmaxf(fabsf(block_sum(nq, red)), expf(-m)) + p.floor;     // (synchronises sq, sk)
+  float den = 1.f;
+  if (plain) __syncthreads();            // sq, sk
+  else den = fmaxf(fabsf(block_sum(nq, red)), expf(-m)) + p.floor;
   const int quads = width / 4, lanes = 256 / quads;
   const int cq = threadIdx.x % quads, rl = threadIdx.x / quads;
   float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -123,7 +135,7 @@ __global__ void __launch_bounds__(256) decode_kernel(const Args<T> p) {
   } else {
     __syncthreads();
   }
-  if (blockIdx.x == 0) {
+  if (blockIdx.x == 0 && !plain) {
     for (int d = threadIdx.x; d < p.dim; d += 256) nr[d] = fresh ? sk[d] : keep * nr[d] + sk[d];
     if (threadIdx.x == 0) p.peak[slot * p.H + h] = m;
   }
@@ -131,7 +143,10 @@ __global__ void __launch_bounds__(256) decode_kernel(const Args<T> p) {
 #pragma unroll
   for (int i = 0; i < DC; ++i) {
     const int x = threadIdx.x + i * 256, c = h * p.vdim + c0 + x;
-    if (x < width) stf(y + x, val[i] * inv * p.norm[c] * sigmoid_f(ldf(row + p.g_col + c)));
+    if (x < width) {
+      const float g = ldf(row + p.g_col + c);
+      stf(y + x, val[i] * inv * p.norm[c] * out_gate(p, g, sigmoid_f(g)));
+    }
   }
 }
 
@@ -150,8 +165,8 @@ __global__ void __launch_bounds__(256) scan_kernel(const Args<T> p, float* o) {
   if (len <= 0) return;
   const int lane8 = threadIdx.x & 7, col = threadIdx.x >> 3, c = c0 + col;
   const long long slot = p.slots[b];
-  const bool old = p.start[b] > 0 && slot >= 0;
-  float S[NR], n[NR], m = old ? p.peak[slot * p.H + h] : 0.f;
+  const bool old = p.start[b] > 0 && slot >= 0, plain = p.decay != nullptr;
+  float S[NR], n[NR], m = old && !plain ? p.peak[slot * p.H + h] : 0.f;
   float* Sg = p.memory + (slot * p.H + h) * p.dim * p.vdim;
   float* ng = p.nrm + (slot * p.H + h) * p.dim;
 #pragma unroll
@@ -159,7 +174,7 @@ __global__ void __launch_bounds__(256) scan_kernel(const Args<T> p, float* o) {
     const int r = lane8 + 8 * i;
     const bool in = old && r < p.dim;
     S[i] = in && c < p.vdim ? Sg[(long long)r * p.vdim + c] : 0.f;
-    n[i] = in ? ng[r] : 0.f;
+    n[i] = in && !plain ? ng[r] : 0.f;
   }
   for (int base = 0; base < len; base += ST) {
     const int nt = min(ST, len - base);
@@ -177,9 +192,15 @@ __global__ void __launch_bounds__(256) scan_kernel(const Args<T> p, float* o) {
     if (threadIdx.x < nt) log_gates(p, t0 + base + threadIdx.x, h, sg[threadIdx.x][1], sg[threadIdx.x][0]);
     __syncthreads();
     for (int s = 0; s < nt; ++s) {
-      const float gi = sg[s][1], gf = sg[s][0];
-      const float top = fmaxf(gf + m, gi), keep = expf(gf + m - top), take = expf(gi - top);
-      m = top;
+      float keep = 0.f, take = 1.f;
+      if (plain) {
+        keep = p.decay[h];
+      } else {
+        const float gi = sg[s][1], gf = sg[s][0], top = fmaxf(gf + m, gi);
+        keep = expf(gf + m - top);
+        take = expf(gi - top);
+        m = top;
+      }
       const float v = sv[s][col] * take;
       float acc = 0.f, nq = 0.f;
 #pragma unroll
@@ -199,7 +220,7 @@ __global__ void __launch_bounds__(256) scan_kernel(const Args<T> p, float* o) {
         nq += __shfl_xor_sync(0xffffffffu, nq, x);
       }
       if (lane8 == 0 && c < p.vdim)
-        o[((long long)(t0 + base + s) * p.H + h) * p.vdim + c] = acc / (fmaxf(fabsf(nq), expf(-m)) + p.floor);
+        o[((long long)(t0 + base + s) * p.H + h) * p.vdim + c] = plain ? acc : acc / (fmaxf(fabsf(nq), expf(-m)) + p.floor);
     }
   }
   if (slot < 0) return;
@@ -272,7 +293,7 @@ __global__ void __launch_bounds__(256) finish_kernel(const Args<T> p, const floa
     ldf4(p.proj + t * p.ld + p.g_col + h * p.vdim + c, g);
     ldf4(p.norm + h * p.vdim + c, w);
 #pragma unroll
-    for (int i = 0; i < 4; ++i) f[i] *= inv * w[i] * sigmoid_t<T>(g[i]);
+    for (int i = 0; i < 4; ++i) f[i] *= inv * w[i] * out_gate(p, g[i], sigmoid_t<T>(g[i]));
     stf4(p.y + r * p.vdim + c, f);
   }
 }
@@ -290,7 +311,7 @@ __global__ void __launch_bounds__(256) carry_kernel(const Args<bf16> p, const Ch
   const int h = blockIdx.y, b = blockIdx.z;
   const int t0 = p.cu[b], len = p.cu[b + 1] - t0, n = (len + C - 1) / C;
   const long long size = (long long)p.dim * p.vdim, e = ((long long)blockIdx.x * 256 + threadIdx.x) * 4;
-  if (len <= 0 || e >= size + p.dim) return;
+  if (len <= 0 || e >= size + (p.decay != nullptr ? 0 : p.dim)) return;
   const long long slot = p.slots[b], id0 = chunk_id(t0, b, 0) * p.H + h;
   const bool old = p.start[b] > 0 && slot >= 0;
   float* mine = e < size ? p.memory + (slot * p.H + h) * size + e : p.nrm + (slot * p.H + h) * p.dim + (e - size);
@@ -298,7 +319,7 @@ __global__ void __launch_bounds__(256) carry_kernel(const Args<bf16> p, const Ch
   float m = 0.f;
   if (old) {
     s = *reinterpret_cast<const float4*>(mine);
-    m = p.peak[slot * p.H + h];
+    if (p.decay == nullptr) m = p.peak[slot * p.H + h];
   }
   float* u = ch.state + id0 * (size + p.dim) + e;
   const long long step = p.H * (size + p.dim);
@@ -345,11 +366,12 @@ __global__ void carry_peak_kernel(const Args<bf16> p, const Chunks ch, int batch
 
 using namespace msrl;
 
-// ints: H, dim, vdim (multiples of 16), entries of a head that count in its root mean square, columns of q, k, v, gate;
+// ints: H, dim, vdim (multiples of 16), entries of a head that count in its root mean square, columns of q, k, v, gate,
+// silu gate; decay: see matrix_memory.cuh;
 // floats: scale, cap, floor, eps
 MSRL_API int msrl_memory_decode(const void* proj, long long ld, const float* z, long long z_ld, const int* ints,
-                                const float* floats, const float* bias, const float* norm, float* memory, float* nrm,
-                                float* peak, const int* positions, const long long* slots, void* y, int batch, int is_f32,
+                                const float* floats, const float* bias, const float* decay, const float* norm,
+                                float* memory, float* nrm, float* peak, const int* positions, const long long* slots, void* y, int batch, int is_f32,
                                 cudaStream_t st) {
   if (batch == 0) return 0;
   const int H = ints[0], dim = ints[1], vdim = ints[2];
@@ -362,7 +384,7 @@ MSRL_API int msrl_memory_decode(const void* proj, long long ld, const float* z, 
   if (vdim / slices > 256 * mem::DC) return (int)cudaErrorNotSupported;
   auto run = [&](auto tag) {
     using T = decltype(tag);
-    const auto p = mem::make_args<T>(proj, ld, z, z_ld, ints, floats, bias, norm, memory, nrm, peak, nullptr, positions,
+    const auto p = mem::make_args<T>(proj, ld, z, z_ld, ints, floats, bias, decay, norm, memory, nrm, peak, nullptr, positions,
                                      slots, y);
     cudaLaunchConfig_t cfg{};
     cfg.gridDim = dim3((unsigned)slices, (unsigned)H, (unsigned)batch);
@@ -382,15 +404,15 @@ MSRL_API int msrl_memory_decode(const void* proj, long long ld, const float* z, 
 
 // o: fp32 scratch [tokens, H * vdim]
 MSRL_API int msrl_memory_prefill(const void* proj, long long ld, const float* z, long long z_ld, const int* ints,
-                                 const float* floats, const float* bias, const float* norm, float* memory, float* nrm,
-                                 float* peak, const int* cu, const int* start, const long long* slots, float* o, void* y,
+                                 const float* floats, const float* bias, const float* decay, const float* norm,
+                                 float* memory, float* nrm, float* peak, const int* cu, const int* start, const long long* slots, float* o, void* y,
                                  int tokens, int batch, int is_f32, cudaStream_t st) {
   if (batch == 0 || tokens == 0) return 0;
   const int H = ints[0], dim = ints[1], vdim = ints[2];
   if (dim > 512 || dim % 16 != 0 || vdim % 16 != 0 || batch > 65535 || H > 65535) return (int)cudaErrorNotSupported;
   auto run = [&](auto tag) {
     using T = decltype(tag);
-    const auto p = mem::make_args<T>(proj, ld, z, z_ld, ints, floats, bias, norm, memory, nrm, peak, cu, start, slots, y);
+    const auto p = mem::make_args<T>(proj, ld, z, z_ld, ints, floats, bias, decay, norm, memory, nrm, peak, cu, start, slots, y);
     const dim3 grid((unsigned)((vdim + mem::SC - 1) / mem::SC), (unsigned)H, (unsigned)batch);
     const size_t smem = 2 * mem::ST * (size_t)dim * sizeof(float);
     auto go = [&](auto kernel) {
@@ -402,7 +424,7 @@ MSRL_API int msrl_memory_prefill(const void* proj, long long ld, const float* z,
     const int rc = dim <= 64 ? go(mem::scan_kernel<T, 8>) : dim <= 128 ? go(mem::scan_kernel<T, 16>)
                    : dim <= 256 ? go(mem::scan_kernel<T, 32>) : go(mem::scan_kernel<T, 64>);
     if (rc != 0) return rc;
-    mem::scan_norm_kernel<T><<<dim3((unsigned)H, (unsigned)batch), 256, 0, st>>>(p);
+    if (decay == nullptr) mem::scan_norm_kernel<T><<<dim3((unsigned)H, (unsigned)batch), 256, 0, st>>>(p);
     const long long rows = (long long)tokens * H;
     mem::finish_kernel<T><<<(unsigned)((rows + 7) / 8), 256, 0, st>>>(p, o, rows);
     return (int)cudaGetLastError();
@@ -428,8 +450,8 @@ int launch_chunk_out(const Args<__nv_bfloat16>& p, const Chunks& ch, int most, i
 
 // The same for bf16 rows, in chunks; column starts and ld are multiples of 8.  error: device status word (0 = ok)
 MSRL_API int msrl_memory_prefill_chunked(const void* proj, long long ld, const float* z, long long z_ld, const int* ints,
-                                         const float* floats, const float* bias, const float* norm, float* memory,
-                                         float* nrm, float* peak, const int* cu, const int* start, const long long* slots,
+                                         const float* floats, const float* bias, const float* decay, const float* norm,
+                                         float* memory, float* nrm, float* peak, const int* cu, const int* start, const long long* slots,
                                          float* scratch, void* y, int tokens, int batch, int max_q, int* error,
                                          cudaStream_t st) {
   if (batch == 0 || tokens == 0) return 0;
@@ -437,7 +459,7 @@ MSRL_API int msrl_memory_prefill_chunked(const void* proj, long long ld, const f
   if (!msrl_memory_chunked_serves(ints) || ld % 8 != 0 || batch > 65535 || H > 65535) return (int)cudaErrorNotSupported;
   for (int i = 4; i < 8; ++i)
     if (ints[i] % 8 != 0) return (int)cudaErrorNotSupported;
-  const auto p = mem::make_args<__nv_bfloat16>(proj, ld, z, z_ld, ints, floats, bias, norm, memory, nrm, peak, cu, start,
+  const auto p = mem::make_args<__nv_bfloat16>(proj, ld, z, z_ld, ints, floats, bias, decay, norm, memory, nrm, peak, cu, start,
                                                slots, y);
   const long long chunks = tokens / mem::C + batch, size = (long long)dim * vdim + dim;
   mem::Chunks ch{};
@@ -455,7 +477,7 @@ MSRL_API int msrl_memory_prefill_chunked(const void* proj, long long ld, const f
   int rc = mem::launch_chunk_state(p, ch, most, batch, error, st);
   if (rc != 0) return rc;
   mem::carry_kernel<<<dim3((unsigned)((size + 1023) / 1024), (unsigned)H, (unsigned)batch), 256, 0, st>>>(p, ch);
-  mem::carry_peak_kernel<<<(unsigned)(((long long)batch * H + 127) / 128), 128, 0, st>>>(p, ch, batch);
+  if (decay == nullptr) mem::carry_peak_kernel<<<(unsigned)(((long long)batch * H + 127) / 128), 128, 0, st>>>(p, ch, batch);
   rc = mem::launch_chunk_out(p, ch, most, batch, error, st);
   if (rc != 0 || vdim <= 128) return rc;
   const long long rows = (long long)tokens * H;

@@ -12,8 +12,11 @@ struct Args {
   const float* z;                        // [tokens, z_ld]: input gate logits [H] | forget gate logits [H]
   long long z_ld;
   int H, dim, vdim, rms_dim, q_col, k_col, v_col, g_col;
+  int silu;                              // the output gate: silu, else sigmoid
   float scale, cap, floor, eps;
   const float* bias;                     // [2 H]
+  const float* decay;                    // [2 H]: a constant decay per head and its logarithm, or null.  With it there are no
+                                         // gates (i = 0, so m stays zero) and no denominator; z, bias, nrm and peak are unused
   const float* norm;                     // [H * vdim]
   float *memory, *nrm, *peak;
   const int* cu;
@@ -24,6 +27,11 @@ struct Args {
 
 template <typename T>
 __device__ __forceinline__ void log_gates(const Args<T>& p, long long t, int h, float& i, float& f) {
+  if (p.decay != nullptr) {
+    i = 0.f;
+    f = p.decay[p.H + h];
+    return;
+  }
   const float* z = p.z + t * p.z_ld + h;
   i = p.cap * tanhf((z[0] + p.bias[h]) / p.cap);
   const float x = p.cap * tanhf((z[p.H] + p.bias[p.H + h]) / p.cap);
@@ -31,11 +39,14 @@ __device__ __forceinline__ void log_gates(const Args<T>& p, long long t, int h, 
 }
 
 template <typename T>
+__device__ __forceinline__ float out_gate(const Args<T>& p, float g, float s) { return p.silu ? g * s : s; }   // s = sigmoid(g)
+
+template <typename T>
 Args<T> make_args(const void* proj, long long ld, const float* z, long long z_ld, const int* ints, const float* floats,
-                  const float* bias, const float* norm, float* memory, float* nrm, float* peak, const int* cu,
-                  const int* start, const long long* slots, void* y) {
+                  const float* bias, const float* decay, const float* norm, float* memory, float* nrm, float* peak,
+                  const int* cu, const int* start, const long long* slots, void* y) {
   return Args<T>{(const T*)proj, ld, z, z_ld, ints[0], ints[1], ints[2], ints[3], ints[4], ints[5], ints[6], ints[7],
-                 floats[0], floats[1], floats[2], floats[3], bias, norm, memory, nrm, peak, cu, start, slots, (T*)y};
+                 ints[8], floats[0], floats[1], floats[2], floats[3], bias, decay, norm, memory, nrm, peak, cu, start, slots, (T*)y};
 }
 
 // bf16 prompts in chunks of C tokens

@@ -332,7 +332,8 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
   };
   if (inter) {
     fetch(0);
-    for (int d = threadIdx.x; d < p.dim; d += 256) sN[d] = S[size + d];
+    if (p.decay == nullptr)
+      for (int d = threadIdx.x; d < p.dim; d += 256) sN[d] = S[size + d];
   }
   if (threadIdx.x < C) {
     const int s = threadIdx.x;
@@ -397,7 +398,7 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
       }
       __syncwarp();
     }
-    if (ok) {
+    if (ok && p.decay == nullptr) {
       // q . n of every row, two threads a row
       const int r = threadIdx.x >> 1;
       float s = 0.f;
@@ -409,8 +410,8 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
       }
       s += __shfl_xor_sync(0xffffffffu, s, 1);
       if ((threadIdx.x & 1) == 0) sDen[r] = s;
-      ok = mbar_wait_warp(&q_done, ((p.dim + TB - 1) / TB - 1) & 1, error, ERR_Q);
     }
+    if (ok) ok = mbar_wait_warp(&q_done, ((p.dim + TB - 1) / TB - 1) & 1, error, ERR_Q);
   }
   ok = ok && mbar_wait_warp(&s_full, 0, error, ERR_S);
   ok = __syncthreads_and(ok);            // Q, K and the state terms are read, sDen is written
@@ -500,10 +501,13 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
   }
   if (ok) {
     fence_after();
-    float den = part[0][row] + part[1][row];
     const float weight = sInter[row];
-    if (inter) den += weight * sDen[row];
-    const float inv = 1.f / (fmaxf(fabsf(den), sExp[row]) + p.floor);
+    float inv = 1.f;
+    if (p.decay == nullptr) {
+      float den = part[0][row] + part[1][row];
+      if (inter) den += weight * sDen[row];
+      inv = 1.f / (fmaxf(fabsf(den), sExp[row]) + p.floor);
+    }
     float o[2][32], ss = 0.f;            // the thread's row, its half of the columns
 #pragma unroll
     for (int c = 0; c < 2; ++c) {
@@ -562,8 +566,10 @@ __global__ void __launch_bounds__(256, 2) chunk_out_kernel(const Args<bf16> p, c
           } else {
             const float2 g0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[it].x));
             const float2 g1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[it].y));
-            const float y[4] = {f.x * wn[0] * sigmoid_t<bf16>(g0.x), f.y * wn[1] * sigmoid_t<bf16>(g0.y),
-                                f.z * wn[2] * sigmoid_t<bf16>(g1.x), f.w * wn[3] * sigmoid_t<bf16>(g1.y)};
+            const float y[4] = {f.x * wn[0] * out_gate(p, g0.x, sigmoid_t<bf16>(g0.x)),
+                                f.y * wn[1] * out_gate(p, g0.y, sigmoid_t<bf16>(g0.y)),
+                                f.z * wn[2] * out_gate(p, g1.x, sigmoid_t<bf16>(g1.x)),
+                                f.w * wn[3] * out_gate(p, g1.y, sigmoid_t<bf16>(g1.y))};
             stf4(p.y + at, y);
           }
         }

@@ -7,7 +7,7 @@
 //             Slots with an id outside the experts have no row (destination -1).
 //   permute   x[token] (optionally scaled by the slot's weight) -> rows of the expert-grouped
 //             buffer; pad rows of every segment are zeroed.
-//   route_top the experts of the largest sigmoid scores of every token, with their scores
+//   route_top the experts of the largest logits of every token, with their sigmoids or the soft-max over those chosen
 //   route_softmax_top  those of the largest soft-max score plus correction, with their scores
 //   combine   out[token] = sum_k w[token, k] * y[row(token, k)]   (fp32 accumulation; w optional)
 //   slot_dot  dw[token, k] = <dout[token], y[row(token, k)]>      (gradient of the combine weights)
@@ -152,8 +152,9 @@ moe_permute_f32_kernel(const float* x, const int* pos, const float* w, int T, in
 }
 
 // One warp per token.  Logits stay in registers (NPL per lane) as integers of the same order; the largest is taken out
-// `top` times.  They are ordered by logit: the sigmoid is monotone but saturates.
-template <int NPL>
+// `top` times.  They are ordered by logit: the sigmoid is monotone but saturates.  CHOSEN: scores are a soft-max over the
+// logits taken.
+template <int NPL, bool CHOSEN>
 __global__ void __launch_bounds__(256)
 route_top_kernel(const float* logits, int T, int E, int top, long long* idx, float* score) {
   const long long t = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -168,6 +169,7 @@ route_top_kernel(const float* logits, int T, int E, int top, long long* idx, flo
       key[n] = max(b & 0x80000000u ? ~b : b | 0x80000000u, 1u);
     }
   }
+  float largest = 0.f, sum = 0.f;
   for (int j = 0; j < top; ++j) {
     unsigned mine = 0;
 #pragma unroll
@@ -181,11 +183,18 @@ route_top_kernel(const float* logits, int T, int E, int top, long long* idx, flo
 #pragma unroll
     for (int n = 0; n < NPL; ++n)
       if (n * 32 + lane == first) key[n] = 0;
+    const float z = __uint_as_float(best & 0x80000000u ? best & 0x7fffffffu : ~best);
+    if (j == 0) largest = z;
+    const float e = CHOSEN ? expf(z - largest) : 1.f / (1.f + expf(-z));
+    sum += e;
     if (lane == 0) {
-      const float z = __uint_as_float(best & 0x80000000u ? best & 0x7fffffffu : ~best);
       idx[t * top + j] = first;
-      score[t * top + j] = 1.f / (1.f + expf(-z));
+      score[t * top + j] = e;
     }
+  }
+  if constexpr (CHOSEN) {
+    __syncwarp();
+    for (int j = lane; j < top; j += 32) score[t * top + j] /= sum;
   }
 }
 
@@ -327,15 +336,20 @@ MSRL_API int msrl_moe_permute_f32(const float* x, const int* pos, const float* w
   return (int)cudaGetLastError();
 }
 
-// logits [T, E] -> idx, score [T, top]; at most 1024 experts
-MSRL_API int msrl_route_top(const float* logits, int T, int E, int top, long long* idx, float* score, cudaStream_t st) {
+// logits [T, E] -> idx, score [T, top]; at most 1024 experts.  chosen: scores are a soft-max over the chosen logits
+MSRL_API int msrl_route_top(const float* logits, int T, int E, int top, long long* idx, float* score, int chosen,
+                            cudaStream_t st) {
   if (T == 0) return 0;
   if (E < 1 || E > 1024 || top < 1 || top > E) return (int)cudaErrorInvalidValue;
   const unsigned grid = (unsigned)((T + 7) / 8);
-  if (E <= 64) route_top_kernel<2><<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
-  else if (E <= 256) route_top_kernel<8><<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
-  else route_top_kernel<32><<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
-  return (int)cudaGetLastError();
+  auto go = [&](auto few, auto some, auto many) {
+    if (E <= 64) few<<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
+    else if (E <= 256) some<<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
+    else many<<<grid, 256, 0, st>>>(logits, T, E, top, idx, score);
+    return (int)cudaGetLastError();
+  };
+  return chosen ? go(route_top_kernel<2, true>, route_top_kernel<8, true>, route_top_kernel<32, true>)
+                : go(route_top_kernel<2, false>, route_top_kernel<8, false>, route_top_kernel<32, false>);
 }
 
 // logits [T, E], correction [E] -> idx, score [T, top]; at most 1024 router outputs

@@ -10,7 +10,14 @@
 // residual they just wrote).  A null `y` skips the norm; without a norm weight y is the residual itself.
 //
 //   post_add          d = delta[t], or sum_j w[t, j] * e[pos(t, j)] + sh[t] where a negative pos stands for the residual's
-//                     row; resid[t] += mult * d / sqrt(mean(d^2) + eps) * weight;  y[t] = resid[t] or a norm of it
+//                     row; resid[t] += mult * d / sqrt(mean(d^2) + eps) * weight;  y[t] = resid[t] or a norm of it.
+//                     Between the add and y: resid[t] += again[t] + step (what a pass of a loop adds before it runs)
+//   post_embed        the same with d = table[id[t]] and a residual that starts at zero; `first` keeps it as it was before
+//                     `step`
+//   side_add          the same with d = proj (gelu_tanh(gate resid[t]) * rows[id[t]]), one block per token from the gate to
+//                     the norm; for few tokens
+//   side_gate         g[t] = gelu_tanh(g[t]) * rows[id[t]]  (many tokens: gate and proj are matrix products)
+//   soft_cap          x = cap * tanh(x / cap)
 //
 //   glu               act(gate) * up of rows [gate | up]: silu, tanh-gelu, or the clamped swish with (up + 1)
 #include "dtype_utils.cuh"
@@ -215,6 +222,8 @@ int launch_row_norm(const RowArgs<T>& p, long long rows, cudaStream_t st) {
   return p.centered || p.delta2 != nullptr ? launch_rows<T, SRC, true>(p, rows, st) : launch_rows<T, SRC, false>(p, rows, st);
 }
 
+enum { POST_ROWS = 0, POST_MOE = 1, POST_EMBED = 2 };
+
 template <typename T>
 struct PostArgs {
   const T* delta;                         // the sublayer's rows, or null:
@@ -230,20 +239,69 @@ struct PostArgs {
   float after_eps;
   T* y;
   int W;
+  const float* again;                     // ENTRY: [rows, W] and
+  const float* step;                      // [W] that the sum gets before its norm, or null
+  const long long* ids;                   // POST_EMBED
+  const T* table;
+  float* first;                           // [rows, W] or null
 };
 
+// adds the normed values to the residual (and, with ENTRY, what a pass adds); the sum stays in `a`
+template <typename T, int V, bool ENTRY>
+__device__ __forceinline__ void post_sum(const PostArgs<T>& p, long long t, int c, float inv, const float (&b)[4], float (&a)[4],
+                                         float& sum) {
+  const long long at = t * p.W + c;
+  float w[4];
+  ldv<V>(p.norm_w + c, w);
+#pragma unroll
+  for (int i = 0; i < V; ++i) a[i] += b[i] * inv * w[i];
+  if constexpr (ENTRY) {
+    if (p.first != nullptr) stv<V>(p.first + at, a);
+    if (p.again != nullptr) {
+      ldv<V>(p.again + at, w);
+#pragma unroll
+      for (int i = 0; i < V; ++i) a[i] += w[i];
+    }
+    if (p.step != nullptr) {
+      ldv<V>(p.step + c, w);
+#pragma unroll
+      for (int i = 0; i < V; ++i) a[i] += w[i];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < V; ++i) sum += a[i] * a[i];
+  stv<V>(p.resid + at, a);
+  if (p.after_w == nullptr) stv<V>(p.y + at, a);
+}
+
+template <typename T, int V>
+__device__ __forceinline__ void post_after(const PostArgs<T>& p, long long t, int c, float q, const float (&a)[4]) {
+  float w[4];
+  ldv<V>(p.after_w + c, w);
+#pragma unroll
+  for (int i = 0; i < V; ++i) w[i] *= a[i] * q;
+  stv<V>(p.y + t * p.W + c, w);
+}
+
 // One block per row.  Rows up to NPT * 256 * V entries stay in registers; what is longer is computed again.
-template <typename T, int V, int NPT, bool MOE>
+template <typename T, int V, int NPT, int SRC, bool ENTRY>
 __global__ void __launch_bounds__(RS_THREADS) post_add_kernel(const PostArgs<T> p) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   const int W = p.W;
   float* res = p.resid + t * W;
-  T* y = p.y + t * W;
+  const T* rows = nullptr;
+  if constexpr (SRC == POST_ROWS) rows = p.delta + t * W;
+  if constexpr (SRC == POST_EMBED) rows = p.table + p.ids[t] * W;
   auto value = [&](int c, float (&r)[4], float (&d)[4]) {     // the residual's entries and the sublayer's
-    ldv<V>(res + c, r);
-    if constexpr (!MOE) {
-      ldv<V>(p.delta + t * W + c, d);
+    if constexpr (SRC == POST_EMBED) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) r[i] = 0.f;
+    } else {
+      ldv<V>(res + c, r);
+    }
+    if constexpr (SRC != POST_MOE) {
+      ldv<V>(rows + c, d);
     } else {
 #pragma unroll
       for (int i = 0; i < V; ++i) d[i] = 0.f;
@@ -282,73 +340,167 @@ __global__ void __launch_bounds__(RS_THREADS) post_add_kernel(const PostArgs<T> 
   }
   const float inv = p.mult / sqrtf(block_sum(ss, red) / (float)W + p.eps);
   float sum = 0.f;
-  auto add = [&](int c, float (&a)[4], const float (&b)[4]) {
-    float w[4];
-    ldv<V>(p.norm_w + c, w);
-#pragma unroll
-    for (int i = 0; i < V; ++i) {
-      a[i] += b[i] * inv * w[i];
-      sum += a[i] * a[i];
-    }
-    stv<V>(res + c, a);
-    if (p.after_w == nullptr) stv<V>(y + c, a);
-  };
 #pragma unroll
   for (int k = 0; k < NPT; ++k) {
     const int c = (k * RS_THREADS + threadIdx.x) * V;
-    if (c < W) add(c, r[k], d[k]);
+    if (c < W) post_sum<T, V, ENTRY>(p, t, c, inv, d[k], r[k], sum);
   }
   for (int c = rest; c < W; c += RS_THREADS * V) {
     float a[4], b[4];
     value(c, a, b);
-    add(c, a, b);
+    post_sum<T, V, ENTRY>(p, t, c, inv, b, a, sum);
   }
   if (p.after_w == nullptr) return;
   const float q = 1.f / sqrtf(block_sum(sum, red) / (float)W + p.after_eps);
-  auto norm = [&](int c, const float (&a)[4]) {
-    float w[4];
-    ldv<V>(p.after_w + c, w);
-#pragma unroll
-    for (int i = 0; i < V; ++i) w[i] *= a[i] * q;
-    stv<V>(y + c, w);
-  };
 #pragma unroll
   for (int k = 0; k < NPT; ++k) {
     const int c = (k * RS_THREADS + threadIdx.x) * V;
-    if (c < W) norm(c, r[k]);
+    if (c < W) post_after<T, V>(p, t, c, q, r[k]);
   }
   for (int c = rest; c < W; c += RS_THREADS * V) {
     float a[4];
     ldv<V>(res + c, a);
-    norm(c, a);
+    post_after<T, V>(p, t, c, q, a);
   }
 }
 
-template <typename T, bool MOE>
-int launch_post(const PostArgs<T>& p, long long rows, cudaStream_t st) {
+template <typename T, int SRC, bool ENTRY>
+int launch_post_rows(const PostArgs<T>& p, long long rows, cudaStream_t st) {
   const unsigned g = (unsigned)rows;
   if (p.W % 4 != 0) {
-    post_add_kernel<T, 1, 4, MOE><<<g, RS_THREADS, 0, st>>>(p);
+    post_add_kernel<T, 1, 4, SRC, ENTRY><<<g, RS_THREADS, 0, st>>>(p);
   } else {
     const int units = (p.W / 4 + RS_THREADS - 1) / RS_THREADS;
-    if (units <= 1) post_add_kernel<T, 4, 1, MOE><<<g, RS_THREADS, 0, st>>>(p);
-    else if (units <= 2) post_add_kernel<T, 4, 2, MOE><<<g, RS_THREADS, 0, st>>>(p);
-    else if (units <= 4) post_add_kernel<T, 4, 4, MOE><<<g, RS_THREADS, 0, st>>>(p);
-    else post_add_kernel<T, 4, 8, MOE><<<g, RS_THREADS, 0, st>>>(p);
+    if (units <= 1) post_add_kernel<T, 4, 1, SRC, ENTRY><<<g, RS_THREADS, 0, st>>>(p);
+    else if (units <= 2) post_add_kernel<T, 4, 2, SRC, ENTRY><<<g, RS_THREADS, 0, st>>>(p);
+    else if (units <= 4) post_add_kernel<T, 4, 4, SRC, ENTRY><<<g, RS_THREADS, 0, st>>>(p);
+    else post_add_kernel<T, 4, 8, SRC, ENTRY><<<g, RS_THREADS, 0, st>>>(p);
   }
   return (int)cudaGetLastError();
 }
 
+template <typename T, int SRC>
+int launch_post(const PostArgs<T>& p, long long rows, cudaStream_t st) {
+  if constexpr (SRC == POST_EMBED) return launch_post_rows<T, SRC, true>(p, rows, st);
+  else return p.again != nullptr || p.step != nullptr ? launch_post_rows<T, SRC, true>(p, rows, st)
+                                                      : launch_post_rows<T, SRC, false>(p, rows, st);
+}
+
+template <typename T>
+__device__ __forceinline__ float gelu_tanh_t(float g) {
+  const float k = 2.f * 0.7978845608028654f;             // 0.5 (1 + tanh(z)) = sigmoid(2 z), z = sqrt(2 / pi) (...)
+  return g * sigmoid_t<T>(k * (g + 0.044715f * g * g * g));
+}
+
+template <typename T>
+struct SideArgs {
+  const T* gate;                          // [dim, W]
+  const T* proj;                          // [W, dim]
+  const T* rows;                          // [vocabulary, ld]; the layer's entries start at `col`
+  const long long* ids;
+  long long ld;
+  int col, dim;
+};
+
+// One block per token.  dynamic shared memory: the residual's row, the gate's outputs
+template <typename T, bool ENTRY>
+__global__ void __launch_bounds__(RS_THREADS) side_add_kernel(const PostArgs<T> p, const SideArgs<T> s) {
+  extern __shared__ float sm[];
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  const int W = p.W, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  float* row = sm;
+  float* d = sm + W;                      // what is to be normed
+  float* g = d + W;
+  const float* res = p.resid + t * W;
+  for (int c = threadIdx.x; c < W; c += RS_THREADS) row[c] = res[c];
+  __syncthreads();
+  const T* tab = s.rows + s.ids[t] * s.ld + s.col;
+  const bool v4 = W % 4 == 0;
+  for (int j = warp; j < s.dim; j += RS_THREADS / 32) {
+    const T* w = s.gate + (long long)j * W;
+    float acc = 0.f;
+    if (v4) {
+#pragma unroll 4
+      for (int c = lane * 4; c < W; c += 128) {
+        float f[4];
+        ldf4(w + c, f);
+        const float4 x = *reinterpret_cast<const float4*>(row + c);
+        acc += f[0] * x.x + f[1] * x.y + f[2] * x.z + f[3] * x.w;
+      }
+    } else {
+      for (int c = lane; c < W; c += 32) acc += ldf(w + c) * row[c];
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) g[j] = gelu_tanh_t<T>(acc) * ldf(tab + j);
+  }
+  __syncthreads();
+  float ss = 0.f;
+  const bool quads = s.dim % 4 == 0;
+  for (int c = threadIdx.x; c < W; c += RS_THREADS) {
+    const T* w = s.proj + (long long)c * s.dim;
+    float acc = 0.f;
+    if (quads) {
+#pragma unroll 4
+      for (int j = 0; j < s.dim; j += 4) {
+        float f[4];
+        ldf4(w + j, f);
+        acc += f[0] * g[j] + f[1] * g[j + 1] + f[2] * g[j + 2] + f[3] * g[j + 3];
+      }
+    } else {
+      for (int j = 0; j < s.dim; ++j) acc += ldf(w + j) * g[j];
+    }
+    d[c] = acc;
+    ss += acc * acc;
+  }
+  const float inv = p.mult / sqrtf(block_sum(ss, red) / (float)W + p.eps);
+  float sum = 0.f;
+  for (int c = threadIdx.x; c < W; c += RS_THREADS) {
+    float a[4], b[4];
+    a[0] = row[c];
+    b[0] = d[c];
+    post_sum<T, 1, ENTRY>(p, t, c, inv, b, a, sum);
+    row[c] = a[0];
+  }
+  if (p.after_w == nullptr) return;
+  const float q = 1.f / sqrtf(block_sum(sum, red) / (float)W + p.after_eps);
+  for (int c = threadIdx.x; c < W; c += RS_THREADS) {
+    float a[4];
+    a[0] = row[c];
+    post_after<T, 1>(p, t, c, q, a);
+  }
+}
+
+// entries past `dim` of a padded row become zero
+template <typename T>
+__global__ void __launch_bounds__(256)
+side_gate_kernel(T* g, long long g_ld, const T* rows, const long long* ids, long long ld, int col, int dim, long long n) {
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= n) return;
+  const long long t = i / g_ld;
+  const int j = (int)(i - t * g_ld);
+  stf(g + i, j < dim ? gelu_tanh_t<T>(ldf(g + i)) * ldf(rows + ids[t] * ld + col + j) : 0.f);
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) soft_cap_kernel(T* x, long long n, float cap) {
+  const long long i = ((long long)blockIdx.x * 256 + threadIdx.x) * V;
+  if (i >= n) return;
+  float f[4];
+  ldv<V>(x + i, f);
+#pragma unroll
+  for (int k = 0; k < V; ++k) f[k] = cap * tanhf(f[k] / cap);
+  stv<V>(x + i, f);
+}
+
 enum { GLU_SILU = 0, GLU_GELU_TANH = 1, GLU_CLAMPED_SWISH = 2 };
 
-// 0.5 (1 + tanh(z)) = sigmoid(2 z) carries the tanh form of gelu on the sigmoid of the storage type
 template <int KIND, typename T>
 __device__ __forceinline__ float glu_one(float g, float u, float limit, float alpha) {
   if constexpr (KIND == GLU_SILU) {
     return g * sigmoid_t<T>(g) * u;
   } else if constexpr (KIND == GLU_GELU_TANH) {
-    const float k = 2.f * 0.7978845608028654f;           // 2 sqrt(2 / pi)
-    return g * sigmoid_t<T>(k * (g + 0.044715f * g * g * g)) * u;
+    return gelu_tanh_t<T>(g) * u;
   } else {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
@@ -466,16 +618,98 @@ MSRL_API int msrl_moe_combine_norm(const void* e, const int* pos, int top, float
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
+template <typename T>
+static PostArgs<T> post_args(float* resid, const float* norm_w, float eps, float mult, const float* after_w, float after_eps,
+                             const float* again, const float* step, void* y, int W) {
+  PostArgs<T> p{};
+  p.resid = resid;
+  p.norm_w = norm_w;
+  p.eps = eps;
+  p.mult = mult;
+  p.after_w = after_w;
+  p.after_eps = after_eps;
+  p.again = again;
+  p.step = step;
+  p.y = (T*)y;
+  p.W = W;
+  return p;
+}
+
 MSRL_API int msrl_post_add(const void* delta, const void* e, const int* pos, const float* weights, int top, const void* shared,
                            float* resid, const float* norm_w, float eps, float mult, const float* after_w, float after_eps,
-                           void* y, long long rows, int W, int is_f32, cudaStream_t st) {
+                           const float* again, const float* step, void* y, long long rows, int W, int is_f32,
+                           cudaStream_t st) {
   if (rows == 0) return 0;
   if (delta == nullptr && (e == nullptr || pos == nullptr || weights == nullptr)) return (int)cudaErrorInvalidValue;
   auto run = [&](auto tag) {
     using T = decltype(tag);
-    const PostArgs<T> p{(const T*)delta, (const T*)e, pos, weights, top, (const T*)shared, resid, norm_w, eps, mult, after_w,
-                        after_eps, (T*)y, W};
-    return delta == nullptr ? launch_post<T, true>(p, rows, st) : launch_post<T, false>(p, rows, st);
+    PostArgs<T> p = post_args<T>(resid, norm_w, eps, mult, after_w, after_eps, again, step, y, W);
+    p.delta = (const T*)delta;
+    p.e = (const T*)e;
+    p.pos = pos;
+    p.weights = weights;
+    p.top = top;
+    p.shared = (const T*)shared;
+    return delta == nullptr ? launch_post<T, POST_MOE>(p, rows, st) : launch_post<T, POST_ROWS>(p, rows, st);
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_post_embed(const long long* ids, const void* table, float* resid, float* first, const float* norm_w, float eps,
+                             float mult, const float* after_w, float after_eps, const float* step, void* y, long long rows,
+                             int W, int is_f32, cudaStream_t st) {
+  if (rows == 0) return 0;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    PostArgs<T> p = post_args<T>(resid, norm_w, eps, mult, after_w, after_eps, nullptr, step, y, W);
+    p.ids = ids;
+    p.table = (const T*)table;
+    p.first = first;
+    return launch_post<T, POST_EMBED>(p, rows, st);
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_side_add(const void* gate, const void* proj, const void* table, const long long* ids, long long ld, int col,
+                           int dim, float* resid, const float* norm_w, float eps, const float* after_w, float after_eps,
+                           const float* again, const float* step, void* y, long long rows, int W, int is_f32,
+                           cudaStream_t st) {
+  if (rows == 0) return 0;
+  const size_t smem = (2 * (size_t)W + dim) * sizeof(float);
+  if (smem > 200 * 1024) return (int)cudaErrorNotSupported;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const PostArgs<T> p = post_args<T>(resid, norm_w, eps, 1.f, after_w, after_eps, again, step, y, W);
+    const SideArgs<T> s{(const T*)gate, (const T*)proj, (const T*)table, ids, ld, col, dim};
+    auto* kernel = again != nullptr || step != nullptr ? side_add_kernel<T, true> : side_add_kernel<T, false>;
+    const cudaError_t rc = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (rc != cudaSuccess) return (int)rc;
+    kernel<<<(unsigned)rows, RS_THREADS, smem, st>>>(p, s);
+    return (int)cudaGetLastError();
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_side_gate(void* g, long long g_ld, const void* table, const long long* ids, long long ld, int col, int dim,
+                            long long rows, int is_f32, cudaStream_t st) {
+  const long long n = rows * g_ld;
+  if (n == 0) return 0;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    side_gate_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, st>>>((T*)g, g_ld, (const T*)table, ids, ld, col, dim, n);
+    return (int)cudaGetLastError();
+  };
+  return is_f32 ? run(float{}) : run(__nv_bfloat16{});
+}
+
+MSRL_API int msrl_soft_cap(void* x, long long n, float cap, int is_f32, cudaStream_t st) {
+  if (n == 0) return 0;
+  if (!(cap > 0.f)) return (int)cudaErrorInvalidValue;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    if (n % 4 == 0) soft_cap_kernel<T, 4><<<(unsigned)((n / 4 + 255) / 256), 256, 0, st>>>((T*)x, n, cap);
+    else soft_cap_kernel<T, 1><<<(unsigned)((n + 255) / 256), 256, 0, st>>>((T*)x, n, cap);
+    return (int)cudaGetLastError();
   };
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }

@@ -282,6 +282,120 @@ class MatrixMemorySpec:
 
 
 @dataclass(frozen=True)
+class RetentionSpec:
+    """Linear attention over a state that decays by a constant per head; neither soft-max nor denominator.  Heads are
+    stored in multiples of 16."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: Tuple[float, ...]
+
+    def slot_state(self, dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
+        return {"memory": ((self.heads, pad16(self.dim), pad16(self.vdim)), torch.float32)}
+
+    def paged_rows(self, dtype) -> dict:
+        return {}
+
+    @classmethod
+    def from_json(cls, m: dict) -> "RetentionSpec":
+        out = cls(int(m["heads"]), int(m["dim"]), int(m["vdim"]), tuple(float(x) for x in m["decay"]))
+        if len(out.decay) != out.heads or not all(0.0 <= x <= 1.0 for x in out.decay):
+            raise ValueError(f"{out.heads} heads need as many decays between 0 and 1, got {out.decay}")
+        return out
+
+
+@dataclass(frozen=True)
+class TurnedAttentionSpec:
+    """Soft-max attention of grouped heads over all earlier tokens, with partial half-split rotation of queries and keys.
+    Values are normed per head and turned by their own position over all their entries; an output is turned back by the
+    query's."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: Rotary
+    keys: KeyRange = None
+
+    @property
+    def value_rot(self) -> Rotary:
+        return Rotary(self.vdim, self.rot.base, halves=True)
+
+    def padded(self, dtype) -> Tuple[int, int]:
+        return padded_heads(self.dim, self.vdim, dtype)
+
+    def paged_rows(self, dtype) -> Dict[str, Tuple[int, ...]]:
+        qp, vp = self.padded(dtype)
+        return {"k": (self.kv_heads, qp), "v": (self.kv_heads, vp)}
+
+    def slot_state(self, dtype) -> dict:
+        return {}
+
+    @classmethod
+    def from_json(cls, m: dict) -> "TurnedAttentionSpec":
+        out = _check_heads(cls(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                               Rotary(int(m["rot"]["dims"]), float(m["rot"]["base"]), halves=True)))
+        _check_rotary(out.rot, out.dim, "dim")
+        _check_rotary(out.value_rot, out.vdim, "vdim")
+        return out
+
+
+@dataclass(frozen=True)
+class MinGRUSpec:
+    """A gated recurrence, element by element, whose gate and candidate read the current token only."""
+    width: int
+
+    def slot_state(self, dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
+        return {"state": ((self.width,), torch.float32)}
+
+    def paged_rows(self, dtype) -> dict:
+        return {}
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Attention and a gated recurrence side by side on the same input; their outputs are scaled and added."""
+    left: TurnedAttentionSpec
+    right: MinGRUSpec
+    left_scale: float
+    right_scale: float
+
+    @property
+    def keys(self) -> KeyRange:
+        return self.left.keys
+
+    def paged_rows(self, dtype) -> Dict[str, Tuple[int, ...]]:
+        return self.left.paged_rows(dtype)
+
+    def slot_state(self, dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
+        return self.right.slot_state(dtype)
+
+    @classmethod
+    def from_json(cls, m: dict) -> "ParallelSpec":
+        return cls(TurnedAttentionSpec.from_json(m["left"]), MinGRUSpec(int(m["right"]["width"])), float(m["left_scale"]),
+                   float(m["right_scale"]))
+
+
+@dataclass(frozen=True)
+class WKVSpec:
+    """Linear attention whose state decays per head and key channel by what the token says, with a bonus for the current
+    token.  Its projections read mixes of the token's input and the one before, which is carried (``model_width`` entries)."""
+    heads: int
+    dim: int
+    model_width: int
+
+    def slot_state(self, dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
+        return {"last": ((self.model_width,), torch.float32), "state": ((self.heads, self.dim, self.dim), torch.float32)}
+
+    def paged_rows(self, dtype) -> dict:
+        return {}
+
+    @classmethod
+    def from_json(cls, m: dict) -> "WKVSpec":
+        return cls(int(m["heads"]), int(m["dim"]), int(m["model_width"]))
+
+
+@dataclass(frozen=True)
 class GluSpec:
     """Gated feed-forward ``W_down(act(W_gate h, W_up h))``; see ``ops.glu_fwd`` for the activations."""
     ff: int
@@ -356,16 +470,38 @@ class SoftmaxMoESpec:
 
 
 @dataclass(frozen=True)
+class ChosenMoESpec:
+    """Experts of the largest router logits (32-bit), their outputs weighted by a soft-max over the chosen logits only."""
+    experts: int
+    top: int
+    expert: GluSpec
+    shared: Optional[GluSpec] = None
+
+    @classmethod
+    def from_json(cls, m: dict) -> "ChosenMoESpec":
+        r = m["router"]
+        out = cls(int(r["experts"]), int(r["top"]), GluSpec(int(m["expert"]["ff"]), "silu"))
+        if not 0 < out.top <= out.experts:
+            raise ValueError(f"top {out.top} of {out.experts} experts")
+        return out
+
+
+@dataclass(frozen=True)
 class Design:
     """What the layers of one architecture have in common.  ``mixers`` and ``feed_forwards``: readers of a layer's entry
     by its type.  ``parallel``: both sublayers read one norm and are added together; ``post_norm``: the sublayers read the
-    residual itself and their outputs are normed before they are added; otherwise the feed-forward reads a second norm of
-    the sum.  ``centered``: norms subtract the mean.  ``norm_offset``: the stored weight of a norm is an offset from this
-    value."""
+    residual itself and their outputs are normed before they are added; ``sandwich``: a norm before and one after each
+    sublayer; otherwise the feed-forward reads a second norm of the sum.  ``embed_norm``: token embeddings are normed.
+    ``loop_input``: every pass of a loop adds a vector of its own before it runs, and passes after the first what the
+    embedding gave.  ``centered``: norms subtract the mean.  ``norm_offset``: the stored weight of a norm is an offset from
+    this value.  Readers of mixers find the model's width under ``model_width``."""
     mixers: Dict[str, Callable[[dict], Any]]
     feed_forwards: Dict[str, Callable[[dict], Any]]
     parallel: bool = False
     post_norm: bool = False
+    sandwich: bool = False
+    embed_norm: bool = False
+    loop_input: bool = False
     centered: bool = False
     norm_offset: float = 0.0
     tied_head: bool = True
@@ -378,6 +514,8 @@ DESIGNS = {
                       {"moe": ScoredMoESpec.from_json}, parallel=True, centered=True, tied_head=False),
     "Gapevik": Design({"attention": ConvAttentionSpec.from_json, "latent_attention": LatentAttentionSpec.gated_from_json,
                        "delta": HeadDeltaSpec.from_json}, {"moe": SoftmaxMoESpec.from_json}, post_norm=True),
+    "Lunelorn": Design({"retention": RetentionSpec.from_json, "parallel": ParallelSpec.from_json, "wkv": WKVSpec.from_json},
+                       {"moe": ChosenMoESpec.from_json}, sandwich=True, embed_norm=True, loop_input=True, tied_head=False),
 }
 
 
@@ -399,6 +537,8 @@ class HybridConfig:
     embedding_scale: float = 1.0
     residual_mult: float = 1.0                       # factor on what a sublayer adds (post-norm designs)
     loop: Optional[Tuple[int, int, int]] = None      # (start, stop, times)
+    token_side: Optional[int] = None                 # entries of a token's row per layer (designs with token inputs)
+    logit_softcap: float = 0.0                       # logits <- cap tanh(logits / cap); 0: as they are
     params_dtype: torch.dtype = torch.bfloat16
     extra: Dict[str, Any] = field(default_factory=dict)
     is_hybrid = True
@@ -442,6 +582,14 @@ class HybridConfig:
         return [*range(a), *(list(range(a, b)) * times), *range(b, n)]
 
     @property
+    def pass_starts(self) -> Dict[int, int]:
+        """Layer run -> number of the pass of the loop that begins with it."""
+        if self.loop is None:
+            return {}
+        a, b, times = self.loop
+        return {a + p * (b - a): p for p in range(times)} if b > a else {}
+
+    @property
     def num_layers(self) -> int:
         return len(self.run_order)
 
@@ -452,7 +600,7 @@ class HybridConfig:
 
     @property
     def is_moe(self) -> bool:
-        return any(isinstance(l.mlp, (TableMoESpec, ScoredMoESpec, SoftmaxMoESpec)) for l in self.layers)
+        return any(isinstance(l.mlp, (TableMoESpec, ScoredMoESpec, SoftmaxMoESpec, ChosenMoESpec)) for l in self.layers)
 
     @property
     def windows(self) -> Tuple[KeyRange, ...]:
@@ -469,13 +617,14 @@ class HybridConfig:
             if mlp is not None and mlp["kind"] not in design.feed_forwards:
                 raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
             of = l.get("weights_of")
-            layers.append(LayerSpec(l["type"], design.mixers[l["type"]](l["mixer"]),
+            layers.append(LayerSpec(l["type"], design.mixers[l["type"]]({"model_width": int(cfg["width"]), **l["mixer"]}),
                                     None if mlp is None else design.feed_forwards[mlp["kind"]](mlp),
                                     None if of is None else int(of)))
-        lp = cfg.get("loop")
+        lp, side = cfg.get("loop"), cfg.get("token_side")
         return cls(architecture=cfg["architecture"], vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
                    layers=layers, norm_epsilon=float(cfg["norm"]["eps"]),
                    embedding_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)),
                    residual_mult=float(cfg.get("residual_mult", 1.0)),
                    loop=None if not lp else (int(lp["start"]), int(lp["stop"]), int(lp["times"])),
+                   token_side=int(side["dim"]) if side else None, logit_softcap=float(cfg.get("logit_softcap") or 0.0),
                    params_dtype=dtype)

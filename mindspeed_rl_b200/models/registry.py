@@ -112,5 +112,6 @@ def _decoder_weights(cfg, state, device):
 register("Pumotar", ModelFamily(HybridConfig.from_json, _hybrid_weights, "pumotar"))
 register("Sunatar", ModelFamily(HybridConfig.from_json, _hybrid_weights, "sunatar"))
 register("Gapevik", ModelFamily(HybridConfig.from_json, _hybrid_weights, "gapevik"))
+register("Lunelorn", ModelFamily(HybridConfig.from_json, _hybrid_weights, "lunelorn"))
 for _name in ("Qwen2ForCausalLM", "Qwen3ForCausalLM", "Qwen3MoeForCausalLM"):
     register(_name, ModelFamily(_decoder_config, _decoder_weights))

@@ -75,19 +75,21 @@ def moe_plan(expert_of: torch.Tensor, num_experts: int) -> MoePlan:
     return MoePlan(counts.int(), offsets.int(), pos.int(), tiles, rows, t, k, num_experts)
 
 
-def route_top(logits: torch.Tensor, top: int) -> Tuple[torch.Tensor, torch.Tensor]:
+def route_top(logits: torch.Tensor, top: int, chosen_softmax: bool = False) -> Tuple[torch.Tensor, torch.Tensor]:
     """Router logits ``[T, E]`` fp32 -> ``(expert ids [T, top] int64, their scores [T, top] fp32)``: the ``top`` largest
-    ``sigmoid(logit)`` in descending order (equal logits: the lower expert first), scores not renormalised."""
+    logits in descending order (equal logits: the lower expert first), scores ``sigmoid(logit)``, not renormalised, or with
+    ``chosen_softmax`` a soft-max over the chosen logits."""
     t, e = logits.shape
     if _lib.use_kernels(logits):
         logits = logits.contiguous()
         idx = guard.empty(t, top, dtype=torch.int64, device=logits.device)
         score = guard.empty(t, top, dtype=torch.float32, device=logits.device)
-        check(_lib.load().msrl_route_top(ptr(logits), c_int(t), c_int(e), c_int(top), ptr(idx), ptr(score), stream()),
-              "route_top")
+        check(_lib.load().msrl_route_top(ptr(logits), c_int(t), c_int(e), c_int(top), ptr(idx), ptr(score),
+                                         c_int(chosen_softmax), stream()), "route_top")
         return idx, score
     z, idx = torch.sort(logits, dim=-1, descending=True, stable=True)
-    return idx[:, :top].contiguous(), torch.sigmoid(z[:, :top])
+    z = z[:, :top]
+    return idx[:, :top].contiguous(), torch.softmax(z, dim=-1) if chosen_softmax else torch.sigmoid(z)
 
 
 def route_softmax_top(logits: torch.Tensor, correction: torch.Tensor, top: int) -> Tuple[torch.Tensor, torch.Tensor]:

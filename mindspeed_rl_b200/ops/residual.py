@@ -4,7 +4,7 @@ follows fused in, and the gated activations.
 The residual ``[T, W]`` is fp32 and updated in place; norm weights are fp32, the activations bf16 or fp32.
 ``norm(x) = x / sqrt(mean(x^2) + eps) * (offset + w)`` in fp32; ``centered`` norms subtract the row's mean from x
 first (a layer norm without bias).  ``post_*`` functions norm what a sublayer gives before it is added and hand on the
-residual itself, rounded to the activation type.  CUDA path: ``csrc/residual_stream.cu``; CPU
+residual itself, rounded to the activation type, or a norm of it; ``entry``: what a pass of a loop adds in between.  CUDA path: ``csrc/residual_stream.cu``; CPU
 tensors run the PyTorch formulation.
 """
 from __future__ import annotations
@@ -18,6 +18,7 @@ from . import guard
 
 from . import _lib
 from ._lib import c_float, c_int, c_ll, check, ptr, stream
+from .gemm import linear_fwd
 
 
 def _is_f32(t: torch.Tensor):
@@ -39,6 +40,22 @@ class PostNorm(NamedTuple):
     weight: torch.Tensor
     eps: float
     mult: float = 1.0
+
+
+class PassEntry(NamedTuple):
+    """What a pass of a loop adds to the residual before it runs: ``again [T, W]`` (or None) and ``step [W]``, fp32."""
+    again: Optional[torch.Tensor]
+    step: torch.Tensor
+
+
+class TokenSide(NamedTuple):
+    """A layer's input from the token itself: ``proj (gelu_tanh(gate x) * table[id, col:col + dim])``.  ``gate [pad, W]`` and
+    ``proj [W, pad]`` are padded with zeros to whole vectors."""
+    gate: torch.Tensor
+    proj: torch.Tensor
+    table: torch.Tensor
+    col: int
+    dim: int
 
 
 def _norm_ref(x: torch.Tensor, w: torch.Tensor, eps: float, offset: float, centered: bool, dtype) -> torch.Tensor:
@@ -75,40 +92,114 @@ def embed(ids: torch.Tensor, table: torch.Tensor, scale: float) -> Tuple[torch.T
     return resid, resid.to(table.dtype, copy=True)
 
 
-def _post_ref(resid, d, post: PostNorm, after: Optional[Norm], dtype):
+def _enter_ref(resid, entry: Optional[PassEntry]) -> None:
+    if entry is not None:
+        if entry.again is not None:
+            resid.add_(entry.again)
+        resid.add_(entry.step)
+
+
+def _post_ref(resid, d, post: PostNorm, after: Optional[Norm], dtype, entry: Optional[PassEntry] = None):
     resid.add_(post.mult * (d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + post.eps) * post.weight))
+    _enter_ref(resid, entry)
     return resid.to(dtype, copy=True) if after is None else _norm_ref(resid, *after, dtype)
 
 
-def post_add_(resid: torch.Tensor, delta: torch.Tensor, post: PostNorm, after: Optional[Norm] = None) -> torch.Tensor:
+def post_embed(ids: torch.Tensor, table: torch.Tensor, post: PostNorm, after: Norm, keep: bool = False,
+               step: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, Optional[torch.Tensor], torch.Tensor]:
+    """Normed embeddings: ``(residual fp32, a copy of it before step or None, after(residual))``; ``step [W]`` is added to the
+    residual, ``keep`` asks for the copy."""
+    t, width = ids.numel(), table.shape[1]
+    if _lib.use_kernels(ids, table, post.weight):
+        _plain(after)
+        resid = guard.empty(t, width, device=table.device, dtype=torch.float32)
+        first = guard.empty(t, width, device=table.device, dtype=torch.float32) if keep else None
+        y = guard.empty(t, width, device=table.device, dtype=table.dtype)
+        check(_lib.load().msrl_post_embed(
+            ptr(ids), ptr(table), ptr(resid), ptr(first), ptr(post.weight), c_float(post.eps), c_float(post.mult),
+            ptr(after.weight), c_float(after.eps), ptr(step), ptr(y), c_ll(t), c_int(width), _is_f32(table), stream()), "post_embed")
+        return resid, first, y
+    resid = torch.zeros(t, width)
+    _post_ref(resid, table[ids].float(), post, None, table.dtype)
+    first = resid.clone() if keep else None
+    if step is not None:
+        resid.add_(step)
+    return resid, first, _norm_ref(resid, *after, table.dtype)
+
+
+def post_add_(resid: torch.Tensor, delta: torch.Tensor, post: PostNorm, after: Optional[Norm] = None,
+              entry: Optional[PassEntry] = None) -> torch.Tensor:
     """Add the normed ``delta`` in place; returns the sum (or, with ``after``, that norm of it) in ``delta``'s type."""
     if _lib.use_kernels(resid, delta, post.weight):
-        return _post(resid, post, after, delta.dtype, delta=delta.contiguous())
-    return _post_ref(resid, delta.float(), post, after, delta.dtype)
+        return _post(resid, post, after, delta.dtype, entry, delta=delta.contiguous())
+    return _post_ref(resid, delta.float(), post, after, delta.dtype, entry)
 
 
 def moe_post_add_(resid: torch.Tensor, expert_rows: torch.Tensor, pos: torch.Tensor, weights: torch.Tensor, post: PostNorm,
-                  after: Optional[Norm] = None, shared: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  after: Optional[Norm] = None, shared: Optional[torch.Tensor] = None,
+                  entry: Optional[PassEntry] = None) -> torch.Tensor:
     """The same for ``d[t] = sum_j weights[t, j] * expert_rows[pos[t, j]] (+ shared[t])``; a negative ``pos`` is an expert
     that gives back its input, the residual's row.  ``weights [T, top]`` fp32."""
     if _lib.use_kernels(resid, expert_rows, pos, weights):
-        return _post(resid, post, after, expert_rows.dtype, rows=expert_rows, pos=pos, weights=weights.contiguous(), shared=shared)
+        return _post(resid, post, after, expert_rows.dtype, entry, rows=expert_rows, pos=pos, weights=weights.contiguous(),
+                     shared=shared)
     pos = pos.long().view(resid.shape[0], -1)
     rows = torch.where((pos < 0)[..., None], resid[:, None, :], expert_rows[pos.clamp(min=0)].float())
     d = (rows * weights[..., None]).sum(1)
-    return _post_ref(resid, d if shared is None else d + shared.float(), post, after, expert_rows.dtype)
+    return _post_ref(resid, d if shared is None else d + shared.float(), post, after, expert_rows.dtype, entry)
 
 
-def _post(resid, post, after, dtype, delta=None, rows=None, pos=None, weights=None, shared=None):
-    t, width = resid.shape
+def _plain(after: Optional[Norm]) -> None:
     if after is not None and (after.centered or after.offset):
-        raise ValueError("the norm behind a post-normed layer is a plain RMS norm")
+        raise ValueError("the norm behind a post-normed sublayer is a plain RMS norm")
+
+
+def _post(resid, post, after, dtype, entry=None, delta=None, rows=None, pos=None, weights=None, shared=None):
+    t, width = resid.shape
+    _plain(after)
+    again, step = entry or (None, None)
     y = guard.empty(t, width, device=resid.device, dtype=dtype)
     check(_lib.load().msrl_post_add(
         ptr(delta), ptr(rows), ptr(pos), ptr(weights), c_int(0 if weights is None else weights.shape[1]), ptr(shared), ptr(resid),
         ptr(post.weight), c_float(post.eps), c_float(post.mult), ptr(after.weight if after else None),
-        c_float(after.eps if after else 0.0), ptr(y), c_ll(t), c_int(width), _is_f32(y), stream()), "post_add")
+        c_float(after.eps if after else 0.0), ptr(again), ptr(step), ptr(y), c_ll(t), c_int(width), _is_f32(y), stream()),
+        "post_add")
     return y
+
+
+FUSED_SIDE_TOKENS = 256        # up to here one kernel does a token input; more tokens make its products matrix products
+
+
+def token_side_(resid: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, side: TokenSide, post: PostNorm,
+                after: Optional[Norm] = None, entry: Optional[PassEntry] = None,
+                fused_tokens: Optional[int] = None) -> torch.Tensor:
+    """Add a layer's token input to the residual like :func:`post_add_`; ``x`` is the residual in the activation type."""
+    t, width = resid.shape
+    if _lib.use_kernels(resid, x, ids, side.gate, side.table):
+        L, pad = _lib.load(), side.gate.shape[0]
+        row = (ptr(side.table), ptr(ids), c_ll(side.table.shape[1]), c_int(side.col))
+        if t <= (FUSED_SIDE_TOKENS if fused_tokens is None else fused_tokens) and pad == side.dim and width <= 16384:
+            _plain(after)
+            again, step = entry or (None, None)
+            y = guard.empty(t, width, device=resid.device, dtype=x.dtype)
+            check(L.msrl_side_add(ptr(side.gate), ptr(side.proj), *row, c_int(side.dim), ptr(resid), ptr(post.weight),
+                                  c_float(post.eps), ptr(after.weight if after else None), c_float(after.eps if after else 0.0),
+                                  ptr(again), ptr(step), ptr(y), c_ll(t), c_int(width), _is_f32(x), stream()), "side_add")
+            return y
+        g = linear_fwd(x, side.gate)
+        check(L.msrl_side_gate(ptr(g), c_ll(pad), *row, c_int(side.dim), c_ll(t), _is_f32(x), stream()), "side_gate")
+        return post_add_(resid, linear_fwd(g, side.proj), post, after, entry)
+    g = F.gelu(linear_fwd(x, side.gate)[:, :side.dim].float(), approximate="tanh")
+    g = (g * side.table[ids, side.col:side.col + side.dim].float()).to(x.dtype)
+    return post_add_(resid, linear_fwd(g, side.proj[:, :side.dim]), post, after, entry)
+
+
+def soft_cap_(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """``x <- cap * tanh(x / cap)`` in place (contiguous), computed in 32-bit."""
+    if _lib.use_kernels(x):
+        check(_lib.load().msrl_soft_cap(ptr(x), c_ll(x.numel()), c_float(cap), _is_f32(x), stream()), "soft_cap")
+        return x
+    return x.copy_(cap * torch.tanh(x.float() / cap))
 
 
 def add_norm_(resid: torch.Tensor, delta: torch.Tensor, w: torch.Tensor, eps: float, offset: float = 0.0,

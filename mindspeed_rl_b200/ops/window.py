@@ -103,6 +103,53 @@ def qkv_prep_(proj: torch.Tensor, lay: GroupedHeads, q_norm: torch.Tensor, k_nor
     v_cache.view(-1, *v_cache.shape[2:])[slots[ok]] = v[ok]
 
 
+def _turned(x: torch.Tensor, cs: torch.Tensor, back: bool = False) -> torch.Tensor:
+    """``x [T, heads, n]`` with entry i turned with entry i + n / 2 by the angles of ``cs [T, n]`` (cos | sin)."""
+    half = cs.shape[1] // 2
+    c, s = cs[:, None, :half], cs[:, None, half:] * (-1.0 if back else 1.0)
+    a, b = x[..., :half], x[..., half:]
+    return torch.cat([a * c - b * s, b * c + a * s], dim=-1)
+
+
+def turned_prep_(proj: torch.Tensor, lay: GroupedHeads, eps: float, table: torch.Tensor, value_table: torch.Tensor,
+                 positions: torch.Tensor, slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor) -> None:
+    """Rotate queries and keys, norm (RMS per head, no weight) and turn values over all their entries, in place, and write keys
+    and values to the cache (``slots[t] < 0``: not written).  ``value_table [length, vdim]``."""
+    t, rot = proj.shape[0], table.shape[1]
+    if _lib.use_kernels(proj, positions, slots, k_cache, v_cache):
+        ints = (ctypes.c_int * 11)(lay.heads, lay.kv_heads, lay.dim, lay.vdim, lay.qp, lay.vp, lay.q_col, lay.k_col, lay.v_col,
+                                   rot, table.shape[0])
+        check(_lib.load().msrl_turned_prep(
+            ptr(proj), c_ll(proj.stride(0)), ints, c_float(eps), ptr(table), ptr(value_table), ptr(positions), ptr(slots),
+            ptr(k_cache), ptr(v_cache), c_int(t), _is_f32(proj), stream()), "turned_prep")
+        return
+    at = positions.long()
+    q, k, v = lay.split(proj)
+    for x in (q, k):
+        x[..., :rot] = _turned(x[..., :rot].float(), table[at]).to(x.dtype)
+    f = v[..., :lay.vdim].float()
+    f = f / torch.sqrt(f.pow(2).mean(-1, keepdim=True) + eps)
+    v[..., :lay.vdim] = _turned(f, value_table[at]).to(v.dtype)
+    ok = slots >= 0
+    k_cache.view(-1, *k_cache.shape[2:])[slots[ok]] = k[ok]
+    v_cache.view(-1, *v_cache.shape[2:])[slots[ok]] = v[ok]
+
+
+def turn_back(attn: torch.Tensor, lay: GroupedHeads, value_table: torch.Tensor, positions: torch.Tensor, scale: float,
+              out: torch.Tensor) -> None:
+    """Attention outputs ``[T, heads * vp]`` turned back by their token's position and scaled, into the first columns of
+    ``out``."""
+    t = attn.shape[0]
+    if _lib.use_kernels(attn, positions, out):
+        check(_lib.load().msrl_turn_back(
+            ptr(attn), ptr(out), c_ll(out.stride(0)), c_int(lay.heads), c_int(lay.vdim), c_int(lay.vp), ptr(value_table),
+            c_int(value_table.shape[0]), ptr(positions), c_float(scale), c_int(t), _is_f32(attn), stream()), "turn_back")
+        return
+    x = attn.view(t, lay.heads, lay.vp).float()
+    y = _turned(x[..., :lay.vdim], value_table[positions.long()], back=True) * scale
+    out[:, :lay.heads * lay.vp] = torch.cat([y, x[..., lay.vdim:] * 0.0], dim=-1).reshape(t, -1).to(out.dtype)
+
+
 def rows_gather(cache: torch.Tensor, block_tables: torch.Tensor, token_seq: torch.Tensor, token_pos: torch.Tensor
                 ) -> torch.Tensor:
     """Cache rows ``[T, *row]`` of tokens given as (block-table row, position)."""

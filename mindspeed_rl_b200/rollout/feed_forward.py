@@ -12,7 +12,7 @@ from typing import Dict, Optional, Tuple
 import torch
 
 from .. import ops
-from ..models.hybrid_config import GluSpec, ScoredMoESpec, SoftmaxMoESpec, TableMoESpec
+from ..models.hybrid_config import ChosenMoESpec, GluSpec, ScoredMoESpec, SoftmaxMoESpec, TableMoESpec
 from ..ops import moe as K
 from ..ops.gemm import linear_f32, linear_fwd
 from .mixers import _pad_cols, _pad_rows
@@ -34,8 +34,8 @@ class Glu:
     def finish_(self, resid, h, done, norm, delta: Optional[torch.Tensor] = None) -> torch.Tensor:
         return ops.add_norm_(resid, done, *norm, delta2=delta)
 
-    def finish_post_(self, resid, done, post, after) -> torch.Tensor:
-        return ops.post_add_(resid, done, post, after)
+    def finish_post_(self, resid, done, post, after, entry=None) -> torch.Tensor:
+        return ops.post_add_(resid, done, post, after, entry)
 
 
 class GroupedExperts:
@@ -100,7 +100,15 @@ class ScoredMoE(GroupedExperts):
         return self.run(h, K.moe_plan(idx, self.spec.experts), score)
 
 
-class SoftmaxMoE(GroupedExperts):
+class WeightedExperts(GroupedExperts):
+    """Experts whose outputs are added with a weight each, in designs that norm a sublayer's output."""
+
+    def finish_post_(self, resid, done, post, after, entry=None) -> torch.Tensor:
+        y, plan, shared, score = done
+        return ops.moe_post_add_(resid, y, plan.pos, score, post, after, shared, entry)
+
+
+class SoftmaxMoE(WeightedExperts):
     """Router scores are a 32-bit soft-max; what is chosen also depends on a correction per output.  Identity experts have
     no rows in the dispatch plan: the combine takes their input, the residual, where it adds the others."""
 
@@ -116,12 +124,23 @@ class SoftmaxMoE(GroupedExperts):
         idx, score = K.route_softmax_top(linear_f32(h, self.router), self.correction, self.spec.top)
         return *self.run(h, K.moe_plan(idx, self.spec.experts)), score
 
-    def finish_post_(self, resid, done, post, after) -> torch.Tensor:
-        y, plan, shared, score = done
-        return ops.moe_post_add_(resid, y, plan.pos, score, post, after, shared)
+
+class ChosenMoE(WeightedExperts):
+    """The experts of the largest 32-bit logits, weighted by a soft-max over the logits chosen."""
+
+    def __init__(self, spec: ChosenMoESpec, w: Dict[str, torch.Tensor], dtype, device):
+        super().__init__(spec, w, dtype, device)
+        self.router = w["router"].to(device=device, dtype=dtype).contiguous()
+        if self.router.shape[0] != spec.experts:
+            raise ValueError(f"router {tuple(self.router.shape)} does not fit {spec.experts} experts")
+
+    def forward(self, h: torch.Tensor, ids: torch.Tensor):
+        idx, score = K.route_top(linear_f32(h, self.router), self.spec.top, chosen_softmax=True)
+        return *self.run(h, K.moe_plan(idx, self.spec.experts)), score
 
 
-FEED_FORWARDS = {GluSpec: Glu, TableMoESpec: TableMoE, ScoredMoESpec: ScoredMoE, SoftmaxMoESpec: SoftmaxMoE}
+FEED_FORWARDS = {GluSpec: Glu, TableMoESpec: TableMoE, ScoredMoESpec: ScoredMoE, SoftmaxMoESpec: SoftmaxMoE,
+                 ChosenMoESpec: ChosenMoE}
 
 
 def build_feed_forward(spec, w: Dict[str, torch.Tensor], dtype, device):

@@ -13,13 +13,15 @@ import torch
 
 from .. import ops
 from ..models.hybrid_config import (ChannelDeltaSpec, Chunk, ConvAttentionSpec, HeadDeltaSpec, KeyRange, LatentAttentionSpec,
-                                    MatrixMemorySpec, WindowAttentionSpec)
+                                    MatrixMemorySpec, ParallelSpec, RetentionSpec, WKVSpec, WindowAttentionSpec)
 from ..ops.conv_qkv import ConvHeads, ConvNormWeights
 from ..ops.delta import DeltaLayout, DeltaWeights
 from ..ops.gemm import linear_f32, linear_fwd
 from ..ops.latent import LatentLayout, pad16
-from ..ops.matrix_memory import MemoryLayout, MemoryWeights
+from ..ops.matrix_memory import MemoryLayout, MemoryWeights, constant_decay
+from ..ops.min_gru import GRULayout
 from ..ops.window import GroupedHeads, ValueSource
+from ..ops.wkv import WKVWeights
 
 
 class KeySpan(NamedTuple):
@@ -379,5 +381,128 @@ class MatrixMemory:
         return linear_fwd(y, self.w_o)
 
 
+class Retention:
+    """The matrix memory with a constant decay per head in place of its gates, no denominator and a silu output gate."""
+
+    def __init__(self, spec, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.spec, self.eps = spec, eps
+        h, d, dv = spec.heads, spec.dim, spec.vdim
+        dp, vp = pad16(d), pad16(dv)
+
+        def put(t, dt=dtype):
+            return t.to(device=device, dtype=dt).contiguous()
+
+        fused, cols = stack_sections([_pad_heads(w["q"], h, d, dp), _pad_heads(w["k"], h, d, dp),
+                                      _pad_heads(w["v"], h, dv, vp), _pad_heads(w["g"], h, dv, vp)])
+        self.lay = MemoryLayout(h, dp, vp, dv, *cols, scale=d ** -0.5, silu_gate=True)
+        self.w_in = put(fused)
+        self.memory = MemoryWeights(bias=None, norm=torch.ones(h * vp, device=device),
+                                    decay=put(constant_decay(spec.decay), torch.float32))
+        self.w_o = put(_pad_cols(w["o"].reshape(-1, h, dv), vp).reshape(-1, h * vp))
+
+    def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        y = ops.memory_prefill(linear_fwd(x, self.w_in), None, self.lay, self.memory, cache.slots[run], meta.cu_q, meta.max_q,
+                               meta.start_pos, meta.state_slots, self.eps)
+        return linear_fwd(y, self.w_o)
+
+    def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        y = ops.memory_decode(linear_fwd(x, self.w_in), None, self.lay, self.memory, cache.slots[run], meta.positions,
+                              meta.state_slots, self.eps)
+        return linear_fwd(y, self.w_o)
+
+
+class ParallelMixer:
+    """Attention with turned values and a minimal gated recurrence on one input.  All projections are one product; both
+    sides write their scaled results next to each other, so that their output projections and the sum are one product too."""
+
+    def __init__(self, spec, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.spec, self.eps = spec, eps
+        s, n = spec.left, spec.right.width
+        h, g = s.heads, s.kv_heads
+        qp, vp = s.padded(dtype)
+
+        def put(t, dt=dtype):
+            return t.to(device=device, dtype=dt).contiguous()
+
+        fused, cols = stack_sections([_pad_heads(w["left.q"], h, s.dim, qp), _pad_heads(w["left.k"], g, s.dim, qp),
+                                      _pad_heads(w["left.v"], g, s.vdim, vp), w["right.z"], w["right.x"], w["right.g"]])
+        self.heads = GroupedHeads(h, g, s.dim, s.vdim, qp, vp, *cols[:3])
+        self.gru = GRULayout(n, _pad8(n), *cols[3:], out_col=h * vp, scale=spec.right_scale)
+        self.w_in = put(fused)
+        self.z_bias, self.x_bias = (put(w[f"right.{i}.b"].reshape(-1), torch.float32) for i in "zx")
+        left = _pad_cols(w["left.o"].reshape(-1, h, s.vdim), vp).reshape(-1, h * vp)
+        self.w_o = put(torch.cat([left, _pad_cols(w["right.o"], _pad8(n))], dim=1))
+
+    def _prepare(self, x: torch.Tensor, meta: StepMeta, rows: Dict[str, torch.Tensor]):
+        s = self.spec.left
+        proj = linear_fwd(x, self.w_in)
+        table, values = (ops.angle_table(_table_rows(meta), r.frequencies(), x.device) for r in (s.rot, s.value_rot))
+        ops.turned_prep_(proj, self.heads, self.eps, table, values, meta.positions, meta.slots, rows["k"], rows["v"])
+        return proj, values
+
+    def _finish(self, attn: torch.Tensor, proj: torch.Tensor, values: torch.Tensor, meta: StepMeta, cache, run: int):
+        out = torch.empty(proj.shape[0], self.w_o.shape[1], dtype=proj.dtype, device=proj.device)
+        ops.turn_back(attn, self.heads, values, meta.positions, self.spec.left_scale, out)
+        args = (proj, self.gru, self.z_bias, self.x_bias, cache.slots[run]["state"], out)
+        if meta.is_decode:
+            ops.min_gru_decode(*args, meta.positions, meta.state_slots)
+        else:
+            ops.min_gru_prefill(*args, meta.cu_q, meta.max_q, meta.start_pos, meta.state_slots)
+        return linear_fwd(out, self.w_o)
+
+    def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        rows, span = cache.rows[run], meta.span_of(self.spec.keys)
+        proj, values = self._prepare(x, meta, rows)
+        attn = ops.window_prefill_attention(proj, self.heads, span.cu_q, span.cu_k, span.max_q, self.spec.left.scale, None,
+                                            _cached_kv(rows, span))
+        return self._finish(attn, proj, values, meta, cache, run)
+
+    def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        rows = cache.rows[run]
+        proj, values = self._prepare(x, meta, rows)
+        attn = ops.window_decode_attention(proj, self.heads, rows["k"], rows["v"], meta.block_tables, meta.context_lens,
+                                           meta.max_context, self.spec.left.scale, None)
+        return self._finish(attn, proj, values, meta, cache, run)
+
+
+class WKV:
+    """Projections read mixes of neighbouring tokens, a row of its own each; those of equal shape are one batched product in
+    small steps.  The decay's bottleneck has 32-bit results."""
+
+    def __init__(self, spec, w: Dict[str, torch.Tensor], eps: float, dtype, device):
+        self.spec, self.eps = spec, eps
+
+        def put(t, dt=dtype):
+            return t.to(device=device, dtype=dt).contiguous()
+
+        f32 = torch.float32
+        self.w_in = put(torch.stack([w[n] for n in "rkvg"]))                   # [4, heads * dim, W]
+        self.w1 = put(w["w1"])
+        self.wkv = WKVWeights(mu=put(torch.stack([w["mu." + n].reshape(-1) for n in "rkvgw"]), f32), w2=put(w["w2"]),
+                              w0=put(w["w0"].reshape(-1), f32), u=put(w["u"].reshape(-1), f32), norm=put(w["norm"].reshape(-1), f32),
+                              heads=spec.heads, dim=spec.dim)
+        self.w_o = put(w["o"])
+
+    def _project(self, mixed: torch.Tensor):
+        a = linear_f32(mixed[4], self.w1)
+        if mixed.shape[1] > 128:
+            return [linear_fwd(x, w) for x, w in zip(mixed, self.w_in)], a
+        return torch.bmm(mixed[:4], self.w_in.transpose(1, 2)).unbind(), a
+
+    def prefill(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        slots = cache.slots[run]
+        rkvg, a = self._project(ops.wkv_mix_prefill(x, self.wkv.mu, slots["last"], meta.tok_seq, meta.cu_q, meta.start_pos,
+                                                    meta.state_slots))
+        y = ops.wkv_prefill(*rkvg, a, self.wkv, slots["state"], meta.cu_q, meta.max_q, meta.start_pos, meta.state_slots, self.eps)
+        return linear_fwd(y, self.w_o)
+
+    def decode(self, x: torch.Tensor, meta: StepMeta, cache, run: int) -> torch.Tensor:
+        slots = cache.slots[run]
+        rkvg, a = self._project(ops.wkv_mix_decode(x, self.wkv.mu, slots["last"], meta.positions, meta.state_slots))
+        y = ops.wkv_decode(*rkvg, a, self.wkv, slots["state"], meta.positions, meta.state_slots, self.eps)
+        return linear_fwd(y, self.w_o)
+
+
 MIXERS = {LatentAttentionSpec: LatentAttention, ChannelDeltaSpec: ChannelDelta, HeadDeltaSpec: HeadDelta,
-          WindowAttentionSpec: WindowAttention, ConvAttentionSpec: ConvAttention, MatrixMemorySpec: MatrixMemory}
+          WindowAttentionSpec: WindowAttention, ConvAttentionSpec: ConvAttention, MatrixMemorySpec: MatrixMemory,
+          RetentionSpec: Retention, ParallelSpec: ParallelMixer, WKVSpec: WKV}

@@ -207,6 +207,8 @@ class ModelRunner:
         order, parallel = c.run_order, c.design.parallel
         if c.design.post_norm:
             return self._forward_post_norm(meta)
+        if c.design.sandwich:
+            return self._forward_sandwich(meta)
 
         def norm(weight):
             return ops.Norm(weight, c.norm_epsilon, c.design.norm_offset, c.design.centered)
@@ -247,6 +249,42 @@ class ModelRunner:
                 self.layer_probe(run, resid)
         return x
 
+    def _forward_sandwich(self, meta: StepMeta) -> torch.Tensor:
+        """The same for designs with a norm before and one after each sublayer, token inputs behind the layers and inputs of
+        a loop's passes: the kernel that adds a layer's last term also adds what the next pass starts with and takes the
+        next norm."""
+        w, c, cache = self.weights, self.cfg, self.cache
+        order, starts = c.run_order, c.pass_starts if c.design.loop_input else {}
+
+        def norm(weight):
+            return ops.Norm(weight, c.norm_epsilon)
+
+        def post(weight):
+            return ops.PostNorm(weight, c.norm_epsilon)
+
+        resid, first, x = ops.post_embed(meta.ids, w.embed, post(w.embed_norm), norm(w.layers[order[0]].norm1),
+                                         keep=len(starts) > 1, step=w.loop_step[starts[0]] if 0 in starts else None)
+        for run, li in enumerate(order):
+            lw = w.layers[li]
+            after = norm(w.layers[order[run + 1]].norm1 if run + 1 < len(order) else w.final_norm)
+            entry = None
+            if run + 1 in starts:
+                t = starts[run + 1]
+                entry = ops.PassEntry(first if t else None, w.loop_step[t])
+            mix = lw.mixer.decode if meta.is_decode else lw.mixer.prefill
+            d, last = mix(x, meta, cache, run), (after, entry)
+            nothing = (None, None)
+            if lw.ff is not None:
+                x = ops.post_add_(resid, d, post(lw.post1), norm(lw.norm2))
+                x = lw.ff.finish_post_(resid, lw.ff.forward(x, meta.ids), post(lw.post2), *(nothing if lw.side else last))
+            else:
+                x = ops.post_add_(resid, d, post(lw.post1), *(nothing if lw.side else last))
+            if lw.side is not None:
+                x = ops.token_side_(resid, x, meta.ids, lw.side, post(lw.side_norm), *last)
+            if self.layer_probe is not None:
+                self.layer_probe(run, resid if entry is None else resid - entry.step - (0.0 if entry.again is None else entry.again))
+        return x
+
     def _beside(self, meta: StepMeta, work):
         """Start ``work`` beside what the caller launches next; the returned function waits for it and gives its
         result.  Small decode steps leave most of the machine idle, so there the two run on two streams (inside
@@ -267,7 +305,8 @@ class ModelRunner:
         return join
 
     def _logits(self, x: torch.Tensor) -> torch.Tensor:
-        return linear_fwd(x, self.weights.lm_head)
+        y, cap = linear_fwd(x, self.weights.lm_head), getattr(self.cfg, "logit_softcap", 0.0)
+        return ops.soft_cap_(y, cap) if cap else y
 
     # ------------------------------------------------------------------------------------------
     @torch.no_grad()
