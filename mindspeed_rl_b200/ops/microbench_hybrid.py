@@ -8,12 +8,14 @@ from __future__ import annotations
 
 import torch
 
-from . import (ConvHeads, ConvNormWeights, DeltaLayout, DeltaWeights, GroupedHeads, LatentLayout, MemoryLayout, MemoryWeights,
-               PostNorm, ScoreForm, add_norm_, angle_table, conv_qkv_decode, conv_qkv_prefill, delta_decode, delta_prefill, embed_norm,
+from . import (ConvHeads, ConvNormWeights, DeltaLayout, DeltaWeights, GRULayout, GroupedHeads, LatentLayout, MemoryLayout,
+               MemoryWeights, Norm, PassEntry, PostNorm, ScoreForm, TokenSide, WKVWeights, add_norm_, angle_table, conv_qkv_decode, conv_qkv_prefill, delta_decode, delta_prefill, embed_norm,
                glu_fwd, latent_decode_attention, latent_prefill_attention, latent_prep, latent_rotate_queries, latent_spread_,
-               memory_decode, memory_prefill, moe_combine_norm_, moe_post_add_, post_add_, qkv_prep_, rope_table, rows_gather,
-               window_decode_attention, window_prefill_attention)
+               memory_decode, memory_prefill, min_gru_decode, min_gru_prefill, moe_combine_norm_, moe_post_add_, post_add_,
+               post_embed, qkv_prep_, rope_table, rows_gather, soft_cap_, token_side_, turn_back, turned_prep_,
+               window_decode_attention, window_prefill_attention, wkv_decode, wkv_mix_decode, wkv_mix_prefill, wkv_prefill)
 from . import moe as K
+from .matrix_memory import constant_decay
 from .microbench import report, timeit
 
 
@@ -128,31 +130,38 @@ def case_stream(small: bool, iters: int):
         report(f"moe_combine_norm T={t} k={k} H={h}", ms, bytes_=t * h * (2.0 * k + 4 + 8 + 2))
 
 
-def _memory(t, slots, heads, dim, vdim):
+def _memory(t, slots, heads, dim, vdim, retention=False):
     n = heads * (2 * dim + 2 * vdim)
-    lay = MemoryLayout(heads, dim, vdim, vdim, 0, heads * dim, 2 * heads * dim, heads * (2 * dim + vdim), dim ** -0.5, 15.0)
-    w = MemoryWeights(torch.zeros(2 * heads, device="cuda"), torch.ones(heads * vdim, device="cuda"))
+    lay = MemoryLayout(heads, dim, vdim, vdim, 0, heads * dim, 2 * heads * dim, heads * (2 * dim + vdim), dim ** -0.5, 15.0,
+                       silu_gate=retention)
+    w = MemoryWeights(torch.zeros(2 * heads, device="cuda"), torch.ones(heads * vdim, device="cuda"),
+                      constant_decay([0.99] * heads).cuda() if retention else None)
     state = {"memory": torch.zeros(slots, heads, dim, vdim, device="cuda"), "norm": torch.zeros(slots, heads, dim, device="cuda"),
              "peak": torch.zeros(slots, heads, device="cuda")}
     return lay, torch.randn(t, n, device="cuda").bfloat16(), torch.randn(t, 2 * heads, device="cuda"), w, state
 
 
-def case_memory(small: bool, iters: int):
+def case_retention(small: bool, iters: int):
+    case_memory(small, iters, True)
+
+
+def case_memory(small: bool, iters: int, retention: bool = False):
     """Roofline of prompts: the rows read and written once (the recurrence's products are far below the tensor peak)."""
+    kind = "retention" if retention else "memory"
     for heads, dim, vdim in ((32, 128, 128), (8, 256, 512)):
         for b, n in ([(1, 2048)] if small else [(1, 8192), (8, 1024), (32, 256)]):
             t = b * n
-            lay, proj, z, w, state = _memory(t, b, heads, dim, vdim)
+            lay, proj, z, w, state = _memory(t, b, heads, dim, vdim, retention)
             cu = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda")
             start, slots = torch.zeros(b, dtype=torch.int32, device="cuda"), torch.arange(b, device="cuda")
             ms = timeit(lambda: memory_prefill(proj, z, lay, w, state, cu, n, start, slots, 1e-5), iters)
-            report(f"memory_prefill {b}x{n} heads={heads} {dim}x{vdim}", ms, bytes_=2.0 * t * heads * (2 * dim + 3 * vdim),
+            report(f"{kind}_prefill {b}x{n} heads={heads} {dim}x{vdim}", ms, bytes_=2.0 * t * heads * (2 * dim + 3 * vdim),
                    flops=4.0 * t * heads * dim * vdim)
         for b in ([32] if small else [1, 32, 256]):
-            lay, proj, z, w, state = _memory(b, b, heads, dim, vdim)
+            lay, proj, z, w, state = _memory(b, b, heads, dim, vdim, retention)
             pos, slots = torch.full((b,), 100, dtype=torch.int32, device="cuda"), torch.randperm(b, device="cuda")
             ms = timeit(lambda: memory_decode(proj, z, lay, w, state, pos, slots, 1e-5), iters)
-            report(f"memory_decode B={b} heads={heads} {dim}x{vdim}", ms, bytes_=8.0 * state["memory"].numel())
+            report(f"{kind}_decode B={b} heads={heads} {dim}x{vdim}", ms, bytes_=8.0 * state["memory"].numel())
 
 
 def case_window(small: bool, iters: int):
@@ -302,6 +311,106 @@ def case_post_norm(small: bool, iters: int):
         report(f"post_add {t}x{h}", ms, bytes_=t * h * 12.0)
 
 
-CASES = {"hybrid_conv": case_conv, "hybrid_gated_latent": case_gated_latent, "hybrid_head_delta": case_head_delta,
+def case_wkv(small: bool, iters: int):
+    """State arithmetic in fp32: three multiply-adds per state entry and token (decayed state, added product, output)."""
+    heads, dim, rank, width = 64, 64, 64, 2304
+    hd = heads * dim
+    g = torch.Generator(device="cuda").manual_seed(0)
+    rnd = lambda *s: torch.randn(*s, device="cuda", generator=g)
+    w = WKVWeights(torch.rand(5, width, device="cuda"), rnd(hd, rank).bfloat16() * 0.1, rnd(hd) - 3, rnd(hd), torch.ones(hd, device="cuda"), heads, dim)
+    for b, n in ([(1, 2048)] if small else [(1, 8192), (8, 1024), (32, 256), (8, 2048)]):
+        t = b * n
+        r, k, v, gate = (rnd(t, hd).bfloat16() for _ in range(4))
+        a, h = rnd(t, rank), rnd(t, width).bfloat16()
+        state, last = torch.zeros(b, heads, dim, dim, device="cuda"), torch.zeros(b, width, device="cuda")
+        cu = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda")
+        seq = torch.arange(b, dtype=torch.int32, device="cuda").repeat_interleave(n)
+        start, slots = torch.zeros(b, dtype=torch.int32, device="cuda"), torch.arange(b, device="cuda")
+        ms = timeit(lambda: wkv_prefill(r, k, v, gate, a, w, state, cu, n, start, slots, 1e-5), iters)
+        flops = 6.0 * t * heads * dim * dim
+        report(f"wkv_prefill {b}x{n} heads={heads} dim={dim}", ms, bytes_=10.0 * t * hd + 4.0 * t * rank,
+               note=f"{flops / ms / 1e9:.1f} TFLOP/s fp32 = {flops / ms / 1e9 / fp32_tflops():.3f} of nominal fp32")
+        ms = timeit(lambda: wkv_mix_prefill(h, w.mu, last, seq, cu, start, slots), iters)
+        report(f"wkv_mix T={t} W={width}", ms, bytes_=12.0 * t * width)
+    for b in ([32] if small else [1, 32, 256]):
+        r, k, v, gate = (rnd(b, hd).bfloat16() for _ in range(4))
+        a, h = rnd(b, rank), rnd(b, width).bfloat16()
+        state, last = torch.zeros(b, heads, dim, dim, device="cuda"), torch.zeros(b, width, device="cuda")
+        pos, slots = torch.full((b,), 100, dtype=torch.int32, device="cuda"), torch.randperm(b, device="cuda")
+        ms = timeit(lambda: wkv_decode(r, k, v, gate, a, w, state, pos, slots, 1e-5), iters)
+        report(f"wkv_decode B={b} heads={heads} dim={dim}", ms, bytes_=8.0 * state.numel() + 10.0 * b * hd + 2.0 * hd * rank)
+        ms = timeit(lambda: wkv_mix_decode(h, w.mu, last, pos, slots), iters)
+        report(f"wkv_mix decode B={b} W={width}", ms, bytes_=20.0 * b * width)
+
+
+def case_parallel(small: bool, iters: int):
+    """Around the attention with turned values, and the gated recurrence beside it."""
+    h, g, d, width = 32, 8, 128, 2304
+    lay = GroupedHeads(h, g, d, d, d, d, 0, h * d, (h + g) * d)
+    c0 = (h + 2 * g) * d
+    gru = GRULayout(width, width, c0, c0 + width, c0 + 2 * width, h * d, 0.7)
+    tab, vtab = (angle_table(8192, tuple(1e4 ** (-i / n) for i in range(n)), "cuda") for n in (32, 64))
+    zb, xb = torch.zeros(width, device="cuda"), torch.zeros(width, device="cuda")
+    for b, n in ([(1, 2048)] if small else [(1, 8192), (8, 2048)]):
+        t = b * n
+        proj = torch.randn(t, c0 + 3 * width, device="cuda").bfloat16()
+        pos, slots = torch.arange(t, dtype=torch.int32, device="cuda") % n, torch.arange(t, device="cuda")
+        kc, vc = (torch.empty(t // 16, 16, g, d, device="cuda").bfloat16() for _ in range(2))
+        ms = timeit(lambda: turned_prep_(proj, lay, 1e-5, tab, vtab, pos, slots, kc, vc), iters)
+        report(f"turned_prep T={t} H={h}/{g} d={d} rot=64", ms, bytes_=2.0 * t * (2 * (h + g) * 64 + 2 * g * d + g * 64 + 2 * g * d))
+        attn, out = torch.randn(t, h * d, device="cuda").bfloat16(), torch.empty(t, h * d + width, device="cuda").bfloat16()
+        ms = timeit(lambda: turn_back(attn, lay, vtab, pos, 0.7, out), iters)
+        report(f"turn_back T={t} H={h} d={d}", ms, bytes_=4.0 * t * h * d)
+        cu = torch.arange(0, t + 1, n, dtype=torch.int32, device="cuda")
+        start, own, state = torch.zeros(b, dtype=torch.int32, device="cuda"), torch.arange(b, device="cuda"), torch.zeros(b, width, device="cuda")
+        ms = timeit(lambda: min_gru_prefill(proj, gru, zb, xb, state, out, cu, n, start, own), iters)
+        report(f"min_gru_prefill {b}x{n} width={width}", ms, bytes_=8.0 * t * width)
+    for b in ([32] if small else [1, 256]):
+        proj, out = torch.randn(b, c0 + 3 * width, device="cuda").bfloat16(), torch.empty(b, h * d + width, device="cuda").bfloat16()
+        pos, own, state = torch.full((b,), 100, dtype=torch.int32, device="cuda"), torch.arange(b, device="cuda"), torch.zeros(b, width, device="cuda")
+        slots, kc, vc = own * 16, *(torch.empty(b, 16, g, d, device="cuda").bfloat16() for _ in range(2))
+        ms = timeit(lambda: turned_prep_(proj, lay, 1e-5, tab, vtab, pos, slots, kc, vc), iters)
+        report(f"turned_prep decode B={b} H={h}/{g}", ms, bytes_=2.0 * b * (2 * (h + g) * 64 + 5 * g * d + g * 64))
+        attn = torch.randn(b, h * d, device="cuda").bfloat16()
+        ms = timeit(lambda: turn_back(attn, lay, vtab, pos, 0.7, out), iters)
+        report(f"turn_back decode B={b} H={h}", ms, bytes_=4.0 * b * h * d)
+        ms = timeit(lambda: min_gru_decode(proj, gru, zb, xb, state, out, pos, own), iters)
+        report(f"min_gru_decode B={b} width={width}", ms, bytes_=16.0 * b * width)
+
+
+def case_sandwich(small: bool, iters: int):
+    """Norms around sublayers, token inputs, pass inputs, the router over the chosen and capped logits."""
+    e, k, h, dim = 64, 8, 2304, 64
+    table, rows = (torch.randn(32768, n, device="cuda").bfloat16() for n in (h, 4 * dim))
+    w, step = torch.ones(h, device="cuda"), torch.ones(h, device="cuda")
+    post, after = PostNorm(w, 1e-5), Norm(w, 1e-5)
+    side = TokenSide(torch.randn(dim, h, device="cuda").bfloat16(), torch.randn(h, dim, device="cuda").bfloat16(), rows, dim, dim)
+    for t in ([2048] if small else [16384, 256, 32, 1]):
+        ids = torch.randint(0, 32768, (t,), device="cuda")
+        x, resid, again = torch.randn(t, h, device="cuda").bfloat16(), torch.zeros(t, h, device="cuda"), torch.zeros(t, h, device="cuda")
+        ms = timeit(lambda: post_embed(ids, table, post, after, True, step), iters)
+        report(f"post_embed {t}x{h}", ms, bytes_=t * h * 12.0)
+        ms = timeit(lambda: post_add_(resid, x, post, after), iters)
+        report(f"post_add + norm {t}x{h}", ms, bytes_=t * h * 12.0)
+        ms = timeit(lambda: post_add_(resid, x, post, after, PassEntry(again, step)), iters)
+        report(f"post_add + pass input + norm {t}x{h}", ms, bytes_=t * h * 16.0)
+        z = torch.randn(t, e, device="cuda")
+        ms = timeit(lambda: K.route_top(z, k, True), iters)
+        report(f"route_top over the chosen T={t} E={e} k={k}", ms, bytes_=t * (4.0 * e + 12 * k))
+        idx, score = K.route_top(z, k, True)
+        plan = K.moe_plan(idx, e)
+        y = torch.randn(plan.max_rows, h, device="cuda").bfloat16()
+        ms = timeit(lambda: moe_post_add_(resid, y, plan.pos, score, post), iters)
+        report(f"moe_post_add T={t} k={k} H={h}", ms, bytes_=t * h * (2.0 * k + 8 + 2))
+        for fused in (0, 1 << 20):
+            ms = timeit(lambda: token_side_(resid, x, ids, side, post, after, fused_tokens=fused), iters)
+            report(f"token_side {'one kernel' if fused else 'products'} {t}x{h} dim={dim}", ms, bytes_=t * h * (10.0 if fused else 16.0) + 4.0 * h * dim)
+    logits = torch.randn(32 if small else 256, 151936, device="cuda").bfloat16()
+    ms = timeit(lambda: soft_cap_(logits, 30.0), iters)
+    report(f"soft_cap {logits.shape[0]}x151936", ms, bytes_=4.0 * logits.numel())
+
+
+CASES = {"hybrid_retention": case_retention, "hybrid_wkv": case_wkv, "hybrid_parallel": case_parallel, "hybrid_sandwich": case_sandwich,
+         "hybrid_conv": case_conv, "hybrid_gated_latent": case_gated_latent, "hybrid_head_delta": case_head_delta,
          "hybrid_post_norm": case_post_norm, "hybrid_memory": case_memory, "hybrid_window": case_window, "hybrid_routed": case_routed,
          "hybrid_delta": case_delta, "hybrid_latent": case_latent, "hybrid_stream": case_stream}

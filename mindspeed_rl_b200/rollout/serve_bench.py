@@ -15,6 +15,9 @@ Gapevik: ``conv`` has convolved attention in chunks everywhere, ``gated`` latent
 and gates, ``delta`` the delta rule with a decay per head, ``gapevik`` the three in turn.  Closest existing models of the same
 width, heads, experts and layer count: ``window``, ``latent`` and ``mixed``.
 
+Lunelorn: ``retention``, ``turned`` (attention with turned values beside the minimal gated recurrence) and ``wkv`` have that mixer
+everywhere, ``lunelorn`` the three in turn; no layer is looped.  Closest existing models: ``memory``, ``gqa`` and ``delta``.
+
 One JSON line per measurement: tokens/s from CUDA events around the engine calls.
 """
 from __future__ import annotations
@@ -25,9 +28,10 @@ from typing import List
 
 import torch
 
-from ..models.hybrid_config import (ChannelDeltaSpec, Chunk, ConvAttentionSpec, GluSpec, HeadDeltaSpec, HybridConfig,
-                                    LatentAttentionSpec, LayerSpec, MatrixMemorySpec, Rotary, ScoredMoESpec, SoftmaxMoESpec,
-                                    TableMoESpec, WavelengthScaling, WindowAttentionSpec)
+from ..models.hybrid_config import (ChannelDeltaSpec, ChosenMoESpec, Chunk, ConvAttentionSpec, GluSpec, HeadDeltaSpec, HybridConfig,
+                                    LatentAttentionSpec, LayerSpec, MatrixMemorySpec, MinGRUSpec, ParallelSpec, RetentionSpec,
+                                    Rotary, ScoredMoESpec, SoftmaxMoESpec, TableMoESpec, TurnedAttentionSpec, WKVSpec,
+                                    WavelengthScaling, WindowAttentionSpec)
 from ..models.transformer_config import TransformerConfig
 from .engine import LLMEngine
 from .scheduler import SamplingParams
@@ -56,7 +60,8 @@ PREFILL = ((1, 8192), (8, 2048))
 DECODE = ((1, 2048), (32, 2048), (256, 2048))
 NEW_TOKENS = 64
 WINDOW = 1024
-MODELS = ("mla", "latent", "mixed", "gqa", "window", "memory", "sunatar", "conv", "gated", "delta", "gapevik")
+MODELS = ("mla", "latent", "mixed", "gqa", "window", "memory", "sunatar", "conv", "gated", "delta", "gapevik", "retention", "turned", "wkv",
+          "lunelorn")
 
 
 def sunatar_config(s: Size, pattern: str) -> HybridConfig:
@@ -83,7 +88,21 @@ def gapevik_config(s: Size, pattern: str) -> HybridConfig:
     return HybridConfig("Gapevik", s.vocab, s.width, layers, 1e-5, residual_mult=0.5)
 
 
+def lunelorn_config(s: Size, pattern: str) -> HybridConfig:
+    left = TurnedAttentionSpec(s.heads, s.heads // 4, 128, 128, 128 ** -0.5, Rotary(64, 500000.0, halves=True))
+    kinds = {"retention": RetentionSpec(s.heads, 128, 128, tuple(1.0 - 2.0 ** (-5 - 8 * i / s.heads) for i in range(s.heads))),
+             "turned": ParallelSpec(left, MinGRUSpec(s.width), 0.7, 0.7), "wkv": WKVSpec(2 * s.heads, 64, s.width)}
+    moe = ChosenMoESpec(s.experts, s.top, GluSpec(s.expert_ff, "silu"))
+    layers = []
+    for i in range(s.layers):
+        name = pattern if pattern in kinds else ("wkv", "retention", "turned")[i % 3]
+        layers.append(LayerSpec("parallel" if name == "turned" else name, kinds[name], moe))
+    return HybridConfig("Lunelorn", s.vocab, s.width, layers, 1e-5, token_side=64, logit_softcap=30.0)
+
+
 def hybrid_config(s: Size, pattern: str) -> HybridConfig:
+    if pattern in ("retention", "turned", "wkv", "lunelorn"):
+        return lunelorn_config(s, pattern)
     if pattern in ("conv", "gated", "delta", "gapevik"):
         return gapevik_config(s, pattern)
     if pattern in ("window", "memory", "sunatar"):
@@ -122,12 +141,48 @@ def random_state(cfg: HybridConfig, device) -> dict:
     vec("final.norm", w, ones)
     if not cfg.design.tied_head:
         lin("head", cfg.vocab_size, w)
+    if cfg.design.embed_norm:
+        vec("embed.norm", w, ones)
+    if cfg.token_side:
+        lin("side.embed", cfg.vocab_size, len(cfg.layers) * cfg.token_side)
     for i, l in enumerate(cfg.layers):
         p, m = f"l{i}.mix.", l.mixer
         vec(f"l{i}.norm1", w, ones)
         if not cfg.design.parallel:
             vec(f"l{i}.norm2", w, ones)
-        if isinstance(m, LatentAttentionSpec):
+        if cfg.design.sandwich:
+            vec(f"l{i}.norm1b", w, ones)
+            vec(f"l{i}.norm2b", w, ones)
+        if cfg.token_side:
+            lin(f"l{i}.side.gate", cfg.token_side, w)
+            lin(f"l{i}.side.proj", w, cfg.token_side)
+            vec(f"l{i}.side.norm", w, ones)
+        if isinstance(m, RetentionSpec):
+            for n, rows in (("q", m.heads * m.dim), ("k", m.heads * m.dim), ("v", m.heads * m.vdim), ("g", m.heads * m.vdim)):
+                lin(p + n, rows, w)
+            lin(p + "o", w, m.heads * m.vdim)
+        elif isinstance(m, ParallelSpec):
+            a, r = m.left, m.right.width
+            for n, rows in (("left.q", a.heads * a.dim), ("left.k", a.kv_heads * a.dim), ("left.v", a.kv_heads * a.vdim),
+                            ("right.z", r), ("right.x", r), ("right.g", r)):
+                lin(p + n, rows, w)
+            vec(p + "right.z.b", r, -2.0)
+            vec(p + "right.x.b", r)
+            lin(p + "left.o", w, a.heads * a.vdim)
+            lin(p + "right.o", w, r)
+        elif isinstance(m, WKVSpec):
+            hd = m.heads * m.dim
+            for n in "rkvgw":
+                vec(p + "mu." + n, w, 0.5)
+            for n in "rkvg":
+                lin(p + n, hd, w)
+            lin(p + "w1", 64, w)
+            lin(p + "w2", hd, 64)
+            vec(p + "w0", hd, -3.0)
+            vec(p + "u", hd, 0.5)
+            vec(p + "norm", hd, 1.0)
+            lin(p + "o", w, hd)
+        elif isinstance(m, LatentAttentionSpec):
             if m.q_rank:
                 lin(p + "dq", m.q_rank, w)
                 vec(p + "dq.norm", m.q_rank, 1.0)
@@ -189,6 +244,10 @@ def random_state(cfg: HybridConfig, device) -> dict:
                 glu(f"{p}e{e}.", l.mlp.expert.ff)
             lin(p + "router", l.mlp.experts, w)
             glu(p + "shared.", l.mlp.shared.ff)
+        elif isinstance(l.mlp, ChosenMoESpec):
+            for e in range(l.mlp.experts):
+                glu(f"{p}e{e}.", l.mlp.expert.ff)
+            lin(p + "router", l.mlp.experts, w)
         elif isinstance(l.mlp, SoftmaxMoESpec):
             for e in range(l.mlp.experts):
                 glu(f"{p}e{e}.", l.mlp.expert.ff)
