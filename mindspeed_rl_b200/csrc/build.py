@@ -33,7 +33,7 @@ NVCC_FLAGS = [
 # without the approximate divisions, square roots, exponentials and flush-to-zero of --use_fast_math
 PRECISE = {"residual_stream", "delta_rule", "latent_attention", "latent_decode_tcgen05", "grouped_gemm_simt",
            "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "conv_qkv", "attention_simt",
-           "moe", "wkv", "min_gru"}
+           "moe", "wkv", "wkv_chunk", "min_gru"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread"]
 
 
@@ -44,7 +44,7 @@ _STREAM = ("residual_stream", "grouped_gemm_simt", "moe", "moe_gemm_tcgen05", "a
 GROUPS = {
     "pumotar": (*_STREAM, "delta_rule", "latent_attention", "latent_decode_tcgen05"),
     "gapevik": (*_STREAM, "delta_rule", "latent_attention", "latent_decode_tcgen05", "conv_qkv", "decode", "decode_prefix_tcgen05"),
-    "lunelorn": (*_STREAM, "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "wkv", "min_gru", "decode", "decode_prefix_tcgen05"),
+    "lunelorn": (*_STREAM, "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "wkv", "wkv_chunk", "min_gru", "decode", "decode_prefix_tcgen05"),
     "sunatar": (*_STREAM, "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "decode", "decode_prefix_tcgen05"),
 }
 

@@ -31,15 +31,30 @@ __device__ __forceinline__ void stf4(__nv_bfloat16* p, const float (&f)[4]) {
   *reinterpret_cast<uint2*>(p) = t;
 }
 
-// V elements (1 or 4) at once
+__device__ __forceinline__ void ldf2(const float* p, float (&f)[4]) {
+  const float2 t = *reinterpret_cast<const float2*>(p);
+  f[0] = t.x; f[1] = t.y;
+}
+__device__ __forceinline__ void ldf2(const __nv_bfloat16* p, float (&f)[4]) {
+  const float2 t = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+  f[0] = t.x; f[1] = t.y;
+}
+__device__ __forceinline__ void stf2(float* p, const float (&f)[4]) { *reinterpret_cast<float2*>(p) = make_float2(f[0], f[1]); }
+__device__ __forceinline__ void stf2(__nv_bfloat16* p, const float (&f)[4]) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(f[0], f[1]);
+}
+
+// V elements (1, 2 or 4) at once
 template <int V, typename T>
 __device__ __forceinline__ void ldv(const T* p, float (&f)[4]) {
   if constexpr (V == 4) ldf4(p, f);
+  else if constexpr (V == 2) ldf2(p, f);
   else f[0] = ldf(p);
 }
 template <int V, typename T>
 __device__ __forceinline__ void stv(T* p, const float (&f)[4]) {
   if constexpr (V == 4) stf4(p, f);
+  else if constexpr (V == 2) stf2(p, f);
   else stf(p, f[0]);
 }
 

@@ -31,12 +31,22 @@ struct Args {
 
 __device__ __forceinline__ long long seg_id(int t0, int b, int j) { return t0 / SEG + b + j; }
 
+// bf16 rows do not need the last bits of the exponential and the division
 template <typename T>
 __device__ __forceinline__ void step_of(float zp, float xp, float zb, float xb, float& keep, float& add) {
   zp += zb;
-  const float u = xp + xb, e = expf(-fabsf(zp)), z = zp >= 0.f ? 1.f / (1.f + e) : e / (1.f + e);
-  keep = zp >= 0.f ? e / (1.f + e) : 1.f / (1.f + e);
-  add = z * (u >= 0.f ? u + 0.5f : sigmoid_f(u));
+  const float u = xp + xb, a = fabsf(zp);
+  float e, inv;
+  if constexpr (sizeof(T) == 2) {
+    e = __expf(-a);
+    inv = __fdividef(1.f, 1.f + e);
+  } else {
+    e = expf(-a);
+    inv = 1.f / (1.f + e);
+  }
+  const float small = e * inv, z = zp >= 0.f ? inv : small;
+  keep = zp >= 0.f ? small : 1.f - small;
+  add = z * (u >= 0.f ? u + 0.5f : sigmoid_t<T>(u));
 }
 
 // OUT: outputs from the state before the segment; otherwise the segment's factor and sum.  WHOLE: one segment holds the
@@ -161,9 +171,9 @@ MSRL_API int msrl_min_gru(const void* z, const void* x, const void* g, long long
     const gru::Args<T> p{(const T*)z, (const T*)x, (const T*)g, ld, z_bias, x_bias, state, cu, start, slots, scale, (T*)y, y_ld,
                          width, padded, scratch, scratch + (n + 3) / 4 * 4};
     const int most = cu == nullptr ? 1 : (max_q + gru::SEG - 1) / gru::SEG;
-    auto at4 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & (4 * sizeof(T) - 1)) == 0; };
-    const bool v4 = width % 4 == 0 && padded % 4 == 0 && ld % 4 == 0 && y_ld % 4 == 0 && at4(z) && at4(x) && at4(g) && at4(y);
-    return v4 ? gru::launch<T, 4>(p, most, batch, st) : gru::launch<T, 1>(p, most, batch, st);
+    auto at2 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & (2 * sizeof(T) - 1)) == 0; };
+    const bool v2 = width % 2 == 0 && padded % 2 == 0 && ld % 2 == 0 && y_ld % 2 == 0 && at2(z) && at2(x) && at2(g) && at2(y);
+    return v2 ? gru::launch<T, 2>(p, most, batch, st) : gru::launch<T, 1>(p, most, batch, st);
   };
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }

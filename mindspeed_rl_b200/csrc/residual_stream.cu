@@ -14,9 +14,7 @@
 //                     Between the add and y: resid[t] += again[t] + step (what a pass of a loop adds before it runs)
 //   post_embed        the same with d = table[id[t]] and a residual that starts at zero; `first` keeps it as it was before
 //                     `step`
-//   side_add          the same with d = proj (gelu_tanh(gate resid[t]) * rows[id[t]]), one block per token from the gate to
-//                     the norm; for few tokens
-//   side_gate         g[t] = gelu_tanh(g[t]) * rows[id[t]]  (many tokens: gate and proj are matrix products)
+//   side_gate         g[t] = gelu_tanh(g[t]) * rows[id[t]], or for few tokens with the product in it: g[t] = x[t] gate^T
 //   soft_cap          x = cap * tanh(x / cap)
 //
 //   glu               act(gate) * up of rows [gate | up]: silu, tanh-gelu, or the clamped swish with (up + 1)
@@ -392,83 +390,28 @@ __device__ __forceinline__ float gelu_tanh_t(float g) {
   return g * sigmoid_t<T>(k * (g + 0.044715f * g * g * g));
 }
 
-template <typename T>
-struct SideArgs {
-  const T* gate;                          // [dim, W]
-  const T* proj;                          // [W, dim]
-  const T* rows;                          // [vocabulary, ld]; the layer's entries start at `col`
-  const long long* ids;
-  long long ld;
-  int col, dim;
-};
-
-// One block per token.  dynamic shared memory: the residual's row, the gate's outputs
-template <typename T, bool ENTRY>
-__global__ void __launch_bounds__(RS_THREADS) side_add_kernel(const PostArgs<T> p, const SideArgs<T> s) {
-  extern __shared__ float sm[];
-  __shared__ float red[32];
-  const long long t = blockIdx.x;
-  const int W = p.W, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  float* row = sm;
-  float* d = sm + W;                      // what is to be normed
-  float* g = d + W;
-  const float* res = p.resid + t * W;
-  for (int c = threadIdx.x; c < W; c += RS_THREADS) row[c] = res[c];
-  __syncthreads();
-  const T* tab = s.rows + s.ids[t] * s.ld + s.col;
-  const bool v4 = W % 4 == 0;
-  for (int j = warp; j < s.dim; j += RS_THREADS / 32) {
-    const T* w = s.gate + (long long)j * W;
-    float acc = 0.f;
-    if (v4) {
-#pragma unroll 4
-      for (int c = lane * 4; c < W; c += 128) {
-        float f[4];
-        ldf4(w + c, f);
-        const float4 x = *reinterpret_cast<const float4*>(row + c);
-        acc += f[0] * x.x + f[1] * x.y + f[2] * x.z + f[3] * x.w;
-      }
-    } else {
-      for (int c = lane; c < W; c += 32) acc += ldf(w + c) * row[c];
+// One warp per token and gate output: few tokens leave a matrix product nothing to share.  grid (padded dim / 8, tokens)
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+side_gate_product_kernel(const T* x, const T* gate, T* g, long long g_ld, const T* rows, const long long* ids, long long ld, int col,
+                         int dim, int W) {
+  const long long t = blockIdx.y;
+  const int j = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (j >= g_ld) return;
+  float acc = 0.f;
+  if (j < dim) {
+    const T *a = x + t * W, *b = gate + (long long)j * W;
+#pragma unroll 8
+    for (int c = lane * V; c < W; c += 32 * V) {
+      float f[4], h[4];
+      ldv<V>(a + c, f);
+      ldv<V>(b + c, h);
+#pragma unroll
+      for (int i = 0; i < V; ++i) acc += f[i] * h[i];
     }
-    acc = warp_sum(acc);
-    if (lane == 0) g[j] = gelu_tanh_t<T>(acc) * ldf(tab + j);
   }
-  __syncthreads();
-  float ss = 0.f;
-  const bool quads = s.dim % 4 == 0;
-  for (int c = threadIdx.x; c < W; c += RS_THREADS) {
-    const T* w = s.proj + (long long)c * s.dim;
-    float acc = 0.f;
-    if (quads) {
-#pragma unroll 4
-      for (int j = 0; j < s.dim; j += 4) {
-        float f[4];
-        ldf4(w + j, f);
-        acc += f[0] * g[j] + f[1] * g[j + 1] + f[2] * g[j + 2] + f[3] * g[j + 3];
-      }
-    } else {
-      for (int j = 0; j < s.dim; ++j) acc += ldf(w + j) * g[j];
-    }
-    d[c] = acc;
-    ss += acc * acc;
-  }
-  const float inv = p.mult / sqrtf(block_sum(ss, red) / (float)W + p.eps);
-  float sum = 0.f;
-  for (int c = threadIdx.x; c < W; c += RS_THREADS) {
-    float a[4], b[4];
-    a[0] = row[c];
-    b[0] = d[c];
-    post_sum<T, 1, ENTRY>(p, t, c, inv, b, a, sum);
-    row[c] = a[0];
-  }
-  if (p.after_w == nullptr) return;
-  const float q = 1.f / sqrtf(block_sum(sum, red) / (float)W + p.after_eps);
-  for (int c = threadIdx.x; c < W; c += RS_THREADS) {
-    float a[4];
-    a[0] = row[c];
-    post_after<T, 1>(p, t, c, q, a);
-  }
+  acc = warp_sum(acc);
+  if (lane == 0) stf(g + t * g_ld + j, j < dim ? gelu_tanh_t<T>(acc) * ldf(rows + ids[t] * ld + col + j) : 0.f);
 }
 
 // entries past `dim` of a padded row become zero
@@ -489,7 +432,8 @@ __global__ void __launch_bounds__(256) soft_cap_kernel(T* x, long long n, float 
   float f[4];
   ldv<V>(x + i, f);
 #pragma unroll
-  for (int k = 0; k < V; ++k) f[k] = cap * tanhf(f[k] / cap);
+  for (int k = 0; k < V; ++k)          // bf16 results: tanh z = 1 - 2 / (e^2z + 1) without the last bits
+    f[k] = sizeof(T) == 2 ? cap - __fdividef(2.f * cap, __expf(2.f * f[k] / cap) + 1.f) : cap * tanhf(f[k] / cap);
   stv<V>(x + i, f);
 }
 
@@ -670,21 +614,17 @@ MSRL_API int msrl_post_embed(const long long* ids, const void* table, float* res
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
-MSRL_API int msrl_side_add(const void* gate, const void* proj, const void* table, const long long* ids, long long ld, int col,
-                           int dim, float* resid, const float* norm_w, float eps, const float* after_w, float after_eps,
-                           const float* again, const float* step, void* y, long long rows, int W, int is_f32,
-                           cudaStream_t st) {
+// x [rows, W] -> g [rows, g_ld] with gate [>= dim, W]
+MSRL_API int msrl_side_gate_product(const void* x, const void* gate, void* g, long long g_ld, const void* table,
+                                    const long long* ids, long long ld, int col, int dim, long long rows, int W, int is_f32,
+                                    cudaStream_t st) {
   if (rows == 0) return 0;
-  const size_t smem = (2 * (size_t)W + dim) * sizeof(float);
-  if (smem > 200 * 1024) return (int)cudaErrorNotSupported;
+  if (rows > 65535) return (int)cudaErrorNotSupported;
+  const dim3 grid((unsigned)((g_ld + 7) / 8), (unsigned)rows);
   auto run = [&](auto tag) {
     using T = decltype(tag);
-    const PostArgs<T> p = post_args<T>(resid, norm_w, eps, 1.f, after_w, after_eps, again, step, y, W);
-    const SideArgs<T> s{(const T*)gate, (const T*)proj, (const T*)table, ids, ld, col, dim};
-    auto* kernel = again != nullptr || step != nullptr ? side_add_kernel<T, true> : side_add_kernel<T, false>;
-    const cudaError_t rc = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (rc != cudaSuccess) return (int)rc;
-    kernel<<<(unsigned)rows, RS_THREADS, smem, st>>>(p, s);
+    auto* kernel = W % 4 == 0 ? side_gate_product_kernel<T, 4> : side_gate_product_kernel<T, 1>;
+    kernel<<<grid, 256, 0, st>>>((const T*)x, (const T*)gate, (T*)g, g_ld, (const T*)table, ids, ld, col, dim, W);
     return (int)cudaGetLastError();
   };
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});

@@ -12,9 +12,10 @@
 // fp32 instructions.  A batch that fills the machine runs each sequence from end to end.  Otherwise sequences are cut into
 // segments: what every segment adds to the state and the product of its decays (all segments in parallel), a pass over the
 // segments that leaves the state before each one, and the scan of every segment from there.  Decays are only ever
-// multiplied.  Decode is one kernel: S read and written once, coalesced.
-#include "dtype_utils.cuh"
+// multiplied.  bf16 rows of the usual sizes take sixteen tokens at a time on the tensor cores (wkv_chunk.cu), others one
+// after the other.  Decode is one kernel: S read and written once, coalesced.
 #include "packed_f32.cuh"
+#include "wkv.cuh"
 
 namespace msrl {
 namespace wkv {
@@ -95,31 +96,7 @@ decay_kernel(const float* a, const T* w2, const float* w0, float* w, int tokens,
     if (s < nt) w[(long long)(t0 + s) * channels + c] = decay_of(acc[s]);
 }
 
-// ---- recurrence ------------------------------------------------------------------------------------------------
-template <typename T>
-struct Args {
-  const T *r, *k, *v, *g;                // [tokens, H * dim]
-  const float* w;                        // decays, [tokens, H * dim]
-  const float *u, *norm;                 // [H * dim]
-  float* state;                          // [slots, H, dim, dim]
-  const int* cu;
-  const int* start;
-  const long long* slots;
-  T* y;                                  // [tokens, H * dim]
-  int H, dim;
-  float eps;
-  int L;                                 // tokens of a segment
-  float* seg;                            // [segments, H, dim, dim]: added states, then the states before the segments
-  float* seg_w;                          // [segments, H, dim]: products of decays
-  float* o;                              // [tokens, H * dim] where a head's columns are spread over blocks, else null
-};
-
-__device__ __forceinline__ long long seg_id(int t0, int b, int j, int L) { return t0 / L + b + j; }
-
-constexpr int TT = 16;                   // tokens per tile
-
-enum { WHOLE = 0, ADDED = 1, FROM_SEGMENT = 2 };
-
+// ---- recurrence, token by token ----------------------------------------------------------------------------------
 constexpr int scan_floats(int DP, int CS) { return TT * (3 * DP + 3 * CS + 1); }
 
 // DP: padded dim; CS value columns of a block; KL lanes share a pair of columns.  grid (segments x column slices, H, B)
@@ -325,11 +302,11 @@ __global__ void __launch_bounds__(256) finish_kernel(const Args<T> p, long long 
 // ---- decode ----------------------------------------------------------------------------------------------------
 constexpr int DB = 4;                    // state rows of a thread in flight
 
-// One block per (head, sequence); `start` holds positions.  V columns of a row per thread.  The decays come from the
-// bottleneck's row a.  dynamic shared memory: r, k, w [dim], tanh(a) [rank], partial outputs [lanes][dim]
+// One block per (head, sequence); `start` holds positions.  V columns of a row per thread.  Decays are read, or come from the
+// bottleneck's row a, `per` lanes a channel.  dynamic shared memory: r, k, w [dim], tanh(a) [rank], partial outputs [lanes][dim]
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
-decode_kernel(const Args<T> p, const float* a, const T* w2, const float* w0, int rank, int lanes) {
+decode_kernel(const Args<T> p, const float* a, const T* w2, const float* w0, int rank, int lanes, int per) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
   const int h = blockIdx.x, b = blockIdx.y, dim = p.dim;
@@ -353,17 +330,36 @@ decode_kernel(const Args<T> p, const float* a, const T* w2, const float* w0, int
     }
   };
   fetch(rl);                             // on its way while the decays are computed
-  for (int j = threadIdx.x; j < rank; j += 256) sa[j] = tanhf(a[(long long)b * rank + j]);
-  __syncthreads();
   float bonus = 0.f;
   for (int d = threadIdx.x; d < dim; d += 256) {
-    const T* row = w2 + (long long)(h * dim + d) * rank;
-    float x = w0[h * dim + d];
-    for (int j = 0; j < rank; ++j) x += sa[j] * ldf(row + j);
     sr[d] = ldf(p.r + at + d);
     sk[d] = ldf(p.k + at + d);
-    sw[d] = decay_of(x);
+    if (p.w != nullptr) sw[d] = p.w[at + d];
     bonus += sr[d] * p.u[h * dim + d] * sk[d];
+  }
+  if (p.w == nullptr) {
+    for (int j = threadIdx.x; j < rank; j += 256) sa[j] = tanhf(a[(long long)b * rank + j]);
+    __syncthreads();
+    const int part_of = threadIdx.x % per;
+    for (int d0 = 0; d0 < dim; d0 += 256 / per) {
+      const int d = d0 + threadIdx.x / per;
+      float x = 0.f;
+      if (d < dim) {
+        const T* row = w2 + (long long)(h * dim + d) * rank;
+        if (rank % 4 == 0) {
+#pragma unroll 4
+          for (int j = part_of * 4; j < rank; j += per * 4) {
+            float f[4];
+            ldf4(row + j, f);
+            x += f[0] * sa[j] + f[1] * sa[j + 1] + f[2] * sa[j + 2] + f[3] * sa[j + 3];
+          }
+        } else {
+          for (int j = part_of; j < rank; j += per) x += ldf(row + j) * sa[j];
+        }
+      }
+      for (int m = per / 2; m > 0; m >>= 1) x += __shfl_xor_sync(0xffffffffu, x, m);
+      if (d < dim && part_of == 0) sw[d] = decay_of(x + w0[h * dim + d]);
+    }
   }
   bonus = block_sum(bonus, red);         // (synchronises sr, sk, sw)
   float v[4], o[4] = {0.f, 0.f, 0.f, 0.f};
@@ -403,6 +399,12 @@ decode_kernel(const Args<T> p, const float* a, const T* w2, const float* w0, int
   }
 }
 
+template <typename T>
+int launch_carry(const Args<T>& p, int batch, cudaStream_t st) {
+  carry_kernel<T><<<dim3((unsigned)((p.dim * p.dim + 255) / 256), (unsigned)p.H, (unsigned)batch), 256, 0, st>>>(p);
+  return (int)cudaGetLastError();
+}
+
 template <typename T, int DP, int CS, int KL, int V>
 int launch_scan(const Args<T>& p, int most, int batch, cudaStream_t st) {
   const int slices = (p.dim + CS - 1) / CS, smem = scan_floats(DP, CS) * (int)sizeof(float);
@@ -413,10 +415,9 @@ int launch_scan(const Args<T>& p, int most, int batch, cudaStream_t st) {
     return (int)cudaGetLastError();
   };
   if (most == 1) return go(scan_kernel<T, DP, CS, KL, WHOLE, V>, 1);
-  const int rc = go(scan_kernel<T, DP, CS, KL, ADDED, V>, most);
-  if (rc != 0) return rc;
-  carry_kernel<T><<<dim3((unsigned)((p.dim * p.dim + 255) / 256), (unsigned)p.H, (unsigned)batch), 256, 0, st>>>(p);
-  return go(scan_kernel<T, DP, CS, KL, FROM_SEGMENT, V>, most);
+  int rc = go(scan_kernel<T, DP, CS, KL, ADDED, V>, most);
+  if (rc == 0) rc = launch_carry(p, batch, st);
+  return rc != 0 ? rc : go(scan_kernel<T, DP, CS, KL, FROM_SEGMENT, V>, most);
 }
 
 template <typename T, int V>
@@ -425,6 +426,13 @@ int launch_by_dim(const Args<T>& p, int most, int batch, cudaStream_t st) {
   if (p.dim <= 64) return launch_scan<T, 64, 64, 4, V>(p, most, batch, st);
   if (p.dim <= 128) return launch_scan<T, 128, 128, 8, V>(p, most, batch, st);
   return launch_scan<T, 256, 64, 16, V>(p, most, batch, st);
+}
+
+static int launch_chunks(const Args<__nv_bfloat16>& p, int most, int batch, cudaStream_t st) {
+  if (most == 1) return launch_chunked(p, WHOLE, 1, batch, st);
+  int rc = launch_chunked(p, ADDED, most, batch, st);
+  if (rc == 0) rc = launch_carry(p, batch, st);
+  return rc != 0 ? rc : launch_chunked(p, FROM_SEGMENT, most, batch, st);
 }
 
 // Tokens per segment: a few blocks for every multiprocessor, no segment shorter than 64 tokens
@@ -477,8 +485,8 @@ MSRL_API long long msrl_wkv_scratch(int H, int dim, int tokens, int batch, int m
 
 MSRL_API int msrl_wkv_prefill(const void* r, const void* k, const void* v, const void* g, const float* w, const float* u,
                               const float* norm, float* state, const int* cu, const int* start, const long long* slots, int H,
-                              int dim, float eps, int tokens, int batch, int max_q, int segment, float* scratch, void* y,
-                              int is_f32, cudaStream_t st) {
+                              int dim, float eps, int tokens, int batch, int max_q, int segment, int chunked, float* scratch,
+                              void* y, int is_f32, cudaStream_t st) {
   if (batch == 0 || tokens == 0) return 0;
   if (dim > 256 || batch > 65535 || H > 65535) return (int)cudaErrorNotSupported;
   const int L = segment > 0 ? segment : wkv::segment_length(H, tokens, max_q);
@@ -489,6 +497,8 @@ MSRL_API int msrl_wkv_prefill(const void* r, const void* k, const void* v, const
                    L, scratch, scratch + segments * H * dim * dim, nullptr};
     if (dim > 128) p.o = p.seg_w + segments * H * dim;
     const int most = (max_q + L - 1) / L;
+    if constexpr (sizeof(T) == 2)
+      if (chunked && dim % 8 == 0 && dim <= 128) return wkv::launch_chunks(p, most, batch, st);
     const int rc = dim % 4 == 0 ? wkv::launch_by_dim<T, 4>(p, most, batch, st) : wkv::launch_by_dim<T, 1>(p, most, batch, st);
     if (rc != 0 || dim <= 128) return rc;
     const long long rows = (long long)tokens * H;
@@ -498,8 +508,8 @@ MSRL_API int msrl_wkv_prefill(const void* r, const void* k, const void* v, const
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});
 }
 
-// One token per sequence; a [batch, rank]: the bottleneck's rows
-MSRL_API int msrl_wkv_decode(const void* r, const void* k, const void* v, const void* g, const float* a, const void* w2,
+// One token per sequence; w: decays [batch, H * dim], or null: from the bottleneck's rows a [batch, rank]
+MSRL_API int msrl_wkv_decode(const void* r, const void* k, const void* v, const void* g, const float* w, const float* a, const void* w2,
                              const float* w0, const float* u, const float* norm, float* state, const int* positions,
                              const long long* slots, int H, int dim, int rank, float eps, int batch, void* y, int is_f32,
                              cudaStream_t st) {
@@ -507,13 +517,15 @@ MSRL_API int msrl_wkv_decode(const void* r, const void* k, const void* v, const 
   if (dim > 256 || rank > 512 || batch > 65535) return (int)cudaErrorNotSupported;
   auto run = [&](auto tag) {
     using T = decltype(tag);
-    const wkv::Args<T> p{(const T*)r, (const T*)k, (const T*)v, (const T*)g, nullptr, u, norm, state, nullptr, positions, slots,
+    const wkv::Args<T> p{(const T*)r, (const T*)k, (const T*)v, (const T*)g, w, u, norm, state, nullptr, positions, slots,
                          (T*)y, H, dim, eps, 1, nullptr, nullptr, nullptr};
     const int units = dim % 4 == 0 ? dim / 4 : dim, lanes = 256 / units;
+    int per = 1;                         // lanes of a channel's decay
+    while (per < 16 && per * 2 * dim <= 256) per *= 2;
     const size_t smem = ((size_t)(lanes + 3) * dim + rank) * sizeof(float);
     const dim3 grid((unsigned)H, (unsigned)batch);
-    if (dim % 4 == 0) wkv::decode_kernel<T, 4><<<grid, 256, smem, st>>>(p, a, (const T*)w2, w0, rank, lanes);
-    else wkv::decode_kernel<T, 1><<<grid, 256, smem, st>>>(p, a, (const T*)w2, w0, rank, lanes);
+    if (dim % 4 == 0) wkv::decode_kernel<T, 4><<<grid, 256, smem, st>>>(p, a, (const T*)w2, w0, rank, lanes, per);
+    else wkv::decode_kernel<T, 1><<<grid, 256, smem, st>>>(p, a, (const T*)w2, w0, rank, lanes, per);
     return (int)cudaGetLastError();
   };
   return is_f32 ? run(float{}) : run(__nv_bfloat16{});

@@ -167,7 +167,7 @@ def _post(resid, post, after, dtype, entry=None, delta=None, rows=None, pos=None
     return y
 
 
-FUSED_SIDE_TOKENS = 256        # up to here one kernel does a token input; more tokens make its products matrix products
+FUSED_SIDE_TOKENS = 64         # up to here the gate's product and activation are one kernel, beyond a matrix product
 
 
 def token_side_(resid: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, side: TokenSide, post: PostNorm,
@@ -178,16 +178,13 @@ def token_side_(resid: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, side: T
     if _lib.use_kernels(resid, x, ids, side.gate, side.table):
         L, pad = _lib.load(), side.gate.shape[0]
         row = (ptr(side.table), ptr(ids), c_ll(side.table.shape[1]), c_int(side.col))
-        if t <= (FUSED_SIDE_TOKENS if fused_tokens is None else fused_tokens) and pad == side.dim and width <= 16384:
-            _plain(after)
-            again, step = entry or (None, None)
-            y = guard.empty(t, width, device=resid.device, dtype=x.dtype)
-            check(L.msrl_side_add(ptr(side.gate), ptr(side.proj), *row, c_int(side.dim), ptr(resid), ptr(post.weight),
-                                  c_float(post.eps), ptr(after.weight if after else None), c_float(after.eps if after else 0.0),
-                                  ptr(again), ptr(step), ptr(y), c_ll(t), c_int(width), _is_f32(x), stream()), "side_add")
-            return y
-        g = linear_fwd(x, side.gate)
-        check(L.msrl_side_gate(ptr(g), c_ll(pad), *row, c_int(side.dim), c_ll(t), _is_f32(x), stream()), "side_gate")
+        if t <= (FUSED_SIDE_TOKENS if fused_tokens is None else fused_tokens):
+            g = guard.empty(t, pad, device=x.device, dtype=x.dtype)
+            check(L.msrl_side_gate_product(ptr(x), ptr(side.gate), ptr(g), c_ll(pad), *row, c_int(side.dim), c_ll(t), c_int(width),
+                                           _is_f32(x), stream()), "side_gate_product")
+        else:
+            g = linear_fwd(x, side.gate)
+            check(L.msrl_side_gate(ptr(g), c_ll(pad), *row, c_int(side.dim), c_ll(t), _is_f32(x), stream()), "side_gate")
         return post_add_(resid, linear_fwd(g, side.proj), post, after, entry)
     g = F.gelu(linear_fwd(x, side.gate)[:, :side.dim].float(), approximate="tanh")
     g = (g * side.table[ids, side.col:side.col + side.dim].float()).to(x.dtype)

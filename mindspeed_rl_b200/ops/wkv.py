@@ -6,7 +6,7 @@ sequence's first token); the last token's h is carried in ``last [slots, W]`` fp
     w = exp(-exp(tanh(a) w2^T + w0))
     o = S^T r + (sum_k r u k) v,   S <- diag(w) S + k v^T,   y = o / rms(o) * norm * silu(gate)
 
-``state [slots, H, dim, dim]`` fp32; a sequence's first token ignores what its slots hold.  CUDA path: ``csrc/wkv.cu``; CPU
+``state [slots, H, dim, dim]`` fp32; a sequence's first token ignores what its slots hold.  CUDA path: ``csrc/wkv.cu``, ``csrc/wkv_chunk.cu``; CPU
 tensors run the PyTorch formulation.
 """
 from __future__ import annotations
@@ -24,6 +24,7 @@ from .elementwise import _workspace
 from .residual import _is_f32
 
 MIXES = 5
+DECAY_IN_DECODE = 8            # sequences up to which a decode step computes its decays inside the recurrence
 
 
 @dataclass
@@ -106,9 +107,10 @@ def _reference(r, k, v, g, a, w: WKVWeights, state, bounds, starts, slots, eps):
 
 def wkv_prefill(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, a: torch.Tensor, w: WKVWeights,
                 state: torch.Tensor, cu: torch.Tensor, max_q: int, start_pos: torch.Tensor, slots: torch.Tensor, eps: float,
-                segment: int = 0) -> torch.Tensor:
+                segment: int = 0, chunked: bool = True) -> torch.Tensor:
     """Packed prompt portions, rows ``[T, heads * dim]`` -> ``[T, heads * dim]``.  ``segment``: tokens of the pieces that
-    sequences are cut into (0: what fills the machine)."""
+    sequences are cut into (0: what fills the machine).  bf16 rows of the sizes that the tensor-core kernel serves go through
+    it (``chunked=False`` keeps to the token-by-token kernel)."""
     t, batch = r.shape[0], cu.numel() - 1
     if _lib.use_kernels(r, k, v, g, a, state, cu):
         L, decay = _lib.load(), wkv_decay(a, w)
@@ -117,7 +119,7 @@ def wkv_prefill(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tens
         y = guard.empty(t, w.heads * w.dim, device=r.device, dtype=r.dtype)
         check(L.msrl_wkv_prefill(*(ptr(x.contiguous()) for x in (r, k, v, g)), ptr(decay), ptr(w.u), ptr(w.norm), ptr(state), ptr(cu),
                                  ptr(start_pos), ptr(slots), c_int(w.heads), c_int(w.dim), c_float(eps), c_int(t), c_int(batch),
-                                 c_int(max_q), c_int(segment), ptr(_workspace("wkv", int(n), r.device)), ptr(y), _is_f32(r), stream()),
+                                 c_int(max_q), c_int(segment), c_int(chunked), ptr(_workspace("wkv", int(n), r.device)), ptr(y), _is_f32(r), stream()),
               "wkv_prefill")
         return y
     return _reference(r, k, v, g, a, w, state, cu.tolist(), start_pos.tolist(), slots.tolist(), eps)
@@ -129,8 +131,9 @@ def wkv_decode(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tenso
     b = r.shape[0]
     if _lib.use_kernels(r, k, v, g, a, state, positions):
         y = guard.empty(b, w.heads * w.dim, device=r.device, dtype=r.dtype)
-        check(_lib.load().msrl_wkv_decode(*(ptr(x.contiguous()) for x in (r, k, v, g)), ptr(a.contiguous()), ptr(w.w2), ptr(w.w0),
-                                          ptr(w.u), ptr(w.norm), ptr(state), ptr(positions), ptr(slots), c_int(w.heads),
+        decay = wkv_decay(a, w) if b > DECAY_IN_DECODE else None
+        check(_lib.load().msrl_wkv_decode(*(ptr(x.contiguous()) for x in (r, k, v, g)), ptr(decay), ptr(a.contiguous()), ptr(w.w2),
+                                          ptr(w.w0), ptr(w.u), ptr(w.norm), ptr(state), ptr(positions), ptr(slots), c_int(w.heads),
                                           c_int(w.dim), c_int(a.shape[1]), c_float(eps), c_int(b), ptr(y), _is_f32(r), stream()),
               "wkv_decode")
         return y

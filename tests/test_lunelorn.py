@@ -19,6 +19,7 @@ from mindspeed_rl_b200 import ops
 from mindspeed_rl_b200.models import registry
 from mindspeed_rl_b200.models.hybrid_config import HybridConfig
 from mindspeed_rl_b200.ops import moe as K
+from mindspeed_rl_b200.ops import wkv as W
 from mindspeed_rl_b200.ops.matrix_memory import constant_decay
 from mindspeed_rl_b200.rollout.engine import LLMEngine
 from mindspeed_rl_b200.rollout.hybrid_weights import build_hybrid_weights
@@ -115,7 +116,7 @@ def test_token_side(device, width, dim):
         side = ops.TokenSide(torch.nn.functional.pad(gate, (0, 0, 0, pad - dim)).to(device),
                              torch.nn.functional.pad(proj, (0, pad - dim)).contiguous().to(device), table.to(device), li * dim, dim)
         post, after = ops.PostNorm(norm.to(device), 1e-3), ops.Norm(nxt.to(device), 1e-2)
-        for fused in (None, 0):            # one kernel, and products
+        for fused in (None, 0):            # the gate's product in its kernel, and as a matrix product
             for entry in (None, ops.PassEntry(x.to(device) * 3, nxt.to(device))):
                 resid = x.to(device).clone()
                 y = ops.token_side_(resid, x.to(device, dtype), ids.to(device), side, post, after, entry, fused_tokens=fused)
@@ -405,19 +406,25 @@ def _to(w, device):
 
 
 @pytest.mark.parametrize("device", DEVICES)
-@pytest.mark.parametrize("h,d,rank", [(3, 12, 5), (2, 10, 1), (2, 32, 16), (3, 64, 20), (1, 100, 8), (2, 128, 64), (1, 200, 3)])
-@pytest.mark.parametrize("segment", [0, 16, 48])
-def test_wkv_portions_and_decode(device, h, d, rank, segment):
-    if device == "cpu" and segment:
+@pytest.mark.parametrize("h,d,rank", [(3, 12, 5), (2, 10, 1), (3, 16, 4), (2, 32, 16), (2, 40, 6), (3, 64, 20), (1, 100, 8), (1, 104, 12),
+                                       (2, 128, 64), (1, 200, 3)])
+@pytest.mark.parametrize("segment,chunked", [(0, True), (0, False), (16, True), (48, True), (48, False)])
+def test_wkv_portions_and_decode(device, h, d, rank, segment, chunked, monkeypatch):
+    """Sequences from end to end and cut into segments, on the tensor cores and token by token; decays computed ahead of a
+    decode step and inside it."""
+    if device == "cpu" and (segment or not chunked):
         pytest.skip("one CPU formulation")
     n, eps = 200, 1e-4
+    monkeypatch.setattr(W, "DECAY_IN_DECODE", 0 if segment else 8)
     for dtype in dtypes(device):
+        if dtype == torch.float32 and not chunked:
+            continue
         rows, a, w = _wkv_case(2 * n, h, d, rank, dtype)
         want = torch.cat([_wkv_want([x[i:i + n] for x in rows], a[i:i + n], w, eps) for i in (0, n)])
         wd, state = _to(w, device), _filled(device, 4, h, d, d)
         pick = lambda r: [x[r].to(device) for x in (*rows, a)]
         got = _walk(n, device,
-                    lambda r, cu, m, st, own, _: ops.wkv_prefill(*pick(r), wd, state, cu, m, st, own, eps, segment=segment),
+                    lambda r, cu, m, st, own, _: ops.wkv_prefill(*pick(r), wd, state, cu, m, st, own, eps, segment=segment, chunked=chunked),
                     lambda r, pos, own: ops.wkv_decode(*pick(r), wd, state, pos, own, eps))
         close(got, want, tol=5e-5 if dtype == torch.float32 else 2e-2)
         if dtype == torch.bfloat16:
