@@ -11,7 +11,8 @@
 namespace msrl {
 namespace gru {
 
-constexpr int SEG = 64, AHEAD = 8;       // tokens of a segment; tokens whose rows are loaded together
+constexpr int SEG = 64;                  // tokens of a segment
+constexpr int AHEAD = 8, SEGS_AHEAD = 32;     // tokens, segments whose rows are loaded together
 
 template <typename T>
 struct Args {
@@ -49,6 +50,11 @@ __device__ __forceinline__ void step_of(float zp, float xp, float zb, float xb, 
   add = z * (u >= 0.f ? u + 0.5f : sigmoid_t<T>(u));
 }
 
+// V entries as they are stored
+template <typename T, int V>
+struct alignas(V * sizeof(T)) Packed {
+  T v[V];
+};
 // OUT: outputs from the state before the segment; otherwise the segment's factor and sum.  WHOLE: one segment holds the
 // sequence, its state comes from the slot and goes back.  grid (channels / (128 V), segments, B)
 template <typename T, int V, bool OUT, bool WHOLE>
@@ -72,32 +78,44 @@ __global__ void __launch_bounds__(128) scan_kernel(const Args<T> p) {
     if (!WHOLE) ldv<V>(p.sum + at, S);
     else if (p.start[b] > 0 && slot >= 0) ldv<V>(p.state + slot * p.width + c, S);
   }
-  for (int i0 = 0; i0 < len; i0 += AHEAD) {
-    float z[AHEAD][4], x[AHEAD][4], g[AHEAD][4];
+  using R = Packed<T, V>;
+  struct Rows {
+    R z[AHEAD], x[AHEAD], g[AHEAD];
+  } now, next;
+  const T *zp = p.z + (long long)t0 * p.ld + c, *xp = p.x + (long long)t0 * p.ld + c, *gp = p.g + (long long)t0 * p.ld + c;
+  auto fetch = [&](Rows& rows, int i0) {
 #pragma unroll
     for (int i = 0; i < AHEAD; ++i) {
       if (i0 + i < len) {
-        const long long row = (long long)(t0 + i0 + i) * p.ld + c;
-        ldv<V>(p.z + row, z[i]);
-        ldv<V>(p.x + row, x[i]);
-        if (OUT) ldv<V>(p.g + row, g[i]);
+        const long long at = (i0 + i) * p.ld;
+        rows.z[i] = *reinterpret_cast<const R*>(zp + at);
+        rows.x[i] = *reinterpret_cast<const R*>(xp + at);
+        if (OUT) rows.g[i] = *reinterpret_cast<const R*>(gp + at);
       }
     }
+  };
+  fetch(now, 0);
+  for (int i0 = 0; i0 < len; i0 += AHEAD) {
+    fetch(next, i0 + AHEAD);
 #pragma unroll
     for (int i = 0; i < AHEAD; ++i) {
       if (i0 + i < len) {
-        float y[4];
+        float z[4], x[4], g[4], y[4];
+        ldv<V>(reinterpret_cast<const T*>(&now.z[i]), z);
+        ldv<V>(reinterpret_cast<const T*>(&now.x[i]), x);
+        if (OUT) ldv<V>(reinterpret_cast<const T*>(&now.g[i]), g);
 #pragma unroll
         for (int e = 0; e < V; ++e) {
           float keep, add;
-          step_of<T>(z[i][e], x[i][e], zb[e], xb[e], keep, add);
+          step_of<T>(z[e], x[e], zb[e], xb[e], keep, add);
           S[e] = keep * S[e] + add;
-          if (OUT) y[e] = S[e] * g[i][e] * sigmoid_t<T>(g[i][e]) * p.scale;
+          if (OUT) y[e] = S[e] * g[e] * sigmoid_t<T>(g[e]) * p.scale;
           else A[e] *= keep;
         }
         if (OUT) stv<V>(p.y + (long long)(t0 + i0 + i) * p.y_ld + c, y);
       }
     }
+    now = next;
   }
   if (!OUT) {
     stv<V>(p.keep + at, A);
@@ -115,17 +133,17 @@ __global__ void __launch_bounds__(128) carry_kernel(const Args<T> p) {
   if (len <= 0 || c >= p.width) return;
   const long long slot = p.slots[b], at = seg_id(t0, b, 0) * p.width + c;
   float s = p.start[b] > 0 && slot >= 0 ? p.state[slot * p.width + c] : 0.f;
-  for (int j0 = 0; j0 < n; j0 += AHEAD) {
-    float keep[AHEAD], sum[AHEAD];
+  for (int j0 = 0; j0 < n; j0 += SEGS_AHEAD) {
+    float keep[SEGS_AHEAD], sum[SEGS_AHEAD];
 #pragma unroll
-    for (int i = 0; i < AHEAD; ++i) {
+    for (int i = 0; i < SEGS_AHEAD; ++i) {
       if (j0 + i < n) {
         keep[i] = p.keep[at + (long long)(j0 + i) * p.width];
         sum[i] = p.sum[at + (long long)(j0 + i) * p.width];
       }
     }
 #pragma unroll
-    for (int i = 0; i < AHEAD; ++i) {
+    for (int i = 0; i < SEGS_AHEAD; ++i) {
       if (j0 + i < n) {
         p.sum[at + (long long)(j0 + i) * p.width] = s;
         s = keep[i] * s + sum[i];

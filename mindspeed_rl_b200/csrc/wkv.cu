@@ -329,13 +329,20 @@ decode_kernel(const Args<T> p, const float* a, const T* w2, const float* w0, int
       if (rl < lanes && !fresh && r < dim) ldv<V>(S + (long long)r * dim, s[i]);
     }
   };
-  fetch(rl);                             // on its way while the decays are computed
-  float bonus = 0.f;
-  for (int d = threadIdx.x; d < dim; d += 256) {
-    sr[d] = ldf(p.r + at + d);
-    sk[d] = ldf(p.k + at + d);
-    if (p.w != nullptr) sw[d] = p.w[at + d];
-    bonus += sr[d] * p.u[h * dim + d] * sk[d];
+  fetch(rl);                             // everything that comes from memory is on its way before the first wait
+  const int own = threadIdx.x;           // the thread's column of the output and key channel (dim <= 256)
+  const bool mine = own < dim;
+  float v[4], bonus = 0.f, value = 0.f, z = 0.f, weight = 0.f;
+  if (rl < lanes) ldv<V>(p.v + at + cu * V, v);
+  if (mine) {
+    const float r = ldf(p.r + at + own), k = ldf(p.k + at + own), u = p.u[h * dim + own];
+    if (p.w != nullptr) sw[own] = p.w[at + own];
+    value = ldf(p.v + at + own);
+    z = ldf(p.g + at + own);
+    weight = p.norm[h * dim + own];
+    sr[own] = r;
+    sk[own] = k;
+    bonus = r * u * k;
   }
   if (p.w == nullptr) {
     for (int j = threadIdx.x; j < rank; j += 256) sa[j] = tanhf(a[(long long)b * rank + j]);
@@ -362,9 +369,8 @@ decode_kernel(const Args<T> p, const float* a, const T* w2, const float* w0, int
     }
   }
   bonus = block_sum(bonus, red);         // (synchronises sr, sk, sw)
-  float v[4], o[4] = {0.f, 0.f, 0.f, 0.f};
+  float o[4] = {0.f, 0.f, 0.f, 0.f};
   if (rl < lanes) {
-    ldv<V>(p.v + at + cu * V, v);
     for (int r0 = rl; r0 < dim; r0 += lanes * DB) {
       if (r0 != rl) fetch(r0);
 #pragma unroll
@@ -381,22 +387,16 @@ decode_kernel(const Args<T> p, const float* a, const T* w2, const float* w0, int
         }
       }
     }
-#pragma unroll
-    for (int x = 0; x < V; ++x) part[rl * dim + cu * V + x] = o[x];
+    stv<V>(part + rl * dim + cu * V, o);
   }
   __syncthreads();
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < dim; c += 256) {
-    float x = bonus * ldf(p.v + at + c);
-    for (int l = 0; l < lanes; ++l) x += part[l * dim + c];
-    part[c] = x;                         // the only reader of column c
-    ss += x * x;
+  float x = 0.f;
+  if (mine) {
+    x = bonus * value;
+    for (int l = 0; l < lanes; ++l) x += part[l * dim + own];
   }
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)dim + p.eps);
-  for (int c = threadIdx.x; c < dim; c += 256) {
-    const float z = ldf(p.g + at + c);
-    stf(p.y + at + c, part[c] * inv * p.norm[h * dim + c] * z * sigmoid_t<T>(z));
-  }
+  const float inv = 1.f / sqrtf(block_sum(x * x, red) / (float)dim + p.eps);
+  if (mine) stf(p.y + at + own, x * inv * weight * z * sigmoid_t<T>(z));
 }
 
 template <typename T>
@@ -466,6 +466,8 @@ MSRL_API int msrl_wkv_decay(const float* a, const void* w2, const float* w0, flo
                             int is_f32, cudaStream_t st) {
   if (tokens == 0) return 0;
   if (rank > 512) return (int)cudaErrorNotSupported;
+  if (!is_f32 && channels % 2 == 0 && rank <= 128)
+    return wkv::launch_decay(a, (const __nv_bfloat16*)w2, w0, w, tokens, rank, channels, st);
   const dim3 grid((unsigned)((channels + 255) / 256), (unsigned)((tokens + wkv::DT - 1) / wkv::DT));
   const size_t smem = (size_t)rank * wkv::DT * sizeof(float);
   auto run = [&](auto tag) {

@@ -31,6 +31,9 @@ enum { WHOLE = 0, ADDED = 1, FROM_SEGMENT = 2 };
 
 // wkv_chunk.cu: the same for bf16 rows with dim a multiple of 8 up to 128, sixteen tokens at a time on the tensor cores
 int launch_chunked(const Args<__nv_bfloat16>& p, int mode, int segments, int batch, cudaStream_t st);
+// decays of bf16 weights on the tensor cores: an even number of channels, rank up to 128
+int launch_decay(const float* a, const __nv_bfloat16* w2, const float* w0, float* w, int tokens, int rank, int channels,
+                 cudaStream_t st);
 
 }  // namespace wkv
 }  // namespace msrl

@@ -333,6 +333,98 @@ __global__ void __launch_bounds__(2 * DP, DP == 128 ? 2 : DP == 64 ? 4 : 8) chun
   if (MODE == ADDED && tid < dim) p.seg_w[(seg_id(s0, b, j, p.L) * p.H + h) * dim + tid] = product;
 }
 
+// ---- decays: w = exp(-exp(tanh(a) w2^T + w0)), tanh(a) as three bf16 terms ------------------------------------------
+constexpr int DM = 64, DN = 256, DTILES = 4;     // tokens of a tile, channels and tiles of a block
+
+__host__ __device__ inline int rank_pitch(int rank) { return (rank + 15) / 16 * 16 + 8; }
+__host__ __device__ inline int decay_smem(int rank) { return (TERMS * DM + DN) * rank_pitch(rank) * 2; }
+
+// grid (channels / DN, tokens / (DM DTILES)); eight warps of 32 channels
+__global__ void __launch_bounds__(256, 2)
+decay_mma_kernel(const float* a, const bf16* w2, const float* w0, float* w, int tokens, int rank, int channels) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int rp = rank_pitch(rank), k16 = rp - 8;
+  bf16 *sA = reinterpret_cast<bf16*>(raw), *sB = sA + TERMS * DM * rp;
+  const int c0 = blockIdx.x * DN, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (rank % 16 == 0) {
+    for (int i = threadIdx.x; i < DN * rank / 8; i += 256) {
+      const int c = i / (rank / 8), k = i % (rank / 8) * 8;
+      const bool ok = c0 + c < channels;
+      cp_async16(sB + c * rp + k, w2 + (ok ? (long long)(c0 + c) * rank + k : 0), ok);
+    }
+    cp_async_commit();
+  } else {
+    for (int i = threadIdx.x; i < DN * k16; i += 256) {
+      const int c = i / k16, k = i % k16;
+      sB[c * rp + k] = c0 + c < channels && k < rank ? w2[(long long)(c0 + c) * rank + k] : __float2bfloat16_rn(0.f);
+    }
+  }
+  const uint32_t a_at = smem_u32(sA), b_at = smem_u32(sB);
+  const int quad = lane >> 3, in8 = lane & 7, n0 = warp * 32, gid = lane >> 2, tig = lane & 3;
+  float2 bias[4];
+#pragma unroll
+  for (int n = 0; n < 4; ++n) {
+    const int c = c0 + n0 + n * 8 + 2 * tig;                       // channels are even
+    bias[n] = c < channels ? *reinterpret_cast<const float2*>(w0 + c) : make_float2(0.f, 0.f);
+  }
+  for (int tile = 0; tile < DTILES; ++tile) {
+    const int t0 = (blockIdx.y * DTILES + tile) * DM;
+    if (t0 >= tokens) break;
+    if (tile > 0) __syncthreads();       // the products of the tile before are done
+    for (int i = threadIdx.x; i < DM * k16 / 2; i += 256) {
+      const int s = i / (k16 / 2), k = i % (k16 / 2) * 2;
+      float x[2] = {0.f, 0.f};
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        if (t0 + s < tokens && k + e < rank) x[e] = tanhf(a[(long long)(t0 + s) * rank + k + e]);
+      uint32_t t[TERMS];
+      split2(x[0], x[1], t);
+#pragma unroll
+      for (int e = 0; e < TERMS; ++e) *reinterpret_cast<uint32_t*>(sA + (e * DM + s) * rp + k) = t[e];
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    float acc[4][4][4] = {};             // [sixteen tokens][eight channels]
+    for (int k = 0; k < k16; k += 16) {
+      uint32_t bt[2][4];
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+        ldmatrix_x4(bt[n], b_at + ((n0 + n * 16 + (quad >> 1) * 8 + in8) * rp + k + (quad & 1) * 8) * 2);
+#pragma unroll
+      for (int e = 0; e < TERMS; ++e)
+#pragma unroll
+        for (int m = 0; m < 4; ++m) {
+          uint32_t at[4];
+          ldmatrix_x4(at, a_at + ((e * DM + m * 16 + (quad & 1) * 8 + in8) * rp + k + (quad >> 1) * 8) * 2);
+#pragma unroll
+          for (int n = 0; n < 4; ++n) mma_16816(acc[m][n], at, bt[n >> 1][(n & 1) * 2], bt[n >> 1][(n & 1) * 2 + 1]);
+        }
+    }
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      const int c = c0 + n0 + n * 8 + 2 * tig;
+#pragma unroll
+      for (int m = 0; m < 4; ++m)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int t = t0 + m * 16 + gid + e * 8;
+          if (t < tokens && c < channels)
+            *reinterpret_cast<float2*>(w + (long long)t * channels + c) =
+                make_float2(expf(-__expf(acc[m][n][2 * e] + bias[n].x)), expf(-__expf(acc[m][n][2 * e + 1] + bias[n].y)));
+        }
+    }
+  }
+}
+
+int launch_decay(const float* a, const bf16* w2, const float* w0, float* w, int tokens, int rank, int channels, cudaStream_t st) {
+  const int smem = decay_smem(rank);
+  const cudaError_t rc = cudaFuncSetAttribute(decay_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+  if (rc != cudaSuccess) return (int)rc;
+  const dim3 grid((unsigned)((channels + DN - 1) / DN), (unsigned)((tokens + DM * DTILES - 1) / (DM * DTILES)));
+  decay_mma_kernel<<<grid, 256, smem, st>>>(a, w2, w0, w, tokens, rank, channels);
+  return (int)cudaGetLastError();
+}
+
 template <int DP>
 static int launch_dim(const Args<bf16>& p, int mode, int segments, int batch, cudaStream_t st) {
   auto go = [&](auto* kernel) {
