@@ -334,14 +334,14 @@ __global__ void __launch_bounds__(2 * DP, DP == 128 ? 2 : DP == 64 ? 4 : 8) chun
 }
 
 // ---- decays: w = exp(-exp(tanh(a) w2^T + w0)), tanh(a) as three bf16 terms ------------------------------------------
-constexpr int DM = 64, DN = 256, DTILES = 4;     // tokens of a tile, channels and tiles of a block
+constexpr int DM = 64, DN = 256;         // tokens of a tile, channels of a block
 
 __host__ __device__ inline int rank_pitch(int rank) { return (rank + 15) / 16 * 16 + 8; }
 __host__ __device__ inline int decay_smem(int rank) { return (TERMS * DM + DN) * rank_pitch(rank) * 2; }
 
-// grid (channels / DN, tokens / (DM DTILES)); eight warps of 32 channels
+// grid (channels / DN, tokens / (DM tiles)); eight warps of 32 channels
 __global__ void __launch_bounds__(256, 2)
-decay_mma_kernel(const float* a, const bf16* w2, const float* w0, float* w, int tokens, int rank, int channels) {
+decay_mma_kernel(const float* a, const bf16* w2, const float* w0, float* w, int tokens, int rank, int channels, int tiles) {
   extern __shared__ __align__(16) unsigned char raw[];
   const int rp = rank_pitch(rank), k16 = rp - 8;
   bf16 *sA = reinterpret_cast<bf16*>(raw), *sB = sA + TERMS * DM * rp;
@@ -367,8 +367,8 @@ decay_mma_kernel(const float* a, const bf16* w2, const float* w0, float* w, int 
     const int c = c0 + n0 + n * 8 + 2 * tig;                       // channels are even
     bias[n] = c < channels ? *reinterpret_cast<const float2*>(w0 + c) : make_float2(0.f, 0.f);
   }
-  for (int tile = 0; tile < DTILES; ++tile) {
-    const int t0 = (blockIdx.y * DTILES + tile) * DM;
+  for (int tile = 0; tile < tiles; ++tile) {
+    const int t0 = (blockIdx.y * tiles + tile) * DM;
     if (t0 >= tokens) break;
     if (tile > 0) __syncthreads();       // the products of the tile before are done
     for (int i = threadIdx.x; i < DM * k16 / 2; i += 256) {
@@ -420,8 +420,10 @@ int launch_decay(const float* a, const bf16* w2, const float* w0, float* w, int 
   const int smem = decay_smem(rank);
   const cudaError_t rc = cudaFuncSetAttribute(decay_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (rc != cudaSuccess) return (int)rc;
-  const dim3 grid((unsigned)((channels + DN - 1) / DN), (unsigned)((tokens + DM * DTILES - 1) / (DM * DTILES)));
-  decay_mma_kernel<<<grid, 256, smem, st>>>(a, w2, w0, w, tokens, rank, channels);
+  const int columns = (channels + DN - 1) / DN, rows = (tokens + DM - 1) / DM;
+  const int tiles = columns * rows >= 8 * sm_count() ? 4 : 1;      // of a block: they share the weights
+  decay_mma_kernel<<<dim3((unsigned)columns, (unsigned)((rows + tiles - 1) / tiles)), 256, smem, st>>>(a, w2, w0, w, tokens, rank,
+                                                                                                       channels, tiles);
   return (int)cudaGetLastError();
 }
 
