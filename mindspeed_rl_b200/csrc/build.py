@@ -44,7 +44,8 @@ _STREAM = ("residual_stream", "grouped_gemm_simt", "moe", "moe_gemm_tcgen05", "a
 GROUPS = {
     "pumotar": (*_STREAM, "delta_rule", "latent_attention", "latent_decode_tcgen05"),
     "gapevik": (*_STREAM, "delta_rule", "latent_attention", "latent_decode_tcgen05", "conv_qkv", "decode", "decode_prefix_tcgen05"),
-    "lunelorn": (*_STREAM, "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "wkv", "wkv_chunk", "min_gru", "decode", "decode_prefix_tcgen05"),
+    "lunelorn": (*_STREAM, "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "wkv", "wkv_chunk", "min_gru", "decode",
+                 "decode_prefix_tcgen05"),
     "sunatar": (*_STREAM, "matrix_memory", "matrix_memory_tcgen05", "qkv_prep", "decode", "decode_prefix_tcgen05"),
 }
 

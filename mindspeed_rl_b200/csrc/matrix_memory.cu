@@ -371,8 +371,8 @@ using namespace msrl;
 // floats: scale, cap, floor, eps
 MSRL_API int msrl_memory_decode(const void* proj, long long ld, const float* z, long long z_ld, const int* ints,
                                 const float* floats, const float* bias, const float* decay, const float* norm,
-                                float* memory, float* nrm, float* peak, const int* positions, const long long* slots, void* y, int batch, int is_f32,
-                                cudaStream_t st) {
+                                float* memory, float* nrm, float* peak, const int* positions, const long long* slots,
+                                void* y, int batch, int is_f32, cudaStream_t st) {
   if (batch == 0) return 0;
   const int H = ints[0], dim = ints[1], vdim = ints[2];
   if (dim % 16 != 0 || vdim % 16 != 0 || batch > 65535 || H > 65535) return (int)cudaErrorInvalidValue;
@@ -405,8 +405,8 @@ MSRL_API int msrl_memory_decode(const void* proj, long long ld, const float* z, 
 // o: fp32 scratch [tokens, H * vdim]
 MSRL_API int msrl_memory_prefill(const void* proj, long long ld, const float* z, long long z_ld, const int* ints,
                                  const float* floats, const float* bias, const float* decay, const float* norm,
-                                 float* memory, float* nrm, float* peak, const int* cu, const int* start, const long long* slots, float* o, void* y,
-                                 int tokens, int batch, int is_f32, cudaStream_t st) {
+                                 float* memory, float* nrm, float* peak, const int* cu, const int* start,
+                                 const long long* slots, float* o, void* y, int tokens, int batch, int is_f32, cudaStream_t st) {
   if (batch == 0 || tokens == 0) return 0;
   const int H = ints[0], dim = ints[1], vdim = ints[2];
   if (dim > 512 || dim % 16 != 0 || vdim % 16 != 0 || batch > 65535 || H > 65535) return (int)cudaErrorNotSupported;
@@ -451,8 +451,8 @@ int launch_chunk_out(const Args<__nv_bfloat16>& p, const Chunks& ch, int most, i
 // The same for bf16 rows, in chunks; column starts and ld are multiples of 8.  error: device status word (0 = ok)
 MSRL_API int msrl_memory_prefill_chunked(const void* proj, long long ld, const float* z, long long z_ld, const int* ints,
                                          const float* floats, const float* bias, const float* decay, const float* norm,
-                                         float* memory, float* nrm, float* peak, const int* cu, const int* start, const long long* slots,
-                                         float* scratch, void* y, int tokens, int batch, int max_q, int* error,
+                                         float* memory, float* nrm, float* peak, const int* cu, const int* start,
+                                         const long long* slots, float* scratch, void* y, int tokens, int batch, int max_q, int* error,
                                          cudaStream_t st) {
   if (batch == 0 || tokens == 0) return 0;
   const int H = ints[0], dim = ints[1], vdim = ints[2];

@@ -511,8 +511,8 @@ MSRL_API int msrl_wkv_prefill(const void* r, const void* k, const void* v, const
 }
 
 // One token per sequence; w: decays [batch, H * dim], or null: from the bottleneck's rows a [batch, rank]
-MSRL_API int msrl_wkv_decode(const void* r, const void* k, const void* v, const void* g, const float* w, const float* a, const void* w2,
-                             const float* w0, const float* u, const float* norm, float* state, const int* positions,
+MSRL_API int msrl_wkv_decode(const void* r, const void* k, const void* v, const void* g, const float* w, const float* a,
+                             const void* w2, const float* w0, const float* u, const float* norm, float* state, const int* positions,
                              const long long* slots, int H, int dim, int rank, float eps, int batch, void* y, int is_f32,
                              cudaStream_t st) {
   if (batch == 0) return 0;

@@ -435,7 +435,8 @@ static int launch_dim(const Args<bf16>& p, int mode, int segments, int batch, cu
     kernel<<<dim3((unsigned)segments, (unsigned)p.H, (unsigned)batch), 2 * DP, Smem<DP>::BYTES, st>>>(p);
     return (int)cudaGetLastError();
   };
-  return mode == WHOLE ? go(chunk_kernel<DP, WHOLE>) : mode == ADDED ? go(chunk_kernel<DP, ADDED>) : go(chunk_kernel<DP, FROM_SEGMENT>);
+  if (mode == WHOLE) return go(chunk_kernel<DP, WHOLE>);
+  return mode == ADDED ? go(chunk_kernel<DP, ADDED>) : go(chunk_kernel<DP, FROM_SEGMENT>);
 }
 
 int launch_chunked(const Args<bf16>& p, int mode, int segments, int batch, cudaStream_t st) {

@@ -13,8 +13,8 @@ Per head, with log gates ``i = cap tanh(z_i / cap)`` and ``f = log sigmoid(cap t
 ``MemoryLayout.silu_gate``: the output gate is ``silu(gate)``.
 
 A sequence starts with S, n and m zero.  ``slots`` holds the state of all sequences: ``memory [slots, H, dim, vdim]``,
-``norm [slots, H, dim]`` and ``peak [slots, H]``, all fp32 (with ``decay`` the memory alone); a sequence's first token ignores what its slot holds.  CUDA
-path: ``csrc/matrix_memory.cu``, ``csrc/matrix_memory_tcgen05.cu``; CPU tensors run the PyTorch formulation.
+``norm [slots, H, dim]`` and ``peak [slots, H]``, all fp32 (with ``decay`` the memory alone); a sequence's first token
+ignores what its slot holds.  CUDA path: ``csrc/matrix_memory.cu``, ``csrc/matrix_memory_tcgen05.cu``; CPU tensors run the PyTorch formulation.
 """
 from __future__ import annotations
 
@@ -128,17 +128,22 @@ def _run(proj, z, lay, w, slots, starts, cu, owner, eps):
     return y
 
 
-def memory_prefill(proj: torch.Tensor, z: Optional[torch.Tensor], lay: MemoryLayout, w: MemoryWeights, slots: Dict[str, torch.Tensor],
-                   cu_q: torch.Tensor, max_q: int, start_pos: torch.Tensor, state_slots: torch.Tensor, eps: float,
-                   chunked: bool = True) -> torch.Tensor:
-    """Prompt portions: ``proj [T, ...]``, gate logits ``z [T, 2 * heads]`` fp32 (None with a constant decay) -> ``y [T, heads * vdim]``.  bf16 rows of
-    the sizes that the tensor-core kernels serve run in chunks (``chunked=False`` keeps to the token-by-token kernel)."""
+def _arguments(proj, z, lay: MemoryLayout, w: MemoryWeights, slots, eps: float):
+    """What the kernels of both kinds of steps take first."""
+    return (ptr(proj), c_ll(proj.stride(0)), ptr(z), c_ll(0 if z is None else z.stride(0)), lay.ints(), lay.floats(eps), ptr(w.bias),
+            ptr(w.decay), ptr(w.norm), ptr(slots["memory"]), ptr(slots.get("norm")), ptr(slots.get("peak")))
+
+
+def memory_prefill(proj: torch.Tensor, z: Optional[torch.Tensor], lay: MemoryLayout, w: MemoryWeights,
+                   slots: Dict[str, torch.Tensor], cu_q: torch.Tensor, max_q: int, start_pos: torch.Tensor,
+                   state_slots: torch.Tensor, eps: float, chunked: bool = True) -> torch.Tensor:
+    """Prompt portions: ``proj [T, ...]``, gate logits ``z [T, 2 * heads]`` fp32 (None with a constant decay) ->
+    ``y [T, heads * vdim]``.  bf16 rows of the sizes that the tensor-core kernels serve run in chunks (``chunked=False`` keeps to the token-by-token kernel)."""
     t, batch = proj.shape[0], cu_q.numel() - 1
     if _lib.use_kernels(proj, cu_q, state_slots):
         L = _lib.load()
         y = guard.empty(t, lay.heads * lay.vdim, device=proj.device, dtype=proj.dtype)
-        args = (ptr(proj), c_ll(proj.stride(0)), ptr(z), c_ll(0 if z is None else z.stride(0)), lay.ints(), lay.floats(eps), ptr(w.bias),
-                ptr(w.decay), ptr(w.norm), ptr(slots["memory"]), ptr(slots.get("norm")), ptr(slots.get("peak")), ptr(cu_q), ptr(start_pos), ptr(state_slots))
+        args = (*_arguments(proj, z, lay, w, slots, eps), ptr(cu_q), ptr(start_pos), ptr(state_slots))
         if chunked and proj.dtype == torch.bfloat16 and L.msrl_memory_chunked_serves(lay.ints()):
             size = L.msrl_memory_chunk_scratch
             size.restype = ctypes.c_longlong
@@ -152,15 +157,13 @@ def memory_prefill(proj: torch.Tensor, z: Optional[torch.Tensor], lay: MemoryLay
     return _run(proj, z, lay, w, slots, start_pos.tolist(), cu_q.tolist(), state_slots.tolist(), eps)
 
 
-def memory_decode(proj: torch.Tensor, z: Optional[torch.Tensor], lay: MemoryLayout, w: MemoryWeights, slots: Dict[str, torch.Tensor],
-                  positions: torch.Tensor, state_slots: torch.Tensor, eps: float) -> torch.Tensor:
+def memory_decode(proj: torch.Tensor, z: Optional[torch.Tensor], lay: MemoryLayout, w: MemoryWeights,
+                  slots: Dict[str, torch.Tensor], positions: torch.Tensor, state_slots: torch.Tensor, eps: float) -> torch.Tensor:
     """One token per sequence: state read and written once (``state_slots[b] < 0``: neither)."""
     b = proj.shape[0]
     if _lib.use_kernels(proj, positions, state_slots):
         y = guard.empty(b, lay.heads * lay.vdim, device=proj.device, dtype=proj.dtype)
-        check(_lib.load().msrl_memory_decode(
-            ptr(proj), c_ll(proj.stride(0)), ptr(z), c_ll(0 if z is None else z.stride(0)), lay.ints(), lay.floats(eps), ptr(w.bias),
-            ptr(w.decay), ptr(w.norm), ptr(slots["memory"]), ptr(slots.get("norm")), ptr(slots.get("peak")), ptr(positions), ptr(state_slots), ptr(y), c_int(b),
-            _is_f32(proj), stream()), "memory_decode")
+        check(_lib.load().msrl_memory_decode(*_arguments(proj, z, lay, w, slots, eps), ptr(positions), ptr(state_slots), ptr(y),
+                                             c_int(b), _is_f32(proj), stream()), "memory_decode")
         return y
     return _run(proj, z, lay, w, slots, positions.tolist(), range(b + 1), state_slots.tolist(), eps)

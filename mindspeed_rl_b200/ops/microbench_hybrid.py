@@ -8,12 +8,13 @@ from __future__ import annotations
 
 import torch
 
-from . import (ConvHeads, ConvNormWeights, DeltaLayout, DeltaWeights, GRULayout, GroupedHeads, LatentLayout, MemoryLayout,
-               MemoryWeights, Norm, PassEntry, PostNorm, ScoreForm, TokenSide, WKVWeights, add_norm_, angle_table, conv_qkv_decode, conv_qkv_prefill, delta_decode, delta_prefill, embed_norm,
-               glu_fwd, latent_decode_attention, latent_prefill_attention, latent_prep, latent_rotate_queries, latent_spread_,
-               memory_decode, memory_prefill, min_gru_decode, min_gru_prefill, moe_combine_norm_, moe_post_add_, post_add_,
-               post_embed, qkv_prep_, rope_table, rows_gather, soft_cap_, token_side_, turn_back, turned_prep_,
-               window_decode_attention, window_prefill_attention, wkv_decode, wkv_mix_decode, wkv_mix_prefill, wkv_prefill)
+from . import (ConvHeads, ConvNormWeights, DeltaLayout, DeltaWeights, GroupedHeads, GRULayout, LatentLayout, MemoryLayout,
+               MemoryWeights, Norm, PassEntry, PostNorm, ScoreForm, TokenSide, WKVWeights, add_norm_, angle_table,
+               conv_qkv_decode, conv_qkv_prefill, delta_decode, delta_prefill, embed_norm, glu_fwd, latent_decode_attention,
+               latent_prefill_attention, latent_prep, latent_rotate_queries, latent_spread_, memory_decode, memory_prefill,
+               min_gru_decode, min_gru_prefill, moe_combine_norm_, moe_post_add_, post_add_, post_embed, qkv_prep_, rope_table,
+               rows_gather, soft_cap_, token_side_, turn_back, turned_prep_, window_decode_attention, window_prefill_attention,
+               wkv_decode, wkv_mix_decode, wkv_mix_prefill, wkv_prefill)
 from . import moe as K
 from .matrix_memory import constant_decay
 from .microbench import report, timeit

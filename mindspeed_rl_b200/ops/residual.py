@@ -4,8 +4,8 @@ follows fused in, and the gated activations.
 The residual ``[T, W]`` is fp32 and updated in place; norm weights are fp32, the activations bf16 or fp32.
 ``norm(x) = x / sqrt(mean(x^2) + eps) * (offset + w)`` in fp32; ``centered`` norms subtract the row's mean from x
 first (a layer norm without bias).  ``post_*`` functions norm what a sublayer gives before it is added and hand on the
-residual itself, rounded to the activation type, or a norm of it; ``entry``: what a pass of a loop adds in between.  CUDA path: ``csrc/residual_stream.cu``; CPU
-tensors run the PyTorch formulation.
+residual itself, rounded to the activation type, or a norm of it; ``entry``: what a pass of a loop adds in between.  CUDA
+path: ``csrc/residual_stream.cu``; CPU tensors run the PyTorch formulation.
 """
 from __future__ import annotations
 
