@@ -1,4 +1,4 @@
-// Gated recurrence whose gate and candidate read the current token only, element by element in fp32:
+// Element-wise recurrence whose gate and candidate do not depend on the state, in fp32:
 //
 //   z = sigmoid(z_proj + z_bias),  u = x_proj + x_bias,  c = u + 1/2 for u >= 0, else sigmoid(u)
 //   S <- (1 - z) S + z c;          y = S * silu(g_proj) * scale

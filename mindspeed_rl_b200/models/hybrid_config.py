@@ -283,8 +283,7 @@ class MatrixMemorySpec:
 
 @dataclass(frozen=True)
 class RetentionSpec:
-    """Linear attention over a state that decays by a constant per head; neither soft-max nor denominator.  Heads are
-    stored in multiples of 16."""
+    """Linear attention over a matrix state whose heads forget at constant rates.  Heads are stored in multiples of 16."""
     heads: int
     dim: int
     vdim: int
@@ -342,7 +341,7 @@ class TurnedAttentionSpec:
 
 @dataclass(frozen=True)
 class MinGRUSpec:
-    """A gated recurrence, element by element, whose gate and candidate read the current token only."""
+    """An element-wise recurrence; its gate and its candidate are functions of the token, not of the state."""
     width: int
 
     def slot_state(self, dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:

@@ -1,6 +1,6 @@
 """Minimal gated recurrence over state slots: prompt portions and decode steps.
 
-Element by element, gate and candidate reading the current token only::
+Element by element; gate and candidate do not depend on the state::
 
     z = sigmoid(z_proj + z_bias),  u = x_proj + x_bias,  c = u + 1/2 where u >= 0, else sigmoid(u)
     S <- (1 - z) S + z c,          y = S * silu(g_proj) * scale

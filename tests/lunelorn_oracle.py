@@ -38,7 +38,7 @@ def turn(x: torch.Tensor, dims: int, base: float, sign: float = 1.0) -> torch.Te
 
 
 def attend(q, k, v, scale: float) -> torch.Tensor:
-    """``q [T, H, d]`` over ``k [T, G, d]``, ``v [T, G, dv]``: token i sees every j <= i."""
+    """Causal soft-max of ``q [T, H, d]`` over ``k [T, G, d]``, ``v [T, G, dv]``."""
     t, h = q.shape[:2]
     of = torch.arange(h) // (h // k.shape[1])
     out = torch.empty(t, h, v.shape[-1], dtype=q.dtype)
